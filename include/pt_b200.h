@@ -45,6 +45,12 @@ uint64_t pt_launch_count(void);
 #define PT_W_INT4 0 /* signed nibbles, 2 per byte, high nibble = even k, fp16 group scales */
 #define PT_W_FP16 1
 #define PT_W_FP8 2  /* OCP E4M3, per-tensor fp32 scale                                    */
+#define PT_W_BF16 3 /* bfloat16 weights and activations, fp32 accumulation                */
+
+/* Element types of activations, caches and outputs where an entry point takes more than one. */
+#define PT_DT_F16 0
+#define PT_DT_F32 1
+#define PT_DT_BF16 2
 
 /* Prologues fused in front of a linear layer (applied to the activation rows). */
 #define PT_PRO_NONE 0
@@ -60,6 +66,7 @@ uint64_t pt_launch_count(void);
 #define PT_EPI_BIAS 3         /* y = fp16(fp16(acc) + bias)          layers/linear.py:42-46 */
 #define PT_EPI_BIAS_GELU 4    /* y = gelu(fp16(fp16(acc) + bias))    layers/mlp.py:34-41   */
 #define PT_EPI_BIAS_RESIDUAL 5/* y = fp16(res + fp16(fp16(acc) + bias))                  */
+#define PT_EPI_RELU2 6        /* y = max(acc, 0)^2, squared in fp32 (PT_W_BF16 and pt_gemm_f32) */
 
 /* ---- Int4ToHalf -------------------------------------------------------------------
  * Replaces the `Int4ToHalf` custom op (poptransformer/ops/customized.py:115-124;
@@ -110,6 +117,8 @@ typedef struct pt_linear_args {
   size_t workspace_bytes;
   int32_t *error_flag;   /* optional device int, set non-zero if a bounded wait gave up        */
   const void *norm_beta; /* fp16 [k_in]   (PT_PRO_NORMCE)                           */
+  int out_dtype;         /* PT_W_BF16: PT_DT_BF16 or PT_DT_F32 (the other formats write fp16 and ignore it)  */
+  float alpha;           /* PT_W_BF16: factor on the fp32 sum before the epilogue; 0 = 1                     */
 } pt_linear_args;
 
 size_t pt_linear_workspace_bytes(int batch, int n_out, int max_ksplit);
@@ -142,10 +151,12 @@ int pt_linear_static_scratch(const pt_linear_args *args, void *stream);
  *   PT_W_INT4: x = fp16 [m, k_in], w = pt_gemm_repack of the reference's int8 [n_out, k_in/2] rows (w_tiled = 1), scales fp16
  *              [n_out, k_in/group]; every weight becomes fp16(q) * scale with one rounding (Int4ToHalf,
  *              custom_ops/int4_to_half_codelets.cpp:18-38) on its way to the tensor core.
- * k_in must be a multiple of 128.  Accumulation is fp32.  k-slices (ksplit, 0 = chosen by the library) are summed in a fixed
+ *   PT_W_BF16: x = bf16 [m, k_in], w = bf16 [n_out, k_in], row-major or tiled by pt_gemm_repack; out = bf16 or fp32 (out_dtype),
+ *              epilogue PT_EPI_STORE or PT_EPI_RELU2 on alpha * (x . w^T).  k_in a multiple of 64.
+ * FP8 and INT4: k_in must be a multiple of 128.  Accumulation is fp32.  k-slices (ksplit, 0 = chosen by the library) are summed in a fixed
  * order; with more than one slice a workspace is needed (zeroed once by the caller; every launch leaves its counters at zero). */
 typedef struct pt_gemm_args {
-  int wfmt;               /* PT_W_FP8 or PT_W_INT4                                  */
+  int wfmt;               /* PT_W_FP8, PT_W_INT4 or PT_W_BF16                       */
   int m, n_out, k_in;
   int group;              /* INT4: scale group along k (a multiple of 128)          */
   int epilogue;           /* PT_EPI_STORE, PT_EPI_RESIDUAL or PT_EPI_BIAS            */
@@ -161,9 +172,15 @@ typedef struct pt_gemm_args {
   size_t workspace_bytes;
   int32_t *error_flag;    /* optional device int, set non-zero (21..24) if a bounded wait gave up */
   const void *bias;       /* fp16 [n_out] (PT_EPI_BIAS)                              */
+  int out_dtype;          /* PT_W_BF16: PT_DT_BF16 or PT_DT_F32                      */
+  float alpha;            /* PT_W_BF16: factor on the fp32 sum; 0 = 1                */
 } pt_gemm_args;
 size_t pt_gemm_workspace_bytes(int m, int n_out, int max_ksplit);
 int pt_gemm(const pt_gemm_args *args, void *stream);
+/* y[m, n] = epilogue(alpha * sum_k x[m, k] w[n, k]) in true fp32 (fused multiply-adds, no TF32): x, w, y fp32 with row strides in
+ * elements, any sizes.  epilogue: PT_EPI_STORE or PT_EPI_RELU2. */
+int pt_gemm_f32(const float *x, int x_ld, const float *w, int w_ld, int m, int n, int k, float alpha, int epilogue, float *y, int y_ld,
+                void *stream);
 /* One-time tiling of a weight matrix for pt_gemm: [128-row tile][k block] with every tile contiguous.  FP8: E4M3 bytes
  * [n_out, k_in] -> 16 KB tiles in the 128-byte-swizzled image the tensor core reads.  INT4: the reference's int8
  * [n_out, k_in/2] rows (high nibble = even k, two's complement) -> 4 KB tiles of offset-binary nibbles in the word order
@@ -428,6 +445,96 @@ int pt_rms_norm_fp8(const void *x, const void *gamma, int rows, int dim, float e
 int pt_swiglu_fp8(const void *gate_up, int rows, int f, float act_scale, void *out, int out_ld, void *stream);
 /* Elementwise fp16: out = fp16(a + b) (ops.add). */
 int pt_add_f16(const void *a, const void *b, int64_t n, void *out, void *stream);
+
+/* ---- layers with per-sequence positions (hybrid attention / state-space models) --------------------------------------
+ * The rows of these entry points are the new tokens of n_seq sequences, packed one sequence after the other: row cu[s] + i is
+ * position start[s] + i of sequence s, which lives in slot[s] of the caches.  Several tokens per sequence are a prompt (or a
+ * portion of one), exactly one per sequence is a decode step.  All arrays are device int32. */
+typedef struct pt_batch_view {
+  int n_seq, n_tok;
+  const int32_t *cu;      /* [n_seq + 1]                                             */
+  const int32_t *start;   /* [n_seq]                                                 */
+  const int32_t *slot;    /* [n_seq]                                                 */
+  const int32_t *tok_seq; /* [n_tok]: the sequence of every row                      */
+} pt_batch_view;
+
+/* Hyper-connections (csrc/hyper.cu): `streams` fp32 residual streams per token, xs [rows, streams, width].
+ *   table != NULL : every stream <- table[ids[row * ids_ld + *step_dev]] (step_dev NULL: column 0; pos_out[row] <- the step)
+ *   y != NULL     : x_t <- sum_s mix[s, t] x_s + mult * w_out[t] * y     (all streams from the old ones)
+ *   then u = sum_s w_in[s] x_s (w_in NULL: plain sum, the streams are not written back) and, with h, h = rms_norm(u) * norm_w in
+ *   the activation type; columns width .. h_ld - 1 of h are zeroed.  row_index (optional) picks the rows of xs and y. */
+typedef struct pt_hyper_args {
+  int rows, width, streams, dtype;
+  float eps, mult;
+  float *xs;
+  const void *table;
+  int table_ld, vocab;
+  const int32_t *ids;
+  int ids_ld;
+  const int32_t *step_dev;
+  int32_t *pos_out;
+  const int32_t *row_index;
+  const float *y;
+  int y_ld;
+  const float *mix, *w_out, *w_in, *norm_w;
+  void *h;
+  int h_ld;
+  float *sum_out;         /* optional fp32 [rows, width]: sum of the new streams    */
+} pt_hyper_args;
+int pt_hyper(const pt_hyper_args *args, void *stream);
+
+/* Masked attention over a paged cache (csrc/window_attn.cu): sliding window with kept first tokens, softmax sink, grouped heads,
+ * separate key and value widths.  pool[page] = K [n_kv][page_size][dim] then V [n_kv][page_size][vdim], page_table
+ * [slots][max_pages].  k / v (NULL for a layer that reads another layer's cache) are appended before anything is read. */
+typedef struct pt_window_attn_args {
+  pt_batch_view batch;
+  int dtype;              /* PT_DT_F32 or PT_DT_BF16: q, k, v, pool and out          */
+  int n_head, n_kv, dim, vdim, page_size, max_pages;
+  int window;             /* a key is visible less than `window` tokens back; 0 = all */
+  int keep_first;         /* ... or when it is one of the first keep_first tokens    */
+  float scale;
+  const float *sink;      /* fp32 [n_head] or NULL                                   */
+  const void *q;
+  int q_ld;
+  const void *k, *v;
+  int kv_ld;
+  void *pool;
+  const int32_t *page_table;
+  void *out;              /* [n_tok, out_ld], columns n_head * vdim .. out_ld - 1 are zeroed */
+  int out_ld;
+  int max_tokens_per_seq; /* most new tokens of one sequence (0 = n_tok)             */
+  int max_len;            /* no position reaches this (0 = page_size * max_pages)    */
+  int plain;              /* 1: the kernel for any sizes, whatever the shape         */
+  void *workspace;        /* decode: pt_window_attn_workspace_bytes, zeroed once     */
+  size_t workspace_bytes;
+  int32_t *error_flag;    /* optional, set to 12 when a position has no page         */
+} pt_window_attn_args;
+size_t pt_window_attn_workspace_bytes(int n_seq, int n_head, int vdim, int page_size, int max_len, int window, int keep_first);
+int pt_window_attn(const pt_window_attn_args *args, void *stream);
+
+/* State-space (SSD) mixer between its two projections (csrc/ssm.cu): convolution, recurrence, gate and group norm.
+ * zx rows hold [z | x | B | C | dt]; inner = heads * vdim, channels = inner + 2 groups * state_dim. */
+typedef struct pt_ssm_args {
+  pt_batch_view batch;
+  int dtype;              /* PT_DT_F32 or PT_DT_BF16: zx, ring, xbc, out             */
+  int heads, vdim, state_dim, groups, taps, norm_groups;
+  float eps;
+  const void *zx;
+  int zx_ld;
+  const float *conv_w, *conv_b;           /* [channels, taps], [channels]            */
+  const float *dt_bias, *A_log, *D;       /* [heads]                                 */
+  const float *norm_w;                    /* [inner]                                 */
+  void *ring;                             /* [slots, taps, channels]                 */
+  float *state;                           /* [slots, heads, state_dim, vdim]         */
+  void *xbc;                              /* scratch of prompts [n_tok, channels]    */
+  float *dt;                              /* scratch of prompts [n_tok, heads]       */
+  float *y;                               /* scratch [n_tok, inner]                  */
+  void *out;                              /* [n_tok, out_ld], columns inner .. out_ld - 1 are zeroed */
+  int out_ld;
+  int plain;              /* 1: the kernels for any sizes, whatever the shape        */
+  int32_t *error_flag;
+} pt_ssm_args;
+int pt_ssm(const pt_ssm_args *args, void *stream);
 
 #ifdef __cplusplus
 }

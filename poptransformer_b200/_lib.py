@@ -24,6 +24,7 @@ class LinearArgs(ctypes.Structure):
         ("norm_eps", c_float), ("act_scale", c_float), ("w_scale", c_float),
         ("bias", c_void_p), ("residual", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("pdl", c_int),
         ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("error_flag", c_void_p), ("norm_beta", c_void_p),
+        ("out_dtype", c_int), ("alpha", c_float),
     ]
 
 
@@ -44,7 +45,7 @@ class GemmArgs(ctypes.Structure):
         ("wfmt", c_int), ("m", c_int), ("n_out", c_int), ("k_in", c_int), ("group", c_int), ("epilogue", c_int), ("ksplit", c_int),
         ("w_tiled", c_int), ("x", c_void_p), ("w", c_void_p), ("scales", c_void_p), ("x_scale", c_float), ("w_scale", c_float),
         ("residual", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t),
-        ("error_flag", c_void_p), ("bias", c_void_p),
+        ("error_flag", c_void_p), ("bias", c_void_p), ("out_dtype", c_int), ("alpha", c_float),
     ]
 
 
@@ -52,6 +53,31 @@ class PrefillAttnArgs(ctypes.Structure):
     _fields_ = [(n, c_int) for n in ("batch", "n_tokens", "start", "n_head", "head_dim", "page_size", "max_pages", "max_len")] + \
                [("score_scale", c_float), ("qkv", c_void_p), ("rope_sin", c_void_p), ("rope_cos", c_void_p), ("pool", c_void_p),
                 ("page_table", c_void_p), ("out", c_void_p)]
+
+
+class BatchView(ctypes.Structure):
+    _fields_ = [("n_seq", c_int), ("n_tok", c_int)] + [(n, c_void_p) for n in ("cu", "start", "slot", "tok_seq")]
+
+
+class HyperArgs(ctypes.Structure):
+    _fields_ = [("rows", c_int), ("width", c_int), ("streams", c_int), ("dtype", c_int), ("eps", c_float), ("mult", c_float), ("xs", c_void_p),
+                ("table", c_void_p), ("table_ld", c_int), ("vocab", c_int), ("ids", c_void_p), ("ids_ld", c_int), ("step_dev", c_void_p),
+                ("pos_out", c_void_p), ("row_index", c_void_p), ("y", c_void_p), ("y_ld", c_int)] + \
+               [(n, c_void_p) for n in ("mix", "w_out", "w_in", "norm_w", "h")] + [("h_ld", c_int), ("sum_out", c_void_p)]
+
+
+class WindowAttnArgs(ctypes.Structure):
+    _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "n_head", "n_kv", "dim", "vdim", "page_size", "max_pages", "window", "keep_first")] + \
+               [("scale", c_float), ("sink", c_void_p), ("q", c_void_p), ("q_ld", c_int), ("k", c_void_p), ("v", c_void_p), ("kv_ld", c_int),
+                ("pool", c_void_p), ("page_table", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("max_tokens_per_seq", c_int), ("max_len", c_int),
+                ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("error_flag", c_void_p)]
+
+
+class SsmArgs(ctypes.Structure):
+    _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "heads", "vdim", "state_dim", "groups", "taps", "norm_groups")] + \
+               [("eps", c_float), ("zx", c_void_p), ("zx_ld", c_int)] + \
+               [(n, c_void_p) for n in ("conv_w", "conv_b", "dt_bias", "A_log", "D", "norm_w", "ring", "state", "xbc", "dt", "y", "out")] + \
+               [("out_ld", c_int), ("plain", c_int), ("error_flag", c_void_p)]
 
 
 class LlamaLayer(ctypes.Structure):
@@ -83,6 +109,11 @@ SIGNATURES = {
     "pt_gemm": (c_int, [ctypes.POINTER(GemmArgs), c_void_p]),
     "pt_gemm_packed_bytes": (c_size_t, [c_int, c_int, c_int]),
     "pt_gemm_repack": (c_int, [c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]),
+    "pt_gemm_f32": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p]),
+    "pt_hyper": (c_int, [ctypes.POINTER(HyperArgs), c_void_p]),
+    "pt_window_attn_workspace_bytes": (c_size_t, [c_int] * 7),
+    "pt_window_attn": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),
+    "pt_ssm": (c_int, [ctypes.POINTER(SsmArgs), c_void_p]),
     "pt_norm_ce": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p]),
     "pt_rms_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p]),
     "pt_softmax": (c_int, [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),

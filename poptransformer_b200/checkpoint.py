@@ -14,6 +14,8 @@ the result for the kernels.
             (utils/param_handler/precision_strategy.py:24-42); `quantize_linears_int4` produces that format (or the group-128
             extension) from fp16 weights.
 """
+import json
+import os
 import re
 
 import torch
@@ -22,15 +24,47 @@ from .quant import quantize_fp8, quantize_int4
 
 
 def load_state_dict(path):
-    """A checkpoint file as a flat {key: CPU tensor} dict: .safetensors (if the safetensors package is present), torch .bin / .pt / .pth."""
+    """A checkpoint file as a flat {key: CPU tensor} dict: .safetensors, torch .bin / .pt / .pth."""
     if path.endswith(".safetensors"):
-        try:
-            from safetensors.torch import load_file
-        except ImportError as e:
-            raise RuntimeError("reading .safetensors needs the safetensors package") from e
-        return load_file(path)
+        return load_safetensors(path)
     sd = torch.load(path, map_location="cpu", weights_only=True)
     return sd.get("state_dict", sd) if isinstance(sd, dict) else sd
+
+
+_SAFETENSORS_DTYPES = {"F64": torch.float64, "F32": torch.float32, "F16": torch.float16, "BF16": torch.bfloat16, "I64": torch.int64, "I32": torch.int32,
+                       "I16": torch.int16, "I8": torch.int8, "U8": torch.uint8, "BOOL": torch.bool, "F8_E4M3": torch.float8_e4m3fn}
+
+
+def load_safetensors(path):
+    """.safetensors: an 8-byte little-endian header length, a JSON header {name: {dtype, shape, data_offsets}}, the raw data."""
+    with open(path, "rb") as f:
+        header = json.loads(f.read(int.from_bytes(f.read(8), "little")))
+        data = memoryview(f.read())
+    out = {}
+    for name, t in header.items():
+        if name == "__metadata__":
+            continue
+        dt = _SAFETENSORS_DTYPES.get(t["dtype"])
+        if dt is None:
+            raise ValueError(f"{path}: tensor {name} has the unknown type {t['dtype']}")
+        lo, hi = t["data_offsets"]
+        flat = torch.frombuffer(bytearray(data[lo:hi]), dtype=dt) if hi > lo else torch.empty(0, dtype=dt)
+        out[name] = flat.reshape(t["shape"])
+    return out
+
+
+def load_model_dir(path):
+    """A model folder: (parsed config.json, state dict of all its weight files)."""
+    with open(os.path.join(path, "config.json")) as f:
+        config = json.load(f)
+    names = sorted(os.listdir(path))
+    files = [n for n in names if n.endswith(".safetensors")] or [n for n in names if n.endswith((".bin", ".pt", ".pth"))]
+    if not files:
+        raise FileNotFoundError(f"{path}: no .safetensors, .bin, .pt or .pth file")
+    sd = {}
+    for n in files:
+        sd.update(load_state_dict(os.path.join(path, n)))
+    return config, sd
 
 
 def gpt2_from_hf(sd, n_embd, n_head):

@@ -1,5 +1,6 @@
 // Shared host/device helpers for libpt_b200 (sm_100a only).
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_fp8.h>
 #include <cuda_runtime.h>

@@ -3,6 +3,8 @@
 //
 //   * FP8:  W and X are OCP E4M3 bytes with per-tensor scales (the reference's FP8MatMul, custom_ops/matmul_fp8.cpp:885-1091,
 //           in the E4M3 form): tcgen05.mma kind::f8f6f4, fp32 accumulation in tensor memory, scales applied in the epilogue.
+//   * BF16: W and X bfloat16, tcgen05.mma kind::f16, bf16 or fp32 output with a factor and an optional relu^2: the same kernel as FP8
+//           with 64 elements of k per 128-byte operand row.
 //   * INT4: W is packed nibbles with fp16 group scales (utils/param_handler/precision_strategy.py:24-42,56-60).  A transform
 //           warpgroup turns every staged tile into fp16(q) * scale - one fp16 rounding per weight, exactly the reference's
 //           Int4ToHalf (custom_ops/int4_to_half_codelets.cpp:18-38) - in the shared-memory layout the tensor core reads;
@@ -50,7 +52,8 @@ struct GemmParams {
   int kb_per_split, n_kb; // k blocks (of 128 bytes of operand row) per k-slice / in total
   int ksplit, stages, raw_stages;
   int w_tiled;            // weights tiled by pt_gemm_repack (one contiguous tile per stage) instead of row-major
-  int epilogue;           // PT_EPI_STORE, PT_EPI_RESIDUAL or PT_EPI_BIAS
+  int epilogue;           // PT_EPI_STORE, PT_EPI_RESIDUAL or PT_EPI_BIAS (BF16: PT_EPI_STORE or PT_EPI_RELU2)
+  int out_dt;             // BF16: PT_DT_BF16 or PT_DT_F32
   float out_scale;
   const unsigned char *w; // tiled weights (w_tiled)
   const __half *scales;   // INT4: [N][K / group]
@@ -145,14 +148,13 @@ __device__ __forceinline__ uint64_t smem_desc_sw128(uint32_t addr) {
   return d;
 }
 // Instruction descriptor: fp32 accumulator, both operands K-major, M = 128, N = n.
-__host__ __device__ inline uint32_t instr_desc(bool f8, int n) {
+__host__ __device__ inline uint32_t instr_desc(bool bf16, int n) {
   uint32_t d = 0;
   d |= 1u << 4;                 // D format: fp32
-  d |= 0u << 7;                 // A format: E4M3 (f8f6f4) / F16 (f16)
-  d |= 0u << 10;                // B format: the same
+  d |= (bf16 ? 1u : 0u) << 7;   // A format: E4M3 (f8f6f4) / F16 or BF16 (f16)
+  d |= (bf16 ? 1u : 0u) << 10;  // B format: the same
   d |= (uint32_t)(n >> 3) << 17;
   d |= (uint32_t)(BM >> 4) << 24;
-  (void)f8;
   return d;
 }
 
@@ -170,8 +172,24 @@ __device__ __forceinline__ void give_up(SharedCtl &ctl, int *error_flag, int cod
   ctl.abort = 1;
 }
 
+// One finished sum of the FP8 / INT4 kernels (fp16 output) or of the BF16 kernel.
+template <bool BF16> __device__ __forceinline__ void store_out(const GemmParams &p, float acc, int m, int n) {
+  if constexpr (BF16) {
+    float y = acc * p.out_scale;
+    if (p.epilogue == PT_EPI_RELU2) { y = fmaxf(y, 0.f); y *= y; }
+    if (p.out_dt == PT_DT_F32) reinterpret_cast<float *>(p.out)[(size_t)m * p.out_ld + n] = y;
+    else reinterpret_cast<__nv_bfloat16 *>(p.out)[(size_t)m * p.out_ld + n] = __float2bfloat16_rn(y);
+  } else {
+    __half y = __float2half_rn(acc * p.out_scale);
+    if (p.epilogue == PT_EPI_RESIDUAL) y = h_add(__ldcg(p.residual + (size_t)m * p.N + n), y);
+    else if (p.epilogue == PT_EPI_BIAS) y = h_add(y, p.bias[n]);
+    p.out[(size_t)m * p.out_ld + n] = y;
+  }
+}
+
 // Epilogue of the warps that own the tile's rows (tensor-memory lane quarter warp % 4): `part` of `parts` warps share a quarter
 // and take alternate 16-column chunks.
+template <bool BF16>
 __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int q, int lane, int part, int parts, int n0, int m0, int ks) {
   const int n = n0 + q * 32 + lane;
   for (int c0 = part * 16; c0 < p.mb; c0 += 16 * parts) {
@@ -189,10 +207,7 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
         if (p.ksplit > 1) {
           p.partial[((size_t)ks * p.M + m) * p.N + n] = acc;
         } else {
-          __half y = __float2half_rn(acc * p.out_scale);
-          if (p.epilogue == PT_EPI_RESIDUAL) y = h_add(__ldcg(p.residual + (size_t)m * p.N + n), y);
-          else if (p.epilogue == PT_EPI_BIAS) y = h_add(y, p.bias[n]);
-          p.out[(size_t)m * p.out_ld + n] = y;
+          store_out<BF16>(p, acc, m, n);
         }
       }
     }
@@ -200,6 +215,7 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 }
 
 // k-slices of this tile meet: the last CTA to arrive sums them in slice order.
+template <bool BF16>
 __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ctl, int n0, int m0, int threads) {
   const int tid = threadIdx.x;
   __threadfence();
@@ -225,18 +241,17 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc += part[j];
       }
-      __half y = __float2half_rn(acc * p.out_scale);
-      if (p.epilogue == PT_EPI_RESIDUAL) y = h_add(__ldcg(p.residual + (size_t)m * p.N + n), y);
-      else if (p.epilogue == PT_EPI_BIAS) y = h_add(y, p.bias[n]);
-      p.out[(size_t)m * p.out_ld + n] = y;
+      store_out<BF16>(p, acc, m, n);
     }
   }
 }
 
-// ------------------------------------------------------------------------------------------ FP8
+// ------------------------------------------------------------------------------------------ FP8 and BF16
 // Dynamic shared memory: [stage][A tile 16 KB | B tile mb * 128 B], every tile 1024-byte aligned.
-__global__ void __launch_bounds__(THREADS_F8, 1) gemm_fp8_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
-                                                                 const GemmParams p) {
+template <bool BF16>
+__global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
+                                                                   const GemmParams p) {
+  constexpr int KX = BF16 ? BKB / 2 : BKB;   // elements of k per stage
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   __shared__ SharedCtl ctl;
   unsigned char *smem = (unsigned char *)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -272,7 +287,7 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_fp8_kernel(const __grid_co
       const unsigned char *wt = p.w + ((size_t)blockIdx.x * p.n_kb + kb0) * A_TILE;
       const uint32_t tx = A_TILE + b_bytes, full0 = sa(&ctl.full[0]), empty0 = sa(&ctl.empty[0]);
       const bool tiled = p.w_tiled != 0;
-      int s = 0, kx = kb0 * BKB;
+      int s = 0, kx = kb0 * KX;
       uint32_t par = 1;   // parity of the `empty` phase that must have completed before slot s is refilled (none in the first round)
       bool first_round = true;
       for (int it = 0; it < n_it; ++it) {
@@ -284,7 +299,7 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_fp8_kernel(const __grid_co
         else tma_load_2d(st, &map_w, kx, n0, fb);
         tma_load_2d(st + A_TILE, &map_x, kx, m0, fb);
         wt += A_TILE;
-        kx += BKB;
+        kx += KX;
         if (++s == p.stages) { s = 0; par ^= 1u; first_round = false; }
       }
     }
@@ -293,7 +308,7 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_fp8_kernel(const __grid_co
       // One thread issues every MMA of the CTA, so its loop is kept to a few dozen instructions per stage: descriptors are one
       // 64-bit add away from the stage-0 descriptors (the start-address field counts 16-byte units), ring position and parity
       // are counters.  (Measured: with divisions and descriptor rebuilds in this loop a stage took 0.6 us whatever its size.)
-      const uint32_t idesc = instr_desc(true, p.mb);
+      const uint32_t idesc = instr_desc(BF16, p.mb);
       const uint64_t adesc0 = smem_desc_sw128(smem_s), bdesc0 = smem_desc_sw128(smem_s + A_TILE);
       const uint32_t full0 = sa(&ctl.full[0]), empty0 = sa(&ctl.empty[0]), stage16 = stage_bytes >> 4;
       int s = 0;
@@ -303,10 +318,10 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_fp8_kernel(const __grid_co
         if (ctl.abort) break;
         fence_after();
         const uint64_t adesc = adesc0 + (uint64_t)(s * stage16), bdesc = bdesc0 + (uint64_t)(s * stage16);
-        umma<true>(tmem, adesc, bdesc, idesc, acc);   // four MMAs of 32 bytes of k each; inside the swizzle atom the start address moves by 32 bytes
-        umma<true>(tmem, adesc + 2, bdesc + 2, idesc, 1u);
-        umma<true>(tmem, adesc + 4, bdesc + 4, idesc, 1u);
-        umma<true>(tmem, adesc + 6, bdesc + 6, idesc, 1u);
+        umma<!BF16>(tmem, adesc, bdesc, idesc, acc);   // four MMAs of 32 bytes of k each; inside the swizzle atom the start address moves by 32 bytes
+        umma<!BF16>(tmem, adesc + 2, bdesc + 2, idesc, 1u);
+        umma<!BF16>(tmem, adesc + 4, bdesc + 4, idesc, 1u);
+        umma<!BF16>(tmem, adesc + 6, bdesc + 6, idesc, 1u);
         umma_commit(empty0 + s * 8);
         acc = 1u;
         if (++s == p.stages) { s = 0; par ^= 1u; }
@@ -316,10 +331,10 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_fp8_kernel(const __grid_co
   } else {
     if (!mbar_wait(sa(&ctl.accum), 0, &ctl.abort)) give_up(ctl, p.error_flag, 24);
     fence_after();
-    if (!ctl.abort && n_it > 0) epilogue(p, tmem, warp & 3, lane, 0, 1, n0, m0, ks);
+    if (!ctl.abort && n_it > 0) epilogue<BF16>(p, tmem, warp & 3, lane, 0, 1, n0, m0, ks);
     fence_before();
   }
-  if (p.ksplit > 1) reduce_slices(p, ctl, n0, m0, THREADS_F8);
+  if (p.ksplit > 1) reduce_slices<BF16>(p, ctl, n0, m0, THREADS_F8);
   __syncthreads();
   fence_after();
   if (warp == 1) tmem_dealloc(tmem, tmem_cols);
@@ -480,17 +495,17 @@ __global__ void __launch_bounds__(THREADS_I4, 1) gemm_int4_kernel(const __grid_c
     }
     if (!mbar_wait(sa(&ctl.accum), 0, &ctl.abort)) give_up(ctl, p.error_flag, 24);
     fence_after();
-    if (!ctl.abort && n_it > 0) epilogue(p, tmem, q, lane, half, 2, n0, m0, ks);
+    if (!ctl.abort && n_it > 0) epilogue<false>(p, tmem, q, lane, half, 2, n0, m0, ks);
     fence_before();
   }
-  if (p.ksplit > 1) reduce_slices(p, ctl, n0, m0, THREADS_I4);
+  if (p.ksplit > 1) reduce_slices<false>(p, ctl, n0, m0, THREADS_I4);
   __syncthreads();
   fence_after();
   if (warp == 1) tmem_dealloc(tmem, tmem_cols);
 }
 
 // ------------------------------------------------------------------------------------------ load-time tiling
-// FP8 bytes W[n, k] (k contiguous) -> tiles [n tile][k block of 128]: 16 KB each, the image of a 128 x 128-byte tile under the
+// FP8 bytes W[n, k] (k contiguous; BF16: k counts bytes) -> tiles [n tile][k block of 128 bytes]: 16 KB each, the image of a 128 x 128-byte tile under the
 // 128-byte swizzle (row r at (r / 8) * 1024 + (r % 8) * 128, its 16-byte chunk c at position c ^ (r % 8)); rows beyond n are zero.
 __global__ void fp8_tile_kernel(const uint4 *__restrict__ src, uint4 *__restrict__ dst, int n, int k, int n_kb, size_t n_units) {
   for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n_units; i += (size_t)gridDim.x * blockDim.x) {
@@ -564,23 +579,24 @@ using namespace pt;
 
 extern "C" size_t pt_gemm_packed_bytes(int wfmt, int n_out, int k_in) {
   const size_t rows = (size_t)ceil_div(n_out, tc::BM) * tc::BM;
-  return wfmt == PT_W_INT4 ? rows * (size_t)(k_in / 2) : rows * (size_t)k_in;
+  return wfmt == PT_W_INT4 ? rows * (size_t)(k_in / 2) : rows * (size_t)k_in * (wfmt == PT_W_BF16 ? 2 : 1);
 }
 
 extern "C" int pt_gemm_repack(int wfmt, const void *w, int n_out, int k_in, void *packed, void *stream) {
-  PT_REQUIRE(wfmt == PT_W_INT4 || wfmt == PT_W_FP8, "pt_gemm_repack: weight format %d (INT4 or FP8)", wfmt);
+  PT_REQUIRE(wfmt == PT_W_INT4 || wfmt == PT_W_FP8 || wfmt == PT_W_BF16, "pt_gemm_repack: weight format %d (INT4, FP8 or BF16)", wfmt);
   PT_REQUIRE(w && packed && w != packed, "pt_gemm_repack: needs distinct source and destination buffers");
   PT_REQUIRE(((uintptr_t)w & 15) == 0 && ((uintptr_t)packed & 15) == 0, "pt_gemm_repack: buffers must be 16-byte aligned");
-  PT_REQUIRE(n_out > 0 && k_in > 0 && k_in % 128 == 0, "pt_gemm_repack: k_in=%d must be a positive multiple of 128", k_in);
+  const int k_step = wfmt == PT_W_BF16 ? 64 : 128;
+  PT_REQUIRE(n_out > 0 && k_in > 0 && k_in % k_step == 0, "pt_gemm_repack: k_in=%d must be a positive multiple of %d", k_in, k_step);
   const int n_tiles = ceil_div(n_out, tc::BM);
   if (wfmt == PT_W_INT4) {
     const int n_kb = k_in / 64;
     const size_t n_words = (size_t)n_tiles * n_kb * 1024;
     tc::int4_tile_kernel<<<sm_count() * 8, 256, 0, as_stream(stream)>>>((const uint32_t *)w, (uint32_t *)packed, n_out, k_in, n_kb, n_words);
   } else {
-    const int n_kb = k_in / 128;
+    const int k_bytes = wfmt == PT_W_BF16 ? 2 * k_in : k_in, n_kb = k_bytes / 128;
     const size_t n_units = (size_t)n_tiles * n_kb * 1024;
-    tc::fp8_tile_kernel<<<sm_count() * 8, 256, 0, as_stream(stream)>>>((const uint4 *)w, (uint4 *)packed, n_out, k_in, n_kb, n_units);
+    tc::fp8_tile_kernel<<<sm_count() * 8, 256, 0, as_stream(stream)>>>((const uint4 *)w, (uint4 *)packed, n_out, k_bytes, n_kb, n_units);
   }
   PT_LAUNCH_CHECK("pt_gemm_repack");
   return PT_OK;
@@ -599,14 +615,20 @@ extern "C" size_t pt_gemm_workspace_bytes(int m, int n_out, int max_ksplit) {
 
 extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   PT_REQUIRE(a, "pt_gemm: null args");
-  PT_REQUIRE(a->wfmt == PT_W_INT4 || a->wfmt == PT_W_FP8, "pt_gemm: weight format %d (INT4 or FP8)", a->wfmt);
-  const bool int4 = a->wfmt == PT_W_INT4;
-  PT_REQUIRE(a->m >= 1 && a->n_out >= 1 && a->k_in >= 128 && a->k_in % 128 == 0, "pt_gemm: bad shape m=%d n_out=%d k_in=%d (k_in a multiple of 128)",
-             a->m, a->n_out, a->k_in);
+  PT_REQUIRE(a->wfmt == PT_W_INT4 || a->wfmt == PT_W_FP8 || a->wfmt == PT_W_BF16, "pt_gemm: weight format %d (INT4, FP8 or BF16)", a->wfmt);
+  const bool int4 = a->wfmt == PT_W_INT4, bf16 = a->wfmt == PT_W_BF16;
+  const int k_step = bf16 ? 64 : 128;
+  PT_REQUIRE(a->m >= 1 && a->n_out >= 1 && a->k_in >= k_step && a->k_in % k_step == 0, "pt_gemm: bad shape m=%d n_out=%d k_in=%d (k_in a multiple of %d)",
+             a->m, a->n_out, a->k_in, k_step);
   PT_REQUIRE(a->x && a->w && a->out, "pt_gemm: null x / w / out");
   PT_REQUIRE(((uintptr_t)a->x & 15) == 0 && ((uintptr_t)a->w & 15) == 0, "pt_gemm: x and w must be 16-byte aligned");
-  PT_REQUIRE(a->epilogue == PT_EPI_STORE || a->epilogue == PT_EPI_RESIDUAL || a->epilogue == PT_EPI_BIAS, "pt_gemm: epilogue %d (store, residual or bias)",
-             a->epilogue);
+  if (bf16) {
+    PT_REQUIRE(a->epilogue == PT_EPI_STORE || a->epilogue == PT_EPI_RELU2, "pt_gemm: BF16 epilogue %d (store or relu2)", a->epilogue);
+    PT_REQUIRE(a->out_dtype == PT_DT_BF16 || a->out_dtype == PT_DT_F32, "pt_gemm: BF16 weights write bf16 or fp32, got type %d", a->out_dtype);
+  } else {
+    PT_REQUIRE(a->epilogue == PT_EPI_STORE || a->epilogue == PT_EPI_RESIDUAL || a->epilogue == PT_EPI_BIAS, "pt_gemm: epilogue %d (store, residual or bias)",
+               a->epilogue);
+  }
   PT_REQUIRE(a->epilogue != PT_EPI_RESIDUAL || a->residual, "pt_gemm: residual epilogue needs residual");
   PT_REQUIRE(a->epilogue != PT_EPI_BIAS || a->bias, "pt_gemm: bias epilogue needs bias");
   PT_REQUIRE(!int4 || a->w_tiled, "pt_gemm: INT4 weights must be tiled with pt_gemm_repack");
@@ -623,7 +645,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   p.mb = std::min(256, ceil_div(a->m, 16) * 16);
   const int m_tiles = ceil_div(a->m, p.mb);
   const int n_tiles = ceil_div(a->n_out, tc::BM);
-  p.n_kb = int4 ? a->k_in / 64 : a->k_in / 128;
+  p.n_kb = (int4 || bf16) ? a->k_in / 64 : a->k_in / 128;
   // k-slices: fill the GPU when there are few tiles, but keep at least PT_TC_MIN_KB k-blocks per CTA
 #ifndef PT_TC_MIN_KB
 #define PT_TC_MIN_KB 8
@@ -641,6 +663,8 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   p.ksplit = ceil_div(p.n_kb, p.kb_per_split);
   p.epilogue = a->epilogue;
   p.out_scale = int4 ? 1.0f : (a->x_scale > 0.f ? a->x_scale : 1.0f) * (a->w_scale > 0.f ? a->w_scale : 1.0f);
+  if (bf16) p.out_scale = a->alpha != 0.f ? a->alpha : 1.0f;
+  p.out_dt = a->out_dtype;
   p.scales = (const __half *)a->scales;
   p.residual = (const __half *)a->residual;
   p.bias = (const __half *)a->bias;
@@ -682,6 +706,10 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   memset(&map_w, 0, sizeof(map_w));
   if (int4) {
     if (int rc = tc::make_map(&map_x, a->x, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (uint64_t)a->k_in, (uint64_t)a->m, 64, (uint32_t)p.mb, CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
+  } else if (bf16) {
+    if (!p.w_tiled)
+      if (int rc = tc::make_map(&map_w, a->w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->k_in, (uint64_t)a->n_out, 64, tc::BM, CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
+    if (int rc = tc::make_map(&map_x, a->x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->k_in, (uint64_t)a->m, 64, (uint32_t)p.mb, CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
   } else {
     if (!p.w_tiled)
       if (int rc = tc::make_map(&map_w, a->w, CU_TENSOR_MAP_DATA_TYPE_UINT8, 1, (uint64_t)a->k_in, (uint64_t)a->n_out, 128, tc::BM, CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
@@ -689,15 +717,18 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   }
   static bool attr_set = false;
   if (!attr_set) {
-    PT_CUDA(cudaFuncSetAttribute(tc::gemm_fp8_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     PT_CUDA(cudaFuncSetAttribute(tc::gemm_int4_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     attr_set = true;
   }
   dim3 grid(n_tiles, p.ksplit, m_tiles);
   if (int4)
     tc::gemm_int4_kernel<<<grid, tc::THREADS_I4, smem, as_stream(stream)>>>(map_x, p);
+  else if (bf16)
+    tc::gemm_dense_kernel<true><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
   else
-    tc::gemm_fp8_kernel<<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
+    tc::gemm_dense_kernel<false><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
   PT_LAUNCH_CHECK("pt_gemm");
   return PT_OK;
 }

@@ -46,6 +46,7 @@ struct LinearParams {
   float *partial;
   int *counters, *error_flag;
   int B, N, K, n_rt, nchunks, chunks_per_split, ksplit, pro, epi, xs_stride, out_ld, pdl;
+  int out_dt;   // PT_W_BF16: PT_DT_BF16 or PT_DT_F32
   float eps, inv_act_scale, out_scale;
 };
 
@@ -294,6 +295,9 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
           if constexpr (WFMT == PT_W_INT4) {
             mma16816(c[t], fa[0], fb[0], fa[1], fb[1], xv.x, xv.y);
             mma16816(c[t], fa[2], fb[2], fa[3], fb[3], xv.z, xv.w);
+          } else if constexpr (WFMT == PT_W_BF16) {
+            mma16816_bf16(acc[t], fa[0], fb[0], fa[1], fb[1], xv.x, xv.y);
+            mma16816_bf16(acc[t], fa[2], fb[2], fa[3], fb[3], xv.z, xv.w);
           } else {
             mma16816(acc[t], fa[0], fb[0], fa[1], fb[1], xv.x, xv.y);
             mma16816(acc[t], fa[2], fb[2], fa[3], fb[3], xv.z, xv.w);
@@ -373,6 +377,19 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
       const int b = t * 8 + 2 * tig + jb;
       if (b >= p.B) continue;
       const float lo = acc[t][jb] * p.out_scale, hi = acc[t][2 + jb] * p.out_scale;  // rows g and g + 8
+      if constexpr (WFMT == PT_W_BF16) {
+#pragma unroll
+        for (int hr = 0; hr < 2; ++hr) {
+          const int n = rt * 16 + g + 8 * hr;
+          if (n >= p.N) continue;
+          float y = hr ? hi : lo;
+          if (p.epi == PT_EPI_RELU2) { y = fmaxf(y, 0.f); y *= y; }
+          const size_t o = (size_t)b * p.out_ld + n;
+          if (p.out_dt == PT_DT_F32) reinterpret_cast<float *>(p.out)[o] = y;
+          else reinterpret_cast<__nv_bfloat16 *>(p.out)[o] = __float2bfloat16_rn(y);
+        }
+        continue;
+      }
       if (p.epi == PT_EPI_SWIGLU) {
         const int n = rt * 8 + g;  // rows 0..7 of the tile are gate rows, 8..15 the matching up rows
         if (n < p.N / 2) p.out[(size_t)b * p.out_ld + n] = h_mul(__float2half_rn(hi), swish_h(__float2half_rn(lo)));
@@ -542,7 +559,7 @@ SplitPlan plan_split(int wfmt, int batch, int n_out, int k_in, int ksplit_req) {
 
 extern "C" int pt_linear_repack(int wfmt, const void *w, const void *scale, int n_out, int k_in, int group, int interleave_rows,
                                 void *packed_w, void *stream) {
-  PT_REQUIRE(wfmt == PT_W_INT4 || wfmt == PT_W_FP16 || wfmt == PT_W_FP8, "pt_linear_repack: unknown weight format %d", wfmt);
+  PT_REQUIRE(wfmt == PT_W_INT4 || wfmt == PT_W_FP16 || wfmt == PT_W_FP8 || wfmt == PT_W_BF16, "pt_linear_repack: unknown weight format %d", wfmt);
   PT_REQUIRE(n_out > 0 && k_in > 0 && k_in % chunk_k(wfmt) == 0, "pt_linear_repack: k_in=%d must be a positive multiple of %d", k_in,
              chunk_k(wfmt));
   PT_REQUIRE(!interleave_rows || n_out % 16 == 0, "pt_linear_repack: interleaved (gate|up) layout needs n_out %% 16 == 0, got %d", n_out);
@@ -566,20 +583,26 @@ extern "C" int pt_linear_repack(int wfmt, const void *w, const void *scale, int 
 
 extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   PT_REQUIRE(a, "pt_linear: null args");
-  PT_REQUIRE(a->wfmt == PT_W_INT4 || a->wfmt == PT_W_FP16 || a->wfmt == PT_W_FP8, "pt_linear: unknown weight format %d", a->wfmt);
+  PT_REQUIRE(a->wfmt == PT_W_INT4 || a->wfmt == PT_W_FP16 || a->wfmt == PT_W_FP8 || a->wfmt == PT_W_BF16, "pt_linear: unknown weight format %d", a->wfmt);
   PT_REQUIRE(a->batch >= 1 && a->batch <= 32, "pt_linear: batch=%d outside 1..32 (larger batches use the GEMM path)", a->batch);
   const int ck = chunk_k(a->wfmt);
   PT_REQUIRE(a->n_out > 0 && a->k_in > 0 && a->k_in % ck == 0, "pt_linear: k_in=%d must be a positive multiple of %d", a->k_in, ck);
   PT_REQUIRE(a->x && a->packed_w && a->out, "pt_linear: null x / packed_w / out");
   PT_REQUIRE(a->prologue >= PT_PRO_NONE && a->prologue <= PT_PRO_NORMCE, "pt_linear: bad prologue %d", a->prologue);
-  PT_REQUIRE(a->epilogue >= PT_EPI_STORE && a->epilogue <= PT_EPI_BIAS_RESIDUAL, "pt_linear: bad epilogue %d", a->epilogue);
+  if (a->wfmt == PT_W_BF16) {
+    PT_REQUIRE(a->prologue == PT_PRO_NONE && (a->epilogue == PT_EPI_STORE || a->epilogue == PT_EPI_RELU2),
+               "pt_linear: bf16 weights take no prologue and the store or relu2 epilogue, got %d / %d", a->prologue, a->epilogue);
+    PT_REQUIRE(a->out_dtype == PT_DT_BF16 || a->out_dtype == PT_DT_F32, "pt_linear: bf16 weights write bf16 or fp32, got type %d", a->out_dtype);
+  } else {
+    PT_REQUIRE(a->epilogue >= PT_EPI_STORE && a->epilogue <= PT_EPI_BIAS_RESIDUAL, "pt_linear: bad epilogue %d", a->epilogue);
+  }
   const bool norm = a->prologue == PT_PRO_RMSNORM || a->prologue == PT_PRO_RMSNORM_CAST_FP8 || a->prologue == PT_PRO_NORMCE;
   PT_REQUIRE(a->prologue != PT_PRO_NORMCE || a->norm_beta, "pt_linear: NormCE prologue needs norm_beta");
   const bool cast = a->prologue == PT_PRO_CAST_FP8 || a->prologue == PT_PRO_RMSNORM_CAST_FP8;
   PT_REQUIRE(!norm || a->norm_gamma, "pt_linear: RMSNorm prologue needs norm_gamma");
   PT_REQUIRE(!cast || a->act_scale > 0.f, "pt_linear: FP8 activation cast needs act_scale > 0");
   if (a->epilogue == PT_EPI_RESIDUAL || a->epilogue == PT_EPI_BIAS_RESIDUAL) PT_REQUIRE(a->residual, "pt_linear: residual epilogue needs residual");
-  if (a->epilogue >= PT_EPI_BIAS) PT_REQUIRE(a->bias, "pt_linear: bias epilogue needs bias");
+  if (a->epilogue >= PT_EPI_BIAS && a->epilogue <= PT_EPI_BIAS_RESIDUAL) PT_REQUIRE(a->bias, "pt_linear: bias epilogue needs bias");
   if (a->epilogue == PT_EPI_SWIGLU) PT_REQUIRE(a->n_out % 16 == 0, "pt_linear: SwiGLU epilogue needs n_out %% 16 == 0, got %d", a->n_out);
   if (a->wfmt == PT_W_INT4)
     PT_REQUIRE(a->group > 0 && a->group % 128 == 0 && a->k_in % a->group == 0, "pt_linear: INT4 group=%d must be a multiple of 128 dividing k_in=%d",
@@ -603,6 +626,8 @@ extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   p.eps = a->norm_eps;
   p.inv_act_scale = cast ? 1.0f / a->act_scale : 1.0f;
   p.out_scale = 1.0f;
+  p.out_dt = a->out_dtype;
+  if (a->wfmt == PT_W_BF16 && a->alpha != 0.f) p.out_scale = a->alpha;
   if (a->wfmt == PT_W_FP8) p.out_scale = (a->w_scale > 0.f ? a->w_scale : 1.0f) * (cast ? a->act_scale : 1.0f);
 
   const SplitPlan plan = plan_split(a->wfmt, a->batch, a->n_out, a->k_in, a->ksplit);
@@ -624,6 +649,7 @@ extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   switch (a->wfmt) {
     case PT_W_INT4: return dispatch_nb<PT_W_INT4>(p, smem, st);
     case PT_W_FP16: return dispatch_nb<PT_W_FP16>(p, smem, st);
+    case PT_W_BF16: return dispatch_nb<PT_W_BF16>(p, smem, st);
     default: return dispatch_nb<PT_W_FP8>(p, smem, st);
   }
 }

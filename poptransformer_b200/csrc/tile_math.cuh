@@ -7,6 +7,7 @@ namespace pt {
 template <int WFMT> struct WTraits;
 template <> struct WTraits<PT_W_INT4> { static constexpr int kChunkK = 128, kUnits = 4, kTileBytes = 1056; };
 template <> struct WTraits<PT_W_FP8> { static constexpr int kChunkK = 64, kUnits = 2, kTileBytes = 1024; };
+template <> struct WTraits<PT_W_BF16> { static constexpr int kChunkK = 32, kUnits = 1, kTileBytes = 1024; };
 template <> struct WTraits<PT_W_FP16> { static constexpr int kChunkK = 32, kUnits = 1, kTileBytes = 1024; };
 
 static inline int chunk_k(int wfmt) { return wfmt == PT_W_INT4 ? 128 : (wfmt == PT_W_FP8 ? 64 : 32); }
@@ -16,6 +17,11 @@ static inline int row_bytes(int wfmt, int k) { return wfmt == PT_W_INT4 ? k / 2 
 __device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void mma16816_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }

@@ -471,25 +471,6 @@ class LlamaDecoder(DecodeLoop):
             self._norm_linear_raw(self.x, L["ln2"], L["gu"], self.act.data_ptr(), self.act.shape[1])
             ops.linear(self.act, L["down"], self.part, workspace=self.lin_ws)
 
-    def capture(self):
-        """Captures one loop iteration in a CUDA graph (one eager iteration first so lazy initialisation is done)."""
-        saved = (self.ids.clone(), self.step_t.clone())
-        s = torch.cuda.Stream()
-        s.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(s):
-            self.enqueue_step()
-        torch.cuda.current_stream().wait_stream(s)
-        torch.cuda.synchronize()
-        self.ids.copy_(saved[0])
-        self.step_t.copy_(saved[1])
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self.enqueue_step()
-        self.graph = g
-        self.ids.copy_(saved[0])
-        self.step_t.copy_(saved[1])
-        torch.cuda.synchronize()
-
     def reset(self, input_ids):
         """input_ids int32 [batch, max_len] (host or device), right-padded with pad_id; step <- 0."""
         ids = torch.as_tensor(input_ids, dtype=torch.int32)

@@ -29,6 +29,25 @@ class DecodeLoop:
         """The device flag handed to the loop-carry kernel (None when the loop always runs max_loop iterations)."""
         return self.done_flag if self.early_stop else None
 
+    def capture(self):
+        """Captures one loop iteration in a CUDA graph (one eager iteration first so lazy initialisation is done)."""
+        saved = (self.ids.clone(), self.step_t.clone())
+        s = torch.cuda.Stream()
+        s.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(s):
+            self.enqueue_step()
+        torch.cuda.current_stream().wait_stream(s)
+        torch.cuda.synchronize()
+        self.ids.copy_(saved[0])
+        self.step_t.copy_(saved[1])
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            self.enqueue_step()
+        self.graph = g
+        self.ids.copy_(saved[0])
+        self.step_t.copy_(saved[1])
+        torch.cuda.synchronize()
+
     def run(self, input_ids, max_loop=None, poll_every=16, prefill=False):
         """Session.run equivalent (poptransformer/sessions.py:47-49): feeds the id container, runs at most `max_loop` loop
         iterations on the device and returns the reference's anchors {'Loop:0': ids, 'Loop:1': step}.  `prefill=True` (decoders that

@@ -20,11 +20,12 @@ import ctypes
 import torch
 
 from . import _lib
-from ._lib import AttnArgs, GemmArgs, LinearArgs, PtError, check
+from ._lib import AttnArgs, BatchView, GemmArgs, HyperArgs, LinearArgs, PtError, SsmArgs, WindowAttnArgs, check
 
-W_INT4, W_FP16, W_FP8 = 0, 1, 2
+W_INT4, W_FP16, W_FP8, W_BF16 = 0, 1, 2, 3
+DT_F16, DT_F32, DT_BF16 = 0, 1, 2
 PRO_NONE, PRO_RMSNORM, PRO_CAST_FP8, PRO_RMSNORM_CAST_FP8, PRO_NORMCE = 0, 1, 2, 3, 4
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL = 0, 1, 2, 3, 4, 5
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL, EPI_RELU2 = 0, 1, 2, 3, 4, 5, 6
 ROPE_NONE, ROPE_LLAMA, ROPE_CHATGLM2 = 0, 1, 2
 SOFTMAX_F32, SOFTMAX_F16 = 0, 1
 
@@ -41,6 +42,13 @@ def _ptr(t):
     if not t.is_contiguous():
         raise PtError("libpt_b200 ops need contiguous tensors")
     return ctypes.c_void_p(t.data_ptr())
+
+
+def dtype_code(dt):
+    code = {torch.float16: DT_F16, torch.float32: DT_F32, torch.bfloat16: DT_BF16}.get(dt)
+    if code is None:
+        raise PtError(f"unsupported element type {dt}")
+    return code
 
 
 def launch_count():
@@ -64,7 +72,7 @@ class PackedLinear:
     w: [n_out, k] with k contiguous — INT4: int8 [n_out, k/2] in the reference checkpoint format
     (precision_strategy.py:24-42) with fp16 scales [n_out] or [n_out, k/group]; FP16: fp16 [n_out, k]
     (the HF [out, in] layout, i.e. before the reference's load-time transpose, layers/linear.py:32);
-    FP8: uint8 E4M3 [n_out, k] with a per-tensor scale."""
+    FP8: uint8 E4M3 [n_out, k] with a per-tensor scale; BF16: bfloat16 [n_out, k]."""
 
     def __init__(self, wfmt, w, scale=None, group=0, interleave_gate_up=False, w_scale=1.0):
         L = _lib.lib()
@@ -88,7 +96,7 @@ class PackedLinear:
         """Algorithmic bytes one launch streams from HBM: weights plus one fp16 scale per row and group.  (The
         packed tiles repeat a scale for every 128-k chunk of its group, so the buffer itself can be larger.)"""
         sb = self.n_out * (self.k_in // self.group) * 2 if self.wfmt == W_INT4 else 0
-        wb = self.n_out * self.k_in // 2 if self.wfmt == W_INT4 else self.n_out * self.k_in * (2 if self.wfmt == W_FP16 else 1)
+        wb = self.n_out * self.k_in // 2 if self.wfmt == W_INT4 else self.n_out * self.k_in * (1 if self.wfmt == W_FP8 else 2)
         return wb + sb
 
 
@@ -100,7 +108,7 @@ def linear_workspace(batch, n_out_max, max_ksplit=16, device="cuda"):
 
 
 def linear_args(x, pl, out, prologue=PRO_NONE, epilogue=EPI_STORE, gamma=None, eps=0.0, act_scale=0.0, bias=None,
-                residual=None, workspace=None, ksplit=0, out_ld=0, pdl=0, error_flag=None, beta=None):
+                residual=None, workspace=None, ksplit=0, out_ld=0, pdl=0, error_flag=None, beta=None, alpha=1.0):
     a = LinearArgs()
     a.wfmt, a.batch, a.n_out, a.k_in, a.group = pl.wfmt, x.shape[0], pl.n_out, pl.k_in, pl.group
     a.prologue, a.epilogue, a.ksplit = prologue, epilogue, ksplit
@@ -108,6 +116,7 @@ def linear_args(x, pl, out, prologue=PRO_NONE, epilogue=EPI_STORE, gamma=None, e
     a.norm_gamma, a.norm_eps, a.act_scale, a.w_scale = _ptr(gamma), eps, act_scale, pl.w_scale
     a.bias, a.residual, a.out, a.out_ld, a.pdl = _ptr(bias), _ptr(residual), _ptr(out), out_ld, pdl
     a.error_flag, a.norm_beta = _ptr(error_flag), _ptr(beta)
+    a.out_dtype, a.alpha = dtype_code(out.dtype), float(alpha)
     a.workspace = _ptr(workspace)
     a.workspace_bytes = workspace.numel() if workspace is not None else 0
     return a
@@ -128,26 +137,33 @@ def linear(x, pl, out=None, **kw):
 # ------------------------------------------------------------------------------------------ tensor-core GEMMs (16+ rows)
 class GemmWeight:
     """A weight matrix tiled once for pt_gemm (pt_gemm_repack): FP8 bytes [n_out, k], or INT4 rows in the reference's int8
-    [n_out, k/2] format plus fp16 scales [n_out, k/group]."""
+    [n_out, k/2] format plus fp16 scales [n_out, k/group], or bfloat16 [n_out, k].  tiled=False (BF16) keeps the row-major
+    matrix, which the kernel then fetches with strided TMA boxes: for a matrix that exists in that form anyway."""
 
-    def __init__(self, wfmt, w, scale=None, group=0, w_scale=1.0):
+    def __init__(self, wfmt, w, scale=None, group=0, w_scale=1.0, tiled=True):
         L = _lib.lib()
+        self.tiled = bool(tiled)
         self.wfmt, self.n_out, self.w_scale = wfmt, w.shape[0], float(w_scale)
         if wfmt == W_INT4:
             self.k_in = w.shape[1] * 2
             self.group = int(group) if group else self.k_in
             self.scales = scale.reshape(self.n_out, self.k_in // self.group).to(torch.float16).contiguous()
-        elif wfmt == W_FP8:
+        elif wfmt in (W_FP8, W_BF16):
             self.k_in, self.group, self.scales = w.shape[1], 0, None
         else:
-            raise PtError("GemmWeight: INT4 or FP8")
+            raise PtError("GemmWeight: INT4, FP8 or BF16")
+        if not self.tiled:
+            if wfmt != W_BF16:
+                raise PtError("GemmWeight: only BF16 weights can stay row-major")
+            self.w = w.contiguous()
+            return
         self.w = torch.empty(L.pt_gemm_packed_bytes(wfmt, self.n_out, self.k_in), dtype=torch.uint8, device=w.device)
         check(L.pt_gemm_repack(wfmt, _ptr(w.contiguous()), self.n_out, self.k_in, _ptr(self.w), _stream()), "pt_gemm_repack")
 
     @property
     def nbytes(self):
         """Algorithmic bytes one launch streams from HBM."""
-        wb = self.n_out * self.k_in // 2 if self.wfmt == W_INT4 else self.n_out * self.k_in
+        wb = self.n_out * self.k_in // 2 if self.wfmt == W_INT4 else self.n_out * self.k_in * (2 if self.wfmt == W_BF16 else 1)
         return wb + (self.scales.numel() * 2 if self.scales is not None else 0)
 
 
@@ -155,8 +171,10 @@ def gemm_workspace(m, n_out_max, max_ksplit=8, device="cuda"):
     return torch.zeros(_lib.lib().pt_gemm_workspace_bytes(m, n_out_max, max_ksplit), dtype=torch.uint8, device=device)
 
 
-def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, workspace=None, ksplit=0, error_flag=None, bias=None):
-    """y = x @ W^T on the tcgen05 GEMM.  INT4: x fp16 [m, k]; FP8: x E4M3 bytes [m, k] quantised with `x_scale`."""
+def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, workspace=None, ksplit=0, error_flag=None, bias=None,
+         out_ld=0, alpha=1.0):
+    """y = x @ W^T on the tcgen05 GEMM.  INT4: x fp16 [m, k]; FP8: x E4M3 bytes [m, k] quantised with `x_scale`; BF16: x bfloat16,
+    `out` bfloat16 or float32."""
     m = x.shape[0]
     if x.shape[1] != gw.k_in:
         raise PtError(f"gemm: x has k={x.shape[1]}, weight has k={gw.k_in}")
@@ -164,14 +182,128 @@ def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, worksp
         out = torch.empty((m, gw.n_out), dtype=torch.float16, device=x.device)
     a = GemmArgs()
     a.wfmt, a.m, a.n_out, a.k_in, a.group, a.epilogue, a.ksplit = gw.wfmt, m, gw.n_out, gw.k_in, gw.group, epilogue, ksplit
-    a.w_tiled = 1
+    a.w_tiled = 1 if gw.tiled else 0
     a.x, a.w, a.scales = _ptr(x), _ptr(gw.w), _ptr(gw.scales)
     a.x_scale, a.w_scale = float(x_scale), gw.w_scale
-    a.residual, a.out, a.out_ld = _ptr(residual), _ptr(out), 0
+    a.residual, a.out, a.out_ld = _ptr(residual), _ptr(out), out_ld
+    a.out_dtype, a.alpha = dtype_code(out.dtype), float(alpha)
     a.workspace, a.workspace_bytes = _ptr(workspace), (workspace.numel() if workspace is not None else 0)
     a.error_flag, a.bias = _ptr(error_flag), _ptr(bias)
     check(_lib.lib().pt_gemm(ctypes.byref(a), _stream()), "pt_gemm")
     return out
+
+
+# ------------------------------------------------------------------------------------------ linears of bf16 / fp32 models
+def pad_to(n, m):
+    return (n + m - 1) // m * m
+
+
+class DenseLinear:
+    """W [n_out, k] of a model whose activations are bfloat16 or float32.  bfloat16: the skinny-matmul kernel up to 32 rows and the
+    tcgen05 GEMM beyond (one tiling of the weights each), k padded to `K_PAD` with zero columns, so inputs have `ld` columns.
+    float32: true 32-bit products, no padding.  Outputs may have more columns than n_out (`out_ld`)."""
+    K_PAD = 64
+    SKINNY_ROWS = 32
+
+    def __init__(self, w, dtype, pad_rows=0, row_major=False):
+        """pad_rows: zero rows are appended up to this many outputs (an output that is the padded input of the next linear).
+        row_major: the GEMM reads the matrix as it is instead of a tiled copy (a table that also serves look-ups)."""
+        self.dtype, self.n_out, self.k_in = dtype, w.shape[0], w.shape[1]
+        self.ld = pad_to(self.k_in, self.K_PAD) if dtype == torch.bfloat16 else self.k_in
+        if self.ld != self.k_in or pad_rows > self.n_out:
+            full = torch.zeros((max(pad_rows, self.n_out), self.ld), dtype=w.dtype, device=w.device)
+            full[:self.n_out, :self.k_in] = w
+            w, self.n_out = full, full.shape[0]
+        w = w.to(dtype).contiguous()
+        if dtype == torch.bfloat16:
+            self.skinny, self.gemm = PackedLinear(W_BF16, w), GemmWeight(W_BF16, w, tiled=not row_major)
+            self.w = w if row_major else None
+        elif dtype == torch.float32:
+            self.w = w
+        else:
+            raise PtError(f"DenseLinear: bfloat16 or float32, got {dtype}")
+
+    @property
+    def nbytes(self):
+        """Algorithmic bytes of one launch: the weights once."""
+        return self.n_out * self.k_in * (2 if self.dtype == torch.bfloat16 else 4)
+
+    def __call__(self, x, out, rows, out_ld, epilogue=EPI_STORE, alpha=1.0, linear_ws=None, gemm_ws=None, error_flag=None):
+        """out[:rows, :n_out] = epilogue(alpha * x[:rows] @ W^T); x and out are flat or 2-D buffers of row strides `ld` and `out_ld`."""
+        x = x.reshape(-1)[:rows * self.ld].view(rows, self.ld)
+        L = _lib.lib()
+        if self.dtype == torch.float32:
+            check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, float(alpha), epilogue, _ptr(out), out_ld, _stream()),
+                  "pt_gemm_f32")
+        elif rows <= self.SKINNY_ROWS:
+            a = linear_args(x, self.skinny, out, epilogue=epilogue, workspace=linear_ws, out_ld=out_ld, error_flag=error_flag, alpha=alpha)
+            check(L.pt_linear(ctypes.byref(a), _stream()), "pt_linear")
+        else:
+            gemm(x, self.gemm, out=out, epilogue=epilogue, workspace=gemm_ws, error_flag=error_flag, out_ld=out_ld, alpha=alpha)
+
+
+# ------------------------------------------------------------------------------------------ layers with per-sequence positions
+def batch_view(n_seq, n_tok, cu, start, slot, tok_seq):
+    """The packed tokens of one launch (pt_batch_view): device int32 tensors."""
+    v = BatchView()
+    v.n_seq, v.n_tok = n_seq, n_tok
+    v.cu, v.start, v.slot, v.tok_seq = _ptr(cu), _ptr(start), _ptr(slot), _ptr(tok_seq)
+    v.keep = (cu, start, slot, tok_seq)
+    return v
+
+
+def hyper(xs, rows, eps, norm_w=None, h=None, h_ld=0, w_in=None, y=None, y_ld=0, mix=None, w_out=None, mult=1.0, table=None, ids=None, ids_ld=1,
+          step=None, pos_out=None, row_index=None, sum_out=None, vocab=0):
+    """Hyper-connection step on the fp32 streams xs [rows, streams, width] (see pt_hyper): write the finished sublayer's y, read and
+    normalise the next one's input into h.  `table` starts tokens from an embedding table instead."""
+    a = HyperArgs()
+    a.rows, a.width, a.streams = rows, xs.shape[2], xs.shape[1]
+    a.dtype = dtype_code(h.dtype if h is not None else (table.dtype if table is not None else torch.float32))
+    a.eps, a.mult, a.xs = float(eps), float(mult), _ptr(xs)
+    if table is not None:
+        a.table, a.table_ld, a.vocab = _ptr(table), table.shape[1], vocab or table.shape[0]
+        a.ids, a.ids_ld, a.step_dev, a.pos_out = _ptr(ids), ids_ld, _ptr(step), _ptr(pos_out)
+    a.row_index, a.y, a.y_ld, a.mix, a.w_out, a.w_in = _ptr(row_index), _ptr(y), y_ld, _ptr(mix), _ptr(w_out), _ptr(w_in)
+    a.norm_w, a.h, a.h_ld, a.sum_out = _ptr(norm_w), _ptr(h), h_ld, _ptr(sum_out)
+    check(_lib.lib().pt_hyper(ctypes.byref(a), _stream()), "pt_hyper")
+
+
+def window_attn_workspace(n_seq, n_head, vdim, page_size, max_len, window, keep_first, device="cuda"):
+    n = _lib.lib().pt_window_attn_workspace_bytes(n_seq, n_head, vdim, page_size, max_len, window, keep_first)
+    return torch.zeros(n, dtype=torch.uint8, device=device)
+
+
+def window_attn(view, qkv, qkv_ld, cache, out, out_ld, n_head, scale, window=0, keep_first=0, sink=None, append=True, max_tokens_per_seq=0,
+                workspace=None, error_flag=None, plain=False):
+    """Masked attention of the packed tokens of `view` over a paged cache (see pt_window_attn).  qkv rows hold [q | k | v]
+    (append=True: k and v go to the cache first) or only q (a layer that reads another layer's cache)."""
+    a = WindowAttnArgs()
+    a.batch, a.dtype = view, dtype_code(qkv.dtype)
+    a.n_head, a.n_kv, a.dim, a.vdim = n_head, cache.n_kv, cache.head_dim, cache.v_dim
+    a.page_size, a.max_pages, a.max_len = cache.page_size, cache.page_table.shape[1], cache.max_len
+    a.window, a.keep_first, a.scale, a.sink = window, keep_first, float(scale), _ptr(sink)
+    a.q, a.q_ld, a.kv_ld = _ptr(qkv), qkv_ld, qkv_ld
+    if append:
+        k = qkv.data_ptr() + n_head * cache.head_dim * qkv.element_size()
+        a.k, a.v = k, k + cache.n_kv * cache.head_dim * qkv.element_size()
+    a.pool, a.page_table, a.out, a.out_ld = _ptr(cache.pool), _ptr(cache.page_table), _ptr(out), out_ld
+    a.max_tokens_per_seq, a.plain = max_tokens_per_seq, 1 if plain else 0
+    a.workspace, a.workspace_bytes = _ptr(workspace), workspace.numel() if workspace is not None else 0
+    a.error_flag = _ptr(error_flag)
+    check(_lib.lib().pt_window_attn(ctypes.byref(a), _stream()), "pt_window_attn")
+
+
+def ssm(view, zx, zx_ld, out, out_ld, w, ring, state, y, xbc=None, dt=None, error_flag=None, plain=False):
+    """State-space mixer between its projections (see pt_ssm).  w: an object with heads, vdim, state, groups, taps, norm_groups, eps
+    and the fp32 tensors conv_w, conv_b, dt_bias, A_log, D, norm_w."""
+    a = SsmArgs()
+    a.batch, a.dtype = view, dtype_code(zx.dtype)
+    a.heads, a.vdim, a.state_dim, a.groups, a.taps, a.norm_groups, a.eps = w.heads, w.vdim, w.state, w.groups, w.taps, w.norm_groups, float(w.eps)
+    a.zx, a.zx_ld, a.out, a.out_ld = _ptr(zx), zx_ld, _ptr(out), out_ld
+    a.conv_w, a.conv_b, a.dt_bias, a.A_log, a.D, a.norm_w = (_ptr(t) for t in (w.conv_w, w.conv_b, w.dt_bias, w.A_log, w.D, w.norm_w))
+    a.ring, a.state, a.xbc, a.dt, a.y = _ptr(ring), _ptr(state), _ptr(xbc), _ptr(dt), _ptr(y)
+    a.plain, a.error_flag = 1 if plain else 0, _ptr(error_flag)
+    check(_lib.lib().pt_ssm(ctypes.byref(a), _stream()), "pt_ssm")
 
 
 # ------------------------------------------------------------------------------------------ norms / softmax
@@ -297,14 +429,19 @@ def kv_cache_pipeline(state, step, updater):
 
 # ------------------------------------------------------------------------------------------ paged cache + attention
 class PagedKVCache:
-    """Page pool of one layer plus the (shared) page table.  pool[page][2][n_kv][page_size][head_dim]."""
+    """Page pool of one layer plus the (shared) page table.  pool[page][2][n_kv][page_size][head_dim]; with a value width of its own
+    (v_dim) a page is K [n_kv][page_size][head_dim] followed by V [n_kv][page_size][v_dim].  n_pages: size of the pool where pages
+    are handed out on demand (cache.SequenceSlots) instead of max_len tokens per row."""
 
-    def __init__(self, rows, n_kv, head_dim, max_len, page_size=64, device="cuda", page_table=None, extra_pages=0):
+    def __init__(self, rows, n_kv, head_dim, max_len, page_size=64, device="cuda", page_table=None, extra_pages=0, v_dim=None, dtype=torch.float16,
+                 n_pages=None):
         self.rows, self.n_kv, self.head_dim, self.page_size = rows, n_kv, head_dim, page_size
+        self.v_dim = head_dim if v_dim is None else v_dim
         self.max_len = max_len
         self.max_pages = (max_len + page_size - 1) // page_size
-        n_pages = rows * self.max_pages + extra_pages
-        self.pool = torch.zeros((n_pages, 2, n_kv, page_size, head_dim), dtype=torch.float16, device=device)
+        n_pages = (rows * self.max_pages if n_pages is None else n_pages) + extra_pages
+        shape = (n_pages, 2, n_kv, page_size, head_dim) if self.v_dim == head_dim else (n_pages, n_kv * page_size * (head_dim + self.v_dim))
+        self.pool = torch.zeros(shape, dtype=dtype, device=device)
         if page_table is None:
             page_table = torch.arange(rows * self.max_pages, dtype=torch.int32, device=device).reshape(rows, self.max_pages)
         self.page_table = page_table
