@@ -11,6 +11,7 @@
 //
 //   ssm_conv_kernel    prompts: convolution + silu of all tokens, step sizes
 //   ssm_scan_kernel    prompts, any sizes and types: the recurrence token by token, state in shared memory
+//   ssm_chunk_kernel   bf16 prompts: the same recurrence 64 tokens at a time on the tensor cores
 //   ssm_step_kernel    one token per sequence: convolution, step size, state update and readout in one launch
 //   ssm_norm_kernel    gate, group norm, and the ring update
 #include "elem.cuh"
@@ -94,6 +95,238 @@ template <typename T> __global__ void __launch_bounds__(SCAN_WARPS * 32) ssm_sca
   }
   for (int n = warp; n < p.N; n += SCAN_WARPS)
     if (in) gS[(size_t)n * p.P + col] = S[n * SCAN_P + lane];
+}
+
+// ------------------------------------------------------------------------------------------ recurrence in chunks of 64 tokens
+// With c_t = sum_{r <= t} log decay_r inside a chunk and S the state before it, the recurrence is four matrix products:
+//     y_t = exp(c_t) C_t S  +  sum_{s <= t} (C_t . B_s) exp(c_t - c_s) dt_s x_s  +  D x_t
+//     S  <- exp(c_last) S  +  sum_s B_s (exp(c_last - c_s) dt_s x_s)^T
+// Block: 32 columns of one head's state, one sequence; it walks the chunks in order with the state in fp32 accumulators.  Operands
+// that are not already bf16 (the state, the decayed products, the weighted x) enter the tensor cores as hi + lo pairs.  c is kept
+// as a pair of floats, so differences of neighbours stay exact however far the sum has run.
+// NP: state size rounded up to 64, 128 or 256 (padding is zero).
+constexpr int CHUNK = 64, CP = 32, CHUNK_THREADS = 128;
+__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
+}
+__device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+template <int NP> struct ChunkSmem {
+  static constexpr int BLD = NP + 8, XLD = CP + 8;
+  __nv_bfloat16 B[2][CHUNK][BLD], C[2][CHUNK][BLD], X[2][CHUNK][XLD];
+  __nv_bfloat16 Sh[NP][XLD], Sl[NP][XLD];      // state before the chunk, hi and lo
+  __nv_bfloat16 Wh[CHUNK][XLD], Wl[CHUNK][XLD];   // exp(c_last - c_s) dt_s x_s
+  float c_hi[CHUNK], c_lo[CHUNK], dt[CHUNK];
+};
+
+template <int NP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_chunk_kernel(const Params p) {
+  typedef __nv_bfloat16 T;
+  constexpr int MT = NP / 64;                       // 16-row tiles of the state per warp
+  extern __shared__ __align__(16) unsigned char smraw[];
+  ChunkSmem<NP> &sm = *reinterpret_cast<ChunkSmem<NP> *>(smraw);
+  const int s = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * CP;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
+  const int grp = h / (p.heads / p.groups);
+  const int row0 = p.cu[s], len = p.cu[s + 1] - row0;
+  const T *xbc = reinterpret_cast<const T *>(p.xbc) + (size_t)row0 * p.C;
+  const float a = -expf(p.A_log[h]), D = p.D[h];
+  float *gS = p.state + ((size_t)p.slot[s] * p.heads + h) * p.N * p.P;
+
+  auto load_chunk = [&](int t0, int stage) {
+    for (int e = tid; e < CHUNK * (NP / 8); e += CHUNK_THREADS) {
+      const int r = e / (NP / 8), c = (e % (NP / 8)) * 8;
+      const bool in = t0 + r < len && c < p.N;
+      const T *row = xbc + (in ? (size_t)(t0 + r) * p.C + p.inner + grp * p.N + c : 0);
+      cp16(&sm.B[stage][r][c], row, in);
+      cp16(&sm.C[stage][r][c], row + (in ? p.groups * p.N : 0), in);
+    }
+    for (int e = tid; e < CHUNK * (CP / 8); e += CHUNK_THREADS) {
+      const int r = e / (CP / 8), c = (e % (CP / 8)) * 8;
+      const bool in = t0 + r < len && col0 + c < p.P;
+      cp16(&sm.X[stage][r][c], xbc + (in ? (size_t)(t0 + r) * p.C + (size_t)h * p.P + col0 + c : 0), in);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load_chunk(0, 0);
+
+  // state accumulators: warp w owns rows w NP / 4 ..; tile i, column tile j, lane (g, tig): rows g and g + 8, columns 2 tig, + 1
+  float S[MT][CP / 8][4];
+  const int srow = warp * (NP / 4) + g;
+  const bool fresh = p.start[s] == 0;
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + j * 8 + 2 * tig + (e & 1);
+        S[i][j][e] = (!fresh && n < p.N && c < p.P) ? gS[(size_t)n * p.P + c] : 0.f;
+      }
+  auto publish_state = [&]() {
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          uint32_t hi, lo;
+          split_bf2(S[i][j][2 * r], S[i][j][2 * r + 1], hi, lo);
+          *reinterpret_cast<uint32_t *>(&sm.Sh[srow + i * 16 + 8 * r][j * 8 + 2 * tig]) = hi;
+          *reinterpret_cast<uint32_t *>(&sm.Sl[srow + i * 16 + 8 * r][j * 8 + 2 * tig]) = lo;
+        }
+  };
+  publish_state();
+
+  int stage = 0;
+  for (int t0 = 0; t0 < len; t0 += CHUNK, stage ^= 1) {
+    if (t0 + CHUNK < len) {
+      load_chunk(t0 + CHUNK, stage ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    if (warp == 0) {   // step sizes and running log decays of the chunk (zero beyond the sequence: decay 1, no contribution)
+      const int r0 = t0 + 2 * lane, r1 = r0 + 1;
+      const float d0 = r0 < len ? p.dt[(size_t)(row0 + r0) * p.heads + h] : 0.f, d1 = r1 < len ? p.dt[(size_t)(row0 + r1) * p.heads + h] : 0.f;
+      const double l0 = (double)(a * d0), l1 = (double)(a * d1);
+      double sum = l0 + l1;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const double v = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += v;
+      }
+      const double c1 = sum, c0 = sum - l1;
+      sm.dt[2 * lane] = d0; sm.dt[2 * lane + 1] = d1;
+      sm.c_hi[2 * lane] = (float)c0; sm.c_lo[2 * lane] = (float)(c0 - (double)(float)c0);
+      sm.c_hi[2 * lane + 1] = (float)c1; sm.c_lo[2 * lane + 1] = (float)(c1 - (double)(float)c1);
+    }
+    __syncthreads();   // operands, step sizes and the published state are in shared memory
+    const float ce_hi = sm.c_hi[CHUNK - 1], ce_lo = sm.c_lo[CHUNK - 1];
+    for (int e = tid; e < CHUNK * (CP / 2); e += CHUNK_THREADS) {   // weighted x for the state update
+      const int r = e / (CP / 2), c = (e % (CP / 2)) * 2;
+      const float w = expf((ce_hi - sm.c_hi[r]) + (ce_lo - sm.c_lo[r])) * sm.dt[r];
+      const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[stage][r][c]);
+      uint32_t hi, lo;
+      split_bf2(w * __low2float(x2), w * __high2float(x2), hi, lo);
+      *reinterpret_cast<uint32_t *>(&sm.Wh[r][c]) = hi;
+      *reinterpret_cast<uint32_t *>(&sm.Wl[r][c]) = lo;
+    }
+    // ---- rows 16 warp .. + 15 of the chunk's output
+    const int tr = warp * 16 + g;
+    float y[CP / 8][4], G[CHUNK / 8][4];
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+#pragma unroll
+    for (int j = 0; j < CHUNK / 8; ++j) G[j][0] = G[j][1] = G[j][2] = G[j][3] = 0.f;
+    const uint32_t sh_lane = smem_addr(&sm.Sh[lane & 15][(lane >> 4) * 8]), sl_lane = smem_addr(&sm.Sl[lane & 15][(lane >> 4) * 8]);
+#pragma unroll 2
+    for (int kk = 0; kk < NP / 16; ++kk) {
+      const T *c0 = &sm.C[stage][tr][kk * 16 + 2 * tig], *c1 = &sm.C[stage][tr + 8][kk * 16 + 2 * tig];
+      const uint32_t a0 = *reinterpret_cast<const uint32_t *>(c0), a1 = *reinterpret_cast<const uint32_t *>(c1);
+      const uint32_t a2 = *reinterpret_cast<const uint32_t *>(c0 + 8), a3 = *reinterpret_cast<const uint32_t *>(c1 + 8);
+#pragma unroll
+      for (int j = 0; j < CHUNK / 8; ++j) {
+        if (j > 2 * warp + 1) break;      // columns behind the diagonal only
+        const T *b = &sm.B[stage][j * 8 + g][kk * 16 + 2 * tig];
+        mma16816_bf16(G[j], a0, a1, a2, a3, *reinterpret_cast<const uint32_t *>(b), *reinterpret_cast<const uint32_t *>(b + 8));
+      }
+#pragma unroll
+      for (int j = 0; j < CP / 8; j += 2) {
+        uint32_t b0, b1, b2, b3;
+        ldsm4t(sh_lane + (uint32_t)(kk * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, b0, b1, b2, b3);
+        mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
+        mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
+        ldsm4t(sl_lane + (uint32_t)(kk * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, b0, b1, b2, b3);
+        mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
+        mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
+      }
+    }
+    const float h0 = sm.c_hi[tr], l0 = sm.c_lo[tr], h1 = sm.c_hi[tr + 8], l1 = sm.c_lo[tr + 8];
+    const float e0 = expf(h0 + l0), e1 = expf(h1 + l1);
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
+#pragma unroll
+    for (int j = 0; j < CHUNK / 8; ++j) {
+      if (j > 2 * warp + 1) break;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int sc = j * 8 + 2 * tig + (e & 1), t = e < 2 ? tr : tr + 8;
+        const float d = e < 2 ? (h0 - sm.c_hi[sc]) + (l0 - sm.c_lo[sc]) : (h1 - sm.c_hi[sc]) + (l1 - sm.c_lo[sc]);
+        G[j][e] = sc <= t ? G[j][e] * expf(d) * sm.dt[sc] : 0.f;
+      }
+    }
+    const uint32_t x_lane = smem_addr(&sm.X[stage][lane & 15][(lane >> 4) * 8]);
+#pragma unroll
+    for (int k2 = 0; k2 < CHUNK / 16; ++k2) {
+      if (k2 > warp) break;
+      uint32_t hi[4], lo[4];
+      split_bf2(G[2 * k2][0], G[2 * k2][1], hi[0], lo[0]);
+      split_bf2(G[2 * k2][2], G[2 * k2][3], hi[1], lo[1]);
+      split_bf2(G[2 * k2 + 1][0], G[2 * k2 + 1][1], hi[2], lo[2]);
+      split_bf2(G[2 * k2 + 1][2], G[2 * k2 + 1][3], hi[3], lo[3]);
+#pragma unroll
+      for (int j = 0; j < CP / 8; j += 2) {
+        uint32_t b0, b1, b2, b3;
+        ldsm4t(x_lane + (uint32_t)(k2 * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, b0, b1, b2, b3);
+        mma16816_bf16(y[j], hi[0], hi[1], hi[2], hi[3], b0, b1);
+        mma16816_bf16(y[j + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
+        mma16816_bf16(y[j], lo[0], lo[1], lo[2], lo[3], b0, b1);
+        mma16816_bf16(y[j + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int t = tr + 8 * r, c = j * 8 + 2 * tig;
+        if (t0 + t >= len || col0 + c >= p.P) continue;
+        const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[stage][t][c]);
+        *reinterpret_cast<float2 *>(p.y + (size_t)(row0 + t0 + t) * p.inner + (size_t)h * p.P + col0 + c) =
+            make_float2(fmaf(D, __low2float(x2), y[j][2 * r]), fmaf(D, __high2float(x2), y[j][2 * r + 1]));
+      }
+    __syncthreads();   // the weighted x is complete; nobody reads the old state any more
+    // ---- state update: B^T [state rows x tokens] times the weighted x
+    const float keep = expf(ce_hi + ce_lo);
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[i][j][e] *= keep;
+    const uint32_t wh_lane = smem_addr(&sm.Wh[lane & 15][(lane >> 4) * 8]), wl_lane = smem_addr(&sm.Wl[lane & 15][(lane >> 4) * 8]);
+#pragma unroll
+    for (int k2 = 0; k2 < CHUNK / 16; ++k2) {
+      uint32_t wh[CP / 8][2], wl[CP / 8][2];
+#pragma unroll
+      for (int j = 0; j < CP / 8; j += 2) {
+        ldsm4t(wh_lane + (uint32_t)(k2 * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, wh[j][0], wh[j][1], wh[j + 1][0], wh[j + 1][1]);
+        ldsm4t(wl_lane + (uint32_t)(k2 * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, wl[j][0], wl[j][1], wl[j + 1][0], wl[j + 1][1]);
+      }
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        // A fragment (rows = state, k = tokens) from the token-major tile: matrices (tokens 0-7 | 8-15) x (state 0-7 | 8-15), transposed
+        uint32_t a0, a1, a2, a3;
+        ldsm4t(smem_addr(&sm.B[stage][k2 * 16 + (lane & 7) + (lane >> 4) * 8][warp * (NP / 4) + i * 16 + ((lane >> 3) & 1) * 8]), a0, a1, a2, a3);
+#pragma unroll
+        for (int j = 0; j < CP / 8; ++j) {
+          mma16816_bf16(S[i][j], a0, a1, a2, a3, wh[j][0], wh[j][1]);
+          mma16816_bf16(S[i][j], a0, a1, a2, a3, wl[j][0], wl[j][1]);
+        }
+      }
+    }
+    publish_state();
+    __syncthreads();   // this stage of the operands may be refilled
+  }
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + j * 8 + 2 * tig + (e & 1);
+        if (n < p.N && c < p.P) gS[(size_t)n * p.P + c] = S[i][j][e];
+      }
 }
 
 // ------------------------------------------------------------------------------------------ one token per sequence
@@ -215,7 +448,15 @@ template <typename T, int VEC> __global__ void ssm_norm_kernel(const Params p) {
 
 static bool al(const void *q, int bytes) { return ((uintptr_t)q & (bytes - 1)) == 0; }
 
-template <typename T> static int run(const Params &p, cudaStream_t st) {
+template <int NP> static int launch_chunk(const Params &p, cudaStream_t st) {
+  static bool set = false;
+  if (!set) { PT_CUDA(cudaFuncSetAttribute(ssm_chunk_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(ChunkSmem<NP>))); set = true; }
+  ssm_chunk_kernel<NP><<<dim3(ceil_div(p.P, CP), p.heads, p.n_seq), CHUNK_THREADS, sizeof(ChunkSmem<NP>), st>>>(p);
+  PT_LAUNCH_CHECK("pt_ssm");
+  return PT_OK;
+}
+
+template <typename T> static int run(const Params &p, bool plain, cudaStream_t st) {
   if (p.n_tok == p.n_seq) {
     const bool v4 = p.P % 4 == 0 && p.P / 4 <= STEP_THREADS && al(p.state, 16);
     const int pq = v4 ? p.P / 4 : p.P, ng = std::max(1, STEP_THREADS / pq);
@@ -228,11 +469,17 @@ template <typename T> static int run(const Params &p, cudaStream_t st) {
   } else {
     ssm_conv_kernel<T><<<dim3(ceil_div(p.C + p.heads, 256), p.n_tok), 256, 0, st>>>(p);
     PT_LAUNCH_CHECK("pt_ssm");
-    const size_t smem = ((size_t)p.N * SCAN_P + 2 * p.N + SCAN_WARPS * 32) * sizeof(float);
-    PT_REQUIRE(smem <= 200 * 1024, "pt_ssm: state %d needs %zu bytes of shared memory", p.N, smem);
-    if (smem > 48 * 1024) PT_CUDA(cudaFuncSetAttribute(ssm_scan_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    ssm_scan_kernel<T><<<dim3(ceil_div(p.P, SCAN_P), p.heads, p.n_seq), SCAN_WARPS * 32, smem, st>>>(p);
-    PT_LAUNCH_CHECK("pt_ssm");
+    // the chunked form: bf16, rows that are whole 16-byte units, state of at most 256
+    if (!plain && sizeof(T) == 2 && p.N <= 256 && p.N % 8 == 0 && p.P % 8 == 0 && al(p.xbc, 16) && al(p.y, 8)) {
+      const int rc = p.N <= 64 ? launch_chunk<64>(p, st) : (p.N <= 128 ? launch_chunk<128>(p, st) : launch_chunk<256>(p, st));
+      if (rc != PT_OK) return rc;
+    } else {
+      const size_t smem = ((size_t)p.N * SCAN_P + 2 * p.N + SCAN_WARPS * 32) * sizeof(float);
+      PT_REQUIRE(smem <= 200 * 1024, "pt_ssm: state %d needs %zu bytes of shared memory", p.N, smem);
+      if (smem > 48 * 1024) PT_CUDA(cudaFuncSetAttribute(ssm_scan_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+      ssm_scan_kernel<T><<<dim3(ceil_div(p.P, SCAN_P), p.heads, p.n_seq), SCAN_WARPS * 32, smem, st>>>(p);
+      PT_LAUNCH_CHECK("pt_ssm");
+    }
   }
   const int len = p.inner / p.norm_groups;
   const bool v4 = len % 4 == 0 && al(p.out, 4 * sizeof(T)) && p.out_ld % 4 == 0;
@@ -274,5 +521,5 @@ extern "C" int pt_ssm(const pt_ssm_args *a, void *stream) {
   p.cu = b.cu; p.start = b.start; p.slot = b.slot; p.tok_seq = b.tok_seq;
   p.zx = a->zx; p.conv_w = a->conv_w; p.conv_b = a->conv_b; p.dt_bias = a->dt_bias; p.A_log = a->A_log; p.D = a->D; p.norm_w = a->norm_w;
   p.ring = a->ring; p.xbc = a->xbc; p.out = a->out; p.state = a->state; p.dt = a->dt; p.y = a->y;
-  return a->dtype == PT_DT_F32 ? ssm::run<float>(p, as_stream(stream)) : ssm::run<__nv_bfloat16>(p, as_stream(stream));
+  return a->dtype == PT_DT_F32 ? ssm::run<float>(p, a->plain != 0, as_stream(stream)) : ssm::run<__nv_bfloat16>(p, a->plain != 0, as_stream(stream));
 }

@@ -22,7 +22,7 @@ namespace wa {
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct Params {
-  int n_seq, n_head, n_kv, qpk, dim, vdim, page, max_pages, window, keep_first;
+  int n_seq, n_head, n_kv, qpk, dim, vdim, page, max_pages, max_len, window, keep_first;
   int q_ld, kv_ld, out_ld;
   float scale;
   const float *sink;
@@ -55,7 +55,7 @@ __device__ __forceinline__ int kept_pages(const Params &p, int pos) { return (mi
 // ------------------------------------------------------------------------------------------ append
 template <typename T> __global__ void kv_append_kernel(const Params p) {
   const int t = blockIdx.x, s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
-  if (pos < 0 || pos >= p.page * p.max_pages) {
+  if (pos < 0 || pos >= p.max_len) {
     if (threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
   }
@@ -74,7 +74,7 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
   float *q = sm, *sc = q + p.qpk * p.dim, *o = sc + p.qpk * p.page, *st = o + p.qpk * p.vdim;   // st: running max, sum, correction
   const int t = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
-  if (pos < 0 || pos >= p.page * p.max_pages) {
+  if (pos < 0 || pos >= p.max_len) {
     if (tid == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
   }
@@ -133,6 +133,390 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
     for (int i = p.n_head * p.vdim + tid; i < p.out_ld; i += PLAIN_THREADS) reinterpret_cast<T *>(p.out)[(size_t)t * p.out_ld + i] = from_f<T>(0.f);
 }
 
+// ------------------------------------------------------------------------------------------ tensor cores
+constexpr int TC_THREADS = 128, TILE = 64;   // TILE = the page size the tensor-core kernels take
+
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
+}
+// 16-byte asynchronous copy; zeros instead of the source when !in (the source address is then not read).
+__device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+
+// ------------------------------------------------------------------------------------------ prompts
+// Block: 64 new tokens of one sequence, one head; warp w owns queries 16 w .. 16 w + 15, their q fragments stay in registers.  Key
+// tiles (one page each) are double-buffered in shared memory; tiles without a visible key are skipped, tiles that every query of
+// the warp sees completely take no mask.  DK / DV: dim / vdim rounded up to 32, 64 or 128 (the padding holds zeros).
+template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_prompt_kernel(const Params p) {
+  constexpr int KLD = DK + 8, VLD = DV + 8;
+  extern __shared__ __align__(16) __nv_bfloat16 smb[];
+  __nv_bfloat16 *Ks = smb, *Vs = smb + 2 * TILE * KLD;      // [2][TILE][KLD], [2][TILE][VLD]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
+  const int s = blockIdx.z, head = blockIdx.y, t0 = blockIdx.x * TILE, kvh = head / p.qpk;
+  const int row0 = p.cu[s], len = p.cu[s + 1] - row0, start = p.start[s];
+  if (t0 >= len) return;
+  if (start < 0 || start + len > p.max_len) {
+    if (tid == 0 && p.error_flag) atomicExch(p.error_flag, 12);
+    return;
+  }
+  const int *table = p.page_table + (size_t)p.slot[s] * p.max_pages;
+  const int q0 = t0 + warp * 16 + g, q1 = q0 + 8;           // this lane's two queries
+  const bool ok0 = q0 < len, ok1 = q1 < len;
+  const int pos0 = start + q0, pos1 = start + q1;
+  const int lo = start + t0, hi = start + min(len, t0 + TILE) - 1;                                  // positions of the block's queries
+  const int wlo = start + t0 + warp * 16, whi = start + min(len, t0 + warp * 16 + 16) - 1;          // ... and of the warp's (whi < wlo: none)
+  uint32_t qa[DK / 16][4];
+  {
+    const __nv_bfloat16 *q = reinterpret_cast<const __nv_bfloat16 *>(p.q) + (size_t)head * p.dim + 2 * tig;
+    const __nv_bfloat16 *r0 = q + (size_t)(row0 + (ok0 ? q0 : 0)) * p.q_ld, *r1 = q + (size_t)(row0 + (ok1 ? q1 : 0)) * p.q_ld;
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      const bool in0 = kk * 16 < p.dim, in1 = kk * 16 + 8 < p.dim;
+      qa[kk][0] = (ok0 && in0) ? *reinterpret_cast<const uint32_t *>(r0 + kk * 16) : 0u;
+      qa[kk][1] = (ok1 && in0) ? *reinterpret_cast<const uint32_t *>(r1 + kk * 16) : 0u;
+      qa[kk][2] = (ok0 && in1) ? *reinterpret_cast<const uint32_t *>(r0 + kk * 16 + 8) : 0u;
+      qa[kk][3] = (ok1 && in1) ? *reinterpret_cast<const uint32_t *>(r1 + kk * 16 + 8) : 0u;
+    }
+  }
+  auto load_tile = [&](int kt, int stage) {
+    const int phys = table[kt];
+    const __nv_bfloat16 *gK = k_page<__nv_bfloat16>(p, phys, kvh), *gV = v_page<__nv_bfloat16>(p, phys, kvh);
+    __nv_bfloat16 *k = Ks + stage * TILE * KLD, *v = Vs + stage * TILE * VLD;
+    for (int e = tid; e < TILE * (DK / 8); e += TC_THREADS) {
+      const int r = e / (DK / 8), c = (e % (DK / 8)) * 8;
+      const bool in = kt * TILE + r <= hi && c < p.dim;
+      cp16(k + r * KLD + c, gK + (in ? (size_t)r * p.dim + c : 0), in);
+    }
+    for (int e = tid; e < TILE * (DV / 8); e += TC_THREADS) {
+      const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
+      const bool in = kt * TILE + r <= hi && c < p.vdim;
+      cp16(v + r * VLD + c, gV + (in ? (size_t)r * p.vdim + c : 0), in);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int kept = kept_pages(p, hi), wtile = window_page(p, lo), last = hi / TILE;
+  auto next_tile = [&](int kt) { return (kt >= kept && kt < wtile) ? wtile : kt; };
+  const float sc2 = p.scale * kLog2e, sink2 = p.sink ? p.sink[head] * kLog2e : -INFINITY;
+  float o[DV / 8][4];
+#pragma unroll
+  for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  float m_run[2] = {sink2, sink2}, l_run[2] = {0.f, 0.f};
+  int kt = next_tile(0), stage = 0;
+  load_tile(kt, 0);
+  for (; kt <= last; stage ^= 1) {
+    const int nt = next_tile(kt + 1);
+    if (nt <= last) {
+      load_tile(nt, stage ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const int k0 = kt * TILE;
+    // anything of this tile for this warp?  (uniform over the warp)
+    if (wlo <= whi && k0 <= whi && (p.window == 0 || k0 + TILE - 1 > wlo - p.window || k0 < p.keep_first)) {
+      const __nv_bfloat16 *K = Ks + stage * TILE * KLD;
+      float sc[TILE / 8][4];
+#pragma unroll
+      for (int j = 0; j < TILE / 8; ++j) {
+        sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+        const __nv_bfloat16 *kr = K + (j * 8 + g) * KLD + 2 * tig;
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk)
+          mma16816_bf16(sc[j], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], *reinterpret_cast<const uint32_t *>(kr + kk * 16),
+                        *reinterpret_cast<const uint32_t *>(kr + kk * 16 + 8));
+      }
+      const bool whole = k0 + TILE - 1 <= wlo && (p.window == 0 || whi - k0 < p.window || k0 + TILE <= p.keep_first);
+      float m_new[2] = {m_run[0], m_run[1]};
+#pragma unroll
+      for (int j = 0; j < TILE / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int key = k0 + j * 8 + 2 * tig + (e & 1);
+          float v = sc[j][e] * sc2;
+          if (!whole && !visible(p, e < 2 ? pos0 : pos1, key)) v = -INFINITY;
+          sc[j][e] = v;
+          m_new[e >> 1] = fmaxf(m_new[e >> 1], v);
+        }
+      float corr[2], base[2], l_tile[2] = {0.f, 0.f};
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 1));
+        m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 2));
+        base[r] = m_new[r] == -INFINITY ? 0.f : m_new[r];       // nothing seen yet: every weight below is exp2(-inf) = 0
+        corr[r] = exp2f(m_run[r] - base[r]);
+        m_run[r] = m_new[r];
+      }
+#pragma unroll
+      for (int j = 0; j < TILE / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sc[j][e] = exp2f(sc[j][e] - base[e >> 1]);
+          l_tile[e >> 1] += sc[j][e];
+        }
+      l_run[0] = l_run[0] * corr[0] + l_tile[0];                // per lane; the four lanes of a row are added at the end
+      l_run[1] = l_run[1] * corr[1] + l_tile[1];
+#pragma unroll
+      for (int j = 0; j < DV / 8; ++j) {
+        o[j][0] *= corr[0]; o[j][1] *= corr[0];
+        o[j][2] *= corr[1]; o[j][3] *= corr[1];
+      }
+      const uint32_t v_lane = smem_addr(Vs + stage * TILE * VLD + (lane & 15) * VLD + (lane >> 4) * 8);
+#pragma unroll
+      for (int k2 = 0; k2 < TILE / 16; ++k2) {
+        uint32_t h[4], l[4];                                    // weights as hi + lo: A fragments of two products
+        split_bf2(sc[2 * k2][0], sc[2 * k2][1], h[0], l[0]);
+        split_bf2(sc[2 * k2][2], sc[2 * k2][3], h[1], l[1]);
+        split_bf2(sc[2 * k2 + 1][0], sc[2 * k2 + 1][1], h[2], l[2]);
+        split_bf2(sc[2 * k2 + 1][2], sc[2 * k2 + 1][3], h[3], l[3]);
+#pragma unroll
+        for (int jn = 0; jn < DV / 8; jn += 2) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(v_lane + (uint32_t)(k2 * 16 * VLD + jn * 8) * 2u, b0, b1, b2, b3);
+          mma16816_bf16(o[jn], h[0], h[1], h[2], h[3], b0, b1);
+          mma16816_bf16(o[jn + 1], h[0], h[1], h[2], h[3], b2, b3);
+          mma16816_bf16(o[jn], l[0], l[1], l[2], l[3], b0, b1);
+          mma16816_bf16(o[jn + 1], l[0], l[1], l[2], l[3], b2, b3);
+        }
+      }
+    }
+    __syncthreads();                                            // the stage may be refilled
+    kt = nt;
+  }
+  float inv[2];
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    float l = l_run[r];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    if (p.sink) l += exp2f(sink2 - m_run[r]);                   // counts once, in the units of the running maximum
+    inv[r] = 1.0f / l;
+  }
+  __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(p.out) + (size_t)head * p.vdim + 2 * tig;
+#pragma unroll
+  for (int j = 0; j < DV / 8; ++j) {
+    if (j * 8 >= p.vdim) break;
+    if (ok0) *reinterpret_cast<uint32_t *>(out + (size_t)(row0 + q0) * p.out_ld + j * 8) = pack_bf2(o[j][0] * inv[0], o[j][1] * inv[0]);
+    if (ok1) *reinterpret_cast<uint32_t *>(out + (size_t)(row0 + q1) * p.out_ld + j * 8) = pack_bf2(o[j][2] * inv[1], o[j][3] * inv[1]);
+  }
+  const int pad = p.out_ld - p.n_head * p.vdim;
+  if (head == p.n_head - 1)
+    for (int i = tid; i < TILE * pad; i += TC_THREADS) {
+      const int r = t0 + i / pad;
+      if (r < len) reinterpret_cast<__nv_bfloat16 *>(p.out)[(size_t)(row0 + r) * p.out_ld + p.n_head * p.vdim + i % pad] = from_f<__nv_bfloat16>(0.f);
+    }
+}
+
+// ------------------------------------------------------------------------------------------ one token per sequence
+// Block: one visible page of one (sequence, kv head, part of the group's query heads).  scores^T [keys x heads] = K q^T with the K
+// rows straight from global memory as A fragments (the k order is a permutation of the channels that q follows); out [heads x vdim]
+// = P V with V staged in shared memory.  Rows 0..7 of P's A fragment are the hi parts of up to 8 heads' weights, rows 8..15 the lo
+// parts, so the split costs no extra product.  The block of the newest page takes the new key and value from the projection and
+// appends them.
+constexpr int NQ = 8;
+template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_decode_kernel(const Params p) {
+  constexpr int VLD = DV + 8, QLD = DK + 32, PSLD = TILE + 8;
+  typedef __nv_bfloat16 T;
+  extern __shared__ __align__(16) unsigned char smd[];
+  T *Vs = reinterpret_cast<T *>(smd);                          // [TILE][VLD]
+  T *qs = Vs + TILE * VLD;                                     // [NQ][QLD]
+  float *ps = reinterpret_cast<float *>(qs + NQ * QLD);        // [NQ][PSLD]
+  float *ml = ps + NQ * PSLD;                                  // [NQ][2]
+  float *cw = ml + NQ * 2;                                     // combine: [NQ][grid_pages] weights
+  __shared__ int s_last;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
+  const int s = blockIdx.z, kvh = blockIdx.y / p.qsplit, part = blockIdx.y - kvh * p.qsplit;
+  const int nq = p.qpk / p.qsplit, h0 = kvh * p.qpk + part * nq;           // this block's query heads h0 .. h0 + nq - 1
+  const int pos = p.start[s], t = p.cu[s];
+  if (pos < 0 || pos >= p.max_len) {
+    if (tid == 0 && p.error_flag) atomicExch(p.error_flag, 12);
+    return;
+  }
+  const int last = pos / TILE, kept = kept_pages(p, pos), wp = window_page(p, pos);
+  const int n_act = kept >= wp ? last + 1 : kept + last - wp + 1;
+  const int x = blockIdx.x;
+  if (x >= n_act) return;
+  const int pg = (kept >= wp || x < kept) ? x : wp + x - kept;
+  const int phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pg];
+  const int k0 = pg * TILE, n_valid = min(TILE, pos + 1 - k0);
+  const bool owner = pg == last && p.k != nullptr;
+  const int n_load = owner ? n_valid - 1 : n_valid, at = n_valid - 1;      // owner: the newest key is not in the pool yet
+  T *gK = k_page<T>(p, phys, kvh), *gV = v_page<T>(p, phys, kvh);
+  const T *knew = reinterpret_cast<const T *>(p.k) + (size_t)t * p.kv_ld + (size_t)kvh * p.dim;
+  const T *vnew = reinterpret_cast<const T *>(p.v) + (size_t)t * p.kv_ld + (size_t)kvh * p.vdim;
+
+  uint4 kf[2][DK / 32];                                        // K rows 16 warp + g and + 8 of the page
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int key = warp * 16 + g + 8 * r;
+#pragma unroll
+    for (int pp = 0; pp < DK / 32; ++pp) {
+      const int c = pp * 32 + tig * 8;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (c < p.dim) {
+        if (key < n_load) v = __ldcg(reinterpret_cast<const uint4 *>(gK + (size_t)key * p.dim + c));
+        else if (owner && key == at) v = *reinterpret_cast<const uint4 *>(knew + c);
+      }
+      kf[r][pp] = v;
+    }
+  }
+  for (int e = tid; e < TILE * (DV / 8); e += TC_THREADS) {
+    const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
+    const bool in = c < p.vdim && (r < n_load || (owner && r == at));
+    const T *src = (owner && r == at) ? vnew + c : gV + (size_t)r * p.vdim + c;
+    cp16(Vs + r * VLD + c, in ? src : gV, in);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * p.dim;
+  for (int i = tid; i < NQ * (DK / 8); i += TC_THREADS) {
+    const int h = i / (DK / 8), c = (i % (DK / 8)) * 8;
+    *reinterpret_cast<uint4 *>(qs + h * QLD + c) = (h < nq && c < p.dim) ? *reinterpret_cast<const uint4 *>(q + (size_t)h * p.dim + c) : make_uint4(0, 0, 0, 0);
+  }
+  for (int i = tid; i < NQ * PSLD; i += TC_THREADS) ps[i] = -INFINITY;
+  if (owner && part == 0) {
+    for (int c = tid; c < p.dim; c += TC_THREADS) gK[(size_t)at * p.dim + c] = knew[c];
+    for (int c = tid; c < p.vdim; c += TC_THREADS) gV[(size_t)at * p.vdim + c] = vnew[c];
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+
+  if (warp * 16 < n_valid) {
+    float sc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int pp = 0; pp < DK / 32; ++pp) {
+      const uint4 qv = *reinterpret_cast<const uint4 *>(qs + g * QLD + pp * 32 + tig * 8);
+      mma16816_bf16(sc, kf[0][pp].x, kf[1][pp].x, kf[0][pp].y, kf[1][pp].y, qv.x, qv.y);
+      mma16816_bf16(sc, kf[0][pp].z, kf[1][pp].z, kf[0][pp].w, kf[1][pp].w, qv.z, qv.w);
+    }
+    const float sc2 = p.scale * kLog2e;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {                              // keys 16 warp + g (+ 8) against heads 2 tig, 2 tig + 1
+      const int key = warp * 16 + g + 8 * (e >> 1), h = 2 * tig + (e & 1);
+      if (h < nq && key < n_valid && visible(p, pos, k0 + key)) ps[h * PSLD + key] = sc[e] * sc2;
+    }
+  }
+  __syncthreads();
+  for (int h = warp; h < NQ; h += TC_THREADS / 32) {
+    float *pr = ps + h * PSLD;
+    if (h >= nq) {
+      pr[lane] = pr[lane + 32] = 0.f;
+      continue;
+    }
+    const float a = pr[lane], b = pr[lane + 32], m = warp_max(fmaxf(a, b));
+    const float base = m == -INFINITY ? 0.f : m, ea = exp2f(a - base), eb = exp2f(b - base);
+    pr[lane] = ea;
+    pr[lane + 32] = eb;
+    const float l = warp_sum(ea + eb);
+    if (lane == 0) { ml[2 * h] = m; ml[2 * h + 1] = l; }
+  }
+  __syncthreads();
+  const size_t head0 = (size_t)s * p.n_head + h0;
+  {
+    constexpr int NT = DV / 32;                                // 8-channel tiles per warp
+    float o[NT][4];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    const float *pr = ps + g * PSLD + 2 * tig;
+    const uint32_t v_lane = smem_addr(Vs + (lane & 15) * VLD + warp * (DV / 4) + (NT > 1 ? (lane >> 4) * 8 : 0));
+    for (int k2 = 0; k2 * 16 < n_valid; ++k2) {
+      const float2 p0 = *reinterpret_cast<const float2 *>(pr + k2 * 16), p1 = *reinterpret_cast<const float2 *>(pr + k2 * 16 + 8);
+      uint32_t a0, a1, a2, a3;
+      split_bf2(p0.x, p0.y, a0, a1);
+      split_bf2(p1.x, p1.y, a2, a3);
+#pragma unroll
+      for (int j = 0; j < NT; j += 2) {
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4_trans(v_lane + (uint32_t)(k2 * 16 * VLD + j * 8) * 2u, b0, b1, b2, b3);
+        mma16816_bf16(o[j], a0, a1, a2, a3, b0, b1);
+        if (j + 1 < NT) mma16816_bf16(o[j + 1], a0, a1, a2, a3, b2, b3);
+      }
+    }
+    if (g < nq) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const int c = warp * (DV / 4) + j * 8 + 2 * tig;
+        if (c < p.vdim)
+          *reinterpret_cast<float2 *>(&p.ws_o[((head0 + g) * p.grid_pages + x) * p.vdim + c]) = make_float2(o[j][0] + o[j][2], o[j][1] + o[j][3]);
+      }
+    }
+  }
+  if (tid < nq) p.ws_ml[(head0 + tid) * p.grid_pages + x] = make_float2(ml[2 * tid], ml[2 * tid + 1]);
+
+  // ---- the last block of this (sequence, kv head, part) combines the pages in page order
+  __threadfence();
+  __syncthreads();
+  int *ctr = p.counters + ((size_t)s * p.n_kv + kvh) * p.qsplit + part;
+  if (tid == 0) s_last = atomicAdd(ctr, 1) == n_act - 1;
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+  if (tid == 0) *ctr = 0;
+  for (int h = warp; h < nq; h += TC_THREADS / 32) {
+    const float2 *src = p.ws_ml + (head0 + h) * p.grid_pages;
+    const float sink2 = p.sink ? p.sink[h0 + h] * kLog2e : -INFINITY;
+    float m = sink2;
+    for (int i = lane; i < n_act; i += 32) m = fmaxf(m, __ldcg(&src[i]).x);
+    m = warp_max(m);
+    float l = 0.f;
+    for (int i = lane; i < n_act; i += 32) {
+      const float2 v = __ldcg(&src[i]);
+      const float w = exp2f(v.x - m);
+      cw[h * p.grid_pages + i] = w;
+      l += v.y * w;
+    }
+    l = warp_sum(l);
+    if (lane == 0) ml[2 * h] = 1.0f / (l + (p.sink ? exp2f(sink2 - m) : 0.f));
+  }
+  __syncthreads();
+  T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld;
+  for (int i = tid; i < nq * p.vdim; i += TC_THREADS) {
+    const int h = i / p.vdim, c = i - h * p.vdim;
+    const float *src = p.ws_o + ((head0 + h) * p.grid_pages) * p.vdim + c, *w = cw + h * p.grid_pages;
+    constexpr int PB = 8;                                      // pages in flight
+    float acc = 0.f;
+    for (int i0 = 0; i0 < n_act; i0 += PB) {
+      float v[PB];
+#pragma unroll
+      for (int j = 0; j < PB; ++j) v[j] = i0 + j < n_act ? __ldcg(src + (size_t)(i0 + j) * p.vdim) : 0.f;
+#pragma unroll
+      for (int j = 0; j < PB; ++j)
+        if (i0 + j < n_act) acc = fmaf(v[j], w[i0 + j], acc);
+    }
+    out[(size_t)(h0 + h) * p.vdim + c] = from_f<T>(acc * ml[2 * h]);
+  }
+  if (h0 + nq == p.n_head)
+    for (int i = p.n_head * p.vdim + tid; i < p.out_ld; i += TC_THREADS) out[i] = from_f<T>(0.f);
+}
+
+template <int DK, int DV> static int launch_prompt(const Params &p, int longest, cudaStream_t st) {
+  constexpr size_t smem = 2 * (size_t)TILE * (DK + 8 + DV + 8) * sizeof(__nv_bfloat16);
+  static bool set = false;
+  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_prompt_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set = true; }
+  attn_prompt_kernel<DK, DV><<<dim3(ceil_div(longest, TILE), p.n_head, p.n_seq), TC_THREADS, smem, st>>>(p);
+  PT_LAUNCH_CHECK("pt_window_attn");
+  return PT_OK;
+}
+template <int DK, int DV> static int launch_decode(const Params &p, cudaStream_t st) {
+  const size_t smem = (size_t)(TILE * (DV + 8) + NQ * (DK + 32)) * sizeof(__nv_bfloat16) + (size_t)(NQ * (TILE + 8) + NQ * 2 + NQ * p.grid_pages) * sizeof(float);
+  PT_REQUIRE(smem <= 200 * 1024, "pt_window_attn: %d pages per sequence need %zu bytes of shared memory", p.grid_pages, smem);
+  static bool set = false;
+  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
+  attn_decode_kernel<DK, DV><<<dim3(p.grid_pages, p.n_kv * p.qsplit, p.n_seq), TC_THREADS, smem, st>>>(p);
+  PT_LAUNCH_CHECK("pt_window_attn");
+  return PT_OK;
+}
+template <int DK> static int dispatch_v(const Params &p, bool decode, int longest, cudaStream_t st) {
+  if (p.vdim <= 32) return decode ? launch_decode<DK, 32>(p, st) : launch_prompt<DK, 32>(p, longest, st);
+  if (p.vdim <= 64) return decode ? launch_decode<DK, 64>(p, st) : launch_prompt<DK, 64>(p, longest, st);
+  return decode ? launch_decode<DK, 128>(p, st) : launch_prompt<DK, 128>(p, longest, st);
+}
+static int dispatch_tc(const Params &p, bool decode, int longest, cudaStream_t st) {
+  if (p.dim <= 32) return dispatch_v<32>(p, decode, longest, st);
+  if (p.dim <= 64) return dispatch_v<64>(p, decode, longest, st);
+  return dispatch_v<128>(p, decode, longest, st);
+}
+
 }  // namespace wa
 }  // namespace pt
 
@@ -144,10 +528,13 @@ static int decode_pages(int page_size, int max_len, int window, int keep_first) 
   return window == 0 ? all : std::min(all, ceil_div(keep_first, page_size) + ceil_div(window - 1, page_size) + 1);
 }
 static size_t align256(size_t v) { return (v + 255) / 256 * 256; }
+// Workspace layout: [arrival counters][(max, sum) per page][outputs per page].  The counter region has ONE size, so that layers and
+// batches of different shapes can share a workspace: the statistics of one never land where another expects zeroed counters.
+constexpr size_t kCounterBytes = 1u << 18;
 
 extern "C" size_t pt_window_attn_workspace_bytes(int n_seq, int n_head, int vdim, int page_size, int max_len, int window, int keep_first) {
   const size_t heads = (size_t)n_seq * n_head, pages = decode_pages(page_size, max_len, window, keep_first);
-  return align256(heads * sizeof(int)) + align256(heads * pages * sizeof(float2)) + heads * pages * vdim * sizeof(float);
+  return kCounterBytes + align256(heads * pages * sizeof(float2)) + heads * pages * vdim * sizeof(float);
 }
 
 extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
@@ -168,12 +555,37 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
   p.q_ld = a->q_ld; p.kv_ld = a->kv_ld; p.out_ld = a->out_ld; p.scale = a->scale; p.sink = a->sink;
   p.q = a->q; p.k = a->k; p.v = a->v; p.pool = a->pool; p.out = a->out; p.page_table = a->page_table;
   p.cu = b.cu; p.start = b.start; p.slot = b.slot; p.tok_seq = b.tok_seq; p.error_flag = a->error_flag;
+  p.max_len = a->max_len > 0 ? a->max_len : a->page_size * a->max_pages;
+  PT_REQUIRE(p.max_len <= a->page_size * a->max_pages, "pt_window_attn: max_len=%d exceeds the %d positions of the page table", p.max_len,
+             a->page_size * a->max_pages);
   cudaStream_t st = as_stream(stream);
+  // the tensor-core kernels: bf16, 64-position pages, head widths of at most 128 whose rows are whole 16-byte units
+  auto al16 = [](const void *x) { return ((uintptr_t)x & 15) == 0; };
+  const bool tc = !a->plain && a->dtype == PT_DT_BF16 && a->page_size == wa::TILE && a->dim <= 128 && a->vdim <= 128 && a->dim % 8 == 0 && a->vdim % 8 == 0 &&
+                  a->q_ld % 8 == 0 && a->out_ld % 2 == 0 && al16(a->q) && al16(a->pool) && (!a->k || (a->kv_ld % 8 == 0 && al16(a->k) && al16(a->v)));
+  if (tc && b.n_tok == b.n_seq && b.n_seq <= 65535) {
+    const size_t need = pt_window_attn_workspace_bytes(b.n_seq, a->n_head, a->vdim, a->page_size, p.max_len, a->window, a->keep_first);
+    PT_REQUIRE(a->workspace && a->workspace_bytes >= need, "pt_window_attn: a decode step needs %zu workspace bytes, got %zu", need, a->workspace_bytes);
+    p.grid_pages = decode_pages(a->page_size, p.max_len, a->window, a->keep_first);
+    int nq = std::min(p.qpk, wa::NQ);
+    while (p.qpk % nq) --nq;
+    p.qsplit = p.qpk / nq;
+    const size_t heads = (size_t)b.n_seq * a->n_head;
+    char *ws = (char *)a->workspace;
+    PT_REQUIRE((size_t)b.n_seq * a->n_kv * p.qsplit <= kCounterBytes / sizeof(int), "pt_window_attn: %d sequences x %d heads exceed the arrival counters", b.n_seq,
+               a->n_head);
+    p.counters = (int *)ws; ws += kCounterBytes;
+    p.ws_ml = (float2 *)ws; ws += align256(heads * p.grid_pages * sizeof(float2));
+    p.ws_o = (float *)ws;
+    return wa::dispatch_tc(p, true, 1, st);
+  }
   if (p.k) {
     if (a->dtype == PT_DT_F32) wa::kv_append_kernel<float><<<b.n_tok, 128, 0, st>>>(p);
     else wa::kv_append_kernel<__nv_bfloat16><<<b.n_tok, 128, 0, st>>>(p);
     PT_LAUNCH_CHECK("pt_window_attn");
   }
+  if (tc && b.n_seq <= 65535)
+    return wa::dispatch_tc(p, false, a->max_tokens_per_seq > 0 ? a->max_tokens_per_seq : b.n_tok, st);
   const size_t smem = (size_t)p.qpk * (p.dim + p.page + p.vdim + 3) * sizeof(float);
   PT_REQUIRE(smem <= 200 * 1024, "pt_window_attn: %d query heads per kv head of widths %d / %d need %zu bytes of shared memory", p.qpk, p.dim, p.vdim, smem);
   if (smem > 48 * 1024) {
