@@ -598,6 +598,132 @@ def run_secondary(args):
     }))
 
 
+# ------------------------------------------------------------------------------------------ the hybrid architecture
+def hybrid_config(width, n_layer, ff, heads, kv_heads, dim, ssm_heads, ssm_dim, state, groups, vocab, window, keep_first, streams):
+    """A Sabisun of real-model layer sizes: three state-space layers, then one attention layer, repeated."""
+    mamba = {"type": "mamba2", "mixer": {"heads": ssm_heads, "vdim": ssm_dim, "state": state, "groups": groups, "conv": 4, "norm_groups": groups}}
+    attn = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                           "mask": {"size": window, "keep_first": keep_first}}}
+    return {"architecture": "Sabisun", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": 1e-5}, "residual_mult": 1.0, "logit_scale": 1.0,
+            "layers": [dict(attn if i % 4 == 3 else mamba, mlp={"ff": ff, "kind": "dense"}) for i in range(n_layer)]}
+
+
+HYBRID = {   # name: configuration, then the Llama of equal width, depth, feed-forward width and vocabulary that is timed beside it
+    "sabisun-2k": (dict(width=2048, n_layer=16, ff=8192, heads=16, kv_heads=4, dim=128, ssm_heads=64, ssm_dim=64, state=128, groups=8, vocab=32000, window=1024,
+                        keep_first=64, streams=2), dict(n_layer=16, d_model=2048, n_head=16, ffn=8192, vocab=32000)),
+    "sabisun-4k": (dict(width=4096, n_layer=16, ff=14336, heads=32, kv_heads=8, dim=128, ssm_heads=128, ssm_dim=64, state=128, groups=8, vocab=32000, window=1024,
+                        keep_first=64, streams=4), dict(n_layer=16, d_model=4096, n_head=32, ffn=14336, vocab=32000)),
+}
+
+
+def run_hybrid(args):
+    """Decode and prompt throughput of a Sabisun beside the Llama of equal size (fp16 weights, per-op kernels, for decode; INT4
+    weights for the prompt pass, the only one Llama has).  One JSON line, marked `secondary`."""
+    import torch
+    from poptransformer_b200 import llama, registry, synth
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device (there is no CPU fallback)")
+    dims, ldims = HYBRID[args.workload]
+    cfg = hybrid_config(**dims)
+    dev = torch.device("cuda", 0)
+    ctx, prompt, K = 2048, 2048, max(8, min(args.steps, 64))
+    max_len = ctx + K + 16
+    sd = synth.sabisun_state_dict(cfg, device=dev)
+    lsd = synth.llama_state_dict(**ldims, device=dev)
+    peak, _ = peaks()
+    sampler = ClockSampler(0)
+    sampler.start()
+    rows = []
+    for batch in (1, 8, 32):
+        dec = registry.build_decoder(cfg, sd, batch, max_len, "bfloat16", pad_id=-1)
+        dec._need_loop_rows()
+        for c in dec.caches.values():
+            c.pool.normal_(std=0.5)
+        dec.step_t.fill_(ctx)
+        dec.capture()
+        dec.step_t.fill_(ctx)
+
+        def steps(d):
+            for _ in range(3):
+                d.step()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            d.step_t.fill_(ctx)
+            torch.cuda.synchronize()
+            e0.record()
+            for _ in range(K):
+                d.step()
+            e1.record()
+            torch.cuda.synchronize()
+            if int(d.error_flag.item()):
+                raise SystemExit(f"device-side error flag {int(d.error_flag.item())}")
+            return e0.elapsed_time(e1) / K
+
+        ms = steps(dec)
+        w_bytes = dec.weight_bytes()
+        mixers = [lay["mixer"] for lay in cfg["layers"]]
+        state = sum(2 * 4 * m["heads"] * m["state"] * m["vdim"] for m in mixers if "state" in m)
+        kv = sum(2 * m["kv_heads"] * m["dim"] * 2 * (m["mask"]["size"] + m["mask"]["keep_first"]) for m in mixers if "mask" in m)
+        need = w_bytes + batch * (state + kv)
+        row = {"batch": batch, "decode_ms": ms, "decode_tokens_per_s": batch / ms * 1e3, "bytes_per_step": need, "decode_frac_of_measured": need / ms / 1e6 / peak}
+        del dec
+        ld = llama.LlamaDecoder(llama.LlamaConfig(**ldims, max_len=max_len), lsd, batch, device=dev, persistent=False)
+        for c in ld.caches:
+            c.pool.normal_(std=0.5)
+        ld.step_t.fill_(ctx)
+        ld.capture()
+        lms = steps(ld)
+        lneed = ld.weight_bytes() + batch * ld.kv_bytes_per_token_total() * ctx
+        row.update(llama_fp16_decode_ms=lms, llama_fp16_tokens_per_s=batch / lms * 1e3, llama_frac_of_measured=lneed / lms / 1e6 / peak)
+        del ld
+        torch.cuda.empty_cache()
+        rows.append(row)
+    # prompts
+    dec = registry.build_decoder(cfg, sd, 4, max_len, "bfloat16", pad_id=-1)
+    lin_flops = 2 * prompt * sum(s.proj.n_out * s.proj.k_in + s.out.n_out * s.out.k_in for s in dec.subs)
+    pre = []
+    r = np.random.default_rng(0)
+    for n_seq in (1, 4):
+        toks = [r.integers(0, cfg["vocab"], prompt).astype(np.int32) for _ in range(n_seq)]
+        best = None
+        for _ in range(4):
+            seqs = [dec.open() for _ in range(n_seq)]
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            dec.extend([(s, t, [prompt - 1]) for s, t in zip(seqs, toks)])
+            e1.record()
+            torch.cuda.synchronize()
+            ms = e0.elapsed_time(e1)
+            best = ms if best is None else min(best, ms)
+            for s in seqs:
+                dec.close(s)
+        pre.append({"sequences": n_seq, "prompt": prompt, "ms": best, "tokens_per_s": n_seq * prompt / best * 1e3, "linear_tflops": n_seq * lin_flops / best / 1e9})
+    del dec, lsd
+    torch.cuda.empty_cache()
+    qsd = synth.llama_state_dict(**ldims, device=dev, int4_group=GROUP)
+    ld = llama.LlamaDecoder(llama.LlamaConfig(**ldims, max_len=max_len, int4_group=GROUP), qsd, 1, device=dev, persistent=False, prefill=True)
+    ids = synth.prompt_ids(1, prompt, max_len, ldims["vocab"], ld.pad_id, seed=0)
+    times = []
+    for _ in range(4):
+        ld.reset(ids)
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        ld.prefill(prompt, chunk=prompt)
+        e1.record()
+        torch.cuda.synchronize()
+        times.append(e0.elapsed_time(e1))
+    lms = min(times)
+    lflops = 2 * prompt * ldims["n_layer"] * (4 * ldims["d_model"] ** 2 + 3 * ldims["d_model"] * ldims["ffn"])
+    clocks = sampler.stop()
+    print(json.dumps({"secondary": "not the headline workload; the hybrid architecture beside the Llama of equal size on one GPU", "metric": f"decode tokens/s ({args.workload}, batch 32)",
+                      "value": rows[-1]["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": 3, "ms_per_step": rows[-1]["decode_ms"],
+                      "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16 (float32 streams, softmax, state)", "data": "synthetic",
+                      "config": {"workload": args.workload, **dims, "ctx": ctx, "cuda_graph": True, "l2": "weights larger than L2 streamed per step"},
+                      "clocks": clocks, "decode": rows, "prompt_pass": pre,
+                      "llama_int4_prompt_pass": {"sequences": 1, "prompt": prompt, "ms": lms, "tokens_per_s": prompt / lms * 1e3, "linear_tflops": lflops / lms / 1e9}}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -614,13 +740,16 @@ def main():
                     "stays small; the line is then marked profiling_only and is not a benchmark result")
     ap.add_argument("--pdl", type=int, default=-1, help="secondary workloads: programmatic dependent launch, bit 0 = linear kernels, bit 1 = "
                     "attention kernel (-1: the decoder's default)")
-    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY),
-                    help="llama2-7b-int4 is the benchmark; the others time a parity configuration on one GPU (line marked `secondary`)")
+    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY) + list(HYBRID),
+                    help="llama2-7b-int4 is the benchmark; the others time a parity configuration, or the hybrid architecture beside the Llama of "
+                    "equal size, on one GPU (line marked `secondary`)")
     args = ap.parse_args()
     if args.impl == "reference":
         run_reference(args)
     elif args.workload in SECONDARY:
         run_secondary(args)
+    elif args.workload in HYBRID:
+        run_hybrid(args)
     else:
         run_b200(args)
 

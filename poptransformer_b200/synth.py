@@ -41,6 +41,52 @@ def llama_state_dict(n_layer, d_model, n_head, ffn, vocab, seed=0, device="cpu",
     return sd
 
 
+def sabisun_state_dict(config, seed=0, device="cpu"):
+    """Sabisun architecture (a parsed config.json), bfloat16: linears N(0, 1 / in_features), norms 1 + N(0, 0.02), stream weights near
+    the identity, decays and step sizes spread over slow and fast heads."""
+    gen = torch.Generator(device=device)
+    gen.manual_seed(seed)
+    sd = {}
+    W, S = config["width"], config["streams"]
+
+    def put(key, shape, std=1.0, mean=0.0):
+        sd[key] = (torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * std + mean).to(torch.bfloat16)
+
+    def lin(key, o, i):
+        put(key, (o, i), i ** -0.5)
+
+    put("embed", (config["vocab"], W))
+    put("final.norm", (W,), 0.02, 1.0)
+    for i, lay in enumerate(config["layers"]):
+        p, m, mlp = f"l{i}.", lay["mixer"], lay.get("mlp")
+        for q in ("1", "2") if mlp else ("1",):
+            put(p + "norm" + q, (W,), 0.02, 1.0)
+            put(p + f"hc{q}.in", (S,), 0.02, 1.0 / S)
+            put(p + f"hc{q}.out", (S,), 0.02, 1.0)
+            sd[p + f"hc{q}.mix"] = (torch.eye(S, device=device) + 0.02 * torch.randn((S, S), generator=gen, device=device)).to(torch.bfloat16)
+        if lay["type"] == "attention":
+            lin(p + "mix.q", m["heads"] * m["dim"], W)
+            if m.get("kv_from") is None:
+                lin(p + "mix.k", m["kv_heads"] * m["dim"], W)
+                lin(p + "mix.v", m["kv_heads"] * m["vdim"], W)
+            put(p + "mix.sink", (m["heads"],))
+            lin(p + "mix.o", W, m["heads"] * m["vdim"])
+        else:
+            inner, channels = m["heads"] * m["vdim"], m["heads"] * m["vdim"] + 2 * m["groups"] * m["state"]
+            lin(p + "mix.in", inner + channels + m["heads"], W)
+            put(p + "mix.conv", (channels, m["conv"]), 0.5)
+            put(p + "mix.conv.b", (channels,), 0.1)
+            put(p + "mix.dt_bias", (m["heads"],), 1.0, -3.0)
+            put(p + "mix.A_log", (m["heads"],), 1.0, 1.0)
+            put(p + "mix.D", (m["heads"],), 0.1, 1.0)
+            put(p + "mix.norm", (inner,), 0.02, 1.0)
+            lin(p + "mix.o", W, inner)
+        if mlp:
+            lin(p + "mlp.up", mlp["ff"], W)
+            lin(p + "mlp.down", W, mlp["ff"])
+    return sd
+
+
 def gpt2_state_dict(n_layer, d_model, n_head, vocab, n_positions, seed=0, device="cpu"):
     """GPT-2 architecture with the reference's key names after its checkpoint pre-processing (gpt2/model.py:154-166): linear
     weights [out, in], the query third of c_attn (weight and bias) multiplied by 1/sqrt(head_size).  fp16, N(0, 0.02);
