@@ -12,7 +12,28 @@ template <typename T> __device__ __forceinline__ T from_f(float x);
 template <> __device__ __forceinline__ float from_f<float>(float x) { return x; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float x) { return __float2bfloat16_rn(x); }
 
-// VEC consecutive values (VEC 1, 2 or 4; the address is aligned to VEC elements).
+template <int VEC> __device__ __forceinline__ void load_vec(const float *p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const float4 r = *reinterpret_cast<const float4 *>(p);
+    v[0] = r.x; v[1] = r.y; v[2] = r.z; v[3] = r.w;
+  } else {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = p[j];
+  }
+}
+template <int VEC> __device__ __forceinline__ void load_vec(const __nv_bfloat16 *p, float (&v)[VEC]) {
+  if constexpr (VEC == 8 || VEC == 4) {
+    __nv_bfloat162 h[VEC / 2];
+    if constexpr (VEC == 8) *reinterpret_cast<uint4 *>(h) = *reinterpret_cast<const uint4 *>(p);
+    else *reinterpret_cast<uint2 *>(h) = *reinterpret_cast<const uint2 *>(p);
+#pragma unroll
+    for (int j = 0; j < VEC / 2; ++j) { v[2 * j] = __low2float(h[j]); v[2 * j + 1] = __high2float(h[j]); }
+  } else {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = to_f(p[j]);
+  }
+}
+// VEC consecutive values (the address is aligned to VEC elements).
 template <int VEC> __device__ __forceinline__ void store_vec(float *p, const float (&v)[VEC]) {
   if constexpr (VEC == 4) *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
   else if constexpr (VEC == 2) *reinterpret_cast<float2 *>(p) = make_float2(v[0], v[1]);

@@ -14,6 +14,8 @@
 //   ssm_chunk_kernel   bf16 prompts: the same recurrence 64 tokens at a time on the tensor cores
 //   ssm_step_kernel    one token per sequence: convolution, step size, state update and readout in one launch
 //   ssm_norm_kernel    gate, group norm, and the ring update
+#include <type_traits>
+
 #include "elem.cuh"
 #include "tile_math.cuh"
 
@@ -52,6 +54,69 @@ template <typename T> __global__ void ssm_conv_kernel(const Params p) {
   } else if (c < p.C + p.heads) {
     const int h = c - p.C;
     p.dt[(size_t)t * p.heads + h] = softplus_f(to_f(zx[(size_t)t * p.zx_ld + p.inner + c]) + p.dt_bias[h]);
+  }
+}
+
+// The same for bf16 rows of whole 16-byte units and at most 4 taps: a thread slides over CONV_TOKENS tokens of 8 channels with the
+// window in registers; the last column of blocks computes the step sizes.
+constexpr int CONV_TOKENS = 16, CONV_THREADS = 128;
+template <int TAPS> __global__ void __launch_bounds__(CONV_THREADS) ssm_conv8_kernel(const Params p) {
+  typedef __nv_bfloat16 T;
+  const T *zx = reinterpret_cast<const T *>(p.zx);
+  const int ta = blockIdx.y * CONV_TOKENS, tb = min(p.n_tok, ta + CONV_TOKENS);
+  if (blockIdx.x == gridDim.x - 1) {
+    for (int i = threadIdx.x; i < (tb - ta) * p.heads; i += CONV_THREADS) {
+      const int t = ta + i / p.heads, h = i % p.heads;
+      p.dt[(size_t)t * p.heads + h] = softplus_f(to_f(zx[(size_t)t * p.zx_ld + p.inner + p.C + h]) + p.dt_bias[h]);
+    }
+    return;
+  }
+  const int c = (blockIdx.x * CONV_THREADS + threadIdx.x) * 8;
+  if (c >= p.C) return;
+  float w[8][TAPS], b[8], x[TAPS][8];     // x[k]: the input k tokens back
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    b[j] = p.conv_b[c + j];
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) w[j][k] = p.conv_w[(size_t)(c + j) * TAPS + k];
+  }
+  int seq = -1;
+#pragma unroll 4
+  for (int t = ta; t < tb; ++t) {
+    const int s = p.tok_seq[t];
+    if (s != seq) {                       // first token of this thread or of a sequence: the window as it stands before it
+      seq = s;
+      const int t0 = p.cu[s], pos = p.start[s] + t - t0;
+      const T *ring = reinterpret_cast<const T *>(p.ring) + (size_t)p.slot[s] * TAPS * p.C;
+#pragma unroll
+      for (int k = 1; k < TAPS; ++k) {
+        if (k > pos) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) x[k - 1][j] = 0.f;
+        } else if (t - k >= t0) {
+          load_vec<8>(zx + (size_t)(t - k) * p.zx_ld + p.inner + c, x[k - 1]);
+        } else {
+          load_vec<8>(ring + (size_t)((pos - k) % TAPS) * p.C + c, x[k - 1]);
+        }
+      }
+    }
+#pragma unroll
+    for (int k = TAPS - 1; k > 0; --k)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[k][j] = x[k - 1][j];
+    load_vec<8>(zx + (size_t)t * p.zx_ld + p.inner + c, x[0]);
+    __nv_bfloat162 o[4];
+    float y[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      float a = b[j];
+#pragma unroll
+      for (int k = 0; k < TAPS; ++k) a = fmaf(w[j][k], x[TAPS - 1 - k][j], a);
+      y[j] = silu_f(a);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j] = __floats2bfloat162_rn(y[2 * j], y[2 * j + 1]);
+    *reinterpret_cast<uint4 *>(reinterpret_cast<T *>(p.xbc) + (size_t)t * p.C + c) = *reinterpret_cast<const uint4 *>(o);
   }
 }
 
@@ -104,10 +169,15 @@ template <typename T> __global__ void __launch_bounds__(SCAN_WARPS * 32) ssm_sca
 // Block: 32 columns of one head's state, one sequence; it walks the chunks in order with the state in fp32 accumulators.  Operands
 // that are not already bf16 (the state, the decayed products, the weighted x) enter the tensor cores as hi + lo pairs.  c is kept
 // as a pair of floats, so differences of neighbours stay exact however far the sum has run.
+// Eight warps: two share 16 tokens of the output, each with half of the state rows (first product) and every other 16 tokens s
+// (second product); all eight share the state rows of the update.  One warp scans the next chunk's decays meanwhile.
 // NP: state size rounded up to 64, 128 or 256 (padding is zero).
-constexpr int CHUNK = 64, CP = 32, CHUNK_THREADS = 128;
+constexpr int CHUNK = 64, CP = 32, CHUNK_THREADS = 256;
 __device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
 }
 __device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
@@ -115,14 +185,17 @@ __device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
 template <int NP> struct ChunkSmem {
   static constexpr int BLD = NP + 8, XLD = CP + 8;
   __nv_bfloat16 B[2][CHUNK][BLD], C[2][CHUNK][BLD], X[2][CHUNK][XLD];
-  __nv_bfloat16 Sh[NP][XLD], Sl[NP][XLD];      // state before the chunk, hi and lo
+  __nv_bfloat16 Sh[NP][XLD], Sl[NP][XLD];         // state before the chunk, hi and lo
   __nv_bfloat16 Wh[CHUNK][XLD], Wl[CHUNK][XLD];   // exp(c_last - c_s) dt_s x_s
-  float c_hi[CHUNK], c_lo[CHUNK], dt[CHUNK];
+  float ypart[4][16][CP + 4];                     // the second warp's share of the output rows
+  float c_hi[2][CHUNK], c_lo[2][CHUNK], dt[2][CHUNK], ec[2][CHUNK], w[2][CHUNK], keep[2];
 };
 
 template <int NP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_chunk_kernel(const Params p) {
   typedef __nv_bfloat16 T;
-  constexpr int MT = NP / 64;                       // 16-row tiles of the state per warp
+  constexpr int MT = NP > 128 ? NP / 128 : 1;       // 16-row tiles of the state per warp ...
+  constexpr int NJ = NP == 64 ? 2 : 4;              // ... and 8-column tiles (64 rows are four row tiles: two warps share each)
+  constexpr int XLD = ChunkSmem<NP>::XLD;
   extern __shared__ __align__(16) unsigned char smraw[];
   ChunkSmem<NP> &sm = *reinterpret_cast<ChunkSmem<NP> *>(smraw);
   const int s = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * CP;
@@ -148,168 +221,210 @@ template <int NP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_chunk_ker
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
+  // Step sizes of the chunk at t0 (two per lane; zero beyond the sequence: decay 1, no contribution) ...
+  auto load_dt = [&](int t0, float (&d)[2]) {
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int r = t0 + 2 * lane + k;
+      d[k] = r < len ? p.dt[(size_t)(row0 + r) * p.heads + h] : 0.f;
+    }
+  };
+  // ... and what follows from them, by one warp.
+  auto scan_chunk = [&](const float (&d)[2], int stage) {
+    const double l1 = (double)(a * d[1]);
+    double sum = (double)(a * d[0]) + l1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const double v = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += v;
+    }
+    const double last = __shfl_sync(0xffffffffu, sum, 31);
+    const double c[2] = {sum - l1, sum};
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int r = 2 * lane + k;
+      sm.c_hi[stage][r] = (float)c[k];
+      sm.c_lo[stage][r] = (float)(c[k] - (double)(float)c[k]);
+      sm.dt[stage][r] = d[k];
+      sm.ec[stage][r] = expf((float)c[k]);
+      sm.w[stage][r] = expf((float)(last - c[k])) * d[k];
+    }
+    if (lane == 0) sm.keep[stage] = expf((float)last);
+  };
   load_chunk(0, 0);
+  constexpr int SCAN_WARP = 1;   // its output rows have the least work
+  float dnext[2];
+  if (warp == SCAN_WARP) {
+    load_dt(0, dnext);
+    scan_chunk(dnext, 0);
+  }
 
-  // state accumulators: warp w owns rows w NP / 4 ..; tile i, column tile j, lane (g, tig): rows g and g + 8, columns 2 tig, + 1
-  float S[MT][CP / 8][4];
-  const int srow = warp * (NP / 4) + g;
+  // state accumulators; lane (g, tig) of tile (i, j): rows g and g + 8, columns 2 tig, + 1
+  float S[MT][NJ][4];
+  const int srow = (NP == 64 ? (warp & 3) * 16 : warp * MT * 16) + g, sj0 = NP == 64 ? (warp >> 2) * NJ : 0;
   const bool fresh = p.start[s] == 0;
 #pragma unroll
   for (int i = 0; i < MT; ++i)
 #pragma unroll
-    for (int j = 0; j < CP / 8; ++j)
+    for (int j = 0; j < NJ; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + j * 8 + 2 * tig + (e & 1);
+        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + (sj0 + j) * 8 + 2 * tig + (e & 1);
         S[i][j][e] = (!fresh && n < p.N && c < p.P) ? gS[(size_t)n * p.P + c] : 0.f;
       }
   auto publish_state = [&]() {
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
-      for (int j = 0; j < CP / 8; ++j)
+      for (int j = 0; j < NJ; ++j)
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           uint32_t hi, lo;
           split_bf2(S[i][j][2 * r], S[i][j][2 * r + 1], hi, lo);
-          *reinterpret_cast<uint32_t *>(&sm.Sh[srow + i * 16 + 8 * r][j * 8 + 2 * tig]) = hi;
-          *reinterpret_cast<uint32_t *>(&sm.Sl[srow + i * 16 + 8 * r][j * 8 + 2 * tig]) = lo;
+          *reinterpret_cast<uint32_t *>(&sm.Sh[srow + i * 16 + 8 * r][(sj0 + j) * 8 + 2 * tig]) = hi;
+          *reinterpret_cast<uint32_t *>(&sm.Sl[srow + i * 16 + 8 * r][(sj0 + j) * 8 + 2 * tig]) = lo;
         }
   };
   publish_state();
 
+  const int rb = warp >> 1, half = warp & 1, tr = rb * 16 + g;      // this warp's output rows tr and tr + 8
   int stage = 0;
   for (int t0 = 0; t0 < len; t0 += CHUNK, stage ^= 1) {
-    if (t0 + CHUNK < len) {
+    const bool more = t0 + CHUNK < len;
+    if (more) {
       load_chunk(t0 + CHUNK, stage ^ 1);
+      if (warp == SCAN_WARP) load_dt(t0 + CHUNK, dnext);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
-    if (warp == 0) {   // step sizes and running log decays of the chunk (zero beyond the sequence: decay 1, no contribution)
-      const int r0 = t0 + 2 * lane, r1 = r0 + 1;
-      const float d0 = r0 < len ? p.dt[(size_t)(row0 + r0) * p.heads + h] : 0.f, d1 = r1 < len ? p.dt[(size_t)(row0 + r1) * p.heads + h] : 0.f;
-      const double l0 = (double)(a * d0), l1 = (double)(a * d1);
-      double sum = l0 + l1;
+    __syncthreads();   // operands, decays and the published state are in shared memory
 #pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const double v = __shfl_up_sync(0xffffffffu, sum, o);
-        if (lane >= o) sum += v;
-      }
-      const double c1 = sum, c0 = sum - l1;
-      sm.dt[2 * lane] = d0; sm.dt[2 * lane + 1] = d1;
-      sm.c_hi[2 * lane] = (float)c0; sm.c_lo[2 * lane] = (float)(c0 - (double)(float)c0);
-      sm.c_hi[2 * lane + 1] = (float)c1; sm.c_lo[2 * lane + 1] = (float)(c1 - (double)(float)c1);
-    }
-    __syncthreads();   // operands, step sizes and the published state are in shared memory
-    const float ce_hi = sm.c_hi[CHUNK - 1], ce_lo = sm.c_lo[CHUNK - 1];
     for (int e = tid; e < CHUNK * (CP / 2); e += CHUNK_THREADS) {   // weighted x for the state update
       const int r = e / (CP / 2), c = (e % (CP / 2)) * 2;
-      const float w = expf((ce_hi - sm.c_hi[r]) + (ce_lo - sm.c_lo[r])) * sm.dt[r];
+      const float w = sm.w[stage][r];
       const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[stage][r][c]);
       uint32_t hi, lo;
       split_bf2(w * __low2float(x2), w * __high2float(x2), hi, lo);
       *reinterpret_cast<uint32_t *>(&sm.Wh[r][c]) = hi;
       *reinterpret_cast<uint32_t *>(&sm.Wl[r][c]) = lo;
     }
-    // ---- rows 16 warp .. + 15 of the chunk's output
-    const int tr = warp * 16 + g;
-    float y[CP / 8][4], G[CHUNK / 8][4];
+    // ---- output rows: C S over half of the state rows, C B^T for this warp's tokens s (16 k2 .. + 15 with k2 = half, half + 2)
+    float y[CP / 8][4], G[2][2][4];
 #pragma unroll
     for (int j = 0; j < CP / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
 #pragma unroll
-    for (int j = 0; j < CHUNK / 8; ++j) G[j][0] = G[j][1] = G[j][2] = G[j][3] = 0.f;
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) G[u][j][0] = G[u][j][1] = G[u][j][2] = G[u][j][3] = 0.f;
+    const uint32_t c_lane = smem_addr(&sm.C[stage][rb * 16 + (lane & 15)][(lane >> 4) * 8]);
+    // (B rows are the n side: matrices (s 0-7, k 0-7), (s 0-7, k 8-15), (s 8-15, k 0-7), (s 8-15, k 8-15))
+    const uint32_t b_lane = smem_addr(&sm.B[stage][half * 16 + (lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]);
     const uint32_t sh_lane = smem_addr(&sm.Sh[lane & 15][(lane >> 4) * 8]), sl_lane = smem_addr(&sm.Sl[lane & 15][(lane >> 4) * 8]);
-#pragma unroll 2
+#pragma unroll 4
     for (int kk = 0; kk < NP / 16; ++kk) {
-      const T *c0 = &sm.C[stage][tr][kk * 16 + 2 * tig], *c1 = &sm.C[stage][tr + 8][kk * 16 + 2 * tig];
-      const uint32_t a0 = *reinterpret_cast<const uint32_t *>(c0), a1 = *reinterpret_cast<const uint32_t *>(c1);
-      const uint32_t a2 = *reinterpret_cast<const uint32_t *>(c0 + 8), a3 = *reinterpret_cast<const uint32_t *>(c1 + 8);
+      uint32_t a0, a1, a2, a3;
+      ldsm4(c_lane + (uint32_t)kk * 32u, a0, a1, a2, a3);
 #pragma unroll
-      for (int j = 0; j < CHUNK / 8; ++j) {
-        if (j > 2 * warp + 1) break;      // columns behind the diagonal only
-        const T *b = &sm.B[stage][j * 8 + g][kk * 16 + 2 * tig];
-        mma16816_bf16(G[j], a0, a1, a2, a3, *reinterpret_cast<const uint32_t *>(b), *reinterpret_cast<const uint32_t *>(b + 8));
-      }
-#pragma unroll
-      for (int j = 0; j < CP / 8; j += 2) {
+      for (int u = 0; u < 2; ++u) {
+        if (half + 2 * u > rb) break;     // tokens behind the diagonal only
         uint32_t b0, b1, b2, b3;
-        ldsm4t(sh_lane + (uint32_t)(kk * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, b0, b1, b2, b3);
-        mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
-        mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
-        ldsm4t(sl_lane + (uint32_t)(kk * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, b0, b1, b2, b3);
-        mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
-        mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
+        ldsm4(b_lane + (uint32_t)(u * 32 * ChunkSmem<NP>::BLD + kk * 16) * 2u, b0, b1, b2, b3);
+        mma16816_bf16(G[u][0], a0, a1, a2, a3, b0, b1);
+        mma16816_bf16(G[u][1], a0, a1, a2, a3, b2, b3);
+      }
+      if ((kk & 1) == half) {
+#pragma unroll
+        for (int j = 0; j < CP / 8; j += 2) {
+          uint32_t b0, b1, b2, b3;
+          ldsm4t(sh_lane + (uint32_t)(kk * 16 * XLD + j * 8) * 2u, b0, b1, b2, b3);
+          mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
+          mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
+          ldsm4t(sl_lane + (uint32_t)(kk * 16 * XLD + j * 8) * 2u, b0, b1, b2, b3);
+          mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
+          mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
+        }
       }
     }
-    const float h0 = sm.c_hi[tr], l0 = sm.c_lo[tr], h1 = sm.c_hi[tr + 8], l1 = sm.c_lo[tr + 8];
-    const float e0 = expf(h0 + l0), e1 = expf(h1 + l1);
+    const float e0 = sm.ec[stage][tr], e1 = sm.ec[stage][tr + 8];
 #pragma unroll
     for (int j = 0; j < CP / 8; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
+    const float h0 = sm.c_hi[stage][tr], l0 = sm.c_lo[stage][tr], h1 = sm.c_hi[stage][tr + 8], l1 = sm.c_lo[stage][tr + 8];
+    const uint32_t x_lane = smem_addr(&sm.X[stage][half * 16 + (lane & 15)][(lane >> 4) * 8]);
 #pragma unroll
-    for (int j = 0; j < CHUNK / 8; ++j) {
-      if (j > 2 * warp + 1) break;
+    for (int u = 0; u < 2; ++u) {
+      const int k2 = half + 2 * u;
+      if (k2 > rb) break;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int sc = j * 8 + 2 * tig + (e & 1), t = e < 2 ? tr : tr + 8;
-        const float d = e < 2 ? (h0 - sm.c_hi[sc]) + (l0 - sm.c_lo[sc]) : (h1 - sm.c_hi[sc]) + (l1 - sm.c_lo[sc]);
-        G[j][e] = sc <= t ? G[j][e] * expf(d) * sm.dt[sc] : 0.f;
+      for (int j = 0; j < 2; ++j) {
+        const int sc = k2 * 16 + j * 8 + 2 * tig;
+        const float2 ch = *reinterpret_cast<const float2 *>(&sm.c_hi[stage][sc]), cl = *reinterpret_cast<const float2 *>(&sm.c_lo[stage][sc]);
+        const float2 dt = *reinterpret_cast<const float2 *>(&sm.dt[stage][sc]);
+        G[u][j][0] = sc <= tr ? G[u][j][0] * expf((h0 - ch.x) + (l0 - cl.x)) * dt.x : 0.f;
+        G[u][j][1] = sc + 1 <= tr ? G[u][j][1] * expf((h0 - ch.y) + (l0 - cl.y)) * dt.y : 0.f;
+        G[u][j][2] = sc <= tr + 8 ? G[u][j][2] * expf((h1 - ch.x) + (l1 - cl.x)) * dt.x : 0.f;
+        G[u][j][3] = sc + 1 <= tr + 8 ? G[u][j][3] * expf((h1 - ch.y) + (l1 - cl.y)) * dt.y : 0.f;
       }
-    }
-    const uint32_t x_lane = smem_addr(&sm.X[stage][lane & 15][(lane >> 4) * 8]);
-#pragma unroll
-    for (int k2 = 0; k2 < CHUNK / 16; ++k2) {
-      if (k2 > warp) break;
       uint32_t hi[4], lo[4];
-      split_bf2(G[2 * k2][0], G[2 * k2][1], hi[0], lo[0]);
-      split_bf2(G[2 * k2][2], G[2 * k2][3], hi[1], lo[1]);
-      split_bf2(G[2 * k2 + 1][0], G[2 * k2 + 1][1], hi[2], lo[2]);
-      split_bf2(G[2 * k2 + 1][2], G[2 * k2 + 1][3], hi[3], lo[3]);
+      split_bf2(G[u][0][0], G[u][0][1], hi[0], lo[0]);
+      split_bf2(G[u][0][2], G[u][0][3], hi[1], lo[1]);
+      split_bf2(G[u][1][0], G[u][1][1], hi[2], lo[2]);
+      split_bf2(G[u][1][2], G[u][1][3], hi[3], lo[3]);
 #pragma unroll
       for (int j = 0; j < CP / 8; j += 2) {
         uint32_t b0, b1, b2, b3;
-        ldsm4t(x_lane + (uint32_t)(k2 * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, b0, b1, b2, b3);
+        ldsm4t(x_lane + (uint32_t)(u * 32 * XLD + j * 8) * 2u, b0, b1, b2, b3);
         mma16816_bf16(y[j], hi[0], hi[1], hi[2], hi[3], b0, b1);
         mma16816_bf16(y[j + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
         mma16816_bf16(y[j], lo[0], lo[1], lo[2], lo[3], b0, b1);
         mma16816_bf16(y[j + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
       }
     }
-#pragma unroll
-    for (int j = 0; j < CP / 8; ++j)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int t = tr + 8 * r, c = j * 8 + 2 * tig;
-        if (t0 + t >= len || col0 + c >= p.P) continue;
-        const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[stage][t][c]);
-        *reinterpret_cast<float2 *>(p.y + (size_t)(row0 + t0 + t) * p.inner + (size_t)h * p.P + col0 + c) =
-            make_float2(fmaf(D, __low2float(x2), y[j][2 * r]), fmaf(D, __high2float(x2), y[j][2 * r + 1]));
-      }
-    __syncthreads();   // the weighted x is complete; nobody reads the old state any more
-    // ---- state update: B^T [state rows x tokens] times the weighted x
-    const float keep = expf(ce_hi + ce_lo);
-#pragma unroll
-    for (int i = 0; i < MT; ++i)
+    if (half) {
 #pragma unroll
       for (int j = 0; j < CP / 8; ++j)
 #pragma unroll
+        for (int r = 0; r < 2; ++r) *reinterpret_cast<float2 *>(&sm.ypart[rb][g + 8 * r][j * 8 + 2 * tig]) = make_float2(y[j][2 * r], y[j][2 * r + 1]);
+    }
+    if (warp == SCAN_WARP && more) scan_chunk(dnext, stage ^ 1);
+    __syncthreads();   // weighted x and partial rows are complete; nobody reads the old state any more
+    if (!half) {
+#pragma unroll
+      for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = tr + 8 * r, c = j * 8 + 2 * tig;
+          if (t0 + t >= len || col0 + c >= p.P) continue;
+          const float2 o = *reinterpret_cast<const float2 *>(&sm.ypart[rb][g + 8 * r][c]);
+          const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[stage][t][c]);
+          *reinterpret_cast<float2 *>(p.y + (size_t)(row0 + t0 + t) * p.inner + (size_t)h * p.P + col0 + c) =
+              make_float2(fmaf(D, __low2float(x2), y[j][2 * r] + o.x), fmaf(D, __high2float(x2), y[j][2 * r + 1] + o.y));
+        }
+    }
+    // ---- state update: B^T [state rows x tokens] times the weighted x
+    const float keep = sm.keep[stage];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < NJ; ++j)
+#pragma unroll
         for (int e = 0; e < 4; ++e) S[i][j][e] *= keep;
-    const uint32_t wh_lane = smem_addr(&sm.Wh[lane & 15][(lane >> 4) * 8]), wl_lane = smem_addr(&sm.Wl[lane & 15][(lane >> 4) * 8]);
+    const uint32_t wh_lane = smem_addr(&sm.Wh[lane & 15][sj0 * 8 + (lane >> 4) * 8]), wl_lane = smem_addr(&sm.Wl[lane & 15][sj0 * 8 + (lane >> 4) * 8]);
 #pragma unroll
     for (int k2 = 0; k2 < CHUNK / 16; ++k2) {
-      uint32_t wh[CP / 8][2], wl[CP / 8][2];
+      uint32_t wh[NJ][2], wl[NJ][2];
 #pragma unroll
-      for (int j = 0; j < CP / 8; j += 2) {
-        ldsm4t(wh_lane + (uint32_t)(k2 * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, wh[j][0], wh[j][1], wh[j + 1][0], wh[j + 1][1]);
-        ldsm4t(wl_lane + (uint32_t)(k2 * 16 * ChunkSmem<NP>::XLD + j * 8) * 2u, wl[j][0], wl[j][1], wl[j + 1][0], wl[j + 1][1]);
+      for (int j = 0; j < NJ; j += 2) {
+        ldsm4t(wh_lane + (uint32_t)(k2 * 16 * XLD + j * 8) * 2u, wh[j][0], wh[j][1], wh[j + 1][0], wh[j + 1][1]);
+        ldsm4t(wl_lane + (uint32_t)(k2 * 16 * XLD + j * 8) * 2u, wl[j][0], wl[j][1], wl[j + 1][0], wl[j + 1][1]);
       }
 #pragma unroll
       for (int i = 0; i < MT; ++i) {
         // A fragment (rows = state, k = tokens) from the token-major tile: matrices (tokens 0-7 | 8-15) x (state 0-7 | 8-15), transposed
         uint32_t a0, a1, a2, a3;
-        ldsm4t(smem_addr(&sm.B[stage][k2 * 16 + (lane & 7) + (lane >> 4) * 8][warp * (NP / 4) + i * 16 + ((lane >> 3) & 1) * 8]), a0, a1, a2, a3);
+        ldsm4t(smem_addr(&sm.B[stage][k2 * 16 + (lane & 7) + (lane >> 4) * 8][srow - g + i * 16 + ((lane >> 3) & 1) * 8]), a0, a1, a2, a3);
 #pragma unroll
-        for (int j = 0; j < CP / 8; ++j) {
+        for (int j = 0; j < NJ; ++j) {
           mma16816_bf16(S[i][j], a0, a1, a2, a3, wh[j][0], wh[j][1]);
           mma16816_bf16(S[i][j], a0, a1, a2, a3, wl[j][0], wl[j][1]);
         }
@@ -321,10 +436,10 @@ template <int NP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_chunk_ker
 #pragma unroll
   for (int i = 0; i < MT; ++i)
 #pragma unroll
-    for (int j = 0; j < CP / 8; ++j)
+    for (int j = 0; j < NJ; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + j * 8 + 2 * tig + (e & 1);
+        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + (sj0 + j) * 8 + 2 * tig + (e & 1);
         if (n < p.N && c < p.P) gS[(size_t)n * p.P + c] = S[i][j][e];
       }
 }
@@ -343,6 +458,22 @@ template <typename T, int VEC> __global__ void __launch_bounds__(STEP_THREADS) s
   float *gS = p.state + ((size_t)slot * p.heads + h) * p.N * p.P;
   const T *zx = reinterpret_cast<const T *>(p.zx) + (size_t)t * p.zx_ld;
   const T *ring = reinterpret_cast<const T *>(p.ring) + (size_t)slot * p.taps * p.C;
+  constexpr int U = 8;                    // state rows in flight per thread
+  float v[U][VEC];
+  auto load_rows = [&](int n0, int q0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int n = n0 + u * ng;
+      if (n < p.N && pos > 0) {
+        if constexpr (VEC == 4) *reinterpret_cast<float4 *>(v[u]) = __ldcs(reinterpret_cast<const float4 *>(gS + (size_t)n * p.P + q0 * 4));
+        else v[u][0] = gS[(size_t)n * p.P + q0];
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v[u][j] = 0.f;
+      }
+    }
+  };
+  if (ngrp < ng && q < pq) load_rows(ngrp, q);   // on their way while the convolution is computed
   for (int i = tid; i < p.P + 2 * p.N; i += STEP_THREADS) {
     const int c = i < p.P ? h * p.P + i : (i < p.P + p.N ? p.inner + g * p.N + i - p.P : p.inner + (p.groups + g) * p.N + i - p.P - p.N);
     float a = p.conv_b[c];
@@ -362,20 +493,8 @@ template <typename T, int VEC> __global__ void __launch_bounds__(STEP_THREADS) s
     float y[VEC], dx[VEC];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) { y[j] = 0.f; dx[j] = dt * x[q0 * VEC + j]; }
-    constexpr int U = 4;
     for (int n0 = ngrp; n0 < p.N; n0 += U * ng) {
-      float v[U][VEC];
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const int n = n0 + u * ng;
-        if (n < p.N && pos > 0) {
-          if constexpr (VEC == 4) *reinterpret_cast<float4 *>(v[u]) = *reinterpret_cast<const float4 *>(gS + (size_t)n * p.P + q0 * 4);
-          else v[u][0] = gS[(size_t)n * p.P + q0];
-        } else {
-#pragma unroll
-          for (int j = 0; j < VEC; ++j) v[u][j] = 0.f;
-        }
-      }
+      if (n0 != ngrp || q0 != q) load_rows(n0, q0);
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const int n = n0 + u * ng;
@@ -413,10 +532,12 @@ template <typename T, int VEC> __global__ void ssm_norm_kernel(const Params p) {
     if (warp >= wpg * gstep) break;
     float ss = 0.f;
     for (int i = ((warp % wpg) * 32 + lane) * VEC; i < len; i += wpg * 32 * VEC) {
-      float v[VEC];
+      float v[VEC], z[VEC];
+      load_vec<VEC>(y + g * len + i, v);
+      load_vec<VEC>(zx + g * len + i, z);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
-        v[j] = y[g * len + i + j] * silu_f(to_f(zx[g * len + i + j]));
+        v[j] *= silu_f(z[j]);
         ss += v[j] * v[j];
       }
       store_vec<VEC>(gbuf + g * len + i, v);
@@ -426,7 +547,13 @@ template <typename T, int VEC> __global__ void ssm_norm_kernel(const Params p) {
   }
   if (t >= t1 - p.taps) {   // the last `taps` raw convolution inputs of the sequence stay in its ring
     T *ring = reinterpret_cast<T *>(p.ring) + ((size_t)p.slot[s] * p.taps + pos % p.taps) * p.C;
-    for (int c = tid; c < p.C; c += blockDim.x) ring[c] = zx[p.inner + c];
+    if constexpr (VEC == 4) {
+      typedef typename std::conditional<sizeof(T) == 4, uint4, uint2>::type V;
+#pragma unroll 4
+      for (int c = tid; c < p.C / 4; c += blockDim.x) reinterpret_cast<V *>(ring)[c] = reinterpret_cast<const V *>(zx + p.inner)[c];
+    } else {
+      for (int c = tid; c < p.C; c += blockDim.x) ring[c] = zx[p.inner + c];
+    }
   }
   __syncthreads();
   for (int g = tid; g < p.norm_groups; g += blockDim.x) {
@@ -438,9 +565,11 @@ template <typename T, int VEC> __global__ void ssm_norm_kernel(const Params p) {
   T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld;
   for (int i = tid * VEC; i < p.inner; i += blockDim.x * VEC) {
     const float inv = sums[i / len * wpg];
-    float v[VEC];
+    float v[VEC], w[VEC];
+    load_vec<VEC>(gbuf + i, v);
+    load_vec<VEC>(p.norm_w + i, w);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) v[j] = gbuf[i + j] * inv * p.norm_w[i + j];
+    for (int j = 0; j < VEC; ++j) v[j] *= inv * w[j];
     store_vec<VEC>(out + i, v);
   }
   for (int i = p.inner + tid; i < p.out_ld; i += blockDim.x) out[i] = from_f<T>(0.f);   // k padding of the output product
@@ -467,7 +596,17 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
     else ssm_step_kernel<T, 1><<<grid, STEP_THREADS, smem, st>>>(p);
     PT_LAUNCH_CHECK("pt_ssm");
   } else {
-    ssm_conv_kernel<T><<<dim3(ceil_div(p.C + p.heads, 256), p.n_tok), 256, 0, st>>>(p);
+    if (!plain && sizeof(T) == 2 && p.taps <= 4 && p.C % 8 == 0 && p.inner % 8 == 0 && p.zx_ld % 8 == 0 && al(p.zx, 16) && al(p.xbc, 16) && al(p.ring, 16)) {
+      const dim3 grid(ceil_div(p.C / 8, CONV_THREADS) + 1, ceil_div(p.n_tok, CONV_TOKENS));
+      switch (p.taps) {
+        case 1: ssm_conv8_kernel<1><<<grid, CONV_THREADS, 0, st>>>(p); break;
+        case 2: ssm_conv8_kernel<2><<<grid, CONV_THREADS, 0, st>>>(p); break;
+        case 3: ssm_conv8_kernel<3><<<grid, CONV_THREADS, 0, st>>>(p); break;
+        default: ssm_conv8_kernel<4><<<grid, CONV_THREADS, 0, st>>>(p); break;
+      }
+    } else {
+      ssm_conv_kernel<T><<<dim3(ceil_div(p.C + p.heads, 256), p.n_tok), 256, 0, st>>>(p);
+    }
     PT_LAUNCH_CHECK("pt_ssm");
     // the chunked form: bf16, rows that are whole 16-byte units, state of at most 256
     if (!plain && sizeof(T) == 2 && p.N <= 256 && p.N % 8 == 0 && p.P % 8 == 0 && al(p.xbc, 16) && al(p.y, 8)) {
@@ -482,8 +621,10 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
     }
   }
   const int len = p.inner / p.norm_groups;
-  const bool v4 = len % 4 == 0 && al(p.out, 4 * sizeof(T)) && p.out_ld % 4 == 0;
-  const int threads = 256;
+  const bool v4 = len % 4 == 0 && p.C % 4 == 0 && p.zx_ld % 4 == 0 && p.out_ld % 4 == 0 && al(p.out, 4 * sizeof(T)) && al(p.zx, 4 * sizeof(T)) &&
+                  al(p.ring, 4 * sizeof(T)) && al(p.y, 16) && al(p.norm_w, 16);
+  // few rows: as many threads per row as it has work for (the launch is one chain of latencies); many rows: more rows per SM
+  const int threads = p.n_tok <= 2 * sm_count() ? std::min(1024, std::max(128, ceil_div(p.inner / (v4 ? 4 : 1), 32) * 32)) : 256;
   const size_t smem = ((size_t)(p.inner + 3) / 4 * 4 + (size_t)std::max(p.norm_groups, threads / 32)) * sizeof(float);
   PT_REQUIRE(smem <= 200 * 1024, "pt_ssm: inner width %d needs %zu bytes of shared memory", p.inner, smem);
   if (smem > 48 * 1024) {
