@@ -136,6 +136,18 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
   asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
 
+__device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&v)[32]) {
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
+               "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+               : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]), "=r"(v[10]),
+                 "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]), "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]),
+                 "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]),
+                 "=r"(v[31])
+               : "r"(taddr)
+               : "memory");
+  asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+}
+
 // Shared-memory matrix descriptor of a K-major operand tile stored as rows of 128 bytes with the 128-byte swizzle (the layout
 // TMA writes with CU_TENSOR_MAP_SWIZZLE_128B and the transform warps reproduce): 8-row groups are 1024 bytes apart.
 __device__ __forceinline__ uint64_t smem_desc_sw128(uint32_t addr) {
@@ -190,9 +202,9 @@ template <bool BF16> __device__ __forceinline__ void store_out(const GemmParams 
 // Epilogue of the warps that own the tile's rows (tensor-memory lane quarter warp % 4): `part` of `parts` warps share a quarter
 // and take alternate 16-column chunks.
 template <bool BF16>
-__device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int q, int lane, int part, int parts, int n0, int m0, int ks) {
+__device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int q, int lane, int part, int parts, int n0, int m0, int ks, int c_first = 0) {
   const int n = n0 + q * 32 + lane;
-  for (int c0 = part * 16; c0 < p.mb; c0 += 16 * parts) {
+  for (int c0 = c_first + part * 16; c0 < p.mb; c0 += 16 * parts) {
     uint32_t v[16];
     float sum[16];
     tmem_ld16(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, v);
@@ -212,6 +224,55 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
       }
     }
   }
+}
+
+// The BF16 kernel's epilogue of a whole 32-column group without k-slices: uniform branches outside the element loop, pointer
+// increments instead of index arithmetic (the general form above costs as much as the products of a 2048-deep tile).  bf16 output:
+// neighbouring lanes (n, n + 1) trade values of two columns, so every store writes 4 bytes per lane.
+template <bool F32, bool RELU2>
+__device__ __forceinline__ void epilogue_rows32(const GemmParams &p, const uint32_t (&v)[32], int n, int m, int lane) {
+  auto fin = [&](uint32_t x) {
+    float y = __uint_as_float(x) * p.out_scale;
+    if (RELU2) { y = fmaxf(y, 0.f); y *= y; }
+    return y;
+  };
+  if (F32) {
+    float *o = reinterpret_cast<float *>(p.out) + (size_t)m * p.out_ld + n;
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+      *o = fin(v[j]);
+      o += p.out_ld;
+    }
+  } else {
+    const int odd = lane & 1;
+    __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(p.out) + (size_t)(m + odd) * p.out_ld + (n - odd);
+#pragma unroll
+    for (int j = 0; j < 32; j += 2) {
+      const float a = fin(v[j]), b = fin(v[j + 1]);
+      const float t = __shfl_xor_sync(0xffffffffu, odd ? a : b, 1);     // even lane: column j of n + 1; odd lane: column j + 1 of n - 1
+      *reinterpret_cast<__nv_bfloat162 *>(o) = odd ? __floats2bfloat162_rn(t, b) : __floats2bfloat162_rn(a, t);
+      o += 2 * (size_t)p.out_ld;
+    }
+  }
+}
+__device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem, int q, int lane, int n0, int m0, int ks) {
+  const int n = n0 + q * 32 + lane;
+  const bool f32 = p.out_dt == PT_DT_F32;
+  // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16 (warp-uniform conditions)
+  const bool fast = p.ksplit == 1 && n0 + q * 32 + 32 <= p.N && (f32 || (p.out_ld % 2 == 0 && ((uintptr_t)p.out & 3) == 0));
+  const int whole = fast ? min(p.mb, p.M - m0) & ~31 : 0;
+  for (int c0 = 0; c0 < whole; c0 += 32) {
+    uint32_t v[32];
+    tmem_ld32(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, v);
+    if (f32) {
+      if (p.epilogue == PT_EPI_RELU2) epilogue_rows32<true, true>(p, v, n, m0 + c0, lane);
+      else epilogue_rows32<true, false>(p, v, n, m0 + c0, lane);
+    } else {
+      if (p.epilogue == PT_EPI_RELU2) epilogue_rows32<false, true>(p, v, n, m0 + c0, lane);
+      else epilogue_rows32<false, false>(p, v, n, m0 + c0, lane);
+    }
+  }
+  if (whole < p.mb) epilogue<true>(p, tmem, q, lane, 0, 1, n0, m0, ks, whole);
 }
 
 // k-slices of this tile meet: the last CTA to arrive sums them in slice order.
@@ -331,7 +392,10 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
   } else {
     if (!mbar_wait(sa(&ctl.accum), 0, &ctl.abort)) give_up(ctl, p.error_flag, 24);
     fence_after();
-    if (!ctl.abort && n_it > 0) epilogue<BF16>(p, tmem, warp & 3, lane, 0, 1, n0, m0, ks);
+    if (!ctl.abort && n_it > 0) {
+      if constexpr (BF16) epilogue_bf16(p, tmem, warp & 3, lane, n0, m0, ks);
+      else epilogue<false>(p, tmem, warp & 3, lane, 0, 1, n0, m0, ks);
+    }
     fence_before();
   }
   if (p.ksplit > 1) reduce_slices<BF16>(p, ctl, n0, m0, THREADS_F8);
@@ -688,7 +752,9 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
 #ifndef PT_TC_BUDGET_SMALL_KB
 #define PT_TC_BUDGET_SMALL_KB 100
 #endif
-  const bool small = p.mb <= 64;
+  // BF16 also with large tiles when there are more of them than SMs: the epilogue of one CTA then hides behind the products of the
+  // other (two accumulators of 256 columns fill the tensor memory).
+  const bool small = p.mb <= 64 || (bf16 && (long long)n_tiles * m_tiles * p.ksplit > sm_count());
   const uint32_t budget = (small ? PT_TC_BUDGET_SMALL_KB : 200) * 1024u;
   size_t smem;
   if (int4) {
@@ -700,6 +766,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
     p.stages = (int)std::min<uint32_t>(8, budget / stage_bytes);
     PT_REQUIRE(p.stages >= 2, "pt_gemm: tile does not fit shared memory");
     smem = (size_t)p.stages * stage_bytes + 1024;
+    if (bf16 && p.mb > 64) smem = std::max<size_t>(smem, 80 * 1024);   // never more CTAs on an SM than its tensor memory holds accumulators for
   }
 
   CUtensorMap map_w, map_x;

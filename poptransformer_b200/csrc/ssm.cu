@@ -77,34 +77,36 @@ template <int TAPS> __global__ void __launch_bounds__(CONV_THREADS) ssm_conv8_ke
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     b[j] = p.conv_b[c + j];
+    if constexpr (TAPS == 4) load_vec<4>(p.conv_w + (size_t)(c + j) * 4, w[j]);
+    else {
 #pragma unroll
-    for (int k = 0; k < TAPS; ++k) w[j][k] = p.conv_w[(size_t)(c + j) * TAPS + k];
+      for (int k = 0; k < TAPS; ++k) w[j][k] = p.conv_w[(size_t)(c + j) * TAPS + k];
+    }
   }
-  int seq = -1;
-#pragma unroll 4
-  for (int t = ta; t < tb; ++t) {
-    const int s = p.tok_seq[t];
-    if (s != seq) {                       // first token of this thread or of a sequence: the window as it stands before it
-      seq = s;
-      const int t0 = p.cu[s], pos = p.start[s] + t - t0;
-      const T *ring = reinterpret_cast<const T *>(p.ring) + (size_t)p.slot[s] * TAPS * p.C;
+  // the window in front of token t of sequence s
+  auto fill_window = [&](int t, int s) {
+    const int t0 = p.cu[s], pos = p.start[s] + t - t0;
+    const T *ring = reinterpret_cast<const T *>(p.ring) + (size_t)p.slot[s] * TAPS * p.C;
 #pragma unroll
-      for (int k = 1; k < TAPS; ++k) {
-        if (k > pos) {
+    for (int k = 1; k < TAPS; ++k) {
+      if (k > pos) {
 #pragma unroll
-          for (int j = 0; j < 8; ++j) x[k - 1][j] = 0.f;
-        } else if (t - k >= t0) {
-          load_vec<8>(zx + (size_t)(t - k) * p.zx_ld + p.inner + c, x[k - 1]);
-        } else {
-          load_vec<8>(ring + (size_t)((pos - k) % TAPS) * p.C + c, x[k - 1]);
-        }
+        for (int j = 0; j < 8; ++j) x[k - 1][j] = 0.f;
+      } else if (t - k >= t0) {
+        load_vec<8>(zx + (size_t)(t - k) * p.zx_ld + p.inner + c, x[k - 1]);
+      } else {
+        load_vec<8>(ring + (size_t)((pos - k) % TAPS) * p.C + c, x[k - 1]);
       }
     }
+  };
+  auto one_token = [&](int t, const uint4 &raw) {
 #pragma unroll
     for (int k = TAPS - 1; k > 0; --k)
 #pragma unroll
       for (int j = 0; j < 8; ++j) x[k][j] = x[k - 1][j];
-    load_vec<8>(zx + (size_t)t * p.zx_ld + p.inner + c, x[0]);
+    const __nv_bfloat162 *r = reinterpret_cast<const __nv_bfloat162 *>(&raw);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { x[0][2 * j] = __low2float(r[j]); x[0][2 * j + 1] = __high2float(r[j]); }
     __nv_bfloat162 o[4];
     float y[8];
 #pragma unroll
@@ -112,11 +114,32 @@ template <int TAPS> __global__ void __launch_bounds__(CONV_THREADS) ssm_conv8_ke
       float a = b[j];
 #pragma unroll
       for (int k = 0; k < TAPS; ++k) a = fmaf(w[j][k], x[TAPS - 1 - k][j], a);
-      y[j] = silu_f(a);
+      y[j] = __fdividef(a, 1.0f + __expf(-a));   // (rounded to bf16 below; for a very negative the quotient is 0 either way)
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) o[j] = __floats2bfloat162_rn(y[2 * j], y[2 * j + 1]);
     *reinterpret_cast<uint4 *>(reinterpret_cast<T *>(p.xbc) + (size_t)t * p.C + c) = *reinterpret_cast<const uint4 *>(o);
+  };
+  auto src = [&](int t) { return reinterpret_cast<const uint4 *>(zx + (size_t)t * p.zx_ld + p.inner + c); };
+  int seq = p.tok_seq[ta];
+  fill_window(ta, seq);
+  if (seq == p.tok_seq[tb - 1]) {         // all tokens of one sequence: four loads in flight
+    for (int t = ta; t < tb; t += 4) {
+      uint4 raw[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) raw[u] = t + u < tb ? *src(t + u) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (t + u < tb) one_token(t + u, raw[u]);
+    }
+    return;
+  }
+  for (int t = ta; t < tb; ++t) {
+    if (p.tok_seq[t] != seq) {
+      seq = p.tok_seq[t];
+      fill_window(t, seq);
+    }
+    one_token(t, *src(t));
   }
 }
 
@@ -596,7 +619,7 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
     else ssm_step_kernel<T, 1><<<grid, STEP_THREADS, smem, st>>>(p);
     PT_LAUNCH_CHECK("pt_ssm");
   } else {
-    if (!plain && sizeof(T) == 2 && p.taps <= 4 && p.C % 8 == 0 && p.inner % 8 == 0 && p.zx_ld % 8 == 0 && al(p.zx, 16) && al(p.xbc, 16) && al(p.ring, 16)) {
+    if (!plain && sizeof(T) == 2 && p.taps <= 4 && p.C % 8 == 0 && p.inner % 8 == 0 && p.zx_ld % 8 == 0 && al(p.zx, 16) && al(p.xbc, 16) && al(p.ring, 16) && al(p.conv_w, 16)) {
       const dim3 grid(ceil_div(p.C / 8, CONV_THREADS) + 1, ceil_div(p.n_tok, CONV_TOKENS));
       switch (p.taps) {
         case 1: ssm_conv8_kernel<1><<<grid, CONV_THREADS, 0, st>>>(p); break;
