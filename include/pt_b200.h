@@ -151,7 +151,7 @@ int pt_linear_static_scratch(const pt_linear_args *args, void *stream);
  *   PT_W_INT4: x = fp16 [m, k_in], w = pt_gemm_repack of the reference's int8 [n_out, k_in/2] rows (w_tiled = 1), scales fp16
  *              [n_out, k_in/group]; every weight becomes fp16(q) * scale with one rounding (Int4ToHalf,
  *              custom_ops/int4_to_half_codelets.cpp:18-38) on its way to the tensor core.
- *   PT_W_BF16: x = bf16 [m, k_in], w = bf16 [n_out, k_in], row-major or tiled by pt_gemm_repack; out = bf16 or fp32 (out_dtype),
+ *   PT_W_BF16: x = bf16 [m, k_in], w = pt_gemm_repack of bf16 [n_out, k_in] (w_tiled = 1); out = bf16 or fp32 (out_dtype),
  *              epilogue PT_EPI_STORE or PT_EPI_RELU2 on alpha * (x . w^T).  k_in a multiple of 64.
  * FP8 and INT4: k_in must be a multiple of 128.  Accumulation is fp32.  k-slices (ksplit, 0 = chosen by the library) are summed in a fixed
  * order; with more than one slice a workspace is needed (zeroed once by the caller; every launch leaves its counters at zero). */
@@ -532,8 +532,10 @@ typedef struct pt_ssm_args {
   void *out;                              /* [n_tok, out_ld], columns inner .. out_ld - 1 are zeroed */
   int out_ld;
   int plain;              /* 1: the kernels for any sizes, whatever the shape        */
-  int32_t *error_flag;
+  void *workspace;        /* bf16 prompts: pt_ssm_workspace_bytes, 16-byte aligned; without it they run token by token */
+  size_t workspace_bytes;
 } pt_ssm_args;
+size_t pt_ssm_workspace_bytes(int n_tok, int n_seq, int heads, int vdim, int state_dim);
 int pt_ssm(const pt_ssm_args *args, void *stream);
 
 #ifdef __cplusplus

@@ -77,7 +77,7 @@ class SsmArgs(ctypes.Structure):
     _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "heads", "vdim", "state_dim", "groups", "taps", "norm_groups")] + \
                [("eps", c_float), ("zx", c_void_p), ("zx_ld", c_int)] + \
                [(n, c_void_p) for n in ("conv_w", "conv_b", "dt_bias", "A_log", "D", "norm_w", "ring", "state", "xbc", "dt", "y", "out")] + \
-               [("out_ld", c_int), ("plain", c_int), ("error_flag", c_void_p)]
+               [("out_ld", c_int), ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t)]
 
 
 class LlamaLayer(ctypes.Structure):
@@ -113,6 +113,7 @@ SIGNATURES = {
     "pt_hyper": (c_int, [ctypes.POINTER(HyperArgs), c_void_p]),
     "pt_window_attn_workspace_bytes": (c_size_t, [c_int] * 7),
     "pt_window_attn": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),
+    "pt_ssm_workspace_bytes": (c_size_t, [c_int] * 5),
     "pt_ssm": (c_int, [ctypes.POINTER(SsmArgs), c_void_p]),
     "pt_norm_ce": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p]),
     "pt_rms_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p]),

@@ -291,6 +291,28 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
     __threadfence();
     // every thread sums the slices of one output element at a time, all slices' loads in flight together (at most 8 per batch)
     const int rows = min(p.mb, p.M - m0);
+    if constexpr (BF16) {
+      if (p.N % 4 == 0) {   // four outputs per thread and step: a quarter of the trips to L2
+        for (int i = tid; i < rows * (BM / 4); i += threads) {
+          const int m = m0 + i / (BM / 4), n = n0 + (i % (BM / 4)) * 4;
+          if (n >= p.N) continue;
+          float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+          for (int s0 = 0; s0 < p.ksplit; s0 += 4) {
+            float4 part[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+              part[j] = (s0 + j < p.ksplit) ? __ldcg(reinterpret_cast<const float4 *>(p.partial + ((size_t)(s0 + j) * p.M + m) * p.N + n)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) { acc.x += part[j].x; acc.y += part[j].y; acc.z += part[j].z; acc.w += part[j].w; }
+          }
+          store_out<true>(p, acc.x, m, n);
+          store_out<true>(p, acc.y, m, n + 1);
+          store_out<true>(p, acc.z, m, n + 2);
+          store_out<true>(p, acc.w, m, n + 3);
+        }
+        return;
+      }
+    }
     for (int i = tid; i < rows * BM; i += threads) {
       const int m = m0 + i / BM, n = n0 + (i % BM);
       if (n >= p.N) continue;
@@ -695,7 +717,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   }
   PT_REQUIRE(a->epilogue != PT_EPI_RESIDUAL || a->residual, "pt_gemm: residual epilogue needs residual");
   PT_REQUIRE(a->epilogue != PT_EPI_BIAS || a->bias, "pt_gemm: bias epilogue needs bias");
-  PT_REQUIRE(!int4 || a->w_tiled, "pt_gemm: INT4 weights must be tiled with pt_gemm_repack");
+  PT_REQUIRE(!(int4 || bf16) || a->w_tiled, "pt_gemm: INT4 and BF16 weights must be tiled with pt_gemm_repack");
   if (int4)
     PT_REQUIRE(a->scales && a->group >= 128 && a->group % 128 == 0 && a->k_in % a->group == 0,
                "pt_gemm: INT4 needs scales and a group (%d) that is a multiple of 128 dividing k_in=%d", a->group, a->k_in);
@@ -707,8 +729,11 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   p.w_tiled = a->w_tiled ? 1 : 0;
   p.w = (const unsigned char *)a->w;
   p.mb = std::min(256, ceil_div(a->m, 16) * 16);
-  const int m_tiles = ceil_div(a->m, p.mb);
   const int n_tiles = ceil_div(a->n_out, tc::BM);
+  // BF16: fewer activation rows per tile before k-slices (whose sums take a detour over HBM) when there are not enough tiles
+  if (bf16)
+    while (p.mb > 64 && n_tiles * ceil_div(a->m, p.mb) * 4 < sm_count() * 3) p.mb = ceil_div(p.mb, 32) * 16;
+  const int m_tiles = ceil_div(a->m, p.mb);
   p.n_kb = (int4 || bf16) ? a->k_in / 64 : a->k_in / 128;
   // k-slices: fill the GPU when there are few tiles, but keep at least PT_TC_MIN_KB k-blocks per CTA
 #ifndef PT_TC_MIN_KB
@@ -774,8 +799,6 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   if (int4) {
     if (int rc = tc::make_map(&map_x, a->x, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (uint64_t)a->k_in, (uint64_t)a->m, 64, (uint32_t)p.mb, CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
   } else if (bf16) {
-    if (!p.w_tiled)
-      if (int rc = tc::make_map(&map_w, a->w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->k_in, (uint64_t)a->n_out, 64, tc::BM, CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
     if (int rc = tc::make_map(&map_x, a->x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->k_in, (uint64_t)a->m, 64, (uint32_t)p.mb, CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
   } else {
     if (!p.w_tiled)

@@ -11,7 +11,7 @@
 //
 //   ssm_conv_kernel    prompts: convolution + silu of all tokens, step sizes
 //   ssm_scan_kernel    prompts, any sizes and types: the recurrence token by token, state in shared memory
-//   ssm_chunk_kernel   bf16 prompts: the same recurrence 64 tokens at a time on the tensor cores
+//   ssm_chunk_* , ssm_carry_kernel   bf16 prompts: the same recurrence 64 tokens at a time on the tensor cores
 //   ssm_step_kernel    one token per sequence: convolution, step size, state update and readout in one launch
 //   ssm_norm_kernel    gate, group norm, and the ring update
 #include <type_traits>
@@ -30,6 +30,8 @@ struct Params {
   const float *conv_w, *conv_b, *dt_bias, *A_log, *D, *norm_w;
   void *ring, *xbc, *out;
   float *state, *dt, *y;
+  float *chunk_state;                // [n_tok / 64 + n_seq][heads][N][P]
+  struct Decays *chunk_decays;       // [n_tok / 64 + n_seq][heads]
 };
 
 // ------------------------------------------------------------------------------------------ convolution of a prompt
@@ -189,13 +191,16 @@ template <typename T> __global__ void __launch_bounds__(SCAN_WARPS * 32) ssm_sca
 // With c_t = sum_{r <= t} log decay_r inside a chunk and S the state before it, the recurrence is four matrix products:
 //     y_t = exp(c_t) C_t S  +  sum_{s <= t} (C_t . B_s) exp(c_t - c_s) dt_s x_s  +  D x_t
 //     S  <- exp(c_last) S  +  sum_s B_s (exp(c_last - c_s) dt_s x_s)^T
-// Block: 32 columns of one head's state, one sequence; it walks the chunks in order with the state in fp32 accumulators.  Operands
-// that are not already bf16 (the state, the decayed products, the weighted x) enter the tensor cores as hi + lo pairs.  c is kept
-// as a pair of floats, so differences of neighbours stay exact however far the sum has run.
-// Eight warps: two share 16 tokens of the output, each with half of the state rows (first product) and every other 16 tokens s
-// (second product); all eight share the state rows of the update.  One warp scans the next chunk's decays meanwhile.
-// NP: state size rounded up to 64, 128 or 256 (padding is zero).
-constexpr int CHUNK = 64, CP = 32, CHUNK_THREADS = 256;
+// Four launches, so that all chunks of all sequences work at once and only an elementwise pass runs along the sequence:
+//   ssm_decay_kernel         the decay factors of every chunk and head
+//   ssm_chunk_state_kernel   the sum of the second line, per chunk and head
+//   ssm_carry_kernel         the second line along the chunks: leaves the state BEFORE every chunk in place of its sum
+//   ssm_chunk_out_kernel     the first line, per chunk and head
+// Chunk ci of sequence s lives in slot cu[s] / 64 + s + ci of the scratch (distinct, below n_tok / 64 + n_seq).  Operands that are
+// not already bf16 (the state, the decayed products, the weighted x) enter the tensor cores as hi + lo pairs.  c is kept as a pair
+// of floats, so differences of neighbours stay exact however far the sum has run.
+// NP: state size rounded up to 64, 128 or 256, CP: columns of a head per block (padding is zero).
+constexpr int CHUNK = 64, CHUNK_THREADS = 256;
 __device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
 }
@@ -205,266 +210,324 @@ __device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t &r0, uint32_t &r1,
 __device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
 }
-template <int NP> struct ChunkSmem {
-  static constexpr int BLD = NP + 8, XLD = CP + 8;
-  __nv_bfloat16 B[2][CHUNK][BLD], C[2][CHUNK][BLD], X[2][CHUNK][XLD];
-  __nv_bfloat16 Sh[NP][XLD], Sl[NP][XLD];         // state before the chunk, hi and lo
-  __nv_bfloat16 Wh[CHUNK][XLD], Wl[CHUNK][XLD];   // exp(c_last - c_s) dt_s x_s
-  float ypart[4][16][CP + 4];                     // the second warp's share of the output rows
-  float c_hi[2][CHUNK], c_lo[2][CHUNK], dt[2][CHUNK], ec[2][CHUNK], w[2][CHUNK], keep[2];
-};
-
-template <int NP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_chunk_kernel(const Params p) {
-  typedef __nv_bfloat16 T;
-  constexpr int MT = NP > 128 ? NP / 128 : 1;       // 16-row tiles of the state per warp ...
-  constexpr int NJ = NP == 64 ? 2 : 4;              // ... and 8-column tiles (64 rows are four row tiles: two warps share each)
-  constexpr int XLD = ChunkSmem<NP>::XLD;
-  extern __shared__ __align__(16) unsigned char smraw[];
-  ChunkSmem<NP> &sm = *reinterpret_cast<ChunkSmem<NP> *>(smraw);
-  const int s = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * CP;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
-  const int grp = h / (p.heads / p.groups);
-  const int row0 = p.cu[s], len = p.cu[s + 1] - row0;
-  const T *xbc = reinterpret_cast<const T *>(p.xbc) + (size_t)row0 * p.C;
-  const float a = -expf(p.A_log[h]), D = p.D[h];
-  float *gS = p.state + ((size_t)p.slot[s] * p.heads + h) * p.N * p.P;
-
-  auto load_chunk = [&](int t0, int stage) {
-    for (int e = tid; e < CHUNK * (NP / 8); e += CHUNK_THREADS) {
-      const int r = e / (NP / 8), c = (e % (NP / 8)) * 8;
-      const bool in = t0 + r < len && c < p.N;
-      const T *row = xbc + (in ? (size_t)(t0 + r) * p.C + p.inner + grp * p.N + c : 0);
-      cp16(&sm.B[stage][r][c], row, in);
-      cp16(&sm.C[stage][r][c], row + (in ? p.groups * p.N : 0), in);
-    }
-    for (int e = tid; e < CHUNK * (CP / 8); e += CHUNK_THREADS) {
-      const int r = e / (CP / 8), c = (e % (CP / 8)) * 8;
-      const bool in = t0 + r < len && col0 + c < p.P;
-      cp16(&sm.X[stage][r][c], xbc + (in ? (size_t)(t0 + r) * p.C + (size_t)h * p.P + col0 + c : 0), in);
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  // Step sizes of the chunk at t0 (two per lane; zero beyond the sequence: decay 1, no contribution) ...
-  auto load_dt = [&](int t0, float (&d)[2]) {
-#pragma unroll
-    for (int k = 0; k < 2; ++k) {
-      const int r = t0 + 2 * lane + k;
-      d[k] = r < len ? p.dt[(size_t)(row0 + r) * p.heads + h] : 0.f;
-    }
-  };
-  // ... and what follows from them, by one warp.
-  auto scan_chunk = [&](const float (&d)[2], int stage) {
-    const double l1 = (double)(a * d[1]);
-    double sum = (double)(a * d[0]) + l1;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const double v = __shfl_up_sync(0xffffffffu, sum, o);
-      if (lane >= o) sum += v;
-    }
-    const double last = __shfl_sync(0xffffffffu, sum, 31);
-    const double c[2] = {sum - l1, sum};
-#pragma unroll
-    for (int k = 0; k < 2; ++k) {
-      const int r = 2 * lane + k;
-      sm.c_hi[stage][r] = (float)c[k];
-      sm.c_lo[stage][r] = (float)(c[k] - (double)(float)c[k]);
-      sm.dt[stage][r] = d[k];
-      sm.ec[stage][r] = expf((float)c[k]);
-      sm.w[stage][r] = expf((float)(last - c[k])) * d[k];
-    }
-    if (lane == 0) sm.keep[stage] = expf((float)last);
-  };
-  load_chunk(0, 0);
-  constexpr int SCAN_WARP = 1;   // its output rows have the least work
-  float dnext[2];
-  if (warp == SCAN_WARP) {
-    load_dt(0, dnext);
-    scan_chunk(dnext, 0);
+__device__ __forceinline__ int chunk_slot(const Params &p, int s) { return p.cu[s] / CHUNK + s; }
+// Sequence and first token (within it) of a scratch slot; false for a slot that no chunk uses.
+__device__ __forceinline__ bool chunk_of_slot(const Params &p, int slot, int &s, int &t0) {
+  int lo = 0, hi = p.n_seq - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) / 2;
+    if (chunk_slot(p, mid) <= slot) lo = mid;
+    else hi = mid - 1;
   }
+  s = lo;
+  t0 = (slot - chunk_slot(p, lo)) * CHUNK;
+  return t0 < p.cu[lo + 1] - p.cu[lo];
+}
+struct __align__(16) Decays {
+  float c_hi[CHUNK], c_lo[CHUNK], dt[CHUNK], ec[CHUNK], w[CHUNK];   // ec = exp(c_t), w = exp(c_last - c_s) dt_s
+  float keep, pad[3];                                               // exp(c_last)
+};
+// One warp: step sizes of the chunk and what follows from them (tokens beyond the sequence: decay 1, no contribution).
+__device__ __forceinline__ void scan_decays(const Params &p, int row0, int valid, int h, Decays &d) {
+  const int lane = threadIdx.x & 31;
+  const float a = -expf(p.A_log[h]);
+  float dt[2];
+#pragma unroll
+  for (int k = 0; k < 2; ++k) dt[k] = 2 * lane + k < valid ? p.dt[(size_t)(row0 + 2 * lane + k) * p.heads + h] : 0.f;
+  const double l1 = (double)(a * dt[1]);
+  double sum = (double)(a * dt[0]) + l1;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const double v = __shfl_up_sync(0xffffffffu, sum, o);
+    if (lane >= o) sum += v;
+  }
+  const double last = __shfl_sync(0xffffffffu, sum, 31);
+  const double c[2] = {sum - l1, sum};
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int r = 2 * lane + k;
+    d.c_hi[r] = (float)c[k];
+    d.c_lo[r] = (float)(c[k] - (double)(float)c[k]);
+    d.dt[r] = dt[k];
+    d.ec[r] = expf((float)c[k]);
+    d.w[r] = expf((float)(last - c[k])) * dt[k];
+  }
+  if (lane == 0) d.keep = expf((float)last);
+}
+__global__ void ssm_decay_kernel(const Params p) {   // one warp per (chunk, head)
+  const int slot = blockIdx.y, h = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  int s, t0;
+  if (h >= p.heads || !chunk_of_slot(p, slot, s, t0)) return;
+  const int row0 = p.cu[s] + t0;
+  scan_decays(p, row0, min(CHUNK, p.cu[s + 1] - row0), h, p.chunk_decays[(size_t)slot * p.heads + h]);
+}
+__device__ __forceinline__ void load_decays(const Params &p, int slot, int h, Decays &d) {
+  const unsigned char *src = reinterpret_cast<const unsigned char *>(p.chunk_decays + (size_t)slot * p.heads + h);
+  for (int i = threadIdx.x; i < (int)(sizeof(Decays) / 16); i += blockDim.x) cp16(reinterpret_cast<unsigned char *>(&d) + i * 16, src + i * 16, true);
+}
 
-  // state accumulators; lane (g, tig) of tile (i, j): rows g and g + 8, columns 2 tig, + 1
+template <int NP, int CP> struct StateSmem {
+  __nv_bfloat16 B[CHUNK][NP + 8], X[CHUNK][CP + 8], Wh[CHUNK][CP + 8], Wl[CHUNK][CP + 8];
+  Decays d;
+};
+// Block: one chunk, one head, CP columns.  The warps share the 16-row tiles of the state (and the columns when there are fewer tiles).
+template <int NP, int CP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_chunk_state_kernel(const Params p) {
+  typedef __nv_bfloat16 T;
+  constexpr int XLD = CP + 8, MTILES = NP / 16, WPT = MTILES >= 8 ? 1 : 8 / MTILES;      // warps per row tile
+  constexpr int MT = MTILES >= 8 ? MTILES / 8 : 1, NJ = CP / 8 / WPT;
+  extern __shared__ __align__(16) unsigned char smraw[];
+  StateSmem<NP, CP> &sm = *reinterpret_cast<StateSmem<NP, CP> *>(smraw);
+  const int slot = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * CP;
+  int s, t0;
+  if (!chunk_of_slot(p, slot, s, t0)) return;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
+  const int grp = h / (p.heads / p.groups), row0 = p.cu[s] + t0, valid = min(CHUNK, p.cu[s + 1] - row0);
+  const T *xbc = reinterpret_cast<const T *>(p.xbc) + (size_t)row0 * p.C;
+  for (int e = tid; e < CHUNK * (NP / 8); e += CHUNK_THREADS) {
+    const int r = e / (NP / 8), c = (e % (NP / 8)) * 8;
+    const bool in = r < valid && c < p.N;
+    cp16(&sm.B[r][c], xbc + (in ? (size_t)r * p.C + p.inner + grp * p.N + c : 0), in);
+  }
+  for (int e = tid; e < CHUNK * (CP / 8); e += CHUNK_THREADS) {
+    const int r = e / (CP / 8), c = (e % (CP / 8)) * 8;
+    const bool in = r < valid && col0 + c < p.P;
+    cp16(&sm.X[r][c], xbc + (in ? (size_t)r * p.C + (size_t)h * p.P + col0 + c : 0), in);
+  }
+  load_decays(p, slot, h, sm.d);
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+#pragma unroll
+  for (int e = tid; e < CHUNK * (CP / 2); e += CHUNK_THREADS) {
+    const int r = e / (CP / 2), c = (e % (CP / 2)) * 2;
+    const float w = sm.d.w[r];
+    const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[r][c]);
+    uint32_t hi, lo;
+    split_bf2(w * __low2float(x2), w * __high2float(x2), hi, lo);
+    *reinterpret_cast<uint32_t *>(&sm.Wh[r][c]) = hi;
+    *reinterpret_cast<uint32_t *>(&sm.Wl[r][c]) = lo;
+  }
+  __syncthreads();
+  const int n0 = (MTILES >= 8 ? warp * MT : warp / WPT) * 16, j0 = MTILES >= 8 ? 0 : (warp % WPT) * NJ;
   float S[MT][NJ][4];
-  const int srow = (NP == 64 ? (warp & 3) * 16 : warp * MT * 16) + g, sj0 = NP == 64 ? (warp >> 2) * NJ : 0;
-  const bool fresh = p.start[s] == 0;
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) S[i][j][0] = S[i][j][1] = S[i][j][2] = S[i][j][3] = 0.f;
+  const uint32_t wh_lane = smem_addr(&sm.Wh[lane & 15][j0 * 8 + (lane >> 4) * 8]), wl_lane = smem_addr(&sm.Wl[lane & 15][j0 * 8 + (lane >> 4) * 8]);
+#pragma unroll
+  for (int k2 = 0; k2 < CHUNK / 16; ++k2) {
+    uint32_t a[MT][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)   // A fragment (rows = state, k = tokens) from the token-major tile, transposed on the way
+      ldsm4t(smem_addr(&sm.B[k2 * 16 + (lane & 7) + (lane >> 4) * 8][n0 + i * 16 + ((lane >> 3) & 1) * 8]), a[i][0], a[i][1], a[i][2], a[i][3]);
+#pragma unroll
+    for (int j = 0; j < NJ; j += 2) {
+      uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+      ldsm4t(wh_lane + (uint32_t)(k2 * 16 * XLD + j * 8) * 2u, h0, h1, h2, h3);
+      ldsm4t(wl_lane + (uint32_t)(k2 * 16 * XLD + j * 8) * 2u, l0, l1, l2, l3);
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        mma16816_bf16(S[i][j], a[i][0], a[i][1], a[i][2], a[i][3], h0, h1);
+        mma16816_bf16(S[i][j + 1], a[i][0], a[i][1], a[i][2], a[i][3], h2, h3);
+        mma16816_bf16(S[i][j], a[i][0], a[i][1], a[i][2], a[i][3], l0, l1);
+        mma16816_bf16(S[i][j + 1], a[i][0], a[i][1], a[i][2], a[i][3], l2, l3);
+      }
+    }
+  }
+  float *out = p.chunk_state + ((size_t)slot * p.heads + h) * p.N * p.P;
 #pragma unroll
   for (int i = 0; i < MT; ++i)
 #pragma unroll
     for (int j = 0; j < NJ; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + (sj0 + j) * 8 + 2 * tig + (e & 1);
-        S[i][j][e] = (!fresh && n < p.N && c < p.P) ? gS[(size_t)n * p.P + c] : 0.f;
+      for (int r = 0; r < 2; ++r) {
+        const int n = n0 + i * 16 + g + 8 * r, c = col0 + (j0 + j) * 8 + 2 * tig;
+        if (n < p.N && c < p.P) *reinterpret_cast<float2 *>(out + (size_t)n * p.P + c) = make_float2(S[i][j][2 * r], S[i][j][2 * r + 1]);
       }
-  auto publish_state = [&]() {
-#pragma unroll
-    for (int i = 0; i < MT; ++i)
-#pragma unroll
-      for (int j = 0; j < NJ; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          uint32_t hi, lo;
-          split_bf2(S[i][j][2 * r], S[i][j][2 * r + 1], hi, lo);
-          *reinterpret_cast<uint32_t *>(&sm.Sh[srow + i * 16 + 8 * r][(sj0 + j) * 8 + 2 * tig]) = hi;
-          *reinterpret_cast<uint32_t *>(&sm.Sl[srow + i * 16 + 8 * r][(sj0 + j) * 8 + 2 * tig]) = lo;
-        }
-  };
-  publish_state();
+}
 
-  const int rb = warp >> 1, half = warp & 1, tr = rb * 16 + g;      // this warp's output rows tr and tr + 8
-  int stage = 0;
-  for (int t0 = 0; t0 < len; t0 += CHUNK, stage ^= 1) {
-    const bool more = t0 + CHUNK < len;
-    if (more) {
-      load_chunk(t0 + CHUNK, stage ^ 1);
-      if (warp == SCAN_WARP) load_dt(t0 + CHUNK, dnext);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();   // operands, decays and the published state are in shared memory
+// Thread: eight consecutive elements of one head's state, along the chunks of its sequence.  In place: sum of the chunk -> state
+// before the chunk, as eight bf16 hi parts and eight lo parts.
+__global__ void ssm_carry_kernel(const Params p) {
+  const int s = blockIdx.z, h = blockIdx.y, i = (blockIdx.x * blockDim.x + threadIdx.x) * 8, n = p.N * p.P;
+  if (i >= n) return;
+  const int chunks = (p.cu[s + 1] - p.cu[s] + CHUNK - 1) / CHUNK;
+  const size_t stride = (size_t)p.heads * n;
+  float *x = p.chunk_state + (size_t)chunk_slot(p, s) * stride + (size_t)h * n + i;
+  const Decays *dec = p.chunk_decays + (size_t)chunk_slot(p, s) * p.heads + h;
+  float *state = p.state + ((size_t)p.slot[s] * p.heads + h) * n + i;
+  float cur[8];
 #pragma unroll
-    for (int e = tid; e < CHUNK * (CP / 2); e += CHUNK_THREADS) {   // weighted x for the state update
-      const int r = e / (CP / 2), c = (e % (CP / 2)) * 2;
-      const float w = sm.w[stage][r];
-      const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[stage][r][c]);
-      uint32_t hi, lo;
-      split_bf2(w * __low2float(x2), w * __high2float(x2), hi, lo);
-      *reinterpret_cast<uint32_t *>(&sm.Wh[r][c]) = hi;
-      *reinterpret_cast<uint32_t *>(&sm.Wl[r][c]) = lo;
-    }
-    // ---- output rows: C S over half of the state rows, C B^T for this warp's tokens s (16 k2 .. + 15 with k2 = half, half + 2)
-    float y[CP / 8][4], G[2][2][4];
+  for (int j = 0; j < 8; ++j) cur[j] = 0.f;
+  if (p.start[s] != 0) {
 #pragma unroll
-    for (int j = 0; j < CP / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+    for (int j = 0; j < 8; j += 4) *reinterpret_cast<float4 *>(cur + j) = *reinterpret_cast<const float4 *>(state + j);
+  }
+  constexpr int U = 4;
+  for (int c0 = 0; c0 < chunks; c0 += U) {
+    float v[U][8], k[U];
 #pragma unroll
-    for (int u = 0; u < 2; ++u)
+    for (int u = 0; u < U; ++u)
+      if (c0 + u < chunks) {
 #pragma unroll
-      for (int j = 0; j < 2; ++j) G[u][j][0] = G[u][j][1] = G[u][j][2] = G[u][j][3] = 0.f;
-    const uint32_t c_lane = smem_addr(&sm.C[stage][rb * 16 + (lane & 15)][(lane >> 4) * 8]);
-    // (B rows are the n side: matrices (s 0-7, k 0-7), (s 0-7, k 8-15), (s 8-15, k 0-7), (s 8-15, k 8-15))
-    const uint32_t b_lane = smem_addr(&sm.B[stage][half * 16 + (lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]);
-    const uint32_t sh_lane = smem_addr(&sm.Sh[lane & 15][(lane >> 4) * 8]), sl_lane = smem_addr(&sm.Sl[lane & 15][(lane >> 4) * 8]);
-#pragma unroll 4
-    for (int kk = 0; kk < NP / 16; ++kk) {
-      uint32_t a0, a1, a2, a3;
-      ldsm4(c_lane + (uint32_t)kk * 32u, a0, a1, a2, a3);
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        if (half + 2 * u > rb) break;     // tokens behind the diagonal only
-        uint32_t b0, b1, b2, b3;
-        ldsm4(b_lane + (uint32_t)(u * 32 * ChunkSmem<NP>::BLD + kk * 16) * 2u, b0, b1, b2, b3);
-        mma16816_bf16(G[u][0], a0, a1, a2, a3, b0, b1);
-        mma16816_bf16(G[u][1], a0, a1, a2, a3, b2, b3);
+        for (int j = 0; j < 8; j += 4) *reinterpret_cast<float4 *>(v[u] + j) = *reinterpret_cast<const float4 *>(x + (size_t)(c0 + u) * stride + j);
+        k[u] = dec[(size_t)(c0 + u) * p.heads].keep;
       }
-      if ((kk & 1) == half) {
 #pragma unroll
-        for (int j = 0; j < CP / 8; j += 2) {
-          uint32_t b0, b1, b2, b3;
-          ldsm4t(sh_lane + (uint32_t)(kk * 16 * XLD + j * 8) * 2u, b0, b1, b2, b3);
-          mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
-          mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
-          ldsm4t(sl_lane + (uint32_t)(kk * 16 * XLD + j * 8) * 2u, b0, b1, b2, b3);
-          mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
-          mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
-        }
+    for (int u = 0; u < U; ++u)
+      if (c0 + u < chunks) {
+        uint4 hi, lo;
+        split_bf2(cur[0], cur[1], hi.x, lo.x);
+        split_bf2(cur[2], cur[3], hi.y, lo.y);
+        split_bf2(cur[4], cur[5], hi.z, lo.z);
+        split_bf2(cur[6], cur[7], hi.w, lo.w);
+        uint4 *o = reinterpret_cast<uint4 *>(x + (size_t)(c0 + u) * stride);
+        o[0] = hi;
+        o[1] = lo;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) cur[j] = fmaf(k[u], cur[j], v[u][j]);
       }
-    }
-    const float e0 = sm.ec[stage][tr], e1 = sm.ec[stage][tr + 8];
+  }
 #pragma unroll
-    for (int j = 0; j < CP / 8; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
-    const float h0 = sm.c_hi[stage][tr], l0 = sm.c_lo[stage][tr], h1 = sm.c_hi[stage][tr + 8], l1 = sm.c_lo[stage][tr + 8];
-    const uint32_t x_lane = smem_addr(&sm.X[stage][half * 16 + (lane & 15)][(lane >> 4) * 8]);
+  for (int j = 0; j < 8; j += 4) *reinterpret_cast<float4 *>(state + j) = *reinterpret_cast<const float4 *>(cur + j);
+}
+
+template <int NP, int CP> struct OutSmem {
+  __nv_bfloat16 C[CHUNK][NP + 8], X[CHUNK][CP + 8], Sh[NP][CP + 8], Sl[NP][CP + 8];
+  union {
+    __nv_bfloat16 B[CHUNK][NP + 8];
+    float ypart[4][16][CP + 4];     // the second warp's share of the output rows, once B is no longer needed
+  };
+  Decays d;
+};
+// Block: one chunk, one head, CP columns.  Two warps share 16 output rows, each with every other 16 state rows (first product) and
+// every other 16 tokens s (second product).
+template <int NP, int CP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_chunk_out_kernel(const Params p) {
+  typedef __nv_bfloat16 T;
+  constexpr int XLD = CP + 8, BLD = NP + 8;
+  extern __shared__ __align__(16) unsigned char smraw[];
+  OutSmem<NP, CP> &sm = *reinterpret_cast<OutSmem<NP, CP> *>(smraw);
+  const int slot = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * CP;
+  int s, t0;
+  if (!chunk_of_slot(p, slot, s, t0)) return;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
+  const int grp = h / (p.heads / p.groups), row0 = p.cu[s] + t0, valid = min(CHUNK, p.cu[s + 1] - row0);
+  const T *xbc = reinterpret_cast<const T *>(p.xbc) + (size_t)row0 * p.C;
+  for (int e = tid; e < CHUNK * (NP / 8); e += CHUNK_THREADS) {
+    const int r = e / (NP / 8), c = (e % (NP / 8)) * 8;
+    const bool in = r < valid && c < p.N;
+    const T *row = xbc + (in ? (size_t)r * p.C + p.inner + grp * p.N + c : 0);
+    cp16(&sm.B[r][c], row, in);
+    cp16(&sm.C[r][c], row + (in ? p.groups * p.N : 0), in);
+  }
+  for (int e = tid; e < CHUNK * (CP / 8); e += CHUNK_THREADS) {
+    const int r = e / (CP / 8), c = (e % (CP / 8)) * 8;
+    const bool in = r < valid && col0 + c < p.P;
+    cp16(&sm.X[r][c], xbc + (in ? (size_t)r * p.C + (size_t)h * p.P + col0 + c : 0), in);
+  }
+  load_decays(p, slot, h, sm.d);
+  const float *st = p.chunk_state + ((size_t)slot * p.heads + h) * p.N * p.P;
+  for (int e = tid; e < NP * (CP / 8); e += CHUNK_THREADS) {
+    const int n = e / (CP / 8), c = (e % (CP / 8)) * 8;
+    const bool in = n < p.N && col0 + c < p.P;
+    const float *src = st + (in ? (size_t)n * p.P + col0 + c : 0);
+    cp16(&sm.Sh[n][c], src, in);
+    cp16(&sm.Sl[n][c], src + 4, in);
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+  const int rb = warp >> 1, half = warp & 1, tr = rb * 16 + g;      // this lane's output rows tr and tr + 8
+  float y[CP / 8][4], G[2][2][4];
+#pragma unroll
+  for (int j = 0; j < CP / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+#pragma unroll
+  for (int u = 0; u < 2; ++u)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) G[u][j][0] = G[u][j][1] = G[u][j][2] = G[u][j][3] = 0.f;
+  const uint32_t c_lane = smem_addr(&sm.C[rb * 16 + (lane & 15)][(lane >> 4) * 8]);
+  // (B rows are the n side: matrices (s 0-7, k 0-7), (s 0-7, k 8-15), (s 8-15, k 0-7), (s 8-15, k 8-15))
+  const uint32_t b_lane = smem_addr(&sm.B[half * 16 + (lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]);
+  const uint32_t sh_lane = smem_addr(&sm.Sh[lane & 15][(lane >> 4) * 8]), sl_lane = smem_addr(&sm.Sl[lane & 15][(lane >> 4) * 8]);
+#pragma unroll 2
+  for (int kk = 0; kk < NP / 16; ++kk) {
+    uint32_t a0, a1, a2, a3;
+    ldsm4(c_lane + (uint32_t)kk * 32u, a0, a1, a2, a3);
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
-      const int k2 = half + 2 * u;
-      if (k2 > rb) break;
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int sc = k2 * 16 + j * 8 + 2 * tig;
-        const float2 ch = *reinterpret_cast<const float2 *>(&sm.c_hi[stage][sc]), cl = *reinterpret_cast<const float2 *>(&sm.c_lo[stage][sc]);
-        const float2 dt = *reinterpret_cast<const float2 *>(&sm.dt[stage][sc]);
-        G[u][j][0] = sc <= tr ? G[u][j][0] * expf((h0 - ch.x) + (l0 - cl.x)) * dt.x : 0.f;
-        G[u][j][1] = sc + 1 <= tr ? G[u][j][1] * expf((h0 - ch.y) + (l0 - cl.y)) * dt.y : 0.f;
-        G[u][j][2] = sc <= tr + 8 ? G[u][j][2] * expf((h1 - ch.x) + (l1 - cl.x)) * dt.x : 0.f;
-        G[u][j][3] = sc + 1 <= tr + 8 ? G[u][j][3] * expf((h1 - ch.y) + (l1 - cl.y)) * dt.y : 0.f;
-      }
-      uint32_t hi[4], lo[4];
-      split_bf2(G[u][0][0], G[u][0][1], hi[0], lo[0]);
-      split_bf2(G[u][0][2], G[u][0][3], hi[1], lo[1]);
-      split_bf2(G[u][1][0], G[u][1][1], hi[2], lo[2]);
-      split_bf2(G[u][1][2], G[u][1][3], hi[3], lo[3]);
+      if (half + 2 * u > rb) break;     // tokens behind the diagonal only
+      uint32_t b0, b1, b2, b3;
+      ldsm4(b_lane + (uint32_t)(u * 32 * BLD + kk * 16) * 2u, b0, b1, b2, b3);
+      mma16816_bf16(G[u][0], a0, a1, a2, a3, b0, b1);
+      mma16816_bf16(G[u][1], a0, a1, a2, a3, b2, b3);
+    }
+    if ((kk & 1) == half) {
 #pragma unroll
       for (int j = 0; j < CP / 8; j += 2) {
         uint32_t b0, b1, b2, b3;
-        ldsm4t(x_lane + (uint32_t)(u * 32 * XLD + j * 8) * 2u, b0, b1, b2, b3);
-        mma16816_bf16(y[j], hi[0], hi[1], hi[2], hi[3], b0, b1);
-        mma16816_bf16(y[j + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
-        mma16816_bf16(y[j], lo[0], lo[1], lo[2], lo[3], b0, b1);
-        mma16816_bf16(y[j + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
+        ldsm4t(sh_lane + (uint32_t)(kk * 16 * XLD + j * 8) * 2u, b0, b1, b2, b3);
+        mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
+        mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
+        ldsm4t(sl_lane + (uint32_t)(kk * 16 * XLD + j * 8) * 2u, b0, b1, b2, b3);
+        mma16816_bf16(y[j], a0, a1, a2, a3, b0, b1);
+        mma16816_bf16(y[j + 1], a0, a1, a2, a3, b2, b3);
       }
     }
-    if (half) {
-#pragma unroll
-      for (int j = 0; j < CP / 8; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) *reinterpret_cast<float2 *>(&sm.ypart[rb][g + 8 * r][j * 8 + 2 * tig]) = make_float2(y[j][2 * r], y[j][2 * r + 1]);
-    }
-    if (warp == SCAN_WARP && more) scan_chunk(dnext, stage ^ 1);
-    __syncthreads();   // weighted x and partial rows are complete; nobody reads the old state any more
-    if (!half) {
-#pragma unroll
-      for (int j = 0; j < CP / 8; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int t = tr + 8 * r, c = j * 8 + 2 * tig;
-          if (t0 + t >= len || col0 + c >= p.P) continue;
-          const float2 o = *reinterpret_cast<const float2 *>(&sm.ypart[rb][g + 8 * r][c]);
-          const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[stage][t][c]);
-          *reinterpret_cast<float2 *>(p.y + (size_t)(row0 + t0 + t) * p.inner + (size_t)h * p.P + col0 + c) =
-              make_float2(fmaf(D, __low2float(x2), y[j][2 * r] + o.x), fmaf(D, __high2float(x2), y[j][2 * r + 1] + o.y));
-        }
-    }
-    // ---- state update: B^T [state rows x tokens] times the weighted x
-    const float keep = sm.keep[stage];
-#pragma unroll
-    for (int i = 0; i < MT; ++i)
-#pragma unroll
-      for (int j = 0; j < NJ; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[i][j][e] *= keep;
-    const uint32_t wh_lane = smem_addr(&sm.Wh[lane & 15][sj0 * 8 + (lane >> 4) * 8]), wl_lane = smem_addr(&sm.Wl[lane & 15][sj0 * 8 + (lane >> 4) * 8]);
-#pragma unroll
-    for (int k2 = 0; k2 < CHUNK / 16; ++k2) {
-      uint32_t wh[NJ][2], wl[NJ][2];
-#pragma unroll
-      for (int j = 0; j < NJ; j += 2) {
-        ldsm4t(wh_lane + (uint32_t)(k2 * 16 * XLD + j * 8) * 2u, wh[j][0], wh[j][1], wh[j + 1][0], wh[j + 1][1]);
-        ldsm4t(wl_lane + (uint32_t)(k2 * 16 * XLD + j * 8) * 2u, wl[j][0], wl[j][1], wl[j + 1][0], wl[j + 1][1]);
-      }
-#pragma unroll
-      for (int i = 0; i < MT; ++i) {
-        // A fragment (rows = state, k = tokens) from the token-major tile: matrices (tokens 0-7 | 8-15) x (state 0-7 | 8-15), transposed
-        uint32_t a0, a1, a2, a3;
-        ldsm4t(smem_addr(&sm.B[stage][k2 * 16 + (lane & 7) + (lane >> 4) * 8][srow - g + i * 16 + ((lane >> 3) & 1) * 8]), a0, a1, a2, a3);
-#pragma unroll
-        for (int j = 0; j < NJ; ++j) {
-          mma16816_bf16(S[i][j], a0, a1, a2, a3, wh[j][0], wh[j][1]);
-          mma16816_bf16(S[i][j], a0, a1, a2, a3, wl[j][0], wl[j][1]);
-        }
-      }
-    }
-    publish_state();
-    __syncthreads();   // this stage of the operands may be refilled
   }
+  const float e0 = sm.d.ec[tr], e1 = sm.d.ec[tr + 8];
 #pragma unroll
-  for (int i = 0; i < MT; ++i)
+  for (int j = 0; j < CP / 8; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
+  const float h0 = sm.d.c_hi[tr], l0 = sm.d.c_lo[tr], h1 = sm.d.c_hi[tr + 8], l1 = sm.d.c_lo[tr + 8];
+  const uint32_t x_lane = smem_addr(&sm.X[half * 16 + (lane & 15)][(lane >> 4) * 8]);
 #pragma unroll
-    for (int j = 0; j < NJ; ++j)
+  for (int u = 0; u < 2; ++u) {
+    const int k2 = half + 2 * u;
+    if (k2 > rb) break;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int n = srow + i * 16 + 8 * (e >> 1), c = col0 + (sj0 + j) * 8 + 2 * tig + (e & 1);
-        if (n < p.N && c < p.P) gS[(size_t)n * p.P + c] = S[i][j][e];
-      }
+    for (int j = 0; j < 2; ++j) {
+      const int sc = k2 * 16 + j * 8 + 2 * tig;
+      const float2 ch = *reinterpret_cast<const float2 *>(&sm.d.c_hi[sc]), cl = *reinterpret_cast<const float2 *>(&sm.d.c_lo[sc]);
+      const float2 dt = *reinterpret_cast<const float2 *>(&sm.d.dt[sc]);
+      G[u][j][0] = sc <= tr ? G[u][j][0] * expf((h0 - ch.x) + (l0 - cl.x)) * dt.x : 0.f;
+      G[u][j][1] = sc + 1 <= tr ? G[u][j][1] * expf((h0 - ch.y) + (l0 - cl.y)) * dt.y : 0.f;
+      G[u][j][2] = sc <= tr + 8 ? G[u][j][2] * expf((h1 - ch.x) + (l1 - cl.x)) * dt.x : 0.f;
+      G[u][j][3] = sc + 1 <= tr + 8 ? G[u][j][3] * expf((h1 - ch.y) + (l1 - cl.y)) * dt.y : 0.f;
+    }
+    uint32_t hi[4], lo[4];
+    split_bf2(G[u][0][0], G[u][0][1], hi[0], lo[0]);
+    split_bf2(G[u][0][2], G[u][0][3], hi[1], lo[1]);
+    split_bf2(G[u][1][0], G[u][1][1], hi[2], lo[2]);
+    split_bf2(G[u][1][2], G[u][1][3], hi[3], lo[3]);
+#pragma unroll
+    for (int j = 0; j < CP / 8; j += 2) {
+      uint32_t b0, b1, b2, b3;
+      ldsm4t(x_lane + (uint32_t)(u * 32 * XLD + j * 8) * 2u, b0, b1, b2, b3);
+      mma16816_bf16(y[j], hi[0], hi[1], hi[2], hi[3], b0, b1);
+      mma16816_bf16(y[j + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
+      mma16816_bf16(y[j], lo[0], lo[1], lo[2], lo[3], b0, b1);
+      mma16816_bf16(y[j + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
+    }
+  }
+  __syncthreads();   // B is no longer needed: its place takes the second warp's rows
+  if (half) {
+#pragma unroll
+    for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) *reinterpret_cast<float2 *>(&sm.ypart[rb][g + 8 * r][j * 8 + 2 * tig]) = make_float2(y[j][2 * r], y[j][2 * r + 1]);
+  }
+  __syncthreads();
+  if (half) return;
+  const float D = p.D[h];
+#pragma unroll
+  for (int j = 0; j < CP / 8; ++j)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int t = tr + 8 * r, c = j * 8 + 2 * tig;
+      if (t >= valid || col0 + c >= p.P) continue;
+      const float2 o = *reinterpret_cast<const float2 *>(&sm.ypart[rb][g + 8 * r][c]);
+      const __nv_bfloat162 x2 = *reinterpret_cast<const __nv_bfloat162 *>(&sm.X[t][c]);
+      *reinterpret_cast<float2 *>(p.y + (size_t)(row0 + t) * p.inner + (size_t)h * p.P + col0 + c) =
+          make_float2(fmaf(D, __low2float(x2), y[j][2 * r] + o.x), fmaf(D, __high2float(x2), y[j][2 * r + 1] + o.y));
+    }
 }
 
 // ------------------------------------------------------------------------------------------ one token per sequence
@@ -600,12 +663,26 @@ template <typename T, int VEC> __global__ void ssm_norm_kernel(const Params p) {
 
 static bool al(const void *q, int bytes) { return ((uintptr_t)q & (bytes - 1)) == 0; }
 
-template <int NP> static int launch_chunk(const Params &p, cudaStream_t st) {
+template <int NP, int CP> static int launch_chunks(const Params &p, cudaStream_t st) {
   static bool set = false;
-  if (!set) { PT_CUDA(cudaFuncSetAttribute(ssm_chunk_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(ChunkSmem<NP>))); set = true; }
-  ssm_chunk_kernel<NP><<<dim3(ceil_div(p.P, CP), p.heads, p.n_seq), CHUNK_THREADS, sizeof(ChunkSmem<NP>), st>>>(p);
+  if (!set) {
+    PT_CUDA(cudaFuncSetAttribute(ssm_chunk_state_kernel<NP, CP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(StateSmem<NP, CP>)));
+    PT_CUDA(cudaFuncSetAttribute(ssm_chunk_out_kernel<NP, CP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(OutSmem<NP, CP>)));
+    set = true;
+  }
+  const dim3 grid(ceil_div(p.P, CP), p.heads, p.n_tok / CHUNK + p.n_seq);
+  ssm_decay_kernel<<<dim3(ceil_div(p.heads, 4), grid.z), 128, 0, st>>>(p);
+  PT_LAUNCH_CHECK("pt_ssm");
+  ssm_chunk_state_kernel<NP, CP><<<grid, CHUNK_THREADS, sizeof(StateSmem<NP, CP>), st>>>(p);
+  PT_LAUNCH_CHECK("pt_ssm");
+  ssm_carry_kernel<<<dim3(ceil_div(p.N * p.P / 8, 64), p.heads, p.n_seq), 64, 0, st>>>(p);
+  PT_LAUNCH_CHECK("pt_ssm");
+  ssm_chunk_out_kernel<NP, CP><<<grid, CHUNK_THREADS, sizeof(OutSmem<NP, CP>), st>>>(p);
   PT_LAUNCH_CHECK("pt_ssm");
   return PT_OK;
+}
+template <int CP> static int dispatch_chunks(const Params &p, cudaStream_t st) {
+  return p.N <= 64 ? launch_chunks<64, CP>(p, st) : (p.N <= 128 ? launch_chunks<128, CP>(p, st) : launch_chunks<256, CP>(p, st));
 }
 
 template <typename T> static int run(const Params &p, bool plain, cudaStream_t st) {
@@ -631,9 +708,9 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
       ssm_conv_kernel<T><<<dim3(ceil_div(p.C + p.heads, 256), p.n_tok), 256, 0, st>>>(p);
     }
     PT_LAUNCH_CHECK("pt_ssm");
-    // the chunked form: bf16, rows that are whole 16-byte units, state of at most 256
-    if (!plain && sizeof(T) == 2 && p.N <= 256 && p.N % 8 == 0 && p.P % 8 == 0 && al(p.xbc, 16) && al(p.y, 8)) {
-      const int rc = p.N <= 64 ? launch_chunk<64>(p, st) : (p.N <= 128 ? launch_chunk<128>(p, st) : launch_chunk<256>(p, st));
+    // the chunked form: bf16, rows that are whole 16-byte units, state of at most 256, with its scratch
+    if (!plain && sizeof(T) == 2 && p.chunk_state && al(p.state, 16) && p.N <= 256 && p.N % 8 == 0 && p.P % 8 == 0 && al(p.xbc, 16) && al(p.y, 8)) {
+      const int rc = p.P <= 32 ? dispatch_chunks<32>(p, st) : dispatch_chunks<64>(p, st);
       if (rc != PT_OK) return rc;
     } else {
       const size_t smem = ((size_t)p.N * SCAN_P + 2 * p.N + SCAN_WARPS * 32) * sizeof(float);
@@ -665,6 +742,11 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
 
 using namespace pt;
 
+extern "C" size_t pt_ssm_workspace_bytes(int n_tok, int n_seq, int heads, int vdim, int state_dim) {
+  const size_t slots = (size_t)n_tok / ssm::CHUNK + n_seq;
+  return slots * heads * ((size_t)state_dim * vdim * sizeof(float) + sizeof(ssm::Decays)) + 16;
+}
+
 extern "C" int pt_ssm(const pt_ssm_args *a, void *stream) {
   PT_REQUIRE(a, "pt_ssm: null args");
   const pt_batch_view &b = a->batch;
@@ -685,5 +767,10 @@ extern "C" int pt_ssm(const pt_ssm_args *a, void *stream) {
   p.cu = b.cu; p.start = b.start; p.slot = b.slot; p.tok_seq = b.tok_seq;
   p.zx = a->zx; p.conv_w = a->conv_w; p.conv_b = a->conv_b; p.dt_bias = a->dt_bias; p.A_log = a->A_log; p.D = a->D; p.norm_w = a->norm_w;
   p.ring = a->ring; p.xbc = a->xbc; p.out = a->out; p.state = a->state; p.dt = a->dt; p.y = a->y;
+  if (a->workspace && ((uintptr_t)a->workspace & 15) == 0 && a->workspace_bytes >= pt_ssm_workspace_bytes(b.n_tok, b.n_seq, a->heads, a->vdim, a->state_dim)) {
+    p.chunk_state = (float *)a->workspace;
+    const size_t n = ((size_t)b.n_tok / ssm::CHUNK + b.n_seq) * a->heads * a->state_dim * a->vdim;
+    p.chunk_decays = (ssm::Decays *)(p.chunk_state + (n + 3) / 4 * 4);
+  }
   return a->dtype == PT_DT_F32 ? ssm::run<float>(p, a->plain != 0, as_stream(stream)) : ssm::run<__nv_bfloat16>(p, a->plain != 0, as_stream(stream));
 }

@@ -107,7 +107,7 @@ class SabisunDecoder(DecodeLoop):
             return SimpleNamespace(w_in=f32(p + f"hc{q}.in", (s,)), w_out=f32(p + f"hc{q}.out", (s,)), mix=f32(p + f"hc{q}.mix", (s, s)))
 
         W = c.width
-        self.head = lin(["embed"], [(c.vocab, W)], row_major=True)     # also the look-up table (rows padded like the head's k)
+        self.head = lin(["embed"], [(c.vocab, W)], keep=True)     # also the look-up table (rows padded like the head's k)
         self.table = self.head.w
         self.final_norm = f32("final.norm", (W,))
         self.subs = []                                                # sublayers in order: mixer, feed-forward, mixer, ...
@@ -205,7 +205,7 @@ class SabisunDecoder(DecodeLoop):
         r.xbc = torch.empty(rows * max((m.channels for m in mm), default=1), dtype=dt, device=dev)
         r.dt = torch.empty(rows * max((m.heads for m in mm), default=1), **f32)
         r.yin = torch.empty(rows * max((m.inner for m in mm), default=1), **f32)
-        r.lin_ws = r.gemm_ws = None
+        r.lin_ws = r.gemm_ws = r.ssm_ws = None
         if dt == torch.bfloat16:
             L = ops._lib.lib()
             lins = [self.head] + [x for s in self.subs for x in (s.proj, s.out)]
@@ -215,6 +215,9 @@ class SabisunDecoder(DecodeLoop):
             if rows > ops.DenseLinear.SKINNY_ROWS:   # k-slices only while there are fewer tiles than SMs: 40 MB hold every such product's
                 n = min(max(L.pt_gemm_workspace_bytes(rows, x.n_out, 8) for x in lins), (40 << 20) + 65536)
                 r.gemm_ws = torch.zeros(n, dtype=torch.uint8, device=dev)
+            if mm:
+                n = max(L.pt_ssm_workspace_bytes(rows, min(self.batch, rows), m.heads, m.vdim, m.state) for m in mm)
+                r.ssm_ws = torch.empty(n, dtype=torch.uint8, device=dev)
         return r
 
     # ---- the layers -----------------------------------------------------------------------------
@@ -247,7 +250,7 @@ class SabisunDecoder(DecodeLoop):
                 ops.window_attn(view, r.a, s.ld, self.caches[s.layer], r.b, s.out.ld, m.heads, m.scale, m.window, m.keep_first, s.sink,
                                 append=m.kv_from is None, max_tokens_per_seq=longest, workspace=self.attn_ws, error_flag=self.error_flag, plain=self.plain)
             else:
-                ops.ssm(view, r.a, s.ld, r.b, s.out.ld, s.w, self.rings[s.layer], self.states[s.layer], r.yin, r.xbc, r.dt, error_flag=self.error_flag,
+                ops.ssm(view, r.a, s.ld, r.b, s.out.ld, s.w, self.rings[s.layer], self.states[s.layer], r.yin, r.xbc, r.dt, r.ssm_ws,
                         plain=self.plain)
             self._linear(s.out, r.b, r.y, n, c.width, r)
 

@@ -80,10 +80,10 @@ def test_true_fp32_product(cuda, m, n, k):
         assert (out[:, n:] == -7).all()
 
 
-@pytest.mark.parametrize("rows", [1, 5, 16, 31, 32, 33, 70, 257, 600])
+@pytest.mark.parametrize("rows", [1, 5, 7, 8, 16, 33, 70, 257, 600])
 @pytest.mark.parametrize("n,k", [(24, 40), (200, 64), (513, 328), (128, 2048)])
 def test_bf16_linear(cuda, rows, n, k):
-    """Skinny-matmul kernel up to 32 rows, tcgen05 GEMM beyond; k that is no multiple of a block, n that is no multiple of a tile."""
+    """Skinny-matmul kernel for few rows, tcgen05 GEMM beyond; k that is no multiple of a block, n that is no multiple of a tile."""
     from poptransformer_b200 import ops
     r = np.random.default_rng(3)
     x, w = bf16(r.standard_normal((rows, k))), bf16(r.standard_normal((n, k)) * k ** -0.5)
@@ -92,16 +92,15 @@ def test_bf16_linear(cuda, rows, n, k):
     L = ops._lib.lib()
     lws = torch.zeros(L.pt_linear_workspace_bytes(min(rows, 32), n, 32), dtype=torch.uint8, device=cuda)
     gws = torch.zeros(L.pt_gemm_workspace_bytes(rows, n, 8), dtype=torch.uint8, device=cuda)
-    for row_major in (False, True):
-        lin = ops.DenseLinear(as_type(w, torch.bfloat16, cuda), torch.bfloat16, row_major=row_major)
-        xp = torch.zeros((rows, lin.ld), dtype=torch.bfloat16, device=cuda)
-        xp[:, :k] = as_type(x, torch.bfloat16, cuda)
-        for dt, tol in ((torch.float32, 1e-5), (torch.bfloat16, 4e-3)):
-            for epi, f in ((ops.EPI_STORE, lambda v: v), (ops.EPI_RELU2, lambda v: np.maximum(v, 0) ** 2)):
-                out = torch.full((rows, n + 8), -7.0, dtype=dt, device=cuda)
-                lin(xp, out, rows, n + 8, epilogue=epi, alpha=0.7, linear_ws=lws, gemm_ws=gws, error_flag=flag)
-                assert rel(out[:, :n].float().cpu(), f(want)) < tol, (row_major, dt, epi)
-                assert (out[:, n:] == -7).all()
+    lin = ops.DenseLinear(as_type(w, torch.bfloat16, cuda), torch.bfloat16)
+    xp = torch.zeros((rows, lin.ld), dtype=torch.bfloat16, device=cuda)
+    xp[:, :k] = as_type(x, torch.bfloat16, cuda)
+    for dt, tol in ((torch.float32, 1e-5), (torch.bfloat16, 4e-3)):
+        for epi, f in ((ops.EPI_STORE, lambda v: v), (ops.EPI_RELU2, lambda v: np.maximum(v, 0) ** 2)):
+            out = torch.full((rows, n + 8), -7.0, dtype=dt, device=cuda)
+            lin(xp, out, rows, n + 8, epilogue=epi, alpha=0.7, linear_ws=lws, gemm_ws=gws, error_flag=flag)
+            assert rel(out[:, :n].float().cpu(), f(want)) < tol, (dt, epi)
+            assert (out[:, n:] == -7).all()
     assert int(flag.item()) == 0
 
 
@@ -242,8 +241,10 @@ class SsmSite:
         buf = torch.zeros((T, ld), dtype=self.dt, device=dev)
         buf[:, :self.width] = as_type(zx, self.dt, dev)
         out = torch.full((T, out_ld), float("nan"), dtype=self.dt, device=dev)
+        n = ops._lib.lib().pt_ssm_workspace_bytes(T, len(lens), self.w.heads, self.w.vdim, self.w.state)
         ops.ssm(view_of(lens, starts, slots, dev), buf, ld, out, out_ld, self.w, self.ring, self.state, torch.empty((T, self.inner), device=dev),
-                torch.empty((T, self.C), dtype=self.dt, device=dev), torch.empty((T, self.w.heads), device=dev), plain=plain)
+                torch.empty((T, self.C), dtype=self.dt, device=dev), torch.empty((T, self.w.heads), device=dev),
+                torch.full((n,), 255, dtype=torch.uint8, device=dev), plain=plain)
         assert not out[:, self.inner:].any()
         return out[:, :self.inner].float().cpu().numpy()
 
