@@ -154,6 +154,16 @@ SIGNATURES = {
 }
 
 _lib = None
+_partial = False
+
+
+def use_library(path):
+    """Loads `path` instead of the full library (before the first call of lib()): it may lack the kernels of other models."""
+    global LIB_PATH, _partial
+    if _lib is not None and path != LIB_PATH:
+        raise PtError(f"{LIB_PATH} is already loaded")
+    _partial = path != LIB_PATH
+    LIB_PATH = path
 
 
 def lib():
@@ -169,6 +179,8 @@ def lib():
     except OSError as e:  # no fallback on purpose
         raise PtError(f"libpt_b200.so could not be loaded from {LIB_PATH}: {e}") from e
     for name, (res, args) in SIGNATURES.items():
+        if _partial and not hasattr(handle, name):
+            continue                     # calling it raises AttributeError
         fn = getattr(handle, name)
         fn.restype, fn.argtypes = res, args
     _lib = handle

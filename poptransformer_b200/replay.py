@@ -21,12 +21,12 @@ def main(argv=None):
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that open requests hold at any time")
     args = ap.parse_args(argv)
 
-    from . import build, checkpoint, registry
+    from . import _lib, build, checkpoint, registry
     config, sd = checkpoint.load_model_dir(args.model)
     if args.dtype not in registry.dtypes(config):
         sys.stderr.write(f"{registry.architecture(config)} does not run in {args.dtype}\n")
         return 3
-    build.build()
+    _lib.use_library(build.build_for(registry.architecture(config)))
     page = 64
     dec, seqs = None, {}
     for line in sys.stdin:

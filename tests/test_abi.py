@@ -31,6 +31,18 @@ def test_library_exports_every_declared_symbol():
     assert handle.pt_version() >= 100
 
 
+def test_parts_link_on_their_own(tmp_path, monkeypatch):
+    """A library with one architecture's sources resolves all of its symbols and has the entry points that the decoder calls."""
+    from poptransformer_b200 import build
+    monkeypatch.setattr(build, "LIB", str(tmp_path / "libpt_b200.so"))
+    path = build.build_for("Sabisun")
+    assert path == build.part_path("Sabisun") and not os.path.exists(build.LIB)
+    handle = ctypes.CDLL(path, mode=os.RTLD_NOW)
+    for s in ("pt_linear", "pt_gemm", "pt_gemm_f32", "pt_hyper", "pt_window_attn", "pt_ssm", "pt_topk", "pt_step_containers"):
+        assert hasattr(handle, s)
+    assert not hasattr(handle, "pt_llama_decode_step")
+
+
 def test_argument_checks_run_without_a_gpu():
     """Shape violations are rejected before any launch, like the reference's setup()-time errors."""
     from poptransformer_b200 import _lib
