@@ -460,7 +460,7 @@ typedef struct pt_batch_view {
 
 /* Hyper-connections (csrc/hyper.cu): `streams` fp32 residual streams per token, xs [rows, streams, width].
  *   table != NULL : every stream <- table[ids[row * ids_ld + *step_dev]] (step_dev NULL: column 0; pos_out[row] <- the step)
- *   y != NULL     : x_t <- sum_s mix[s, t] x_s + mult * w_out[t] * y     (all streams from the old ones)
+ *   y != NULL     : x_t <- sum_s mix[s, t] x_s + mult * w_out[t] * y     (simultaneously)
  *   then u = sum_s w_in[s] x_s (w_in NULL: plain sum, the streams are not written back) and, with h, h = rms_norm(u) * norm_w in
  *   the activation type; columns width .. h_ld - 1 of h are zeroed.  row_index (optional) picks the rows of xs and y. */
 typedef struct pt_hyper_args {

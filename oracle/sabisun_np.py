@@ -1,7 +1,7 @@
 """Plain restatement of the Sabisun decoder in numpy, one function per mechanism, whole sequences only (no cache, no batching).
 
-Everything is float64 unless a dtype is given.  It is the checker of `tests/test_gpu_sabisun*.py`; it shares no code with the
-product path and is never timed.  Conventions: rows are tokens, linears are W[out, in] applied as x @ W.T.
+Everything is float64 unless a dtype is given.  `tests/test_gpu_sabisun.py` compares the kernels with it; it shares no code with
+the product path and is never timed.  Conventions: rows are tokens, linears are W[out, in] applied as x @ W.T.
 """
 import numpy as np
 

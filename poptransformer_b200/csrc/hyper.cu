@@ -1,6 +1,6 @@
 // Hyper-connections: several fp32 residual streams per token instead of one, with learned read, write and mixing weights.
 //
-// A sublayer reads u = sum_s in[s] x_s, computes y = f(rms_norm(u)), and then all streams are replaced at once:
+// A sublayer reads u = sum_s in[s] x_s, computes y = f(rms_norm(u)), and then every stream becomes a mix of the previous streams plus its share of y:
 //     x_t <- sum_s mix[s, t] x_s + mult * out[t] * y .
 // One launch does everything that lies between two sublayers' matrix products: the write of the finished sublayer, the read of
 // the next one and its RMS norm, so the streams cross HBM once in each direction per sublayer.  The same kernel starts a token

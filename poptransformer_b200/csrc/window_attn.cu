@@ -1,6 +1,6 @@
 // Masked attention over a paged cache with per-sequence positions: a sliding window, kept first tokens, a softmax sink, grouped
 // heads, key and value widths of their own, no rotation.  Position i sees key j when j <= i and (i - j < window or j < keep_first);
-// window = 0 means every earlier key.  sink adds exp(sink[h]) to the softmax denominator of head h (no key, no value, not scaled).
+// window = 0 means every earlier key.  sink[h] acts as one more logit of head h that brings weight to the denominator only.
 //
 // The tokens of a launch are packed sequence after sequence (pt_batch_view): row cu[s] + i is position start[s] + i of sequence s,
 // whose pages are page_table[slot[s]].  A page holds K [n_kv][page][dim] and then V [n_kv][page][vdim].  New keys and values are
@@ -290,7 +290,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_pro
     float l = l_run[r];
     l += __shfl_xor_sync(0xffffffffu, l, 1);
     l += __shfl_xor_sync(0xffffffffu, l, 2);
-    if (p.sink) l += exp2f(sink2 - m_run[r]);                   // counts once, in the units of the running maximum
+    if (p.sink) l += exp2f(sink2 - m_run[r]);                   // the sink, in the units of the running maximum
     inv[r] = 1.0f / l;
   }
   __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(p.out) + (size_t)head * p.vdim + 2 * tig;

@@ -52,7 +52,7 @@ def test_hyper_connections(cuda, dtype, streams, width):
     assert np.array_equal(xs.cpu().numpy(), X.transpose(1, 0, 2).astype(np.float32))
     assert rel(h[:, :width].float().cpu(), ref.rms(ref.stream_read(X, w_in), eps) * nw) < tol
     assert not h[:, width:].any()
-    # a write of all streams from the old ones, the next read, and the sum
+    # write, next read, and the sum
     sums = torch.empty((rows, width), device=cuda)
     X = r.standard_normal((streams, rows, width))
     xs.copy_(f(X.transpose(1, 0, 2).astype(np.float32)))
