@@ -1,5 +1,6 @@
 // Matrix product in true fp32 for models that run in 32-bit: y[m, n] = epilogue(alpha * sum_k x[m, k] w[n, k]).
-// 64 x 64 output tiles, 16 k per step through shared memory, 4 x 4 outputs per thread, fused multiply-adds in k order.
+// 64 x 64 output tiles, 16 k per step through shared memory, 4 x 4 outputs per thread, fused multiply-adds in k order.  Every step
+// is summed on its own and then added, so the rounding error grows with the number of steps, not with k.
 #include "common.cuh"
 
 namespace pt {
@@ -21,6 +22,7 @@ __global__ void __launch_bounds__(THREADS) gemm_f32_kernel(const float *__restri
       ws[k][r] = (in && n0 + r < N) ? w[(size_t)(n0 + r) * w_ld + k0 + k] : 0.f;
     }
     __syncthreads();
+    float part[4][4] = {};
 #pragma unroll
     for (int k = 0; k < BK; ++k) {
       float a[4], b[4];
@@ -29,8 +31,12 @@ __global__ void __launch_bounds__(THREADS) gemm_f32_kernel(const float *__restri
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        for (int j = 0; j < 4; ++j) part[i][j] = fmaf(a[i], b[j], part[i][j]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j];
     __syncthreads();
   }
 #pragma unroll
