@@ -67,6 +67,29 @@ uint64_t pt_launch_count(void);
 #define PT_EPI_BIAS_GELU 4    /* y = gelu(fp16(fp16(acc) + bias))    layers/mlp.py:34-41   */
 #define PT_EPI_BIAS_RESIDUAL 5/* y = fp16(res + fp16(fp16(acc) + bias))                  */
 #define PT_EPI_RELU2 6        /* y = max(acc, 0)^2, squared in fp32 (PT_W_BF16 and pt_gemm_f32) */
+#define PT_EPI_GLU 7          /* clamped gated unit of row pairs (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
+#define PT_EPI_GELU_MUL 8     /* gelu_tanh(acc) * mul[mul_ids[row]]  (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
+
+/* Further arguments of the linears of bf16 and fp32 models: pt_linear and pt_gemm with PT_W_BF16, and pt_gemm_f32 (csrc/dense_out.cuh).
+ *   bias       fp32 [n_out], added to alpha * sum before the epilogue; outputs from split_n on (a multiple of 32) skip the epilogue
+ *              and go to out2 in fp32
+ *   PT_EPI_GLU weight rows alternate: eight gate features, the same eight up features; g = min(gate, limit), u = clamp(up, -limit,
+ *              limit), out = g sigmoid(1.702 g) (u + 1), half as many columns as rows
+ *   PT_EPI_GELU_MUL  out[m, n] = gelu_tanh(y) * mul[mul_ids[m] * mul_ld + n], mul of the output's type
+ *   groups     n_groups > 0: the weights are n_groups matrices one after the other (each as packed for the entry point), and tile t of
+ *              group_rows activation rows is multiplied with matrix group_of[t] (device; negative: the tile is skipped).  pt_gemm:
+ *              group_rows a multiple of 16 up to 256; pt_gemm_f32: 64; pt_linear: 1, and row t reads input row t / group_x_div */
+typedef struct pt_dense_ext {
+  const float *bias;
+  float *out2;
+  int out2_ld, split_n;
+  float limit;
+  const void *mul;
+  int mul_ld;
+  const int32_t *mul_ids;
+  int n_groups, group_rows, group_x_div;
+  const int32_t *group_of;
+} pt_dense_ext;
 
 /* ---- Int4ToHalf -------------------------------------------------------------------
  * Replaces the `Int4ToHalf` custom op (poptransformer/ops/customized.py:115-124;
@@ -119,6 +142,7 @@ typedef struct pt_linear_args {
   const void *norm_beta; /* fp16 [k_in]   (PT_PRO_NORMCE)                           */
   int out_dtype;         /* PT_W_BF16: PT_DT_BF16 or PT_DT_F32 (the other formats write fp16 and ignore it)  */
   float alpha;           /* PT_W_BF16: factor on the fp32 sum before the epilogue; 0 = 1                     */
+  const pt_dense_ext *ext; /* PT_W_BF16: further arguments, or NULL                                          */
 } pt_linear_args;
 
 size_t pt_linear_workspace_bytes(int batch, int n_out, int max_ksplit);
@@ -152,7 +176,7 @@ int pt_linear_static_scratch(const pt_linear_args *args, void *stream);
  *              [n_out, k_in/group]; every weight becomes fp16(q) * scale with one rounding (Int4ToHalf,
  *              custom_ops/int4_to_half_codelets.cpp:18-38) on its way to the tensor core.
  *   PT_W_BF16: x = bf16 [m, k_in], w = pt_gemm_repack of bf16 [n_out, k_in] (w_tiled = 1); out = bf16 or fp32 (out_dtype),
- *              epilogue PT_EPI_STORE or PT_EPI_RELU2 on alpha * (x . w^T).  k_in a multiple of 64.
+ *              epilogue PT_EPI_STORE, _RELU2, _GLU or _GELU_MUL on alpha * (x . w^T).  k_in a multiple of 64.
  * FP8 and INT4: k_in must be a multiple of 128.  Accumulation is fp32.  k-slices (ksplit, 0 = chosen by the library) are summed in a fixed
  * order; with more than one slice a workspace is needed (zeroed once by the caller; every launch leaves its counters at zero). */
 typedef struct pt_gemm_args {
@@ -174,12 +198,14 @@ typedef struct pt_gemm_args {
   const void *bias;       /* fp16 [n_out] (PT_EPI_BIAS)                              */
   int out_dtype;          /* PT_W_BF16: PT_DT_BF16 or PT_DT_F32                      */
   float alpha;            /* PT_W_BF16: factor on the fp32 sum; 0 = 1                */
+  const pt_dense_ext *ext; /* PT_W_BF16: further arguments, or NULL                  */
 } pt_gemm_args;
 size_t pt_gemm_workspace_bytes(int m, int n_out, int max_ksplit);
 int pt_gemm(const pt_gemm_args *args, void *stream);
 /* y[m, n] = epilogue(alpha * sum_k x[m, k] w[n, k]) in true fp32 (fused multiply-adds, no TF32): x, w, y fp32 with row strides in
- * elements, any sizes.  epilogue: PT_EPI_STORE or PT_EPI_RELU2. */
+ * elements, any sizes.  epilogue: PT_EPI_STORE, _RELU2, _GLU or _GELU_MUL; ext may be NULL. */
 int pt_gemm_f32(const float *x, int x_ld, const float *w, int w_ld, int m, int n, int k, float alpha, int epilogue, float *y, int y_ld,
+                const pt_dense_ext *ext,
                 void *stream);
 /* One-time tiling of a weight matrix for pt_gemm: [128-row tile][k block] with every tile contiguous.  FP8: E4M3 bytes
  * [n_out, k_in] -> 16 KB tiles in the 128-byte-swizzled image the tensor core reads.  INT4: the reference's int8
@@ -483,6 +509,54 @@ typedef struct pt_hyper_args {
 } pt_hyper_args;
 int pt_hyper(const pt_hyper_args *args, void *stream);
 
+/* Residual stream with norms on the sublayers' outputs (csrc/post_norm.cu), x fp32 [rows, width]:
+ *   table != NULL : x_out[r] = h[r] = table[ids[r * ids_ld + *step_dev]] (step_dev NULL: column 0; pos_out[r] <- the step, id_out[r] <- the id)
+ *   otherwise     : s = row_index ? row_index[r] : r;  Y = y[s] + sum_k pair_w[s, k] pair_y[pair_row[s, k]]  (pair_row NULL: s * top + k);
+ *                   x = x_in[s] + rms_norm(Y) * norm_w;  x_out[r] = x;  h[r] = x, or rms_norm(x) * final_w
+ * x_out, h, y (with top > 0) and final_w may be NULL; x_out may be x_in without row_index.  Columns width .. h_ld - 1 of h are zeroed. */
+typedef struct pt_post_norm_args {
+  int rows, width, dtype;
+  float eps;
+  const float *x_in;
+  float *x_out;
+  const void *table;
+  int table_ld, vocab;
+  const int32_t *ids;
+  int ids_ld;
+  const int32_t *step_dev;
+  int32_t *pos_out, *id_out;
+  const int32_t *row_index;
+  const float *y;
+  int y_ld;
+  const float *pair_y;    /* fp32 rows of width                                      */
+  int pair_ld, top;       /* top at most 64                                          */
+  const float *pair_w;
+  const int32_t *pair_row;
+  const float *norm_w, *final_w;
+  void *h;
+  int h_ld;
+} pt_post_norm_args;
+int pt_post_norm(const pt_post_norm_args *args, void *stream);
+
+/* Mixture of experts (csrc/moe.cu): the `top` experts of every token by router logit, softmax weights over the chosen ones, and the
+ * layout of the grouped products.  tile = 0: only expert and weight are written.  tile > 0: the pairs (token, choice) are sorted by
+ * expert into tiles of `tile` rows: pair_row [n_tok, top], tile_expert [max_tiles] (-1: unused), row_token [max_tiles * tile] (-1:
+ * padding), and with h the rows of h_bytes each are copied to gathered [max_tiles * tile]. */
+typedef struct pt_moe_route_args {
+  int n_tok, experts, top;        /* at most 64 of 1024                              */
+  const float *logits;
+  int logits_ld;
+  int32_t *expert;                /* [n_tok, top]                                    */
+  float *weight;                  /* [n_tok, top]                                    */
+  int tile, max_tiles;
+  int32_t *pair_row, *tile_expert, *row_token;
+  const void *h;
+  int h_bytes;
+  void *gathered;
+} pt_moe_route_args;
+int pt_moe_max_tiles(int n_tok, int experts, int top, int tile);
+int pt_moe_route(const pt_moe_route_args *args, void *stream);
+
 /* Masked attention over a paged cache (csrc/window_attn.cu): sliding window with kept first tokens, softmax sink, grouped heads,
  * separate key and value widths.  pool[page] = K [n_kv][page_size][dim] then V [n_kv][page_size][vdim], page_table
  * [slots][max_pages].  k / v (NULL for a layer that reads another layer's cache) are appended before anything is read. */
@@ -508,6 +582,15 @@ typedef struct pt_window_attn_args {
   void *workspace;        /* decode: pt_window_attn_workspace_bytes, zeroed once     */
   size_t workspace_bytes;
   int32_t *error_flag;    /* optional, set to 12 when a position has no page         */
+  /* Before they are used or cached, q and k (never v, which may be the same rows as k) are divided by their root mean square and
+   * multiplied with q_norm / k_norm (fp32 [dim] or NULL), and their first rope_dims dimensions are rotated: dimension i with
+   * i + rope_dims / 2 by the angle whose (cos, sin) is rope[position][i].  Prompts normalise and rotate q in place. */
+  const float *q_norm, *k_norm;
+  float norm_eps;
+  int rope_dims;
+  const float *rope;      /* fp32 [positions, rope_dims / 2, 2]                      */
+  float out_scale;        /* factor on the output, 0 = 1                             */
+  int out_cols;           /* columns of out that are written or zeroed, 0 = out_ld   */
 } pt_window_attn_args;
 size_t pt_window_attn_workspace_bytes(int n_seq, int n_head, int vdim, int page_size, int max_len, int window, int keep_first);
 int pt_window_attn(const pt_window_attn_args *args, void *stream);
@@ -537,6 +620,34 @@ typedef struct pt_ssm_args {
 } pt_ssm_args;
 size_t pt_ssm_workspace_bytes(int n_tok, int n_seq, int heads, int vdim, int state_dim);
 int pt_ssm(const pt_ssm_args *args, void *stream);
+
+/* Matrix memory with exponential gates (csrc/mlstm.cu) between its projections, with the per-head norm and the output gate. */
+typedef struct pt_mlstm_args {
+  pt_batch_view batch;
+  int dtype;              /* PT_DT_F32 or PT_DT_BF16: q, k, v, gate, out             */
+  int heads, dim, vdim;
+  float gate_cap, q_scale, eps;
+  float out_scale;        /* factor on the output, 0 = 1                             */
+  const void *q, *k;      /* rows of heads * dim                                     */
+  const void *v, *gate;   /* rows of heads * vdim                                    */
+  int ld;                 /* row stride of the four                                  */
+  const float *log_i, *log_f;             /* pre-activations of the gates, rows of heads */
+  int gate_ld;
+  const float *norm_w;                    /* [heads * vdim]                          */
+  float *state;                           /* [slots, pt_mlstm_state_floats(.., 0)]   */
+  float *nm;                              /* [slots, pt_mlstm_state_floats(.., 1)]   */
+  float *y;                               /* scratch [n_tok, heads * vdim]           */
+  void *out;
+  int out_ld;
+  int out_cols;           /* columns of out that are written or zeroed, 0 = out_ld   */
+  int plain;              /* 1: the kernels for any sizes, whatever the shape        */
+  void *workspace;        /* pt_mlstm_workspace_bytes, zeroed once, 16-byte aligned; prompts without it run token by token */
+  size_t workspace_bytes;
+} pt_mlstm_args;
+size_t pt_mlstm_workspace_bytes(int n_tok, int n_seq, int heads, int dim, int vdim);
+/* Floats a sequence slot keeps: which = 0 the matrix, 1 the normaliser and the running maximum. */
+size_t pt_mlstm_state_floats(int heads, int dim, int vdim, int which);
+int pt_mlstm(const pt_mlstm_args *args, void *stream);
 
 #ifdef __cplusplus
 }

@@ -16,6 +16,11 @@ class PtError(RuntimeError):
     popart::error / poplar_error at graph-build time for the same violations)."""
 
 
+class DenseExt(ctypes.Structure):
+    _fields_ = [("bias", c_void_p), ("out2", c_void_p), ("out2_ld", c_int), ("split_n", c_int), ("limit", c_float), ("mul", c_void_p), ("mul_ld", c_int),
+                ("mul_ids", c_void_p), ("n_groups", c_int), ("group_rows", c_int), ("group_x_div", c_int), ("group_of", c_void_p)]
+
+
 class LinearArgs(ctypes.Structure):
     _fields_ = [
         ("wfmt", c_int), ("batch", c_int), ("n_out", c_int), ("k_in", c_int), ("group", c_int),
@@ -24,7 +29,7 @@ class LinearArgs(ctypes.Structure):
         ("norm_eps", c_float), ("act_scale", c_float), ("w_scale", c_float),
         ("bias", c_void_p), ("residual", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("pdl", c_int),
         ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("error_flag", c_void_p), ("norm_beta", c_void_p),
-        ("out_dtype", c_int), ("alpha", c_float),
+        ("out_dtype", c_int), ("alpha", c_float), ("ext", ctypes.POINTER(DenseExt)),
     ]
 
 
@@ -45,7 +50,7 @@ class GemmArgs(ctypes.Structure):
         ("wfmt", c_int), ("m", c_int), ("n_out", c_int), ("k_in", c_int), ("group", c_int), ("epilogue", c_int), ("ksplit", c_int),
         ("w_tiled", c_int), ("x", c_void_p), ("w", c_void_p), ("scales", c_void_p), ("x_scale", c_float), ("w_scale", c_float),
         ("residual", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t),
-        ("error_flag", c_void_p), ("bias", c_void_p), ("out_dtype", c_int), ("alpha", c_float),
+        ("error_flag", c_void_p), ("bias", c_void_p), ("out_dtype", c_int), ("alpha", c_float), ("ext", ctypes.POINTER(DenseExt)),
     ]
 
 
@@ -70,7 +75,8 @@ class WindowAttnArgs(ctypes.Structure):
     _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "n_head", "n_kv", "dim", "vdim", "page_size", "max_pages", "window", "keep_first")] + \
                [("scale", c_float), ("sink", c_void_p), ("q", c_void_p), ("q_ld", c_int), ("k", c_void_p), ("v", c_void_p), ("kv_ld", c_int),
                 ("pool", c_void_p), ("page_table", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("max_tokens_per_seq", c_int), ("max_len", c_int),
-                ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("error_flag", c_void_p)]
+                ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("error_flag", c_void_p), ("q_norm", c_void_p), ("k_norm", c_void_p),
+                ("norm_eps", c_float), ("rope_dims", c_int), ("rope", c_void_p), ("out_scale", c_float), ("out_cols", c_int)]
 
 
 class SsmArgs(ctypes.Structure):
@@ -78,6 +84,26 @@ class SsmArgs(ctypes.Structure):
                [("eps", c_float), ("zx", c_void_p), ("zx_ld", c_int)] + \
                [(n, c_void_p) for n in ("conv_w", "conv_b", "dt_bias", "A_log", "D", "norm_w", "ring", "state", "xbc", "dt", "y", "out")] + \
                [("out_ld", c_int), ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t)]
+
+
+class MlstmArgs(ctypes.Structure):
+    _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "heads", "dim", "vdim")] + [(n, c_float) for n in ("gate_cap", "q_scale", "eps", "out_scale")] + \
+               [(n, c_void_p) for n in ("q", "k", "v", "gate")] + [("ld", c_int), ("log_i", c_void_p), ("log_f", c_void_p), ("gate_ld", c_int)] + \
+               [(n, c_void_p) for n in ("norm_w", "state", "nm", "y", "out")] + [("out_ld", c_int), ("out_cols", c_int), ("plain", c_int), ("workspace", c_void_p),
+                                                                                 ("workspace_bytes", c_size_t)]
+
+
+class PostNormArgs(ctypes.Structure):
+    _fields_ = [("rows", c_int), ("width", c_int), ("dtype", c_int), ("eps", c_float), ("x_in", c_void_p), ("x_out", c_void_p), ("table", c_void_p),
+                ("table_ld", c_int), ("vocab", c_int), ("ids", c_void_p), ("ids_ld", c_int)] + \
+               [(n, c_void_p) for n in ("step_dev", "pos_out", "id_out", "row_index", "y")] + [("y_ld", c_int), ("pair_y", c_void_p), ("pair_ld", c_int), ("top", c_int)] + \
+               [(n, c_void_p) for n in ("pair_w", "pair_row", "norm_w", "final_w", "h")] + [("h_ld", c_int)]
+
+
+class MoeRouteArgs(ctypes.Structure):
+    _fields_ = [("n_tok", c_int), ("experts", c_int), ("top", c_int), ("logits", c_void_p), ("logits_ld", c_int), ("expert", c_void_p), ("weight", c_void_p),
+                ("tile", c_int), ("max_tiles", c_int), ("pair_row", c_void_p), ("tile_expert", c_void_p), ("row_token", c_void_p), ("h", c_void_p), ("h_bytes", c_int),
+                ("gathered", c_void_p)]
 
 
 class LlamaLayer(ctypes.Structure):
@@ -109,7 +135,13 @@ SIGNATURES = {
     "pt_gemm": (c_int, [ctypes.POINTER(GemmArgs), c_void_p]),
     "pt_gemm_packed_bytes": (c_size_t, [c_int, c_int, c_int]),
     "pt_gemm_repack": (c_int, [c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]),
-    "pt_gemm_f32": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p]),
+    "pt_gemm_f32": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, ctypes.POINTER(DenseExt), c_void_p]),
+    "pt_post_norm": (c_int, [ctypes.POINTER(PostNormArgs), c_void_p]),
+    "pt_moe_max_tiles": (c_int, [c_int] * 4),
+    "pt_moe_route": (c_int, [ctypes.POINTER(MoeRouteArgs), c_void_p]),
+    "pt_mlstm_workspace_bytes": (c_size_t, [c_int] * 5),
+    "pt_mlstm_state_floats": (c_size_t, [c_int] * 4),
+    "pt_mlstm": (c_int, [ctypes.POINTER(MlstmArgs), c_void_p]),
     "pt_hyper": (c_int, [ctypes.POINTER(HyperArgs), c_void_p]),
     "pt_window_attn_workspace_bytes": (c_size_t, [c_int] * 7),
     "pt_window_attn": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),

@@ -6,6 +6,8 @@
 
 namespace pt {
 
+static inline bool aligned_to(const void *q, int bytes) { return ((uintptr_t)q & (bytes - 1)) == 0; }
+
 __device__ __forceinline__ float to_f(float x) { return x; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 x) { return __bfloat162float(x); }
 template <typename T> __device__ __forceinline__ T from_f(float x);

@@ -3,8 +3,8 @@
 //
 //   * FP8:  W and X are OCP E4M3 bytes with per-tensor scales (the reference's FP8MatMul, custom_ops/matmul_fp8.cpp:885-1091,
 //           in the E4M3 form): tcgen05.mma kind::f8f6f4, fp32 accumulation in tensor memory, scales applied in the epilogue.
-//   * BF16: W and X bfloat16, tcgen05.mma kind::f16, bf16 or fp32 output with a factor and an optional relu^2: the same kernel as FP8
-//           with 64 elements of k per 128-byte operand row.
+//   * BF16: W and X bfloat16, tcgen05.mma kind::f16, bf16 or fp32 output with the epilogues of dense_out.cuh: the same kernel as FP8
+//           with 64 elements of k per 128-byte operand row.  Grouped: every tile of activation rows names its weight matrix.
 //   * INT4: W is packed nibbles with fp16 group scales (utils/param_handler/precision_strategy.py:24-42,56-60).  A transform
 //           warpgroup turns every staged tile into fp16(q) * scale - one fp16 rounding per weight, exactly the reference's
 //           Int4ToHalf (custom_ops/int4_to_half_codelets.cpp:18-38) - in the shared-memory layout the tensor core reads;
@@ -28,6 +28,7 @@
 #include <cstdlib>
 #include <cstring>
 
+#include "dense_out.cuh"
 #include "tile_math.cuh"
 
 namespace pt {
@@ -52,8 +53,7 @@ struct GemmParams {
   int kb_per_split, n_kb; // k blocks (of 128 bytes of operand row) per k-slice / in total
   int ksplit, stages, raw_stages;
   int w_tiled;            // weights tiled by pt_gemm_repack (one contiguous tile per stage) instead of row-major
-  int epilogue;           // PT_EPI_STORE, PT_EPI_RESIDUAL or PT_EPI_BIAS (BF16: PT_EPI_STORE or PT_EPI_RELU2)
-  int out_dt;             // BF16: PT_DT_BF16 or PT_DT_F32
+  int epilogue;           // PT_EPI_STORE, PT_EPI_RESIDUAL or PT_EPI_BIAS (BF16: see dense)
   float out_scale;
   const unsigned char *w; // tiled weights (w_tiled)
   const __half *scales;   // INT4: [N][K / group]
@@ -64,6 +64,9 @@ struct GemmParams {
   float *partial;         // [ksplit][M][N] (ksplit > 1)
   int *counters;          // [n tiles * m tiles]
   int *error_flag;
+  DenseOut dense;         // BF16: what becomes of a finished sum
+  const int *group_of;    // BF16, grouped: the weight matrix of every tile of mb rows (negative: none)
+  size_t group_stride;    // bytes between weight matrices
 };
 
 // ------------------------------------------------------------------------------------------ PTX
@@ -187,10 +190,7 @@ __device__ __forceinline__ void give_up(SharedCtl &ctl, int *error_flag, int cod
 // One finished sum of the FP8 / INT4 kernels (fp16 output) or of the BF16 kernel.
 template <bool BF16> __device__ __forceinline__ void store_out(const GemmParams &p, float acc, int m, int n) {
   if constexpr (BF16) {
-    float y = acc * p.out_scale;
-    if (p.epilogue == PT_EPI_RELU2) { y = fmaxf(y, 0.f); y *= y; }
-    if (p.out_dt == PT_DT_F32) reinterpret_cast<float *>(p.out)[(size_t)m * p.out_ld + n] = y;
-    else reinterpret_cast<__nv_bfloat16 *>(p.out)[(size_t)m * p.out_ld + n] = __float2bfloat16_rn(y);
+    dense_store(p.dense, m, n, acc);
   } else {
     __half y = __float2half_rn(acc * p.out_scale);
     if (p.epilogue == PT_EPI_RESIDUAL) y = h_add(__ldcg(p.residual + (size_t)m * p.N + n), y);
@@ -210,6 +210,16 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
     tmem_ld16(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, v);
 #pragma unroll
     for (int j = 0; j < 16; ++j) sum[j] = __uint_as_float(v[j]);
+    if constexpr (BF16) {
+      if (p.ksplit == 1 && p.dense.epilogue == PT_EPI_GLU && n0 + q * 32 < p.dense.split_n) {   // (uniform over the warp)
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          const float up = __shfl_xor_sync(0xffffffffu, sum[j], 8);
+          if (n < p.N && m0 + c0 + j < p.M && (lane & 8) == 0) dense_store_glu(p.dense, m0 + c0 + j, n, sum[j], up);
+        }
+        continue;
+      }
+    }
     if (n < p.N) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
@@ -227,49 +237,69 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 }
 
 // The BF16 kernel's epilogue of a whole 32-column group without k-slices: uniform branches outside the element loop, pointer
-// increments instead of index arithmetic (the general form above costs as much as the products of a 2048-deep tile).  bf16 output:
-// neighbouring lanes (n, n + 1) trade values of two columns, so every store writes 4 bytes per lane.
-template <bool F32, bool RELU2>
-__device__ __forceinline__ void epilogue_rows32(const GemmParams &p, const uint32_t (&v)[32], int n, int m, int lane) {
+// increments instead of index arithmetic (the general form above costs as much as the products of a 2048-deep tile).
+// bf16 output: neighbouring lanes (n, n + 1) trade values of two columns, so every store writes 4 bytes per lane.
+// Gated features: lanes n and n + 8 trade likewise, and each computes one column of the pair's feature.
+enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_GLU = 2 };
+template <int KIND, bool RELU2>
+__device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, int ld, const uint32_t (&v)[32], int n, int m, int lane) {
+  const float b = d.bias ? __ldg(d.bias + n + (KIND == OUT_F32 && out == d.out2 ? d.split_n : 0)) : 0.f;
   auto fin = [&](uint32_t x) {
-    float y = __uint_as_float(x) * p.out_scale;
+    float y = fmaf(__uint_as_float(x), d.alpha, b);
     if (RELU2) { y = fmaxf(y, 0.f); y *= y; }
     return y;
   };
-  if (F32) {
-    float *o = reinterpret_cast<float *>(p.out) + (size_t)m * p.out_ld + n;
+  if (KIND == OUT_F32) {
+    float *o = reinterpret_cast<float *>(out) + (size_t)m * ld + n;
 #pragma unroll
     for (int j = 0; j < 32; ++j) {
       *o = fin(v[j]);
-      o += p.out_ld;
+      o += ld;
     }
-  } else {
+  } else if (KIND == OUT_BF16) {
     const int odd = lane & 1;
-    __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(p.out) + (size_t)(m + odd) * p.out_ld + (n - odd);
+    __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(out) + (size_t)(m + odd) * ld + (n - odd);
 #pragma unroll
     for (int j = 0; j < 32; j += 2) {
-      const float a = fin(v[j]), b = fin(v[j + 1]);
-      const float t = __shfl_xor_sync(0xffffffffu, odd ? a : b, 1);     // even lane: column j of n + 1; odd lane: column j + 1 of n - 1
-      *reinterpret_cast<__nv_bfloat162 *>(o) = odd ? __floats2bfloat162_rn(t, b) : __floats2bfloat162_rn(a, t);
-      o += 2 * (size_t)p.out_ld;
+      const float a = fin(v[j]), c = fin(v[j + 1]);
+      const float t = __shfl_xor_sync(0xffffffffu, odd ? a : c, 1);     // even lane: column j of n + 1; odd lane: column j + 1 of n - 1
+      *reinterpret_cast<__nv_bfloat162 *>(o) = odd ? __floats2bfloat162_rn(t, c) : __floats2bfloat162_rn(a, t);
+      o += 2 * (size_t)ld;
+    }
+  } else {
+    const bool up = lane & 8;
+    __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(out) + (size_t)(m + (up ? 1 : 0)) * ld + n / 16 * 8 + n % 8;
+#pragma unroll
+    for (int j = 0; j < 32; j += 2) {
+      const float a = fin(v[j]), c = fin(v[j + 1]);
+      const float t = __shfl_xor_sync(0xffffffffu, up ? a : c, 8);      // gate lane: the up value of column j; up lane: the gate value of j + 1
+      *o = __float2bfloat16_rn(up ? glu_f<true>(t, c, d.limit) : glu_f<true>(a, t, d.limit));
+      o += 2 * (size_t)ld;
     }
   }
 }
 __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem, int q, int lane, int n0, int m0, int ks) {
-  const int n = n0 + q * 32 + lane;
-  const bool f32 = p.out_dt == PT_DT_F32;
-  // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16 (warp-uniform conditions)
-  const bool fast = p.ksplit == 1 && n0 + q * 32 + 32 <= p.N && (f32 || (p.out_ld % 2 == 0 && ((uintptr_t)p.out & 3) == 0));
+  const DenseOut &d = p.dense;
+  const int nq = n0 + q * 32, n = nq + lane;
+  // (warp-uniform) where this warp's 32 outputs go
+  const bool second = nq >= d.split_n, glu = d.epilogue == PT_EPI_GLU && !second, f32 = second || d.out_dt == PT_DT_F32;
+  // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16
+  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && (second || d.epilogue != PT_EPI_GELU_MUL) && !(glu && f32) &&
+                    (f32 || glu || (d.out_ld % 2 == 0 && ((uintptr_t)d.out & 3) == 0));
   const int whole = fast ? min(p.mb, p.M - m0) & ~31 : 0;
   for (int c0 = 0; c0 < whole; c0 += 32) {
     uint32_t v[32];
     tmem_ld32(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, v);
-    if (f32) {
-      if (p.epilogue == PT_EPI_RELU2) epilogue_rows32<true, true>(p, v, n, m0 + c0, lane);
-      else epilogue_rows32<true, false>(p, v, n, m0 + c0, lane);
+    if (second) {
+      epilogue_rows32<OUT_F32, false>(d, d.out2, d.out2_ld, v, n - d.split_n, m0 + c0, lane);
+    } else if (glu) {
+      epilogue_rows32<OUT_GLU, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+    } else if (f32) {
+      if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_F32, true>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else epilogue_rows32<OUT_F32, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     } else {
-      if (p.epilogue == PT_EPI_RELU2) epilogue_rows32<false, true>(p, v, n, m0 + c0, lane);
-      else epilogue_rows32<false, false>(p, v, n, m0 + c0, lane);
+      if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_BF16, true>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else epilogue_rows32<OUT_BF16, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     }
   }
   if (whole < p.mb) epilogue<true>(p, tmem, q, lane, 0, 1, n0, m0, ks, whole);
@@ -296,15 +326,28 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
         for (int i = tid; i < rows * (BM / 4); i += threads) {
           const int m = m0 + i / (BM / 4), n = n0 + (i % (BM / 4)) * 4;
           if (n >= p.N) continue;
-          float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-          for (int s0 = 0; s0 < p.ksplit; s0 += 4) {
-            float4 part[4];
+          auto sum4 = [&](int nn) {
+            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int s0 = 0; s0 < p.ksplit; s0 += 4) {
+              float4 part[4];
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
-              part[j] = (s0 + j < p.ksplit) ? __ldcg(reinterpret_cast<const float4 *>(p.partial + ((size_t)(s0 + j) * p.M + m) * p.N + n)) : make_float4(0.f, 0.f, 0.f, 0.f);
+              for (int j = 0; j < 4; ++j)
+                part[j] = (s0 + j < p.ksplit) ? __ldcg(reinterpret_cast<const float4 *>(p.partial + ((size_t)(s0 + j) * p.M + m) * p.N + nn)) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) { acc.x += part[j].x; acc.y += part[j].y; acc.z += part[j].z; acc.w += part[j].w; }
+              for (int j = 0; j < 4; ++j) { acc.x += part[j].x; acc.y += part[j].y; acc.z += part[j].z; acc.w += part[j].w; }
+            }
+            return acc;
+          };
+          if (p.dense.epilogue == PT_EPI_GLU && n < p.dense.split_n) {   // gate features n % 16 < 8, their up features eight further
+            if (n & 8) continue;
+            const float4 gt = sum4(n), up = sum4(n + 8);
+            dense_store_glu(p.dense, m, n, gt.x, up.x);
+            dense_store_glu(p.dense, m, n + 1, gt.y, up.y);
+            dense_store_glu(p.dense, m, n + 2, gt.z, up.z);
+            dense_store_glu(p.dense, m, n + 3, gt.w, up.w);
+            continue;
           }
+          const float4 acc = sum4(n);
           store_out<true>(p, acc.x, m, n);
           store_out<true>(p, acc.y, m, n + 1);
           store_out<true>(p, acc.z, m, n + 2);
@@ -316,15 +359,24 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
     for (int i = tid; i < rows * BM; i += threads) {
       const int m = m0 + i / BM, n = n0 + (i % BM);
       if (n >= p.N) continue;
-      float acc = 0.f;
-      for (int s0 = 0; s0 < p.ksplit; s0 += 8) {
-        float part[8];
+      auto sum1 = [&](int nn) {
+        float acc = 0.f;
+        for (int s0 = 0; s0 < p.ksplit; s0 += 8) {
+          float part[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) part[j] = (s0 + j < p.ksplit) ? __ldcg(p.partial + ((size_t)(s0 + j) * p.M + m) * p.N + n) : 0.f;
+          for (int j = 0; j < 8; ++j) part[j] = (s0 + j < p.ksplit) ? __ldcg(p.partial + ((size_t)(s0 + j) * p.M + m) * p.N + nn) : 0.f;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc += part[j];
+          for (int j = 0; j < 8; ++j) acc += part[j];
+        }
+        return acc;
+      };
+      if constexpr (BF16) {
+        if (p.dense.epilogue == PT_EPI_GLU && n < p.dense.split_n) {
+          if (!(n & 8)) dense_store_glu(p.dense, m, n, sum1(n), sum1(n + 8));
+          continue;
+        }
       }
-      store_out<BF16>(p, acc, m, n);
+      store_out<BF16>(p, sum1(n), m, n);
     }
   }
 }
@@ -345,6 +397,14 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
   const uint32_t b_bytes = (uint32_t)p.mb * BKB;
   const uint32_t stage_bytes = A_TILE + ((b_bytes + 1023u) & ~1023u);
   const uint32_t smem_s = sa(smem);
+  size_t w_base = 0;
+  if constexpr (BF16) {
+    if (p.group_of) {
+      const int grp = p.group_of[blockIdx.z];
+      if (grp < 0) return;                     // a tile without rows: nothing is initialised yet
+      w_base = (size_t)grp * p.group_stride;
+    }
+  }
   uint32_t tmem_cols = 32;
   while ((int)tmem_cols < p.mb) tmem_cols <<= 1;
 
@@ -367,7 +427,7 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
   if (warp == 0) {
     if (lane == 0) {
       // (ring positions and parities are carried as counters: this thread's instruction count per stage is what limits a CTA)
-      const unsigned char *wt = p.w + ((size_t)blockIdx.x * p.n_kb + kb0) * A_TILE;
+      const unsigned char *wt = p.w + w_base + ((size_t)blockIdx.x * p.n_kb + kb0) * A_TILE;
       const uint32_t tx = A_TILE + b_bytes, full0 = sa(&ctl.full[0]), empty0 = sa(&ctl.empty[0]);
       const bool tiled = p.w_tiled != 0;
       int s = 0, kx = kb0 * KX;
@@ -709,7 +769,9 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   PT_REQUIRE(a->x && a->w && a->out, "pt_gemm: null x / w / out");
   PT_REQUIRE(((uintptr_t)a->x & 15) == 0 && ((uintptr_t)a->w & 15) == 0, "pt_gemm: x and w must be 16-byte aligned");
   if (bf16) {
-    PT_REQUIRE(a->epilogue == PT_EPI_STORE || a->epilogue == PT_EPI_RELU2, "pt_gemm: BF16 epilogue %d (store or relu2)", a->epilogue);
+    PT_REQUIRE(dense_epilogue_known(a->epilogue), "pt_gemm: BF16 epilogue %d (store, relu2, glu or gelu-mul)", a->epilogue);
+    const char *bad = dense_ext_error(a->epilogue, a->n_out, a->ext);
+    PT_REQUIRE(!bad, "pt_gemm: %s", bad);
     PT_REQUIRE(a->out_dtype == PT_DT_BF16 || a->out_dtype == PT_DT_F32, "pt_gemm: BF16 weights write bf16 or fp32, got type %d", a->out_dtype);
   } else {
     PT_REQUIRE(a->epilogue == PT_EPI_STORE || a->epilogue == PT_EPI_RESIDUAL || a->epilogue == PT_EPI_BIAS, "pt_gemm: epilogue %d (store, residual or bias)",
@@ -729,9 +791,16 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   p.w_tiled = a->w_tiled ? 1 : 0;
   p.w = (const unsigned char *)a->w;
   p.mb = std::min(256, ceil_div(a->m, 16) * 16);
+  const bool grouped = bf16 && a->ext && a->ext->n_groups > 0;
   const int n_tiles = ceil_div(a->n_out, tc::BM);
   // BF16: fewer activation rows per tile before k-slices (whose sums take a detour over HBM) when there are not enough tiles
-  if (bf16)
+  if (grouped) {
+    p.mb = a->ext->group_rows;
+    PT_REQUIRE(p.mb % 16 == 0 && p.mb >= 16 && p.mb <= 256 && a->m % p.mb == 0 && a->m / p.mb <= 65535, "pt_gemm: groups of %d rows (16 .. 256 in steps of 16) in %d rows",
+               p.mb, a->m);
+    p.group_of = a->ext->group_of;
+    p.group_stride = pt_gemm_packed_bytes(a->wfmt, a->n_out, a->k_in);
+  } else if (bf16)
     while (p.mb > 64 && n_tiles * ceil_div(a->m, p.mb) * 4 < sm_count() * 3) p.mb = ceil_div(p.mb, 32) * 16;
   const int m_tiles = ceil_div(a->m, p.mb);
   p.n_kb = (int4 || bf16) ? a->k_in / 64 : a->k_in / 128;
@@ -752,13 +821,12 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   p.ksplit = ceil_div(p.n_kb, p.kb_per_split);
   p.epilogue = a->epilogue;
   p.out_scale = int4 ? 1.0f : (a->x_scale > 0.f ? a->x_scale : 1.0f) * (a->w_scale > 0.f ? a->w_scale : 1.0f);
-  if (bf16) p.out_scale = a->alpha != 0.f ? a->alpha : 1.0f;
-  p.out_dt = a->out_dtype;
   p.scales = (const __half *)a->scales;
   p.residual = (const __half *)a->residual;
   p.bias = (const __half *)a->bias;
   p.out = (__half *)a->out;
   p.out_ld = a->out_ld > 0 ? a->out_ld : a->n_out;
+  if (bf16) p.dense = make_dense_out(a->out, p.out_ld, a->out_dtype, a->epilogue, a->alpha, a->ext);
   p.error_flag = a->error_flag;
   if (p.ksplit > 1) {
     const size_t need = pt_gemm_workspace_bytes(a->m, a->n_out, p.ksplit);

@@ -29,6 +29,7 @@
 // logit tolerance, and pt_int4_to_half remains the bit-exact form of that op.
 #include <algorithm>
 
+#include "dense_out.cuh"
 #include "tile_math.cuh"
 
 namespace pt {
@@ -46,8 +47,12 @@ struct LinearParams {
   float *partial;
   int *counters, *error_flag;
   int B, N, K, n_rt, nchunks, chunks_per_split, ksplit, pro, epi, xs_stride, out_ld, pdl;
-  int out_dt;   // PT_W_BF16: PT_DT_BF16 or PT_DT_F32
   float eps, inv_act_scale, out_scale;
+  // PT_W_BF16
+  DenseOut dense;
+  const int *group_of;       // grouped: blockIdx.z is a row of its own, multiplied with weight matrix group_of[z]; its input is row z / group_x_div
+  int group_x_div, rows;     // rows: B, or the number of grouped rows (B is then 1)
+  size_t group_stride;       // bytes between weight matrices
 };
 
 // ------------------------------------------------------------------------------------------ device helpers
@@ -85,9 +90,18 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
   __shared__ float s_stat[32], s_mean[32];
   __shared__ float s_part[32 * kWarps], s_part1[32 * kWarps];
   __shared__ int s_last;
+  const int z = WFMT == PT_W_BF16 ? blockIdx.z : 0;   // the first output row of this block
+  size_t w_base = 0;
+  const __half *px = p.x;
+  if constexpr (WFMT == PT_W_BF16) {
+    if (p.group_of) {
+      w_base = (size_t)p.group_of[z] * p.group_stride;
+      px += (size_t)(z / p.group_x_div) * p.K;
+    }
+  }
 
   // ---- start streaming this warp's tiles before anything else (they do not depend on the previous kernel)
-  const unsigned char *wsrc = p.w + ((size_t)(active ? rt : 0) * p.nchunks + c_begin) * TILE + lane * 16;
+  const unsigned char *wsrc = p.w + w_base + ((size_t)(active ? rt : 0) * p.nchunks + c_begin) * TILE + lane * 16;
   const uint32_t ring_lane = smem_addr(ring) + lane * 16;
   auto issue = [&](int i) {   // tile i of the slice -> stage i % kStages; always commits so that group counting stays uniform
     if (active && i < nslice) {
@@ -120,7 +134,7 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
   const bool fits = total_units <= PRE * kThreads;
   auto unit_src = [&](int i) {
     const int b = i / slice_units, u = i - b * slice_units;
-    return reinterpret_cast<const uint4 *>(p.x + (size_t)b * p.K + (size_t)c_begin * CHUNK_K + (size_t)u * 8);
+    return reinterpret_cast<const uint4 *>(px + (size_t)b * p.K + (size_t)c_begin * CHUNK_K + (size_t)u * 8);
   };
   uint4 pre[PRE];
   if (fits) {
@@ -137,7 +151,7 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
     const int part = warp % wpr;
     for (int b = warp / wpr; b < p.B; b += kWarps / wpr) {
       float ss = 0.f, s1 = 0.f;
-      const uint4 *xr = reinterpret_cast<const uint4 *>(p.x + (size_t)b * p.K);
+      const uint4 *xr = reinterpret_cast<const uint4 *>(px + (size_t)b * p.K);
       for (int i0 = part * 32 + lane; i0 < units; i0 += 4 * 32 * wpr) {
         uint4 v[4];
 #pragma unroll
@@ -327,16 +341,17 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int bcol = t * 8 + 2 * tig + (j & 1), row = g + 8 * (j >> 1);
-          if (bcol < p.B) p.partial[((size_t)ks * p.B + bcol) * npad + rt * 16 + row] = acc[t][j];
+          if (bcol < p.B) p.partial[((size_t)ks * p.rows + z + bcol) * npad + rt * 16 + row] = acc[t][j];
         }
     }
     __threadfence();
     __syncthreads();
-    if (tid == 0) s_last = (atomicAdd(p.counters + blockIdx.x, 1) == p.ksplit - 1);
+    int *counter = p.counters + (size_t)z * gridDim.x + blockIdx.x;
+    if (tid == 0) s_last = (atomicAdd(counter, 1) == p.ksplit - 1);
     __syncthreads();
     if (!s_last) return;
     __threadfence();
-    if (tid == 0) p.counters[blockIdx.x] = 0;  // ready for the next launch on this stream
+    if (tid == 0) *counter = 0;  // ready for the next launch on this stream
     if (active) {
       // Sum in split order (deterministic).  The loads of two splits (2 x 4 NB values) are issued together, so the reduction
       // costs ksplit / 2 trips to L2 instead of one per (value, split).
@@ -354,8 +369,8 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
           for (int j = 0; j < 4; ++j) {
             const int bcol = t * 8 + 2 * tig + (j & 1), row8 = 8 * (j >> 1);
             const bool ok = bcol < p.B;
-            a0[t][j] = ok ? __ldcg(base + ((size_t)s0 * p.B + bcol) * npad + row8) : 0.f;
-            a1[t][j] = (ok && two) ? __ldcg(base + ((size_t)(s0 + 1) * p.B + bcol) * npad + row8) : 0.f;
+            a0[t][j] = ok ? __ldcg(base + ((size_t)s0 * p.rows + z + bcol) * npad + row8) : 0.f;
+            a1[t][j] = (ok && two) ? __ldcg(base + ((size_t)(s0 + 1) * p.rows + z + bcol) * npad + row8) : 0.f;
           }
 #pragma unroll
         for (int t = 0; t < NB; ++t)
@@ -378,15 +393,12 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
       if (b >= p.B) continue;
       const float lo = acc[t][jb] * p.out_scale, hi = acc[t][2 + jb] * p.out_scale;  // rows g and g + 8
       if constexpr (WFMT == PT_W_BF16) {
-#pragma unroll
-        for (int hr = 0; hr < 2; ++hr) {
-          const int n = rt * 16 + g + 8 * hr;
-          if (n >= p.N) continue;
-          float y = hr ? hi : lo;
-          if (p.epi == PT_EPI_RELU2) { y = fmaxf(y, 0.f); y *= y; }
-          const size_t o = (size_t)b * p.out_ld + n;
-          if (p.out_dt == PT_DT_F32) reinterpret_cast<float *>(p.out)[o] = y;
-          else reinterpret_cast<__nv_bfloat16 *>(p.out)[o] = __float2bfloat16_rn(y);
+        const int n = rt * 16 + g;
+        if (p.epi == PT_EPI_GLU && n < p.dense.split_n) {      // rows 0..7 of the tile are gate rows, 8..15 the matching up rows
+          if (n < p.N) dense_store_glu(p.dense, z + b, n, acc[t][jb], acc[t][2 + jb]);
+        } else {
+          if (n < p.N) dense_store(p.dense, z + b, n, acc[t][jb]);
+          if (n + 8 < p.N) dense_store(p.dense, z + b, n + 8, acc[t][2 + jb]);
         }
         continue;
       }
@@ -479,7 +491,7 @@ template <int WFMT, int NB, int ST> static int launch_linear(const LinearParams 
     attr_set = true;
   }
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(ceil_div(p.n_rt, kWarps), p.ksplit);
+  cfg.gridDim = dim3(ceil_div(p.n_rt, kWarps), p.ksplit, p.group_of ? p.rows : 1);
   cfg.blockDim = dim3(kThreads);
   cfg.dynamicSmemBytes = smem;
   cfg.stream = st;
@@ -584,14 +596,18 @@ extern "C" int pt_linear_repack(int wfmt, const void *w, const void *scale, int 
 extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   PT_REQUIRE(a, "pt_linear: null args");
   PT_REQUIRE(a->wfmt == PT_W_INT4 || a->wfmt == PT_W_FP16 || a->wfmt == PT_W_FP8 || a->wfmt == PT_W_BF16, "pt_linear: unknown weight format %d", a->wfmt);
-  PT_REQUIRE(a->batch >= 1 && a->batch <= 32, "pt_linear: batch=%d outside 1..32 (larger batches use the GEMM path)", a->batch);
+  const bool grouped = a->wfmt == PT_W_BF16 && a->ext && a->ext->n_groups > 0;     // every row has a weight matrix of its own
+  PT_REQUIRE(a->batch >= 1 && a->batch <= (grouped ? 65535 : 32), "pt_linear: batch=%d outside 1..32 (larger batches use the GEMM path)", a->batch);
   const int ck = chunk_k(a->wfmt);
   PT_REQUIRE(a->n_out > 0 && a->k_in > 0 && a->k_in % ck == 0, "pt_linear: k_in=%d must be a positive multiple of %d", a->k_in, ck);
   PT_REQUIRE(a->x && a->packed_w && a->out, "pt_linear: null x / packed_w / out");
   PT_REQUIRE(a->prologue >= PT_PRO_NONE && a->prologue <= PT_PRO_NORMCE, "pt_linear: bad prologue %d", a->prologue);
   if (a->wfmt == PT_W_BF16) {
-    PT_REQUIRE(a->prologue == PT_PRO_NONE && (a->epilogue == PT_EPI_STORE || a->epilogue == PT_EPI_RELU2),
-               "pt_linear: bf16 weights take no prologue and the store or relu2 epilogue, got %d / %d", a->prologue, a->epilogue);
+    PT_REQUIRE(a->prologue == PT_PRO_NONE && dense_epilogue_known(a->epilogue),
+               "pt_linear: bf16 weights take no prologue and the store, relu2, glu or gelu-mul epilogue, got %d / %d", a->prologue, a->epilogue);
+    const char *bad = dense_ext_error(a->epilogue, a->n_out, a->ext);
+    PT_REQUIRE(!bad, "pt_linear: %s", bad);
+    PT_REQUIRE(!grouped || (a->ext->group_rows == 1 && a->ext->group_x_div >= 1), "pt_linear: groups come row by row");
     PT_REQUIRE(a->out_dtype == PT_DT_BF16 || a->out_dtype == PT_DT_F32, "pt_linear: bf16 weights write bf16 or fp32, got type %d", a->out_dtype);
   } else {
     PT_REQUIRE(a->epilogue >= PT_EPI_STORE && a->epilogue <= PT_EPI_BIAS_RESIDUAL, "pt_linear: bad epilogue %d", a->epilogue);
@@ -618,7 +634,7 @@ extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   p.out = (__half *)a->out;
   p.error_flag = a->error_flag;
   p.pdl = a->pdl ? 1 : 0;
-  p.B = a->batch; p.N = a->n_out; p.K = a->k_in;
+  p.B = grouped ? 1 : a->batch; p.rows = a->batch; p.N = a->n_out; p.K = a->k_in;
   p.out_ld = a->out_ld > 0 ? a->out_ld : (a->epilogue == PT_EPI_SWIGLU ? a->n_out / 2 : a->n_out);
   p.n_rt = ceil_div(a->n_out, 16);
   p.nchunks = a->k_in / ck;
@@ -626,11 +642,20 @@ extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   p.eps = a->norm_eps;
   p.inv_act_scale = cast ? 1.0f / a->act_scale : 1.0f;
   p.out_scale = 1.0f;
-  p.out_dt = a->out_dtype;
-  if (a->wfmt == PT_W_BF16 && a->alpha != 0.f) p.out_scale = a->alpha;
+  if (a->wfmt == PT_W_BF16) p.dense = make_dense_out(a->out, p.out_ld, a->out_dtype, a->epilogue, a->alpha, a->ext);
   if (a->wfmt == PT_W_FP8) p.out_scale = (a->w_scale > 0.f ? a->w_scale : 1.0f) * (cast ? a->act_scale : 1.0f);
 
-  const SplitPlan plan = plan_split(a->wfmt, a->batch, a->n_out, a->k_in, a->ksplit);
+  int want_split = a->ksplit;
+  if (grouped) {
+    p.group_of = a->ext->group_of;
+    p.group_x_div = a->ext->group_x_div;
+    p.group_stride = pt_linear_packed_bytes(a->wfmt, a->n_out, a->k_in);
+    // as many warps in total as one matrix gets, and no more counters and partial sums than the workspace holds
+    if (want_split <= 0) want_split = std::max(1, std::min(sm_count() * 24 / (p.n_rt * a->batch), p.nchunks / 8));
+    while (want_split > 1 && (a->workspace_bytes < pt_linear_workspace_bytes(a->batch, a->n_out, want_split) || ceil_div(p.n_rt, kWarps) * a->batch > kMaxCounters))
+      --want_split;
+  }
+  const SplitPlan plan = plan_split(a->wfmt, p.B, a->n_out, a->k_in, want_split);
   PT_REQUIRE(plan.fits, "pt_linear: activation slice does not fit shared memory (batch=%d k=%d)", a->batch, a->k_in);
   p.chunks_per_split = plan.chunks_per_split;
   p.ksplit = plan.ksplit;
@@ -639,7 +664,7 @@ extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
     const size_t need = pt_linear_workspace_bytes(a->batch, a->n_out, p.ksplit);
     PT_REQUIRE(a->workspace && a->workspace_bytes >= need, "pt_linear: split-k=%d needs %zu workspace bytes, got %zu", p.ksplit, need,
                a->workspace_bytes);
-    PT_REQUIRE(ceil_div(p.n_rt, kWarps) <= kMaxCounters, "pt_linear: n_out=%d exceeds the %d arrival counters of a split-k workspace", a->n_out,
+    PT_REQUIRE(ceil_div(p.n_rt, kWarps) * (grouped ? a->batch : 1) <= kMaxCounters, "pt_linear: n_out=%d exceeds the %d arrival counters of a split-k workspace", a->n_out,
                kMaxCounters);
     p.counters = (int *)a->workspace;
     p.partial = (float *)((char *)a->workspace + kCounterBytes);

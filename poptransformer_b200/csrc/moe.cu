@@ -1,0 +1,164 @@
+// Mixture of experts: which experts a token goes to, and where its rows lie for the grouped products.
+//   choose   per token the `top` experts with the largest router logits (the lowest index first among equals), and the softmax over
+//            those logits as weights.  fp32.
+//   place    pair i = token i / top with its choice i % top gets a row of its own among its expert's rows.  The rows of an expert are
+//            padded to whole tiles; tile_expert names the expert of every tile (-1: unused), so a grouped product can look its weights
+//            up per tile.  Pairs keep their order within an expert.
+//   gather   the tokens' activations are copied to their pairs' rows (zeros in the padding).
+// With few tokens every pair is a tile of one row and nothing is placed or copied.
+#include <limits.h>
+
+#include "elem.cuh"
+
+namespace pt {
+namespace moe {
+
+constexpr int kMaxExperts = 1024, kMaxTop = 64, PLACE_THREADS = 1024;
+
+struct Params {
+  int n_tok, experts, top, logits_ld, tile, max_tiles;
+  const float *logits;
+  int *expert, *pair_row, *tile_expert, *row_token;   // [n_tok][top] x 2, [max_tiles], [max_tiles * tile]
+  float *weight;                                      // [n_tok][top]
+};
+
+// One warp per token; lane l holds the logits of experts l, l + 32, ...
+__global__ void choose_kernel(const Params p) {
+  const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= p.n_tok) return;
+  const float *z = p.logits + (size_t)t * p.logits_ld;
+  __shared__ float zs[4][kMaxExperts];
+  float *mine = zs[threadIdx.x >> 5];
+  for (int e = lane; e < p.experts; e += 32) mine[e] = z[e];
+  __syncwarp();
+  float first = 0.f, sum = 0.f, w0 = 0.f, w1 = 0.f;     // lane k keeps the weights of choices k and k + 32
+  for (int k = 0; k < p.top; ++k) {
+    float best = -INFINITY;
+    int at = INT_MAX;
+    for (int e = lane; e < p.experts; e += 32)
+      if (mine[e] > best) { best = mine[e]; at = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float b = __shfl_xor_sync(0xffffffffu, best, o);
+      const int a = __shfl_xor_sync(0xffffffffu, at, o);
+      if (b > best || (b == best && a < at)) { best = b; at = a; }
+    }
+    if (at == INT_MAX) at = k;                          // only infinities or NaN are left
+    if (k == 0) first = best;
+    const float w = expf(best - first);
+    sum += w;
+    if (lane == (k & 31)) {
+      (k < 32 ? w0 : w1) = w;
+      p.expert[(size_t)t * p.top + k] = at;
+      mine[at] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  if (lane < p.top) p.weight[(size_t)t * p.top + lane] = w0 / sum;
+  if (lane + 32 < p.top) p.weight[(size_t)t * p.top + lane + 32] = w1 / sum;
+}
+
+// Block e places the pairs of expert e: every block counts all experts' pairs (for the tiles in front of its own), then walks the pairs once more.
+__global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
+  __shared__ int count[kMaxExperts], warps[PLACE_THREADS / 32];
+  __shared__ int first, total;
+  const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, pairs = p.n_tok * p.top;
+  for (int i = tid; i < p.experts; i += PLACE_THREADS) count[i] = 0;
+  __syncthreads();
+  for (int i = tid; i < pairs; i += PLACE_THREADS) atomicAdd(&count[p.expert[i]], 1);
+  __syncthreads();
+  if (warp == 0) {
+    int before = 0, all = 0;
+    for (int i = lane; i < p.experts; i += 32) {
+      const int tiles = (count[i] + p.tile - 1) / p.tile;
+      all += tiles;
+      if (i < e) before += tiles;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      before += __shfl_xor_sync(0xffffffffu, before, o);
+      all += __shfl_xor_sync(0xffffffffu, all, o);
+    }
+    if (lane == 0) { first = before; total = all; }
+  }
+  __syncthreads();
+  const int mine = count[e], tiles = (mine + p.tile - 1) / p.tile, row0 = first * p.tile;
+  for (int i = tid; i < tiles; i += PLACE_THREADS) p.tile_expert[first + i] = e;
+  for (int i = mine + tid; i < tiles * p.tile; i += PLACE_THREADS) p.row_token[row0 + i] = -1;
+  if (e == 0) {
+    for (int i = total + tid; i < p.max_tiles; i += PLACE_THREADS) p.tile_expert[i] = -1;
+    for (int i = total * p.tile + tid; i < p.max_tiles * p.tile; i += PLACE_THREADS) p.row_token[i] = -1;
+  }
+  int next = row0;
+  for (int i0 = 0; i0 < pairs; i0 += PLACE_THREADS) {
+    const int i = i0 + tid;
+    const bool hit = i < pairs && p.expert[i] == e;
+    const unsigned vote = __ballot_sync(0xffffffffu, hit);
+    if (lane == 0) warps[warp] = __popc(vote);
+    __syncthreads();
+    int before = 0, all = 0;
+    for (int w = 0; w < PLACE_THREADS / 32; ++w) {
+      const int n = warps[w];
+      all += n;
+      if (w < warp) before += n;
+    }
+    if (hit) {
+      const int row = next + before + __popc(vote & ((1u << lane) - 1u));
+      p.pair_row[i] = row;
+      p.row_token[row] = i / p.top;
+    }
+    next += all;
+    __syncthreads();
+  }
+}
+
+// Rows of h (whole 16-byte units) to where row_token says.
+__global__ void gather_kernel(const uint4 *h, uint4 *out, int units, const int *row_token) {
+  const int tok = row_token[blockIdx.x];
+  uint4 *o = out + (size_t)blockIdx.x * units;
+  const uint4 *src = h + (size_t)max(tok, 0) * units;
+  for (int i = threadIdx.x; i < units; i += blockDim.x) o[i] = tok >= 0 ? src[i] : make_uint4(0, 0, 0, 0);
+}
+__global__ void gather4_kernel(const uint32_t *h, uint32_t *out, int units, const int *row_token) {
+  const int tok = row_token[blockIdx.x];
+  for (int i = threadIdx.x; i < units; i += blockDim.x) out[(size_t)blockIdx.x * units + i] = tok >= 0 ? h[(size_t)tok * units + i] : 0u;
+}
+
+}  // namespace moe
+}  // namespace pt
+
+using namespace pt;
+
+extern "C" int pt_moe_max_tiles(int n_tok, int experts, int top, int tile) {
+  const int pairs = n_tok * top, used = std::min(experts, pairs);     // every expert in use pads less than a tile
+  return (pairs + used * (tile - 1)) / tile;
+}
+
+extern "C" int pt_moe_route(const pt_moe_route_args *a, void *stream) {
+  PT_REQUIRE(a, "pt_moe_route: null args");
+  PT_REQUIRE(a->n_tok > 0 && a->experts > 0 && a->experts <= moe::kMaxExperts && a->top > 0 && a->top <= std::min(a->experts, moe::kMaxTop),
+             "pt_moe_route: %d tokens, %d of %d experts (at most %d of %d)", a->n_tok, a->top, a->experts, moe::kMaxTop, moe::kMaxExperts);
+  PT_REQUIRE((long long)a->n_tok * a->top < (1 << 28), "pt_moe_route: %d tokens x %d choices", a->n_tok, a->top);
+  PT_REQUIRE(a->logits && a->logits_ld >= a->experts && a->expert && a->weight, "pt_moe_route: null pointer argument");
+  moe::Params p{};
+  p.n_tok = a->n_tok; p.experts = a->experts; p.top = a->top; p.logits_ld = a->logits_ld; p.logits = a->logits; p.expert = a->expert; p.weight = a->weight;
+  cudaStream_t st = as_stream(stream);
+  moe::choose_kernel<<<ceil_div(p.n_tok, 4), 128, 0, st>>>(p);
+  PT_LAUNCH_CHECK("pt_moe_route");
+  if (!a->tile) return PT_OK;
+  PT_REQUIRE(a->tile > 0 && a->pair_row && a->tile_expert && a->row_token && a->max_tiles >= pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile),
+             "pt_moe_route: tiles of %d rows need pair_row, row_token and %d entries of tile_expert", a->tile, pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile));
+  p.tile = a->tile; p.max_tiles = a->max_tiles; p.pair_row = a->pair_row; p.tile_expert = a->tile_expert; p.row_token = a->row_token;
+  moe::place_kernel<<<p.experts, moe::PLACE_THREADS, 0, st>>>(p);
+  PT_LAUNCH_CHECK("pt_moe_route");
+  if (a->h) {
+    PT_REQUIRE(a->gathered && a->h_bytes > 0 && a->h_bytes % 4 == 0, "pt_moe_route: rows of %d bytes", a->h_bytes);
+    const int rows = a->max_tiles * a->tile;
+    if (a->h_bytes % 16 == 0 && aligned_to(a->h, 16) && aligned_to(a->gathered, 16))
+      moe::gather_kernel<<<rows, 128, 0, st>>>((const uint4 *)a->h, (uint4 *)a->gathered, a->h_bytes / 16, p.row_token);
+    else
+      moe::gather4_kernel<<<rows, 128, 0, st>>>((const uint32_t *)a->h, (uint32_t *)a->gathered, a->h_bytes / 4, p.row_token);
+    PT_LAUNCH_CHECK("pt_moe_route");
+  }
+  return PT_OK;
+}

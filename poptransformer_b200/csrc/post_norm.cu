@@ -1,0 +1,155 @@
+// Residual stream with norms on the sublayers' outputs only:
+//     x <- x + rms(y) * norm_w        and h = x in the activation type, the input of the next matrix product.
+// y may be a sum: a dense output plus a weighted sum over the experts a token went to (their rows lie where the router put them).
+// One launch does everything between two sublayers' matrix products.  The same kernel starts a token (x is its embedding row) and ends
+// the model (h = rms(x) * final_w for the output layer).  All of it is fp32; only h is rounded.
+#include "elem.cuh"
+
+namespace pt {
+namespace post {
+
+constexpr int kMaxTop = 64;
+
+struct Params {
+  int rows, width, h_ld, table_ld, vocab, ids_ld, y_ld, pair_ld, top;
+  float eps;
+  const float *x_in;
+  float *x_out;
+  const void *table;
+  const int *ids, *step;
+  int *pos_out, *id_out;
+  const int *row_index;
+  const float *y, *pair_y, *pair_w;
+  const int *pair_row;
+  const float *norm_w, *final_w;
+  void *h;
+};
+
+template <int VEC> __device__ __forceinline__ void put_f32(float *p, const float (&v)[VEC]) { store_vec<VEC>(p, v); }
+
+template <typename T, int VEC> __global__ void post_norm_kernel(const Params p) {
+  extern __shared__ __align__(16) float row[];     // [width]: y, then the new x
+  __shared__ float red[32], pw[kMaxTop];
+  __shared__ int pr[kMaxTop];
+  const int r = blockIdx.x, src = p.row_index ? p.row_index[r] : r, tid = threadIdx.x;
+  float *xo = p.x_out ? p.x_out + (size_t)r * p.width : nullptr;
+  T *hrow = p.h ? reinterpret_cast<T *>(p.h) + (size_t)r * p.h_ld : nullptr;
+  if (hrow)
+    for (int i = p.width + tid; i < p.h_ld; i += blockDim.x) hrow[i] = from_f<T>(0.f);     // k padding of the next product
+  if (p.table) {
+    const int step = p.step ? *p.step : 0;
+    const int id = min(max(p.ids[(size_t)src * p.ids_ld + step], 0), p.vocab - 1);
+    const T *emb = reinterpret_cast<const T *>(p.table) + (size_t)id * p.table_ld;
+    if (tid == 0) {
+      if (p.pos_out) p.pos_out[r] = step;
+      if (p.id_out) p.id_out[r] = id;
+    }
+    for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
+      float v[VEC];
+      load_vec<VEC>(emb + i, v);
+      put_f32<VEC>(xo + i, v);
+      if (hrow) store_vec<VEC>(hrow + i, v);
+    }
+    return;
+  }
+  if (tid < p.top) {
+    const size_t k = (size_t)src * p.top + tid;
+    pw[tid] = p.pair_w[k];
+    pr[tid] = p.pair_row ? p.pair_row[k] : (int)k;
+  }
+  __syncthreads();
+  const float *x = p.x_in + (size_t)src * p.width;
+  float ss = 0.f;
+  for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
+    float v[VEC];
+    if (p.y) {
+      load_vec<VEC>(p.y + (size_t)src * p.y_ld + i, v);
+    } else {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+    }
+#pragma unroll 4
+    for (int k = 0; k < p.top; ++k) {
+      float e[VEC];
+      load_vec<VEC>(p.pair_y + (size_t)pr[k] * p.pair_ld + i, e);
+      const float w = pw[k];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] = fmaf(w, e[j], v[j]);
+    }
+    put_f32<VEC>(row + i, v);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+  ss = 0.f;
+  for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
+    float v[VEC], w[VEC], o[VEC];
+    load_vec<VEC>(row + i, v);
+    load_vec<VEC>(p.norm_w + i, w);
+    load_vec<VEC>(x + i, o);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      o[j] += v[j] * inv * w[j];
+      ss = fmaf(o[j], o[j], ss);
+    }
+    if (xo) put_f32<VEC>(xo + i, o);
+    if (p.final_w) put_f32<VEC>(row + i, o);
+    else if (hrow) store_vec<VEC>(hrow + i, o);
+  }
+  if (!p.final_w || !hrow) return;
+  const float end = 1.0f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+  for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
+    float v[VEC], w[VEC];
+    load_vec<VEC>(row + i, v);
+    load_vec<VEC>(p.final_w + i, w);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] *= end * w[j];
+    store_vec<VEC>(hrow + i, v);
+  }
+}
+
+template <typename T, int VEC> static int launch(const Params &p, cudaStream_t st) {
+  const size_t smem = (size_t)p.width * sizeof(float);
+  if (smem > 48 * 1024) {
+    static bool set = false;
+    if (!set) { PT_CUDA(cudaFuncSetAttribute(post_norm_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
+  }
+  // few rows: as many threads per row as it has work for; many rows: more rows per SM
+  const int want = ceil_div(ceil_div(p.width, VEC), 32) * 32, cap = p.rows <= 2 * sm_count() ? 1024 : 256;
+  post_norm_kernel<T, VEC><<<p.rows, std::max(64, std::min(want, cap)), smem, st>>>(p);
+  PT_LAUNCH_CHECK("pt_post_norm");
+  return PT_OK;
+}
+
+}  // namespace post
+}  // namespace pt
+
+using namespace pt;
+
+extern "C" int pt_post_norm(const pt_post_norm_args *a, void *stream) {
+  PT_REQUIRE(a, "pt_post_norm: null args");
+  PT_REQUIRE(a->rows > 0 && a->width > 0 && a->width <= 48 * 1024, "pt_post_norm: bad shape rows=%d width=%d", a->rows, a->width);
+  PT_REQUIRE(a->dtype == PT_DT_F32 || a->dtype == PT_DT_BF16, "pt_post_norm: activation type %d (fp32 or bf16)", a->dtype);
+  PT_REQUIRE(!a->h || a->h_ld >= a->width, "pt_post_norm: h_ld=%d", a->h_ld);
+  if (a->table) {
+    PT_REQUIRE(a->ids && a->vocab > 0 && a->table_ld >= a->width && a->ids_ld >= 1 && a->x_out, "pt_post_norm: an embedding start needs ids, vocab, table_ld and x_out");
+  } else {
+    PT_REQUIRE(a->x_in && a->norm_w && (a->y || a->top > 0), "pt_post_norm: null x, norm weight or sublayer output");
+    PT_REQUIRE(!a->y || a->y_ld >= a->width, "pt_post_norm: y_ld=%d", a->y_ld);
+    PT_REQUIRE(a->top >= 0 && a->top <= post::kMaxTop && (!a->top || (a->pair_y && a->pair_w && a->pair_ld >= a->width)),
+               "pt_post_norm: %d experts per token (at most %d) need pair_y, pair_w and pair_ld", a->top, post::kMaxTop);
+  }
+  post::Params p{};
+  p.rows = a->rows; p.width = a->width; p.h_ld = a->h_ld; p.table_ld = a->table_ld; p.vocab = a->vocab; p.ids_ld = a->ids_ld; p.y_ld = a->y_ld;
+  p.pair_ld = a->pair_ld; p.top = a->table ? 0 : a->top; p.eps = a->eps;
+  p.x_in = a->x_in; p.x_out = a->x_out; p.table = a->table; p.ids = a->ids; p.step = a->step_dev; p.pos_out = a->pos_out; p.id_out = a->id_out;
+  p.row_index = a->row_index; p.y = a->y; p.pair_y = a->pair_y; p.pair_w = a->pair_w; p.pair_row = a->pair_row;
+  p.norm_w = a->norm_w; p.final_w = a->final_w; p.h = a->h;
+  const int vb = a->dtype == PT_DT_F32 ? 16 : 8;
+  const bool v4 = a->width % 4 == 0 && aligned_to(a->x_in, 16) && aligned_to(a->x_out, 16) && aligned_to(a->y, 16) && a->y_ld % 4 == 0 && aligned_to(a->pair_y, 16) &&
+                  a->pair_ld % 4 == 0 && aligned_to(a->norm_w, 16) && aligned_to(a->final_w, 16) && aligned_to(a->h, vb) && a->h_ld % 4 == 0 && aligned_to(a->table, vb) &&
+                  a->table_ld % 4 == 0;
+  cudaStream_t st = as_stream(stream);
+  if (a->dtype == PT_DT_F32) return v4 ? post::launch<float, 4>(p, st) : post::launch<float, 1>(p, st);
+  return v4 ? post::launch<__nv_bfloat16, 4>(p, st) : post::launch<__nv_bfloat16, 1>(p, st);
+}

@@ -16,8 +16,7 @@
 //   ssm_norm_kernel    gate, group norm, and the ring update
 #include <type_traits>
 
-#include "elem.cuh"
-#include "tile_math.cuh"
+#include "chunk.cuh"
 
 namespace pt {
 namespace ssm {
@@ -196,33 +195,9 @@ template <typename T> __global__ void __launch_bounds__(SCAN_WARPS * 32) ssm_sca
 //   ssm_chunk_state_kernel   the sum of the second line, per chunk and head
 //   ssm_carry_kernel         the second line along the chunks: leaves the state BEFORE every chunk in place of its sum
 //   ssm_chunk_out_kernel     the first line, per chunk and head
-// Chunk ci of sequence s lives in slot cu[s] / 64 + s + ci of the scratch (distinct, below n_tok / 64 + n_seq).  Operands that are
-// not already bf16 (the state, the decayed products, the weighted x) enter the tensor cores as hi + lo pairs.  c is kept as a pair
+// Operands that are not already bf16 (the state, the decayed products, the weighted x) enter the tensor cores as hi + lo pairs.  c is kept as a pair
 // of floats, so differences of neighbours stay exact however far the sum has run.
 // NP: state size rounded up to 64, 128 or 256, CP: columns of a head per block (padding is zero).
-constexpr int CHUNK = 64, CHUNK_THREADS = 256;
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ int chunk_slot(const Params &p, int s) { return p.cu[s] / CHUNK + s; }
-// Sequence and first token (within it) of a scratch slot; false for a slot that no chunk uses.
-__device__ __forceinline__ bool chunk_of_slot(const Params &p, int slot, int &s, int &t0) {
-  int lo = 0, hi = p.n_seq - 1;
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) / 2;
-    if (chunk_slot(p, mid) <= slot) lo = mid;
-    else hi = mid - 1;
-  }
-  s = lo;
-  t0 = (slot - chunk_slot(p, lo)) * CHUNK;
-  return t0 < p.cu[lo + 1] - p.cu[lo];
-}
 struct __align__(16) Decays {
   float c_hi[CHUNK], c_lo[CHUNK], dt[CHUNK], ec[CHUNK], w[CHUNK];   // ec = exp(c_t), w = exp(c_last - c_s) dt_s
   float keep, pad[3];                                               // exp(c_last)
@@ -257,7 +232,7 @@ __device__ __forceinline__ void scan_decays(const Params &p, int row0, int valid
 __global__ void ssm_decay_kernel(const Params p) {   // one warp per (chunk, head)
   const int slot = blockIdx.y, h = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   int s, t0;
-  if (h >= p.heads || !chunk_of_slot(p, slot, s, t0)) return;
+  if (h >= p.heads || !chunk_of_slot(p.cu, p.n_seq, slot, s, t0)) return;
   const int row0 = p.cu[s] + t0;
   scan_decays(p, row0, min(CHUNK, p.cu[s + 1] - row0), h, p.chunk_decays[(size_t)slot * p.heads + h]);
 }
@@ -279,7 +254,7 @@ template <int NP, int CP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_c
   StateSmem<NP, CP> &sm = *reinterpret_cast<StateSmem<NP, CP> *>(smraw);
   const int slot = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * CP;
   int s, t0;
-  if (!chunk_of_slot(p, slot, s, t0)) return;
+  if (!chunk_of_slot(p.cu, p.n_seq, slot, s, t0)) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
   const int grp = h / (p.heads / p.groups), row0 = p.cu[s] + t0, valid = min(CHUNK, p.cu[s + 1] - row0);
   const T *xbc = reinterpret_cast<const T *>(p.xbc) + (size_t)row0 * p.C;
@@ -353,8 +328,8 @@ __global__ void ssm_carry_kernel(const Params p) {
   if (i >= n) return;
   const int chunks = (p.cu[s + 1] - p.cu[s] + CHUNK - 1) / CHUNK;
   const size_t stride = (size_t)p.heads * n;
-  float *x = p.chunk_state + (size_t)chunk_slot(p, s) * stride + (size_t)h * n + i;
-  const Decays *dec = p.chunk_decays + (size_t)chunk_slot(p, s) * p.heads + h;
+  float *x = p.chunk_state + (size_t)chunk_slot(p.cu, s) * stride + (size_t)h * n + i;
+  const Decays *dec = p.chunk_decays + (size_t)chunk_slot(p.cu, s) * p.heads + h;
   float *state = p.state + ((size_t)p.slot[s] * p.heads + h) * n + i;
   float cur[8];
 #pragma unroll
@@ -409,7 +384,7 @@ template <int NP, int CP> __global__ void __launch_bounds__(CHUNK_THREADS) ssm_c
   OutSmem<NP, CP> &sm = *reinterpret_cast<OutSmem<NP, CP> *>(smraw);
   const int slot = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * CP;
   int s, t0;
-  if (!chunk_of_slot(p, slot, s, t0)) return;
+  if (!chunk_of_slot(p.cu, p.n_seq, slot, s, t0)) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
   const int grp = h / (p.heads / p.groups), row0 = p.cu[s] + t0, valid = min(CHUNK, p.cu[s + 1] - row0);
   const T *xbc = reinterpret_cast<const T *>(p.xbc) + (size_t)row0 * p.C;
@@ -661,8 +636,6 @@ template <typename T, int VEC> __global__ void ssm_norm_kernel(const Params p) {
   for (int i = p.inner + tid; i < p.out_ld; i += blockDim.x) out[i] = from_f<T>(0.f);   // k padding of the output product
 }
 
-static bool al(const void *q, int bytes) { return ((uintptr_t)q & (bytes - 1)) == 0; }
-
 template <int NP, int CP> static int launch_chunks(const Params &p, cudaStream_t st) {
   static bool set = false;
   if (!set) {
@@ -687,7 +660,7 @@ template <int CP> static int dispatch_chunks(const Params &p, cudaStream_t st) {
 
 template <typename T> static int run(const Params &p, bool plain, cudaStream_t st) {
   if (p.n_tok == p.n_seq) {
-    const bool v4 = p.P % 4 == 0 && p.P / 4 <= STEP_THREADS && al(p.state, 16);
+    const bool v4 = p.P % 4 == 0 && p.P / 4 <= STEP_THREADS && aligned_to(p.state, 16);
     const int pq = v4 ? p.P / 4 : p.P, ng = std::max(1, STEP_THREADS / pq);
     const size_t smem = ((size_t)(p.P + 2 * p.N + 3) / 4 * 4 + (size_t)ng * p.P) * sizeof(float);
     PT_REQUIRE(smem <= 48 * 1024, "pt_ssm: head width %d and state %d need %zu bytes of shared memory", p.P, p.N, smem);
@@ -696,7 +669,7 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
     else ssm_step_kernel<T, 1><<<grid, STEP_THREADS, smem, st>>>(p);
     PT_LAUNCH_CHECK("pt_ssm");
   } else {
-    if (!plain && sizeof(T) == 2 && p.taps <= 4 && p.C % 8 == 0 && p.inner % 8 == 0 && p.zx_ld % 8 == 0 && al(p.zx, 16) && al(p.xbc, 16) && al(p.ring, 16) && al(p.conv_w, 16)) {
+    if (!plain && sizeof(T) == 2 && p.taps <= 4 && p.C % 8 == 0 && p.inner % 8 == 0 && p.zx_ld % 8 == 0 && aligned_to(p.zx, 16) && aligned_to(p.xbc, 16) && aligned_to(p.ring, 16) && aligned_to(p.conv_w, 16)) {
       const dim3 grid(ceil_div(p.C / 8, CONV_THREADS) + 1, ceil_div(p.n_tok, CONV_TOKENS));
       switch (p.taps) {
         case 1: ssm_conv8_kernel<1><<<grid, CONV_THREADS, 0, st>>>(p); break;
@@ -709,7 +682,7 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
     }
     PT_LAUNCH_CHECK("pt_ssm");
     // the chunked form: bf16, rows that are whole 16-byte units, state of at most 256, with its scratch
-    if (!plain && sizeof(T) == 2 && p.chunk_state && al(p.state, 16) && p.N <= 256 && p.N % 8 == 0 && p.P % 8 == 0 && al(p.xbc, 16) && al(p.y, 8)) {
+    if (!plain && sizeof(T) == 2 && p.chunk_state && aligned_to(p.state, 16) && p.N <= 256 && p.N % 8 == 0 && p.P % 8 == 0 && aligned_to(p.xbc, 16) && aligned_to(p.y, 8)) {
       const int rc = p.P <= 32 ? dispatch_chunks<32>(p, st) : dispatch_chunks<64>(p, st);
       if (rc != PT_OK) return rc;
     } else {
@@ -721,8 +694,8 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
     }
   }
   const int len = p.inner / p.norm_groups;
-  const bool v4 = len % 4 == 0 && p.C % 4 == 0 && p.zx_ld % 4 == 0 && p.out_ld % 4 == 0 && al(p.out, 4 * sizeof(T)) && al(p.zx, 4 * sizeof(T)) &&
-                  al(p.ring, 4 * sizeof(T)) && al(p.y, 16) && al(p.norm_w, 16);
+  const bool v4 = len % 4 == 0 && p.C % 4 == 0 && p.zx_ld % 4 == 0 && p.out_ld % 4 == 0 && aligned_to(p.out, 4 * sizeof(T)) && aligned_to(p.zx, 4 * sizeof(T)) &&
+                  aligned_to(p.ring, 4 * sizeof(T)) && aligned_to(p.y, 16) && aligned_to(p.norm_w, 16);
   // few rows: as many threads per row as it has work for (the launch is one chain of latencies); many rows: more rows per SM
   const int threads = p.n_tok <= 2 * sm_count() ? std::min(1024, std::max(128, ceil_div(p.inner / (v4 ? 4 : 1), 32) * 32)) : 256;
   const size_t smem = ((size_t)(p.inner + 3) / 4 * 4 + (size_t)std::max(p.norm_groups, threads / 32)) * sizeof(float);
@@ -743,7 +716,7 @@ template <typename T> static int run(const Params &p, bool plain, cudaStream_t s
 using namespace pt;
 
 extern "C" size_t pt_ssm_workspace_bytes(int n_tok, int n_seq, int heads, int vdim, int state_dim) {
-  const size_t slots = (size_t)n_tok / ssm::CHUNK + n_seq;
+  const size_t slots = (size_t)n_tok / CHUNK + n_seq;
   return slots * heads * ((size_t)state_dim * vdim * sizeof(float) + sizeof(ssm::Decays)) + 16;
 }
 
@@ -769,7 +742,7 @@ extern "C" int pt_ssm(const pt_ssm_args *a, void *stream) {
   p.ring = a->ring; p.xbc = a->xbc; p.out = a->out; p.state = a->state; p.dt = a->dt; p.y = a->y;
   if (a->workspace && ((uintptr_t)a->workspace & 15) == 0 && a->workspace_bytes >= pt_ssm_workspace_bytes(b.n_tok, b.n_seq, a->heads, a->vdim, a->state_dim)) {
     p.chunk_state = (float *)a->workspace;
-    const size_t n = ((size_t)b.n_tok / ssm::CHUNK + b.n_seq) * a->heads * a->state_dim * a->vdim;
+    const size_t n = ((size_t)b.n_tok / CHUNK + b.n_seq) * a->heads * a->state_dim * a->vdim;
     p.chunk_decays = (ssm::Decays *)(p.chunk_state + (n + 3) / 4 * 4);
   }
   return a->dtype == PT_DT_F32 ? ssm::run<float>(p, a->plain != 0, as_stream(stream)) : ssm::run<__nv_bfloat16>(p, a->plain != 0, as_stream(stream));

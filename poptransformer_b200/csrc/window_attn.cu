@@ -1,20 +1,20 @@
 // Masked attention over a paged cache with per-sequence positions: a sliding window, kept first tokens, a softmax sink, grouped
-// heads, key and value widths of their own, no rotation.  Position i sees key j when j <= i and (i - j < window or j < keep_first);
+// heads, key and value widths of their own, optionally a norm and a rotation of every query and key head.  Position i sees key j when j <= i and (i - j < window or j < keep_first);
 // window = 0 means every earlier key.  sink[h] acts as one more logit of head h that brings weight to the denominator only.
 //
 // The tokens of a launch are packed sequence after sequence (pt_batch_view): row cu[s] + i is position start[s] + i of sequence s,
 // whose pages are page_table[slot[s]].  A page holds K [n_kv][page][dim] and then V [n_kv][page][vdim].  New keys and values are
 // appended first; a layer that shares another layer's cache passes none and reads what is there.
 //
+//   attn_prep_kernel    norm and rotation of a prompt's queries and keys, and the append
 //   attn_plain_kernel   any sizes, fp32 or bf16 caches, CUDA cores: the 32-bit path and the shapes the others do not take
 //   attn_prompt_kernel  bf16 prompts: 64 queries of one head per block, Q K^T and P V on the tensor cores, online softmax; only key
 //                       tiles that hold a visible key are touched
 //   attn_decode_kernel  bf16, one token per sequence: one block per (visible page, kv head, sequence), scores and P V on the tensor
-//                       cores, pages combined by the last block to arrive; the append is fused
+//                       cores, pages combined by the last block to arrive; norm, rotation and append are fused
 // Scores, softmax and weights are fp32.  The tensor-core kernels multiply V with weights split into two bf16 parts (hi + lo), which
 // keeps 16 significant bits of each weight.
-#include "elem.cuh"
-#include "tile_math.cuh"
+#include "chunk.cuh"
 
 namespace pt {
 namespace wa {
@@ -30,6 +30,11 @@ struct Params {
   void *pool, *out;
   const int *page_table, *cu, *start, *slot, *tok_seq;
   int *error_flag;
+  const float *q_norm, *k_norm;
+  const float2 *rope;        // [positions][rope_half]
+  float norm_eps, out_scale;
+  int rope_half, out_cols;
+  bool prep;                 // queries and keys are normalised or rotated
   // decode
   int grid_pages, qsplit;
   float *ws_o;      // [n_seq, n_head, grid_pages, vdim]
@@ -52,7 +57,52 @@ __device__ __forceinline__ int window_page(const Params &p, int pos) { return p.
 // Pages that hold the kept first tokens (as far as they exist at position pos).
 __device__ __forceinline__ int kept_pages(const Params &p, int pos) { return (min(p.keep_first, pos + 1) + p.page - 1) / p.page; }
 
-// ------------------------------------------------------------------------------------------ append
+// ------------------------------------------------------------------------------------------ norm, rotation, append
+// One warp: a head's row of a query or key.  put(i, value) may write over src (a lane reads what it writes).
+template <typename T, typename Put>
+__device__ __forceinline__ void norm_rotate(const Params &p, const T *src, const float *norm, int pos, Put put) {
+  const int lane = threadIdx.x & 31;
+  float inv = 1.f;
+  if (norm) {
+    float ss = 0.f;
+    for (int i = lane; i < p.dim; i += 32) {
+      const float x = to_f(src[i]);
+      ss = fmaf(x, x, ss);
+    }
+    inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.norm_eps);
+  }
+  auto at = [&](int i) { return to_f(src[i]) * inv * (norm ? __ldg(norm + i) : 1.f); };
+  const float2 *cs = p.rope + (size_t)pos * p.rope_half;
+  for (int i = lane; i < p.rope_half; i += 32) {
+    const float u = at(i), v = at(i + p.rope_half);
+    const float2 c = __ldg(cs + i);
+    put(i, u * c.x - v * c.y);
+    put(i + p.rope_half, v * c.x + u * c.y);
+  }
+  for (int i = 2 * p.rope_half + lane; i < p.dim; i += 32) put(i, at(i));
+}
+
+constexpr int PREP_WARPS = 4;
+template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const Params p) {   // warp: one token, one query or key head
+  const int t = blockIdx.y, h = blockIdx.x * PREP_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
+  if (h >= p.n_head + (p.k ? p.n_kv : 0)) return;
+  if (pos < 0 || pos >= p.max_len) {
+    if (lane == 0 && p.error_flag) atomicExch(p.error_flag, 12);
+    return;
+  }
+  if (h < p.n_head) {
+    T *q = reinterpret_cast<T *>(const_cast<void *>(p.q)) + (size_t)t * p.q_ld + (size_t)h * p.dim;
+    norm_rotate<T>(p, q, p.q_norm, pos, [&](int i, float y) { q[i] = from_f<T>(y); });
+    return;
+  }
+  const int g = h - p.n_head, phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page], at = pos % p.page;
+  const T *k = reinterpret_cast<const T *>(p.k) + (size_t)t * p.kv_ld + (size_t)g * p.dim, *v = reinterpret_cast<const T *>(p.v) + (size_t)t * p.kv_ld + (size_t)g * p.vdim;
+  T *kc = k_page<T>(p, phys, g) + (size_t)at * p.dim, *vc = v_page<T>(p, phys, g) + (size_t)at * p.vdim;
+  norm_rotate<T>(p, k, p.k_norm, pos, [&](int i, float y) { kc[i] = from_f<T>(y); });
+  for (int i = lane; i < p.vdim; i += 32) vc[i] = v[i];
+}
+
 template <typename T> __global__ void kv_append_kernel(const Params p) {
   const int t = blockIdx.x, s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
   if (pos < 0 || pos >= p.max_len) {
@@ -128,21 +178,13 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
     }
   }
   T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld + (size_t)g * p.qpk * p.vdim;
-  for (int i = tid; i < p.qpk * p.vdim; i += PLAIN_THREADS) out[i] = from_f<T>(o[i] / st[3 * (i / p.vdim) + 1]);
+  for (int i = tid; i < p.qpk * p.vdim; i += PLAIN_THREADS) out[i] = from_f<T>(o[i] / st[3 * (i / p.vdim) + 1] * p.out_scale);
   if (g == p.n_kv - 1)   // k padding of the output product
-    for (int i = p.n_head * p.vdim + tid; i < p.out_ld; i += PLAIN_THREADS) reinterpret_cast<T *>(p.out)[(size_t)t * p.out_ld + i] = from_f<T>(0.f);
+    for (int i = p.n_head * p.vdim + tid; i < p.out_cols; i += PLAIN_THREADS) reinterpret_cast<T *>(p.out)[(size_t)t * p.out_ld + i] = from_f<T>(0.f);
 }
 
 // ------------------------------------------------------------------------------------------ tensor cores
 constexpr int TC_THREADS = 128, TILE = 64;   // TILE = the page size the tensor-core kernels take
-
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t &r0, uint32_t &r1, uint32_t &r2, uint32_t &r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-// 16-byte asynchronous copy; zeros instead of the source when !in (the source address is then not read).
-__device__ __forceinline__ void cp16(void *dst, const void *src, bool in) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
-}
 
 // ------------------------------------------------------------------------------------------ prompts
 // Block: 64 new tokens of one sequence, one head; warp w owns queries 16 w .. 16 w + 15, their q fragments stay in registers.  Key
@@ -273,7 +315,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_pro
 #pragma unroll
         for (int jn = 0; jn < DV / 8; jn += 2) {
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(v_lane + (uint32_t)(k2 * 16 * VLD + jn * 8) * 2u, b0, b1, b2, b3);
+          ldsm4t(v_lane + (uint32_t)(k2 * 16 * VLD + jn * 8) * 2u, b0, b1, b2, b3);
           mma16816_bf16(o[jn], h[0], h[1], h[2], h[3], b0, b1);
           mma16816_bf16(o[jn + 1], h[0], h[1], h[2], h[3], b2, b3);
           mma16816_bf16(o[jn], l[0], l[1], l[2], l[3], b0, b1);
@@ -291,7 +333,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_pro
     l += __shfl_xor_sync(0xffffffffu, l, 1);
     l += __shfl_xor_sync(0xffffffffu, l, 2);
     if (p.sink) l += exp2f(sink2 - m_run[r]);                   // the sink, in the units of the running maximum
-    inv[r] = 1.0f / l;
+    inv[r] = p.out_scale / l;
   }
   __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(p.out) + (size_t)head * p.vdim + 2 * tig;
 #pragma unroll
@@ -300,7 +342,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_pro
     if (ok0) *reinterpret_cast<uint32_t *>(out + (size_t)(row0 + q0) * p.out_ld + j * 8) = pack_bf2(o[j][0] * inv[0], o[j][1] * inv[0]);
     if (ok1) *reinterpret_cast<uint32_t *>(out + (size_t)(row0 + q1) * p.out_ld + j * 8) = pack_bf2(o[j][2] * inv[1], o[j][3] * inv[1]);
   }
-  const int pad = p.out_ld - p.n_head * p.vdim;
+  const int pad = p.out_cols - p.n_head * p.vdim;
   if (head == p.n_head - 1)
     for (int i = tid; i < TILE * pad; i += TC_THREADS) {
       const int r = t0 + i / pad;
@@ -323,7 +365,8 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
   T *qs = Vs + TILE * VLD;                                     // [NQ][QLD]
   float *ps = reinterpret_cast<float *>(qs + NQ * QLD);        // [NQ][PSLD]
   float *ml = ps + NQ * PSLD;                                  // [NQ][2]
-  float *cw = ml + NQ * 2;                                     // combine: [NQ][grid_pages] weights
+  T *kn = reinterpret_cast<T *>(ml + NQ * 2);                  // [DK] the newest key, normalised and rotated
+  float *cw = reinterpret_cast<float *>(kn + DK);              // combine: [NQ][grid_pages] weights
   __shared__ int s_last;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
   const int s = blockIdx.z, kvh = blockIdx.y / p.qsplit, part = blockIdx.y - kvh * p.qsplit;
@@ -356,7 +399,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
       uint4 v = make_uint4(0, 0, 0, 0);
       if (c < p.dim) {
         if (key < n_load) v = __ldcg(reinterpret_cast<const uint4 *>(gK + (size_t)key * p.dim + c));
-        else if (owner && key == at) v = *reinterpret_cast<const uint4 *>(knew + c);
+        else if (owner && !p.prep && key == at) v = *reinterpret_cast<const uint4 *>(knew + c);
       }
       kf[r][pp] = v;
     }
@@ -369,17 +412,35 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * p.dim;
-  for (int i = tid; i < NQ * (DK / 8); i += TC_THREADS) {
+  if (p.prep) {
+    for (int h = warp; h < NQ + 1; h += TC_THREADS / 32) {
+      T *dst = h < NQ ? qs + h * QLD : kn;
+      const bool have = h < NQ ? h < nq : owner;
+      if (have) norm_rotate<T>(p, h < NQ ? q + (size_t)h * p.dim : knew, h < NQ ? p.q_norm : p.k_norm, pos, [&](int i, float y) { dst[i] = from_f<T>(y); });
+      for (int i = (have ? p.dim : 0) + lane; i < DK; i += 32) dst[i] = from_f<T>(0.f);
+    }
+  } else for (int i = tid; i < NQ * (DK / 8); i += TC_THREADS) {
     const int h = i / (DK / 8), c = (i % (DK / 8)) * 8;
     *reinterpret_cast<uint4 *>(qs + h * QLD + c) = (h < nq && c < p.dim) ? *reinterpret_cast<const uint4 *>(q + (size_t)h * p.dim + c) : make_uint4(0, 0, 0, 0);
   }
   for (int i = tid; i < NQ * PSLD; i += TC_THREADS) ps[i] = -INFINITY;
   if (owner && part == 0) {
-    for (int c = tid; c < p.dim; c += TC_THREADS) gK[(size_t)at * p.dim + c] = knew[c];
+    if (!p.prep)
+      for (int c = tid; c < p.dim; c += TC_THREADS) gK[(size_t)at * p.dim + c] = knew[c];
     for (int c = tid; c < p.vdim; c += TC_THREADS) gV[(size_t)at * p.vdim + c] = vnew[c];
   }
   asm volatile("cp.async.wait_all;" ::: "memory");
   __syncthreads();
+  if (owner && p.prep) {
+    if (part == 0)
+      for (int c = tid; c < p.dim; c += TC_THREADS) gK[(size_t)at * p.dim + c] = kn[c];
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (warp * 16 + g + 8 * r == at) {
+#pragma unroll
+        for (int pp = 0; pp < DK / 32; ++pp) kf[r][pp] = *reinterpret_cast<const uint4 *>(kn + pp * 32 + tig * 8);
+      }
+  }
 
   if (warp * 16 < n_valid) {
     float sc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -427,7 +488,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
 #pragma unroll
       for (int j = 0; j < NT; j += 2) {
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(v_lane + (uint32_t)(k2 * 16 * VLD + j * 8) * 2u, b0, b1, b2, b3);
+        ldsm4t(v_lane + (uint32_t)(k2 * 16 * VLD + j * 8) * 2u, b0, b1, b2, b3);
         mma16816_bf16(o[j], a0, a1, a2, a3, b0, b1);
         if (j + 1 < NT) mma16816_bf16(o[j + 1], a0, a1, a2, a3, b2, b3);
       }
@@ -466,7 +527,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
       l += v.y * w;
     }
     l = warp_sum(l);
-    if (lane == 0) ml[2 * h] = 1.0f / (l + (p.sink ? exp2f(sink2 - m) : 0.f));
+    if (lane == 0) ml[2 * h] = p.out_scale / (l + (p.sink ? exp2f(sink2 - m) : 0.f));
   }
   __syncthreads();
   T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld;
@@ -486,7 +547,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
     out[(size_t)(h0 + h) * p.vdim + c] = from_f<T>(acc * ml[2 * h]);
   }
   if (h0 + nq == p.n_head)
-    for (int i = p.n_head * p.vdim + tid; i < p.out_ld; i += TC_THREADS) out[i] = from_f<T>(0.f);
+    for (int i = p.n_head * p.vdim + tid; i < p.out_cols; i += TC_THREADS) out[i] = from_f<T>(0.f);
 }
 
 template <int DK, int DV> static int launch_prompt(const Params &p, int longest, cudaStream_t st) {
@@ -498,7 +559,7 @@ template <int DK, int DV> static int launch_prompt(const Params &p, int longest,
   return PT_OK;
 }
 template <int DK, int DV> static int launch_decode(const Params &p, cudaStream_t st) {
-  const size_t smem = (size_t)(TILE * (DV + 8) + NQ * (DK + 32)) * sizeof(__nv_bfloat16) + (size_t)(NQ * (TILE + 8) + NQ * 2 + NQ * p.grid_pages) * sizeof(float);
+  const size_t smem = (size_t)(TILE * (DV + 8) + NQ * (DK + 32) + DK) * sizeof(__nv_bfloat16) + (size_t)(NQ * (TILE + 8) + NQ * 2 + NQ * p.grid_pages) * sizeof(float);
   PT_REQUIRE(smem <= 200 * 1024, "pt_window_attn: %d pages per sequence need %zu bytes of shared memory", p.grid_pages, smem);
   static bool set = false;
   if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
@@ -555,6 +616,13 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
   p.q_ld = a->q_ld; p.kv_ld = a->kv_ld; p.out_ld = a->out_ld; p.scale = a->scale; p.sink = a->sink;
   p.q = a->q; p.k = a->k; p.v = a->v; p.pool = a->pool; p.out = a->out; p.page_table = a->page_table;
   p.cu = b.cu; p.start = b.start; p.slot = b.slot; p.tok_seq = b.tok_seq; p.error_flag = a->error_flag;
+  p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.norm_eps = a->norm_eps; p.rope = (const float2 *)a->rope; p.rope_half = a->rope_dims / 2;
+  p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.0f;
+  p.out_cols = a->out_cols > 0 ? a->out_cols : a->out_ld;
+  p.prep = a->q_norm || a->k_norm || a->rope_dims;
+  PT_REQUIRE(a->rope_dims >= 0 && a->rope_dims % 2 == 0 && a->rope_dims <= a->dim && (!a->rope_dims || a->rope), "pt_window_attn: %d rotated dimensions of %d",
+             a->rope_dims, a->dim);
+  PT_REQUIRE(p.out_cols >= a->n_head * a->vdim && p.out_cols <= a->out_ld, "pt_window_attn: out_cols=%d", a->out_cols);
   p.max_len = a->max_len > 0 ? a->max_len : a->page_size * a->max_pages;
   PT_REQUIRE(p.max_len <= a->page_size * a->max_pages, "pt_window_attn: max_len=%d exceeds the %d positions of the page table", p.max_len,
              a->page_size * a->max_pages);
@@ -579,7 +647,13 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
     p.ws_o = (float *)ws;
     return wa::dispatch_tc(p, true, 1, st);
   }
-  if (p.k) {
+  if (p.prep) {
+    PT_REQUIRE(b.n_tok <= 65535, "pt_window_attn: %d tokens", b.n_tok);
+    const dim3 grid(ceil_div(a->n_head + (p.k ? a->n_kv : 0), wa::PREP_WARPS), b.n_tok);
+    if (a->dtype == PT_DT_F32) wa::attn_prep_kernel<float><<<grid, wa::PREP_WARPS * 32, 0, st>>>(p);
+    else wa::attn_prep_kernel<__nv_bfloat16><<<grid, wa::PREP_WARPS * 32, 0, st>>>(p);
+    PT_LAUNCH_CHECK("pt_window_attn");
+  } else if (p.k) {
     if (a->dtype == PT_DT_F32) wa::kv_append_kernel<float><<<b.n_tok, 128, 0, st>>>(p);
     else wa::kv_append_kernel<__nv_bfloat16><<<b.n_tok, 128, 0, st>>>(p);
     PT_LAUNCH_CHECK("pt_window_attn");

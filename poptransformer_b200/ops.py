@@ -20,12 +20,13 @@ import ctypes
 import torch
 
 from . import _lib
-from ._lib import AttnArgs, BatchView, GemmArgs, HyperArgs, LinearArgs, PtError, SsmArgs, WindowAttnArgs, check
+from ._lib import (AttnArgs, BatchView, DenseExt, GemmArgs, HyperArgs, LinearArgs, MlstmArgs, MoeRouteArgs, PostNormArgs, PtError, SsmArgs,
+                   WindowAttnArgs, check)
 
 W_INT4, W_FP16, W_FP8, W_BF16 = 0, 1, 2, 3
 DT_F16, DT_F32, DT_BF16 = 0, 1, 2
 PRO_NONE, PRO_RMSNORM, PRO_CAST_FP8, PRO_RMSNORM_CAST_FP8, PRO_NORMCE = 0, 1, 2, 3, 4
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL, EPI_RELU2 = 0, 1, 2, 3, 4, 5, 6
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL, EPI_RELU2, EPI_GLU, EPI_GELU_MUL = 0, 1, 2, 3, 4, 5, 6, 7, 8
 ROPE_NONE, ROPE_LLAMA, ROPE_CHATGLM2 = 0, 1, 2
 SOFTMAX_F32, SOFTMAX_F16 = 0, 1
 
@@ -108,7 +109,7 @@ def linear_workspace(batch, n_out_max, max_ksplit=16, device="cuda"):
 
 
 def linear_args(x, pl, out, prologue=PRO_NONE, epilogue=EPI_STORE, gamma=None, eps=0.0, act_scale=0.0, bias=None,
-                residual=None, workspace=None, ksplit=0, out_ld=0, pdl=0, error_flag=None, beta=None, alpha=1.0):
+                residual=None, workspace=None, ksplit=0, out_ld=0, pdl=0, error_flag=None, beta=None, alpha=1.0, ext=None):
     a = LinearArgs()
     a.wfmt, a.batch, a.n_out, a.k_in, a.group = pl.wfmt, x.shape[0], pl.n_out, pl.k_in, pl.group
     a.prologue, a.epilogue, a.ksplit = prologue, epilogue, ksplit
@@ -117,6 +118,8 @@ def linear_args(x, pl, out, prologue=PRO_NONE, epilogue=EPI_STORE, gamma=None, e
     a.bias, a.residual, a.out, a.out_ld, a.pdl = _ptr(bias), _ptr(residual), _ptr(out), out_ld, pdl
     a.error_flag, a.norm_beta = _ptr(error_flag), _ptr(beta)
     a.out_dtype, a.alpha = dtype_code(out.dtype), float(alpha)
+    if ext is not None:
+        a.ext = ctypes.pointer(ext)
     a.workspace = _ptr(workspace)
     a.workspace_bytes = workspace.numel() if workspace is not None else 0
     return a
@@ -165,7 +168,7 @@ def gemm_workspace(m, n_out_max, max_ksplit=8, device="cuda"):
 
 
 def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, workspace=None, ksplit=0, error_flag=None, bias=None,
-         out_ld=0, alpha=1.0):
+         out_ld=0, alpha=1.0, ext=None):
     """y = x @ W^T on the tcgen05 GEMM.  INT4: x fp16 [m, k]; FP8: x E4M3 bytes [m, k] quantised with `x_scale`; BF16: x bfloat16,
     `out` bfloat16 or float32."""
     m = x.shape[0]
@@ -182,6 +185,8 @@ def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, worksp
     a.out_dtype, a.alpha = dtype_code(out.dtype), float(alpha)
     a.workspace, a.workspace_bytes = _ptr(workspace), (workspace.numel() if workspace is not None else 0)
     a.error_flag, a.bias = _ptr(error_flag), _ptr(bias)
+    if ext is not None:
+        a.ext = ctypes.pointer(ext)
     check(_lib.lib().pt_gemm(ctypes.byref(a), _stream()), "pt_gemm")
     return out
 
@@ -189,6 +194,18 @@ def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, worksp
 # ------------------------------------------------------------------------------------------ linears of bf16 / fp32 models
 def pad_to(n, m):
     return (n + m - 1) // m * m
+
+
+def glu_rows(gate, up, features):
+    """Weight rows of a gated product (EPI_GLU): blocks of eight gate features and the same eight up features, with zero rows up to
+    `features` (a multiple of eight)."""
+    n, k = gate.shape
+    out = torch.zeros((features // 8, 2, 8, k), dtype=gate.dtype, device=gate.device)
+    for j, w in enumerate((gate, up)):
+        full = torch.zeros((features, k), dtype=w.dtype, device=w.device)
+        full[:n] = w
+        out[:, j] = full.view(-1, 8, k)
+    return out.reshape(-1, k)
 
 
 class DenseLinear:
@@ -199,15 +216,21 @@ class DenseLinear:
     # Measured on B200 over 2048 x 4096 .. 32000 x 4096: at 8 rows the GEMM is level (2048-wide) to 20 % faster, at 32 rows 10 % to 3x.
     SKINNY_ROWS = 7
 
-    def __init__(self, w, dtype, pad_rows=0, keep=False):
+    def __init__(self, w, dtype, pad_rows=0, keep=False, bias=None, split=None, limit=0.0):
         """pad_rows: zero rows are appended up to this many outputs (an output that is the padded input of the next linear).
-        keep: keep the padded matrix itself as `w` (a table that also serves look-ups)."""
+        keep: keep the padded matrix itself as `w` (a table that also serves look-ups).  bias: fp32 [n_out].  split: outputs from this
+        row on (a multiple of 32) go to a second, fp32 output and skip the epilogue.  limit: of a gated epilogue (rows as glu_rows)."""
         self.dtype, self.n_out, self.k_in = dtype, w.shape[0], w.shape[1]
+        self.split, self.limit = split, float(limit)
         self.ld = pad_to(self.k_in, self.K_PAD) if dtype == torch.bfloat16 else self.k_in
         if self.ld != self.k_in or pad_rows > self.n_out:
             full = torch.zeros((max(pad_rows, self.n_out), self.ld), dtype=w.dtype, device=w.device)
             full[:self.n_out, :self.k_in] = w
             w, self.n_out = full, full.shape[0]
+        self.bias = None
+        if bias is not None:
+            self.bias = torch.zeros(self.n_out, dtype=torch.float32, device=w.device)
+            self.bias[:len(bias)] = bias
         w = w.to(dtype).contiguous()
         if dtype == torch.bfloat16:
             self.skinny, self.gemm = PackedLinear(W_BF16, w), GemmWeight(W_BF16, w)
@@ -222,18 +245,91 @@ class DenseLinear:
         """Algorithmic bytes of one launch: the weights once."""
         return self.n_out * self.k_in * (2 if self.dtype == torch.bfloat16 else 4)
 
-    def __call__(self, x, out, rows, out_ld, epilogue=EPI_STORE, alpha=1.0, linear_ws=None, gemm_ws=None, error_flag=None):
-        """out[:rows, :n_out] = epilogue(alpha * x[:rows] @ W^T); x and out are flat or 2-D buffers of row strides `ld` and `out_ld`."""
+    def _ext(self, out2, out2_ld, mul, mul_ids):
+        """mul: (a table of the output's type, its row stride, its first column)."""
+        if self.bias is None and self.split is None and mul is None and not self.limit:
+            return None
+        e = DenseExt()
+        e.bias, e.limit = _ptr(self.bias), self.limit
+        if self.split is not None:
+            e.out2, e.out2_ld, e.split_n = _ptr(out2), out2_ld, self.split
+        if mul is not None:
+            table, ld, col = mul
+            e.mul, e.mul_ld, e.mul_ids = table.data_ptr() + col * table.element_size(), ld, _ptr(mul_ids)
+        return e
+
+    def __call__(self, x, out, rows, out_ld, epilogue=EPI_STORE, alpha=1.0, linear_ws=None, gemm_ws=None, error_flag=None, out2=None, out2_ld=0, mul=None,
+                 mul_ids=None):
+        """out[:rows, :n_out] = epilogue(alpha * x[:rows] @ W^T + bias); x and out are flat or 2-D buffers of row strides `ld` and
+        `out_ld`."""
         x = x.reshape(-1)[:rows * self.ld].view(rows, self.ld)
         L = _lib.lib()
+        ext = self._ext(out2, out2_ld, mul, mul_ids)
         if self.dtype == torch.float32:
-            check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, float(alpha), epilogue, _ptr(out), out_ld, _stream()),
-                  "pt_gemm_f32")
+            check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, float(alpha), epilogue, _ptr(out), out_ld,
+                                ctypes.byref(ext) if ext else None, _stream()), "pt_gemm_f32")
         elif rows <= self.SKINNY_ROWS:
-            a = linear_args(x, self.skinny, out, epilogue=epilogue, workspace=linear_ws, out_ld=out_ld, error_flag=error_flag, alpha=alpha)
+            a = linear_args(x, self.skinny, out, epilogue=epilogue, workspace=linear_ws, out_ld=out_ld, error_flag=error_flag, alpha=alpha, ext=ext)
             check(L.pt_linear(ctypes.byref(a), _stream()), "pt_linear")
         else:
-            gemm(x, self.gemm, out=out, epilogue=epilogue, workspace=gemm_ws, error_flag=error_flag, out_ld=out_ld, alpha=alpha)
+            gemm(x, self.gemm, out=out, epilogue=epilogue, workspace=gemm_ws, error_flag=error_flag, out_ld=out_ld, alpha=alpha, ext=ext)
+
+
+class GroupedLinear:
+    """Matrices [n_out, k] of one shape (experts), one after the other in a buffer: every tile of activation rows is multiplied with
+    the matrix that `group_of` names for it.  bfloat16: tiles of one row on the skinny-matmul kernel, tiles of 16 .. 256 rows on the
+    tcgen05 GEMM; float32: tiles of 64 rows."""
+
+    def __init__(self, ws, dtype, pad_rows=0, limit=0.0):
+        self.dtype, self.groups, self.k_in, self.limit = dtype, len(ws), ws[0].shape[1], float(limit)
+        self.n_out = max(pad_rows, ws[0].shape[0])
+        self.ld = pad_to(self.k_in, DenseLinear.K_PAD) if dtype == torch.bfloat16 else self.k_in
+        L = _lib.lib()
+        dev = ws[0].device
+        if dtype == torch.bfloat16:
+            skinny, tiled = L.pt_linear_packed_bytes(W_BF16, self.n_out, self.ld), L.pt_gemm_packed_bytes(W_BF16, self.n_out, self.ld)
+            self.skinny = torch.empty((self.groups, skinny), dtype=torch.uint8, device=dev)
+            self.tiled = torch.empty((self.groups, tiled), dtype=torch.uint8, device=dev)
+        elif dtype == torch.float32:
+            self.w = torch.zeros((self.groups, self.n_out, self.k_in), dtype=dtype, device=dev)
+        else:
+            raise PtError(f"GroupedLinear: bfloat16 or float32, got {dtype}")
+        for g, w in enumerate(ws):
+            if dtype == torch.float32:
+                self.w[g, :w.shape[0]] = w
+                continue
+            full = torch.zeros((self.n_out, self.ld), dtype=dtype, device=dev)
+            full[:w.shape[0], :self.k_in] = w
+            check(L.pt_linear_repack(W_BF16, _ptr(full), None, self.n_out, self.ld, 0, 0, _ptr(self.skinny[g]), _stream()), "pt_linear_repack")
+            check(L.pt_gemm_repack(W_BF16, _ptr(full), self.n_out, self.ld, _ptr(self.tiled[g]), _stream()), "pt_gemm_repack")
+
+    @property
+    def nbytes(self):
+        """Bytes of one matrix."""
+        return self.n_out * self.k_in * (2 if self.dtype == torch.bfloat16 else 4)
+
+    def __call__(self, x, out, rows, out_ld, tile, group_of, x_div=1, epilogue=EPI_STORE, linear_ws=None, gemm_ws=None, error_flag=None):
+        """out[:rows] = epilogue(x rows @ matrix^T).  tile: rows per entry of group_of; with tile 1 row r reads x row r // x_div."""
+        L = _lib.lib()
+        e = DenseExt()
+        e.limit, e.n_groups, e.group_rows, e.group_x_div, e.group_of = self.limit, self.groups, tile, x_div, _ptr(group_of)
+        if self.dtype == torch.float32:
+            check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, 1.0, epilogue, _ptr(out), out_ld, ctypes.byref(e), _stream()),
+                  "pt_gemm_f32")
+        elif tile == 1:
+            a = LinearArgs()
+            a.wfmt, a.batch, a.n_out, a.k_in, a.epilogue, a.x, a.packed_w = W_BF16, rows, self.n_out, self.ld, epilogue, _ptr(x), _ptr(self.skinny)
+            a.out, a.out_ld, a.out_dtype, a.alpha, a.error_flag = _ptr(out), out_ld, dtype_code(out.dtype), 1.0, _ptr(error_flag)
+            a.workspace, a.workspace_bytes = _ptr(linear_ws), linear_ws.numel() if linear_ws is not None else 0
+            a.ext = ctypes.pointer(e)
+            check(L.pt_linear(ctypes.byref(a), _stream()), "pt_linear")
+        else:
+            a = GemmArgs()
+            a.wfmt, a.m, a.n_out, a.k_in, a.epilogue, a.w_tiled, a.x, a.w = W_BF16, rows, self.n_out, self.ld, epilogue, 1, _ptr(x), _ptr(self.tiled)
+            a.out, a.out_ld, a.out_dtype, a.alpha, a.error_flag = _ptr(out), out_ld, dtype_code(out.dtype), 1.0, _ptr(error_flag)
+            a.workspace, a.workspace_bytes = _ptr(gemm_ws), gemm_ws.numel() if gemm_ws is not None else 0
+            a.ext = ctypes.pointer(e)
+            check(L.pt_gemm(ctypes.byref(a), _stream()), "pt_gemm")
 
 
 # ------------------------------------------------------------------------------------------ layers with per-sequence positions
@@ -268,9 +364,11 @@ def window_attn_workspace(n_seq, n_head, vdim, page_size, max_len, window, keep_
 
 
 def window_attn(view, qkv, qkv_ld, cache, out, out_ld, n_head, scale, window=0, keep_first=0, sink=None, append=True, max_tokens_per_seq=0,
-                workspace=None, error_flag=None, plain=False):
+                workspace=None, error_flag=None, plain=False, values_are_keys=False, q_norm=None, k_norm=None, eps=0.0, rope=None, rope_dims=0, out_scale=1.0,
+                out_cols=0):
     """Masked attention of the packed tokens of `view` over a paged cache (see pt_window_attn).  qkv rows hold [q | k | v]
-    (append=True: k and v go to the cache first) or only q (a layer that reads another layer's cache)."""
+    (append=True: k and v go to the cache first), [q | k] (values_are_keys: the keys as they are in the row are the values) or only q
+    (a layer that reads another layer's cache).  q_norm, k_norm, rope: per-head norm and rotation of q and k; q is then rewritten."""
     a = WindowAttnArgs()
     a.batch, a.dtype = view, dtype_code(qkv.dtype)
     a.n_head, a.n_kv, a.dim, a.vdim = n_head, cache.n_kv, cache.head_dim, cache.v_dim
@@ -279,7 +377,9 @@ def window_attn(view, qkv, qkv_ld, cache, out, out_ld, n_head, scale, window=0, 
     a.q, a.q_ld, a.kv_ld = _ptr(qkv), qkv_ld, qkv_ld
     if append:
         k = qkv.data_ptr() + n_head * cache.head_dim * qkv.element_size()
-        a.k, a.v = k, k + cache.n_kv * cache.head_dim * qkv.element_size()
+        a.k, a.v = k, k if values_are_keys else k + cache.n_kv * cache.head_dim * qkv.element_size()
+    a.q_norm, a.k_norm, a.norm_eps, a.rope, a.rope_dims = _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(rope), rope_dims
+    a.out_scale, a.out_cols = float(out_scale), out_cols
     a.pool, a.page_table, a.out, a.out_ld = _ptr(cache.pool), _ptr(cache.page_table), _ptr(out), out_ld
     a.max_tokens_per_seq, a.plain = max_tokens_per_seq, 1 if plain else 0
     a.workspace, a.workspace_bytes = _ptr(workspace), workspace.numel() if workspace is not None else 0
@@ -299,6 +399,53 @@ def ssm(view, zx, zx_ld, out, out_ld, w, ring, state, y, xbc=None, dt=None, work
     a.plain = 1 if plain else 0
     a.workspace, a.workspace_bytes = _ptr(workspace), workspace.numel() if workspace is not None else 0
     check(_lib.lib().pt_ssm(ctypes.byref(a), _stream()), "pt_ssm")
+
+
+def mlstm(view, rows, ld, cols, gates, gate_ld, out, out_ld, w, state, nm, y, workspace, out_scale=1.0, out_cols=0, plain=False):
+    """Matrix memory between its projections (see pt_mlstm).  cols: first columns of q, k, v and the output gate in `rows`; gates: fp32
+    rows [log input | log forget]; w: an object with heads, dim, vdim, cap, eps and the fp32 tensor norm_w.  out: a view that starts
+    at the output's first column."""
+    a = MlstmArgs()
+    es = rows.element_size()
+    a.batch, a.dtype, a.heads, a.dim, a.vdim = view, dtype_code(rows.dtype), w.heads, w.dim, w.vdim
+    a.gate_cap, a.q_scale, a.eps, a.out_scale = float(w.cap), float(w.dim) ** -0.5, float(w.eps), float(out_scale)
+    a.q, a.k, a.v, a.gate = (rows.data_ptr() + c * es for c in cols)
+    a.ld, a.log_i, a.log_f, a.gate_ld = ld, gates.data_ptr(), gates.data_ptr() + w.heads * 4, gate_ld
+    a.norm_w, a.state, a.nm, a.y = _ptr(w.norm_w), _ptr(state), _ptr(nm), _ptr(y)
+    a.out, a.out_ld, a.out_cols, a.plain = out.data_ptr(), out_ld, out_cols, 1 if plain else 0
+    a.workspace, a.workspace_bytes = _ptr(workspace), workspace.numel() if workspace is not None else 0
+    check(_lib.lib().pt_mlstm(ctypes.byref(a), _stream()), "pt_mlstm")
+
+
+def post_norm(rows, width, eps, dtype, x_in=None, x_out=None, y=None, y_ld=0, pair_y=None, pair_ld=0, top=0, pair_w=None, pair_row=None, norm_w=None,
+              final_w=None, h=None, h_ld=0, row_index=None, table=None, vocab=0, ids=None, ids_ld=1, step=None, pos_out=None, id_out=None):
+    """Residual step with a norm on the sublayer's output (see pt_post_norm), or the start of a token from an embedding table."""
+    a = PostNormArgs()
+    a.rows, a.width, a.dtype, a.eps, a.x_in, a.x_out = rows, width, dtype_code(dtype), float(eps), _ptr(x_in), _ptr(x_out)
+    if table is not None:
+        a.table, a.table_ld, a.vocab, a.ids, a.ids_ld = _ptr(table), table.shape[1], vocab or table.shape[0], _ptr(ids), ids_ld
+        a.step_dev, a.pos_out, a.id_out = _ptr(step), _ptr(pos_out), _ptr(id_out)
+    a.row_index, a.y, a.y_ld = _ptr(row_index), _ptr(y), y_ld
+    a.pair_y, a.pair_ld, a.top, a.pair_w, a.pair_row = _ptr(pair_y), pair_ld, top, _ptr(pair_w), _ptr(pair_row)
+    a.norm_w, a.final_w, a.h, a.h_ld = _ptr(norm_w), _ptr(final_w), _ptr(h), h_ld
+    check(_lib.lib().pt_post_norm(ctypes.byref(a), _stream()), "pt_post_norm")
+
+
+def moe_max_tiles(n_tok, experts, top, tile):
+    return int(_lib.lib().pt_moe_max_tiles(n_tok, experts, top, tile))
+
+
+def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, row_token=None, h=None, h_ld=0, gathered=None):
+    """Experts and weights of every token, and with `tile` the rows of the grouped products (see pt_moe_route)."""
+    a = MoeRouteArgs()
+    a.n_tok, a.experts, a.top, a.logits, a.logits_ld = n_tok, experts, top, _ptr(logits), logits.shape[-1]
+    a.expert, a.weight, a.tile = _ptr(expert), _ptr(weight), tile
+    if tile:
+        a.max_tiles = moe_max_tiles(n_tok, experts, top, tile)
+        a.pair_row, a.tile_expert, a.row_token = _ptr(pair_row), _ptr(tile_expert), _ptr(row_token)
+        if h is not None:
+            a.h, a.h_bytes, a.gathered = _ptr(h), h_ld * h.element_size(), _ptr(gathered)
+    check(_lib.lib().pt_moe_route(ctypes.byref(a), _stream()), "pt_moe_route")
 
 
 # ------------------------------------------------------------------------------------------ norms / softmax

@@ -41,6 +41,11 @@ def _sabisun(c, sd, batch, max_len, dtype, **kw):
     return SabisunDecoder(SabisunConfig(c, max_len), sd, batch, dtype=dtype, **kw)
 
 
+def _padetar(c, sd, batch, max_len, dtype, **kw):
+    from .padetar import PadetarConfig, PadetarDecoder
+    return PadetarDecoder(PadetarConfig(c, max_len), sd, batch, dtype=dtype, **kw)
+
+
 # name -> (builder, dtypes the decoder runs in; the first is the default)
 ARCHITECTURES = {
     "LlamaForCausalLM": (_llama, ("float16",)),
@@ -49,6 +54,7 @@ ARCHITECTURES = {
     "ChatGLMForConditionalGeneration": (_chatglm2, ("float16",)),
     "RwkvForCausalLM": (_rwkv, ("float16",)),
     "Sabisun": (_sabisun, ("bfloat16", "float32")),
+    "Padetar": (_padetar, ("bfloat16", "float32")),
 }
 
 
