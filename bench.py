@@ -616,6 +616,87 @@ HYBRID = {   # name: configuration, then the Llama of equal width, depth, feed-f
 }
 
 
+def expert_config(width, n_layer, heads, kv_heads, dim, mem_heads, mem_dim, mem_vdim, experts, top, ff, shared_ff, side, vocab):
+    """A Padetar of real-model layer sizes."""
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+            "rot": {"base": 5e5, "dims": dim, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    right = {"heads": mem_heads, "dim": mem_dim, "vdim": mem_vdim, "gate_cap": 15.0}
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff, "limit": 7.0}, "shared": {"ff": shared_ff, "limit": 7.0}}
+    return {"architecture": "Padetar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "token_side": {"dim": side},
+            "layers": [{"type": "parallel", "mixer": {"left": left, "left_scale": 1.0, "right": right, "right_scale": 1.0}, "mlp": mlp} for _ in range(n_layer)]}
+
+
+EXPERTS = {   # name: configuration, then the Sabisun of equal width, depth and vocabulary whose feed-forward has as many weights as a token uses here
+    "padetar-2k": (dict(width=2048, n_layer=16, heads=16, kv_heads=4, dim=128, mem_heads=16, mem_dim=128, mem_vdim=128, experts=32, top=4, ff=1024, shared_ff=2048,
+                        side=128, vocab=32000),
+                   dict(width=2048, n_layer=16, ff=9216, heads=16, kv_heads=4, dim=128, ssm_heads=64, ssm_dim=64, state=128, groups=8, vocab=32000, window=1024,
+                        keep_first=64, streams=2)),
+    "padetar-4k": (dict(width=4096, n_layer=8, heads=32, kv_heads=8, dim=128, mem_heads=16, mem_dim=128, mem_vdim=256, experts=32, top=4, ff=1536, shared_ff=4096,
+                        side=256, vocab=32000),
+                   dict(width=4096, n_layer=8, ff=15360, heads=32, kv_heads=8, dim=128, ssm_heads=128, ssm_dim=64, state=128, groups=8, vocab=32000, window=1024,
+                        keep_first=64, streams=4)),
+}
+
+
+def time_decode(dec, ctx, K):
+    """ms per step of a captured decode loop at context `ctx`: the mean of K steps after three."""
+    import torch
+    for _ in range(3):
+        dec.step()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    dec.step_t.fill_(ctx)
+    torch.cuda.synchronize()
+    e0.record()
+    for _ in range(K):
+        dec.step()
+    e1.record()
+    torch.cuda.synchronize()
+    if int(dec.error_flag.item()):
+        raise SystemExit(f"device-side error flag {int(dec.error_flag.item())}")
+    return e0.elapsed_time(e1) / K
+
+
+def sequence_decoder(cfg, sd, batch, max_len, ctx):
+    """A decoder of packed sequences (bf16) with a captured step, at context `ctx` over random caches."""
+    from poptransformer_b200 import registry
+    dec = registry.build_decoder(cfg, sd, batch, max_len, "bfloat16", pad_id=-1)
+    dec._need_loop_rows()
+    for c in dec.caches.values():
+        c.pool.normal_(std=0.5)
+    dec.ids.random_(0, cfg["vocab"])          # rows that differ, so that a router spreads them over its experts
+    dec.step_t.fill_(ctx)
+    dec.capture()
+    dec.step_t.fill_(ctx)
+    return dec
+
+
+def time_prompts(dec, vocab, n_seq, prompt):
+    """Best of four passes (ms) over n_seq prompts, from the ids on the host to the logits of the last tokens."""
+    import torch
+    r = np.random.default_rng(0)
+    toks = [r.integers(0, vocab, prompt).astype(np.int32) for _ in range(n_seq)]
+    times = []
+    for _ in range(4):
+        seqs = [dec.open() for _ in range(n_seq)]
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        dec.extend([(s, t, [prompt - 1]) for s, t in zip(seqs, toks)])
+        e1.record()
+        torch.cuda.synchronize()
+        times.append(e0.elapsed_time(e1))
+        for s in seqs:
+            dec.close(s)
+    return min(times)
+
+
+def sabisun_state_bytes(cfg):
+    """Recurrent state (read and written) and visible keys and values of one row and step."""
+    mixers = [lay["mixer"] for lay in cfg["layers"]]
+    return sum(2 * 4 * m["heads"] * m["state"] * m["vdim"] for m in mixers if "state" in m) + \
+        sum(2 * m["kv_heads"] * m["dim"] * 2 * (m["mask"]["size"] + m["mask"]["keep_first"]) for m in mixers if "mask" in m)
+
+
 def run_hybrid(args):
     """Decode and prompt throughput of a Sabisun beside the Llama of equal size (fp16 weights, per-op kernels, for decode; INT4
     weights for the prompt pass, the only one Llama has).  One JSON line, marked `secondary`."""
@@ -635,35 +716,9 @@ def run_hybrid(args):
     sampler.start()
     rows = []
     for batch in (1, 8, 32):
-        dec = registry.build_decoder(cfg, sd, batch, max_len, "bfloat16", pad_id=-1)
-        dec._need_loop_rows()
-        for c in dec.caches.values():
-            c.pool.normal_(std=0.5)
-        dec.step_t.fill_(ctx)
-        dec.capture()
-        dec.step_t.fill_(ctx)
-
-        def steps(d):
-            for _ in range(3):
-                d.step()
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            d.step_t.fill_(ctx)
-            torch.cuda.synchronize()
-            e0.record()
-            for _ in range(K):
-                d.step()
-            e1.record()
-            torch.cuda.synchronize()
-            if int(d.error_flag.item()):
-                raise SystemExit(f"device-side error flag {int(d.error_flag.item())}")
-            return e0.elapsed_time(e1) / K
-
-        ms = steps(dec)
-        w_bytes = dec.weight_bytes()
-        mixers = [lay["mixer"] for lay in cfg["layers"]]
-        state = sum(2 * 4 * m["heads"] * m["state"] * m["vdim"] for m in mixers if "state" in m)
-        kv = sum(2 * m["kv_heads"] * m["dim"] * 2 * (m["mask"]["size"] + m["mask"]["keep_first"]) for m in mixers if "mask" in m)
-        need = w_bytes + batch * (state + kv)
+        dec = sequence_decoder(cfg, sd, batch, max_len, ctx)
+        ms = time_decode(dec, ctx, K)
+        need = dec.weight_bytes() + batch * sabisun_state_bytes(cfg)
         row = {"batch": batch, "decode_ms": ms, "decode_tokens_per_s": batch / ms * 1e3, "bytes_per_step": need, "decode_frac_of_measured": need / ms / 1e6 / peak}
         del dec
         ld = llama.LlamaDecoder(llama.LlamaConfig(**ldims, max_len=max_len), lsd, batch, device=dev, persistent=False)
@@ -671,7 +726,7 @@ def run_hybrid(args):
             c.pool.normal_(std=0.5)
         ld.step_t.fill_(ctx)
         ld.capture()
-        lms = steps(ld)
+        lms = time_decode(ld, ctx, K)
         lneed = ld.weight_bytes() + batch * ld.kv_bytes_per_token_total() * ctx
         row.update(llama_fp16_decode_ms=lms, llama_fp16_tokens_per_s=batch / lms * 1e3, llama_frac_of_measured=lneed / lms / 1e6 / peak)
         del ld
@@ -681,22 +736,8 @@ def run_hybrid(args):
     dec = registry.build_decoder(cfg, sd, 4, max_len, "bfloat16", pad_id=-1)
     lin_flops = 2 * prompt * sum(s.proj.n_out * s.proj.k_in + s.out.n_out * s.out.k_in for s in dec.subs)
     pre = []
-    r = np.random.default_rng(0)
     for n_seq in (1, 4):
-        toks = [r.integers(0, cfg["vocab"], prompt).astype(np.int32) for _ in range(n_seq)]
-        best = None
-        for _ in range(4):
-            seqs = [dec.open() for _ in range(n_seq)]
-            torch.cuda.synchronize()
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            dec.extend([(s, t, [prompt - 1]) for s, t in zip(seqs, toks)])
-            e1.record()
-            torch.cuda.synchronize()
-            ms = e0.elapsed_time(e1)
-            best = ms if best is None else min(best, ms)
-            for s in seqs:
-                dec.close(s)
+        best = time_prompts(dec, cfg["vocab"], n_seq, prompt)
         pre.append({"sequences": n_seq, "prompt": prompt, "ms": best, "tokens_per_s": n_seq * prompt / best * 1e3, "linear_tflops": n_seq * lin_flops / best / 1e9})
     del dec, lsd
     torch.cuda.empty_cache()
@@ -724,6 +765,61 @@ def run_hybrid(args):
                       "llama_int4_prompt_pass": {"sequences": 1, "prompt": prompt, "ms": lms, "tokens_per_s": prompt / lms * 1e3, "linear_tflops": lflops / lms / 1e9}}))
 
 
+def run_experts(args):
+    """Decode and prompt throughput of a Padetar beside the Sabisun of equal size.  One JSON line, marked `secondary`."""
+    import torch
+    from poptransformer_b200 import registry, synth
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device (there is no CPU fallback)")
+    dims, sdims = EXPERTS[args.workload]
+    dev = torch.device("cuda", 0)
+    ctx, prompt, K = 2048, 2048, max(8, min(args.steps, 64))
+    max_len = ctx + K + 16
+    peak, _ = peaks()
+    sampler = ClockSampler(0)
+    sampler.start()
+    E, top, n_layer = dims["experts"], dims["top"], dims["n_layer"]
+    res = {}
+    for name, cfg, make in (("padetar", expert_config(**dims), synth.padetar_state_dict), ("sabisun", hybrid_config(**sdims), synth.sabisun_state_dict)):
+        sd = make(cfg, device=dev)
+        rows, pre = [], []
+        for batch in (1, 8, 32):
+            dec = sequence_decoder(cfg, sd, batch, max_len, ctx)
+            ms = time_decode(dec, ctx, K)
+            if name == "padetar":
+                # every linear once, and the experts that `batch` independent choices are expected to hit
+                hit = E * (1.0 - (1.0 - top / E) ** batch)
+                moe = [s for s in dec.subs if s.kind == "moe"]
+                weights = sum(x.nbytes for x in dec._linears()) + sum(hit * (s.up.nbytes + s.back.nbytes) for s in moe)
+                state = n_layer * (2 * 4 * dims["mem_heads"] * dims["mem_dim"] * dims["mem_vdim"] + 2 * 2 * dims["kv_heads"] * dims["dim"] * ctx)
+            else:
+                weights, state = dec.weight_bytes(), sabisun_state_bytes(cfg)
+            need = weights + batch * state
+            rows.append({"batch": batch, "decode_ms": ms, "decode_tokens_per_s": batch / ms * 1e3, "bytes_per_step": int(need), "decode_frac_of_measured": need / ms / 1e6 / peak})
+            del dec
+            torch.cuda.empty_cache()
+        dec = registry.build_decoder(cfg, sd, 4, max_len, "bfloat16", pad_id=-1)
+        size = lambda x: x.n_out * x.k_in
+        if name == "padetar":
+            flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(top * (size(s.up) + size(s.back)) for s in dec.subs if s.kind == "moe"))
+        else:
+            flops = 2 * prompt * sum(size(s.proj) + size(s.out) for s in dec.subs)
+        for n_seq in (1, 4):
+            best = time_prompts(dec, cfg["vocab"], n_seq, prompt)
+            pre.append({"sequences": n_seq, "prompt": prompt, "ms": best, "tokens_per_s": n_seq * prompt / best * 1e3, "linear_tflops": n_seq * flops / best / 1e9})
+        res[name] = {"decode": rows, "prompt_pass": pre}
+        del dec, sd
+        torch.cuda.empty_cache()
+    clocks = sampler.stop()
+    last = res["padetar"]["decode"][-1]
+    print(json.dumps({"secondary": "not the headline workload; a decoder with experts and a matrix memory beside the Sabisun of equal size on one GPU",
+                      "metric": f"decode tokens/s ({args.workload}, batch 32)", "value": last["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": 3,
+                      "ms_per_step": last["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+                      "dtype": "bf16 (float32 residual, router, gates, softmax, state)", "data": "synthetic",
+                      "config": {"workload": args.workload, **dims, "ctx": ctx, "cuda_graph": True, "l2": "weights larger than L2 streamed per step"},
+                      "clocks": clocks, **res["padetar"], "sabisun_config": sdims, "sabisun": res["sabisun"]}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -740,9 +836,9 @@ def main():
                     "stays small; the line is then marked profiling_only and is not a benchmark result")
     ap.add_argument("--pdl", type=int, default=-1, help="secondary workloads: programmatic dependent launch, bit 0 = linear kernels, bit 1 = "
                     "attention kernel (-1: the decoder's default)")
-    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY) + list(HYBRID),
-                    help="llama2-7b-int4 is the benchmark; the others time a parity configuration, or the hybrid architecture beside the Llama of "
-                    "equal size, on one GPU (line marked `secondary`)")
+    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY) + list(HYBRID) + list(EXPERTS),
+                    help="llama2-7b-int4 is the benchmark; the others time a parity configuration, or an architecture of this framework beside the "
+                    "closest one of equal size, on one GPU (line marked `secondary`)")
     args = ap.parse_args()
     if args.impl == "reference":
         run_reference(args)
@@ -750,6 +846,8 @@ def main():
         run_secondary(args)
     elif args.workload in HYBRID:
         run_hybrid(args)
+    elif args.workload in EXPERTS:
+        run_experts(args)
     else:
         run_b200(args)
 

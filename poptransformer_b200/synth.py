@@ -87,6 +87,58 @@ def sabisun_state_dict(config, seed=0, device="cpu"):
     return sd
 
 
+def padetar_state_dict(config, seed=0, device="cpu"):
+    """Padetar architecture (a parsed config.json), bfloat16: linears N(0, 1 / in_features), norms 1 + N(0, 0.02), forget gates spread
+    over slow and fast heads."""
+    gen = torch.Generator(device=device)
+    gen.manual_seed(seed)
+    sd = {}
+    W, V = config["width"], config["vocab"]
+
+    def put(key, shape, std=1.0, mean=0.0):
+        sd[key] = torch.empty(shape, dtype=torch.bfloat16, device=device).normal_(mean, std, generator=gen)
+
+    def lin(key, o, i):
+        put(key, (o, i), i ** -0.5)
+
+    put("embed", (V, W))
+    put("final.norm", (W,), 0.02, 1.0)
+    lin("head", V, W)
+    side = (config.get("token_side") or {}).get("dim", 0)
+    if side:
+        put("side.embed", (V, side * len(config["layers"])))
+    for i, lay in enumerate(config["layers"]):
+        p, a, b, mlp = f"l{i}.", lay["mixer"]["left"], lay["mixer"]["right"], lay.get("mlp")
+        L, R, M = p + "mix.left.", p + "mix.right.", p + "mlp."
+        put(p + "norm1", (W,), 0.02, 1.0)
+        for n, rows in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"])):
+            lin(L + n, rows, W)
+            put(L + n + ".b", (rows,), 0.1)
+            put(L + n + ".norm", (a["dim"],), 0.02, 1.0)
+        lin(L + "o", W, a["heads"] * a["dim"])
+        put(L + "o.b", (W,), 0.1)
+        for n, rows in (("q", b["heads"] * b["dim"]), ("k", b["heads"] * b["dim"]), ("v", b["heads"] * b["vdim"]), ("g", b["heads"] * b["vdim"]), ("i", b["heads"]), ("f", b["heads"])):
+            lin(R + n, rows, W)
+        lin(R + "o", W, b["heads"] * b["vdim"])
+        put(R + "norm", (b["heads"] * b["vdim"],), 0.02, 1.0)
+        put(R + "i.b", (b["heads"],), 1.0, -2.0)
+        put(R + "f.b", (b["heads"],), 1.5, 4.0)
+        if mlp:
+            put(p + "norm2", (W,), 0.02, 1.0)
+            lin(M + "router", mlp["router"]["experts"], W)
+            put(M + "router.b", (mlp["router"]["experts"],), 0.1)
+            units = [(f"e{e}.", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])] + ([("shared.", mlp["shared"]["ff"])] if mlp.get("shared") else [])
+            for n, ff in units:
+                lin(M + n + "gate", ff, W)
+                lin(M + n + "up", ff, W)
+                lin(M + n + "down", W, ff)
+        if side:
+            lin(p + "side.gate", side, W)
+            lin(p + "side.proj", W, side)
+            put(p + "side.norm", (W,), 0.02, 1.0)
+    return sd
+
+
 def gpt2_state_dict(n_layer, d_model, n_head, vocab, n_positions, seed=0, device="cpu"):
     """GPT-2 architecture with the reference's key names after its checkpoint pre-processing (gpt2/model.py:154-166): linear
     weights [out, in], the query third of c_attn (weight and bias) multiplied by 1/sqrt(head_size).  fp16, N(0, 0.02);

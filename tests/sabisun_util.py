@@ -1,8 +1,7 @@
-"""Small Sabisun configurations, random weights and model folders for the tests."""
-import json
-import os
-
+"""Small Sabisun configurations and random weights for the tests."""
 import numpy as np
+
+from seq_util import bf16, tensors
 
 
 def attn(heads=4, kv_heads=2, dim=32, vdim=32, scale=None, size=None, keep_first=0, kv_from=None):
@@ -25,12 +24,6 @@ def config(mixers, width=96, vocab=160, ff=128, streams=2, eps=1e-5, mult=0.9, l
               for m, f in zip(mixers, ffs)]
     return {"architecture": "Sabisun", "layers": layers, "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": eps}, "residual_mult": mult,
             "logit_scale": logit_scale}
-
-
-def bf16(x):
-    """float array rounded to bfloat16 (as float32)."""
-    import torch
-    return torch.from_numpy(np.ascontiguousarray(x, dtype=np.float32)).to(torch.bfloat16).float().numpy()
 
 
 def weights(cfg, seed=0, sinks=True):
@@ -65,36 +58,9 @@ def weights(cfg, seed=0, sinks=True):
     return {k: bf16(v) for k, v in w.items()}
 
 
-def tensors(w):
-    import torch
-    return {k: torch.from_numpy(v).to(torch.bfloat16) for k, v in w.items()}
-
-
 def decoder(cfg, w, batch, max_len, dtype="float32", **kw):
     from poptransformer_b200 import registry
     return registry.build_decoder(cfg, tensors(w), batch, max_len, dtype, **kw)
-
-
-def write_model(path, cfg, w):
-    """config.json + model.safetensors (bfloat16)."""
-    import torch
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(cfg, f)
-    head, blobs, at = {}, [], 0
-    for k, t in tensors(w).items():
-        b = t.contiguous().view(torch.int16).numpy().tobytes()
-        head[k] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [at, at + len(b)]}
-        blobs.append(b)
-        at += len(b)
-    h = json.dumps(head).encode()
-    with open(os.path.join(path, "model.safetensors"), "wb") as f:
-        f.write(len(h).to_bytes(8, "little") + h + b"".join(blobs))
-
-
-def rel(got, want):
-    """rms of the difference over the rms of the expected values."""
-    got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
-    return float(np.sqrt(((got - want) ** 2).mean()) / np.sqrt((want ** 2).mean()))
 
 
 # configurations that differ in every size, the order of the layers, and the optional parts

@@ -11,25 +11,12 @@ import pytest
 import torch
 
 from oracle import sabisun_np as ref
-from sabisun_util import CONFIGS, attn, bf16, config, decoder, mamba, rel, weights, write_model
+from sabisun_util import CONFIGS, attn, config, decoder, mamba, weights
+from seq_util import PagedAttention, as_type, bf16, greedy_ok, i32, prompt, rel, run_cut, view_of, write_model
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 TOL = {"float32": 2e-5, "bfloat16": 2e-2}       # rms of the difference over the rms of the logits, whole model
-
-
-def i32(x, dev):
-    return torch.tensor(np.asarray(x), dtype=torch.int32, device=dev)
-
-
-def view_of(lens, starts, slots, dev):
-    from poptransformer_b200 import ops
-    cu = np.concatenate([[0], np.cumsum(lens)])
-    return ops.batch_view(len(lens), int(cu[-1]), i32(cu, dev), i32(starts, dev), i32(slots, dev), i32(np.repeat(np.arange(len(lens)), lens), dev))
-
-
-def as_type(x, dt, dev):
-    return torch.from_numpy(np.ascontiguousarray(x, dtype=np.float32)).to(dev).to(dt)
 
 
 # ------------------------------------------------------------------------------------------ mechanisms
@@ -106,37 +93,6 @@ def test_bf16_linear(cuda, rows, n, k):
         ops.linear(xp, lin.skinny, out, workspace=lws, alpha=0.7)
         assert rel(out.cpu(), want) < 1e-5
     assert int(flag.item()) == 0
-
-
-class PagedAttention:
-    """One attention call site over a cache whose pages lie in shuffled order."""
-
-    def __init__(self, dev, dt, n_seq, G, D, V, max_len, poison=True, page=64, seed=0):
-        from poptransformer_b200 import ops
-        self.ops, self.dev, self.dt, self.G, self.D, self.V = ops, dev, dt, G, D, V
-        pages = -(-max_len // page)
-        table = np.random.default_rng(seed).permutation(n_seq * pages).reshape(n_seq, pages)
-        self.cache = ops.PagedKVCache(n_seq, G, D, max_len, page, dev, i32(table, dev), v_dim=V, dtype=dt)
-        if poison:                                   # nothing may be read that was not written
-            self.cache.pool.fill_(float("nan"))
-        self.flag = torch.zeros(1, dtype=torch.int32, device=dev)
-
-    def __call__(self, q, k, v, lens, starts, slots, scale, window, keep, sink, plain):
-        """q [T, H, D], k [T, G, D], v [T, G, V] (None: read the cache only), packed.  Returns [T, H V]."""
-        ops, dev, T, H = self.ops, self.dev, q.shape[0], q.shape[1]
-        parts = [q.reshape(T, -1)] + ([] if k is None else [k.reshape(T, -1), v.reshape(T, -1)])
-        x = np.concatenate(parts, 1)
-        ld = x.shape[1] + (-x.shape[1]) % 8
-        buf = torch.zeros((T, ld), dtype=self.dt, device=dev)
-        buf[:, :x.shape[1]] = as_type(x, self.dt, dev)
-        out_ld = ops.pad_to(H * self.V, 64)
-        out = torch.full((T, out_ld), float("nan"), dtype=self.dt, device=dev)
-        ws = ops.window_attn_workspace(len(lens), H, self.V, self.cache.page_size, self.cache.max_len, window, keep, dev)
-        ops.window_attn(view_of(lens, starts, slots, dev), buf, ld, self.cache, out, out_ld, H, scale, window, keep,
-                        None if sink is None else as_type(sink, torch.float32, dev), append=k is not None, max_tokens_per_seq=max(lens), workspace=ws,
-                        error_flag=self.flag, plain=plain)
-        assert not out[:, H * self.V:].any() and int(self.flag.item()) == 0
-        return out[:, :H * self.V].float().cpu().numpy()
 
 
 ATTN_SHAPES = [  # heads, kv heads, dim, vdim, window, keep_first, sink
@@ -303,21 +259,6 @@ def test_decay_survives_long_running_sums(cuda):
 
 
 # ------------------------------------------------------------------------------------------ whole models
-def prompt(n, vocab, seed=0):
-    return np.random.default_rng(100 + seed).integers(0, vocab, n).astype(np.int32)
-
-
-def run_cut(dec, tokens, cuts):
-    """One sequence in portions; logits of every token."""
-    s, out, at = dec.open(), [], 0
-    for n in cuts:
-        out.append(dec.extend([(s, tokens[at:at + n], list(range(n)))]).cpu().numpy())
-        at += n
-    assert at == len(tokens)
-    dec.close(s)
-    return np.concatenate(out)
-
-
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("name", list(CONFIGS))
 def test_model_prompts_portions_and_decoding(cuda, name, dtype):
@@ -431,19 +372,6 @@ def test_first_tokens(cuda):
 
 
 # ------------------------------------------------------------------------------------------ the decode loop
-def greedy_ok(orc, ids, lens, tol):
-    """Every generated id is the oracle's best along the generated stream, or within `tol` of it (relative to the logits' rms)."""
-    exact = total = 0
-    for row, n in zip(ids, lens):
-        lg = orc.forward(row[:-1])
-        for i in range(n, len(row)):
-            best, got = lg[i - 1].max(), lg[i - 1][row[i]]
-            assert best - got <= tol * np.sqrt((lg[i - 1] ** 2).mean()), i
-            exact += int(lg[i - 1].argmax() == row[i])
-            total += 1
-    return exact / total
-
-
 @pytest.mark.parametrize("dtype,tol", [("float32", 1e-4), ("bfloat16", 8e-2)])
 def test_greedy_generation(cuda, dtype, tol):
     cfg = CONFIGS["mixed"]

@@ -9,7 +9,8 @@ import pytest
 import torch
 
 from oracle import sabisun_np as ref
-from sabisun_util import CONFIGS, attn, config, mamba, weights, write_model
+from sabisun_util import CONFIGS, attn, config, mamba, weights
+from seq_util import write_model
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
