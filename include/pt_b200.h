@@ -89,6 +89,7 @@ typedef struct pt_dense_ext {
   const int32_t *mul_ids;
   int n_groups, group_rows, group_x_div;
   const int32_t *group_of;
+  const int32_t *group_used; /* pt_gemm, optional: rows in use of every tile (the rest is neither multiplied nor written) */
 } pt_dense_ext;
 
 /* ---- Int4ToHalf -------------------------------------------------------------------
@@ -528,7 +529,8 @@ typedef struct pt_post_norm_args {
   const int32_t *row_index;
   const float *y;
   int y_ld;
-  const float *pair_y;    /* fp32 rows of width                                      */
+  const void *pair_y;     /* rows of width, pair_dtype PT_DT_F32 or PT_DT_BF16       */
+  int pair_dtype;
   int pair_ld, top;       /* top at most 64                                          */
   const float *pair_w;
   const int32_t *pair_row;
@@ -540,8 +542,8 @@ int pt_post_norm(const pt_post_norm_args *args, void *stream);
 
 /* Mixture of experts (csrc/moe.cu): the `top` experts of every token by router logit, softmax weights over the chosen ones, and the
  * layout of the grouped products.  tile = 0: only expert and weight are written.  tile > 0: the pairs (token, choice) are sorted by
- * expert into tiles of `tile` rows: pair_row [n_tok, top], tile_expert [max_tiles] (-1: unused), row_token [max_tiles * tile] (-1:
- * padding), and with h the rows of h_bytes each are copied to gathered [max_tiles * tile]. */
+ * expert into tiles of `tile` rows: pair_row [n_tok, top], tile_expert [max_tiles] (-1: unused), tile_rows [max_tiles] (rows in use), row_token
+ * [max_tiles * tile] (-1: padding), and with h the rows of h_bytes each are copied to gathered [max_tiles * tile]. */
 typedef struct pt_moe_route_args {
   int n_tok, experts, top;        /* at most 64 of 1024                              */
   const float *logits;
@@ -549,7 +551,7 @@ typedef struct pt_moe_route_args {
   int32_t *expert;                /* [n_tok, top]                                    */
   float *weight;                  /* [n_tok, top]                                    */
   int tile, max_tiles;
-  int32_t *pair_row, *tile_expert, *row_token;
+  int32_t *pair_row, *tile_expert, *tile_rows, *row_token;
   const void *h;
   int h_bytes;
   void *gathered;

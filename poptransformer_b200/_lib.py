@@ -18,7 +18,8 @@ class PtError(RuntimeError):
 
 class DenseExt(ctypes.Structure):
     _fields_ = [("bias", c_void_p), ("out2", c_void_p), ("out2_ld", c_int), ("split_n", c_int), ("limit", c_float), ("mul", c_void_p), ("mul_ld", c_int),
-                ("mul_ids", c_void_p), ("n_groups", c_int), ("group_rows", c_int), ("group_x_div", c_int), ("group_of", c_void_p)]
+                ("mul_ids", c_void_p), ("n_groups", c_int), ("group_rows", c_int), ("group_x_div", c_int), ("group_of", c_void_p),
+                ("group_used", c_void_p)]
 
 
 class LinearArgs(ctypes.Structure):
@@ -96,13 +97,13 @@ class MlstmArgs(ctypes.Structure):
 class PostNormArgs(ctypes.Structure):
     _fields_ = [("rows", c_int), ("width", c_int), ("dtype", c_int), ("eps", c_float), ("x_in", c_void_p), ("x_out", c_void_p), ("table", c_void_p),
                 ("table_ld", c_int), ("vocab", c_int), ("ids", c_void_p), ("ids_ld", c_int)] + \
-               [(n, c_void_p) for n in ("step_dev", "pos_out", "id_out", "row_index", "y")] + [("y_ld", c_int), ("pair_y", c_void_p), ("pair_ld", c_int), ("top", c_int)] + \
+               [(n, c_void_p) for n in ("step_dev", "pos_out", "id_out", "row_index", "y")] + [("y_ld", c_int), ("pair_y", c_void_p), ("pair_dtype", c_int), ("pair_ld", c_int), ("top", c_int)] + \
                [(n, c_void_p) for n in ("pair_w", "pair_row", "norm_w", "final_w", "h")] + [("h_ld", c_int)]
 
 
 class MoeRouteArgs(ctypes.Structure):
     _fields_ = [("n_tok", c_int), ("experts", c_int), ("top", c_int), ("logits", c_void_p), ("logits_ld", c_int), ("expert", c_void_p), ("weight", c_void_p),
-                ("tile", c_int), ("max_tiles", c_int), ("pair_row", c_void_p), ("tile_expert", c_void_p), ("row_token", c_void_p), ("h", c_void_p), ("h_bytes", c_int),
+                ("tile", c_int), ("max_tiles", c_int), ("pair_row", c_void_p), ("tile_expert", c_void_p), ("tile_rows", c_void_p), ("row_token", c_void_p), ("h", c_void_p), ("h_bytes", c_int),
                 ("gathered", c_void_p)]
 
 

@@ -66,6 +66,8 @@ struct GemmParams {
   int *error_flag;
   DenseOut dense;         // BF16: what becomes of a finished sum
   const int *group_of;    // BF16, grouped: the weight matrix of every tile of mb rows (negative: none)
+  const int *group_used;  // ... and how many of its rows are in use (null: all)
+  int n_tiles;            // tiles of 128 weight rows
   size_t group_stride;    // bytes between weight matrices
 };
 
@@ -202,9 +204,9 @@ template <bool BF16> __device__ __forceinline__ void store_out(const GemmParams 
 // Epilogue of the warps that own the tile's rows (tensor-memory lane quarter warp % 4): `part` of `parts` warps share a quarter
 // and take alternate 16-column chunks.
 template <bool BF16>
-__device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int q, int lane, int part, int parts, int n0, int m0, int ks, int c_first = 0) {
+__device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int q, int lane, int part, int parts, int n0, int m0, int m_end, int ks, int c_first = 0) {
   const int n = n0 + q * 32 + lane;
-  for (int c0 = c_first + part * 16; c0 < p.mb; c0 += 16 * parts) {
+  for (int c0 = c_first + part * 16; c0 < min(p.mb, m_end - m0); c0 += 16 * parts) {
     uint32_t v[16];
     float sum[16];
     tmem_ld16(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, v);
@@ -215,7 +217,7 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           const float up = __shfl_xor_sync(0xffffffffu, sum[j], 8);
-          if (n < p.N && m0 + c0 + j < p.M && (lane & 8) == 0) dense_store_glu(p.dense, m0 + c0 + j, n, sum[j], up);
+          if (n < p.N && m0 + c0 + j < m_end && (lane & 8) == 0) dense_store_glu(p.dense, m0 + c0 + j, n, sum[j], up);
         }
         continue;
       }
@@ -224,7 +226,7 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
         const int m = m0 + c0 + j;
-        if (m >= p.M) break;
+        if (m >= m_end) break;
         const float acc = sum[j];
         if (p.ksplit > 1) {
           p.partial[((size_t)ks * p.M + m) * p.N + n] = acc;
@@ -278,7 +280,7 @@ __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, in
     }
   }
 }
-__device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem, int q, int lane, int n0, int m0, int ks) {
+__device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem, int q, int lane, int n0, int m0, int m_end, int ks) {
   const DenseOut &d = p.dense;
   const int nq = n0 + q * 32, n = nq + lane;
   // (warp-uniform) where this warp's 32 outputs go
@@ -286,7 +288,7 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
   // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16
   const bool fast = p.ksplit == 1 && nq + 32 <= p.N && (second || d.epilogue != PT_EPI_GELU_MUL) && !(glu && f32) &&
                     (f32 || glu || (d.out_ld % 2 == 0 && ((uintptr_t)d.out & 3) == 0));
-  const int whole = fast ? min(p.mb, p.M - m0) & ~31 : 0;
+  const int rows = min(p.mb, m_end - m0), whole = fast ? rows & ~31 : 0;
   for (int c0 = 0; c0 < whole; c0 += 32) {
     uint32_t v[32];
     tmem_ld32(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, v);
@@ -302,12 +304,12 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
       else epilogue_rows32<OUT_BF16, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     }
   }
-  if (whole < p.mb) epilogue<true>(p, tmem, q, lane, 0, 1, n0, m0, ks, whole);
+  if (whole < rows) epilogue<true>(p, tmem, q, lane, 0, 1, n0, m0, m_end, ks, whole);
 }
 
 // k-slices of this tile meet: the last CTA to arrive sums them in slice order.
 template <bool BF16>
-__device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ctl, int n0, int m0, int threads) {
+__device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ctl, int n0, int m0, int m_end, int threads) {
   const int tid = threadIdx.x;
   __threadfence();
   __syncthreads();
@@ -320,7 +322,7 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
   if (ctl.last && !ctl.abort) {
     __threadfence();
     // every thread sums the slices of one output element at a time, all slices' loads in flight together (at most 8 per batch)
-    const int rows = min(p.mb, p.M - m0);
+    const int rows = min(p.mb, m_end - m0);
     if constexpr (BF16) {
       if (p.N % 4 == 0) {   // four outputs per thread and step: a quarter of the trips to L2
         for (int i = tid; i < rows * (BM / 4); i += threads) {
@@ -382,8 +384,9 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
 }
 
 // ------------------------------------------------------------------------------------------ FP8 and BF16
-// Dynamic shared memory: [stage][A tile 16 KB | B tile mb * 128 B], every tile 1024-byte aligned.
-template <bool BF16>
+// Dynamic shared memory: [stage][NA A tiles of 16 KB | B tile mb * 128 B], every tile 1024-byte aligned.  NA = 2: a CTA takes 256 weight
+// rows (two accumulators), which fetches a third less per product than NA = 1; without k-slices.
+template <bool BF16, int NA>
 __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                                                                    const GemmParams p) {
   constexpr int KX = BF16 ? BKB / 2 : BKB;   // elements of k per stage
@@ -391,22 +394,28 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
   __shared__ SharedCtl ctl;
   unsigned char *smem = (unsigned char *)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int n0 = blockIdx.x * BM, m0 = blockIdx.z * p.mb, ks = blockIdx.y;
+  const int n0 = blockIdx.x * (BM * NA), m0 = blockIdx.z * p.mb, ks = blockIdx.y;
   const int kb0 = ks * p.kb_per_split, kb1 = min(p.n_kb, kb0 + p.kb_per_split);
-  const int n_it = kb1 - kb0;
+  const int n_it = kb1 - kb0, na = NA == 1 ? 1 : min(NA, p.n_tiles - (int)blockIdx.x * NA);
   const uint32_t b_bytes = (uint32_t)p.mb * BKB;
-  const uint32_t stage_bytes = A_TILE + ((b_bytes + 1023u) & ~1023u);
+  const uint32_t stage_bytes = NA * A_TILE + ((b_bytes + 1023u) & ~1023u);
   const uint32_t smem_s = sa(smem);
+  int m_end = min(p.M, m0 + p.mb), mma_n = p.mb;
   size_t w_base = 0;
   if constexpr (BF16) {
     if (p.group_of) {
       const int grp = p.group_of[blockIdx.z];
       if (grp < 0) return;                     // a tile without rows: nothing is initialised yet
       w_base = (size_t)grp * p.group_stride;
+      if (p.group_used) {
+        m_end = m0 + min(p.mb, p.group_used[blockIdx.z]);
+        mma_n = max(16, (m_end - m0 + 15) & ~15);
+      }
     }
   }
-  uint32_t tmem_cols = 32;
-  while ((int)tmem_cols < p.mb) tmem_cols <<= 1;
+  uint32_t acc_cols = 32;
+  while ((int)acc_cols < p.mb) acc_cols <<= 1;
+  const uint32_t tmem_cols = NA * acc_cols;
 
   if (tid == 0) {
     for (int s = 0; s < p.stages; ++s) {
@@ -427,8 +436,9 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
   if (warp == 0) {
     if (lane == 0) {
       // (ring positions and parities are carried as counters: this thread's instruction count per stage is what limits a CTA)
-      const unsigned char *wt = p.w + w_base + ((size_t)blockIdx.x * p.n_kb + kb0) * A_TILE;
-      const uint32_t tx = A_TILE + b_bytes, full0 = sa(&ctl.full[0]), empty0 = sa(&ctl.empty[0]);
+      const unsigned char *wt = p.w + w_base + ((size_t)blockIdx.x * NA * p.n_kb + kb0) * A_TILE;
+      const size_t next_tile = (size_t)p.n_kb * A_TILE;
+      const uint32_t tx = na * A_TILE + b_bytes, full0 = sa(&ctl.full[0]), empty0 = sa(&ctl.empty[0]);
       const bool tiled = p.w_tiled != 0;
       int s = 0, kx = kb0 * KX;
       uint32_t par = 1;   // parity of the `empty` phase that must have completed before slot s is refilled (none in the first round)
@@ -438,9 +448,13 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
         if (ctl.abort) break;
         const uint32_t st = smem_s + s * stage_bytes, fb = full0 + s * 8;
         mbar_expect_tx(fb, tx);
-        if (tiled) bulk_g2s(st, wt, A_TILE, fb);
-        else tma_load_2d(st, &map_w, kx, n0, fb);
-        tma_load_2d(st + A_TILE, &map_x, kx, m0, fb);
+        if (tiled) {
+          bulk_g2s(st, wt, A_TILE, fb);
+          if (NA == 2 && na == 2) bulk_g2s(st + A_TILE, wt + next_tile, A_TILE, fb);
+        } else {
+          tma_load_2d(st, &map_w, kx, n0, fb);
+        }
+        tma_load_2d(st + NA * A_TILE, &map_x, kx, m0, fb);
         wt += A_TILE;
         kx += KX;
         if (++s == p.stages) { s = 0; par ^= 1u; first_round = false; }
@@ -451,8 +465,8 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
       // One thread issues every MMA of the CTA, so its loop is kept to a few dozen instructions per stage: descriptors are one
       // 64-bit add away from the stage-0 descriptors (the start-address field counts 16-byte units), ring position and parity
       // are counters.  (Measured: with divisions and descriptor rebuilds in this loop a stage took 0.6 us whatever its size.)
-      const uint32_t idesc = instr_desc(BF16, p.mb);
-      const uint64_t adesc0 = smem_desc_sw128(smem_s), bdesc0 = smem_desc_sw128(smem_s + A_TILE);
+      const uint32_t idesc = instr_desc(BF16, mma_n);
+      const uint64_t adesc0 = smem_desc_sw128(smem_s), bdesc0 = smem_desc_sw128(smem_s + NA * A_TILE);
       const uint32_t full0 = sa(&ctl.full[0]), empty0 = sa(&ctl.empty[0]), stage16 = stage_bytes >> 4;
       int s = 0;
       uint32_t par = 0, acc = 0;
@@ -465,6 +479,13 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
         umma<!BF16>(tmem, adesc + 2, bdesc + 2, idesc, 1u);
         umma<!BF16>(tmem, adesc + 4, bdesc + 4, idesc, 1u);
         umma<!BF16>(tmem, adesc + 6, bdesc + 6, idesc, 1u);
+        if (NA == 2 && na == 2) {
+          const uint64_t a2 = adesc + (A_TILE >> 4);
+          umma<!BF16>(tmem + acc_cols, a2, bdesc, idesc, acc);
+          umma<!BF16>(tmem + acc_cols, a2 + 2, bdesc + 2, idesc, 1u);
+          umma<!BF16>(tmem + acc_cols, a2 + 4, bdesc + 4, idesc, 1u);
+          umma<!BF16>(tmem + acc_cols, a2 + 6, bdesc + 6, idesc, 1u);
+        }
         umma_commit(empty0 + s * 8);
         acc = 1u;
         if (++s == p.stages) { s = 0; par ^= 1u; }
@@ -475,12 +496,15 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
     if (!mbar_wait(sa(&ctl.accum), 0, &ctl.abort)) give_up(ctl, p.error_flag, 24);
     fence_after();
     if (!ctl.abort && n_it > 0) {
-      if constexpr (BF16) epilogue_bf16(p, tmem, warp & 3, lane, n0, m0, ks);
-      else epilogue<false>(p, tmem, warp & 3, lane, 0, 1, n0, m0, ks);
+      if constexpr (BF16) {
+        for (int a = 0; a < na; ++a) epilogue_bf16(p, tmem + a * acc_cols, warp & 3, lane, n0 + a * BM, m0, m_end, ks);
+      } else {
+        epilogue<false>(p, tmem, warp & 3, lane, 0, 1, n0, m0, m_end, ks);
+      }
     }
     fence_before();
   }
-  if (p.ksplit > 1) reduce_slices<BF16>(p, ctl, n0, m0, THREADS_F8);
+  if (NA == 1 && p.ksplit > 1) reduce_slices<BF16>(p, ctl, n0, m0, m_end, THREADS_F8);
   __syncthreads();
   fence_after();
   if (warp == 1) tmem_dealloc(tmem, tmem_cols);
@@ -641,10 +665,10 @@ __global__ void __launch_bounds__(THREADS_I4, 1) gemm_int4_kernel(const __grid_c
     }
     if (!mbar_wait(sa(&ctl.accum), 0, &ctl.abort)) give_up(ctl, p.error_flag, 24);
     fence_after();
-    if (!ctl.abort && n_it > 0) epilogue<false>(p, tmem, q, lane, half, 2, n0, m0, ks);
+    if (!ctl.abort && n_it > 0) epilogue<false>(p, tmem, q, lane, half, 2, n0, m0, p.M, ks);
     fence_before();
   }
-  if (p.ksplit > 1) reduce_slices<false>(p, ctl, n0, m0, THREADS_I4);
+  if (p.ksplit > 1) reduce_slices<false>(p, ctl, n0, m0, p.M, THREADS_I4);
   __syncthreads();
   fence_after();
   if (warp == 1) tmem_dealloc(tmem, tmem_cols);
@@ -799,6 +823,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
     PT_REQUIRE(p.mb % 16 == 0 && p.mb >= 16 && p.mb <= 256 && a->m % p.mb == 0 && a->m / p.mb <= 65535, "pt_gemm: groups of %d rows (16 .. 256 in steps of 16) in %d rows",
                p.mb, a->m);
     p.group_of = a->ext->group_of;
+    p.group_used = a->ext->group_used;
     p.group_stride = pt_gemm_packed_bytes(a->wfmt, a->n_out, a->k_in);
   } else if (bf16)
     while (p.mb > 64 && n_tiles * ceil_div(a->m, p.mb) * 4 < sm_count() * 3) p.mb = ceil_div(p.mb, 32) * 16;
@@ -837,8 +862,15 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
     p.partial = (float *)((char *)a->workspace + kGemmCounterBytes);
   }
 
+  // BF16 without k-slices: two weight tiles per CTA when half as many CTAs still fill the GPU
+#ifndef PT_TC_PAIR
+#define PT_TC_PAIR 1
+#endif
+  const bool pair = PT_TC_PAIR && bf16 && p.ksplit == 1 && p.mb >= 128 && n_tiles >= 2 && (long long)ceil_div(n_tiles, 2) * m_tiles >= sm_count();
+  const int na = pair ? 2 : 1;
+  p.n_tiles = n_tiles;
   const uint32_t b_bytes = (uint32_t)p.mb * tc::BKB;
-  const uint32_t stage_bytes = tc::A_TILE + ((b_bytes + 1023u) & ~1023u);
+  const uint32_t stage_bytes = na * tc::A_TILE + ((b_bytes + 1023u) & ~1023u);
   // Up to 64 activation rows a stage is small, and what limits the kernel is the one thread per CTA that issues the MMAs (about
   // 75 cycles per tcgen05.mma whatever its N): two CTAs per SM (half the shared memory each) issue side by side.  Measured on
   // B200, FP8 65024 x 4096 at 8 / 32 rows: 63 / 66 us with one CTA per SM, 45 / 47 us with two.
@@ -847,7 +879,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
 #endif
   // BF16 also with large tiles when there are more of them than SMs: the epilogue of one CTA then hides behind the products of the
   // other (two accumulators of 256 columns fill the tensor memory).
-  const bool small = p.mb <= 64 || (bf16 && (long long)n_tiles * m_tiles * p.ksplit > sm_count());
+  const bool small = p.mb <= 64 || (bf16 && na * p.mb <= 256 && (long long)n_tiles * m_tiles * p.ksplit > sm_count());
   const uint32_t budget = (small ? PT_TC_BUDGET_SMALL_KB : 200) * 1024u;
   size_t smem;
   if (int4) {
@@ -859,7 +891,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
     p.stages = (int)std::min<uint32_t>(8, budget / stage_bytes);
     PT_REQUIRE(p.stages >= 2, "pt_gemm: tile does not fit shared memory");
     smem = (size_t)p.stages * stage_bytes + 1024;
-    if (bf16 && p.mb > 64) smem = std::max<size_t>(smem, 80 * 1024);   // never more CTAs on an SM than its tensor memory holds accumulators for
+    if (bf16 && p.mb > 64) smem = std::max<size_t>(smem, (na * p.mb > 256 ? 120 : 80) * 1024);   // never more CTAs on an SM than its tensor memory holds accumulators for
   }
 
   CUtensorMap map_w, map_x;
@@ -875,18 +907,19 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   }
   static bool attr_set = false;
   if (!attr_set) {
-    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<false, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     PT_CUDA(cudaFuncSetAttribute(tc::gemm_int4_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     attr_set = true;
   }
-  dim3 grid(n_tiles, p.ksplit, m_tiles);
+  dim3 grid(ceil_div(n_tiles, na), p.ksplit, m_tiles);
   if (int4)
     tc::gemm_int4_kernel<<<grid, tc::THREADS_I4, smem, as_stream(stream)>>>(map_x, p);
   else if (bf16)
-    tc::gemm_dense_kernel<true><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
+    (pair ? tc::gemm_dense_kernel<true, 2> : tc::gemm_dense_kernel<true, 1>)<<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
   else
-    tc::gemm_dense_kernel<false><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
+    tc::gemm_dense_kernel<false, 1><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
   PT_LAUNCH_CHECK("pt_gemm");
   return PT_OK;
 }

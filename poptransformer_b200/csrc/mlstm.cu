@@ -514,22 +514,50 @@ template <typename T, int VEC> __device__ __forceinline__ void norm_gate_row(con
       v[0] = __ldcg(y + i);
     }
   };
-  float ss = 0.f;
-  for (int i = lane * VEC; i < p.P; i += 32 * VEC) {
-    float v[VEC];
-    load(i, v);
+  auto squares = [](const float (&v)[VEC]) {
+    float s = 0.f;
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
-  }
-  const float inv = p.out_scale / sqrtf(warp_sum(ss) / (float)p.P + p.eps);
-  for (int i = lane * VEC; i < p.P; i += 32 * VEC) {
-    float v[VEC], a[VEC], b[VEC];
-    load(i, v);
+    for (int j = 0; j < VEC; ++j) s = fmaf(v[j], v[j], s);
+    return s;
+  };
+  auto scale = [&](float ss) { return p.out_scale / sqrtf(warp_sum(ss) / (float)p.P + p.eps); };
+  auto finish = [&](int i, float (&v)[VEC], float (&b)[VEC], float inv) {
+    float a[VEC];
     load_vec<VEC>(w + i, a);
-    load_vec<VEC>(gate + i, b);
 #pragma unroll
     for (int j = 0; j < VEC; ++j) v[j] *= inv * a[j] * sigmoid_f(b[j]);
     store_vec<VEC>(out + i, v);
+  };
+  constexpr int R = 2;                          // a head of up to 32 R VEC values stays in registers
+  if (p.P <= 32 * R * VEC) {
+    float v[R][VEC], b[R][VEC], ss = 0.f;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = (lane + 32 * r) * VEC;
+      if (i < p.P) {
+        load(i, v[r]);
+        load_vec<VEC>(gate + i, b[r]);
+        ss += squares(v[r]);
+      }
+    }
+    const float inv = scale(ss);
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if ((lane + 32 * r) * VEC < p.P) finish((lane + 32 * r) * VEC, v[r], b[r], inv);
+  } else {
+    float ss = 0.f;
+    for (int i = lane * VEC; i < p.P; i += 32 * VEC) {
+      float v[VEC];
+      load(i, v);
+      ss += squares(v);
+    }
+    const float inv = scale(ss);
+    for (int i = lane * VEC; i < p.P; i += 32 * VEC) {
+      float v[VEC], b[VEC];
+      load(i, v);
+      load_vec<VEC>(gate + i, b);
+      finish(i, v, b, inv);
+    }
   }
   if (h == p.heads - 1)   // k padding of the output product
     for (int i = p.inner + lane; i < p.out_cols; i += 32) reinterpret_cast<T *>(p.out)[(size_t)t * p.out_ld + i] = from_f<T>(0.f);

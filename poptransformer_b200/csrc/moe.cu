@@ -2,8 +2,8 @@
 //   choose   per token the `top` experts with the largest router logits (the lowest index first among equals), and the softmax over
 //            those logits as weights.  fp32.
 //   place    pair i = token i / top with its choice i % top gets a row of its own among its expert's rows.  The rows of an expert are
-//            padded to whole tiles; tile_expert names the expert of every tile (-1: unused), so a grouped product can look its weights
-//            up per tile.  Pairs keep their order within an expert.
+//            padded to whole tiles; tile_expert names the expert of every tile (-1: unused) and tile_rows its rows in use, so a grouped
+//            product can look its weights up per tile.  Pairs keep their order within an expert.
 //   gather   the tokens' activations are copied to their pairs' rows (zeros in the padding).
 // With few tokens every pair is a tile of one row and nothing is placed or copied.
 #include <limits.h>
@@ -16,9 +16,9 @@ namespace moe {
 constexpr int kMaxExperts = 1024, kMaxTop = 64, PLACE_THREADS = 1024;
 
 struct Params {
-  int n_tok, experts, top, logits_ld, tile, max_tiles;
+  int n_tok, experts, top, logits_ld, tile, max_tiles, hist_copies;
   const float *logits;
-  int *expert, *pair_row, *tile_expert, *row_token;   // [n_tok][top] x 2, [max_tiles], [max_tiles * tile]
+  int *expert, *pair_row, *tile_expert, *tile_rows, *row_token;   // [n_tok][top] x 2, [max_tiles] x 2, [max_tiles * tile]
   float *weight;                                      // [n_tok][top]
 };
 
@@ -58,19 +58,41 @@ __global__ void choose_kernel(const Params p) {
   if (lane + 32 < p.top) p.weight[(size_t)t * p.top + lane + 32] = w1 / sum;
 }
 
-// Block e places the pairs of expert e: every block counts all experts' pairs (for the tiles in front of its own), then walks the pairs once more.
+// Block e places the pairs of expert e: every block counts all experts' pairs (for the tiles in front of its own), then its own pairs
+// get their rows.  Thread i looks at a run of consecutive pairs, so the order within an expert is the order of the pairs.
 __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
-  __shared__ int count[kMaxExperts], warps[PLACE_THREADS / 32];
+  extern __shared__ int hist[];                   // [copies][experts]: warps count into copies of their own while they fit
+  __shared__ int warps[PLACE_THREADS / 32];
   __shared__ int first, total;
   const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, pairs = p.n_tok * p.top;
-  for (int i = tid; i < p.experts; i += PLACE_THREADS) count[i] = 0;
+  const int per = (pairs + PLACE_THREADS - 1) / PLACE_THREADS, i0 = min(pairs, tid * per), i1 = min(pairs, i0 + per);
+  int *mine = hist + (warp % p.hist_copies) * p.experts;
+  for (int i = tid; i < p.hist_copies * p.experts; i += PLACE_THREADS) hist[i] = 0;
   __syncthreads();
-  for (int i = tid; i < pairs; i += PLACE_THREADS) atomicAdd(&count[p.expert[i]], 1);
+  int hits = 0;
+  for (int i = i0; i < i1; ++i) {
+    const int x = p.expert[i];
+    atomicAdd(mine + x, 1);
+    hits += x == e;
+  }
+  __syncthreads();
+  for (int i = tid; i < p.experts; i += PLACE_THREADS) {
+    int n = 0;
+    for (int c = 0; c < p.hist_copies; ++c) n += hist[c * p.experts + i];
+    hist[i] = n;                                  // (the same thread read copy 0 of this expert just before)
+  }
+  int scan = hits;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int v = __shfl_up_sync(0xffffffffu, scan, o);
+    if (lane >= o) scan += v;
+  }
+  if (lane == 31) warps[warp] = scan;
   __syncthreads();
   if (warp == 0) {
     int before = 0, all = 0;
     for (int i = lane; i < p.experts; i += 32) {
-      const int tiles = (count[i] + p.tile - 1) / p.tile;
+      const int tiles = (hist[i] + p.tile - 1) / p.tile;
       all += tiles;
       if (i < e) before += tiles;
     }
@@ -80,36 +102,33 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
       all += __shfl_xor_sync(0xffffffffu, all, o);
     }
     if (lane == 0) { first = before; total = all; }
+  } else if (warp == 1) {
+    const int own = warps[lane];
+    int sum = own;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += v;
+    }
+    warps[lane] = sum - own;
   }
   __syncthreads();
-  const int mine = count[e], tiles = (mine + p.tile - 1) / p.tile, row0 = first * p.tile;
-  for (int i = tid; i < tiles; i += PLACE_THREADS) p.tile_expert[first + i] = e;
-  for (int i = mine + tid; i < tiles * p.tile; i += PLACE_THREADS) p.row_token[row0 + i] = -1;
+  const int count = hist[e], tiles = (count + p.tile - 1) / p.tile, row0 = first * p.tile;
+  for (int i = tid; i < tiles; i += PLACE_THREADS) {
+    p.tile_expert[first + i] = e;
+    p.tile_rows[first + i] = min(p.tile, count - i * p.tile);
+  }
+  for (int i = count + tid; i < tiles * p.tile; i += PLACE_THREADS) p.row_token[row0 + i] = -1;
   if (e == 0) {
-    for (int i = total + tid; i < p.max_tiles; i += PLACE_THREADS) p.tile_expert[i] = -1;
+    for (int i = total + tid; i < p.max_tiles; i += PLACE_THREADS) { p.tile_expert[i] = -1; p.tile_rows[i] = 0; }
     for (int i = total * p.tile + tid; i < p.max_tiles * p.tile; i += PLACE_THREADS) p.row_token[i] = -1;
   }
-  int next = row0;
-  for (int i0 = 0; i0 < pairs; i0 += PLACE_THREADS) {
-    const int i = i0 + tid;
-    const bool hit = i < pairs && p.expert[i] == e;
-    const unsigned vote = __ballot_sync(0xffffffffu, hit);
-    if (lane == 0) warps[warp] = __popc(vote);
-    __syncthreads();
-    int before = 0, all = 0;
-    for (int w = 0; w < PLACE_THREADS / 32; ++w) {
-      const int n = warps[w];
-      all += n;
-      if (w < warp) before += n;
-    }
-    if (hit) {
-      const int row = next + before + __popc(vote & ((1u << lane) - 1u));
+  int row = row0 + warps[warp] + scan - hits;
+  for (int i = i0; hits > 0 && i < i1; ++i)
+    if (p.expert[i] == e) {
       p.pair_row[i] = row;
-      p.row_token[row] = i / p.top;
+      p.row_token[row++] = i / p.top;
     }
-    next += all;
-    __syncthreads();
-  }
 }
 
 // Rows of h (whole 16-byte units) to where row_token says.
@@ -146,10 +165,11 @@ extern "C" int pt_moe_route(const pt_moe_route_args *a, void *stream) {
   moe::choose_kernel<<<ceil_div(p.n_tok, 4), 128, 0, st>>>(p);
   PT_LAUNCH_CHECK("pt_moe_route");
   if (!a->tile) return PT_OK;
-  PT_REQUIRE(a->tile > 0 && a->pair_row && a->tile_expert && a->row_token && a->max_tiles >= pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile),
+  PT_REQUIRE(a->tile > 0 && a->pair_row && a->tile_expert && a->tile_rows && a->row_token && a->max_tiles >= pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile),
              "pt_moe_route: tiles of %d rows need pair_row, row_token and %d entries of tile_expert", a->tile, pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile));
-  p.tile = a->tile; p.max_tiles = a->max_tiles; p.pair_row = a->pair_row; p.tile_expert = a->tile_expert; p.row_token = a->row_token;
-  moe::place_kernel<<<p.experts, moe::PLACE_THREADS, 0, st>>>(p);
+  p.tile = a->tile; p.max_tiles = a->max_tiles; p.pair_row = a->pair_row; p.tile_expert = a->tile_expert; p.tile_rows = a->tile_rows; p.row_token = a->row_token;
+  p.hist_copies = std::max(1, std::min(32, 8192 / p.experts));
+  moe::place_kernel<<<p.experts, moe::PLACE_THREADS, (size_t)p.hist_copies * p.experts * sizeof(int), st>>>(p);
   PT_LAUNCH_CHECK("pt_moe_route");
   if (a->h) {
     PT_REQUIRE(a->gathered && a->h_bytes > 0 && a->h_bytes % 4 == 0, "pt_moe_route: rows of %d bytes", a->h_bytes);

@@ -19,7 +19,8 @@ struct Params {
   const int *ids, *step;
   int *pos_out, *id_out;
   const int *row_index;
-  const float *y, *pair_y, *pair_w;
+  const float *y, *pair_w;
+  const void *pair_y;
   const int *pair_row;
   const float *norm_w, *final_w;
   void *h;
@@ -27,7 +28,7 @@ struct Params {
 
 template <int VEC> __device__ __forceinline__ void put_f32(float *p, const float (&v)[VEC]) { store_vec<VEC>(p, v); }
 
-template <typename T, int VEC> __global__ void post_norm_kernel(const Params p) {
+template <typename T, typename E, int VEC> __global__ void post_norm_kernel(const Params p) {
   extern __shared__ __align__(16) float row[];     // [width]: y, then the new x
   __shared__ float red[32], pw[kMaxTop];
   __shared__ int pr[kMaxTop];
@@ -71,7 +72,7 @@ template <typename T, int VEC> __global__ void post_norm_kernel(const Params p) 
 #pragma unroll 4
     for (int k = 0; k < p.top; ++k) {
       float e[VEC];
-      load_vec<VEC>(p.pair_y + (size_t)pr[k] * p.pair_ld + i, e);
+      load_vec<VEC>(reinterpret_cast<const E *>(p.pair_y) + (size_t)pr[k] * p.pair_ld + i, e);
       const float w = pw[k];
 #pragma unroll
       for (int j = 0; j < VEC; ++j) v[j] = fmaf(w, e[j], v[j]);
@@ -108,15 +109,15 @@ template <typename T, int VEC> __global__ void post_norm_kernel(const Params p) 
   }
 }
 
-template <typename T, int VEC> static int launch(const Params &p, cudaStream_t st) {
+template <typename T, typename E, int VEC> static int launch(const Params &p, cudaStream_t st) {
   const size_t smem = (size_t)p.width * sizeof(float);
   if (smem > 48 * 1024) {
     static bool set = false;
-    if (!set) { PT_CUDA(cudaFuncSetAttribute(post_norm_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
+    if (!set) { PT_CUDA(cudaFuncSetAttribute(post_norm_kernel<T, E, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
   }
   // few rows: as many threads per row as it has work for; many rows: more rows per SM
   const int want = ceil_div(ceil_div(p.width, VEC), 32) * 32, cap = p.rows <= 2 * sm_count() ? 1024 : 256;
-  post_norm_kernel<T, VEC><<<p.rows, std::max(64, std::min(want, cap)), smem, st>>>(p);
+  post_norm_kernel<T, E, VEC><<<p.rows, std::max(64, std::min(want, cap)), smem, st>>>(p);
   PT_LAUNCH_CHECK("pt_post_norm");
   return PT_OK;
 }
@@ -138,6 +139,8 @@ extern "C" int pt_post_norm(const pt_post_norm_args *a, void *stream) {
     PT_REQUIRE(!a->y || a->y_ld >= a->width, "pt_post_norm: y_ld=%d", a->y_ld);
     PT_REQUIRE(a->top >= 0 && a->top <= post::kMaxTop && (!a->top || (a->pair_y && a->pair_w && a->pair_ld >= a->width)),
                "pt_post_norm: %d experts per token (at most %d) need pair_y, pair_w and pair_ld", a->top, post::kMaxTop);
+    PT_REQUIRE(!a->top || a->pair_dtype == PT_DT_F32 || (a->pair_dtype == PT_DT_BF16 && a->dtype == PT_DT_BF16), "pt_post_norm: experts' outputs of type %d",
+               a->pair_dtype);
   }
   post::Params p{};
   p.rows = a->rows; p.width = a->width; p.h_ld = a->h_ld; p.table_ld = a->table_ld; p.vocab = a->vocab; p.ids_ld = a->ids_ld; p.y_ld = a->y_ld;
@@ -146,10 +149,12 @@ extern "C" int pt_post_norm(const pt_post_norm_args *a, void *stream) {
   p.row_index = a->row_index; p.y = a->y; p.pair_y = a->pair_y; p.pair_w = a->pair_w; p.pair_row = a->pair_row;
   p.norm_w = a->norm_w; p.final_w = a->final_w; p.h = a->h;
   const int vb = a->dtype == PT_DT_F32 ? 16 : 8;
-  const bool v4 = a->width % 4 == 0 && aligned_to(a->x_in, 16) && aligned_to(a->x_out, 16) && aligned_to(a->y, 16) && a->y_ld % 4 == 0 && aligned_to(a->pair_y, 16) &&
+  const bool v4 = a->width % 4 == 0 && aligned_to(a->x_in, 16) && aligned_to(a->x_out, 16) && aligned_to(a->y, 16) && a->y_ld % 4 == 0 && aligned_to(a->pair_y, a->pair_dtype == PT_DT_F32 ? 16 : 8) &&
                   a->pair_ld % 4 == 0 && aligned_to(a->norm_w, 16) && aligned_to(a->final_w, 16) && aligned_to(a->h, vb) && a->h_ld % 4 == 0 && aligned_to(a->table, vb) &&
                   a->table_ld % 4 == 0;
   cudaStream_t st = as_stream(stream);
-  if (a->dtype == PT_DT_F32) return v4 ? post::launch<float, 4>(p, st) : post::launch<float, 1>(p, st);
-  return v4 ? post::launch<__nv_bfloat16, 4>(p, st) : post::launch<__nv_bfloat16, 1>(p, st);
+  typedef __nv_bfloat16 B;
+  if (a->dtype == PT_DT_F32) return v4 ? post::launch<float, float, 4>(p, st) : post::launch<float, float, 1>(p, st);
+  if (p.top > 0 && a->pair_dtype == PT_DT_BF16) return v4 ? post::launch<B, B, 4>(p, st) : post::launch<B, B, 1>(p, st);
+  return v4 ? post::launch<B, float, 4>(p, st) : post::launch<B, float, 1>(p, st);
 }

@@ -58,28 +58,57 @@ __device__ __forceinline__ int window_page(const Params &p, int pos) { return p.
 __device__ __forceinline__ int kept_pages(const Params &p, int pos) { return (min(p.keep_first, pos + 1) + p.page - 1) / p.page; }
 
 // ------------------------------------------------------------------------------------------ norm, rotation, append
-// One warp: a head's row of a query or key.  put(i, value) may write over src (a lane reads what it writes).
+// One warp: a head's row of a query or key.  put(i, value) may write over src (a lane reads what it writes).  A unit is the pair
+// (u, u + half) that turns together, or two neighbours behind the rotated dimensions.  Up to 128 dimensions the row stays in registers.
 template <typename T, typename Put>
 __device__ __forceinline__ void norm_rotate(const Params &p, const T *src, const float *norm, int pos, Put put) {
-  const int lane = threadIdx.x & 31;
-  float inv = 1.f;
-  if (norm) {
-    float ss = 0.f;
-    for (int i = lane; i < p.dim; i += 32) {
-      const float x = to_f(src[i]);
-      ss = fmaf(x, x, ss);
+  const int lane = threadIdx.x & 31, half = p.rope_half, units = (p.dim + 1) / 2;
+  const float2 *cs = p.rope + (size_t)pos * half;
+  auto first = [&](int u) { return u < half ? u : 2 * u; };            // 2 half + 2 (u - half)
+  auto second = [&](int u) { return u < half ? u + half : 2 * u + 1; };
+  auto load = [&](int u, float &x, float &y) {
+    x = to_f(src[first(u)]);
+    y = second(u) < p.dim ? to_f(src[second(u)]) : 0.f;
+  };
+  auto finish = [&](int u, float x, float y, float inv) {
+    const int i = first(u), j = second(u);
+    if (norm) {
+      x *= inv * __ldg(norm + i);
+      if (j < p.dim) y *= inv * __ldg(norm + j);
     }
-    inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.norm_eps);
+    if (u < half) {
+      const float2 c = __ldg(cs + u);
+      put(i, x * c.x - y * c.y);
+      put(j, y * c.x + x * c.y);
+    } else {
+      put(i, x);
+      if (j < p.dim) put(j, y);
+    }
+  };
+  auto scale = [&](float ss) { return norm ? 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.norm_eps) : 1.f; };
+  if (units <= 64) {
+    float x[2] = {0.f, 0.f}, y[2] = {0.f, 0.f};
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      if (lane + 32 * k < units) load(lane + 32 * k, x[k], y[k]);
+    const float inv = scale(fmaf(x[0], x[0], y[0] * y[0]) + fmaf(x[1], x[1], y[1] * y[1]));
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      if (lane + 32 * k < units) finish(lane + 32 * k, x[k], y[k], inv);
+    return;
   }
-  auto at = [&](int i) { return to_f(src[i]) * inv * (norm ? __ldg(norm + i) : 1.f); };
-  const float2 *cs = p.rope + (size_t)pos * p.rope_half;
-  for (int i = lane; i < p.rope_half; i += 32) {
-    const float u = at(i), v = at(i + p.rope_half);
-    const float2 c = __ldg(cs + i);
-    put(i, u * c.x - v * c.y);
-    put(i + p.rope_half, v * c.x + u * c.y);
+  float ss = 0.f;
+  for (int u = lane; u < units; u += 32) {
+    float x, y;
+    load(u, x, y);
+    ss += fmaf(x, x, y * y);
   }
-  for (int i = 2 * p.rope_half + lane; i < p.dim; i += 32) put(i, at(i));
+  const float inv = scale(ss);
+  for (int u = lane; u < units; u += 32) {
+    float x, y;
+    load(u, x, y);
+    finish(u, x, y, inv);
+  }
 }
 
 constexpr int PREP_WARPS = 4;

@@ -308,11 +308,12 @@ class GroupedLinear:
         """Bytes of one matrix."""
         return self.n_out * self.k_in * (2 if self.dtype == torch.bfloat16 else 4)
 
-    def __call__(self, x, out, rows, out_ld, tile, group_of, x_div=1, epilogue=EPI_STORE, linear_ws=None, gemm_ws=None, error_flag=None):
-        """out[:rows] = epilogue(x rows @ matrix^T).  tile: rows per entry of group_of; with tile 1 row r reads x row r // x_div."""
+    def __call__(self, x, out, rows, out_ld, tile, group_of, used=None, x_div=1, epilogue=EPI_STORE, linear_ws=None, gemm_ws=None, error_flag=None):
+        """out[:rows] = epilogue(x rows @ matrix^T).  tile: rows per entry of group_of; with tile 1 row r reads x row r // x_div.
+        used: rows of every tile that matter (the GEMM leaves the others out)."""
         L = _lib.lib()
         e = DenseExt()
-        e.limit, e.n_groups, e.group_rows, e.group_x_div, e.group_of = self.limit, self.groups, tile, x_div, _ptr(group_of)
+        e.limit, e.n_groups, e.group_rows, e.group_x_div, e.group_of, e.group_used = self.limit, self.groups, tile, x_div, _ptr(group_of), _ptr(used)
         if self.dtype == torch.float32:
             check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, 1.0, epilogue, _ptr(out), out_ld, ctypes.byref(e), _stream()),
                   "pt_gemm_f32")
@@ -426,6 +427,8 @@ def post_norm(rows, width, eps, dtype, x_in=None, x_out=None, y=None, y_ld=0, pa
         a.table, a.table_ld, a.vocab, a.ids, a.ids_ld = _ptr(table), table.shape[1], vocab or table.shape[0], _ptr(ids), ids_ld
         a.step_dev, a.pos_out, a.id_out = _ptr(step), _ptr(pos_out), _ptr(id_out)
     a.row_index, a.y, a.y_ld = _ptr(row_index), _ptr(y), y_ld
+    if pair_y is not None:
+        a.pair_dtype = dtype_code(pair_y.dtype)
     a.pair_y, a.pair_ld, a.top, a.pair_w, a.pair_row = _ptr(pair_y), pair_ld, top, _ptr(pair_w), _ptr(pair_row)
     a.norm_w, a.final_w, a.h, a.h_ld = _ptr(norm_w), _ptr(final_w), _ptr(h), h_ld
     check(_lib.lib().pt_post_norm(ctypes.byref(a), _stream()), "pt_post_norm")
@@ -435,14 +438,14 @@ def moe_max_tiles(n_tok, experts, top, tile):
     return int(_lib.lib().pt_moe_max_tiles(n_tok, experts, top, tile))
 
 
-def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, row_token=None, h=None, h_ld=0, gathered=None):
+def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, tile_rows=None, row_token=None, h=None, h_ld=0, gathered=None):
     """Experts and weights of every token, and with `tile` the rows of the grouped products (see pt_moe_route)."""
     a = MoeRouteArgs()
     a.n_tok, a.experts, a.top, a.logits, a.logits_ld = n_tok, experts, top, _ptr(logits), logits.shape[-1]
     a.expert, a.weight, a.tile = _ptr(expert), _ptr(weight), tile
     if tile:
         a.max_tiles = moe_max_tiles(n_tok, experts, top, tile)
-        a.pair_row, a.tile_expert, a.row_token = _ptr(pair_row), _ptr(tile_expert), _ptr(row_token)
+        a.pair_row, a.tile_expert, a.tile_rows, a.row_token = _ptr(pair_row), _ptr(tile_expert), _ptr(tile_rows), _ptr(row_token)
         if h is not None:
             a.h, a.h_bytes, a.gathered = _ptr(h), h_ld * h.element_size(), _ptr(gathered)
     check(_lib.lib().pt_moe_route(ctypes.byref(a), _stream()), "pt_moe_route")

@@ -205,10 +205,10 @@ class PadetarDecoder(SequenceDecoder):
             padded = [self._moe_tile(rows, s.m) * ops.moe_max_tiles(rows, s.m.experts, s.m.top, self._moe_tile(rows, s.m)) for s in moes]
             r.logits = torch.empty(rows * max(s.m.experts for s in moes), **f32)
             r.expert, r.pair_row, r.weight = torch.empty(rows * top, **i32), torch.empty(rows * top, **i32), torch.empty(rows * top, **f32)
-            r.tile_expert, r.row_token = torch.empty(max(padded), **i32), torch.empty(max(padded), **i32)
+            r.tile_expert, r.tile_rows, r.row_token = (torch.empty(max(padded), **i32) for _ in range(3))
             r.gathered = torch.empty(max(padded) * self.h_ld, dtype=dt, device=dev)
             r.act = torch.empty(max(p * s.ff for p, s in zip(padded, moes)), dtype=dt, device=dev)
-            r.pair_y = torch.empty((max(padded), c.width), **f32)
+            r.pair_y = torch.empty((max(padded), c.width), dtype=dt, device=dev)
             if r.lin_ws is not None:
                 pairs = min(rows, ops.DenseLinear.SKINNY_ROWS) * top
                 n = max(L.pt_linear_workspace_bytes(pairs, x.n_out, 4) for s in moes for x in (s.up, s.back))
@@ -240,9 +240,9 @@ class PadetarDecoder(SequenceDecoder):
             s.back(r.act, r.pair_y, n * m.top, W, 1, r.expert, **ws)
         else:
             rows = tile * ops.moe_max_tiles(n, m.experts, m.top, tile)
-            ops.moe_route(logits, n, m.experts, m.top, r.expert, r.weight, tile, r.pair_row, r.tile_expert, r.row_token, r.h, self.h_ld, r.gathered)
-            s.up(r.gathered, r.act, rows, s.ff, tile, r.tile_expert, epilogue=ops.EPI_GLU, **ws)
-            s.back(r.act, r.pair_y, rows, W, tile, r.tile_expert, **ws)
+            ops.moe_route(logits, n, m.experts, m.top, r.expert, r.weight, tile, r.pair_row, r.tile_expert, r.tile_rows, r.row_token, r.h, self.h_ld, r.gathered)
+            s.up(r.gathered, r.act, rows, s.ff, tile, r.tile_expert, r.tile_rows, epilogue=ops.EPI_GLU, **ws)
+            s.back(r.act, r.pair_y, rows, W, tile, r.tile_expert, r.tile_rows, **ws)
         if s.down:
             self._linear(s.down, r.a, r.y, n, W, r)
         return dict(y=r.y if s.down else None, y_ld=W, pair_y=r.pair_y, pair_ld=W, top=m.top, pair_w=r.weight, pair_row=None if tile == 1 else r.pair_row)

@@ -171,9 +171,9 @@ def test_router(cuda, tokens, experts, top, tile):
     h = bf16(r.standard_normal((tokens, 24)))
     if tile:
         tiles = ops.moe_max_tiles(tokens, experts, top, tile)
-        tile_expert, row_token = torch.full((tiles,), -5, dtype=torch.int32, device=cuda), torch.full((tiles * tile,), -5, dtype=torch.int32, device=cuda)
+        tile_expert, tile_rows, row_token = (torch.full((n,), -5, dtype=torch.int32, device=cuda) for n in (tiles, tiles, tiles * tile))
         gathered = torch.full((tiles * tile, 24), -7.0, dtype=BF16, device=cuda)
-        kw = dict(tile=tile, pair_row=pair_row, tile_expert=tile_expert, row_token=row_token, h=as_type(h, BF16, cuda), h_ld=24, gathered=gathered)
+        kw = dict(tile=tile, pair_row=pair_row, tile_expert=tile_expert, tile_rows=tile_rows, row_token=row_token, h=as_type(h, BF16, cuda), h_ld=24, gathered=gathered)
     ops.moe_route(as_type(z, F32, cuda), tokens, experts, top, expert, weight, **kw)
     assert np.array_equal(expert.cpu().numpy(), idx) and np.abs(weight.cpu().numpy() - wt).max() < 1e-6
     if not tile:
@@ -186,6 +186,8 @@ def test_router(cuda, tokens, experts, top, tile):
     assert (rt >= 0).sum() == tokens * top and ((rt == -1) | (rt >= 0)).all()
     used = -(-np.bincount(idx.ravel(), minlength=experts) // tile)
     assert np.array_equal(np.bincount(te[te >= 0], minlength=experts), used) and (te[used.sum():] == -1).all()
+    assert np.array_equal(tile_rows.cpu().numpy(), (rt.reshape(tiles, tile) >= 0).sum(1))
+    assert all((np.diff(np.sort(rows[idx == e])) == 1).sum() >= (idx == e).sum() - used[e] and (np.diff(rows[idx == e]) > 0).all() for e in range(experts))   # in order
     assert np.array_equal(g, np.where(rt[:, None] >= 0, h[np.maximum(rt, 0)], 0))
 
 
