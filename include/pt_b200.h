@@ -200,6 +200,7 @@ typedef struct pt_gemm_args {
   int out_dtype;          /* PT_W_BF16: PT_DT_BF16 or PT_DT_F32                      */
   float alpha;            /* PT_W_BF16: factor on the fp32 sum; 0 = 1                */
   const pt_dense_ext *ext; /* PT_W_BF16: further arguments, or NULL                  */
+  int pdl;                /* PT_W_BF16: 1: programmatic dependent launch (see pt_linear_args.pdl) */
 } pt_gemm_args;
 size_t pt_gemm_workspace_bytes(int m, int n_out, int max_ksplit);
 int pt_gemm(const pt_gemm_args *args, void *stream);

@@ -52,6 +52,7 @@ class GemmArgs(ctypes.Structure):
         ("w_tiled", c_int), ("x", c_void_p), ("w", c_void_p), ("scales", c_void_p), ("x_scale", c_float), ("w_scale", c_float),
         ("residual", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t),
         ("error_flag", c_void_p), ("bias", c_void_p), ("out_dtype", c_int), ("alpha", c_float), ("ext", ctypes.POINTER(DenseExt)),
+        ("pdl", c_int),
     ]
 
 

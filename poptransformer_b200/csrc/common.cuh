@@ -40,6 +40,11 @@ static inline cudaStream_t as_stream(void *s) { return reinterpret_cast<cudaStre
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 
 #ifdef __CUDACC__
+// Programmatic dependent launch: the next kernel of the stream may start (it waits for this one's results before it reads them), and
+// the wait for everything launched before.  Both do nothing when no such launch is involved.
+__device__ __forceinline__ void launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+__device__ __forceinline__ void wait_for_prerequisites() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+
 // ---- fp16 arithmetic with the reference's "one rounding per op" semantics -------------
 __device__ __forceinline__ __half h_mul(__half a, __half b) { return __hmul_rn(a, b); }
 __device__ __forceinline__ __half h_add(__half a, __half b) { return __hadd_rn(a, b); }

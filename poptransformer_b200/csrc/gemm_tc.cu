@@ -68,6 +68,7 @@ struct GemmParams {
   const int *group_of;    // BF16, grouped: the weight matrix of every tile of mb rows (negative: none)
   const int *group_used;  // ... and how many of its rows are in use (null: all)
   int n_tiles;            // tiles of 128 weight rows
+  int pdl;                // BF16: programmatic dependent launch: weights are fetched before the producer of x has finished
   size_t group_stride;    // bytes between weight matrices
 };
 
@@ -404,6 +405,7 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
   size_t w_base = 0;
   if constexpr (BF16) {
     if (p.group_of) {
+      if (p.pdl) wait_for_prerequisites();     // the router may be among the kernels before
       const int grp = p.group_of[blockIdx.z];
       if (grp < 0) return;                     // a tile without rows: nothing is initialised yet
       w_base = (size_t)grp * p.group_stride;
@@ -432,6 +434,8 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
   __syncthreads();
   fence_after();
   const uint32_t tmem = ctl.tmem_base;
+  // Not before: a CTA of the next GEMM that found the tensor memory free would keep it while it waits for this kernel to end.
+  if (BF16 && p.pdl) launch_dependents();
 
   if (warp == 0) {
     if (lane == 0) {
@@ -443,19 +447,32 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
       int s = 0, kx = kb0 * KX;
       uint32_t par = 1;   // parity of the `empty` phase that must have completed before slot s is refilled (none in the first round)
       bool first_round = true;
-      for (int it = 0; it < n_it; ++it) {
-        if (!first_round && !mbar_wait(empty0 + s * 8, par, &ctl.abort)) give_up(ctl, p.error_flag, 21);
-        if (ctl.abort) break;
-        const uint32_t st = smem_s + s * stage_bytes, fb = full0 + s * 8;
-        mbar_expect_tx(fb, tx);
+      auto load_w = [&](uint32_t st, uint32_t fb) {
         if (tiled) {
           bulk_g2s(st, wt, A_TILE, fb);
           if (NA == 2 && na == 2) bulk_g2s(st + A_TILE, wt + next_tile, A_TILE, fb);
         } else {
           tma_load_2d(st, &map_w, kx, n0, fb);
         }
-        tma_load_2d(st + NA * A_TILE, &map_x, kx, m0, fb);
         wt += A_TILE;
+      };
+      int early = 0;                         // stages whose weights are already on their way
+      if (BF16 && p.pdl) {
+        for (; early < min(p.stages, n_it); ++early) {
+          mbar_expect_tx(full0 + early * 8, tx);
+          load_w(smem_s + early * stage_bytes, full0 + early * 8);
+        }
+        wait_for_prerequisites();
+      }
+      for (int it = 0; it < n_it; ++it) {
+        if (!first_round && !mbar_wait(empty0 + s * 8, par, &ctl.abort)) give_up(ctl, p.error_flag, 21);
+        if (ctl.abort) break;
+        const uint32_t st = smem_s + s * stage_bytes, fb = full0 + s * 8;
+        if (it >= early) {
+          mbar_expect_tx(fb, tx);
+          load_w(st, fb);
+        }
+        tma_load_2d(st + NA * A_TILE, &map_x, kx, m0, fb);
         kx += KX;
         if (++s == p.stages) { s = 0; par ^= 1u; first_round = false; }
       }
@@ -836,7 +853,9 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   int ksplit = a->ksplit;
   if (ksplit <= 0) {
     ksplit = std::max(1, (p.mb <= 64 ? 2 : 1) * sm_count() / (n_tiles * m_tiles));   // two CTAs fit an SM up to 64 activation rows
-    ksplit = std::max(1, std::min(ksplit, p.n_kb / PT_TC_MIN_KB));
+    // (with several blocks of activation rows a slice's sums cost more than its share of a short k saves: 128 x 2048 at 512 .. 8192
+    // rows takes 19 - 21 us whole and 27 - 41 us in slices)
+    ksplit = std::max(1, std::min(ksplit, p.n_kb / (bf16 && m_tiles > 1 ? 32 : PT_TC_MIN_KB)));
     ksplit = std::min(ksplit, 8);                                           // what pt_gemm_workspace_bytes is usually asked for ...
     while (ksplit > 1 && pt_gemm_workspace_bytes(a->m, a->n_out, ksplit) > a->workspace_bytes) --ksplit;   // ... and never more than the caller's workspace holds
     if ((size_t)n_tiles * m_tiles > kGemmMaxCounters) ksplit = 1;
@@ -869,6 +888,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   const bool pair = PT_TC_PAIR && bf16 && p.ksplit == 1 && p.mb >= 128 && n_tiles >= 2 && (long long)ceil_div(n_tiles, 2) * m_tiles >= sm_count();
   const int na = pair ? 2 : 1;
   p.n_tiles = n_tiles;
+  p.pdl = bf16 && a->pdl ? 1 : 0;
   const uint32_t b_bytes = (uint32_t)p.mb * tc::BKB;
   const uint32_t stage_bytes = na * tc::A_TILE + ((b_bytes + 1023u) & ~1023u);
   // Up to 64 activation rows a stage is small, and what limits the kernel is the one thread per CTA that issues the MMAs (about
@@ -916,9 +936,20 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   dim3 grid(ceil_div(n_tiles, na), p.ksplit, m_tiles);
   if (int4)
     tc::gemm_int4_kernel<<<grid, tc::THREADS_I4, smem, as_stream(stream)>>>(map_x, p);
-  else if (bf16)
-    (pair ? tc::gemm_dense_kernel<true, 2> : tc::gemm_dense_kernel<true, 1>)<<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
-  else
+  else if (bf16) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(tc::THREADS_F8);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = as_stream(stream);
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = p.pdl ? 1 : 0;
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, pair ? tc::gemm_dense_kernel<true, 2> : tc::gemm_dense_kernel<true, 1>, map_w, map_x, p);
+    if (e != cudaSuccess) return pt::set_error(PT_ERR_CUDA, "pt_gemm: %s", cudaGetErrorString(e));
+  } else
     tc::gemm_dense_kernel<false, 1><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
   PT_LAUNCH_CHECK("pt_gemm");
   return PT_OK;

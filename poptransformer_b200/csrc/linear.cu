@@ -95,6 +95,7 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
   const __half *px = p.x;
   if constexpr (WFMT == PT_W_BF16) {
     if (p.group_of) {
+      if (p.pdl) wait_for_prerequisites();            // the router may be among the kernels before
       w_base = (size_t)p.group_of[z] * p.group_stride;
       px += (size_t)(z / p.group_x_div) * p.K;
     }
@@ -117,8 +118,8 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
   for (int s = 0; s < kStages - 1; ++s) issue(s);
   if (p.pdl) {
     // let the next kernel of the stream start its own weight prefetch, then wait for the producer of x
-    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-    asm volatile("griddepcontrol.wait;" ::: "memory");
+    launch_dependents();
+    wait_for_prerequisites();
   }
 
   // ---- prologue: stage (and optionally normalise / quantise) the activation slice
@@ -353,31 +354,32 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
     __threadfence();
     if (tid == 0) *counter = 0;  // ready for the next launch on this stream
     if (active) {
-      // Sum in split order (deterministic).  The loads of two splits (2 x 4 NB values) are issued together, so the reduction
-      // costs ksplit / 2 trips to L2 instead of one per (value, split).
+      // Sum in split order (deterministic).  The loads of SP splits (4 NB values each) are issued together, so the reduction costs
+      // ksplit / SP trips to L2 instead of one per (value, split).
+      constexpr int SP = NB == 1 ? 8 : 2;
 #pragma unroll
       for (int t = 0; t < NB; ++t)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[t][j] = 0.f;
       const float *base = p.partial + (size_t)rt * 16 + g;
-      for (int s0 = 0; s0 < p.ksplit; s0 += 2) {
-        float a0[NB][4], a1[NB][4];
-        const bool two = s0 + 1 < p.ksplit;
+      for (int s0 = 0; s0 < p.ksplit; s0 += SP) {
+        float a[SP][NB][4];
 #pragma unroll
-        for (int t = 0; t < NB; ++t)
+        for (int u = 0; u < SP; ++u)
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const int bcol = t * 8 + 2 * tig + (j & 1), row8 = 8 * (j >> 1);
-            const bool ok = bcol < p.B;
-            a0[t][j] = ok ? __ldcg(base + ((size_t)s0 * p.rows + z + bcol) * npad + row8) : 0.f;
-            a1[t][j] = (ok && two) ? __ldcg(base + ((size_t)(s0 + 1) * p.rows + z + bcol) * npad + row8) : 0.f;
-          }
+          for (int t = 0; t < NB; ++t)
 #pragma unroll
-        for (int t = 0; t < NB; ++t)
+            for (int j = 0; j < 4; ++j) {
+              const int bcol = t * 8 + 2 * tig + (j & 1), row8 = 8 * (j >> 1);
+              a[u][t][j] = (bcol < p.B && s0 + u < p.ksplit) ? __ldcg(base + ((size_t)(s0 + u) * p.rows + z + bcol) * npad + row8) : 0.f;
+            }
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            acc[t][j] += a0[t][j];
-            if (two) acc[t][j] += a1[t][j];
+        for (int u = 0; u < SP; ++u)
+          if (s0 + u < p.ksplit) {
+#pragma unroll
+            for (int t = 0; t < NB; ++t)
+#pragma unroll
+              for (int j = 0; j < 4; ++j) acc[t][j] += a[u][t][j];
           }
       }
     }

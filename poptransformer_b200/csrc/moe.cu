@@ -24,6 +24,7 @@ struct Params {
 
 // One warp per token; lane l holds the logits of experts l, l + 32, ...
 __global__ void choose_kernel(const Params p) {
+  launch_dependents();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= p.n_tok) return;
   const float *z = p.logits + (size_t)t * p.logits_ld;
@@ -65,16 +66,25 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
   __shared__ int warps[PLACE_THREADS / 32];
   __shared__ int first, total;
   const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, pairs = p.n_tok * p.top;
-  const int per = (pairs + PLACE_THREADS - 1) / PLACE_THREADS, i0 = min(pairs, tid * per), i1 = min(pairs, i0 + per);
+  const int per = ((pairs + PLACE_THREADS - 1) / PLACE_THREADS + 3) & ~3, i0 = min(pairs, tid * per), i1 = min(pairs, i0 + per);
   int *mine = hist + (warp % p.hist_copies) * p.experts;
   for (int i = tid; i < p.hist_copies * p.experts; i += PLACE_THREADS) hist[i] = 0;
   __syncthreads();
   int hits = 0;
-  for (int i = i0; i < i1; ++i) {
-    const int x = p.expert[i];
+  auto count_one = [&](int x) {
     atomicAdd(mine + x, 1);
     hits += x == e;
-  }
+  };
+  int i = i0;
+  if (((uintptr_t)p.expert & 15) == 0)
+    for (; i + 4 <= i1; i += 4) {
+      const int4 x = *reinterpret_cast<const int4 *>(p.expert + i);
+      count_one(x.x);
+      count_one(x.y);
+      count_one(x.z);
+      count_one(x.w);
+    }
+  for (; i < i1; ++i) count_one(p.expert[i]);
   __syncthreads();
   for (int i = tid; i < p.experts; i += PLACE_THREADS) {
     int n = 0;
@@ -133,6 +143,7 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
 
 // Rows of h (whole 16-byte units) to where row_token says.
 __global__ void gather_kernel(const uint4 *h, uint4 *out, int units, const int *row_token) {
+  launch_dependents();
   const int tok = row_token[blockIdx.x];
   uint4 *o = out + (size_t)blockIdx.x * units;
   const uint4 *src = h + (size_t)max(tok, 0) * units;

@@ -32,6 +32,7 @@ template <typename T, typename E, int VEC> __global__ void post_norm_kernel(cons
   extern __shared__ __align__(16) float row[];     // [width]: y, then the new x
   __shared__ float red[32], pw[kMaxTop];
   __shared__ int pr[kMaxTop];
+  launch_dependents();
   const int r = blockIdx.x, src = p.row_index ? p.row_index[r] : r, tid = threadIdx.x;
   float *xo = p.x_out ? p.x_out + (size_t)r * p.width : nullptr;
   T *hrow = p.h ? reinterpret_cast<T *>(p.h) + (size_t)r * p.h_ld : nullptr;

@@ -112,24 +112,26 @@ __device__ __forceinline__ void norm_rotate(const Params &p, const T *src, const
 }
 
 constexpr int PREP_WARPS = 4;
-template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const Params p) {   // warp: one token, one query or key head
-  const int t = blockIdx.y, h = blockIdx.x * PREP_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const Params p) {   // block: one token, warp: a head at a time
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
-  if (h >= p.n_head + (p.k ? p.n_kv : 0)) return;
   if (pos < 0 || pos >= p.max_len) {
     if (lane == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
   }
-  if (h < p.n_head) {
+#pragma unroll 2
+  for (int h = warp; h < p.n_head; h += PREP_WARPS) {
     T *q = reinterpret_cast<T *>(const_cast<void *>(p.q)) + (size_t)t * p.q_ld + (size_t)h * p.dim;
     norm_rotate<T>(p, q, p.q_norm, pos, [&](int i, float y) { q[i] = from_f<T>(y); });
-    return;
   }
-  const int g = h - p.n_head, phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page], at = pos % p.page;
-  const T *k = reinterpret_cast<const T *>(p.k) + (size_t)t * p.kv_ld + (size_t)g * p.dim, *v = reinterpret_cast<const T *>(p.v) + (size_t)t * p.kv_ld + (size_t)g * p.vdim;
-  T *kc = k_page<T>(p, phys, g) + (size_t)at * p.dim, *vc = v_page<T>(p, phys, g) + (size_t)at * p.vdim;
-  norm_rotate<T>(p, k, p.k_norm, pos, [&](int i, float y) { kc[i] = from_f<T>(y); });
-  for (int i = lane; i < p.vdim; i += 32) vc[i] = v[i];
+  if (!p.k) return;
+  const int phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page], at = pos % p.page;
+  for (int g = warp; g < p.n_kv; g += PREP_WARPS) {
+    const T *k = reinterpret_cast<const T *>(p.k) + (size_t)t * p.kv_ld + (size_t)g * p.dim, *v = reinterpret_cast<const T *>(p.v) + (size_t)t * p.kv_ld + (size_t)g * p.vdim;
+    T *kc = k_page<T>(p, phys, g) + (size_t)at * p.dim, *vc = v_page<T>(p, phys, g) + (size_t)at * p.vdim;
+    norm_rotate<T>(p, k, p.k_norm, pos, [&](int i, float y) { kc[i] = from_f<T>(y); });
+    for (int i = lane; i < p.vdim; i += 32) vc[i] = v[i];
+  }
 }
 
 template <typename T> __global__ void kv_append_kernel(const Params p) {
@@ -560,20 +562,31 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
   }
   __syncthreads();
   T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld;
-  for (int i = tid; i < nq * p.vdim; i += TC_THREADS) {
-    const int h = i / p.vdim, c = i - h * p.vdim;
+  const int v4 = p.vdim / 4;                                    // (vdim is a multiple of 8 here)
+  for (int i = tid; i < nq * v4; i += TC_THREADS) {
+    const int h = i / v4, c = (i - h * v4) * 4;
     const float *src = p.ws_o + ((head0 + h) * p.grid_pages) * p.vdim + c, *w = cw + h * p.grid_pages;
     constexpr int PB = 8;                                      // pages in flight
-    float acc = 0.f;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
     for (int i0 = 0; i0 < n_act; i0 += PB) {
-      float v[PB];
+      float4 v[PB];
 #pragma unroll
-      for (int j = 0; j < PB; ++j) v[j] = i0 + j < n_act ? __ldcg(src + (size_t)(i0 + j) * p.vdim) : 0.f;
+      for (int j = 0; j < PB; ++j) v[j] = i0 + j < n_act ? __ldcg(reinterpret_cast<const float4 *>(src + (size_t)(i0 + j) * p.vdim)) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
       for (int j = 0; j < PB; ++j)
-        if (i0 + j < n_act) acc = fmaf(v[j], w[i0 + j], acc);
+        if (i0 + j < n_act) {
+          const float x = w[i0 + j];
+          acc[0] = fmaf(v[j].x, x, acc[0]);
+          acc[1] = fmaf(v[j].y, x, acc[1]);
+          acc[2] = fmaf(v[j].z, x, acc[2]);
+          acc[3] = fmaf(v[j].w, x, acc[3]);
+        }
     }
-    out[(size_t)(h0 + h) * p.vdim + c] = from_f<T>(acc * ml[2 * h]);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[j] *= ml[2 * h];
+    T *o = out + (size_t)(h0 + h) * p.vdim + c;                // (rows of an even number of elements)
+    *reinterpret_cast<__nv_bfloat162 *>(o) = __floats2bfloat162_rn(acc[0], acc[1]);
+    *reinterpret_cast<__nv_bfloat162 *>(o + 2) = __floats2bfloat162_rn(acc[2], acc[3]);
   }
   if (h0 + nq == p.n_head)
     for (int i = p.n_head * p.vdim + tid; i < p.out_cols; i += TC_THREADS) out[i] = from_f<T>(0.f);
@@ -677,10 +690,8 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
     return wa::dispatch_tc(p, true, 1, st);
   }
   if (p.prep) {
-    PT_REQUIRE(b.n_tok <= 65535, "pt_window_attn: %d tokens", b.n_tok);
-    const dim3 grid(ceil_div(a->n_head + (p.k ? a->n_kv : 0), wa::PREP_WARPS), b.n_tok);
-    if (a->dtype == PT_DT_F32) wa::attn_prep_kernel<float><<<grid, wa::PREP_WARPS * 32, 0, st>>>(p);
-    else wa::attn_prep_kernel<__nv_bfloat16><<<grid, wa::PREP_WARPS * 32, 0, st>>>(p);
+    if (a->dtype == PT_DT_F32) wa::attn_prep_kernel<float><<<b.n_tok, wa::PREP_WARPS * 32, 0, st>>>(p);
+    else wa::attn_prep_kernel<__nv_bfloat16><<<b.n_tok, wa::PREP_WARPS * 32, 0, st>>>(p);
     PT_LAUNCH_CHECK("pt_window_attn");
   } else if (p.k) {
     if (a->dtype == PT_DT_F32) wa::kv_append_kernel<float><<<b.n_tok, 128, 0, st>>>(p);

@@ -168,7 +168,7 @@ def gemm_workspace(m, n_out_max, max_ksplit=8, device="cuda"):
 
 
 def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, workspace=None, ksplit=0, error_flag=None, bias=None,
-         out_ld=0, alpha=1.0, ext=None):
+         out_ld=0, alpha=1.0, ext=None, pdl=0):
     """y = x @ W^T on the tcgen05 GEMM.  INT4: x fp16 [m, k]; FP8: x E4M3 bytes [m, k] quantised with `x_scale`; BF16: x bfloat16,
     `out` bfloat16 or float32."""
     m = x.shape[0]
@@ -187,6 +187,7 @@ def gemm(x, gw, out=None, x_scale=1.0, epilogue=EPI_STORE, residual=None, worksp
     a.error_flag, a.bias = _ptr(error_flag), _ptr(bias)
     if ext is not None:
         a.ext = ctypes.pointer(ext)
+    a.pdl = pdl
     check(_lib.lib().pt_gemm(ctypes.byref(a), _stream()), "pt_gemm")
     return out
 
@@ -259,9 +260,9 @@ class DenseLinear:
         return e
 
     def __call__(self, x, out, rows, out_ld, epilogue=EPI_STORE, alpha=1.0, linear_ws=None, gemm_ws=None, error_flag=None, out2=None, out2_ld=0, mul=None,
-                 mul_ids=None):
+                 mul_ids=None, pdl=0):
         """out[:rows, :n_out] = epilogue(alpha * x[:rows] @ W^T + bias); x and out are flat or 2-D buffers of row strides `ld` and
-        `out_ld`."""
+        `out_ld`.  pdl: programmatic dependent launch behind the kernel before it in the stream (bfloat16)."""
         x = x.reshape(-1)[:rows * self.ld].view(rows, self.ld)
         L = _lib.lib()
         ext = self._ext(out2, out2_ld, mul, mul_ids)
@@ -269,10 +270,10 @@ class DenseLinear:
             check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, float(alpha), epilogue, _ptr(out), out_ld,
                                 ctypes.byref(ext) if ext else None, _stream()), "pt_gemm_f32")
         elif rows <= self.SKINNY_ROWS:
-            a = linear_args(x, self.skinny, out, epilogue=epilogue, workspace=linear_ws, out_ld=out_ld, error_flag=error_flag, alpha=alpha, ext=ext)
+            a = linear_args(x, self.skinny, out, epilogue=epilogue, workspace=linear_ws, out_ld=out_ld, error_flag=error_flag, alpha=alpha, ext=ext, pdl=pdl)
             check(L.pt_linear(ctypes.byref(a), _stream()), "pt_linear")
         else:
-            gemm(x, self.gemm, out=out, epilogue=epilogue, workspace=gemm_ws, error_flag=error_flag, out_ld=out_ld, alpha=alpha, ext=ext)
+            gemm(x, self.gemm, out=out, epilogue=epilogue, workspace=gemm_ws, error_flag=error_flag, out_ld=out_ld, alpha=alpha, ext=ext, pdl=pdl)
 
 
 class GroupedLinear:
@@ -308,7 +309,7 @@ class GroupedLinear:
         """Bytes of one matrix."""
         return self.n_out * self.k_in * (2 if self.dtype == torch.bfloat16 else 4)
 
-    def __call__(self, x, out, rows, out_ld, tile, group_of, used=None, x_div=1, epilogue=EPI_STORE, linear_ws=None, gemm_ws=None, error_flag=None):
+    def __call__(self, x, out, rows, out_ld, tile, group_of, used=None, x_div=1, epilogue=EPI_STORE, linear_ws=None, gemm_ws=None, error_flag=None, pdl=0):
         """out[:rows] = epilogue(x rows @ matrix^T).  tile: rows per entry of group_of; with tile 1 row r reads x row r // x_div.
         used: rows of every tile that matter (the GEMM leaves the others out)."""
         L = _lib.lib()
@@ -322,14 +323,14 @@ class GroupedLinear:
             a.wfmt, a.batch, a.n_out, a.k_in, a.epilogue, a.x, a.packed_w = W_BF16, rows, self.n_out, self.ld, epilogue, _ptr(x), _ptr(self.skinny)
             a.out, a.out_ld, a.out_dtype, a.alpha, a.error_flag = _ptr(out), out_ld, dtype_code(out.dtype), 1.0, _ptr(error_flag)
             a.workspace, a.workspace_bytes = _ptr(linear_ws), linear_ws.numel() if linear_ws is not None else 0
-            a.ext = ctypes.pointer(e)
+            a.ext, a.pdl = ctypes.pointer(e), pdl
             check(L.pt_linear(ctypes.byref(a), _stream()), "pt_linear")
         else:
             a = GemmArgs()
             a.wfmt, a.m, a.n_out, a.k_in, a.epilogue, a.w_tiled, a.x, a.w = W_BF16, rows, self.n_out, self.ld, epilogue, 1, _ptr(x), _ptr(self.tiled)
             a.out, a.out_ld, a.out_dtype, a.alpha, a.error_flag = _ptr(out), out_ld, dtype_code(out.dtype), 1.0, _ptr(error_flag)
             a.workspace, a.workspace_bytes = _ptr(gemm_ws), gemm_ws.numel() if gemm_ws is not None else 0
-            a.ext = ctypes.pointer(e)
+            a.ext, a.pdl = ctypes.pointer(e), pdl
             check(L.pt_gemm(ctypes.byref(a), _stream()), "pt_gemm")
 
 

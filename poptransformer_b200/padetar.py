@@ -197,6 +197,9 @@ class PadetarDecoder(SequenceDecoder):
         r.o = torch.empty(rows * max(s.mem.heads * s.mem.vdim for s in mixers), **f32)
         r.gates = torch.empty(rows * max(2 * s.mem.heads for s in mixers), **f32)
         self._linear_workspaces(r, rows, self._linears())
+        r.beside = SimpleNamespace(lin_ws=None, gemm_ws=None)                                  # of the shared expert, which runs beside the others
+        if any(s.down for s in moes):
+            self._linear_workspaces(r.beside, rows, [s.down for s in moes if s.down])
         L = ops._lib.lib()
         n = max(L.pt_mlstm_workspace_bytes(rows + 1, min(self.batch, rows), s.mem.heads, s.mem.dim, s.mem.vdim) for s in mixers)
         r.mem_ws = torch.zeros(n, dtype=torch.uint8, device=dev)
@@ -219,21 +222,26 @@ class PadetarDecoder(SequenceDecoder):
     # ---- the layers -----------------------------------------------------------------------------
     def _mixer(self, s, r, view, longest):
         n, lay, a = view.n_tok, s.lay, s.lay.left
-        self._linear(s.proj, r.h, r.a, n, s.ld, r, out2=r.gates, out2_ld=2 * s.mem.heads)
+        self._linear(s.proj, r.h, r.a, n, s.ld, r, out2=r.gates, out2_ld=2 * s.mem.heads, pdl=1)
+        with self._beside():          # the two mixers read and write columns of their own
+            ops.mlstm(view, r.a, s.ld, s.cols, r.gates, 2 * s.mem.heads, r.b[s.right_col:], s.out.ld, s.mem, self.states[s.layer], self.norms[s.layer], r.o, r.mem_ws,
+                      out_scale=lay.right_scale, out_cols=s.out.ld - s.right_col, plain=self.plain)
         ops.window_attn(view, r.a, s.ld, self.caches[s.layer], r.b, s.out.ld, a.heads, a.scale, max_tokens_per_seq=longest, workspace=self.attn_ws,
                         error_flag=self.error_flag, plain=self.plain, values_are_keys=True, q_norm=s.q_norm, k_norm=s.k_norm, eps=self.cfg.eps, rope=s.rope,
                         rope_dims=a.rot_dims, out_scale=lay.left_scale, out_cols=s.right_col)
-        ops.mlstm(view, r.a, s.ld, s.cols, r.gates, 2 * s.mem.heads, r.b[s.right_col:], s.out.ld, s.mem, self.states[s.layer], self.norms[s.layer], r.o, r.mem_ws,
-                  out_scale=lay.right_scale, out_cols=s.out.ld - s.right_col, plain=self.plain)
+        self._join()
         self._linear(s.out, r.b, r.y, n, self.cfg.width, r)
         return dict(y=r.y, y_ld=self.cfg.width)
 
     def _experts(self, s, r, view, longest):
         n, m, W = view.n_tok, s.m, self.cfg.width
-        self._linear(s.proj, r.h, r.a, n, s.sff, r, epilogue=ops.EPI_GLU if s.down else ops.EPI_STORE, out2=r.logits, out2_ld=m.experts)
+        self._linear(s.proj, r.h, r.a, n, s.sff, r, epilogue=ops.EPI_GLU if s.down else ops.EPI_STORE, out2=r.logits, out2_ld=m.experts, pdl=1)
+        if s.down:
+            with self._beside():
+                self._linear(s.down, r.a, r.y, n, W, r.beside)
         tile = self._moe_tile(n, m)
         logits = r.logits[:n * m.experts].view(n, m.experts)
-        ws = dict(linear_ws=r.lin_ws, gemm_ws=r.gemm_ws, error_flag=self.error_flag)
+        ws = dict(linear_ws=r.lin_ws, gemm_ws=r.gemm_ws, error_flag=self.error_flag, pdl=1)
         if tile == 1:
             ops.moe_route(logits, n, m.experts, m.top, r.expert, r.weight)
             s.up(r.h, r.act, n * m.top, s.ff, 1, r.expert, x_div=m.top, epilogue=ops.EPI_GLU, **ws)
@@ -244,13 +252,13 @@ class PadetarDecoder(SequenceDecoder):
             s.up(r.gathered, r.act, rows, s.ff, tile, r.tile_expert, r.tile_rows, epilogue=ops.EPI_GLU, **ws)
             s.back(r.act, r.pair_y, rows, W, tile, r.tile_expert, r.tile_rows, **ws)
         if s.down:
-            self._linear(s.down, r.a, r.y, n, W, r)
+            self._join()
         return dict(y=r.y if s.down else None, y_ld=W, pair_y=r.pair_y, pair_ld=W, top=m.top, pair_w=r.weight, pair_row=None if tile == 1 else r.pair_row)
 
     def _side(self, s, r, view, longest):
         n, W = view.n_tok, self.cfg.width
-        self._linear(s.proj, r.h, r.a, n, s.ld, r, epilogue=ops.EPI_GELU_MUL, mul=(self.side_table, self.side_table.shape[1], s.layer * self.side_ld), mul_ids=r.tok)
-        self._linear(s.out, r.a, r.y, n, W, r)
+        self._linear(s.proj, r.h, r.a, n, s.ld, r, epilogue=ops.EPI_GELU_MUL, mul=(self.side_table, self.side_table.shape[1], s.layer * self.side_ld), mul_ids=r.tok, pdl=1)
+        self._linear(s.out, r.a, r.y, n, W, r, pdl=1)
         return dict(y=r.y, y_ld=W)
 
     def _layers(self, r, view, longest, ids, ids_ld=1, step=None, pos_out=None, layer_sums=None):
@@ -275,4 +283,4 @@ class PadetarDecoder(SequenceDecoder):
             ops.post_norm(n_tok, c.width, c.eps, self.dtype, x_in=r.x, x_out=layer_sums[-1], **r.pending)
         if n:
             ops.post_norm(n, c.width, c.eps, self.dtype, x_in=r.x, h=r.h, h_ld=self.h_ld, final_w=self.final_norm, row_index=row_index, **r.pending)
-            self._linear(self.head, r.h, out, n, c.vocab, r)
+            self._linear(self.head, r.h, out, n, c.vocab, r, pdl=1)

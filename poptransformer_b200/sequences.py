@@ -5,6 +5,7 @@ A model's class brings its weights (`_load`), the caches and states of its layer
 The decode loop of the other models (`run`, `step`, `prefill`, `capture`): one id container, all rows at the same position, greedy.
 And sequences with positions of their own (`open`, `extend`, `close`): each call takes the next tokens of any number of sequences
 and returns logits."""
+import contextlib
 import copy
 from types import SimpleNamespace
 
@@ -46,6 +47,7 @@ class Weights:
 
 
 class SequenceDecoder(DecodeLoop):
+    _side_stream = None
     PROMPT_TOKENS = 8192     # most packed prompt tokens of one pass (longer prompts go in portions)
 
     def __init__(self, cfg, state_dict, batch, device="cuda", dtype="bfloat16", page_size=64, pad_id=None, eos_id=-1, early_stop=False, n_pages=None,
@@ -134,6 +136,18 @@ class SequenceDecoder(DecodeLoop):
 
     def _linear(self, lin, x, out, rows, out_ld, r, **kw):
         lin(x, out, rows, out_ld, linear_ws=r.lin_ws, gemm_ws=r.gemm_ws, error_flag=self.error_flag, **kw)
+
+    @contextlib.contextmanager
+    def _beside(self):
+        """What is launched inside runs beside what follows on the current stream, until `_join`.  (In a captured graph: a branch.)"""
+        if self._side_stream is None:
+            self._side_stream = torch.cuda.Stream(self.device)
+        self._side_stream.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(self._side_stream):
+            yield
+
+    def _join(self):
+        torch.cuda.current_stream().wait_stream(self._side_stream)
 
     # ---- the decode loop ------------------------------------------------------------------------
     def _need_loop_rows(self):
