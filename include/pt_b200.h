@@ -553,6 +553,7 @@ typedef struct pt_moe_route_args {
   float *weight;                  /* [n_tok, top]                                    */
   int tile, max_tiles;
   int32_t *pair_row, *tile_expert, *tile_rows, *row_token;
+  int32_t *counts;                /* scratch [experts], optional: faster with many pairs */
   const void *h;
   int h_bytes;
   void *gathered;

@@ -104,7 +104,7 @@ class PostNormArgs(ctypes.Structure):
 
 class MoeRouteArgs(ctypes.Structure):
     _fields_ = [("n_tok", c_int), ("experts", c_int), ("top", c_int), ("logits", c_void_p), ("logits_ld", c_int), ("expert", c_void_p), ("weight", c_void_p),
-                ("tile", c_int), ("max_tiles", c_int), ("pair_row", c_void_p), ("tile_expert", c_void_p), ("tile_rows", c_void_p), ("row_token", c_void_p), ("h", c_void_p), ("h_bytes", c_int),
+                ("tile", c_int), ("max_tiles", c_int), ("pair_row", c_void_p), ("tile_expert", c_void_p), ("tile_rows", c_void_p), ("row_token", c_void_p), ("counts", c_void_p), ("h", c_void_p), ("h_bytes", c_int),
                 ("gathered", c_void_p)]
 
 

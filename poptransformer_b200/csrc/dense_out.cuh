@@ -53,6 +53,10 @@ static inline const char *dense_ext_error(int epilogue, int n_out, const pt_dens
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * x * x, x, x)));
 }
+// (rounded to bf16 by the caller)  tanh(z) = 2 sigmoid(2 z) - 1
+__device__ __forceinline__ float gelu_tanh_fast(float x) {
+  return __fdividef(x, 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * x * x, x, x)));
+}
 template <bool FAST> __device__ __forceinline__ float glu_f(float gate, float up, float limit) {
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   if (FAST) return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);   // (rounded to bf16 by the caller; for g very negative the quotient is 0)

@@ -243,7 +243,7 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 // increments instead of index arithmetic (the general form above costs as much as the products of a 2048-deep tile).
 // bf16 output: neighbouring lanes (n, n + 1) trade values of two columns, so every store writes 4 bytes per lane.
 // Gated features: lanes n and n + 8 trade likewise, and each computes one column of the pair's feature.
-enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_GLU = 2 };
+enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_GLU = 2, OUT_GELU_MUL = 3 };
 template <int KIND, bool RELU2>
 __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, int ld, const uint32_t (&v)[32], int n, int m, int lane) {
   const float b = d.bias ? __ldg(d.bias + n + (KIND == OUT_F32 && out == d.out2 ? d.split_n : 0)) : 0.f;
@@ -259,12 +259,22 @@ __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, in
       *o = fin(v[j]);
       o += ld;
     }
-  } else if (KIND == OUT_BF16) {
+  } else if (KIND == OUT_BF16 || KIND == OUT_GELU_MUL) {
+    float w[KIND == OUT_GELU_MUL ? 32 : 1];     // the factors of this lane's column, requested together
+    if (KIND == OUT_GELU_MUL) {
+      const __nv_bfloat16 *mul = reinterpret_cast<const __nv_bfloat16 *>(d.mul) + n;
+#pragma unroll
+      for (int j = 0; j < 32; ++j) w[j] = __bfloat162float(mul[(size_t)__ldg(d.mul_ids + m + j) * d.mul_ld]);
+    }
     const int odd = lane & 1;
     __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(out) + (size_t)(m + odd) * ld + (n - odd);
 #pragma unroll
     for (int j = 0; j < 32; j += 2) {
-      const float a = fin(v[j]), c = fin(v[j + 1]);
+      float a = fin(v[j]), c = fin(v[j + 1]);
+      if (KIND == OUT_GELU_MUL) {
+        a = gelu_tanh_fast(a) * w[KIND == OUT_GELU_MUL ? j : 0];
+        c = gelu_tanh_fast(c) * w[KIND == OUT_GELU_MUL ? j + 1 : 0];
+      }
       const float t = __shfl_xor_sync(0xffffffffu, odd ? a : c, 1);     // even lane: column j of n + 1; odd lane: column j + 1 of n - 1
       *reinterpret_cast<__nv_bfloat162 *>(o) = odd ? __floats2bfloat162_rn(t, c) : __floats2bfloat162_rn(a, t);
       o += 2 * (size_t)ld;
@@ -287,7 +297,7 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
   // (warp-uniform) where this warp's 32 outputs go
   const bool second = nq >= d.split_n, glu = d.epilogue == PT_EPI_GLU && !second, f32 = second || d.out_dt == PT_DT_F32;
   // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16
-  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && (second || d.epilogue != PT_EPI_GELU_MUL) && !(glu && f32) &&
+  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) &&
                     (f32 || glu || (d.out_ld % 2 == 0 && ((uintptr_t)d.out & 3) == 0));
   const int rows = min(p.mb, m_end - m0), whole = fast ? rows & ~31 : 0;
   for (int c0 = 0; c0 < whole; c0 += 32) {
@@ -301,7 +311,8 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
       if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_F32, true>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
       else epilogue_rows32<OUT_F32, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     } else {
-      if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_BF16, true>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      if (d.epilogue == PT_EPI_GELU_MUL) epilogue_rows32<OUT_GELU_MUL, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_BF16, true>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
       else epilogue_rows32<OUT_BF16, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     }
   }

@@ -20,6 +20,7 @@ struct Params {
   const float *logits;
   int *expert, *pair_row, *tile_expert, *tile_rows, *row_token;   // [n_tok][top] x 2, [max_tiles] x 2, [max_tiles * tile]
   float *weight;                                      // [n_tok][top]
+  const int *counts;                                  // [experts], or null: counted while placing
 };
 
 // One warp per token; lane l holds the logits of experts l, l + 32, ...
@@ -59,8 +60,28 @@ __global__ void choose_kernel(const Params p) {
   if (lane + 32 < p.top) p.weight[(size_t)t * p.top + lane + 32] = w1 / sum;
 }
 
-// Block e places the pairs of expert e: every block counts all experts' pairs (for the tiles in front of its own), then its own pairs
-// get their rows.  Thread i looks at a run of consecutive pairs, so the order within an expert is the order of the pairs.
+// Pairs per expert, for many pairs: block e counts those of expert e.
+__global__ void __launch_bounds__(PLACE_THREADS) count_kernel(const int *expert, int pairs, int *counts) {
+  __shared__ int warps[PLACE_THREADS / 32];
+  const int e = blockIdx.x, tid = threadIdx.x, n4 = pairs / 4;
+  int hits = 0;
+  for (int i = tid; i < n4; i += PLACE_THREADS) {
+    const int4 x = reinterpret_cast<const int4 *>(expert)[i];
+    hits += (x.x == e) + (x.y == e) + (x.z == e) + (x.w == e);
+  }
+  for (int i = 4 * n4 + tid; i < pairs; i += PLACE_THREADS) hits += expert[i] == e;
+  for (int o = 16; o > 0; o >>= 1) hits += __shfl_xor_sync(0xffffffffu, hits, o);
+  if ((tid & 31) == 0) warps[tid >> 5] = hits;
+  __syncthreads();
+  if (tid == 0) {
+    int n = 0;
+    for (int w = 0; w < PLACE_THREADS / 32; ++w) n += warps[w];
+    counts[e] = n;
+  }
+}
+
+// Block e places the pairs of expert e: the pairs of all experts are counted (or come from count_kernel) for the tiles in front of its
+// own, then its own pairs get their rows.  Thread i looks at a run of consecutive pairs, so the order within an expert is the order of the pairs.
 __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
   extern __shared__ int hist[];                   // [copies][experts]: warps count into copies of their own while they fit
   __shared__ int warps[PLACE_THREADS / 32];
@@ -72,7 +93,7 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
   __syncthreads();
   int hits = 0;
   auto count_one = [&](int x) {
-    atomicAdd(mine + x, 1);
+    if (!p.counts) atomicAdd(mine + x, 1);
     hits += x == e;
   };
   int i = i0;
@@ -88,7 +109,9 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
   __syncthreads();
   for (int i = tid; i < p.experts; i += PLACE_THREADS) {
     int n = 0;
-    for (int c = 0; c < p.hist_copies; ++c) n += hist[c * p.experts + i];
+    if (p.counts) n = p.counts[i];
+    else
+      for (int c = 0; c < p.hist_copies; ++c) n += hist[c * p.experts + i];
     hist[i] = n;                                  // (the same thread read copy 0 of this expert just before)
   }
   int scan = hits;
@@ -179,7 +202,12 @@ extern "C" int pt_moe_route(const pt_moe_route_args *a, void *stream) {
   PT_REQUIRE(a->tile > 0 && a->pair_row && a->tile_expert && a->tile_rows && a->row_token && a->max_tiles >= pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile),
              "pt_moe_route: tiles of %d rows need pair_row, row_token and %d entries of tile_expert", a->tile, pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile));
   p.tile = a->tile; p.max_tiles = a->max_tiles; p.pair_row = a->pair_row; p.tile_expert = a->tile_expert; p.tile_rows = a->tile_rows; p.row_token = a->row_token;
-  p.hist_copies = std::max(1, std::min(32, 8192 / p.experts));
+  if (p.n_tok * p.top > 4096 && a->counts && aligned_to(p.expert, 16)) {
+    moe::count_kernel<<<p.experts, moe::PLACE_THREADS, 0, st>>>(p.expert, p.n_tok * p.top, a->counts);
+    PT_LAUNCH_CHECK("pt_moe_route");
+    p.counts = a->counts;
+  }
+  p.hist_copies = p.counts ? 1 : std::max(1, std::min(32, 8192 / p.experts));
   moe::place_kernel<<<p.experts, moe::PLACE_THREADS, (size_t)p.hist_copies * p.experts * sizeof(int), st>>>(p);
   PT_LAUNCH_CHECK("pt_moe_route");
   if (a->h) {

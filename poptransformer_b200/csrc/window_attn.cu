@@ -34,7 +34,7 @@ struct Params {
   const float2 *rope;        // [positions][rope_half]
   float norm_eps, out_scale;
   int rope_half, out_cols;
-  bool prep;                 // queries and keys are normalised or rotated
+  bool prep, pair_rows;      // queries and keys are normalised or rotated; their rows can be taken as pairs of neighbours
   // decode
   int grid_pages, qsplit;
   float *ws_o;      // [n_seq, n_head, grid_pages, vdim]
@@ -58,57 +58,72 @@ __device__ __forceinline__ int window_page(const Params &p, int pos) { return p.
 __device__ __forceinline__ int kept_pages(const Params &p, int pos) { return (min(p.keep_first, pos + 1) + p.page - 1) / p.page; }
 
 // ------------------------------------------------------------------------------------------ norm, rotation, append
-// One warp: a head's row of a query or key.  put(i, value) may write over src (a lane reads what it writes).  A unit is the pair
-// (u, u + half) that turns together, or two neighbours behind the rotated dimensions.  Up to 128 dimensions the row stays in registers.
+// One warp, a head's row of a query or key at a time.  put(i, value) may write over src (a lane reads what it writes).
 template <typename T, typename Put>
-__device__ __forceinline__ void norm_rotate(const Params &p, const T *src, const float *norm, int pos, Put put) {
-  const int lane = threadIdx.x & 31, half = p.rope_half, units = (p.dim + 1) / 2;
+__device__ __forceinline__ void norm_rotate_any(const Params &p, const T *src, const float *norm, int pos, Put put) {
+  const int lane = threadIdx.x & 31, half = p.rope_half;
+  float inv = 1.f;
+  if (norm) {
+    float ss = 0.f;
+    for (int i = lane; i < p.dim; i += 32) {
+      const float x = to_f(src[i]);
+      ss = fmaf(x, x, ss);
+    }
+    inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.norm_eps);
+  }
+  auto at = [&](int i) { return to_f(src[i]) * inv * (norm ? __ldg(norm + i) : 1.f); };
   const float2 *cs = p.rope + (size_t)pos * half;
-  auto first = [&](int u) { return u < half ? u : 2 * u; };            // 2 half + 2 (u - half)
-  auto second = [&](int u) { return u < half ? u + half : 2 * u + 1; };
-  auto load = [&](int u, float &x, float &y) {
-    x = to_f(src[first(u)]);
-    y = second(u) < p.dim ? to_f(src[second(u)]) : 0.f;
-  };
-  auto finish = [&](int u, float x, float y, float inv) {
-    const int i = first(u), j = second(u);
-    if (norm) {
-      x *= inv * __ldg(norm + i);
-      if (j < p.dim) y *= inv * __ldg(norm + j);
+  for (int i = lane; i < half; i += 32) {
+    const float u = at(i), v = at(i + half);
+    const float2 c = __ldg(cs + i);
+    put(i, u * c.x - v * c.y);
+    put(i + half, v * c.x + u * c.y);
+  }
+  for (int i = 2 * half + lane; i < p.dim; i += 32) put(i, at(i));
+}
+// The same in registers for rows of up to 128 dimensions (p.pair_rows): a lane holds the neighbours i, i + 1 and their partners j,
+// j + 1.  Behind the rotated dimensions the partners are the next two, and the angle is zero.  Angles and weights serve all heads.
+__device__ __forceinline__ float2 load_pair(const float *p) { return *reinterpret_cast<const float2 *>(p); }
+__device__ __forceinline__ float2 load_pair(const __nv_bfloat16 *p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(p)); }
+struct HeadLane {
+  int i, j;
+  bool on;
+  float2 c0, c1, wi, wj;
+  __device__ __forceinline__ HeadLane(const Params &p, const float *norm, int pos) {
+    const int u = 2 * (threadIdx.x & 31), half = p.rope_half;
+    on = p.pair_rows && u < p.dim / 2;       // (nothing is loaded for rows that are taken the other way)
+    i = u < half ? u : 2 * u;
+    j = u < half ? u + half : 2 * u + 2;
+    c0 = c1 = make_float2(1.f, 0.f);
+    wi = wj = make_float2(1.f, 1.f);
+    if (on && u < half) {
+      const float4 c = __ldg(reinterpret_cast<const float4 *>(p.rope + (size_t)pos * half + u));
+      c0 = make_float2(c.x, c.y);
+      c1 = make_float2(c.z, c.w);
     }
-    if (u < half) {
-      const float2 c = __ldg(cs + u);
-      put(i, x * c.x - y * c.y);
-      put(j, y * c.x + x * c.y);
-    } else {
-      put(i, x);
-      if (j < p.dim) put(j, y);
+    if (on && norm) {
+      wi = __ldg(reinterpret_cast<const float2 *>(norm + i));
+      wj = __ldg(reinterpret_cast<const float2 *>(norm + j));
     }
-  };
-  auto scale = [&](float ss) { return norm ? 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.norm_eps) : 1.f; };
-  if (units <= 64) {
-    float x[2] = {0.f, 0.f}, y[2] = {0.f, 0.f};
-#pragma unroll
-    for (int k = 0; k < 2; ++k)
-      if (lane + 32 * k < units) load(lane + 32 * k, x[k], y[k]);
-    const float inv = scale(fmaf(x[0], x[0], y[0] * y[0]) + fmaf(x[1], x[1], y[1] * y[1]));
-#pragma unroll
-    for (int k = 0; k < 2; ++k)
-      if (lane + 32 * k < units) finish(lane + 32 * k, x[k], y[k], inv);
-    return;
   }
-  float ss = 0.f;
-  for (int u = lane; u < units; u += 32) {
-    float x, y;
-    load(u, x, y);
-    ss += fmaf(x, x, y * y);
+  template <typename T> __device__ __forceinline__ void run(const Params &p, const T *src, bool norm, T *dst) const {
+    float2 x = make_float2(0.f, 0.f), y = x;
+    if (on) {
+      x = load_pair(src + i);
+      y = load_pair(src + j);
+    }
+    const float inv = norm ? 1.0f / sqrtf(warp_sum(fmaf(x.x, x.x, x.y * x.y) + fmaf(y.x, y.x, y.y * y.y)) / (float)p.dim + p.norm_eps) : 1.f;
+    if (!on) return;
+    x.x *= inv * wi.x; x.y *= inv * wi.y;
+    y.x *= inv * wj.x; y.y *= inv * wj.y;
+    const float a[2] = {x.x * c0.x - y.x * c0.y, x.y * c1.x - y.y * c1.y}, b[2] = {y.x * c0.x + x.x * c0.y, y.y * c1.x + x.y * c1.y};
+    store_vec<2>(dst + i, a);
+    store_vec<2>(dst + j, b);
   }
-  const float inv = scale(ss);
-  for (int u = lane; u < units; u += 32) {
-    float x, y;
-    load(u, x, y);
-    finish(u, x, y, inv);
-  }
+};
+template <typename T> __device__ __forceinline__ void norm_rotate(const Params &p, const HeadLane &hl, const T *src, const float *norm, int pos, T *dst) {
+  if (p.pair_rows) hl.run<T>(p, src, norm != nullptr, dst);
+  else norm_rotate_any<T>(p, src, norm, pos, [&](int i, float y) { dst[i] = from_f<T>(y); });
 }
 
 constexpr int PREP_WARPS = 4;
@@ -119,17 +134,21 @@ template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_pr
     if (lane == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
   }
-#pragma unroll 2
-  for (int h = warp; h < p.n_head; h += PREP_WARPS) {
-    T *q = reinterpret_cast<T *>(const_cast<void *>(p.q)) + (size_t)t * p.q_ld + (size_t)h * p.dim;
-    norm_rotate<T>(p, q, p.q_norm, pos, [&](int i, float y) { q[i] = from_f<T>(y); });
+  {
+    const HeadLane hl(p, p.q_norm, pos);
+#pragma unroll 4
+    for (int h = warp; h < p.n_head; h += PREP_WARPS) {
+      T *q = reinterpret_cast<T *>(const_cast<void *>(p.q)) + (size_t)t * p.q_ld + (size_t)h * p.dim;
+      norm_rotate<T>(p, hl, q, p.q_norm, pos, q);
+    }
   }
   if (!p.k) return;
+  const HeadLane hl(p, p.k_norm, pos);
   const int phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page], at = pos % p.page;
   for (int g = warp; g < p.n_kv; g += PREP_WARPS) {
     const T *k = reinterpret_cast<const T *>(p.k) + (size_t)t * p.kv_ld + (size_t)g * p.dim, *v = reinterpret_cast<const T *>(p.v) + (size_t)t * p.kv_ld + (size_t)g * p.vdim;
     T *kc = k_page<T>(p, phys, g) + (size_t)at * p.dim, *vc = v_page<T>(p, phys, g) + (size_t)at * p.vdim;
-    norm_rotate<T>(p, k, p.k_norm, pos, [&](int i, float y) { kc[i] = from_f<T>(y); });
+    norm_rotate<T>(p, hl, k, p.k_norm, pos, kc);
     for (int i = lane; i < p.vdim; i += 32) vc[i] = v[i];
   }
 }
@@ -221,12 +240,12 @@ constexpr int TC_THREADS = 128, TILE = 64;   // TILE = the page size the tensor-
 // Block: 64 new tokens of one sequence, one head; warp w owns queries 16 w .. 16 w + 15, their q fragments stay in registers.  Key
 // tiles (one page each) are double-buffered in shared memory; tiles without a visible key are skipped, tiles that every query of
 // the warp sees completely take no mask.  DK / DV: dim / vdim rounded up to 32, 64 or 128 (the padding holds zeros).
-template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_prompt_kernel(const Params p) {
+template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS, 3) attn_prompt_kernel(const Params p) {
   constexpr int KLD = DK + 8, VLD = DV + 8;
   extern __shared__ __align__(16) __nv_bfloat16 smb[];
   __nv_bfloat16 *Ks = smb, *Vs = smb + 2 * TILE * KLD;      // [2][TILE][KLD], [2][TILE][VLD]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
-  const int s = blockIdx.z, head = blockIdx.y, t0 = blockIdx.x * TILE, kvh = head / p.qpk;
+  const int s = blockIdx.z, head = blockIdx.y, t0 = (gridDim.x - 1 - blockIdx.x) * TILE, kvh = head / p.qpk;   // (the tiles with most keys first)
   const int row0 = p.cu[s], len = p.cu[s + 1] - row0, start = p.start[s];
   if (t0 >= len) return;
   if (start < 0 || start + len > p.max_len) {
@@ -291,15 +310,19 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_pro
     if (wlo <= whi && k0 <= whi && (p.window == 0 || k0 + TILE - 1 > wlo - p.window || k0 < p.keep_first)) {
       const __nv_bfloat16 *K = Ks + stage * TILE * KLD;
       float sc[TILE / 8][4];
+      // (matrices of a load: keys 0-7 with channels 0-7 and 8-15, then keys 8-15 likewise)
+      const uint32_t k_lane = smem_addr(K + ((lane & 7) + (lane >> 4) * 8) * KLD + ((lane >> 3) & 1) * 8);
 #pragma unroll
-      for (int j = 0; j < TILE / 8; ++j) {
-        sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
-        const __nv_bfloat16 *kr = K + (j * 8 + g) * KLD + 2 * tig;
+      for (int j = 0; j < TILE / 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
 #pragma unroll
-        for (int kk = 0; kk < DK / 16; ++kk)
-          mma16816_bf16(sc[j], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], *reinterpret_cast<const uint32_t *>(kr + kk * 16),
-                        *reinterpret_cast<const uint32_t *>(kr + kk * 16 + 8));
-      }
+      for (int kk = 0; kk < DK / 16; ++kk)      // (channels outside: the products of one step are independent)
+#pragma unroll
+        for (int j = 0; j < TILE / 8; j += 2) {
+          uint32_t b0, b1, b2, b3;
+          ldsm4(k_lane + (uint32_t)(j * 8 * KLD + kk * 16) * 2u, b0, b1, b2, b3);
+          mma16816_bf16(sc[j], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b0, b1);
+          mma16816_bf16(sc[j + 1], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b2, b3);
+        }
       const bool whole = k0 + TILE - 1 <= wlo && (p.window == 0 || whi - k0 < p.window || k0 + TILE <= p.keep_first);
       float m_new[2] = {m_run[0], m_run[1]};
 #pragma unroll
@@ -444,10 +467,11 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
   asm volatile("cp.async.commit_group;" ::: "memory");
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * p.dim;
   if (p.prep) {
+    const HeadLane hq(p, p.q_norm, pos), hk(p, p.k_norm, pos);
     for (int h = warp; h < NQ + 1; h += TC_THREADS / 32) {
       T *dst = h < NQ ? qs + h * QLD : kn;
       const bool have = h < NQ ? h < nq : owner;
-      if (have) norm_rotate<T>(p, h < NQ ? q + (size_t)h * p.dim : knew, h < NQ ? p.q_norm : p.k_norm, pos, [&](int i, float y) { dst[i] = from_f<T>(y); });
+      if (have) norm_rotate<T>(p, h < NQ ? hq : hk, h < NQ ? q + (size_t)h * p.dim : knew, h < NQ ? p.q_norm : p.k_norm, pos, dst);
       for (int i = (have ? p.dim : 0) + lane; i < DK; i += 32) dst[i] = from_f<T>(0.f);
     }
   } else for (int i = tid; i < NQ * (DK / 8); i += TC_THREADS) {
@@ -662,6 +686,12 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
   p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.0f;
   p.out_cols = a->out_cols > 0 ? a->out_cols : a->out_ld;
   p.prep = a->q_norm || a->k_norm || a->rope_dims;
+  {
+    const int pair = a->dtype == PT_DT_F32 ? 8 : 4;
+    auto al = [](const void *x, int bytes) { return ((uintptr_t)x & (bytes - 1)) == 0; };
+    p.pair_rows = a->dim % 4 == 0 && a->dim <= 128 && a->rope_dims % 4 == 0 && a->q_ld % 2 == 0 && a->n_kv * a->page_size * (a->dim + a->vdim) % 2 == 0 && al(a->q, pair) && al(a->pool, pair) && al(a->rope, 16) && al(a->q_norm, 8) &&
+                  al(a->k_norm, 8) && (!a->k || (a->kv_ld % 2 == 0 && al(a->k, pair)));
+  }
   PT_REQUIRE(a->rope_dims >= 0 && a->rope_dims % 2 == 0 && a->rope_dims <= a->dim && (!a->rope_dims || a->rope), "pt_window_attn: %d rotated dimensions of %d",
              a->rope_dims, a->dim);
   PT_REQUIRE(p.out_cols >= a->n_head * a->vdim && p.out_cols <= a->out_ld, "pt_window_attn: out_cols=%d", a->out_cols);

@@ -210,12 +210,13 @@ def glu_rows(gate, up, features):
 
 
 class DenseLinear:
-    """W [n_out, k] of a model whose activations are bfloat16 or float32.  bfloat16: the skinny-matmul kernel up to SKINNY_ROWS rows
+    """W [n_out, k] of a model whose activations are bfloat16 or float32.  bfloat16: the skinny-matmul kernel up to `skinny_rows` rows
     and the tcgen05 GEMM beyond (one tiling of the weights each), k padded to `K_PAD` with zero columns, so inputs have `ld` columns.
     float32: true 32-bit products, no padding.  Outputs may have more columns than n_out (`out_ld`)."""
     K_PAD = 64
     # Measured on B200 over 2048 x 4096 .. 32000 x 4096: at 8 rows the GEMM is level (2048-wide) to 20 % faster, at 32 rows 10 % to 3x.
-    SKINNY_ROWS = 7
+    # Up to a million weights (128 x 2048, 2048 x 128, 1024 x 1024) the skinny kernel takes 0.6 - 0.75 of the GEMM's time at 8 and 16 rows.
+    SKINNY_ROWS, SMALL_ROWS, SMALL_SIZE = 7, 16, 1 << 20
 
     def __init__(self, w, dtype, pad_rows=0, keep=False, bias=None, split=None, limit=0.0):
         """pad_rows: zero rows are appended up to this many outputs (an output that is the padded input of the next linear).
@@ -233,6 +234,7 @@ class DenseLinear:
             self.bias = torch.zeros(self.n_out, dtype=torch.float32, device=w.device)
             self.bias[:len(bias)] = bias
         w = w.to(dtype).contiguous()
+        self.skinny_rows = self.SMALL_ROWS if self.n_out * self.ld <= self.SMALL_SIZE else self.SKINNY_ROWS
         if dtype == torch.bfloat16:
             self.skinny, self.gemm = PackedLinear(W_BF16, w), GemmWeight(W_BF16, w)
             self.w = w if keep else None
@@ -269,7 +271,7 @@ class DenseLinear:
         if self.dtype == torch.float32:
             check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, float(alpha), epilogue, _ptr(out), out_ld,
                                 ctypes.byref(ext) if ext else None, _stream()), "pt_gemm_f32")
-        elif rows <= self.SKINNY_ROWS:
+        elif rows <= self.skinny_rows:
             a = linear_args(x, self.skinny, out, epilogue=epilogue, workspace=linear_ws, out_ld=out_ld, error_flag=error_flag, alpha=alpha, ext=ext, pdl=pdl)
             check(L.pt_linear(ctypes.byref(a), _stream()), "pt_linear")
         else:
@@ -439,7 +441,7 @@ def moe_max_tiles(n_tok, experts, top, tile):
     return int(_lib.lib().pt_moe_max_tiles(n_tok, experts, top, tile))
 
 
-def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, tile_rows=None, row_token=None, h=None, h_ld=0, gathered=None):
+def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, tile_rows=None, row_token=None, counts=None, h=None, h_ld=0, gathered=None):
     """Experts and weights of every token, and with `tile` the rows of the grouped products (see pt_moe_route)."""
     a = MoeRouteArgs()
     a.n_tok, a.experts, a.top, a.logits, a.logits_ld = n_tok, experts, top, _ptr(logits), logits.shape[-1]
@@ -447,6 +449,7 @@ def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None
     if tile:
         a.max_tiles = moe_max_tiles(n_tok, experts, top, tile)
         a.pair_row, a.tile_expert, a.tile_rows, a.row_token = _ptr(pair_row), _ptr(tile_expert), _ptr(tile_rows), _ptr(row_token)
+        a.counts = _ptr(counts)
         if h is not None:
             a.h, a.h_bytes, a.gathered = _ptr(h), h_ld * h.element_size(), _ptr(gathered)
     check(_lib.lib().pt_moe_route(ctypes.byref(a), _stream()), "pt_moe_route")

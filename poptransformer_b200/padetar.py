@@ -209,6 +209,7 @@ class PadetarDecoder(SequenceDecoder):
             r.logits = torch.empty(rows * max(s.m.experts for s in moes), **f32)
             r.expert, r.pair_row, r.weight = torch.empty(rows * top, **i32), torch.empty(rows * top, **i32), torch.empty(rows * top, **f32)
             r.tile_expert, r.tile_rows, r.row_token = (torch.empty(max(padded), **i32) for _ in range(3))
+            r.counts = torch.empty(max(s.m.experts for s in moes), **i32)
             r.gathered = torch.empty(max(padded) * self.h_ld, dtype=dt, device=dev)
             r.act = torch.empty(max(p * s.ff for p, s in zip(padded, moes)), dtype=dt, device=dev)
             r.pair_y = torch.empty((max(padded), c.width), dtype=dt, device=dev)
@@ -248,7 +249,7 @@ class PadetarDecoder(SequenceDecoder):
             s.back(r.act, r.pair_y, n * m.top, W, 1, r.expert, **ws)
         else:
             rows = tile * ops.moe_max_tiles(n, m.experts, m.top, tile)
-            ops.moe_route(logits, n, m.experts, m.top, r.expert, r.weight, tile, r.pair_row, r.tile_expert, r.tile_rows, r.row_token, r.h, self.h_ld, r.gathered)
+            ops.moe_route(logits, n, m.experts, m.top, r.expert, r.weight, tile, r.pair_row, r.tile_expert, r.tile_rows, r.row_token, r.counts, r.h, self.h_ld, r.gathered)
             s.up(r.gathered, r.act, rows, s.ff, tile, r.tile_expert, r.tile_rows, epilogue=ops.EPI_GLU, **ws)
             s.back(r.act, r.pair_y, rows, W, tile, r.tile_expert, r.tile_rows, **ws)
         if s.down:

@@ -87,8 +87,7 @@ class SequenceDecoder(DecodeLoop):
         r.lin_ws = r.gemm_ws = None
         if self.dtype == torch.bfloat16:
             L = ops._lib.lib()
-            skinny = min(rows, ops.DenseLinear.SKINNY_ROWS)
-            n = max(L.pt_linear_workspace_bytes(skinny, x.n_out, max(16, x.ld // 256)) for x in linears)     # at least 256 k per slice
+            n = max(L.pt_linear_workspace_bytes(min(rows, x.skinny_rows), x.n_out, max(16, x.ld // 256)) for x in linears)     # at least 256 k per slice
             r.lin_ws = torch.zeros(n, dtype=torch.uint8, device=self.device)
             if rows > ops.DenseLinear.SKINNY_ROWS:   # k-slices only while there are fewer tiles than SMs: 40 MB hold every such product's
                 n = min(max(L.pt_gemm_workspace_bytes(rows, x.n_out, 8) for x in linears), (40 << 20) + 65536)

@@ -3,6 +3,8 @@ import ctypes
 import os
 import re
 
+import pytest
+
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
@@ -31,16 +33,17 @@ def test_library_exports_every_declared_symbol():
     assert handle.pt_version() >= 100
 
 
-def test_parts_link_on_their_own(tmp_path, monkeypatch):
+@pytest.mark.parametrize("arch,own,other", [("Sabisun", ("pt_hyper", "pt_ssm"), "pt_mlstm"), ("Padetar", ("pt_post_norm", "pt_moe_route", "pt_mlstm"), "pt_ssm")])
+def test_parts_link_on_their_own(tmp_path, monkeypatch, arch, own, other):
     """A library with one architecture's sources resolves all of its symbols and has the entry points that the decoder calls."""
     from poptransformer_b200 import build
     monkeypatch.setattr(build, "LIB", str(tmp_path / "libpt_b200.so"))
-    path = build.build_for("Sabisun")
-    assert path == build.part_path("Sabisun") and not os.path.exists(build.LIB)
+    path = build.build_for(arch)
+    assert path == build.part_path(arch) and not os.path.exists(build.LIB)
     handle = ctypes.CDLL(path, mode=os.RTLD_NOW)
-    for s in ("pt_linear", "pt_gemm", "pt_gemm_f32", "pt_hyper", "pt_window_attn", "pt_ssm", "pt_topk", "pt_step_containers"):
+    for s in ("pt_linear", "pt_gemm", "pt_gemm_f32", "pt_window_attn", "pt_topk", "pt_step_containers", *own):
         assert hasattr(handle, s)
-    assert not hasattr(handle, "pt_llama_decode_step")
+    assert not hasattr(handle, "pt_llama_decode_step") and not hasattr(handle, other)
 
 
 def test_argument_checks_run_without_a_gpu():

@@ -157,7 +157,7 @@ def test_glu_rows_and_clamps(cuda):
 
 # ------------------------------------------------------------------------------------------ router
 @pytest.mark.parametrize("tokens,experts,top,tile", [(1, 5, 5, 0), (3, 33, 4, 0), (7, 64, 8, 0), (9, 6, 2, 16), (40, 33, 4, 16), (300, 12, 3, 64), (1500, 7, 1, 128),
-                                                     (50, 100, 40, 64), (20, 3, 3, 32)])
+                                                     (50, 100, 40, 64), (20, 3, 3, 32), (1901, 11, 5, 64)])
 def test_router(cuda, tokens, experts, top, tile):
     from poptransformer_b200 import ops
     r = np.random.default_rng(4)
@@ -173,7 +173,8 @@ def test_router(cuda, tokens, experts, top, tile):
         tiles = ops.moe_max_tiles(tokens, experts, top, tile)
         tile_expert, tile_rows, row_token = (torch.full((n,), -5, dtype=torch.int32, device=cuda) for n in (tiles, tiles, tiles * tile))
         gathered = torch.full((tiles * tile, 24), -7.0, dtype=BF16, device=cuda)
-        kw = dict(tile=tile, pair_row=pair_row, tile_expert=tile_expert, tile_rows=tile_rows, row_token=row_token, h=as_type(h, BF16, cuda), h_ld=24, gathered=gathered)
+        kw = dict(tile=tile, pair_row=pair_row, tile_expert=tile_expert, tile_rows=tile_rows, row_token=row_token,
+                  counts=torch.full((experts,), -5, dtype=torch.int32, device=cuda) if tokens % 2 else None, h=as_type(h, BF16, cuda), h_ld=24, gathered=gathered)
     ops.moe_route(as_type(z, F32, cuda), tokens, experts, top, expert, weight, **kw)
     assert np.array_equal(expert.cpu().numpy(), idx) and np.abs(weight.cpu().numpy() - wt).max() < 1e-6
     if not tile:

@@ -67,7 +67,7 @@ def test_true_fp32_product(cuda, m, n, k):
         assert (out[:, n:] == -7).all()
 
 
-@pytest.mark.parametrize("rows", [1, 5, 7, 8, 16, 31, 70, 257, 600])
+@pytest.mark.parametrize("rows", [1, 5, 7, 8, 16, 17, 31, 70, 257, 600])
 @pytest.mark.parametrize("n,k", [(24, 40), (200, 64), (513, 328), (128, 2048)])
 def test_bf16_linear(cuda, rows, n, k):
     """Skinny-matmul kernel for few rows, tcgen05 GEMM beyond; k that is no multiple of a block, n that is no multiple of a tile."""
