@@ -544,7 +544,8 @@ int pt_post_norm(const pt_post_norm_args *args, void *stream);
 /* Mixture of experts (csrc/moe.cu): the `top` experts of every token by router logit, softmax weights over the chosen ones, and the
  * layout of the grouped products.  tile = 0: only expert and weight are written.  tile > 0: the pairs (token, choice) are sorted by
  * expert into tiles of `tile` rows: pair_row [n_tok, top], tile_expert [max_tiles] (-1: unused), tile_rows [max_tiles] (rows in use), row_token
- * [max_tiles * tile] (-1: padding), and with h the rows of h_bytes each are copied to gathered [max_tiles * tile]. */
+ * [max_tiles * tile] (-1: padding), and with h the rows of h_bytes each are copied to gathered [max_tiles * tile] (padding
+ * rows are left as they are). */
 typedef struct pt_moe_route_args {
   int n_tok, experts, top;        /* at most 64 of 1024                              */
   const float *logits;

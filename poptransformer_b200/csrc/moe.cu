@@ -4,7 +4,8 @@
 //   place    pair i = token i / top with its choice i % top gets a row of its own among its expert's rows.  The rows of an expert are
 //            padded to whole tiles; tile_expert names the expert of every tile (-1: unused) and tile_rows its rows in use, so a grouped
 //            product can look its weights up per tile.  Pairs keep their order within an expert.
-//   gather   the tokens' activations are copied to their pairs' rows (zeros in the padding).
+//   gather   the tokens' activations are copied to their pairs' rows.  (Rows of the padding keep what they held: rows of a product do
+//            not touch one another, and nothing reads theirs.)
 // With few tokens every pair is a tile of one row and nothing is placed or copied.
 #include <limits.h>
 
@@ -168,13 +169,13 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
 __global__ void gather_kernel(const uint4 *h, uint4 *out, int units, const int *row_token) {
   launch_dependents();
   const int tok = row_token[blockIdx.x];
-  uint4 *o = out + (size_t)blockIdx.x * units;
-  const uint4 *src = h + (size_t)max(tok, 0) * units;
-  for (int i = threadIdx.x; i < units; i += blockDim.x) o[i] = tok >= 0 ? src[i] : make_uint4(0, 0, 0, 0);
+  if (tok < 0) return;
+  for (int i = threadIdx.x; i < units; i += blockDim.x) out[(size_t)blockIdx.x * units + i] = h[(size_t)tok * units + i];
 }
 __global__ void gather4_kernel(const uint32_t *h, uint32_t *out, int units, const int *row_token) {
   const int tok = row_token[blockIdx.x];
-  for (int i = threadIdx.x; i < units; i += blockDim.x) out[(size_t)blockIdx.x * units + i] = tok >= 0 ? h[(size_t)tok * units + i] : 0u;
+  if (tok < 0) return;
+  for (int i = threadIdx.x; i < units; i += blockDim.x) out[(size_t)blockIdx.x * units + i] = h[(size_t)tok * units + i];
 }
 
 }  // namespace moe

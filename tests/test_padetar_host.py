@@ -47,7 +47,7 @@ def test_registry():
     assert registry.architecture({"architecture": "Padetar"}) == "Padetar" and registry.dtypes({"architecture": "Padetar"}) == ("bfloat16", "float32")
 
 
-@pytest.mark.parametrize("dims,base,scaling", [(48, 5e5, (4.0, 1.0, 4.0, 128)), (64, 1e4, (8.0, 2.0, 32.0, 512)), (16, 100.0, None), (2, 1e4, (3.0, 1.0, 2.0, 4))])
+@pytest.mark.parametrize("dims,base,scaling", [(56, 3e5, (5.0, 1.5, 6.0, 200)), (64, 1e4, (8.0, 2.0, 32.0, 512)), (16, 100.0, None), (2, 1e4, (3.0, 1.0, 2.0, 4))])
 def test_frequencies(dims, base, scaling):
     from poptransformer_b200.padetar import rope_frequencies
     sc = dict(zip(("factor", "low", "high", "original"), scaling)) if scaling else None
