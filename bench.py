@@ -790,7 +790,7 @@ def run_experts(args):
                 # every linear once, and the experts that `batch` independent choices are expected to hit
                 hit = E * (1.0 - (1.0 - top / E) ** batch)
                 moe = [s for s in dec.subs if s.kind == "moe"]
-                weights = sum(x.nbytes for x in dec._linears()) + sum(hit * (s.up.nbytes + s.back.nbytes) for s in moe)
+                weights = sum(x.nbytes for x in dec._linears()) + sum(hit * (s.experts.up.nbytes + s.experts.back.nbytes) for s in moe)
                 state = n_layer * (2 * 4 * dims["mem_heads"] * dims["mem_dim"] * dims["mem_vdim"] + 2 * 2 * dims["kv_heads"] * dims["dim"] * ctx)
             else:
                 weights, state = dec.weight_bytes(), sabisun_state_bytes(cfg)
@@ -801,7 +801,7 @@ def run_experts(args):
         dec = registry.build_decoder(cfg, sd, 4, max_len, "bfloat16", pad_id=-1)
         size = lambda x: x.n_out * x.k_in
         if name == "padetar":
-            flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(top * (size(s.up) + size(s.back)) for s in dec.subs if s.kind == "moe"))
+            flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(top * (size(s.experts.up) + size(s.experts.back)) for s in dec.subs if s.kind == "moe"))
         else:
             flops = 2 * prompt * sum(size(s.proj) + size(s.out) for s in dec.subs)
         for n_seq in (1, 4):

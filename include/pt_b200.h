@@ -67,14 +67,21 @@ uint64_t pt_launch_count(void);
 #define PT_EPI_BIAS_GELU 4    /* y = gelu(fp16(fp16(acc) + bias))    layers/mlp.py:34-41   */
 #define PT_EPI_BIAS_RESIDUAL 5/* y = fp16(res + fp16(fp16(acc) + bias))                  */
 #define PT_EPI_RELU2 6        /* y = max(acc, 0)^2, squared in fp32 (PT_W_BF16 and pt_gemm_f32) */
-#define PT_EPI_GLU 7          /* clamped gated unit of row pairs (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
+#define PT_EPI_GLU 7          /* gated unit of row pairs (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
 #define PT_EPI_GELU_MUL 8     /* gelu_tanh(acc) * mul[mul_ids[row]]  (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
+#define PT_EPI_SOFTCAP 9      /* limit * tanh(acc / limit)  (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
+#define PT_GLU_CLAMPED 0      /* kinds of gated units */
+#define PT_GLU_SILU 1
+#define PT_GLU_GELU 2
 
 /* Further arguments of the linears of bf16 and fp32 models: pt_linear and pt_gemm with PT_W_BF16, and pt_gemm_f32 (csrc/dense_out.cuh).
  *   bias       fp32 [n_out], added to alpha * sum before the epilogue; outputs from split_n on (a multiple of 32) skip the epilogue
  *              and go to out2 in fp32
- *   PT_EPI_GLU weight rows alternate: eight gate features, the same eight up features; g = min(gate, limit), u = clamp(up, -limit,
- *              limit), out = g sigmoid(1.702 g) (u + 1), half as many columns as rows
+ *   row_scale  fp32 [rows] or NULL: sums of activation row m are multiplied with row_scale[m] before the bias is added
+ *   PT_EPI_GLU weight rows alternate: eight gate features, the same eight up features; half as many columns as rows.  By `glu`:
+ *              PT_GLU_CLAMPED  g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(1.702 g) (u + 1)
+ *              PT_GLU_SILU     gate sigmoid(gate) up            PT_GLU_GELU  gelu_tanh(gate) up
+ *   PT_EPI_SOFTCAP   out = limit tanh(y / limit)
  *   PT_EPI_GELU_MUL  out[m, n] = gelu_tanh(y) * mul[mul_ids[m] * mul_ld + n], mul of the output's type
  *   groups     n_groups > 0: the weights are n_groups matrices one after the other (each as packed for the entry point), and tile t of
  *              group_rows activation rows is multiplied with matrix group_of[t] (device; negative: the tile is skipped).  pt_gemm:
@@ -90,6 +97,8 @@ typedef struct pt_dense_ext {
   int n_groups, group_rows, group_x_div;
   const int32_t *group_of;
   const int32_t *group_used; /* pt_gemm, optional: rows in use of every tile (the rest is neither multiplied nor written) */
+  int glu;
+  const float *row_scale;
 } pt_dense_ext;
 
 /* ---- Int4ToHalf -------------------------------------------------------------------
@@ -511,11 +520,13 @@ typedef struct pt_hyper_args {
 } pt_hyper_args;
 int pt_hyper(const pt_hyper_args *args, void *stream);
 
-/* Residual stream with norms on the sublayers' outputs (csrc/post_norm.cu), x fp32 [rows, width]:
- *   table != NULL : x_out[r] = h[r] = table[ids[r * ids_ld + *step_dev]] (step_dev NULL: column 0; pos_out[r] <- the step, id_out[r] <- the id)
- *   otherwise     : s = row_index ? row_index[r] : r;  Y = y[s] + sum_k pair_w[s, k] pair_y[pair_row[s, k]]  (pair_row NULL: s * top + k);
- *                   x = x_in[s] + rms_norm(Y) * norm_w;  x_out[r] = x;  h[r] = x, or rms_norm(x) * final_w
- * x_out, h, y (with top > 0) and final_w may be NULL; x_out may be x_in without row_index.  Columns width .. h_ld - 1 of h are zeroed. */
+/* Residual step with norms on the sublayers' outputs, on the next one's input, or both (csrc/post_norm.cu), x fp32 [rows, width]:
+ *   Y = table != NULL ? table[ids[r * ids_ld + *step_dev]] (step_dev NULL: column 0; pos_out[r] <- the step, id_out[r] <- the id)
+ *       : y[s] + sum_k pair_w[s, k] pair_y[pair_row[s, k]],  s = row_index ? row_index[r] : r  (pair_w NULL: ones; pair_row NULL: s * top + k)
+ *   x = x_in[s] + (norm_w ? rms_norm(Y) * norm_w : Y)  (x_in NULL, or a table: without the first term)
+ *   x_out[r] = copy[r] = x;  h[r] = final_w ? rms_norm(x) * final_w : x       (copy and h in the activation type)
+ * x_out, copy, h, y and the weights may be NULL; x_out may be x_in without row_index.  Columns from width up to h_cols of h and
+ * copy_cols of copy are zeroed (0: h_ld, nothing). */
 typedef struct pt_post_norm_args {
   int rows, width, dtype;
   float eps;
@@ -537,15 +548,19 @@ typedef struct pt_post_norm_args {
   const int32_t *pair_row;
   const float *norm_w, *final_w;
   void *h;
-  int h_ld;
+  int h_ld, h_cols;
+  void *copy;
+  int copy_ld, copy_cols;
 } pt_post_norm_args;
 int pt_post_norm(const pt_post_norm_args *args, void *stream);
 
-/* Mixture of experts (csrc/moe.cu): the `top` experts of every token by router logit, softmax weights over the chosen ones, and the
- * layout of the grouped products.  tile = 0: only expert and weight are written.  tile > 0: the pairs (token, choice) are sorted by
+/* Mixture of experts (csrc/moe.cu): the `top` experts of every token by router logit, their weights (by `score`: the softmax over the
+ * chosen logits, or the sigmoid of each), and the layout of the grouped products.  tile = 0: only expert and weight are written.  tile > 0: the pairs (token, choice) are sorted by
  * expert into tiles of `tile` rows: pair_row [n_tok, top], tile_expert [max_tiles] (-1: unused), tile_rows [max_tiles] (rows in use), row_token
  * [max_tiles * tile] (-1: padding), and with h the rows of h_bytes each are copied to gathered [max_tiles * tile] (padding
- * rows are left as they are). */
+ * rows are left as they are), and row_weight [max_tiles * tile] (optional) gets the weight of every placed row. */
+#define PT_MOE_SOFTMAX 0
+#define PT_MOE_SIGMOID 1
 typedef struct pt_moe_route_args {
   int n_tok, experts, top;        /* at most 64 of 1024                              */
   const float *logits;
@@ -558,6 +573,8 @@ typedef struct pt_moe_route_args {
   const void *h;
   int h_bytes;
   void *gathered;
+  int score;                      /* PT_MOE_*                                        */
+  float *row_weight;
 } pt_moe_route_args;
 int pt_moe_max_tiles(int n_tok, int experts, int top, int tile);
 int pt_moe_route(const pt_moe_route_args *args, void *stream);
@@ -565,6 +582,14 @@ int pt_moe_route(const pt_moe_route_args *args, void *stream);
 /* Masked attention over a paged cache (csrc/window_attn.cu): sliding window with kept first tokens, softmax sink, grouped heads,
  * separate key and value widths.  pool[page] = K [n_kv][page_size][dim] then V [n_kv][page_size][vdim], page_table
  * [slots][max_pages].  k / v (NULL for a layer that reads another layer's cache) are appended before anything is read. */
+/* Keys and values of the whole context as bf16 rows instead of pages: row cu[s] + j is position j of sequence s.  Head h's key is
+ * [the first shared_dim dimensions from `shared` (the same for all heads) | columns h (dim - shared_dim) .. of k], its value columns
+ * h vdim .. of v.  k and v have row stride ld. */
+typedef struct pt_context_rows {
+  const void *k, *v, *shared;
+  int ld, shared_ld, shared_dim;
+  const int32_t *cu;      /* [n_seq]                                                 */
+} pt_context_rows;
 typedef struct pt_window_attn_args {
   pt_batch_view batch;
   int dtype;              /* PT_DT_F32 or PT_DT_BF16: q, k, v, pool and out          */
@@ -596,9 +621,77 @@ typedef struct pt_window_attn_args {
   const float *rope;      /* fp32 [positions, rope_dims / 2, 2]                      */
   float out_scale;        /* factor on the output, 0 = 1                             */
   int out_cols;           /* columns of out that are written or zeroed, 0 = out_ld   */
+  float softcap;          /* c: a score s becomes c tanh(s / c); 0 = none            */
+  const void *gate;       /* NULL, or rows of the activation type: the output is multiplied with sigmoid(gate) */
+  int gate_ld, gate_per_head; /* n_head * vdim columns, or one per head              */
+  int values_in_keys;     /* the pool holds keys only; values are dimensions value_col .. value_col + vdim - 1 of them */
+  int value_col;
+  const pt_context_rows *context; /* prompts: where keys and values are instead of the pool, or NULL */
 } pt_window_attn_args;
 size_t pt_window_attn_workspace_bytes(int n_seq, int n_head, int vdim, int page_size, int max_len, int window, int keep_first);
 int pt_window_attn(const pt_window_attn_args *args, void *stream);
+
+/* Attention over a latent (csrc/latent.cu).  A cached row is [rot_dim rotated key dimensions, shared by all heads | rank latent
+ * dimensions]; pool [pages][page_size][rot_dim + rank], one page numbering with the other caches.
+ * pt_latent_prep: cq <- rms_norm(q) * q_norm (columns q_rank .. cq_ld - 1 zeroed); the row of every token <- [rotation of kv[rank ..] |
+ * rms_norm(kv[.. rank]) * kv_norm].  rope: (cos, sin) of rope[position][i] for the pair (i, i + rot_dim / 2). */
+typedef struct pt_latent_prep_args {
+  pt_batch_view batch;
+  int dtype;              /* PT_DT_F32 or PT_DT_BF16: q, kv, cq, pool                */
+  int q_rank, rank, rot_dim;
+  float eps;
+  const void *q, *kv;     /* [n_tok] rows of q_rank and of rank + rot_dim            */
+  int ld;                 /* row stride of both                                      */
+  const float *q_norm, *kv_norm;
+  const float *rope;      /* fp32 [positions, rot_dim / 2, 2]                        */
+  void *cq;
+  int cq_ld;
+  void *pool;
+  const int32_t *page_table;
+  int page_size, max_pages, max_len;
+  int32_t *error_flag;    /* optional, set to 12 when a position has no page         */
+} pt_latent_prep_args;
+int pt_latent_prep(const pt_latent_prep_args *args, void *stream);
+
+/* The cached rows of every sequence's context (bf16), sequence after sequence: shared [n_ctx, rot_dim], latent [n_ctx, latent_ld] (padding
+ * columns zeroed).  Row ctx_cu[s] + j is position j of sequence s. */
+typedef struct pt_latent_context_args {
+  pt_batch_view batch;    /* n_seq and slot are used                                 */
+  const int32_t *ctx_cu;  /* [n_seq + 1]                                             */
+  int n_ctx, rot_dim, rank, page_size, max_pages;
+  const void *pool;
+  const int32_t *page_table;
+  void *shared, *latent;
+  int latent_ld;
+} pt_latent_context_args;
+int pt_latent_context(const pt_latent_context_args *args, void *stream);
+
+/* Causal attention of the packed tokens over the cached latents, without forming keys and values: out[h] = sigmoid(gate[h]) W_v[h] sum_j
+ * w_j latent_j, w = softmax(scale ([rotated q | W_k[h] q] . row_j)).  A query head is [rot_dim, to be rotated | dim]. */
+typedef struct pt_latent_attn_args {
+  pt_batch_view batch;
+  int dtype;              /* PT_DT_F32 or PT_DT_BF16: q, weights, gate, pool, out    */
+  int n_head, dim, rot_dim, vdim, rank;
+  float scale;
+  const void *q;
+  int q_ld;
+  const float *rope;
+  const void *w_k;        /* [n_head, rank, dim]                                     */
+  const void *w_v;        /* [n_head, vdim, rank]                                    */
+  const void *gate;       /* NULL, or one column per head                            */
+  int gate_ld;
+  const void *pool;
+  const int32_t *page_table;
+  int page_size, max_pages, max_len;
+  void *out;
+  int out_ld, out_cols;   /* columns n_head * vdim .. out_cols - 1 are zeroed (0 = out_ld) */
+  int plain;              /* 1: the kernels for any sizes, whatever the shape        */
+  void *workspace;        /* pt_latent_attn_workspace_bytes                          */
+  size_t workspace_bytes;
+  int32_t *error_flag;
+} pt_latent_attn_args;
+size_t pt_latent_attn_workspace_bytes(int n_tok, int n_head, int rot_dim, int rank, int dtype);
+int pt_latent_attn(const pt_latent_attn_args *args, void *stream);
 
 /* State-space (SSD) mixer between its two projections (csrc/ssm.cu): convolution, recurrence, gate and group norm.
  * zx rows hold [z | x | B | C | dt]; inner = heads * vdim, channels = inner + 2 groups * state_dim. */

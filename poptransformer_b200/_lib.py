@@ -19,7 +19,7 @@ class PtError(RuntimeError):
 class DenseExt(ctypes.Structure):
     _fields_ = [("bias", c_void_p), ("out2", c_void_p), ("out2_ld", c_int), ("split_n", c_int), ("limit", c_float), ("mul", c_void_p), ("mul_ld", c_int),
                 ("mul_ids", c_void_p), ("n_groups", c_int), ("group_rows", c_int), ("group_x_div", c_int), ("group_of", c_void_p),
-                ("group_used", c_void_p)]
+                ("group_used", c_void_p), ("glu", c_int), ("row_scale", c_void_p)]
 
 
 class LinearArgs(ctypes.Structure):
@@ -73,12 +73,37 @@ class HyperArgs(ctypes.Structure):
                [(n, c_void_p) for n in ("mix", "w_out", "w_in", "norm_w", "h")] + [("h_ld", c_int), ("sum_out", c_void_p)]
 
 
+class ContextRows(ctypes.Structure):
+    _fields_ = [("k", c_void_p), ("v", c_void_p), ("shared", c_void_p), ("ld", c_int), ("shared_ld", c_int), ("shared_dim", c_int), ("cu", c_void_p)]
+
+
 class WindowAttnArgs(ctypes.Structure):
     _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "n_head", "n_kv", "dim", "vdim", "page_size", "max_pages", "window", "keep_first")] + \
                [("scale", c_float), ("sink", c_void_p), ("q", c_void_p), ("q_ld", c_int), ("k", c_void_p), ("v", c_void_p), ("kv_ld", c_int),
                 ("pool", c_void_p), ("page_table", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("max_tokens_per_seq", c_int), ("max_len", c_int),
                 ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("error_flag", c_void_p), ("q_norm", c_void_p), ("k_norm", c_void_p),
-                ("norm_eps", c_float), ("rope_dims", c_int), ("rope", c_void_p), ("out_scale", c_float), ("out_cols", c_int)]
+                ("norm_eps", c_float), ("rope_dims", c_int), ("rope", c_void_p), ("out_scale", c_float), ("out_cols", c_int),
+                ("softcap", c_float), ("gate", c_void_p), ("gate_ld", c_int), ("gate_per_head", c_int), ("values_in_keys", c_int), ("value_col", c_int),
+                ("context", ctypes.POINTER(ContextRows))]
+
+
+class LatentPrepArgs(ctypes.Structure):
+    _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "q_rank", "rank", "rot_dim")] + [("eps", c_float), ("q", c_void_p), ("kv", c_void_p), ("ld", c_int)] + \
+               [(n, c_void_p) for n in ("q_norm", "kv_norm", "rope", "cq")] + [("cq_ld", c_int), ("pool", c_void_p), ("page_table", c_void_p)] + \
+               [(n, c_int) for n in ("page_size", "max_pages", "max_len")] + [("error_flag", c_void_p)]
+
+
+class LatentContextArgs(ctypes.Structure):
+    _fields_ = [("batch", BatchView), ("ctx_cu", c_void_p)] + [(n, c_int) for n in ("n_ctx", "rot_dim", "rank", "page_size", "max_pages")] + \
+               [(n, c_void_p) for n in ("pool", "page_table", "shared", "latent")] + [("latent_ld", c_int)]
+
+
+class LatentAttnArgs(ctypes.Structure):
+    _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("dtype", "n_head", "dim", "rot_dim", "vdim", "rank")] + \
+               [("scale", c_float), ("q", c_void_p), ("q_ld", c_int)] + [(n, c_void_p) for n in ("rope", "w_k", "w_v", "gate")] + \
+               [("gate_ld", c_int), ("pool", c_void_p), ("page_table", c_void_p)] + [(n, c_int) for n in ("page_size", "max_pages", "max_len")] + \
+               [("out", c_void_p), ("out_ld", c_int), ("out_cols", c_int), ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t),
+                ("error_flag", c_void_p)]
 
 
 class SsmArgs(ctypes.Structure):
@@ -99,13 +124,13 @@ class PostNormArgs(ctypes.Structure):
     _fields_ = [("rows", c_int), ("width", c_int), ("dtype", c_int), ("eps", c_float), ("x_in", c_void_p), ("x_out", c_void_p), ("table", c_void_p),
                 ("table_ld", c_int), ("vocab", c_int), ("ids", c_void_p), ("ids_ld", c_int)] + \
                [(n, c_void_p) for n in ("step_dev", "pos_out", "id_out", "row_index", "y")] + [("y_ld", c_int), ("pair_y", c_void_p), ("pair_dtype", c_int), ("pair_ld", c_int), ("top", c_int)] + \
-               [(n, c_void_p) for n in ("pair_w", "pair_row", "norm_w", "final_w", "h")] + [("h_ld", c_int)]
+               [(n, c_void_p) for n in ("pair_w", "pair_row", "norm_w", "final_w", "h")] + [("h_ld", c_int), ("h_cols", c_int), ("copy", c_void_p), ("copy_ld", c_int), ("copy_cols", c_int)]
 
 
 class MoeRouteArgs(ctypes.Structure):
     _fields_ = [("n_tok", c_int), ("experts", c_int), ("top", c_int), ("logits", c_void_p), ("logits_ld", c_int), ("expert", c_void_p), ("weight", c_void_p),
                 ("tile", c_int), ("max_tiles", c_int), ("pair_row", c_void_p), ("tile_expert", c_void_p), ("tile_rows", c_void_p), ("row_token", c_void_p), ("counts", c_void_p), ("h", c_void_p), ("h_bytes", c_int),
-                ("gathered", c_void_p)]
+                ("gathered", c_void_p), ("score", c_int), ("row_weight", c_void_p)]
 
 
 class LlamaLayer(ctypes.Structure):
@@ -147,6 +172,10 @@ SIGNATURES = {
     "pt_hyper": (c_int, [ctypes.POINTER(HyperArgs), c_void_p]),
     "pt_window_attn_workspace_bytes": (c_size_t, [c_int] * 7),
     "pt_window_attn": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),
+    "pt_latent_prep": (c_int, [ctypes.POINTER(LatentPrepArgs), c_void_p]),
+    "pt_latent_context": (c_int, [ctypes.POINTER(LatentContextArgs), c_void_p]),
+    "pt_latent_attn_workspace_bytes": (c_size_t, [c_int] * 5),
+    "pt_latent_attn": (c_int, [ctypes.POINTER(LatentAttnArgs), c_void_p]),
     "pt_ssm_workspace_bytes": (c_size_t, [c_int] * 5),
     "pt_ssm": (c_int, [ctypes.POINTER(SsmArgs), c_void_p]),
     "pt_norm_ce": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p]),

@@ -4,8 +4,12 @@
 //   STORE      out[m, n] = y
 //   RELU2      out[m, n] = max(y, 0)^2
 //   GELU_MUL   out[m, n] = gelu_tanh(y) * mul[mul_ids[m], n]
-//   GLU        weight rows alternate in blocks of eight, eight gate features and then the same eight up features:
-//              out[m, f] = g sigmoid(1.702 g) (u + 1),  g = min(gate, limit), u = clamp(up, -limit, limit)
+//   SOFTCAP    out[m, n] = limit * tanh(y / limit)
+//   GLU        weight rows alternate in blocks of eight, eight gate features and then the same eight up features; by `glu`:
+//     CLAMPED    out[m, f] = g sigmoid(1.702 g) (u + 1),  g = min(gate, limit), u = clamp(up, -limit, limit)
+//     SILU       out[m, f] = gate sigmoid(gate) up
+//     GELU       out[m, f] = gelu_tanh(gate) up
+// row_scale (optional, one factor per activation row) multiplies the sum before the bias: the product of a scaled row.
 // Outputs from split_n on skip the epilogue and go to a second, fp32 matrix: out2[m, n - split_n] = y.
 #pragma once
 #include <limits.h>
@@ -22,6 +26,8 @@ struct DenseOut {
   const int *mul_ids;
   int out_ld, out2_ld, split_n, mul_ld, epilogue, out_dt;
   float alpha, limit;
+  int glu;
+  const float *row_scale;
 };
 
 static inline DenseOut make_dense_out(void *out, int out_ld, int out_dt, int epilogue, float alpha, const pt_dense_ext *e) {
@@ -31,20 +37,22 @@ static inline DenseOut make_dense_out(void *out, int out_ld, int out_dt, int epi
   o.split_n = INT_MAX;
   if (e) {
     o.bias = e->bias; o.mul = e->mul; o.mul_ids = e->mul_ids; o.mul_ld = e->mul_ld; o.limit = e->limit;
+    o.glu = e->glu; o.row_scale = e->row_scale;
     if (e->out2) { o.out2 = e->out2; o.out2_ld = e->out2_ld; o.split_n = e->split_n; }
   }
   return o;
 }
-static inline bool dense_epilogue_known(int e) { return e == PT_EPI_STORE || e == PT_EPI_RELU2 || e == PT_EPI_GLU || e == PT_EPI_GELU_MUL; }
+static inline bool dense_epilogue_known(int e) { return e == PT_EPI_STORE || e == PT_EPI_RELU2 || e == PT_EPI_GLU || e == PT_EPI_GELU_MUL || e == PT_EPI_SOFTCAP; }
 // nullptr, or what is wrong with the combination.
 static inline const char *dense_ext_error(int epilogue, int n_out, const pt_dense_ext *e) {
-  if ((epilogue == PT_EPI_GLU || epilogue == PT_EPI_GELU_MUL) && !e) return "the epilogue needs its extra arguments";
+  if ((epilogue == PT_EPI_GLU || epilogue == PT_EPI_GELU_MUL || epilogue == PT_EPI_SOFTCAP) && !e) return "the epilogue needs its extra arguments";
   if (!e) return nullptr;
   if (epilogue == PT_EPI_GELU_MUL && !(e->mul && e->mul_ids)) return "a gelu-times-row epilogue needs mul and mul_ids";
   if (e->out2 && (e->split_n < 0 || e->split_n % 32 || e->split_n > n_out || e->out2_ld < n_out - e->split_n))
     return "split_n must be a multiple of 32 within n_out, and out2_ld hold the rest";
   if (epilogue == PT_EPI_GLU && (e->out2 ? e->split_n : n_out) % 16) return "gated features come in blocks of eight";
-  if (epilogue == PT_EPI_GLU && !(e->limit > 0.f)) return "a gated epilogue needs a positive limit";
+  if (epilogue == PT_EPI_GLU && (e->glu < PT_GLU_CLAMPED || e->glu > PT_GLU_GELU)) return "unknown kind of gated unit";
+  if (((epilogue == PT_EPI_GLU && e->glu == PT_GLU_CLAMPED) || epilogue == PT_EPI_SOFTCAP) && !(e->limit > 0.f)) return "the epilogue needs a positive limit";
   if (e->n_groups < 0 || (e->n_groups > 0 && (!e->group_of || e->group_rows < 1))) return "groups need group_of and group_rows";
   return nullptr;
 }
@@ -57,7 +65,10 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
 __device__ __forceinline__ float gelu_tanh_fast(float x) {
   return __fdividef(x, 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * x * x, x, x)));
 }
-template <bool FAST> __device__ __forceinline__ float glu_f(float gate, float up, float limit) {
+template <bool FAST> __device__ __forceinline__ float glu_f(const DenseOut &o, float gate, float up) {
+  if (o.glu == PT_GLU_SILU) return (FAST ? __fdividef(gate, 1.0f + __expf(-gate)) : gate / (1.0f + expf(-gate))) * up;
+  if (o.glu == PT_GLU_GELU) return (FAST ? gelu_tanh_fast(gate) : gelu_tanh_f(gate)) * up;
+  const float limit = o.limit;
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   if (FAST) return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);   // (rounded to bf16 by the caller; for g very negative the quotient is 0)
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
@@ -67,10 +78,11 @@ __device__ __forceinline__ void dense_put(const DenseOut &o, int m, int n, float
   if (o.out_dt == PT_DT_F32) reinterpret_cast<float *>(o.out)[i] = y;
   else reinterpret_cast<__nv_bfloat16 *>(o.out)[i] = __float2bfloat16_rn(y);
 }
-__device__ __forceinline__ float dense_value(const DenseOut &o, int n, float acc) { return fmaf(acc, o.alpha, o.bias ? __ldg(o.bias + n) : 0.f); }
+__device__ __forceinline__ float dense_factor(const DenseOut &o, int m) { return o.row_scale ? o.alpha * __ldcg(o.row_scale + m) : o.alpha; }
+__device__ __forceinline__ float dense_value(const DenseOut &o, int m, int n, float acc) { return fmaf(acc, dense_factor(o, m), o.bias ? __ldg(o.bias + n) : 0.f); }
 // One finished sum (any epilogue but GLU, whose sums come in pairs).
 __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, float acc) {
-  float y = dense_value(o, n, acc);
+  float y = dense_value(o, m, n, acc);
   if (n >= o.split_n) {
     o.out2[(size_t)m * o.out2_ld + n - o.split_n] = y;
     return;
@@ -78,6 +90,8 @@ __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, flo
   if (o.epilogue == PT_EPI_RELU2) {
     y = fmaxf(y, 0.f);
     y *= y;
+  } else if (o.epilogue == PT_EPI_SOFTCAP) {
+    y = o.limit * tanhf(y / o.limit);
   } else if (o.epilogue == PT_EPI_GELU_MUL) {
     const size_t i = (size_t)o.mul_ids[m] * o.mul_ld + n;
     y = gelu_tanh_f(y) * (o.out_dt == PT_DT_F32 ? reinterpret_cast<const float *>(o.mul)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16 *>(o.mul)[i]));
@@ -87,8 +101,8 @@ __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, flo
 // Sums of the gate row n (n % 16 < 8) and the up row n + 8.
 __device__ __forceinline__ void dense_store_glu(const DenseOut &o, int m, int n, float gate, float up) {
   const int f = n / 16 * 8 + n % 8;
-  const float g = dense_value(o, n, gate), u = dense_value(o, n + 8, up);
-  dense_put(o, m, f, o.out_dt == PT_DT_F32 ? glu_f<false>(g, u, o.limit) : glu_f<true>(g, u, o.limit));
+  const float g = dense_value(o, m, n, gate), u = dense_value(o, m, n + 8, up);
+  dense_put(o, m, f, o.out_dt == PT_DT_F32 ? glu_f<false>(o, g, u) : glu_f<true>(o, g, u));
 }
 #endif
 

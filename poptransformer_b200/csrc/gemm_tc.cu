@@ -244,12 +244,14 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 // bf16 output: neighbouring lanes (n, n + 1) trade values of two columns, so every store writes 4 bytes per lane.
 // Gated features: lanes n and n + 8 trade likewise, and each computes one column of the pair's feature.
 enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_GLU = 2, OUT_GELU_MUL = 3 };
-template <int KIND, bool RELU2>
+enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2 };
+template <int KIND, int ACT>
 __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, int ld, const uint32_t (&v)[32], int n, int m, int lane) {
   const float b = d.bias ? __ldg(d.bias + n + (KIND == OUT_F32 && out == d.out2 ? d.split_n : 0)) : 0.f;
   auto fin = [&](uint32_t x) {
     float y = fmaf(__uint_as_float(x), d.alpha, b);
-    if (RELU2) { y = fmaxf(y, 0.f); y *= y; }
+    if (ACT == ACT_RELU2) { y = fmaxf(y, 0.f); y *= y; }
+    if (ACT == ACT_SOFTCAP) y = d.limit * tanhf(y / d.limit);
     return y;
   };
   if (KIND == OUT_F32) {
@@ -282,11 +284,13 @@ __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, in
   } else {
     const bool up = lane & 8;
     __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(out) + (size_t)(m + (up ? 1 : 0)) * ld + n / 16 * 8 + n % 8;
+    const float mine = d.row_scale ? __ldcg(d.row_scale + m + lane) : 1.f;     // lane j: the factor of row m + j
 #pragma unroll
     for (int j = 0; j < 32; j += 2) {
-      const float a = fin(v[j]), c = fin(v[j + 1]);
+      const float s0 = __shfl_sync(0xffffffffu, mine, j), s1 = __shfl_sync(0xffffffffu, mine, j + 1);
+      const float a = fmaf(__uint_as_float(v[j]), d.alpha * s0, b), c = fmaf(__uint_as_float(v[j + 1]), d.alpha * s1, b);
       const float t = __shfl_xor_sync(0xffffffffu, up ? a : c, 8);      // gate lane: the up value of column j; up lane: the gate value of j + 1
-      *o = __float2bfloat16_rn(up ? glu_f<true>(t, c, d.limit) : glu_f<true>(a, t, d.limit));
+      *o = __float2bfloat16_rn(up ? glu_f<true>(d, t, c) : glu_f<true>(d, a, t));
       o += 2 * (size_t)ld;
     }
   }
@@ -297,23 +301,25 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
   // (warp-uniform) where this warp's 32 outputs go
   const bool second = nq >= d.split_n, glu = d.epilogue == PT_EPI_GLU && !second, f32 = second || d.out_dt == PT_DT_F32;
   // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16
-  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) &&
+  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) && (glu || !d.row_scale) &&
+                    (second || f32 || d.epilogue != PT_EPI_SOFTCAP) &&
                     (f32 || glu || (d.out_ld % 2 == 0 && ((uintptr_t)d.out & 3) == 0));
   const int rows = min(p.mb, m_end - m0), whole = fast ? rows & ~31 : 0;
   for (int c0 = 0; c0 < whole; c0 += 32) {
     uint32_t v[32];
     tmem_ld32(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, v);
     if (second) {
-      epilogue_rows32<OUT_F32, false>(d, d.out2, d.out2_ld, v, n - d.split_n, m0 + c0, lane);
+      epilogue_rows32<OUT_F32, ACT_NONE>(d, d.out2, d.out2_ld, v, n - d.split_n, m0 + c0, lane);
     } else if (glu) {
-      epilogue_rows32<OUT_GLU, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      epilogue_rows32<OUT_GLU, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     } else if (f32) {
-      if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_F32, true>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
-      else epilogue_rows32<OUT_F32, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_F32, ACT_RELU2>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (d.epilogue == PT_EPI_SOFTCAP) epilogue_rows32<OUT_F32, ACT_SOFTCAP>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else epilogue_rows32<OUT_F32, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     } else {
-      if (d.epilogue == PT_EPI_GELU_MUL) epilogue_rows32<OUT_GELU_MUL, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
-      else if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_BF16, true>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
-      else epilogue_rows32<OUT_BF16, false>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      if (d.epilogue == PT_EPI_GELU_MUL) epilogue_rows32<OUT_GELU_MUL, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_BF16, ACT_RELU2>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else epilogue_rows32<OUT_BF16, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     }
   }
   if (whole < rows) epilogue<true>(p, tmem, q, lane, 0, 1, n0, m0, m_end, ks, whole);
@@ -821,7 +827,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   PT_REQUIRE(a->x && a->w && a->out, "pt_gemm: null x / w / out");
   PT_REQUIRE(((uintptr_t)a->x & 15) == 0 && ((uintptr_t)a->w & 15) == 0, "pt_gemm: x and w must be 16-byte aligned");
   if (bf16) {
-    PT_REQUIRE(dense_epilogue_known(a->epilogue), "pt_gemm: BF16 epilogue %d (store, relu2, glu or gelu-mul)", a->epilogue);
+    PT_REQUIRE(dense_epilogue_known(a->epilogue), "pt_gemm: BF16 epilogue %d (store, relu2, glu, gelu-mul or softcap)", a->epilogue);
     const char *bad = dense_ext_error(a->epilogue, a->n_out, a->ext);
     PT_REQUIRE(!bad, "pt_gemm: %s", bad);
     PT_REQUIRE(a->out_dtype == PT_DT_BF16 || a->out_dtype == PT_DT_F32, "pt_gemm: BF16 weights write bf16 or fp32, got type %d", a->out_dtype);

@@ -606,7 +606,7 @@ extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   PT_REQUIRE(a->prologue >= PT_PRO_NONE && a->prologue <= PT_PRO_NORMCE, "pt_linear: bad prologue %d", a->prologue);
   if (a->wfmt == PT_W_BF16) {
     PT_REQUIRE(a->prologue == PT_PRO_NONE && dense_epilogue_known(a->epilogue),
-               "pt_linear: bf16 weights take no prologue and the store, relu2, glu or gelu-mul epilogue, got %d / %d", a->prologue, a->epilogue);
+               "pt_linear: bf16 weights take no prologue and the store, relu2, glu, gelu-mul or softcap epilogue, got %d / %d", a->prologue, a->epilogue);
     const char *bad = dense_ext_error(a->epilogue, a->n_out, a->ext);
     PT_REQUIRE(!bad, "pt_linear: %s", bad);
     PT_REQUIRE(!grouped || (a->ext->group_rows == 1 && a->ext->group_x_div >= 1), "pt_linear: groups come row by row");

@@ -1,6 +1,6 @@
 // Mixture of experts: which experts a token goes to, and where its rows lie for the grouped products.
-//   choose   per token the `top` experts with the largest router logits (the lowest index first among equals), and the softmax over
-//            those logits as weights.  fp32.
+//   choose   per token the `top` experts with the largest router logits (the lowest index first among equals), and as weights the
+//            softmax over those logits or their sigmoids.  fp32.
 //   place    pair i = token i / top with its choice i % top gets a row of its own among its expert's rows.  The rows of an expert are
 //            padded to whole tiles; tile_expert names the expert of every tile (-1: unused) and tile_rows its rows in use, so a grouped
 //            product can look its weights up per tile.  Pairs keep their order within an expert.
@@ -20,7 +20,8 @@ struct Params {
   int n_tok, experts, top, logits_ld, tile, max_tiles, hist_copies;
   const float *logits;
   int *expert, *pair_row, *tile_expert, *tile_rows, *row_token;   // [n_tok][top] x 2, [max_tiles] x 2, [max_tiles * tile]
-  float *weight;                                      // [n_tok][top]
+  float *weight, *row_weight;                         // [n_tok][top], [max_tiles * tile] or null: the weight of every placed row
+  int sigmoid;                                        // weights: sigmoid(logit) instead of the softmax over the chosen
   const int *counts;                                  // [experts], or null: counted while placing
 };
 
@@ -48,7 +49,7 @@ __global__ void choose_kernel(const Params p) {
     }
     if (at == INT_MAX) at = k;                          // only infinities or NaN are left
     if (k == 0) first = best;
-    const float w = expf(best - first);
+    const float w = p.sigmoid ? 1.0f / (1.0f + expf(-best)) : expf(best - first);
     sum += w;
     if (lane == (k & 31)) {
       (k < 32 ? w0 : w1) = w;
@@ -57,6 +58,7 @@ __global__ void choose_kernel(const Params p) {
     }
     __syncwarp();
   }
+  if (p.sigmoid) sum = 1.f;
   if (lane < p.top) p.weight[(size_t)t * p.top + lane] = w0 / sum;
   if (lane + 32 < p.top) p.weight[(size_t)t * p.top + lane + 32] = w1 / sum;
 }
@@ -161,6 +163,7 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
   for (int i = i0; hits > 0 && i < i1; ++i)
     if (p.expert[i] == e) {
       p.pair_row[i] = row;
+      if (p.row_weight) p.row_weight[row] = p.weight[i];
       p.row_token[row++] = i / p.top;
     }
 }
@@ -196,6 +199,8 @@ extern "C" int pt_moe_route(const pt_moe_route_args *a, void *stream) {
   PT_REQUIRE(a->logits && a->logits_ld >= a->experts && a->expert && a->weight, "pt_moe_route: null pointer argument");
   moe::Params p{};
   p.n_tok = a->n_tok; p.experts = a->experts; p.top = a->top; p.logits_ld = a->logits_ld; p.logits = a->logits; p.expert = a->expert; p.weight = a->weight;
+  PT_REQUIRE(a->score == PT_MOE_SOFTMAX || a->score == PT_MOE_SIGMOID, "pt_moe_route: weights of kind %d", a->score);
+  p.sigmoid = a->score == PT_MOE_SIGMOID;
   cudaStream_t st = as_stream(stream);
   moe::choose_kernel<<<ceil_div(p.n_tok, 4), 128, 0, st>>>(p);
   PT_LAUNCH_CHECK("pt_moe_route");
@@ -203,6 +208,7 @@ extern "C" int pt_moe_route(const pt_moe_route_args *a, void *stream) {
   PT_REQUIRE(a->tile > 0 && a->pair_row && a->tile_expert && a->tile_rows && a->row_token && a->max_tiles >= pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile),
              "pt_moe_route: tiles of %d rows need pair_row, row_token and %d entries of tile_expert", a->tile, pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile));
   p.tile = a->tile; p.max_tiles = a->max_tiles; p.pair_row = a->pair_row; p.tile_expert = a->tile_expert; p.tile_rows = a->tile_rows; p.row_token = a->row_token;
+  p.row_weight = a->row_weight;
   if (p.n_tok * p.top > 4096 && a->counts && aligned_to(p.expert, 16)) {
     moe::count_kernel<<<p.experts, moe::PLACE_THREADS, 0, st>>>(p.expert, p.n_tok * p.top, a->counts);
     PT_LAUNCH_CHECK("pt_moe_route");

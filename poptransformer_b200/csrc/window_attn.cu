@@ -1,6 +1,9 @@
 // Masked attention over a paged cache with per-sequence positions: a sliding window, kept first tokens, a softmax sink, grouped
 // heads, key and value widths of their own, optionally a norm and a rotation of every query and key head.  Position i sees key j when j <= i and (i - j < window or j < keep_first);
-// window = 0 means every earlier key.  sink[h] acts as one more logit of head h that brings weight to the denominator only.
+// window = 0 means every earlier key.  sink[h] acts as one more logit of head h that brings weight to the denominator only.  With a
+// softcap c a score s becomes c tanh(s / c).  The output can be multiplied with the sigmoid of a gate, per element or per head.
+// The values can be a part of the cached keys (a latent that all heads share), and prompts can read keys and values from rows of the
+// whole context instead of pages (pt_context_rows: a latent that was projected up), with a part of the key shared by all heads.
 //
 // The tokens of a launch are packed sequence after sequence (pt_batch_view): row cu[s] + i is position start[s] + i of sequence s,
 // whose pages are page_table[slot[s]].  A page holds K [n_kv][page][dim] and then V [n_kv][page][vdim].  New keys and values are
@@ -34,6 +37,15 @@ struct Params {
   const float2 *rope;        // [positions][rope_half]
   float norm_eps, out_scale;
   int rope_half, out_cols;
+  const void *gate;          // [n_tok][gate_ld]: n_head * vdim columns, or n_head with gate_heads
+  int gate_ld;
+  bool gate_heads, v_in_k;   // v_in_k: the pool holds keys only, the values are their dimensions v_col ..
+  int v_col, hsplit;         // hsplit: blocks that share a kv head's query heads (plain kernel)
+  float softcap;
+  // rows of the whole context (prompts)
+  const __nv_bfloat16 *ctx_k, *ctx_shared, *ctx_v;
+  int ctx_ld, shared_ld, shared_dim;
+  const int *ctx_cu;
   bool prep, pair_rows;      // queries and keys are normalised or rotated; their rows can be taken as pairs of neighbours
   // decode
   int grid_pages, qsplit;
@@ -42,12 +54,29 @@ struct Params {
   int *counters;    // [n_seq, n_kv, qsplit]
 };
 
-__device__ __forceinline__ size_t page_elems(const Params &p) { return (size_t)p.n_kv * p.page * (p.dim + p.vdim); }
+__device__ __forceinline__ size_t page_elems(const Params &p) { return (size_t)p.n_kv * p.page * (p.v_in_k ? p.dim : p.dim + p.vdim); }
 template <typename T> __device__ __forceinline__ T *k_page(const Params &p, int phys, int g) {
   return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems(p) + (size_t)g * p.page * p.dim;
 }
 template <typename T> __device__ __forceinline__ T *v_page(const Params &p, int phys, int g) {
+  if (p.v_in_k) return k_page<T>(p, phys, g) + p.v_col;
   return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems(p) + (size_t)p.n_kv * p.page * p.dim + (size_t)g * p.page * p.vdim;
+}
+// Scores in the units of exp2 from raw products: scale and softcap.  (tanh z = 1 - 2 / (exp(2 z) + 1))
+struct Score {
+  float a, b;                // without a cap: a = scale log2(e).  With: b = cap log2(e), a = 2 scale log2(e) / cap
+  bool capped;
+  __device__ __forceinline__ Score(const Params &p) {
+    capped = p.softcap > 0.f;
+    a = capped ? 2.0f * p.scale * kLog2e / p.softcap : p.scale * kLog2e;
+    b = p.softcap * kLog2e;
+  }
+  __device__ __forceinline__ float operator()(float s) const { return capped ? b * (1.0f - __fdividef(2.0f, exp2f(a * s) + 1.0f)) : a * s; }
+};
+template <typename T> __device__ __forceinline__ float gate_at(const Params &p, int t, int head, int c) {
+  if (!p.gate) return 1.f;
+  const float z = to_f(reinterpret_cast<const T *>(p.gate)[(size_t)t * p.gate_ld + (p.gate_heads ? head : head * p.vdim + c)]);
+  return 1.0f / (1.0f + expf(-z));
 }
 __device__ __forceinline__ bool visible(const Params &p, int pos, int key) {
   return key <= pos && (p.window == 0 || pos - key < p.window || key < p.keep_first);
@@ -60,16 +89,16 @@ __device__ __forceinline__ int kept_pages(const Params &p, int pos) { return (mi
 // ------------------------------------------------------------------------------------------ norm, rotation, append
 // One warp, a head's row of a query or key at a time.  put(i, value) may write over src (a lane reads what it writes).
 template <typename T, typename Put>
-__device__ __forceinline__ void norm_rotate_any(const Params &p, const T *src, const float *norm, int pos, Put put) {
+__device__ __forceinline__ void norm_rotate_any(const Params &p, int dim, const T *src, const float *norm, int pos, Put put) {
   const int lane = threadIdx.x & 31, half = p.rope_half;
   float inv = 1.f;
   if (norm) {
     float ss = 0.f;
-    for (int i = lane; i < p.dim; i += 32) {
+    for (int i = lane; i < dim; i += 32) {
       const float x = to_f(src[i]);
       ss = fmaf(x, x, ss);
     }
-    inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.norm_eps);
+    inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + p.norm_eps);
   }
   auto at = [&](int i) { return to_f(src[i]) * inv * (norm ? __ldg(norm + i) : 1.f); };
   const float2 *cs = p.rope + (size_t)pos * half;
@@ -79,7 +108,7 @@ __device__ __forceinline__ void norm_rotate_any(const Params &p, const T *src, c
     put(i, u * c.x - v * c.y);
     put(i + half, v * c.x + u * c.y);
   }
-  for (int i = 2 * half + lane; i < p.dim; i += 32) put(i, at(i));
+  for (int i = 2 * half + lane; i < dim; i += 32) put(i, at(i));
 }
 // The same in registers for rows of up to 128 dimensions (p.pair_rows): a lane holds the neighbours i, i + 1 and their partners j,
 // j + 1.  Behind the rotated dimensions the partners are the next two, and the angle is zero.  Angles and weights serve all heads.
@@ -89,9 +118,9 @@ struct HeadLane {
   int i, j;
   bool on;
   float2 c0, c1, wi, wj;
-  __device__ __forceinline__ HeadLane(const Params &p, const float *norm, int pos) {
+  __device__ __forceinline__ HeadLane(const Params &p, int dim, const float *norm, int pos) {
     const int u = 2 * (threadIdx.x & 31), half = p.rope_half;
-    on = p.pair_rows && u < p.dim / 2;       // (nothing is loaded for rows that are taken the other way)
+    on = p.pair_rows && u < dim / 2;       // (nothing is loaded for rows that are taken the other way)
     i = u < half ? u : 2 * u;
     j = u < half ? u + half : 2 * u + 2;
     c0 = c1 = make_float2(1.f, 0.f);
@@ -121,9 +150,9 @@ struct HeadLane {
     store_vec<2>(dst + j, b);
   }
 };
-template <typename T> __device__ __forceinline__ void norm_rotate(const Params &p, const HeadLane &hl, const T *src, const float *norm, int pos, T *dst) {
+template <typename T> __device__ __forceinline__ void norm_rotate(const Params &p, int dim, const HeadLane &hl, const T *src, const float *norm, int pos, T *dst) {
   if (p.pair_rows) hl.run<T>(p, src, norm != nullptr, dst);
-  else norm_rotate_any<T>(p, src, norm, pos, [&](int i, float y) { dst[i] = from_f<T>(y); });
+  else norm_rotate_any<T>(p, dim, src, norm, pos, [&](int i, float y) { dst[i] = from_f<T>(y); });
 }
 
 constexpr int PREP_WARPS = 4;
@@ -135,20 +164,21 @@ template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_pr
     return;
   }
   {
-    const HeadLane hl(p, p.q_norm, pos);
+    const int dim = p.q_norm ? p.dim : 2 * p.rope_half;       // (in place: what is not rotated stays)
+    const HeadLane hl(p, dim, p.q_norm, pos);
 #pragma unroll 4
     for (int h = warp; h < p.n_head; h += PREP_WARPS) {
       T *q = reinterpret_cast<T *>(const_cast<void *>(p.q)) + (size_t)t * p.q_ld + (size_t)h * p.dim;
-      norm_rotate<T>(p, hl, q, p.q_norm, pos, q);
+      norm_rotate<T>(p, dim, hl, q, p.q_norm, pos, q);
     }
   }
   if (!p.k) return;
-  const HeadLane hl(p, p.k_norm, pos);
+  const HeadLane hl(p, p.dim, p.k_norm, pos);
   const int phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page], at = pos % p.page;
   for (int g = warp; g < p.n_kv; g += PREP_WARPS) {
     const T *k = reinterpret_cast<const T *>(p.k) + (size_t)t * p.kv_ld + (size_t)g * p.dim, *v = reinterpret_cast<const T *>(p.v) + (size_t)t * p.kv_ld + (size_t)g * p.vdim;
     T *kc = k_page<T>(p, phys, g) + (size_t)at * p.dim, *vc = v_page<T>(p, phys, g) + (size_t)at * p.vdim;
-    norm_rotate<T>(p, hl, k, p.k_norm, pos, kc);
+    norm_rotate<T>(p, p.dim, hl, k, p.k_norm, pos, kc);
     for (int i = lane; i < p.vdim; i += 32) vc[i] = v[i];
   }
 }
@@ -166,24 +196,25 @@ template <typename T> __global__ void kv_append_kernel(const Params p) {
 }
 
 // ------------------------------------------------------------------------------------------ plain
-// Block: one token and one kv head (all of its query heads).  Dynamic shared memory: q [qpk][dim], scores [qpk][page], o [qpk][vdim],
-// statistics [qpk][3].
+// Block: one token and the query heads of one kv head, or a part of them (nh).  Dynamic shared memory: q [nh][dim], scores [nh][page],
+// o [nh][vdim], statistics [nh][3].
 constexpr int PLAIN_THREADS = 128;
 template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plain_kernel(const Params p) {
   extern __shared__ __align__(16) float sm[];
-  float *q = sm, *sc = q + p.qpk * p.dim, *o = sc + p.qpk * p.page, *st = o + p.qpk * p.vdim;   // st: running max, sum, correction
-  const int t = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int nh = p.qpk / p.hsplit, g = blockIdx.y / p.hsplit, h0 = blockIdx.y * nh, v_ld = p.v_in_k ? p.dim : p.vdim;   // (heads h0 .. h0 + nh - 1)
+  float *q = sm, *sc = q + nh * p.dim, *o = sc + nh * p.page, *st = o + nh * p.vdim;   // st: running max, sum, correction
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
   if (pos < 0 || pos >= p.max_len) {
     if (tid == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
   }
   const int *table = p.page_table + (size_t)p.slot[s] * p.max_pages;
-  const T *qrow = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)g * p.qpk * p.dim;
-  for (int i = tid; i < p.qpk * p.dim; i += PLAIN_THREADS) q[i] = to_f(qrow[i]);
-  for (int i = tid; i < p.qpk * p.vdim; i += PLAIN_THREADS) o[i] = 0.f;
-  for (int h = tid; h < p.qpk; h += PLAIN_THREADS) {
-    st[3 * h] = p.sink ? p.sink[g * p.qpk + h] : -INFINITY;
+  const T *qrow = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * p.dim;
+  for (int i = tid; i < nh * p.dim; i += PLAIN_THREADS) q[i] = to_f(qrow[i]);
+  for (int i = tid; i < nh * p.vdim; i += PLAIN_THREADS) o[i] = 0.f;
+  for (int h = tid; h < nh; h += PLAIN_THREADS) {
+    st[3 * h] = p.sink ? p.sink[h0 + h] : -INFINITY;
     st[3 * h + 1] = p.sink ? 1.f : 0.f;
   }
   const int kept = kept_pages(p, pos), wpage = window_page(p, pos);
@@ -192,15 +223,17 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
     const int k0 = pg * p.page, nk = min(p.page, pos + 1 - k0);
     const T *K = k_page<T>(p, table[pg], g), *V = v_page<T>(p, table[pg], g);
     __syncthreads();
-    for (int i = warp; i < p.qpk * nk; i += PLAIN_THREADS / 32) {
+    for (int i = warp; i < nh * nk; i += PLAIN_THREADS / 32) {
       const int h = i / nk, key = i - h * nk;
       float a = 0.f;
       for (int c = lane; c < p.dim; c += 32) a = fmaf(q[h * p.dim + c], to_f(K[(size_t)key * p.dim + c]), a);
       a = warp_sum(a);
-      if (lane == 0) sc[h * p.page + key] = visible(p, pos, k0 + key) ? a * p.scale : -INFINITY;
+      a *= p.scale;
+      if (p.softcap > 0.f) a = p.softcap * tanhf(a / p.softcap);
+      if (lane == 0) sc[h * p.page + key] = visible(p, pos, k0 + key) ? a : -INFINITY;
     }
     __syncthreads();
-    for (int h = warp; h < p.qpk; h += PLAIN_THREADS / 32) {
+    for (int h = warp; h < nh; h += PLAIN_THREADS / 32) {
       float m = st[3 * h];
       for (int i = lane; i < nk; i += 32) m = fmaxf(m, sc[h * p.page + i]);
       m = warp_max(m);
@@ -220,16 +253,17 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
       }
     }
     __syncthreads();
-    for (int i = tid; i < p.qpk * p.vdim; i += PLAIN_THREADS) {
+    for (int i = tid; i < nh * p.vdim; i += PLAIN_THREADS) {
       const int h = i / p.vdim, c = i - h * p.vdim;
       float a = o[i] * st[3 * h + 2];
-      for (int key = 0; key < nk; ++key) a = fmaf(sc[h * p.page + key], to_f(V[(size_t)key * p.vdim + c]), a);
+      for (int key = 0; key < nk; ++key) a = fmaf(sc[h * p.page + key], to_f(V[(size_t)key * v_ld + c]), a);
       o[i] = a;
     }
   }
-  T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld + (size_t)g * p.qpk * p.vdim;
-  for (int i = tid; i < p.qpk * p.vdim; i += PLAIN_THREADS) out[i] = from_f<T>(o[i] / st[3 * (i / p.vdim) + 1] * p.out_scale);
-  if (g == p.n_kv - 1)   // k padding of the output product
+  T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld + (size_t)h0 * p.vdim;
+  for (int i = tid; i < nh * p.vdim; i += PLAIN_THREADS)
+    out[i] = from_f<T>(o[i] / st[3 * (i / p.vdim) + 1] * p.out_scale * gate_at<T>(p, t, h0 + i / p.vdim, i % p.vdim));
+  if (blockIdx.y == gridDim.y - 1)   // k padding of the output product
     for (int i = p.n_head * p.vdim + tid; i < p.out_cols; i += PLAIN_THREADS) reinterpret_cast<T *>(p.out)[(size_t)t * p.out_ld + i] = from_f<T>(0.f);
 }
 
@@ -239,8 +273,9 @@ constexpr int TC_THREADS = 128, TILE = 64;   // TILE = the page size the tensor-
 // ------------------------------------------------------------------------------------------ prompts
 // Block: 64 new tokens of one sequence, one head; warp w owns queries 16 w .. 16 w + 15, their q fragments stay in registers.  Key
 // tiles (one page each) are double-buffered in shared memory; tiles without a visible key are skipped, tiles that every query of
-// the warp sees completely take no mask.  DK / DV: dim / vdim rounded up to 32, 64 or 128 (the padding holds zeros).
-template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS, 3) attn_prompt_kernel(const Params p) {
+// the warp sees completely take no mask.  DK / DV: dim / vdim rounded up to 32, 64, 128 .. (the padding holds zeros).  CTX: keys and
+// values are rows of the context; the first shared_dim dimensions of a key belong to all heads.
+template <int DK, int DV, bool CTX> __global__ void __launch_bounds__(TC_THREADS, DK > 128 ? 2 : 3) attn_prompt_kernel(const Params p) {
   constexpr int KLD = DK + 8, VLD = DV + 8;
   extern __shared__ __align__(16) __nv_bfloat16 smb[];
   __nv_bfloat16 *Ks = smb, *Vs = smb + 2 * TILE * KLD;      // [2][TILE][KLD], [2][TILE][VLD]
@@ -272,6 +307,25 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS, 3) attn_
     }
   }
   auto load_tile = [&](int kt, int stage) {
+    if constexpr (CTX) {
+      const size_t row = (size_t)p.ctx_cu[s] + kt * TILE;
+      const int own = p.dim - p.shared_dim;
+      const __nv_bfloat16 *gS = p.ctx_shared + row * p.shared_ld, *gK = p.ctx_k + row * p.ctx_ld + (size_t)kvh * own - p.shared_dim,
+                          *gV = p.ctx_v + row * p.ctx_ld + (size_t)kvh * p.vdim;
+      __nv_bfloat16 *k = Ks + stage * TILE * KLD, *v = Vs + stage * TILE * VLD;
+      for (int e = tid; e < TILE * (DK / 8); e += TC_THREADS) {
+        const int r = e / (DK / 8), c = (e % (DK / 8)) * 8;
+        const bool in = kt * TILE + r <= hi && c < p.dim;
+        cp16(k + r * KLD + c, !in ? p.ctx_k : c < p.shared_dim ? gS + (size_t)r * p.shared_ld + c : gK + (size_t)r * p.ctx_ld + c, in);
+      }
+      for (int e = tid; e < TILE * (DV / 8); e += TC_THREADS) {
+        const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
+        const bool in = kt * TILE + r <= hi && c < p.vdim;
+        cp16(v + r * VLD + c, in ? gV + (size_t)r * p.ctx_ld + c : p.ctx_k, in);
+      }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+      return;
+    }
     const int phys = table[kt];
     const __nv_bfloat16 *gK = k_page<__nv_bfloat16>(p, phys, kvh), *gV = v_page<__nv_bfloat16>(p, phys, kvh);
     __nv_bfloat16 *k = Ks + stage * TILE * KLD, *v = Vs + stage * TILE * VLD;
@@ -289,7 +343,8 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS, 3) attn_
   };
   const int kept = kept_pages(p, hi), wtile = window_page(p, lo), last = hi / TILE;
   auto next_tile = [&](int kt) { return (kt >= kept && kt < wtile) ? wtile : kt; };
-  const float sc2 = p.scale * kLog2e, sink2 = p.sink ? p.sink[head] * kLog2e : -INFINITY;
+  const Score score(p);
+  const float sink2 = p.sink ? p.sink[head] * kLog2e : -INFINITY;
   float o[DV / 8][4];
 #pragma unroll
   for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
@@ -330,7 +385,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS, 3) attn_
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = k0 + j * 8 + 2 * tig + (e & 1);
-          float v = sc[j][e] * sc2;
+          float v = score(sc[j][e]);
           if (!whole && !visible(p, e < 2 ? pos0 : pos1, key)) v = -INFINITY;
           sc[j][e] = v;
           m_new[e >> 1] = fmaxf(m_new[e >> 1], v);
@@ -390,9 +445,23 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS, 3) attn_
     inv[r] = p.out_scale / l;
   }
   __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(p.out) + (size_t)head * p.vdim + 2 * tig;
+  if (p.gate && p.gate_heads) {
+    if (ok0) inv[0] *= gate_at<__nv_bfloat16>(p, row0 + q0, head, 0);
+    if (ok1) inv[1] *= gate_at<__nv_bfloat16>(p, row0 + q1, head, 0);
+  }
+  const bool each = p.gate && !p.gate_heads;
 #pragma unroll
   for (int j = 0; j < DV / 8; ++j) {
     if (j * 8 >= p.vdim) break;
+    if (each) {
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        if (!(r ? ok1 : ok0)) continue;
+        const float2 z = load_pair(reinterpret_cast<const __nv_bfloat16 *>(p.gate) + (size_t)(row0 + (r ? q1 : q0)) * p.gate_ld + head * p.vdim + 2 * tig + j * 8);
+        o[j][2 * r] *= __fdividef(1.0f, 1.0f + __expf(-z.x));          // (rounded to bf16 below)
+        o[j][2 * r + 1] *= __fdividef(1.0f, 1.0f + __expf(-z.y));
+      }
+    }
     if (ok0) *reinterpret_cast<uint32_t *>(out + (size_t)(row0 + q0) * p.out_ld + j * 8) = pack_bf2(o[j][0] * inv[0], o[j][1] * inv[0]);
     if (ok1) *reinterpret_cast<uint32_t *>(out + (size_t)(row0 + q1) * p.out_ld + j * 8) = pack_bf2(o[j][2] * inv[1], o[j][3] * inv[1]);
   }
@@ -467,11 +536,11 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
   asm volatile("cp.async.commit_group;" ::: "memory");
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * p.dim;
   if (p.prep) {
-    const HeadLane hq(p, p.q_norm, pos), hk(p, p.k_norm, pos);
+    const HeadLane hq(p, p.dim, p.q_norm, pos), hk(p, p.dim, p.k_norm, pos);
     for (int h = warp; h < NQ + 1; h += TC_THREADS / 32) {
       T *dst = h < NQ ? qs + h * QLD : kn;
       const bool have = h < NQ ? h < nq : owner;
-      if (have) norm_rotate<T>(p, h < NQ ? hq : hk, h < NQ ? q + (size_t)h * p.dim : knew, h < NQ ? p.q_norm : p.k_norm, pos, dst);
+      if (have) norm_rotate<T>(p, p.dim, h < NQ ? hq : hk, h < NQ ? q + (size_t)h * p.dim : knew, h < NQ ? p.q_norm : p.k_norm, pos, dst);
       for (int i = (have ? p.dim : 0) + lane; i < DK; i += 32) dst[i] = from_f<T>(0.f);
     }
   } else for (int i = tid; i < NQ * (DK / 8); i += TC_THREADS) {
@@ -505,11 +574,11 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
       mma16816_bf16(sc, kf[0][pp].x, kf[1][pp].x, kf[0][pp].y, kf[1][pp].y, qv.x, qv.y);
       mma16816_bf16(sc, kf[0][pp].z, kf[1][pp].z, kf[0][pp].w, kf[1][pp].w, qv.z, qv.w);
     }
-    const float sc2 = p.scale * kLog2e;
+    const Score score(p);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {                              // keys 16 warp + g (+ 8) against heads 2 tig, 2 tig + 1
       const int key = warp * 16 + g + 8 * (e >> 1), h = 2 * tig + (e & 1);
-      if (h < nq && key < n_valid && visible(p, pos, k0 + key)) ps[h * PSLD + key] = sc[e] * sc2;
+      if (h < nq && key < n_valid && visible(p, pos, k0 + key)) ps[h * PSLD + key] = score(sc[e]);
     }
   }
   __syncthreads();
@@ -607,7 +676,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
         }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) acc[j] *= ml[2 * h];
+    for (int j = 0; j < 4; ++j) acc[j] *= ml[2 * h] * gate_at<T>(p, t, h0 + h, c + j);
     T *o = out + (size_t)(h0 + h) * p.vdim + c;                // (rows of an even number of elements)
     *reinterpret_cast<__nv_bfloat162 *>(o) = __floats2bfloat162_rn(acc[0], acc[1]);
     *reinterpret_cast<__nv_bfloat162 *>(o + 2) = __floats2bfloat162_rn(acc[2], acc[3]);
@@ -616,11 +685,11 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
     for (int i = p.n_head * p.vdim + tid; i < p.out_cols; i += TC_THREADS) out[i] = from_f<T>(0.f);
 }
 
-template <int DK, int DV> static int launch_prompt(const Params &p, int longest, cudaStream_t st) {
+template <int DK, int DV, bool CTX> static int launch_prompt(const Params &p, int longest, cudaStream_t st) {
   constexpr size_t smem = 2 * (size_t)TILE * (DK + 8 + DV + 8) * sizeof(__nv_bfloat16);
   static bool set = false;
-  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_prompt_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set = true; }
-  attn_prompt_kernel<DK, DV><<<dim3(ceil_div(longest, TILE), p.n_head, p.n_seq), TC_THREADS, smem, st>>>(p);
+  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_prompt_kernel<DK, DV, CTX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set = true; }
+  attn_prompt_kernel<DK, DV, CTX><<<dim3(ceil_div(longest, TILE), p.n_head, p.n_seq), TC_THREADS, smem, st>>>(p);
   PT_LAUNCH_CHECK("pt_window_attn");
   return PT_OK;
 }
@@ -634,14 +703,23 @@ template <int DK, int DV> static int launch_decode(const Params &p, cudaStream_t
   return PT_OK;
 }
 template <int DK> static int dispatch_v(const Params &p, bool decode, int longest, cudaStream_t st) {
-  if (p.vdim <= 32) return decode ? launch_decode<DK, 32>(p, st) : launch_prompt<DK, 32>(p, longest, st);
-  if (p.vdim <= 64) return decode ? launch_decode<DK, 64>(p, st) : launch_prompt<DK, 64>(p, longest, st);
-  return decode ? launch_decode<DK, 128>(p, st) : launch_prompt<DK, 128>(p, longest, st);
+  if (p.vdim <= 32) return decode ? launch_decode<DK, 32>(p, st) : launch_prompt<DK, 32, false>(p, longest, st);
+  if (p.vdim <= 64) return decode ? launch_decode<DK, 64>(p, st) : launch_prompt<DK, 64, false>(p, longest, st);
+  return decode ? launch_decode<DK, 128>(p, st) : launch_prompt<DK, 128, false>(p, longest, st);
+}
+template <int DK> static int dispatch_ctx(const Params &p, int longest, cudaStream_t st) {
+  return p.vdim <= 64 ? launch_prompt<DK, 64, true>(p, longest, st) : launch_prompt<DK, 128, true>(p, longest, st);
 }
 static int dispatch_tc(const Params &p, bool decode, int longest, cudaStream_t st) {
   if (p.dim <= 32) return dispatch_v<32>(p, decode, longest, st);
   if (p.dim <= 64) return dispatch_v<64>(p, decode, longest, st);
   return dispatch_v<128>(p, decode, longest, st);
+}
+static int dispatch_ctx(const Params &p, int longest, cudaStream_t st) {
+  if (p.dim <= 64) return dispatch_ctx<64>(p, longest, st);
+  if (p.dim <= 128) return dispatch_ctx<128>(p, longest, st);
+  if (p.dim <= 192) return dispatch_ctx<192>(p, longest, st);
+  return dispatch_ctx<256>(p, longest, st);
 }
 
 }  // namespace wa
@@ -673,7 +751,8 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
              a->vdim, a->page_size, a->max_pages);
   PT_REQUIRE(a->window >= 0 && a->keep_first >= 0, "pt_window_attn: window=%d keep_first=%d", a->window, a->keep_first);
   PT_REQUIRE(a->dtype == PT_DT_F32 || a->dtype == PT_DT_BF16, "pt_window_attn: type %d (fp32 or bf16)", a->dtype);
-  PT_REQUIRE(a->q && a->pool && a->page_table && a->out && (!a->k == !a->v), "pt_window_attn: null pointer argument");
+  const pt_context_rows *ctx = a->context;
+  PT_REQUIRE(a->q && a->out && (ctx || (a->pool && a->page_table)) && (!a->k == !a->v), "pt_window_attn: null pointer argument");
   PT_REQUIRE(a->q_ld >= a->n_head * a->dim && a->out_ld >= a->n_head * a->vdim && (!a->k || a->kv_ld >= a->n_kv * std::max(a->dim, a->vdim)),
              "pt_window_attn: row strides q %d, kv %d, out %d too small", a->q_ld, a->kv_ld, a->out_ld);
   wa::Params p{};
@@ -683,25 +762,41 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
   p.q = a->q; p.k = a->k; p.v = a->v; p.pool = a->pool; p.out = a->out; p.page_table = a->page_table;
   p.cu = b.cu; p.start = b.start; p.slot = b.slot; p.tok_seq = b.tok_seq; p.error_flag = a->error_flag;
   p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.norm_eps = a->norm_eps; p.rope = (const float2 *)a->rope; p.rope_half = a->rope_dims / 2;
+  PT_REQUIRE(a->softcap >= 0.f && (!a->gate || a->gate_ld >= (a->gate_per_head ? a->n_head : a->n_head * a->vdim)), "pt_window_attn: softcap=%f gate_ld=%d", a->softcap,
+             a->gate_ld);
+  PT_REQUIRE(!a->values_in_keys || (!a->k && !ctx && a->value_col >= 0 && a->value_col + a->vdim <= a->dim),
+             "pt_window_attn: values that are dimensions of the cached keys need value_col + vdim within dim and nothing to append");
+  p.softcap = a->softcap; p.gate = a->gate; p.gate_ld = a->gate_ld; p.gate_heads = a->gate_per_head != 0;
+  p.v_in_k = a->values_in_keys != 0; p.v_col = a->value_col;
   p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.0f;
   p.out_cols = a->out_cols > 0 ? a->out_cols : a->out_ld;
   p.prep = a->q_norm || a->k_norm || a->rope_dims;
   {
     const int pair = a->dtype == PT_DT_F32 ? 8 : 4;
     auto al = [](const void *x, int bytes) { return ((uintptr_t)x & (bytes - 1)) == 0; };
-    p.pair_rows = a->dim % 4 == 0 && a->dim <= 128 && a->rope_dims % 4 == 0 && a->q_ld % 2 == 0 && a->n_kv * a->page_size * (a->dim + a->vdim) % 2 == 0 && al(a->q, pair) && al(a->pool, pair) && al(a->rope, 16) && al(a->q_norm, 8) &&
+    p.pair_rows = a->dim % 4 == 0 && (ctx && !a->q_norm ? a->rope_dims : a->dim) <= 128 && a->rope_dims % 4 == 0 && a->q_ld % 2 == 0 && a->n_kv * a->page_size * (p.v_in_k ? a->dim : a->dim + a->vdim) % 2 == 0 && al(a->q, pair) && al(a->pool, pair) && al(a->rope, 16) && al(a->q_norm, 8) &&
                   al(a->k_norm, 8) && (!a->k || (a->kv_ld % 2 == 0 && al(a->k, pair)));
   }
   PT_REQUIRE(a->rope_dims >= 0 && a->rope_dims % 2 == 0 && a->rope_dims <= a->dim && (!a->rope_dims || a->rope), "pt_window_attn: %d rotated dimensions of %d",
              a->rope_dims, a->dim);
   PT_REQUIRE(p.out_cols >= a->n_head * a->vdim && p.out_cols <= a->out_ld, "pt_window_attn: out_cols=%d", a->out_cols);
   p.max_len = a->max_len > 0 ? a->max_len : a->page_size * a->max_pages;
-  PT_REQUIRE(p.max_len <= a->page_size * a->max_pages, "pt_window_attn: max_len=%d exceeds the %d positions of the page table", p.max_len,
+  PT_REQUIRE(ctx || p.max_len <= a->page_size * a->max_pages, "pt_window_attn: max_len=%d exceeds the %d positions of the page table", p.max_len,
              a->page_size * a->max_pages);
   cudaStream_t st = as_stream(stream);
   // the tensor-core kernels: bf16, 64-position pages, head widths of at most 128 whose rows are whole 16-byte units
   auto al16 = [](const void *x) { return ((uintptr_t)x & 15) == 0; };
-  const bool tc = !a->plain && a->dtype == PT_DT_BF16 && a->page_size == wa::TILE && a->dim <= 128 && a->vdim <= 128 && a->dim % 8 == 0 && a->vdim % 8 == 0 &&
+  const bool gate_ok = !a->gate || (a->gate_ld % 2 == 0 && aligned_to(a->gate, 4));
+  if (ctx) {
+    PT_REQUIRE(a->dtype == PT_DT_BF16 && a->n_kv == a->n_head && !a->k && a->dim <= 256 && a->vdim <= 128 && a->dim % 8 == 0 && a->vdim % 8 == 0 && gate_ok && b.n_seq <= 65535,
+               "pt_window_attn: context rows take bf16 heads of at most 256 / 128 dimensions in steps of 8, one key head per query head, and nothing to append");
+    PT_REQUIRE(ctx->k && ctx->v && ctx->cu && ctx->shared_dim >= 0 && ctx->shared_dim <= a->dim && (!ctx->shared_dim || ctx->shared) && ctx->ld % 8 == 0 && ctx->shared_ld % 8 == 0 &&
+                   ctx->shared_dim % 8 == 0 && al16(ctx->k) && al16(ctx->v) && al16(ctx->shared) && al16(a->q) && a->q_ld % 8 == 0 && a->out_ld % 2 == 0 && aligned_to(a->out, 4),
+               "pt_window_attn: context rows in units of 16 bytes");
+    p.ctx_k = (const __nv_bfloat16 *)ctx->k; p.ctx_v = (const __nv_bfloat16 *)ctx->v; p.ctx_shared = (const __nv_bfloat16 *)ctx->shared;
+    p.ctx_ld = ctx->ld; p.shared_ld = ctx->shared_ld; p.shared_dim = ctx->shared_dim; p.ctx_cu = ctx->cu;
+  }
+  const bool tc = !a->plain && !ctx && !p.v_in_k && gate_ok && a->dtype == PT_DT_BF16 && a->page_size == wa::TILE && a->dim <= 128 && a->vdim <= 128 && a->dim % 8 == 0 && a->vdim % 8 == 0 &&
                   a->q_ld % 8 == 0 && a->out_ld % 2 == 0 && al16(a->q) && al16(a->pool) && (!a->k || (a->kv_ld % 8 == 0 && al16(a->k) && al16(a->v)));
   if (tc && b.n_tok == b.n_seq && b.n_seq <= 65535) {
     const size_t need = pt_window_attn_workspace_bytes(b.n_seq, a->n_head, a->vdim, a->page_size, p.max_len, a->window, a->keep_first);
@@ -728,15 +823,21 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
     else wa::kv_append_kernel<__nv_bfloat16><<<b.n_tok, 128, 0, st>>>(p);
     PT_LAUNCH_CHECK("pt_window_attn");
   }
+  if (ctx) return wa::dispatch_ctx(p, a->max_tokens_per_seq > 0 ? a->max_tokens_per_seq : b.n_tok, st);
   if (tc && b.n_seq <= 65535)
     return wa::dispatch_tc(p, false, a->max_tokens_per_seq > 0 ? a->max_tokens_per_seq : b.n_tok, st);
-  const size_t smem = (size_t)p.qpk * (p.dim + p.page + p.vdim + 3) * sizeof(float);
-  PT_REQUIRE(smem <= 200 * 1024, "pt_window_attn: %d query heads per kv head of widths %d / %d need %zu bytes of shared memory", p.qpk, p.dim, p.vdim, smem);
+  // heads per block: what fits 64 KB of shared memory
+  auto bytes = [&](int nh) { return (size_t)nh * (p.dim + p.page + p.vdim + 3) * sizeof(float); };
+  p.hsplit = 1;
+  while (p.hsplit < p.qpk && (p.qpk % p.hsplit || bytes(p.qpk / p.hsplit) > 64 * 1024)) ++p.hsplit;
+  const size_t smem = bytes(p.qpk / p.hsplit);
+  PT_REQUIRE(smem <= 200 * 1024, "pt_window_attn: a head of widths %d / %d needs %zu bytes of shared memory", p.dim, p.vdim, smem);
   if (smem > 48 * 1024) {
     PT_CUDA(cudaFuncSetAttribute(wa::attn_plain_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     PT_CUDA(cudaFuncSetAttribute(wa::attn_plain_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
   }
-  const dim3 grid(b.n_tok, a->n_kv);
+  PT_REQUIRE(a->n_kv * p.hsplit <= 65535, "pt_window_attn: %d heads", a->n_head);
+  const dim3 grid(b.n_tok, a->n_kv * p.hsplit);
   if (a->dtype == PT_DT_F32) wa::attn_plain_kernel<float><<<grid, wa::PLAIN_THREADS, smem, st>>>(p);
   else wa::attn_plain_kernel<__nv_bfloat16><<<grid, wa::PLAIN_THREADS, smem, st>>>(p);
   PT_LAUNCH_CHECK("pt_window_attn");

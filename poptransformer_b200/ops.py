@@ -20,13 +20,15 @@ import ctypes
 import torch
 
 from . import _lib
-from ._lib import (AttnArgs, BatchView, DenseExt, GemmArgs, HyperArgs, LinearArgs, MlstmArgs, MoeRouteArgs, PostNormArgs, PtError, SsmArgs,
-                   WindowAttnArgs, check)
+from ._lib import (AttnArgs, BatchView, ContextRows, DenseExt, GemmArgs, HyperArgs, LatentAttnArgs, LatentContextArgs, LatentPrepArgs, LinearArgs, MlstmArgs,
+                   MoeRouteArgs, PostNormArgs, PtError, SsmArgs, WindowAttnArgs, check)
 
 W_INT4, W_FP16, W_FP8, W_BF16 = 0, 1, 2, 3
 DT_F16, DT_F32, DT_BF16 = 0, 1, 2
 PRO_NONE, PRO_RMSNORM, PRO_CAST_FP8, PRO_RMSNORM_CAST_FP8, PRO_NORMCE = 0, 1, 2, 3, 4
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL, EPI_RELU2, EPI_GLU, EPI_GELU_MUL = 0, 1, 2, 3, 4, 5, 6, 7, 8
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL, EPI_RELU2, EPI_GLU, EPI_GELU_MUL, EPI_SOFTCAP = range(10)
+GLU_CLAMPED, GLU_SILU, GLU_GELU = 0, 1, 2
+MOE_SOFTMAX, MOE_SIGMOID = 0, 1
 ROPE_NONE, ROPE_LLAMA, ROPE_CHATGLM2 = 0, 1, 2
 SOFTMAX_F32, SOFTMAX_F16 = 0, 1
 
@@ -218,12 +220,13 @@ class DenseLinear:
     # Up to a million weights (128 x 2048, 2048 x 128, 1024 x 1024) the skinny kernel takes 0.6 - 0.75 of the GEMM's time at 8 and 16 rows.
     SKINNY_ROWS, SMALL_ROWS, SMALL_SIZE = 7, 16, 1 << 20
 
-    def __init__(self, w, dtype, pad_rows=0, keep=False, bias=None, split=None, limit=0.0):
+    def __init__(self, w, dtype, pad_rows=0, keep=False, bias=None, split=None, limit=0.0, glu=GLU_CLAMPED):
         """pad_rows: zero rows are appended up to this many outputs (an output that is the padded input of the next linear).
         keep: keep the padded matrix itself as `w` (a table that also serves look-ups).  bias: fp32 [n_out].  split: outputs from this
-        row on (a multiple of 32) go to a second, fp32 output and skip the epilogue.  limit: of a gated epilogue (rows as glu_rows)."""
+        row on (a multiple of 32) go to a second, fp32 output and skip the epilogue.  limit, glu: of a gated epilogue (rows as glu_rows);
+        limit also of the softcap."""
         self.dtype, self.n_out, self.k_in = dtype, w.shape[0], w.shape[1]
-        self.split, self.limit = split, float(limit)
+        self.split, self.limit, self.glu = split, float(limit), glu
         self.ld = pad_to(self.k_in, self.K_PAD) if dtype == torch.bfloat16 else self.k_in
         if self.ld != self.k_in or pad_rows > self.n_out:
             full = torch.zeros((max(pad_rows, self.n_out), self.ld), dtype=w.dtype, device=w.device)
@@ -248,12 +251,13 @@ class DenseLinear:
         """Algorithmic bytes of one launch: the weights once."""
         return self.n_out * self.k_in * (2 if self.dtype == torch.bfloat16 else 4)
 
-    def _ext(self, out2, out2_ld, mul, mul_ids):
+    def _ext(self, out2, out2_ld, mul, mul_ids, bias):
         """mul: (a table of the output's type, its row stride, its first column)."""
-        if self.bias is None and self.split is None and mul is None and not self.limit:
+        bias = self.bias if bias is None else bias
+        if bias is None and self.split is None and mul is None and not self.limit and self.glu == GLU_CLAMPED:
             return None
         e = DenseExt()
-        e.bias, e.limit = _ptr(self.bias), self.limit
+        e.bias, e.limit, e.glu = _ptr(bias), self.limit, self.glu
         if self.split is not None:
             e.out2, e.out2_ld, e.split_n = _ptr(out2), out2_ld, self.split
         if mul is not None:
@@ -262,12 +266,12 @@ class DenseLinear:
         return e
 
     def __call__(self, x, out, rows, out_ld, epilogue=EPI_STORE, alpha=1.0, linear_ws=None, gemm_ws=None, error_flag=None, out2=None, out2_ld=0, mul=None,
-                 mul_ids=None, pdl=0):
+                 mul_ids=None, pdl=0, bias=None):
         """out[:rows, :n_out] = epilogue(alpha * x[:rows] @ W^T + bias); x and out are flat or 2-D buffers of row strides `ld` and
-        `out_ld`.  pdl: programmatic dependent launch behind the kernel before it in the stream (bfloat16)."""
+        `out_ld`.  bias: fp32 [n_out] in place of the linear's own.  pdl: programmatic dependent launch behind the kernel before it in the stream (bfloat16)."""
         x = x.reshape(-1)[:rows * self.ld].view(rows, self.ld)
         L = _lib.lib()
-        ext = self._ext(out2, out2_ld, mul, mul_ids)
+        ext = self._ext(out2, out2_ld, mul, mul_ids, bias)
         if self.dtype == torch.float32:
             check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, float(alpha), epilogue, _ptr(out), out_ld,
                                 ctypes.byref(ext) if ext else None, _stream()), "pt_gemm_f32")
@@ -282,9 +286,10 @@ class GroupedLinear:
     """Matrices [n_out, k] of one shape (experts), one after the other in a buffer: every tile of activation rows is multiplied with
     the matrix that `group_of` names for it.  bfloat16: tiles of one row on the skinny-matmul kernel, tiles of 16 .. 256 rows on the
     tcgen05 GEMM; float32: tiles of 64 rows."""
+    skinny_rows = DenseLinear.SKINNY_ROWS
 
-    def __init__(self, ws, dtype, pad_rows=0, limit=0.0):
-        self.dtype, self.groups, self.k_in, self.limit = dtype, len(ws), ws[0].shape[1], float(limit)
+    def __init__(self, ws, dtype, pad_rows=0, limit=0.0, glu=GLU_CLAMPED):
+        self.dtype, self.groups, self.k_in, self.limit, self.glu = dtype, len(ws), ws[0].shape[1], float(limit), glu
         self.n_out = max(pad_rows, ws[0].shape[0])
         self.ld = pad_to(self.k_in, DenseLinear.K_PAD) if dtype == torch.bfloat16 else self.k_in
         L = _lib.lib()
@@ -311,12 +316,14 @@ class GroupedLinear:
         """Bytes of one matrix."""
         return self.n_out * self.k_in * (2 if self.dtype == torch.bfloat16 else 4)
 
-    def __call__(self, x, out, rows, out_ld, tile, group_of, used=None, x_div=1, epilogue=EPI_STORE, linear_ws=None, gemm_ws=None, error_flag=None, pdl=0):
+    def __call__(self, x, out, rows, out_ld, tile, group_of, used=None, x_div=1, epilogue=EPI_STORE, linear_ws=None, gemm_ws=None, error_flag=None, pdl=0,
+                 row_scale=None):
         """out[:rows] = epilogue(x rows @ matrix^T).  tile: rows per entry of group_of; with tile 1 row r reads x row r // x_div.
-        used: rows of every tile that matter (the GEMM leaves the others out)."""
+        used: rows of every tile that matter (the GEMM leaves the others out).  row_scale: fp32, a factor on every row's sums."""
         L = _lib.lib()
         e = DenseExt()
         e.limit, e.n_groups, e.group_rows, e.group_x_div, e.group_of, e.group_used = self.limit, self.groups, tile, x_div, _ptr(group_of), _ptr(used)
+        e.glu, e.row_scale = self.glu, _ptr(row_scale)
         if self.dtype == torch.float32:
             check(L.pt_gemm_f32(_ptr(x), self.ld, _ptr(self.w), self.ld, rows, self.n_out, self.k_in, 1.0, epilogue, _ptr(out), out_ld, ctypes.byref(e), _stream()),
                   "pt_gemm_f32")
@@ -369,10 +376,12 @@ def window_attn_workspace(n_seq, n_head, vdim, page_size, max_len, window, keep_
 
 def window_attn(view, qkv, qkv_ld, cache, out, out_ld, n_head, scale, window=0, keep_first=0, sink=None, append=True, max_tokens_per_seq=0,
                 workspace=None, error_flag=None, plain=False, values_are_keys=False, q_norm=None, k_norm=None, eps=0.0, rope=None, rope_dims=0, out_scale=1.0,
-                out_cols=0):
+                out_cols=0, softcap=0.0, gate=None, gate_ld=0, gate_per_head=False, context=None):
     """Masked attention of the packed tokens of `view` over a paged cache (see pt_window_attn).  qkv rows hold [q | k | v]
     (append=True: k and v go to the cache first), [q | k] (values_are_keys: the keys as they are in the row are the values) or only q
-    (a layer that reads another layer's cache).  q_norm, k_norm, rope: per-head norm and rotation of q and k; q is then rewritten."""
+    (a layer that reads another layer's cache).  q_norm, k_norm, rope: per-head norm and rotation of q and k; q is then rewritten.  gate: rows
+    whose sigmoid multiplies the output (a view that starts at its first column).  context: an object with k, v, shared, ld, shared_dim
+    and cu that names rows of the whole context as keys and values of a prompt, in place of the cache's pages (see pt_context_rows)."""
     a = WindowAttnArgs()
     a.batch, a.dtype = view, dtype_code(qkv.dtype)
     a.n_head, a.n_kv, a.dim, a.vdim = n_head, cache.n_kv, cache.head_dim, cache.v_dim
@@ -384,11 +393,55 @@ def window_attn(view, qkv, qkv_ld, cache, out, out_ld, n_head, scale, window=0, 
         a.k, a.v = k, k if values_are_keys else k + cache.n_kv * cache.head_dim * qkv.element_size()
     a.q_norm, a.k_norm, a.norm_eps, a.rope, a.rope_dims = _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(rope), rope_dims
     a.out_scale, a.out_cols = float(out_scale), out_cols
+    a.softcap, a.gate, a.gate_ld, a.gate_per_head = float(softcap), gate.data_ptr() if gate is not None else None, gate_ld, 1 if gate_per_head else 0
+    if context is not None:
+        c = ContextRows()
+        c.k, c.v, c.shared, c.ld, c.shared_ld, c.shared_dim, c.cu = context.k.data_ptr(), context.v.data_ptr(), context.shared.data_ptr(), context.ld, context.shared_dim, context.shared_dim, _ptr(context.cu)
+        a.n_kv, a.dim, a.vdim, a.context = n_head, context.dim, context.vdim, ctypes.pointer(c)
     a.pool, a.page_table, a.out, a.out_ld = _ptr(cache.pool), _ptr(cache.page_table), _ptr(out), out_ld
     a.max_tokens_per_seq, a.plain = max_tokens_per_seq, 1 if plain else 0
     a.workspace, a.workspace_bytes = _ptr(workspace), workspace.numel() if workspace is not None else 0
     a.error_flag = _ptr(error_flag)
     check(_lib.lib().pt_window_attn(ctypes.byref(a), _stream()), "pt_window_attn")
+
+
+def latent_prep(view, rows, ld, q_col, kv_col, w, cq, cq_ld, cache, eps, rope, error_flag=None):
+    """Norms of both latents, rotation of the shared key part, append (see pt_latent_prep).  q_col, kv_col: first columns of the query latent
+    and of [latent | key part] in `rows`; w: an object with q_rank, rank, rot_dim and the fp32 tensors q_norm, kv_norm."""
+    a = LatentPrepArgs()
+    es = rows.element_size()
+    a.batch, a.dtype, a.q_rank, a.rank, a.rot_dim, a.eps = view, dtype_code(rows.dtype), w.q_rank, w.rank, w.rot_dim, float(eps)
+    a.q, a.kv, a.ld = rows.data_ptr() + q_col * es, rows.data_ptr() + kv_col * es, ld
+    a.q_norm, a.kv_norm, a.rope, a.cq, a.cq_ld = _ptr(w.q_norm), _ptr(w.kv_norm), _ptr(rope), _ptr(cq), cq_ld
+    a.pool, a.page_table, a.page_size, a.max_pages, a.max_len = _ptr(cache.pool), _ptr(cache.page_table), cache.page_size, cache.page_table.shape[1], cache.max_len
+    a.error_flag = _ptr(error_flag)
+    check(_lib.lib().pt_latent_prep(ctypes.byref(a), _stream()), "pt_latent_prep")
+
+
+def latent_context(view, ctx_cu, n_ctx, w, cache, shared, latent, latent_ld):
+    """The cached rows of every sequence's context, one after the other (see pt_latent_context)."""
+    a = LatentContextArgs()
+    a.batch, a.ctx_cu, a.n_ctx, a.rot_dim, a.rank = view, _ptr(ctx_cu), n_ctx, w.rot_dim, w.rank
+    a.page_size, a.max_pages, a.pool, a.page_table = cache.page_size, cache.page_table.shape[1], _ptr(cache.pool), _ptr(cache.page_table)
+    a.shared, a.latent, a.latent_ld = _ptr(shared), _ptr(latent), latent_ld
+    check(_lib.lib().pt_latent_context(ctypes.byref(a), _stream()), "pt_latent_context")
+
+
+def latent_workspace_bytes(n_tok, w, dtype):
+    return _lib.lib().pt_latent_attn_workspace_bytes(n_tok, w.heads, w.rot_dim, w.rank, dtype_code(dtype))
+
+
+def latent_attn(view, q, q_ld, w, cache, out, out_ld, scale, rope, workspace, gate=None, gate_ld=0, out_cols=0, error_flag=None, plain=False):
+    """Attention over the cached latents (see pt_latent_attn).  w: an object with heads, dim, rot_dim, vdim, rank and the tensors w_k [heads,
+    rank, dim] and w_v [heads, vdim, rank].  gate: a view that starts at the heads' gates."""
+    a = LatentAttnArgs()
+    a.batch, a.dtype, a.n_head, a.dim, a.rot_dim, a.vdim, a.rank, a.scale = view, dtype_code(q.dtype), w.heads, w.dim, w.rot_dim, w.vdim, w.rank, float(scale)
+    a.q, a.q_ld, a.rope, a.w_k, a.w_v = _ptr(q), q_ld, _ptr(rope), _ptr(w.w_k), _ptr(w.w_v)
+    a.gate, a.gate_ld = gate.data_ptr() if gate is not None else None, gate_ld
+    a.pool, a.page_table, a.page_size, a.max_pages, a.max_len = _ptr(cache.pool), _ptr(cache.page_table), cache.page_size, cache.page_table.shape[1], cache.max_len
+    a.out, a.out_ld, a.out_cols, a.plain, a.error_flag = _ptr(out), out_ld, out_cols, 1 if plain else 0, _ptr(error_flag)
+    a.workspace, a.workspace_bytes = _ptr(workspace), workspace.numel()
+    check(_lib.lib().pt_latent_attn(ctypes.byref(a), _stream()), "pt_latent_attn")
 
 
 def ssm(view, zx, zx_ld, out, out_ld, w, ring, state, y, xbc=None, dt=None, workspace=None, plain=False):
@@ -422,8 +475,10 @@ def mlstm(view, rows, ld, cols, gates, gate_ld, out, out_ld, w, state, nm, y, wo
 
 
 def post_norm(rows, width, eps, dtype, x_in=None, x_out=None, y=None, y_ld=0, pair_y=None, pair_ld=0, top=0, pair_w=None, pair_row=None, norm_w=None,
-              final_w=None, h=None, h_ld=0, row_index=None, table=None, vocab=0, ids=None, ids_ld=1, step=None, pos_out=None, id_out=None):
-    """Residual step with a norm on the sublayer's output (see pt_post_norm), or the start of a token from an embedding table."""
+              final_w=None, h=None, h_ld=0, row_index=None, table=None, vocab=0, ids=None, ids_ld=1, step=None, pos_out=None, id_out=None, h_cols=0,
+              copy=None, copy_ld=0, copy_cols=0):
+    """Residual step with a norm on the sublayer's output, on the next one's input or both (see pt_post_norm), or the start of a token
+    from an embedding table.  copy: a view that starts at the first column of the second copy."""
     a = PostNormArgs()
     a.rows, a.width, a.dtype, a.eps, a.x_in, a.x_out = rows, width, dtype_code(dtype), float(eps), _ptr(x_in), _ptr(x_out)
     if table is not None:
@@ -433,7 +488,8 @@ def post_norm(rows, width, eps, dtype, x_in=None, x_out=None, y=None, y_ld=0, pa
     if pair_y is not None:
         a.pair_dtype = dtype_code(pair_y.dtype)
     a.pair_y, a.pair_ld, a.top, a.pair_w, a.pair_row = _ptr(pair_y), pair_ld, top, _ptr(pair_w), _ptr(pair_row)
-    a.norm_w, a.final_w, a.h, a.h_ld = _ptr(norm_w), _ptr(final_w), _ptr(h), h_ld
+    a.norm_w, a.final_w, a.h, a.h_ld, a.h_cols = _ptr(norm_w), _ptr(final_w), _ptr(h), h_ld, h_cols
+    a.copy, a.copy_ld, a.copy_cols = copy.data_ptr() if copy is not None else None, copy_ld, copy_cols
     check(_lib.lib().pt_post_norm(ctypes.byref(a), _stream()), "pt_post_norm")
 
 
@@ -441,11 +497,12 @@ def moe_max_tiles(n_tok, experts, top, tile):
     return int(_lib.lib().pt_moe_max_tiles(n_tok, experts, top, tile))
 
 
-def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, tile_rows=None, row_token=None, counts=None, h=None, h_ld=0, gathered=None):
+def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, tile_rows=None, row_token=None, counts=None, h=None, h_ld=0, gathered=None,
+              score=MOE_SOFTMAX, row_weight=None):
     """Experts and weights of every token, and with `tile` the rows of the grouped products (see pt_moe_route)."""
     a = MoeRouteArgs()
     a.n_tok, a.experts, a.top, a.logits, a.logits_ld = n_tok, experts, top, _ptr(logits), logits.shape[-1]
-    a.expert, a.weight, a.tile = _ptr(expert), _ptr(weight), tile
+    a.expert, a.weight, a.tile, a.score, a.row_weight = _ptr(expert), _ptr(weight), tile, score, _ptr(row_weight)
     if tile:
         a.max_tiles = moe_max_tiles(n_tok, experts, top, tile)
         a.pair_row, a.tile_expert, a.tile_rows, a.row_token = _ptr(pair_row), _ptr(tile_expert), _ptr(tile_rows), _ptr(row_token)

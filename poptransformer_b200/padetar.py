@@ -23,6 +23,7 @@ import numpy as np
 import torch
 
 from . import ops
+from .experts import Experts
 from .sequences import SequenceDecoder
 
 
@@ -127,7 +128,7 @@ class PadetarDecoder(SequenceDecoder):
             # ---- experts
             if lay.moe:
                 m, M = lay.moe, p + "mlp."
-                sub = SimpleNamespace(kind="moe", layer=i, m=m, norm=f32(p + "norm2", (W,)), sff=ops.pad_to(m.shared_ff, pad), ff=ops.pad_to(m.ff, pad), down=None)
+                sub = SimpleNamespace(kind="moe", layer=i, m=m, norm=f32(p + "norm2", (W,)), sff=ops.pad_to(m.shared_ff, pad), down=None)
                 rows = []
                 if m.shared_ff:
                     rows.append(ops.glu_rows(*(mat(M + "shared." + n, (m.shared_ff, W)) for n in ("gate", "up")), sub.sff))
@@ -136,8 +137,8 @@ class PadetarDecoder(SequenceDecoder):
                 bias = torch.zeros(split + m.experts, dtype=torch.float32, device=self.device)
                 bias[split:] = f32(M + "router.b", (m.experts,))
                 sub.proj = ops.DenseLinear(torch.cat(rows + [mat(M + "router", (m.experts, W))], 0), dt, bias=bias, split=split, limit=m.shared_limit)
-                sub.up = ops.GroupedLinear([ops.glu_rows(*(mat(M + f"e{e}." + n, (m.ff, W)) for n in ("gate", "up")), sub.ff) for e in range(m.experts)], dt, limit=m.limit)
-                sub.back = ops.GroupedLinear([down(M + f"e{e}.down", m.ff) for e in range(m.experts)], dt)
+                gates, ups = ([mat(M + f"e{e}." + n, (m.ff, W)) for e in range(m.experts)] for n in ("gate", "up"))
+                sub.experts = Experts(dt, m.top, gates, ups, [mat(M + f"e{e}.down", (W, m.ff)) for e in range(m.experts)], limit=m.limit)
                 self.subs.append(sub)
             # ---- side input
             if c.side:
@@ -159,7 +160,7 @@ class PadetarDecoder(SequenceDecoder):
         """Algorithmic weight bytes one decode step of `rows` tokens streams: every linear once, of the experts as many as the rows
         can choose at most."""
         moe = [s for s in self.subs if s.kind == "moe"]
-        return sum(x.nbytes for x in self._linears()) + sum(min(s.m.experts, rows * s.m.top) * (s.up.nbytes + s.back.nbytes) for s in moe)
+        return sum(x.nbytes for x in self._linears()) + sum(s.experts.step_bytes(rows) for s in moe)
 
     # ---- state ----------------------------------------------------------------------------------
     def _alloc_layers(self):
@@ -171,17 +172,6 @@ class PadetarDecoder(SequenceDecoder):
             self.caches[i] = ops.PagedKVCache(B, a.kv_heads, a.dim, c.max_len, page_size, dev, self.slots.page_table, dtype=self.dtype, n_pages=self.slots.n_pages)
             self.states[i], self.norms[i] = (torch.zeros((B, L.pt_mlstm_state_floats(b.heads, b.dim, b.vdim, k)), dtype=torch.float32, device=dev) for k in (0, 1))
         self.attn_ws = self._attn_workspace([(lay.left.heads, lay.left.dim, 0, 0) for lay in c.layers])
-
-    def _moe_tile(self, n, m):
-        """Rows of a tile of the grouped products for n tokens: 1 for the skinny-matmul kernel, else about an expert's share."""
-        if self.dtype == torch.float32:
-            return 64
-        if n <= ops.DenseLinear.SKINNY_ROWS:
-            return 1
-        share, tile = n * m.top / m.experts, 16
-        while tile < 128 and tile < share:
-            tile *= 2
-        return tile
 
     def _row_buffers(self, rows):
         c, dev, dt = self.cfg, self.device, self.dtype
@@ -204,20 +194,7 @@ class PadetarDecoder(SequenceDecoder):
         n = max(L.pt_mlstm_workspace_bytes(rows + 1, min(self.batch, rows), s.mem.heads, s.mem.dim, s.mem.vdim) for s in mixers)
         r.mem_ws = torch.zeros(n, dtype=torch.uint8, device=dev)
         if moes:
-            top = max(s.m.top for s in moes)
-            padded = [self._moe_tile(rows, s.m) * ops.moe_max_tiles(rows, s.m.experts, s.m.top, self._moe_tile(rows, s.m)) for s in moes]
-            r.logits = torch.empty(rows * max(s.m.experts for s in moes), **f32)
-            r.expert, r.pair_row, r.weight = torch.empty(rows * top, **i32), torch.empty(rows * top, **i32), torch.empty(rows * top, **f32)
-            r.tile_expert, r.tile_rows, r.row_token = (torch.empty(max(padded), **i32) for _ in range(3))
-            r.counts = torch.empty(max(s.m.experts for s in moes), **i32)
-            r.gathered = torch.empty(max(padded) * self.h_ld, dtype=dt, device=dev)
-            r.act = torch.empty(max(p * s.ff for p, s in zip(padded, moes)), dtype=dt, device=dev)
-            r.pair_y = torch.empty((max(padded), c.width), dtype=dt, device=dev)
-            if r.lin_ws is not None:
-                pairs = min(rows, ops.DenseLinear.SKINNY_ROWS) * top
-                n = max(L.pt_linear_workspace_bytes(pairs, x.n_out, 4) for s in moes for x in (s.up, s.back))
-                if n > r.lin_ws.numel():
-                    r.lin_ws = torch.zeros(n, dtype=torch.uint8, device=dev)
+            Experts.buffers(r, rows, [s.experts for s in moes], self.h_ld, dev)
         return r
 
     # ---- the layers -----------------------------------------------------------------------------
@@ -240,21 +217,10 @@ class PadetarDecoder(SequenceDecoder):
         if s.down:
             with self._beside():
                 self._linear(s.down, r.a, r.y, n, W, r.beside)
-        tile = self._moe_tile(n, m)
-        logits = r.logits[:n * m.experts].view(n, m.experts)
-        ws = dict(linear_ws=r.lin_ws, gemm_ws=r.gemm_ws, error_flag=self.error_flag, pdl=1)
-        if tile == 1:
-            ops.moe_route(logits, n, m.experts, m.top, r.expert, r.weight)
-            s.up(r.h, r.act, n * m.top, s.ff, 1, r.expert, x_div=m.top, epilogue=ops.EPI_GLU, **ws)
-            s.back(r.act, r.pair_y, n * m.top, W, 1, r.expert, **ws)
-        else:
-            rows = tile * ops.moe_max_tiles(n, m.experts, m.top, tile)
-            ops.moe_route(logits, n, m.experts, m.top, r.expert, r.weight, tile, r.pair_row, r.tile_expert, r.tile_rows, r.row_token, r.counts, r.h, self.h_ld, r.gathered)
-            s.up(r.gathered, r.act, rows, s.ff, tile, r.tile_expert, r.tile_rows, epilogue=ops.EPI_GLU, **ws)
-            s.back(r.act, r.pair_y, rows, W, tile, r.tile_expert, r.tile_rows, **ws)
+        pairs = s.experts(r, n, self.h_ld, self.error_flag)
         if s.down:
             self._join()
-        return dict(y=r.y if s.down else None, y_ld=W, pair_y=r.pair_y, pair_ld=W, top=m.top, pair_w=r.weight, pair_row=None if tile == 1 else r.pair_row)
+        return dict(y=r.y if s.down else None, y_ld=W, **pairs)
 
     def _side(self, s, r, view, longest):
         n, W = view.n_tok, self.cfg.width

@@ -46,6 +46,11 @@ def _padetar(c, sd, batch, max_len, dtype, **kw):
     return PadetarDecoder(PadetarConfig(c, max_len), sd, batch, dtype=dtype, **kw)
 
 
+def _pivavik(c, sd, batch, max_len, dtype, **kw):
+    from .pivavik import PivavikConfig, PivavikDecoder
+    return PivavikDecoder(PivavikConfig(c, max_len), sd, batch, dtype=dtype, **kw)
+
+
 # name -> (builder, dtypes the decoder runs in; the first is the default)
 ARCHITECTURES = {
     "LlamaForCausalLM": (_llama, ("float16",)),
@@ -55,6 +60,7 @@ ARCHITECTURES = {
     "RwkvForCausalLM": (_rwkv, ("float16",)),
     "Sabisun": (_sabisun, ("bfloat16", "float32")),
     "Padetar": (_padetar, ("bfloat16", "float32")),
+    "Pivavik": (_pivavik, ("bfloat16", "float32")),
 }
 
 

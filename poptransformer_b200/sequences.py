@@ -259,15 +259,16 @@ class SequenceDecoder(DecodeLoop):
         cu = np.concatenate([[0], np.cumsum(lens)]).astype(np.int32)
         rows = [cu[s] + w for s, (_, _, _, want) in enumerate(part) for w, _ in want]
         dest = [o for _, _, _, want in part for _, o in want]
+        ctx = np.concatenate([[0], np.cumsum([s + n for (_, _, s, _), n in zip(part, lens)])])      # all positions so far, sequence after sequence
         fields = [np.concatenate([t for _, t, _, _ in part]), np.repeat(np.arange(n_seq), lens), cu, [s for _, _, s, _ in part], [s for s, _, _, _ in part],
-                  rows, dest]
+                  rows, dest, ctx]
         sizes = [ops.pad_to(len(f), 4) for f in fields]              # every array on a 16-byte boundary of one upload
         host = np.zeros(sum(sizes), dtype=np.int32)
         at = np.concatenate([[0], np.cumsum(sizes)])
         for f, a in zip(fields, at):
             host[a:a + len(f)] = f
         dev = torch.from_numpy(host).to(self.device)
-        ids, tok_seq, cu_d, start, slot, rows_d, dest_d = (dev[a:a + len(f)] for f, a in zip(fields, at))
+        ids, tok_seq, cu_d, start, slot, rows_d, dest_d, ctx_d = (dev[a:a + len(f)] for f, a in zip(fields, at))
         if n <= self.rows_decode.rows:
             r = self.rows_decode
         else:
@@ -275,7 +276,9 @@ class SequenceDecoder(DecodeLoop):
                 self.rows_prompt = None
                 self.rows_prompt = self._row_buffers(n)
             r = self.rows_prompt
-        self._layers(r, ops.batch_view(n_seq, n, cu_d, start, slot, tok_seq), max(lens), ids, layer_sums=layer_sums)
+        view = ops.batch_view(n_seq, n, cu_d, start, slot, tok_seq)
+        view.ctx_cu, view.n_ctx = ctx_d, int(ctx[-1])
+        self._layers(r, view, max(lens), ids, layer_sums=layer_sums)
         k = len(rows)
         logits = torch.empty((k, self.cfg.vocab), dtype=torch.float32, device=self.device) if k else None
         self._head(r, k, logits, row_index=rows_d if k else None, layer_sums=layer_sums, n_tok=n)
