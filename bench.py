@@ -626,6 +626,16 @@ def expert_config(width, n_layer, heads, kv_heads, dim, mem_heads, mem_dim, mem_
             "layers": [{"type": "parallel", "mixer": {"left": left, "left_scale": 1.0, "right": right, "right_scale": 1.0}, "mlp": mlp} for _ in range(n_layer)]}
 
 
+def latent_config(width, n_layer, loop, heads, kv_heads, dim, rot, kv_rank, q_rank, window, softcap, experts, top, ff, dense_ff, vocab):
+    """A Pivavik of real-model layer sizes: latent and windowed attention in turn, the first layer with a dense feed-forward."""
+    lat = {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "kv_rank": kv_rank, "q_rank": q_rank, "rot": {"base": 1e4, "dims": rot},
+                                                 "scale": (dim + rot) ** -0.5}}
+    win = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": softcap, "mask": {"size": window}}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}}
+    return {"architecture": "Pivavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "loop": dict(zip(("start", "stop", "times"), loop)),
+            "layers": [dict(win if i % 2 else lat, mlp=moe if i else {"kind": "dense", "ff": dense_ff}) for i in range(n_layer)]}
+
+
 EXPERTS = {   # name: configuration, then the Sabisun of equal width, depth and vocabulary whose feed-forward has as many weights as a token uses here
     "padetar-2k": (dict(width=2048, n_layer=16, heads=16, kv_heads=4, dim=128, mem_heads=16, mem_dim=128, mem_vdim=128, experts=32, top=4, ff=1024, shared_ff=2048,
                         side=128, vocab=32000),
@@ -635,6 +645,12 @@ EXPERTS = {   # name: configuration, then the Sabisun of equal width, depth and 
                         side=256, vocab=32000),
                    dict(width=4096, n_layer=8, ff=15360, heads=32, kv_heads=8, dim=128, ssm_heads=128, ssm_dim=64, state=128, groups=8, vocab=32000, window=1024,
                         keep_first=64, streams=4)),
+}
+LATENT = {    # name: configuration, then the Padetar of equal width, vocabulary, heads and experts with as many layers as run here
+    "pivavik-2k": (dict(width=2048, n_layer=10, loop=(2, 8, 2), heads=16, kv_heads=4, dim=128, rot=64, kv_rank=512, q_rank=768, window=1024, softcap=50.0, experts=32, top=4, ff=1024,
+                        dense_ff=6144, vocab=32000), EXPERTS["padetar-2k"][0]),
+    "pivavik-4k": (dict(width=4096, n_layer=6, loop=(2, 4, 2), heads=32, kv_heads=8, dim=128, rot=64, kv_rank=512, q_rank=1536, window=1024, softcap=50.0, experts=32, top=4, ff=1536,
+                        dense_ff=12288, vocab=32000), EXPERTS["padetar-4k"][0]),
 }
 
 
@@ -765,45 +781,61 @@ def run_hybrid(args):
                       "llama_int4_prompt_pass": {"sequences": 1, "prompt": prompt, "ms": lms, "tokens_per_s": prompt / lms * 1e3, "linear_tflops": lflops / lms / 1e9}}))
 
 
-def run_experts(args):
-    """Decode and prompt throughput of a Padetar beside the Sabisun of equal size.  One JSON line, marked `secondary`."""
+def padetar_state_bytes(dims, ctx):
+    """Recurrent state (read and written) and keys of one row and step."""
+    return dims["n_layer"] * (2 * 4 * dims["mem_heads"] * dims["mem_dim"] * dims["mem_vdim"] + 2 * 2 * dims["kv_heads"] * dims["dim"] * ctx)
+
+
+def pivavik_state_bytes(dims, ctx):
+    """Cached latents, and visible keys and values, of one row and step."""
+    start, stop, times = dims["loop"]
+    runs = list(range(start)) + list(range(start, stop)) * times + list(range(stop, dims["n_layer"]))
+    return sum(2 * 2 * dims["kv_heads"] * dims["dim"] * min(ctx, dims["window"]) if i % 2 else 2 * (dims["rot"] + dims["kv_rank"]) * ctx for i in runs)
+
+
+def run_beside(args):
+    """Decode and prompt throughput of an architecture beside its closest one of equal size.  One JSON line, marked `secondary`."""
     import torch
     from poptransformer_b200 import registry, synth
     if not torch.cuda.is_available():
         raise SystemExit("bench.py needs a CUDA device (there is no CPU fallback)")
-    dims, sdims = EXPERTS[args.workload]
+    mine, other, table, what = ("pivavik", "padetar", LATENT, "a decoder with latent attention, experts and looped layers") if args.workload in LATENT else \
+        ("padetar", "sabisun", EXPERTS, "a decoder with experts and a matrix memory")
+    make = {"pivavik": (latent_config, synth.pivavik_state_dict, pivavik_state_bytes), "padetar": (expert_config, synth.padetar_state_dict, padetar_state_bytes),
+            "sabisun": (hybrid_config, synth.sabisun_state_dict, None)}
+    dims, odims = table[args.workload]
     dev = torch.device("cuda", 0)
     ctx, prompt, K = 2048, 2048, max(8, min(args.steps, 64))
     max_len = ctx + K + 16
     peak, _ = peaks()
     sampler = ClockSampler(0)
     sampler.start()
-    E, top, n_layer = dims["experts"], dims["top"], dims["n_layer"]
     res = {}
-    for name, cfg, make in (("padetar", expert_config(**dims), synth.padetar_state_dict), ("sabisun", hybrid_config(**sdims), synth.sabisun_state_dict)):
-        sd = make(cfg, device=dev)
+    for name, d in ((mine, dims), (other, odims)):
+        config, weights, state_bytes = make[name]
+        cfg = config(**d)
+        sd = weights(cfg, device=dev)
         rows, pre = [], []
         for batch in (1, 8, 32):
             dec = sequence_decoder(cfg, sd, batch, max_len, ctx)
             ms = time_decode(dec, ctx, K)
-            if name == "padetar":
-                # every linear once, and the experts that `batch` independent choices are expected to hit
-                hit = E * (1.0 - (1.0 - top / E) ** batch)
-                moe = [s for s in dec.subs if s.kind == "moe"]
-                weights = sum(x.nbytes for x in dec._linears()) + sum(hit * (s.experts.up.nbytes + s.experts.back.nbytes) for s in moe)
-                state = n_layer * (2 * 4 * dims["mem_heads"] * dims["mem_dim"] * dims["mem_vdim"] + 2 * 2 * dims["kv_heads"] * dims["dim"] * ctx)
+            if name == "sabisun":
+                need = dec.weight_bytes() + batch * sabisun_state_bytes(cfg)
             else:
-                weights, state = dec.weight_bytes(), sabisun_state_bytes(cfg)
-            need = weights + batch * state
+                # every linear once, and the experts that `batch` independent choices are expected to hit
+                hit = d["experts"] * (1.0 - (1.0 - d["top"] / d["experts"]) ** batch)
+                need = dec.fixed_bytes() + sum(hit * (e.up.nbytes + e.back.nbytes) for e in dec.expert_groups()) + batch * state_bytes(d, ctx)
             rows.append({"batch": batch, "decode_ms": ms, "decode_tokens_per_s": batch / ms * 1e3, "bytes_per_step": int(need), "decode_frac_of_measured": need / ms / 1e6 / peak})
             del dec
             torch.cuda.empty_cache()
         dec = registry.build_decoder(cfg, sd, 4, max_len, "bfloat16", pad_id=-1)
         size = lambda x: x.n_out * x.k_in
-        if name == "padetar":
-            flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(top * (size(s.experts.up) + size(s.experts.back)) for s in dec.subs if s.kind == "moe"))
-        else:
+        if name == "sabisun":
             flops = 2 * prompt * sum(size(s.proj) + size(s.out) for s in dec.subs)
+        else:
+            flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(e.top * (size(e.up) + size(e.back)) for e in dec.expert_groups()))
+            if name == "pivavik":
+                flops += 2 * prompt * sum(size(r.sub.up) for r in dec.runs if r.sub.lay.kind == "latent_attention")
         for n_seq in (1, 4):
             best = time_prompts(dec, cfg["vocab"], n_seq, prompt)
             pre.append({"sequences": n_seq, "prompt": prompt, "ms": best, "tokens_per_s": n_seq * prompt / best * 1e3, "linear_tflops": n_seq * flops / best / 1e9})
@@ -811,13 +843,13 @@ def run_experts(args):
         del dec, sd
         torch.cuda.empty_cache()
     clocks = sampler.stop()
-    last = res["padetar"]["decode"][-1]
-    print(json.dumps({"secondary": "not the headline workload; a decoder with experts and a matrix memory beside the Sabisun of equal size on one GPU",
+    last = res[mine]["decode"][-1]
+    print(json.dumps({"secondary": f"not the headline workload; {what} beside the {other.capitalize()} of equal size on one GPU",
                       "metric": f"decode tokens/s ({args.workload}, batch 32)", "value": last["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": 3,
                       "ms_per_step": last["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
-                      "dtype": "bf16 (float32 residual, router, gates, softmax, state)", "data": "synthetic",
+                      "dtype": "bf16 (float32 residual, norms, scores, softmax, router, recurrences)", "data": "synthetic",
                       "config": {"workload": args.workload, **dims, "ctx": ctx, "cuda_graph": True, "l2": "weights larger than L2 streamed per step"},
-                      "clocks": clocks, **res["padetar"], "sabisun_config": sdims, "sabisun": res["sabisun"]}))
+                      "clocks": clocks, **res[mine], f"{other}_config": odims, other: res[other]}))
 
 
 def main():
@@ -836,7 +868,7 @@ def main():
                     "stays small; the line is then marked profiling_only and is not a benchmark result")
     ap.add_argument("--pdl", type=int, default=-1, help="secondary workloads: programmatic dependent launch, bit 0 = linear kernels, bit 1 = "
                     "attention kernel (-1: the decoder's default)")
-    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY) + list(HYBRID) + list(EXPERTS),
+    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY) + list(HYBRID) + list(EXPERTS) + list(LATENT),
                     help="llama2-7b-int4 is the benchmark; the others time a parity configuration, or an architecture of this framework beside the "
                     "closest one of equal size, on one GPU (line marked `secondary`)")
     args = ap.parse_args()
@@ -846,8 +878,8 @@ def main():
         run_secondary(args)
     elif args.workload in HYBRID:
         run_hybrid(args)
-    elif args.workload in EXPERTS:
-        run_experts(args)
+    elif args.workload in EXPERTS or args.workload in LATENT:
+        run_beside(args)
     else:
         run_b200(args)
 

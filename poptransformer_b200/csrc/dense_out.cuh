@@ -61,17 +61,22 @@ static inline const char *dense_ext_error(int epilogue, int n_out, const pt_dens
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * x * x, x, x)));
 }
-// (rounded to bf16 by the caller)  tanh(z) = 2 sigmoid(2 z) - 1
+// tanh(z) = 2 sigmoid(2 z) - 1, with the fast exponential and quotient (a few units in the last place): what the bf16 kernels use, also
+// because their epilogues stay short
 __device__ __forceinline__ float gelu_tanh_fast(float x) {
   return __fdividef(x, 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * x * x, x, x)));
 }
-template <bool FAST> __device__ __forceinline__ float glu_f(const DenseOut &o, float gate, float up) {
-  if (o.glu == PT_GLU_SILU) return (FAST ? __fdividef(gate, 1.0f + __expf(-gate)) : gate / (1.0f + expf(-gate))) * up;
-  if (o.glu == PT_GLU_GELU) return (FAST ? gelu_tanh_fast(gate) : gelu_tanh_f(gate)) * up;
-  const float limit = o.limit;
+template <bool FAST, int GLU> __device__ __forceinline__ float glu_unit(float gate, float up, float limit) {
+  if (GLU == PT_GLU_SILU) return (FAST ? __fdividef(gate, 1.0f + __expf(-gate)) : gate / (1.0f + expf(-gate))) * up;
+  if (GLU == PT_GLU_GELU) return (FAST ? gelu_tanh_fast(gate) : gelu_tanh_f(gate)) * up;
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   if (FAST) return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);   // (rounded to bf16 by the caller; for g very negative the quotient is 0)
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+template <bool FAST> __device__ __forceinline__ float glu_f(const DenseOut &o, float gate, float up) {
+  if (o.glu == PT_GLU_SILU) return glu_unit<FAST, PT_GLU_SILU>(gate, up, 0.f);
+  if (o.glu == PT_GLU_GELU) return glu_unit<FAST, PT_GLU_GELU>(gate, up, 0.f);
+  return glu_unit<FAST, PT_GLU_CLAMPED>(gate, up, o.limit);
 }
 __device__ __forceinline__ void dense_put(const DenseOut &o, int m, int n, float y) {
   const size_t i = (size_t)m * o.out_ld + n;
@@ -80,8 +85,9 @@ __device__ __forceinline__ void dense_put(const DenseOut &o, int m, int n, float
 }
 __device__ __forceinline__ float dense_factor(const DenseOut &o, int m) { return o.row_scale ? o.alpha * __ldcg(o.row_scale + m) : o.alpha; }
 __device__ __forceinline__ float dense_value(const DenseOut &o, int m, int n, float acc) { return fmaf(acc, dense_factor(o, m), o.bias ? __ldg(o.bias + n) : 0.f); }
-// One finished sum (any epilogue but GLU, whose sums come in pairs).
-__device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, float acc) {
+__device__ __forceinline__ float softcap_fast(float x, float limit) { return limit * (1.0f - __fdividef(2.0f, 1.0f + __expf(__fdividef(2.0f * x, limit)))); }
+// One finished sum (any epilogue but GLU, whose sums come in pairs).  EXACT: for models that run in 32-bit.
+template <bool EXACT = false> __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, float acc) {
   float y = dense_value(o, m, n, acc);
   if (n >= o.split_n) {
     o.out2[(size_t)m * o.out2_ld + n - o.split_n] = y;
@@ -91,18 +97,65 @@ __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, flo
     y = fmaxf(y, 0.f);
     y *= y;
   } else if (o.epilogue == PT_EPI_SOFTCAP) {
-    y = o.limit * tanhf(y / o.limit);
+    y = EXACT ? o.limit * tanhf(y / o.limit) : softcap_fast(y, o.limit);
   } else if (o.epilogue == PT_EPI_GELU_MUL) {
     const size_t i = (size_t)o.mul_ids[m] * o.mul_ld + n;
-    y = gelu_tanh_f(y) * (o.out_dt == PT_DT_F32 ? reinterpret_cast<const float *>(o.mul)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16 *>(o.mul)[i]));
+    y = (EXACT ? gelu_tanh_f(y) : gelu_tanh_fast(y)) * (o.out_dt == PT_DT_F32 ? reinterpret_cast<const float *>(o.mul)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16 *>(o.mul)[i]));
   }
   dense_put(o, m, n, y);
 }
 // Sums of the gate row n (n % 16 < 8) and the up row n + 8.
-__device__ __forceinline__ void dense_store_glu(const DenseOut &o, int m, int n, float gate, float up) {
+template <bool EXACT = false> __device__ __forceinline__ void dense_store_glu(const DenseOut &o, int m, int n, float gate, float up) {
   const int f = n / 16 * 8 + n % 8;
   const float g = dense_value(o, m, n, gate), u = dense_value(o, m, n + 8, up);
-  dense_put(o, m, f, o.out_dt == PT_DT_F32 ? glu_f<false>(o, g, u) : glu_f<true>(o, g, u));
+  dense_put(o, m, f, glu_f<!EXACT>(o, g, u));
+}
+// Four consecutive outputs n .. n + 3 (n a multiple of four).  The plain epilogues leave as one store where the rows allow it.
+__device__ __forceinline__ void dense_put4(void *out, size_t i, bool f32, const float (&y)[4]) {
+  if (f32) {
+    float *o = reinterpret_cast<float *>(out) + i;
+    if (((uintptr_t)o & 15) == 0) *reinterpret_cast<float4 *>(o) = make_float4(y[0], y[1], y[2], y[3]);
+    else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[j] = y[j];
+    }
+  } else {
+    __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(out) + i;
+    if (((uintptr_t)o & 7) == 0) *reinterpret_cast<uint2 *>(o) = make_uint2(pack_bf2(y[0], y[1]), pack_bf2(y[2], y[3]));
+    else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[j] = __float2bfloat16_rn(y[j]);
+    }
+  }
+}
+__device__ __forceinline__ void dense_store4(const DenseOut &o, int m, int n, const float4 &acc) {
+  const float a[4] = {acc.x, acc.y, acc.z, acc.w};
+  const bool second = n >= o.split_n;
+  if (!second && o.epilogue != PT_EPI_STORE && o.epilogue != PT_EPI_RELU2) {
+#pragma unroll 1
+    for (int j = 0; j < 4; ++j) dense_store(o, m, n + j, j == 0 ? acc.x : j == 1 ? acc.y : j == 2 ? acc.z : acc.w);
+    return;
+  }
+  const float f = dense_factor(o, m);
+  float y[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    y[j] = fmaf(a[j], f, o.bias ? __ldg(o.bias + n + j) : 0.f);
+    if (!second && o.epilogue == PT_EPI_RELU2) {
+      y[j] = fmaxf(y[j], 0.f);
+      y[j] *= y[j];
+    }
+  }
+  if (second) dense_put4(o.out2, (size_t)m * o.out2_ld + n - o.split_n, true, y);
+  else dense_put4(o.out, (size_t)m * o.out_ld + n, o.out_dt == PT_DT_F32, y);
+}
+// Four gate rows n .. n + 3 and the up rows n + 8 ..
+__device__ __forceinline__ void dense_store_glu4(const DenseOut &o, int m, int n, const float4 &gate, const float4 &up) {
+  const float f = dense_factor(o, m), g[4] = {gate.x, gate.y, gate.z, gate.w}, u[4] = {up.x, up.y, up.z, up.w};
+  float y[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) y[j] = glu_f<true>(o, fmaf(g[j], f, o.bias ? __ldg(o.bias + n + j) : 0.f), fmaf(u[j], f, o.bias ? __ldg(o.bias + n + 8 + j) : 0.f));
+  dense_put4(o.out, (size_t)m * o.out_ld + n / 16 * 8 + n % 8, o.out_dt == PT_DT_F32, y);
 }
 #endif
 

@@ -244,14 +244,14 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 // bf16 output: neighbouring lanes (n, n + 1) trade values of two columns, so every store writes 4 bytes per lane.
 // Gated features: lanes n and n + 8 trade likewise, and each computes one column of the pair's feature.
 enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_GLU = 2, OUT_GELU_MUL = 3 };
-enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2 };
+enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2, ACT_SCALED = 16 };   // OUT_GLU: the kind of unit, plus ACT_SCALED with a factor per row
 template <int KIND, int ACT>
 __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, int ld, const uint32_t (&v)[32], int n, int m, int lane) {
   const float b = d.bias ? __ldg(d.bias + n + (KIND == OUT_F32 && out == d.out2 ? d.split_n : 0)) : 0.f;
   auto fin = [&](uint32_t x) {
     float y = fmaf(__uint_as_float(x), d.alpha, b);
     if (ACT == ACT_RELU2) { y = fmaxf(y, 0.f); y *= y; }
-    if (ACT == ACT_SOFTCAP) y = d.limit * tanhf(y / d.limit);
+    if (ACT == ACT_SOFTCAP) y = softcap_fast(y, d.limit);
     return y;
   };
   if (KIND == OUT_F32) {
@@ -284,13 +284,13 @@ __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, in
   } else {
     const bool up = lane & 8;
     __nv_bfloat16 *o = reinterpret_cast<__nv_bfloat16 *>(out) + (size_t)(m + (up ? 1 : 0)) * ld + n / 16 * 8 + n % 8;
-    const float mine = d.row_scale ? __ldcg(d.row_scale + m + lane) : 1.f;     // lane j: the factor of row m + j
+    const float mine = (ACT & ACT_SCALED) ? d.alpha * __ldcg(d.row_scale + m + lane) : d.alpha;     // lane j: the factor of row m + j
 #pragma unroll
     for (int j = 0; j < 32; j += 2) {
-      const float s0 = __shfl_sync(0xffffffffu, mine, j), s1 = __shfl_sync(0xffffffffu, mine, j + 1);
-      const float a = fmaf(__uint_as_float(v[j]), d.alpha * s0, b), c = fmaf(__uint_as_float(v[j + 1]), d.alpha * s1, b);
+      const float s0 = (ACT & ACT_SCALED) ? __shfl_sync(0xffffffffu, mine, j) : mine, s1 = (ACT & ACT_SCALED) ? __shfl_sync(0xffffffffu, mine, j + 1) : mine;
+      const float a = fmaf(__uint_as_float(v[j]), s0, b), c = fmaf(__uint_as_float(v[j + 1]), s1, b);
       const float t = __shfl_xor_sync(0xffffffffu, up ? a : c, 8);      // gate lane: the up value of column j; up lane: the gate value of j + 1
-      *o = __float2bfloat16_rn(up ? glu_f<true>(d, t, c) : glu_f<true>(d, a, t));
+      *o = __float2bfloat16_rn(up ? glu_unit<true, ACT & 15>(t, c, d.limit) : glu_unit<true, ACT & 15>(a, t, d.limit));
       o += 2 * (size_t)ld;
     }
   }
@@ -301,7 +301,7 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
   // (warp-uniform) where this warp's 32 outputs go
   const bool second = nq >= d.split_n, glu = d.epilogue == PT_EPI_GLU && !second, f32 = second || d.out_dt == PT_DT_F32;
   // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16
-  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) && (glu || !d.row_scale) &&
+  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) && (!d.row_scale || (glu && d.glu == PT_GLU_SILU)) &&
                     (second || f32 || d.epilogue != PT_EPI_SOFTCAP) &&
                     (f32 || glu || (d.out_ld % 2 == 0 && ((uintptr_t)d.out & 3) == 0));
   const int rows = min(p.mb, m_end - m0), whole = fast ? rows & ~31 : 0;
@@ -311,7 +311,10 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
     if (second) {
       epilogue_rows32<OUT_F32, ACT_NONE>(d, d.out2, d.out2_ld, v, n - d.split_n, m0 + c0, lane);
     } else if (glu) {
-      epilogue_rows32<OUT_GLU, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      if (d.glu == PT_GLU_SILU && d.row_scale) epilogue_rows32<OUT_GLU, PT_GLU_SILU | ACT_SCALED>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (d.glu == PT_GLU_GELU) epilogue_rows32<OUT_GLU, PT_GLU_GELU>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (d.glu == PT_GLU_SILU) epilogue_rows32<OUT_GLU, PT_GLU_SILU>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else epilogue_rows32<OUT_GLU, PT_GLU_CLAMPED>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     } else if (f32) {
       if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_F32, ACT_RELU2>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
       else if (d.epilogue == PT_EPI_SOFTCAP) epilogue_rows32<OUT_F32, ACT_SOFTCAP>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
@@ -361,17 +364,10 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
           if (p.dense.epilogue == PT_EPI_GLU && n < p.dense.split_n) {   // gate features n % 16 < 8, their up features eight further
             if (n & 8) continue;
             const float4 gt = sum4(n), up = sum4(n + 8);
-            dense_store_glu(p.dense, m, n, gt.x, up.x);
-            dense_store_glu(p.dense, m, n + 1, gt.y, up.y);
-            dense_store_glu(p.dense, m, n + 2, gt.z, up.z);
-            dense_store_glu(p.dense, m, n + 3, gt.w, up.w);
+            dense_store_glu4(p.dense, m, n, gt, up);
             continue;
           }
-          const float4 acc = sum4(n);
-          store_out<true>(p, acc.x, m, n);
-          store_out<true>(p, acc.y, m, n + 1);
-          store_out<true>(p, acc.z, m, n + 2);
-          store_out<true>(p, acc.w, m, n + 3);
+          dense_store4(p.dense, m, n, sum4(n));
         }
         return;
       }

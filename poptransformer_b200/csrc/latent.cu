@@ -15,6 +15,8 @@
 //   expand_kernel    the runs of pages combined, then W_uv and the gate per head (expand_plain_kernel: any sizes)
 // Prompts in fp32, or of sizes the tensor-core kernels do not take, go through pt_window_attn's any-size kernel with the values inside
 // the keys.  Norms, angles, scores, softmax and weights are fp32; weights enter the tensor cores as two bf16 parts (hi + lo).
+#include <type_traits>
+
 #include "chunk.cuh"
 
 namespace pt {
@@ -51,21 +53,26 @@ struct PrepParams {
   int *error_flag;
 };
 constexpr int PREP_THREADS = 256;
-template <typename T> __global__ void __launch_bounds__(PREP_THREADS) prep_kernel(const PrepParams p) {
-  __shared__ float red[32];
+template <typename T, int VEC> __global__ void __launch_bounds__(PREP_THREADS) prep_kernel(const PrepParams p) {   // block: one token
+  __shared__ float red[PREP_THREADS / 32];
   launch_dependents();
   wait_for_prerequisites();
   const int t = blockIdx.x, tid = threadIdx.x, s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
+  const bool ok = pos >= 0 && pos < p.max_len;
+  const int phys = ok ? p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page] : 0, half = p.rot / 2;
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.ld, *kv = reinterpret_cast<const T *>(p.kv) + (size_t)t * p.ld;
-  // the first half of the block sums the query latent, the second half the cached one
+  // the first half of the block takes the query latent, the second half the cached one
   constexpr int HALF = PREP_THREADS / 2;
   const bool second = tid >= HALF;
   const T *mine = second ? kv : q;
+  const float *norm = second ? p.kv_norm : p.q_norm;
   const int n = second ? p.rank : p.q_rank, lane = tid & 31, warp = tid >> 5, at = tid & (HALF - 1);
   float ss = 0.f;
-  for (int i = at; i < n; i += HALF) {
-    const float x = to_f(mine[i]);
-    ss = fmaf(x, x, ss);
+  for (int i = at * VEC; i < n; i += HALF * VEC) {
+    float v[VEC];
+    load_vec<VEC>(mine + i, v);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
   }
   ss = warp_sum(ss);
   if (lane == 0) red[warp] = ss;
@@ -73,18 +80,24 @@ template <typename T> __global__ void __launch_bounds__(PREP_THREADS) prep_kerne
   float sum = 0.f;
   for (int i = 0; i < HALF / 32; ++i) sum += red[(second ? HALF / 32 : 0) + i];
   const float inv = 1.0f / sqrtf(sum / (float)n + p.eps);
-  if (!second) {
-    T *out = reinterpret_cast<T *>(p.cq) + (size_t)t * p.cq_ld;
-    for (int i = at; i < p.cq_ld; i += HALF) out[i] = from_f<T>(i < n ? to_f(q[i]) * inv * __ldg(p.q_norm + i) : 0.f);
-    return;
-  }
-  if (pos < 0 || pos >= p.max_len) {
+  if (second && !ok) {
     if (at == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
   }
-  const int phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page], half = p.rot / 2;
   T *row = reinterpret_cast<T *>(p.pool) + ((size_t)phys * p.page + pos % p.page) * (p.rot + p.rank);
-  for (int i = at; i < n; i += HALF) row[p.rot + i] = from_f<T>(to_f(kv[i]) * inv * __ldg(p.kv_norm + i));
+  T *out = second ? row + p.rot : reinterpret_cast<T *>(p.cq) + (size_t)t * p.cq_ld;
+  for (int i = at * VEC; i < n; i += HALF * VEC) {
+    float v[VEC], w[VEC];
+    load_vec<VEC>(mine + i, v);
+    load_vec<VEC>(norm + i, w);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] *= inv * w[j];
+    store_vec<VEC>(out + i, v);
+  }
+  if (!second) {
+    for (int i = n + at; i < p.cq_ld; i += HALF) out[i] = from_f<T>(0.f);
+    return;
+  }
   for (int i = at; i < half; i += HALF) {
     const float u = to_f(kv[p.rank + i]), v = to_f(kv[p.rank + half + i]);
     const float2 c = __ldg(p.rope + (size_t)pos * half + i);
@@ -234,6 +247,53 @@ __global__ void __launch_bounds__(ABSORB_WARPS * 32) absorb_kernel(const Params 
 __device__ __forceinline__ int pages_per_run(int n_pages, int n_split) { return (n_pages + n_split - 1) / n_split; }
 
 constexpr int EXPAND_WARPS = 8;
+// os[m] = sum over the runs of cw[m][run] * o[m][run], V neighbouring dimensions per item; a thread has the loads of U items x PB runs in
+// flight together.
+template <int V, int U, int PB>
+__device__ __forceinline__ void combine_runs(const float *src, size_t m_stride, int rank, int n_split, int tokens, const int *act, const float (*cw)[kMaxSplit + 1], bf *os, int ld) {
+  typedef typename std::conditional<V == 4, float4, float2>::type Vec;
+  const int per = rank / V, items = tokens * per, step = EXPAND_WARPS * 32;
+  for (int i = threadIdx.x; i < items; i += U * step) {
+    float a[U][V] = {};
+    int top = 0;
+    const float *s[U];
+    int ms[U], n_act[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = i + u * step;
+      ms[u] = k < items ? k / per : 0;
+      n_act[u] = k < items ? act[ms[u]] : 0;
+      s[u] = src + ms[u] * m_stride + (k < items ? k - ms[u] * per : 0) * V;
+      top = max(top, n_act[u]);
+    }
+    for (int i0 = 0; i0 < top; i0 += PB) {
+      Vec v[U][PB];
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int j = 0; j < PB; ++j)
+          if (i0 + j < n_act[u]) v[u][j] = __ldcg(reinterpret_cast<const Vec *>(s[u] + (size_t)(i0 + j) * rank));
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int j = 0; j < PB; ++j)
+          if (i0 + j < n_act[u]) {
+            const float x = cw[ms[u]][i0 + j];
+            const float *f = reinterpret_cast<const float *>(&v[u][j]);
+#pragma unroll
+            for (int e = 0; e < V; ++e) a[u][e] = fmaf(f[e], x, a[u][e]);
+          }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = i + u * step;
+      if (k >= items) break;
+      uint32_t *o = reinterpret_cast<uint32_t *>(os + ms[u] * ld + (k - ms[u] * per) * V);
+#pragma unroll
+      for (int e = 0; e < V; e += 2) o[e / 2] = pack_bf2(a[u][e], a[u][e + 1]);
+    }
+  }
+}
 // Grid: (16 ng outputs, head, 16 tokens).  Warp (n group, k group): 8 / ng warps share an output group's k.
 __global__ void __launch_bounds__(EXPAND_WARPS * 32) expand_kernel(const Params p) {
   extern __shared__ __align__(16) unsigned char sm_raw[];
@@ -262,28 +322,12 @@ __global__ void __launch_bounds__(EXPAND_WARPS * 32) expand_kernel(const Params 
     if (lane == 0) act[m] = n_act;
   }
   __syncthreads();
-  const int r4 = p.rank / 4;
-  for (int i = tid; i < 16 * r4; i += blockDim.x) {
-    const int m = i / r4, c = (i - m * r4) * 4, n_act = act[m];
-    const float *src = p.ws_o + ((size_t)(t0 + m) * p.n_head + h) * p.n_split * p.rank + c;
-    constexpr int PB = 8;
-    float a[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int i0 = 0; i0 < n_act; i0 += PB) {
-      float4 v[PB];
-#pragma unroll
-      for (int j = 0; j < PB; ++j) v[j] = i0 + j < n_act ? __ldcg(reinterpret_cast<const float4 *>(src + (size_t)(i0 + j) * p.rank)) : make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-      for (int j = 0; j < PB; ++j) {
-        if (i0 + j >= n_act) break;
-        const float x = cw[m][i0 + j];
-        a[0] = fmaf(v[j].x, x, a[0]);
-        a[1] = fmaf(v[j].y, x, a[1]);
-        a[2] = fmaf(v[j].z, x, a[2]);
-        a[3] = fmaf(v[j].w, x, a[3]);
-      }
-    }
-    *reinterpret_cast<uint2 *>(os + m * ld + c) = make_uint2(pack_bf2(a[0], a[1]), pack_bf2(a[2], a[3]));
-  }
+  const int tokens = min(16, p.n_tok - t0);
+  const float *src = p.ws_o + ((size_t)t0 * p.n_head + h) * p.n_split * p.rank;
+  const size_t m_stride = (size_t)p.n_head * p.n_split * p.rank;
+  if (tokens == 1) combine_runs<2, 1, 16>(src, m_stride, p.rank, p.n_split, tokens, act, cw, os, ld);
+  else combine_runs<4, 4, 4>(src, m_stride, p.rank, p.n_split, tokens, act, cw, os, ld);
+  for (int i = tid; i < (16 - tokens) * p.rank / 2; i += blockDim.x) reinterpret_cast<uint32_t *>(os + (tokens + i / (p.rank / 2)) * ld)[i % (p.rank / 2)] = 0u;
   __syncthreads();
   // ---- W_uv
   float acc[2][4] = {};
@@ -322,18 +366,18 @@ __global__ void __launch_bounds__(EXPAND_WARPS * 32) expand_kernel(const Params 
 
 // ------------------------------------------------------------------------------------------ one token per sequence
 // Block: one run of pages of one sequence, 16 MT heads.  The rows [rotated part | latent] of a page lie once in shared memory and serve
-// as keys (warp w: keys 8 w ..) and, from column rot on, as values (warp w: latent dimensions 8 NT w ..).
-constexpr int DEC_WARPS = 8, DEC_THREADS = DEC_WARPS * 32, P_LD = TILE + 8;
+// as keys (warps w and w + 8: keys 8 w .., half of the row each) and, from column rot on, as values (warp w: latent dimensions 8 NT w ..).
+constexpr int DEC_WARPS = 16, DEC_THREADS = DEC_WARPS * 32, P_LD = TILE + 8;
 template <int MT> static size_t decode_smem(int width_pad) {
-  return (size_t)(16 * MT + 2 * TILE) * (width_pad + 8) * sizeof(bf) + (size_t)16 * MT * (P_LD * (sizeof(float) + 2 * sizeof(bf)) + sizeof(float));
+  return (size_t)(16 * MT + 2 * TILE) * (width_pad + 8) * sizeof(bf) + (size_t)16 * MT * (P_LD * (2 * sizeof(float) + 2 * sizeof(bf)) + sizeof(float));
 }
 template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) decode_kernel(const Params p) {
   constexpr int HB = 16 * MT;
   extern __shared__ __align__(16) unsigned char sm_raw[];
   const int ld = p.width_pad + 8;
   bf *qs = reinterpret_cast<bf *>(sm_raw), *ks = qs + HB * ld;              // [HB][ld], [2][TILE][ld]
-  float *ps = reinterpret_cast<float *>(ks + 2 * TILE * ld);                // [HB][P_LD]
-  bf *ph = reinterpret_cast<bf *>(ps + HB * P_LD), *pl = ph + HB * P_LD;    // [HB][P_LD] the weights' two parts
+  float *ps = reinterpret_cast<float *>(ks + 2 * TILE * ld);                // [2][HB][P_LD] scores, the two halves' sums
+  bf *ph = reinterpret_cast<bf *>(ps + 2 * HB * P_LD), *pl = ph + HB * P_LD;    // [HB][P_LD] the weights' two parts
   float *corr = reinterpret_cast<float *>(pl + HB * P_LD);                  // [HB]
   launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
@@ -369,9 +413,9 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
     }
   load_page(pg0, 0);
   const float sc2 = p.scale * kLog2e;
-  float m_run[2 * MT], l_run[2 * MT];             // heads 2 MT warp .. (the same in all lanes)
+  float m_run[MT], l_run[MT];                     // heads MT warp .. (the same in all lanes)
 #pragma unroll
-  for (int i = 0; i < 2 * MT; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+  for (int i = 0; i < MT; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
   float o[MT][NT][4];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
@@ -390,10 +434,11 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
     const bf *K = ks + stage * TILE * ld;
     {
       float sc[MT][2][4] = {};
-      const uint32_t k_lane = smem_addr(K + (warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8);     // matrices: k 0-7, 8-15, 16-23, 24-31 of eight keys
+      const int keys = (warp & 7) * 8, part = warp >> 3, steps = p.width_pad / 32, k0 = part ? (steps + 1) / 2 * 32 : 0, k1 = part ? p.width_pad : (steps + 1) / 2 * 32;
+      const uint32_t k_lane = smem_addr(K + (keys + (lane & 7)) * ld + (lane >> 3) * 8);     // matrices: k 0-7, 8-15, 16-23, 24-31 of eight keys
       const uint32_t q_lane = smem_addr(qs + (lane & 15) * ld + (lane >> 4) * 8);
-#pragma unroll 2
-      for (int k = 0; k < p.width_pad; k += 32) {
+#pragma unroll 3
+      for (int k = k0; k < k1; k += 32) {
         uint32_t b0, b1, b2, b3;
         ldsm4(k_lane + k * 2u, b0, b1, b2, b3);
 #pragma unroll
@@ -406,20 +451,23 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
           mma16816_bf16(sc[mt][1], a0, a1, a2, a3, b2, b3);
         }
       }
-      const int key = warp * 8 + 2 * tig, seen = pos - pg * TILE;           // keys 0 .. seen of this page
+      const int key = keys + 2 * tig, seen = pos - pg * TILE;           // keys 0 .. seen of this page
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const float a = (sc[mt][0][2 * r] + sc[mt][1][2 * r]) * sc2, b = (sc[mt][0][2 * r + 1] + sc[mt][1][2 * r + 1]) * sc2;
-          *reinterpret_cast<float2 *>(ps + (mt * 16 + g + 8 * r) * P_LD + key) = make_float2(key <= seen ? a : -INFINITY, key + 1 <= seen ? b : -INFINITY);
+          *reinterpret_cast<float2 *>(ps + (part * HB + mt * 16 + g + 8 * r) * P_LD + key) = make_float2(key <= seen ? a : -INFINITY, key + 1 <= seen ? b : -INFINITY);
         }
     }
     __syncthreads();
 #pragma unroll
-    for (int i = 0; i < 2 * MT; ++i) {
-      const int r = warp * 2 * MT + i;
-      const float2 v = *reinterpret_cast<const float2 *>(ps + r * P_LD + 2 * lane);
+    for (int i = 0; i < MT; ++i) {
+      const int r = warp * MT + i;
+      float2 v = *reinterpret_cast<const float2 *>(ps + r * P_LD + 2 * lane);
+      const float2 v2 = *reinterpret_cast<const float2 *>(ps + (HB + r) * P_LD + 2 * lane);
+      v.x += v2.x;
+      v.y += v2.y;
       const float m = fmaxf(m_run[i], warp_max(fmaxf(v.x, v.y)));           // (a page of a run holds at least one visible key)
       const float a = exp2f(v.x - m), b = exp2f(v.y - m), c = exp2f(m_run[i] - m);
       uint32_t hi, lo;
@@ -479,8 +527,8 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
         if (c0 + j * 8 < p.rank) *reinterpret_cast<float2 *>(dst + j * 8) = make_float2(o[mt][j][2 * r], o[mt][j][2 * r + 1]);
     }
 #pragma unroll
-  for (int i = 0; i < 2 * MT; ++i) {
-    const int row = warp * 2 * MT + i;
+  for (int i = 0; i < MT; ++i) {
+    const int row = warp * MT + i;
     if (lane == 0 && row < nh) p.ws_ml[(head0 + row) * p.n_split + x] = make_float2(m_run[i], l_run[i]);
   }
 }
@@ -494,9 +542,7 @@ template <int MT, int NT> static int launch_decode(const Params &p, cudaStream_t
   return PT_OK;
 }
 template <int MT> static int dispatch_decode(const Params &p, cudaStream_t st) {
-  if (p.rank <= 128) return launch_decode<MT, 2>(p, st);
-  if (p.rank <= 256) return launch_decode<MT, 4>(p, st);
-  return launch_decode<MT, 8>(p, st);
+  return p.rank <= 256 ? launch_decode<MT, 2>(p, st) : launch_decode<MT, 4>(p, st);
 }
 
 constexpr size_t kSmemLimit = 226 * 1024;
@@ -532,7 +578,11 @@ extern "C" int pt_latent_prep(const pt_latent_prep_args *a, void *stream) {
   PT_REQUIRE(p.max_len <= a->page_size * a->max_pages, "pt_latent_prep: max_len=%d exceeds the page table", p.max_len);
   p.q = a->q; p.kv = a->kv; p.q_norm = a->q_norm; p.kv_norm = a->kv_norm; p.rope = (const float2 *)a->rope; p.cq = a->cq; p.pool = a->pool;
   p.page_table = a->page_table; p.cu = b.cu; p.start = b.start; p.slot = b.slot; p.tok_seq = b.tok_seq; p.error_flag = a->error_flag;
-  auto kernel = a->dtype == PT_DT_F32 ? lat::prep_kernel<float> : lat::prep_kernel<__nv_bfloat16>;
+  const int es = a->dtype == PT_DT_F32 ? 4 : 2;
+  auto al = [&](const void *x) { return aligned_to(x, 4 * es); };
+  const bool v4 = a->q_rank % 4 == 0 && a->rank % 4 == 0 && a->rot_dim % 4 == 0 && a->ld % 4 == 0 && a->cq_ld % 4 == 0 && al(a->q) && al(a->kv) && al(a->cq) && al(a->pool) &&
+                  aligned_to(a->q_norm, 16) && aligned_to(a->kv_norm, 16);
+  auto kernel = a->dtype == PT_DT_F32 ? (v4 ? lat::prep_kernel<float, 4> : lat::prep_kernel<float, 1>) : (v4 ? lat::prep_kernel<__nv_bfloat16, 4> : lat::prep_kernel<__nv_bfloat16, 1>);
   PT_CUDA(lat::launch_early(kernel, dim3(b.n_tok), lat::PREP_THREADS, 0, as_stream(stream), p));
   count_launch();
   return PT_OK;

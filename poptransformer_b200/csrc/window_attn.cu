@@ -71,7 +71,8 @@ struct Score {
     a = capped ? 2.0f * p.scale * kLog2e / p.softcap : p.scale * kLog2e;
     b = p.softcap * kLog2e;
   }
-  __device__ __forceinline__ float operator()(float s) const { return capped ? b * (1.0f - __fdividef(2.0f, exp2f(a * s) + 1.0f)) : a * s; }
+  __device__ __forceinline__ float cap(float s) const { return b * (1.0f - __fdividef(2.0f, exp2f(a * s) + 1.0f)); }
+  __device__ __forceinline__ float operator()(float s) const { return capped ? cap(s) : a * s; }
 };
 template <typename T> __device__ __forceinline__ float gate_at(const Params &p, int t, int head, int c) {
   if (!p.gate) return 1.f;
@@ -181,6 +182,33 @@ template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_pr
     norm_rotate<T>(p, p.dim, hl, k, p.k_norm, pos, kc);
     for (int i = lane; i < p.vdim; i += 32) vc[i] = v[i];
   }
+}
+
+// Rotation alone, of bf16 queries in place: a thread takes eight neighbouring pairs of one head.
+__global__ void attn_rotate_kernel(const Params p) {
+  const int per = p.rope_half / 8, i = blockIdx.x * blockDim.x + threadIdx.x;
+  const int c = (i % per) * 8, h = i / per % p.n_head, t = i / (per * p.n_head);
+  if (t >= p.cu[p.n_seq]) return;
+  const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
+  if (pos < 0 || pos >= p.max_len) {
+    if (p.error_flag) atomicExch(p.error_flag, 12);
+    return;
+  }
+  __nv_bfloat16 *q = reinterpret_cast<__nv_bfloat16 *>(const_cast<void *>(p.q)) + (size_t)t * p.q_ld + (size_t)h * p.dim + c;
+  const float4 *cs = reinterpret_cast<const float4 *>(p.rope + (size_t)pos * p.rope_half + c);
+  float u[8], v[8];
+  load_vec<8>(q, u);
+  load_vec<8>(q + p.rope_half, v);
+  uint4 a, b;
+  uint32_t *ap = reinterpret_cast<uint32_t *>(&a), *bp = reinterpret_cast<uint32_t *>(&b);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float4 x = __ldg(cs + j);
+    ap[j] = pack_bf2(u[2 * j] * x.x - v[2 * j] * x.y, u[2 * j + 1] * x.z - v[2 * j + 1] * x.w);
+    bp[j] = pack_bf2(v[2 * j] * x.x + u[2 * j] * x.y, v[2 * j + 1] * x.z + u[2 * j + 1] * x.w);
+  }
+  *reinterpret_cast<uint4 *>(q) = a;
+  *reinterpret_cast<uint4 *>(q + p.rope_half) = b;
 }
 
 template <typename T> __global__ void kv_append_kernel(const Params p) {
@@ -379,13 +407,24 @@ template <int DK, int DV, bool CTX> __global__ void __launch_bounds__(TC_THREADS
           mma16816_bf16(sc[j + 1], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b2, b3);
         }
       const bool whole = k0 + TILE - 1 <= wlo && (p.window == 0 || whi - k0 < p.window || k0 + TILE <= p.keep_first);
+      if (score.capped) {                                         // (uniform)
+#pragma unroll
+        for (int j = 0; j < TILE / 8; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sc[j][e] = score.cap(sc[j][e]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < TILE / 8; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sc[j][e] *= score.a;
+      }
       float m_new[2] = {m_run[0], m_run[1]};
 #pragma unroll
       for (int j = 0; j < TILE / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = k0 + j * 8 + 2 * tig + (e & 1);
-          float v = score(sc[j][e]);
+          float v = sc[j][e];
           if (!whole && !visible(p, e < 2 ? pos0 : pos1, key)) v = -INFINITY;
           sc[j][e] = v;
           m_new[e >> 1] = fmaxf(m_new[e >> 1], v);
@@ -676,7 +715,12 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
         }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) acc[j] *= ml[2 * h] * gate_at<T>(p, t, h0 + h, c + j);
+    for (int j = 0; j < 4; ++j) acc[j] *= ml[2 * h];
+    if (p.gate) {
+      const T *gate = reinterpret_cast<const T *>(p.gate) + (size_t)t * p.gate_ld + (p.gate_heads ? h0 + h : (h0 + h) * p.vdim + c);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[j] *= __fdividef(1.0f, 1.0f + __expf(-to_f(gate[p.gate_heads ? 0 : j])));
+    }
     T *o = out + (size_t)(h0 + h) * p.vdim + c;                // (rows of an even number of elements)
     *reinterpret_cast<__nv_bfloat162 *>(o) = __floats2bfloat162_rn(acc[0], acc[1]);
     *reinterpret_cast<__nv_bfloat162 *>(o + 2) = __floats2bfloat162_rn(acc[2], acc[3]);
@@ -814,7 +858,11 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
     p.ws_o = (float *)ws;
     return wa::dispatch_tc(p, true, 1, st);
   }
-  if (p.prep) {
+  if (p.prep && !p.k && !a->q_norm && a->dtype == PT_DT_BF16 && p.rope_half % 8 == 0 && p.dim % 8 == 0 && p.q_ld % 8 == 0 && al16(p.q) && al16(p.rope) &&
+      (long long)b.n_tok * p.n_head * p.rope_half < (1ll << 31)) {
+    wa::attn_rotate_kernel<<<ceil_div(b.n_tok * p.n_head * (p.rope_half / 8), 256), 256, 0, st>>>(p);
+    PT_LAUNCH_CHECK("pt_window_attn");
+  } else if (p.prep) {
     if (a->dtype == PT_DT_F32) wa::attn_prep_kernel<float><<<b.n_tok, wa::PREP_WARPS * 32, 0, st>>>(p);
     else wa::attn_prep_kernel<__nv_bfloat16><<<b.n_tok, wa::PREP_WARPS * 32, 0, st>>>(p);
     PT_LAUNCH_CHECK("pt_window_attn");

@@ -156,11 +156,17 @@ class PadetarDecoder(SequenceDecoder):
     def _linears(self):
         return [self.head] + [x for s in self.subs for x in (s.proj, s.down if s.kind == "moe" else s.out) if x is not None]
 
+    def expert_groups(self):
+        return [s.experts for s in self.subs if s.kind == "moe"]
+
+    def fixed_bytes(self):
+        """Weight bytes that every decode step streams, whatever the experts."""
+        return sum(x.nbytes for x in self._linears())
+
     def weight_bytes(self, rows=1):
         """Algorithmic weight bytes one decode step of `rows` tokens streams: every linear once, of the experts as many as the rows
         can choose at most."""
-        moe = [s for s in self.subs if s.kind == "moe"]
-        return sum(x.nbytes for x in self._linears()) + sum(s.experts.step_bytes(rows) for s in moe)
+        return self.fixed_bytes() + sum(e.step_bytes(rows) for e in self.expert_groups())
 
     # ---- state ----------------------------------------------------------------------------------
     def _alloc_layers(self):

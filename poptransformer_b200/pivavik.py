@@ -159,13 +159,17 @@ class PivavikDecoder(SequenceDecoder):
         once = [self.head] + [self.loop_in for r in self.runs if r.entry is not None]
         return once + [x for r in self.runs for x in (r.sub.proj, r.sub.ff, r.sub.uq if r.sub.lay.kind != "attention" else None, r.sub.out) if x is not None]
 
-    def head_bytes(self):
-        """Bytes of the per-head up-projections that every decode step reads beside the linears."""
-        return sum(x.numel() * x.element_size() for r in self.runs if r.sub.lay.kind != "attention" for x in (r.sub.lat.w_k, r.sub.lat.w_v))
+    def expert_groups(self):
+        return [r.sub.experts for r in self.runs if r.sub.experts]
+
+    def fixed_bytes(self):
+        """Weight bytes that every decode step streams, whatever the experts: the linears and the latents' per-head up-projections."""
+        heads = [x for r in self.runs if r.sub.lay.kind != "attention" for x in (r.sub.lat.w_k, r.sub.lat.w_v)]
+        return sum(x.nbytes for x in self._linears()) + sum(x.numel() * x.element_size() for x in heads)
 
     def weight_bytes(self, rows=1):
         """Algorithmic weight bytes one decode step of `rows` tokens streams, of the experts as many as the rows can choose at most."""
-        return sum(x.nbytes for x in self._linears()) + self.head_bytes() + sum(r.sub.experts.step_bytes(rows) for r in self.runs if r.sub.experts)
+        return self.fixed_bytes() + sum(e.step_bytes(rows) for e in self.expert_groups())
 
     # ---- state ----------------------------------------------------------------------------------
     def _alloc_layers(self):

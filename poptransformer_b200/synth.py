@@ -139,6 +139,60 @@ def padetar_state_dict(config, seed=0, device="cpu"):
     return sd
 
 
+def pivavik_state_dict(config, seed=0, device="cpu"):
+    """Pivavik architecture (a parsed config.json), bfloat16: linears N(0, 1 / in_features), the stream's norms N(0, 0.02) around zero, the
+    latents' 1 + N(0, 0.02)."""
+    gen = torch.Generator(device=device)
+    gen.manual_seed(seed)
+    sd = {}
+    W, V = config["width"], config["vocab"]
+
+    def put(key, shape, std=1.0, mean=0.0):
+        sd[key] = torch.empty(shape, dtype=torch.bfloat16, device=device).normal_(mean, std, generator=gen)
+
+    def lin(key, o, i, bias=False):
+        put(key, (o, i), i ** -0.5)
+        if bias:
+            put(key + ".b", (o,), 0.1)
+
+    lin("embed", V, W)
+    put("embed.norm", (W,), 0.02)
+    put("final.norm", (W,), 0.02)
+    if config.get("loop"):
+        lin("loop.in", W, 2 * W)
+        put("loop.step", (config["loop"]["times"], W), 0.1)
+    for i, lay in enumerate(config["layers"]):
+        p, m, mlp = f"l{i}.", lay["mixer"], lay.get("mlp")
+        M, Q, H = p + "mix.", p + "mlp.", m["heads"]
+        put(p + "norm1", (W,), 0.02)
+        if lay["type"] == "latent_attention":
+            lin(M + "dq", m["q_rank"], W)
+            put(M + "dq.norm", (m["q_rank"],), 0.02, 1.0)
+            lin(M + "uq", H * (m["dim"] + m["rot_dim"]), m["q_rank"])
+            lin(M + "dkv", m["kv_rank"] + m["rot_dim"], W)
+            put(M + "dkv.norm", (m["kv_rank"],), 0.02, 1.0)
+            lin(M + "uk", H * m["dim"], m["kv_rank"])
+            lin(M + "uv", H * m["vdim"], m["kv_rank"])
+            lin(M + "g", H, W)
+        else:
+            lin(M + "q", H * m["dim"], W, True)
+            lin(M + "k", m["kv_heads"] * m["dim"], W, True)
+            lin(M + "v", m["kv_heads"] * m["vdim"], W, True)
+            lin(M + "g", H * m["vdim"], W)
+        lin(M + "o", W, H * m["vdim"])
+        if mlp and mlp["kind"] == "dense":
+            lin(Q + "gate", mlp["ff"], W, True)
+            lin(Q + "up", mlp["ff"], W, True)
+            lin(Q + "down", W, mlp["ff"], True)
+        elif mlp:
+            lin(Q + "router", mlp["router"]["experts"], W)
+            for e in range(mlp["router"]["experts"]):
+                lin(Q + f"e{e}.gate", mlp["expert"]["ff"], W)
+                lin(Q + f"e{e}.up", mlp["expert"]["ff"], W)
+                lin(Q + f"e{e}.down", W, mlp["expert"]["ff"])
+    return sd
+
+
 def gpt2_state_dict(n_layer, d_model, n_head, vocab, n_positions, seed=0, device="cpu"):
     """GPT-2 architecture with the reference's key names after its checkpoint pre-processing (gpt2/model.py:154-166): linear
     weights [out, in], the query third of c_attn (weight and bias) multiplied by 1/sqrt(head_size).  fp16, N(0, 0.02);
