@@ -42,6 +42,7 @@ static inline DenseOut make_dense_out(void *out, int out_ld, int out_dt, int epi
   }
   return o;
 }
+static inline bool dense_needs_ext(int epilogue, const pt_dense_ext *e) { return e && (e->row_scale || epilogue == PT_EPI_SOFTCAP || (epilogue == PT_EPI_GLU && e->glu != PT_GLU_CLAMPED)); }
 static inline bool dense_epilogue_known(int e) { return e == PT_EPI_STORE || e == PT_EPI_RELU2 || e == PT_EPI_GLU || e == PT_EPI_GELU_MUL || e == PT_EPI_SOFTCAP; }
 // nullptr, or what is wrong with the combination.
 static inline const char *dense_ext_error(int epilogue, int n_out, const pt_dense_ext *e) {
@@ -73,7 +74,9 @@ template <bool FAST, int GLU> __device__ __forceinline__ float glu_unit(float ga
   if (FAST) return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);   // (rounded to bf16 by the caller; for g very negative the quotient is 0)
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
-template <bool FAST> __device__ __forceinline__ float glu_f(const DenseOut &o, float gate, float up) {
+// EXT: the kernel serves what dense_needs_ext names (an instantiation of its own, so that the others' epilogues stay short)
+template <bool FAST, bool EXT> __device__ __forceinline__ float glu_f(const DenseOut &o, float gate, float up) {
+  if (!EXT) return glu_unit<FAST, PT_GLU_CLAMPED>(gate, up, o.limit);
   if (o.glu == PT_GLU_SILU) return glu_unit<FAST, PT_GLU_SILU>(gate, up, 0.f);
   if (o.glu == PT_GLU_GELU) return glu_unit<FAST, PT_GLU_GELU>(gate, up, 0.f);
   return glu_unit<FAST, PT_GLU_CLAMPED>(gate, up, o.limit);
@@ -83,12 +86,12 @@ __device__ __forceinline__ void dense_put(const DenseOut &o, int m, int n, float
   if (o.out_dt == PT_DT_F32) reinterpret_cast<float *>(o.out)[i] = y;
   else reinterpret_cast<__nv_bfloat16 *>(o.out)[i] = __float2bfloat16_rn(y);
 }
-__device__ __forceinline__ float dense_factor(const DenseOut &o, int m) { return o.row_scale ? o.alpha * __ldcg(o.row_scale + m) : o.alpha; }
-__device__ __forceinline__ float dense_value(const DenseOut &o, int m, int n, float acc) { return fmaf(acc, dense_factor(o, m), o.bias ? __ldg(o.bias + n) : 0.f); }
+template <bool EXT> __device__ __forceinline__ float dense_factor(const DenseOut &o, int m) { return EXT && o.row_scale ? o.alpha * __ldcg(o.row_scale + m) : o.alpha; }
+template <bool EXT> __device__ __forceinline__ float dense_value(const DenseOut &o, int m, int n, float acc) { return fmaf(acc, dense_factor<EXT>(o, m), o.bias ? __ldg(o.bias + n) : 0.f); }
 __device__ __forceinline__ float softcap_fast(float x, float limit) { return limit * (1.0f - __fdividef(2.0f, 1.0f + __expf(__fdividef(2.0f * x, limit)))); }
 // One finished sum (any epilogue but GLU, whose sums come in pairs).  EXACT: for models that run in 32-bit.
-template <bool EXACT = false> __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, float acc) {
-  float y = dense_value(o, m, n, acc);
+template <bool EXT, bool EXACT = false> __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, float acc) {
+  float y = dense_value<EXT>(o, m, n, acc);
   if (n >= o.split_n) {
     o.out2[(size_t)m * o.out2_ld + n - o.split_n] = y;
     return;
@@ -96,7 +99,7 @@ template <bool EXACT = false> __device__ __forceinline__ void dense_store(const 
   if (o.epilogue == PT_EPI_RELU2) {
     y = fmaxf(y, 0.f);
     y *= y;
-  } else if (o.epilogue == PT_EPI_SOFTCAP) {
+  } else if (EXT && o.epilogue == PT_EPI_SOFTCAP) {
     y = EXACT ? o.limit * tanhf(y / o.limit) : softcap_fast(y, o.limit);
   } else if (o.epilogue == PT_EPI_GELU_MUL) {
     const size_t i = (size_t)o.mul_ids[m] * o.mul_ld + n;
@@ -105,10 +108,10 @@ template <bool EXACT = false> __device__ __forceinline__ void dense_store(const 
   dense_put(o, m, n, y);
 }
 // Sums of the gate row n (n % 16 < 8) and the up row n + 8.
-template <bool EXACT = false> __device__ __forceinline__ void dense_store_glu(const DenseOut &o, int m, int n, float gate, float up) {
+template <bool EXT, bool EXACT = false> __device__ __forceinline__ void dense_store_glu(const DenseOut &o, int m, int n, float gate, float up) {
   const int f = n / 16 * 8 + n % 8;
-  const float g = dense_value(o, m, n, gate), u = dense_value(o, m, n + 8, up);
-  dense_put(o, m, f, glu_f<!EXACT>(o, g, u));
+  const float g = dense_value<EXT>(o, m, n, gate), u = dense_value<EXT>(o, m, n + 8, up);
+  dense_put(o, m, f, glu_f<!EXACT, EXT>(o, g, u));
 }
 // Four consecutive outputs n .. n + 3 (n a multiple of four).  The plain epilogues leave as one store where the rows allow it.
 __device__ __forceinline__ void dense_put4(void *out, size_t i, bool f32, const float (&y)[4]) {
@@ -128,15 +131,15 @@ __device__ __forceinline__ void dense_put4(void *out, size_t i, bool f32, const 
     }
   }
 }
-__device__ __forceinline__ void dense_store4(const DenseOut &o, int m, int n, const float4 &acc) {
+template <bool EXT> __device__ __forceinline__ void dense_store4(const DenseOut &o, int m, int n, const float4 &acc) {
   const float a[4] = {acc.x, acc.y, acc.z, acc.w};
   const bool second = n >= o.split_n;
   if (!second && o.epilogue != PT_EPI_STORE && o.epilogue != PT_EPI_RELU2) {
 #pragma unroll 1
-    for (int j = 0; j < 4; ++j) dense_store(o, m, n + j, j == 0 ? acc.x : j == 1 ? acc.y : j == 2 ? acc.z : acc.w);
+    for (int j = 0; j < 4; ++j) dense_store<EXT>(o, m, n + j, j == 0 ? acc.x : j == 1 ? acc.y : j == 2 ? acc.z : acc.w);
     return;
   }
-  const float f = dense_factor(o, m);
+  const float f = dense_factor<EXT>(o, m);
   float y[4];
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
@@ -150,11 +153,11 @@ __device__ __forceinline__ void dense_store4(const DenseOut &o, int m, int n, co
   else dense_put4(o.out, (size_t)m * o.out_ld + n, o.out_dt == PT_DT_F32, y);
 }
 // Four gate rows n .. n + 3 and the up rows n + 8 ..
-__device__ __forceinline__ void dense_store_glu4(const DenseOut &o, int m, int n, const float4 &gate, const float4 &up) {
-  const float f = dense_factor(o, m), g[4] = {gate.x, gate.y, gate.z, gate.w}, u[4] = {up.x, up.y, up.z, up.w};
+template <bool EXT> __device__ __forceinline__ void dense_store_glu4(const DenseOut &o, int m, int n, const float4 &gate, const float4 &up) {
+  const float f = dense_factor<EXT>(o, m), g[4] = {gate.x, gate.y, gate.z, gate.w}, u[4] = {up.x, up.y, up.z, up.w};
   float y[4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) y[j] = glu_f<true>(o, fmaf(g[j], f, o.bias ? __ldg(o.bias + n + j) : 0.f), fmaf(u[j], f, o.bias ? __ldg(o.bias + n + 8 + j) : 0.f));
+  for (int j = 0; j < 4; ++j) y[j] = glu_f<true, EXT>(o, fmaf(g[j], f, o.bias ? __ldg(o.bias + n + j) : 0.f), fmaf(u[j], f, o.bias ? __ldg(o.bias + n + 8 + j) : 0.f));
   dense_put4(o.out, (size_t)m * o.out_ld + n / 16 * 8 + n % 8, o.out_dt == PT_DT_F32, y);
 }
 #endif

@@ -54,9 +54,9 @@ __global__ void __launch_bounds__(THREADS) gemm_f32_kernel(const float *__restri
       const float other = o.epilogue == PT_EPI_GLU ? __shfl_xor_sync(0xffffffffu, acc[i][j], 2) : 0.f;
       if (m >= M || n >= N) continue;
       if (o.epilogue == PT_EPI_GLU && n < o.split_n) {
-        if (n % 16 < 8) dense_store_glu<true>(o, m, n, acc[i][j], other);
+        if (n % 16 < 8) dense_store_glu<true, true>(o, m, n, acc[i][j], other);
       } else {
-        dense_store<true>(o, m, n, acc[i][j]);
+        dense_store<true, true>(o, m, n, acc[i][j]);
       }
     }
 }

@@ -191,9 +191,9 @@ __device__ __forceinline__ void give_up(SharedCtl &ctl, int *error_flag, int cod
 }
 
 // One finished sum of the FP8 / INT4 kernels (fp16 output) or of the BF16 kernel.
-template <bool BF16> __device__ __forceinline__ void store_out(const GemmParams &p, float acc, int m, int n) {
+template <bool BF16, bool EXT> __device__ __forceinline__ void store_out(const GemmParams &p, float acc, int m, int n) {
   if constexpr (BF16) {
-    dense_store(p.dense, m, n, acc);
+    dense_store<EXT>(p.dense, m, n, acc);
   } else {
     __half y = __float2half_rn(acc * p.out_scale);
     if (p.epilogue == PT_EPI_RESIDUAL) y = h_add(__ldcg(p.residual + (size_t)m * p.N + n), y);
@@ -202,9 +202,24 @@ template <bool BF16> __device__ __forceinline__ void store_out(const GemmParams 
   }
 }
 
+// Sixteen rows of one weight row per lane, gated: lanes n and n + 8 hold a feature's two sums.
+template <int GLU, bool EXT> __device__ __forceinline__ void glu_rows16(const GemmParams &p, const float (&sum)[16], int m, int m_end, int n, int lane) {
+  const DenseOut &d = p.dense;
+  const bool store = n < p.N && (lane & 8) == 0;
+  const float bg = store && d.bias ? __ldg(d.bias + n) : 0.f, bu = store && d.bias ? __ldg(d.bias + n + 8) : 0.f;
+  const int f = n / 16 * 8 + n % 8;
+#pragma unroll
+  for (int j = 0; j < 16; ++j) {
+    const float up = __shfl_xor_sync(0xffffffffu, sum[j], 8);
+    if (!store || m + j >= m_end) continue;
+    const float s = dense_factor<EXT>(d, m + j);
+    dense_put(d, m + j, f, glu_unit<true, GLU>(fmaf(sum[j], s, bg), fmaf(up, s, bu), d.limit));
+  }
+}
+
 // Epilogue of the warps that own the tile's rows (tensor-memory lane quarter warp % 4): `part` of `parts` warps share a quarter
 // and take alternate 16-column chunks.
-template <bool BF16>
+template <bool BF16, bool EXT>
 __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int q, int lane, int part, int parts, int n0, int m0, int m_end, int ks, int c_first = 0) {
   const int n = n0 + q * 32 + lane;
   for (int c0 = c_first + part * 16; c0 < min(p.mb, m_end - m0); c0 += 16 * parts) {
@@ -215,11 +230,9 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
     for (int j = 0; j < 16; ++j) sum[j] = __uint_as_float(v[j]);
     if constexpr (BF16) {
       if (p.ksplit == 1 && p.dense.epilogue == PT_EPI_GLU && n0 + q * 32 < p.dense.split_n) {   // (uniform over the warp)
-#pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          const float up = __shfl_xor_sync(0xffffffffu, sum[j], 8);
-          if (n < p.N && m0 + c0 + j < m_end && (lane & 8) == 0) dense_store_glu(p.dense, m0 + c0 + j, n, sum[j], up);
-        }
+        if (EXT && p.dense.glu == PT_GLU_SILU) glu_rows16<PT_GLU_SILU, EXT>(p, sum, m0 + c0, m_end, n, lane);
+        else if (EXT && p.dense.glu == PT_GLU_GELU) glu_rows16<PT_GLU_GELU, EXT>(p, sum, m0 + c0, m_end, n, lane);
+        else glu_rows16<PT_GLU_CLAMPED, EXT>(p, sum, m0 + c0, m_end, n, lane);
         continue;
       }
     }
@@ -232,7 +245,7 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
         if (p.ksplit > 1) {
           p.partial[((size_t)ks * p.M + m) * p.N + n] = acc;
         } else {
-          store_out<BF16>(p, acc, m, n);
+          store_out<BF16, EXT>(p, acc, m, n);
         }
       }
     }
@@ -295,14 +308,13 @@ __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, in
     }
   }
 }
-__device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem, int q, int lane, int n0, int m0, int m_end, int ks) {
+template <bool EXT> __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem, int q, int lane, int n0, int m0, int m_end, int ks) {
   const DenseOut &d = p.dense;
   const int nq = n0 + q * 32, n = nq + lane;
   // (warp-uniform) where this warp's 32 outputs go
   const bool second = nq >= d.split_n, glu = d.epilogue == PT_EPI_GLU && !second, f32 = second || d.out_dt == PT_DT_F32;
   // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16
-  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) && (!d.row_scale || (glu && d.glu == PT_GLU_SILU)) &&
-                    (second || f32 || d.epilogue != PT_EPI_SOFTCAP) &&
+  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) && (!EXT || ((!d.row_scale || (glu && d.glu == PT_GLU_SILU)) && (second || f32 || d.epilogue != PT_EPI_SOFTCAP))) &&
                     (f32 || glu || (d.out_ld % 2 == 0 && ((uintptr_t)d.out & 3) == 0));
   const int rows = min(p.mb, m_end - m0), whole = fast ? rows & ~31 : 0;
   for (int c0 = 0; c0 < whole; c0 += 32) {
@@ -311,13 +323,13 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
     if (second) {
       epilogue_rows32<OUT_F32, ACT_NONE>(d, d.out2, d.out2_ld, v, n - d.split_n, m0 + c0, lane);
     } else if (glu) {
-      if (d.glu == PT_GLU_SILU && d.row_scale) epilogue_rows32<OUT_GLU, PT_GLU_SILU | ACT_SCALED>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
-      else if (d.glu == PT_GLU_GELU) epilogue_rows32<OUT_GLU, PT_GLU_GELU>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
-      else if (d.glu == PT_GLU_SILU) epilogue_rows32<OUT_GLU, PT_GLU_SILU>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      if (EXT && d.glu == PT_GLU_SILU && d.row_scale) epilogue_rows32<OUT_GLU, PT_GLU_SILU | ACT_SCALED>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (EXT && d.glu == PT_GLU_GELU) epilogue_rows32<OUT_GLU, PT_GLU_GELU>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (EXT && d.glu == PT_GLU_SILU) epilogue_rows32<OUT_GLU, PT_GLU_SILU>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
       else epilogue_rows32<OUT_GLU, PT_GLU_CLAMPED>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     } else if (f32) {
       if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_F32, ACT_RELU2>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
-      else if (d.epilogue == PT_EPI_SOFTCAP) epilogue_rows32<OUT_F32, ACT_SOFTCAP>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (EXT && d.epilogue == PT_EPI_SOFTCAP) epilogue_rows32<OUT_F32, ACT_SOFTCAP>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
       else epilogue_rows32<OUT_F32, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     } else {
       if (d.epilogue == PT_EPI_GELU_MUL) epilogue_rows32<OUT_GELU_MUL, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
@@ -325,11 +337,11 @@ __device__ __forceinline__ void epilogue_bf16(const GemmParams &p, uint32_t tmem
       else epilogue_rows32<OUT_BF16, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     }
   }
-  if (whole < rows) epilogue<true>(p, tmem, q, lane, 0, 1, n0, m0, m_end, ks, whole);
+  if (whole < rows) epilogue<true, EXT>(p, tmem, q, lane, 0, 1, n0, m0, m_end, ks, whole);
 }
 
 // k-slices of this tile meet: the last CTA to arrive sums them in slice order.
-template <bool BF16>
+template <bool BF16, bool EXT>
 __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ctl, int n0, int m0, int m_end, int threads) {
   const int tid = threadIdx.x;
   __threadfence();
@@ -364,10 +376,10 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
           if (p.dense.epilogue == PT_EPI_GLU && n < p.dense.split_n) {   // gate features n % 16 < 8, their up features eight further
             if (n & 8) continue;
             const float4 gt = sum4(n), up = sum4(n + 8);
-            dense_store_glu4(p.dense, m, n, gt, up);
+            dense_store_glu4<EXT>(p.dense, m, n, gt, up);
             continue;
           }
-          dense_store4(p.dense, m, n, sum4(n));
+          dense_store4<EXT>(p.dense, m, n, sum4(n));
         }
         return;
       }
@@ -388,11 +400,11 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
       };
       if constexpr (BF16) {
         if (p.dense.epilogue == PT_EPI_GLU && n < p.dense.split_n) {
-          if (!(n & 8)) dense_store_glu(p.dense, m, n, sum1(n), sum1(n + 8));
+          if (!(n & 8)) dense_store_glu<EXT>(p.dense, m, n, sum1(n), sum1(n + 8));
           continue;
         }
       }
-      store_out<BF16>(p, sum1(n), m, n);
+      store_out<BF16, EXT>(p, sum1(n), m, n);
     }
   }
 }
@@ -400,7 +412,7 @@ __device__ __forceinline__ void reduce_slices(const GemmParams &p, SharedCtl &ct
 // ------------------------------------------------------------------------------------------ FP8 and BF16
 // Dynamic shared memory: [stage][NA A tiles of 16 KB | B tile mb * 128 B], every tile 1024-byte aligned.  NA = 2: a CTA takes 256 weight
 // rows (two accumulators), which fetches a third less per product than NA = 1; without k-slices.
-template <bool BF16, int NA>
+template <bool BF16, int NA, bool EXT>
 __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                                                                    const GemmParams p) {
   constexpr int KX = BF16 ? BKB / 2 : BKB;   // elements of k per stage
@@ -527,14 +539,14 @@ __global__ void __launch_bounds__(THREADS_F8, 1) gemm_dense_kernel(const __grid_
     fence_after();
     if (!ctl.abort && n_it > 0) {
       if constexpr (BF16) {
-        for (int a = 0; a < na; ++a) epilogue_bf16(p, tmem + a * acc_cols, warp & 3, lane, n0 + a * BM, m0, m_end, ks);
+        for (int a = 0; a < na; ++a) epilogue_bf16<EXT>(p, tmem + a * acc_cols, warp & 3, lane, n0 + a * BM, m0, m_end, ks);
       } else {
-        epilogue<false>(p, tmem, warp & 3, lane, 0, 1, n0, m0, m_end, ks);
+        epilogue<false, false>(p, tmem, warp & 3, lane, 0, 1, n0, m0, m_end, ks);
       }
     }
     fence_before();
   }
-  if (NA == 1 && p.ksplit > 1) reduce_slices<BF16>(p, ctl, n0, m0, m_end, THREADS_F8);
+  if (NA == 1 && p.ksplit > 1) reduce_slices<BF16, EXT>(p, ctl, n0, m0, m_end, THREADS_F8);
   __syncthreads();
   fence_after();
   if (warp == 1) tmem_dealloc(tmem, tmem_cols);
@@ -695,10 +707,10 @@ __global__ void __launch_bounds__(THREADS_I4, 1) gemm_int4_kernel(const __grid_c
     }
     if (!mbar_wait(sa(&ctl.accum), 0, &ctl.abort)) give_up(ctl, p.error_flag, 24);
     fence_after();
-    if (!ctl.abort && n_it > 0) epilogue<false>(p, tmem, q, lane, half, 2, n0, m0, p.M, ks);
+    if (!ctl.abort && n_it > 0) epilogue<false, false>(p, tmem, q, lane, half, 2, n0, m0, p.M, ks);
     fence_before();
   }
-  if (p.ksplit > 1) reduce_slices<false>(p, ctl, n0, m0, p.M, THREADS_I4);
+  if (p.ksplit > 1) reduce_slices<false, false>(p, ctl, n0, m0, p.M, THREADS_I4);
   __syncthreads();
   fence_after();
   if (warp == 1) tmem_dealloc(tmem, tmem_cols);
@@ -940,9 +952,11 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   }
   static bool attr_set = false;
   if (!attr_set) {
-    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<false, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<false, 1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    PT_CUDA(cudaFuncSetAttribute(tc::gemm_dense_kernel<true, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     PT_CUDA(cudaFuncSetAttribute(tc::gemm_int4_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     attr_set = true;
   }
@@ -960,10 +974,13 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = p.pdl ? 1 : 0;
-    const cudaError_t e = cudaLaunchKernelEx(&cfg, pair ? tc::gemm_dense_kernel<true, 2> : tc::gemm_dense_kernel<true, 1>, map_w, map_x, p);
+    const bool ext = dense_needs_ext(a->epilogue, a->ext);
+    const auto kernel = pair ? (ext ? tc::gemm_dense_kernel<true, 2, true> : tc::gemm_dense_kernel<true, 2, false>)
+                             : (ext ? tc::gemm_dense_kernel<true, 1, true> : tc::gemm_dense_kernel<true, 1, false>);
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, map_w, map_x, p);
     if (e != cudaSuccess) return pt::set_error(PT_ERR_CUDA, "pt_gemm: %s", cudaGetErrorString(e));
   } else
-    tc::gemm_dense_kernel<false, 1><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
+    tc::gemm_dense_kernel<false, 1, false><<<grid, tc::THREADS_F8, smem, as_stream(stream)>>>(map_w, map_x, p);
   PT_LAUNCH_CHECK("pt_gemm");
   return PT_OK;
 }

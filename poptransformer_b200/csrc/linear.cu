@@ -397,10 +397,10 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
       if constexpr (WFMT == PT_W_BF16) {
         const int n = rt * 16 + g;
         if (p.epi == PT_EPI_GLU && n < p.dense.split_n) {      // rows 0..7 of the tile are gate rows, 8..15 the matching up rows
-          if (n < p.N) dense_store_glu(p.dense, z + b, n, acc[t][jb], acc[t][2 + jb]);
+          if (n < p.N) dense_store_glu<true>(p.dense, z + b, n, acc[t][jb], acc[t][2 + jb]);
         } else {
-          if (n < p.N) dense_store(p.dense, z + b, n, acc[t][jb]);
-          if (n + 8 < p.N) dense_store(p.dense, z + b, n + 8, acc[t][2 + jb]);
+          if (n < p.N) dense_store<true>(p.dense, z + b, n, acc[t][jb]);
+          if (n + 8 < p.N) dense_store<true>(p.dense, z + b, n + 8, acc[t][2 + jb]);
         }
         continue;
       }

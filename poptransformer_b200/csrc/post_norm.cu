@@ -29,20 +29,21 @@ struct Params {
 
 template <int VEC> __device__ __forceinline__ void put_f32(float *p, const float (&v)[VEC]) { store_vec<VEC>(p, v); }
 
-template <typename T, typename E, int VEC> __global__ void post_norm_kernel(const Params p) {
+// NORM_Y: what is added is normalised (a residual step, without a second copy)
+template <typename T, typename E, int VEC, bool NORM_Y> __global__ void __launch_bounds__(1024, NORM_Y ? 2 : 1) post_norm_kernel(const Params p) {
   extern __shared__ __align__(16) float row[];     // [width]: y, then the new x
   __shared__ float red[32], pw[kMaxTop];
   __shared__ int pr[kMaxTop];
   launch_dependents();
   const int r = blockIdx.x, src = p.row_index ? p.row_index[r] : r, tid = threadIdx.x;
   float *xo = p.x_out ? p.x_out + (size_t)r * p.width : nullptr;
-  T *hrow = p.h ? reinterpret_cast<T *>(p.h) + (size_t)r * p.h_ld : nullptr, *crow = p.copy ? reinterpret_cast<T *>(p.copy) + (size_t)r * p.copy_ld : nullptr;
+  T *hrow = p.h ? reinterpret_cast<T *>(p.h) + (size_t)r * p.h_ld : nullptr, *crow = !NORM_Y && p.copy ? reinterpret_cast<T *>(p.copy) + (size_t)r * p.copy_ld : nullptr;
   if (hrow)
     for (int i = p.width + tid; i < p.h_cols; i += blockDim.x) hrow[i] = from_f<T>(0.f);     // k padding of the next product
   if (crow)
     for (int i = p.width + tid; i < p.copy_cols; i += blockDim.x) crow[i] = from_f<T>(0.f);
   const T *emb = nullptr;
-  if (p.table) {
+  if (!NORM_Y && p.table) {
     const int step = p.step ? *p.step : 0;
     const int id = min(max(p.ids[(size_t)src * p.ids_ld + step], 0), p.vocab - 1);
     emb = reinterpret_cast<const T *>(p.table) + (size_t)id * p.table_ld;
@@ -60,7 +61,7 @@ template <typename T, typename E, int VEC> __global__ void post_norm_kernel(cons
   float ss = 0.f;
   for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
     float v[VEC];
-    if (emb) {
+    if (!NORM_Y && emb) {
       load_vec<VEC>(emb + i, v);
     } else if (p.y) {
       load_vec<VEC>(p.y + (size_t)src * p.y_ld + i, v);
@@ -80,19 +81,20 @@ template <typename T, typename E, int VEC> __global__ void post_norm_kernel(cons
 #pragma unroll
     for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
   }
-  const float inv = p.norm_w ? 1.0f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps) : 1.f;     // (every thread reads back what it wrote)
+  const bool norm = NORM_Y || p.norm_w;
+  const float inv = norm ? 1.0f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps) : 1.f;     // (every thread reads back what it wrote)
   const float *x = p.x_in ? p.x_in + (size_t)src * p.width : nullptr;
   ss = 0.f;
   for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
     float v[VEC], o[VEC];
     load_vec<VEC>(row + i, v);
-    if (p.norm_w) {
+    if (norm) {
       float w[VEC];
       load_vec<VEC>(p.norm_w + i, w);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) v[j] *= inv * w[j];
     }
-    if (x) {
+    if (NORM_Y || x) {
       load_vec<VEC>(x + i, o);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) o[j] += v[j];
@@ -119,17 +121,21 @@ template <typename T, typename E, int VEC> __global__ void post_norm_kernel(cons
   }
 }
 
-template <typename T, typename E, int VEC> static int launch(const Params &p, cudaStream_t st) {
+template <typename T, typename E, int VEC, bool NORM_Y> static int launch(const Params &p, cudaStream_t st) {
   const size_t smem = (size_t)p.width * sizeof(float);
   if (smem > 48 * 1024) {
     static bool set = false;
-    if (!set) { PT_CUDA(cudaFuncSetAttribute(post_norm_kernel<T, E, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
+    if (!set) { PT_CUDA(cudaFuncSetAttribute(post_norm_kernel<T, E, VEC, NORM_Y>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
   }
   // few rows: as many threads per row as it has work for; many rows: more rows per SM
   const int want = ceil_div(ceil_div(p.width, VEC), 32) * 32, cap = p.rows <= 2 * sm_count() ? 1024 : 256;
-  post_norm_kernel<T, E, VEC><<<p.rows, std::max(64, std::min(want, cap)), smem, st>>>(p);
+  post_norm_kernel<T, E, VEC, NORM_Y><<<p.rows, std::max(64, std::min(want, cap)), smem, st>>>(p);
   PT_LAUNCH_CHECK("pt_post_norm");
   return PT_OK;
+}
+
+template <typename T, typename E, int VEC> static int launch(const Params &p, cudaStream_t st) {
+  return p.norm_w && p.x_in && !p.copy ? launch<T, E, VEC, true>(p, st) : launch<T, E, VEC, false>(p, st);
 }
 
 }  // namespace post

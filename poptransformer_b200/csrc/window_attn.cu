@@ -13,6 +13,7 @@
 //   attn_plain_kernel   any sizes, fp32 or bf16 caches, CUDA cores: the 32-bit path and the shapes the others do not take
 //   attn_prompt_kernel  bf16 prompts: 64 queries of one head per block, Q K^T and P V on the tensor cores, online softmax; only key
 //                       tiles that hold a visible key are touched
+//   (EXT instantiations of these two take a softcap and a gate)
 //   attn_decode_kernel  bf16, one token per sequence: one block per (visible page, kv head, sequence), scores and P V on the tensor
 //                       cores, pages combined by the last block to arrive; norm, rotation and append are fused
 // Scores, softmax and weights are fp32.  The tensor-core kernels multiply V with weights split into two bf16 parts (hi + lo), which
@@ -54,20 +55,21 @@ struct Params {
   int *counters;    // [n_seq, n_kv, qsplit]
 };
 
-__device__ __forceinline__ size_t page_elems(const Params &p) { return (size_t)p.n_kv * p.page * (p.v_in_k ? p.dim : p.dim + p.vdim); }
-template <typename T> __device__ __forceinline__ T *k_page(const Params &p, int phys, int g) {
-  return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems(p) + (size_t)g * p.page * p.dim;
+// (ANY: the values may be inside the keys; the tensor-core kernels do not take such pools)
+template <bool ANY> __device__ __forceinline__ size_t page_elems(const Params &p) { return (size_t)p.n_kv * p.page * (ANY && p.v_in_k ? p.dim : p.dim + p.vdim); }
+template <typename T, bool ANY = false> __device__ __forceinline__ T *k_page(const Params &p, int phys, int g) {
+  return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems<ANY>(p) + (size_t)g * p.page * p.dim;
 }
-template <typename T> __device__ __forceinline__ T *v_page(const Params &p, int phys, int g) {
-  if (p.v_in_k) return k_page<T>(p, phys, g) + p.v_col;
-  return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems(p) + (size_t)p.n_kv * p.page * p.dim + (size_t)g * p.page * p.vdim;
+template <typename T, bool ANY = false> __device__ __forceinline__ T *v_page(const Params &p, int phys, int g) {
+  if (ANY && p.v_in_k) return k_page<T, ANY>(p, phys, g) + p.v_col;
+  return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems<ANY>(p) + (size_t)p.n_kv * p.page * p.dim + (size_t)g * p.page * p.vdim;
 }
 // Scores in the units of exp2 from raw products: scale and softcap.  (tanh z = 1 - 2 / (exp(2 z) + 1))
 struct Score {
   float a, b;                // without a cap: a = scale log2(e).  With: b = cap log2(e), a = 2 scale log2(e) / cap
   bool capped;
-  __device__ __forceinline__ Score(const Params &p) {
-    capped = p.softcap > 0.f;
+  __device__ __forceinline__ Score(const Params &p, bool may_cap) {
+    capped = may_cap && p.softcap > 0.f;
     a = capped ? 2.0f * p.scale * kLog2e / p.softcap : p.scale * kLog2e;
     b = p.softcap * kLog2e;
   }
@@ -90,16 +92,16 @@ __device__ __forceinline__ int kept_pages(const Params &p, int pos) { return (mi
 // ------------------------------------------------------------------------------------------ norm, rotation, append
 // One warp, a head's row of a query or key at a time.  put(i, value) may write over src (a lane reads what it writes).
 template <typename T, typename Put>
-__device__ __forceinline__ void norm_rotate_any(const Params &p, int dim, const T *src, const float *norm, int pos, Put put) {
+__device__ __forceinline__ void norm_rotate_any(const Params &p, const T *src, const float *norm, int pos, Put put) {
   const int lane = threadIdx.x & 31, half = p.rope_half;
   float inv = 1.f;
   if (norm) {
     float ss = 0.f;
-    for (int i = lane; i < dim; i += 32) {
+    for (int i = lane; i < p.dim; i += 32) {
       const float x = to_f(src[i]);
       ss = fmaf(x, x, ss);
     }
-    inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + p.norm_eps);
+    inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.norm_eps);
   }
   auto at = [&](int i) { return to_f(src[i]) * inv * (norm ? __ldg(norm + i) : 1.f); };
   const float2 *cs = p.rope + (size_t)pos * half;
@@ -109,7 +111,7 @@ __device__ __forceinline__ void norm_rotate_any(const Params &p, int dim, const 
     put(i, u * c.x - v * c.y);
     put(i + half, v * c.x + u * c.y);
   }
-  for (int i = 2 * half + lane; i < dim; i += 32) put(i, at(i));
+  for (int i = 2 * half + lane; i < p.dim; i += 32) put(i, at(i));
 }
 // The same in registers for rows of up to 128 dimensions (p.pair_rows): a lane holds the neighbours i, i + 1 and their partners j,
 // j + 1.  Behind the rotated dimensions the partners are the next two, and the angle is zero.  Angles and weights serve all heads.
@@ -119,9 +121,9 @@ struct HeadLane {
   int i, j;
   bool on;
   float2 c0, c1, wi, wj;
-  __device__ __forceinline__ HeadLane(const Params &p, int dim, const float *norm, int pos) {
+  __device__ __forceinline__ HeadLane(const Params &p, const float *norm, int pos) {
     const int u = 2 * (threadIdx.x & 31), half = p.rope_half;
-    on = p.pair_rows && u < dim / 2;       // (nothing is loaded for rows that are taken the other way)
+    on = p.pair_rows && u < p.dim / 2;       // (nothing is loaded for rows that are taken the other way)
     i = u < half ? u : 2 * u;
     j = u < half ? u + half : 2 * u + 2;
     c0 = c1 = make_float2(1.f, 0.f);
@@ -151,13 +153,13 @@ struct HeadLane {
     store_vec<2>(dst + j, b);
   }
 };
-template <typename T> __device__ __forceinline__ void norm_rotate(const Params &p, int dim, const HeadLane &hl, const T *src, const float *norm, int pos, T *dst) {
+template <typename T> __device__ __forceinline__ void norm_rotate(const Params &p, const HeadLane &hl, const T *src, const float *norm, int pos, T *dst) {
   if (p.pair_rows) hl.run<T>(p, src, norm != nullptr, dst);
-  else norm_rotate_any<T>(p, dim, src, norm, pos, [&](int i, float y) { dst[i] = from_f<T>(y); });
+  else norm_rotate_any<T>(p, src, norm, pos, [&](int i, float y) { dst[i] = from_f<T>(y); });
 }
 
 constexpr int PREP_WARPS = 4;
-template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const Params p) {   // block: one token, warp: a head at a time
+template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32, 5) attn_prep_kernel(const Params p) {   // block: one token, warp: a head at a time
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
   if (pos < 0 || pos >= p.max_len) {
@@ -165,21 +167,20 @@ template <typename T> __global__ void __launch_bounds__(PREP_WARPS * 32) attn_pr
     return;
   }
   {
-    const int dim = p.q_norm ? p.dim : 2 * p.rope_half;       // (in place: what is not rotated stays)
-    const HeadLane hl(p, dim, p.q_norm, pos);
+    const HeadLane hl(p, p.q_norm, pos);
 #pragma unroll 4
     for (int h = warp; h < p.n_head; h += PREP_WARPS) {
       T *q = reinterpret_cast<T *>(const_cast<void *>(p.q)) + (size_t)t * p.q_ld + (size_t)h * p.dim;
-      norm_rotate<T>(p, dim, hl, q, p.q_norm, pos, q);
+      norm_rotate<T>(p, hl, q, p.q_norm, pos, q);
     }
   }
   if (!p.k) return;
-  const HeadLane hl(p, p.dim, p.k_norm, pos);
+  const HeadLane hl(p, p.k_norm, pos);
   const int phys = p.page_table[(size_t)p.slot[s] * p.max_pages + pos / p.page], at = pos % p.page;
   for (int g = warp; g < p.n_kv; g += PREP_WARPS) {
     const T *k = reinterpret_cast<const T *>(p.k) + (size_t)t * p.kv_ld + (size_t)g * p.dim, *v = reinterpret_cast<const T *>(p.v) + (size_t)t * p.kv_ld + (size_t)g * p.vdim;
     T *kc = k_page<T>(p, phys, g) + (size_t)at * p.dim, *vc = v_page<T>(p, phys, g) + (size_t)at * p.vdim;
-    norm_rotate<T>(p, p.dim, hl, k, p.k_norm, pos, kc);
+    norm_rotate<T>(p, hl, k, p.k_norm, pos, kc);
     for (int i = lane; i < p.vdim; i += 32) vc[i] = v[i];
   }
 }
@@ -249,7 +250,7 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
   for (int pg = kept > 0 ? 0 : wpage; pg <= pos / p.page; ++pg) {
     if (pg >= kept && pg < wpage) pg = wpage;
     const int k0 = pg * p.page, nk = min(p.page, pos + 1 - k0);
-    const T *K = k_page<T>(p, table[pg], g), *V = v_page<T>(p, table[pg], g);
+    const T *K = k_page<T, true>(p, table[pg], g), *V = v_page<T, true>(p, table[pg], g);
     __syncthreads();
     for (int i = warp; i < nh * nk; i += PLAIN_THREADS / 32) {
       const int h = i / nk, key = i - h * nk;
@@ -303,7 +304,7 @@ constexpr int TC_THREADS = 128, TILE = 64;   // TILE = the page size the tensor-
 // tiles (one page each) are double-buffered in shared memory; tiles without a visible key are skipped, tiles that every query of
 // the warp sees completely take no mask.  DK / DV: dim / vdim rounded up to 32, 64, 128 .. (the padding holds zeros).  CTX: keys and
 // values are rows of the context; the first shared_dim dimensions of a key belong to all heads.
-template <int DK, int DV, bool CTX> __global__ void __launch_bounds__(TC_THREADS, DK > 128 ? 2 : 3) attn_prompt_kernel(const Params p) {
+template <int DK, int DV, bool CTX, bool EXT> __global__ void __launch_bounds__(TC_THREADS, DK > 128 ? 2 : 3) attn_prompt_kernel(const Params p) {
   constexpr int KLD = DK + 8, VLD = DV + 8;
   extern __shared__ __align__(16) __nv_bfloat16 smb[];
   __nv_bfloat16 *Ks = smb, *Vs = smb + 2 * TILE * KLD;      // [2][TILE][KLD], [2][TILE][VLD]
@@ -371,7 +372,7 @@ template <int DK, int DV, bool CTX> __global__ void __launch_bounds__(TC_THREADS
   };
   const int kept = kept_pages(p, hi), wtile = window_page(p, lo), last = hi / TILE;
   auto next_tile = [&](int kt) { return (kt >= kept && kt < wtile) ? wtile : kt; };
-  const Score score(p);
+  const Score score(p, EXT);
   const float sink2 = p.sink ? p.sink[head] * kLog2e : -INFINITY;
   float o[DV / 8][4];
 #pragma unroll
@@ -407,7 +408,7 @@ template <int DK, int DV, bool CTX> __global__ void __launch_bounds__(TC_THREADS
           mma16816_bf16(sc[j + 1], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b2, b3);
         }
       const bool whole = k0 + TILE - 1 <= wlo && (p.window == 0 || whi - k0 < p.window || k0 + TILE <= p.keep_first);
-      if (score.capped) {                                         // (uniform)
+      if (EXT && score.capped) {                                  // (uniform)
 #pragma unroll
         for (int j = 0; j < TILE / 8; ++j)
 #pragma unroll
@@ -484,11 +485,11 @@ template <int DK, int DV, bool CTX> __global__ void __launch_bounds__(TC_THREADS
     inv[r] = p.out_scale / l;
   }
   __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(p.out) + (size_t)head * p.vdim + 2 * tig;
-  if (p.gate && p.gate_heads) {
+  if (EXT && p.gate && p.gate_heads) {
     if (ok0) inv[0] *= gate_at<__nv_bfloat16>(p, row0 + q0, head, 0);
     if (ok1) inv[1] *= gate_at<__nv_bfloat16>(p, row0 + q1, head, 0);
   }
-  const bool each = p.gate && !p.gate_heads;
+  const bool each = EXT && p.gate && !p.gate_heads;
 #pragma unroll
   for (int j = 0; j < DV / 8; ++j) {
     if (j * 8 >= p.vdim) break;
@@ -519,7 +520,7 @@ template <int DK, int DV, bool CTX> __global__ void __launch_bounds__(TC_THREADS
 // parts, so the split costs no extra product.  The block of the newest page takes the new key and value from the projection and
 // appends them.
 constexpr int NQ = 8;
-template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_decode_kernel(const Params p) {
+template <int DK, int DV, bool EXT> __global__ void __launch_bounds__(TC_THREADS) attn_decode_kernel(const Params p) {
   constexpr int VLD = DV + 8, QLD = DK + 32, PSLD = TILE + 8;
   typedef __nv_bfloat16 T;
   extern __shared__ __align__(16) unsigned char smd[];
@@ -575,11 +576,11 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
   asm volatile("cp.async.commit_group;" ::: "memory");
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * p.dim;
   if (p.prep) {
-    const HeadLane hq(p, p.dim, p.q_norm, pos), hk(p, p.dim, p.k_norm, pos);
+    const HeadLane hq(p, p.q_norm, pos), hk(p, p.k_norm, pos);
     for (int h = warp; h < NQ + 1; h += TC_THREADS / 32) {
       T *dst = h < NQ ? qs + h * QLD : kn;
       const bool have = h < NQ ? h < nq : owner;
-      if (have) norm_rotate<T>(p, p.dim, h < NQ ? hq : hk, h < NQ ? q + (size_t)h * p.dim : knew, h < NQ ? p.q_norm : p.k_norm, pos, dst);
+      if (have) norm_rotate<T>(p, h < NQ ? hq : hk, h < NQ ? q + (size_t)h * p.dim : knew, h < NQ ? p.q_norm : p.k_norm, pos, dst);
       for (int i = (have ? p.dim : 0) + lane; i < DK; i += 32) dst[i] = from_f<T>(0.f);
     }
   } else for (int i = tid; i < NQ * (DK / 8); i += TC_THREADS) {
@@ -613,7 +614,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
       mma16816_bf16(sc, kf[0][pp].x, kf[1][pp].x, kf[0][pp].y, kf[1][pp].y, qv.x, qv.y);
       mma16816_bf16(sc, kf[0][pp].z, kf[1][pp].z, kf[0][pp].w, kf[1][pp].w, qv.z, qv.w);
     }
-    const Score score(p);
+    const Score score(p, EXT);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {                              // keys 16 warp + g (+ 8) against heads 2 tig, 2 tig + 1
       const int key = warp * 16 + g + 8 * (e >> 1), h = 2 * tig + (e & 1);
@@ -716,7 +717,7 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[j] *= ml[2 * h];
-    if (p.gate) {
+    if (EXT && p.gate) {
       const T *gate = reinterpret_cast<const T *>(p.gate) + (size_t)t * p.gate_ld + (p.gate_heads ? h0 + h : (h0 + h) * p.vdim + c);
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[j] *= __fdividef(1.0f, 1.0f + __expf(-to_f(gate[p.gate_heads ? 0 : j])));
@@ -729,30 +730,34 @@ template <int DK, int DV> __global__ void __launch_bounds__(TC_THREADS) attn_dec
     for (int i = p.n_head * p.vdim + tid; i < p.out_cols; i += TC_THREADS) out[i] = from_f<T>(0.f);
 }
 
-template <int DK, int DV, bool CTX> static int launch_prompt(const Params &p, int longest, cudaStream_t st) {
+template <int DK, int DV, bool CTX, bool EXT> static int launch_prompt(const Params &p, int longest, cudaStream_t st) {
   constexpr size_t smem = 2 * (size_t)TILE * (DK + 8 + DV + 8) * sizeof(__nv_bfloat16);
   static bool set = false;
-  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_prompt_kernel<DK, DV, CTX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set = true; }
-  attn_prompt_kernel<DK, DV, CTX><<<dim3(ceil_div(longest, TILE), p.n_head, p.n_seq), TC_THREADS, smem, st>>>(p);
+  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_prompt_kernel<DK, DV, CTX, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set = true; }
+  attn_prompt_kernel<DK, DV, CTX, EXT><<<dim3(ceil_div(longest, TILE), p.n_head, p.n_seq), TC_THREADS, smem, st>>>(p);
   PT_LAUNCH_CHECK("pt_window_attn");
   return PT_OK;
 }
-template <int DK, int DV> static int launch_decode(const Params &p, cudaStream_t st) {
+template <int DK, int DV, bool EXT> static int launch_decode(const Params &p, cudaStream_t st) {
   const size_t smem = (size_t)(TILE * (DV + 8) + NQ * (DK + 32) + DK) * sizeof(__nv_bfloat16) + (size_t)(NQ * (TILE + 8) + NQ * 2 + NQ * p.grid_pages) * sizeof(float);
   PT_REQUIRE(smem <= 200 * 1024, "pt_window_attn: %d pages per sequence need %zu bytes of shared memory", p.grid_pages, smem);
   static bool set = false;
-  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
-  attn_decode_kernel<DK, DV><<<dim3(p.grid_pages, p.n_kv * p.qsplit, p.n_seq), TC_THREADS, smem, st>>>(p);
+  if (!set) { PT_CUDA(cudaFuncSetAttribute(attn_decode_kernel<DK, DV, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
+  attn_decode_kernel<DK, DV, EXT><<<dim3(p.grid_pages, p.n_kv * p.qsplit, p.n_seq), TC_THREADS, smem, st>>>(p);
   PT_LAUNCH_CHECK("pt_window_attn");
   return PT_OK;
 }
+template <int DK, int DV> static int dispatch_ext(const Params &p, bool decode, int longest, cudaStream_t st) {
+  if (p.softcap > 0.f || p.gate) return decode ? launch_decode<DK, DV, true>(p, st) : launch_prompt<DK, DV, false, true>(p, longest, st);
+  return decode ? launch_decode<DK, DV, false>(p, st) : launch_prompt<DK, DV, false, false>(p, longest, st);
+}
 template <int DK> static int dispatch_v(const Params &p, bool decode, int longest, cudaStream_t st) {
-  if (p.vdim <= 32) return decode ? launch_decode<DK, 32>(p, st) : launch_prompt<DK, 32, false>(p, longest, st);
-  if (p.vdim <= 64) return decode ? launch_decode<DK, 64>(p, st) : launch_prompt<DK, 64, false>(p, longest, st);
-  return decode ? launch_decode<DK, 128>(p, st) : launch_prompt<DK, 128, false>(p, longest, st);
+  if (p.vdim <= 32) return dispatch_ext<DK, 32>(p, decode, longest, st);
+  if (p.vdim <= 64) return dispatch_ext<DK, 64>(p, decode, longest, st);
+  return dispatch_ext<DK, 128>(p, decode, longest, st);
 }
 template <int DK> static int dispatch_ctx(const Params &p, int longest, cudaStream_t st) {
-  return p.vdim <= 64 ? launch_prompt<DK, 64, true>(p, longest, st) : launch_prompt<DK, 128, true>(p, longest, st);
+  return p.vdim <= 64 ? launch_prompt<DK, 64, true, true>(p, longest, st) : launch_prompt<DK, 128, true, true>(p, longest, st);
 }
 static int dispatch_tc(const Params &p, bool decode, int longest, cudaStream_t st) {
   if (p.dim <= 32) return dispatch_v<32>(p, decode, longest, st);
@@ -818,7 +823,7 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
   {
     const int pair = a->dtype == PT_DT_F32 ? 8 : 4;
     auto al = [](const void *x, int bytes) { return ((uintptr_t)x & (bytes - 1)) == 0; };
-    p.pair_rows = a->dim % 4 == 0 && (ctx && !a->q_norm ? a->rope_dims : a->dim) <= 128 && a->rope_dims % 4 == 0 && a->q_ld % 2 == 0 && a->n_kv * a->page_size * (p.v_in_k ? a->dim : a->dim + a->vdim) % 2 == 0 && al(a->q, pair) && al(a->pool, pair) && al(a->rope, 16) && al(a->q_norm, 8) &&
+    p.pair_rows = a->dim % 4 == 0 && a->dim <= 128 && a->rope_dims % 4 == 0 && a->q_ld % 2 == 0 && a->n_kv * a->page_size * (p.v_in_k ? a->dim : a->dim + a->vdim) % 2 == 0 && al(a->q, pair) && al(a->pool, pair) && al(a->rope, 16) && al(a->q_norm, 8) &&
                   al(a->k_norm, 8) && (!a->k || (a->kv_ld % 2 == 0 && al(a->k, pair)));
   }
   PT_REQUIRE(a->rope_dims >= 0 && a->rope_dims % 2 == 0 && a->rope_dims <= a->dim && (!a->rope_dims || a->rope), "pt_window_attn: %d rotated dimensions of %d",
