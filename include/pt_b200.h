@@ -626,13 +626,14 @@ typedef struct pt_window_attn_args {
   int gate_ld, gate_per_head; /* n_head * vdim columns, or one per head              */
   int values_in_keys;     /* the pool holds keys only; values are dimensions value_col .. value_col + vdim - 1 of them */
   int value_col;
+  int row_ld;             /* ... elements between its rows, and between the heads of q (0 = dim) */
   const pt_context_rows *context; /* prompts: where keys and values are instead of the pool, or NULL */
 } pt_window_attn_args;
 size_t pt_window_attn_workspace_bytes(int n_seq, int n_head, int vdim, int page_size, int max_len, int window, int keep_first);
 int pt_window_attn(const pt_window_attn_args *args, void *stream);
 
 /* Attention over a latent (csrc/latent.cu).  A cached row is [rot_dim rotated key dimensions, shared by all heads | rank latent
- * dimensions]; pool [pages][page_size][rot_dim + rank], one page numbering with the other caches.
+ * dimensions] and padding: pt_latent_row elements; pool [pages][page_size][pt_latent_row], one page numbering with the other caches.
  * pt_latent_prep: cq <- rms_norm(q) * q_norm (columns q_rank .. cq_ld - 1 zeroed); the row of every token <- [rotation of kv[rank ..] |
  * rms_norm(kv[.. rank]) * kv_norm].  rope: (cos, sin) of rope[position][i] for the pair (i, i + rot_dim / 2). */
 typedef struct pt_latent_prep_args {
@@ -651,6 +652,7 @@ typedef struct pt_latent_prep_args {
   int page_size, max_pages, max_len;
   int32_t *error_flag;    /* optional, set to 12 when a position has no page         */
 } pt_latent_prep_args;
+int pt_latent_row(int rot_dim, int rank);
 int pt_latent_prep(const pt_latent_prep_args *args, void *stream);
 
 /* The cached rows of every sequence's context (bf16), sequence after sequence: shared [n_ctx, rot_dim], latent [n_ctx, latent_ld] (padding

@@ -83,7 +83,7 @@ class WindowAttnArgs(ctypes.Structure):
                 ("pool", c_void_p), ("page_table", c_void_p), ("out", c_void_p), ("out_ld", c_int), ("max_tokens_per_seq", c_int), ("max_len", c_int),
                 ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("error_flag", c_void_p), ("q_norm", c_void_p), ("k_norm", c_void_p),
                 ("norm_eps", c_float), ("rope_dims", c_int), ("rope", c_void_p), ("out_scale", c_float), ("out_cols", c_int),
-                ("softcap", c_float), ("gate", c_void_p), ("gate_ld", c_int), ("gate_per_head", c_int), ("values_in_keys", c_int), ("value_col", c_int),
+                ("softcap", c_float), ("gate", c_void_p), ("gate_ld", c_int), ("gate_per_head", c_int), ("values_in_keys", c_int), ("value_col", c_int), ("row_ld", c_int),
                 ("context", ctypes.POINTER(ContextRows))]
 
 
@@ -172,6 +172,7 @@ SIGNATURES = {
     "pt_hyper": (c_int, [ctypes.POINTER(HyperArgs), c_void_p]),
     "pt_window_attn_workspace_bytes": (c_size_t, [c_int] * 7),
     "pt_window_attn": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),
+    "pt_latent_row": (c_int, [c_int] * 2),
     "pt_latent_prep": (c_int, [ctypes.POINTER(LatentPrepArgs), c_void_p]),
     "pt_latent_context": (c_int, [ctypes.POINTER(LatentContextArgs), c_void_p]),
     "pt_latent_attn_workspace_bytes": (c_size_t, [c_int] * 5),

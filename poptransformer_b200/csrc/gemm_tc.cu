@@ -29,6 +29,7 @@
 #include <cstring>
 
 #include "dense_out.cuh"
+#include "mbarrier.cuh"
 #include "tile_math.cuh"
 
 namespace pt {
@@ -40,10 +41,6 @@ constexpr int THREADS_F8 = 192;    // warp 0: producer, warp 1: MMA + tensor-mem
 constexpr int THREADS_I4 = 352;    // warp 0: raw-tile producer, warp 1: MMA, warps 2-9: transform + epilogue, warp 10: activation producer
 constexpr int A_TILE = BM * BKB;   // 16 KB: 128 rows x 128 bytes of k, 128-byte swizzle
 constexpr int RAW_TILE = BM * 32;  // 4 KB: 128 rows x 64 k of packed nibbles
-constexpr int WAIT_LIMIT = 1 << 22;
-#ifndef PT_TC_HINT
-#define PT_TC_HINT 1000   // suspend-time hint (ns) of the barrier waits; negative: plain polling with test_wait
-#endif
 
 struct GemmParams {
   int M, N, K;
@@ -74,38 +71,9 @@ struct GemmParams {
 
 // ------------------------------------------------------------------------------------------ PTX
 __device__ __forceinline__ uint32_t sa(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void mbar_init(uint32_t bar, int count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count)); }
-__device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(uint32_t bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory"); }
-// Bounded wait; gives up at once when the CTA has already recorded a failure.
-__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int *abort_flag) {
-  for (int it = 0; it < WAIT_LIMIT; ++it) {
-    uint32_t ok;
-#if PT_TC_HINT < 0
-    asm volatile("{\n\t.reg .pred p;\n\tmbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-                 : "=r"(ok)
-                 : "r"(bar), "r"(parity)
-                 : "memory");
-#else
-    asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2, %3;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-                 : "=r"(ok)
-                 : "r"(bar), "r"(parity), "r"((uint32_t)PT_TC_HINT)
-                 : "memory");
-#endif
-    if (ok) return true;
-    if (*abort_flag) return false;
-  }
-  return false;
-}
 __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap *map, int x, int y, uint32_t bar) {
   asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];" ::"r"(dst), "l"(map),
                "r"(bar), "r"(x), "r"(y)
-               : "memory");
-}
-__device__ __forceinline__ void bulk_g2s(uint32_t dst, const void *src, uint32_t bytes, uint32_t bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar)
                : "memory");
 }
 __device__ __forceinline__ void tmem_alloc(uint32_t dst_smem, uint32_t ncols) {

@@ -18,6 +18,7 @@
 #include <type_traits>
 
 #include "chunk.cuh"
+#include "mbarrier.cuh"
 
 namespace pt {
 namespace lat {
@@ -43,7 +44,7 @@ template <typename... A, typename... B> static cudaError_t launch_early(void (*k
 
 // ------------------------------------------------------------------------------------------ norms, rotation, append
 struct PrepParams {
-  int q_rank, rank, rot, page, max_pages, max_len, ld, cq_ld;
+  int q_rank, rank, rot, row_ld, page, max_pages, max_len, ld, cq_ld;
   float eps;
   const void *q, *kv;                // columns of the projection's rows: the query latent; [latent | key part]
   const float *q_norm, *kv_norm;
@@ -84,7 +85,7 @@ template <typename T, int VEC> __global__ void __launch_bounds__(PREP_THREADS) p
     if (at == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
   }
-  T *row = reinterpret_cast<T *>(p.pool) + ((size_t)phys * p.page + pos % p.page) * (p.rot + p.rank);
+  T *row = reinterpret_cast<T *>(p.pool) + ((size_t)phys * p.page + pos % p.page) * p.row_ld;
   T *out = second ? row + p.rot : reinterpret_cast<T *>(p.cq) + (size_t)t * p.cq_ld;
   for (int i = at * VEC; i < n; i += HALF * VEC) {
     float v[VEC], w[VEC];
@@ -104,12 +105,13 @@ template <typename T, int VEC> __global__ void __launch_bounds__(PREP_THREADS) p
     row[i] = from_f<T>(u * c.x - v * c.y);
     row[half + i] = from_f<T>(v * c.x + u * c.y);
   }
+  for (int i = p.rot + p.rank + at; i < p.row_ld - 8; i += HALF) row[i] = from_f<T>(0.f);      // (products go in steps of 16)
 }
 
 // ------------------------------------------------------------------------------------------ the whole context
 // One warp per context row, 16-byte units.
 __global__ void context_kernel(const uint4 *pool, const int *page_table, const int *slot, const int *ctx_cu, int n_seq, int n_ctx, int page, int max_pages,
-                               int rot_units, int units, uint4 *shared, uint4 *latent, int latent_units) {
+                               int rot_units, int units, int row_units, uint4 *shared, uint4 *latent, int latent_units) {
   const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (r >= n_ctx) return;
   int lo = 0, hi = n_seq - 1;
@@ -119,7 +121,7 @@ __global__ void context_kernel(const uint4 *pool, const int *page_table, const i
     else hi = mid - 1;
   }
   const int pos = r - ctx_cu[lo];
-  const uint4 *src = pool + ((size_t)page_table[(size_t)slot[lo] * max_pages + pos / page] * page + pos % page) * units;
+  const uint4 *src = pool + ((size_t)page_table[(size_t)slot[lo] * max_pages + pos / page] * page + pos % page) * row_units;
   for (int i = lane; i < rot_units + latent_units; i += 32) {
     const uint4 v = i < units ? src[i] : make_uint4(0, 0, 0, 0);
     if (i < rot_units) shared[(size_t)r * rot_units + i] = v;
@@ -129,8 +131,8 @@ __global__ void context_kernel(const uint4 *pool, const int *page_table, const i
 
 // ------------------------------------------------------------------------------------------ attention
 struct Params {
-  int n_tok, n_head, dim, rot, vdim, rank, width, width_pad, q_ld, max_pages, max_len, gate_ld, out_ld, out_cols;   // width = rot + rank
-  int n_split, ng;                   // runs of pages; expand: groups of 16 outputs per block
+  int n_tok, n_head, dim, rot, vdim, rank, width, row_ld, q_ld, max_pages, max_len, gate_ld, out_ld, out_cols;   // width = rot + rank, row_ld: cached rows, q_cat rows
+  int n_split, slots, ng;            // runs of pages; slots of the ring; expand: groups of 16 outputs per block
   float scale;
   const void *q, *w_k, *w_v, *gate, *pool;
   const float2 *rope;
@@ -159,7 +161,7 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) absorb_pl
   const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
   if (pos < 0 || pos >= p.max_len) return;         // (reported where the position is cached)
-  T *dst = reinterpret_cast<T *>(p.q_cat) + ((size_t)t * p.n_head + h) * p.width;
+  T *dst = reinterpret_cast<T *>(p.q_cat) + ((size_t)t * p.n_head + h) * p.row_ld;
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h * (p.rot + p.dim) + p.rot;
   const T *w = reinterpret_cast<const T *>(p.w_k) + (size_t)h * p.rank * p.dim;
   for (int i = tid; i < p.rot / 2; i += PLAIN_THREADS) rotate_query<T>(p, t, h, pos, i, dst);
@@ -219,13 +221,17 @@ __global__ void __launch_bounds__(ABSORB_WARPS * 32) absorb_kernel(const Params 
   Frag128 wf, xf;
   load128(wf, w0, w1, 0, p.dim, tig, n0 + g < p.rank, n0 + 8 + g < p.rank, true);
   wait_for_prerequisites();
-  if (blockIdx.x == 0)
+  if (blockIdx.x == 0) {
+    const int pad = p.row_ld - 8 - p.width;          // (products go in steps of 16)
+    for (int i = tid; i < 16 * pad; i += blockDim.x)
+      if (t0 + i / pad < p.n_tok) reinterpret_cast<bf *>(p.q_cat)[((size_t)(t0 + i / pad) * p.n_head + h) * p.row_ld + p.width + i % pad] = from_f<bf>(0.f);
     for (int i = tid; i < 16 * (p.rot / 2); i += blockDim.x) {
       const int m = i / (p.rot / 2), t = t0 + m;
       if (t >= p.n_tok) break;
       const int pos = p.start[t];
-      if (pos >= 0 && pos < p.max_len) rotate_query<bf>(p, t, h, pos, i % (p.rot / 2), reinterpret_cast<bf *>(p.q_cat) + ((size_t)t * p.n_head + h) * p.width);
+      if (pos >= 0 && pos < p.max_len) rotate_query<bf>(p, t, h, pos, i % (p.rot / 2), reinterpret_cast<bf *>(p.q_cat) + ((size_t)t * p.n_head + h) * p.row_ld);
     }
+  }
   const bool ok0 = t0 + g < p.n_tok, ok1 = t0 + g + 8 < p.n_tok;
   const bf *x0 = reinterpret_cast<const bf *>(p.q) + (size_t)(t0 + g) * p.q_ld + (size_t)h * (p.rot + p.dim) + p.rot, *x1 = x0 + (size_t)8 * p.q_ld;
   float acc[2][4] = {};
@@ -238,9 +244,9 @@ __global__ void __launch_bounds__(ABSORB_WARPS * 32) absorb_kernel(const Params 
   for (int j = 0; j < 2; ++j) {
     const int n = n0 + 8 * j + 2 * tig;
     if (n >= p.rank) continue;               // (rank is a multiple of 8)
-    bf *o = reinterpret_cast<bf *>(p.q_cat) + ((size_t)(t0 + g) * p.n_head + h) * p.width + p.rot + n;
+    bf *o = reinterpret_cast<bf *>(p.q_cat) + ((size_t)(t0 + g) * p.n_head + h) * p.row_ld + p.rot + n;
     if (ok0) *reinterpret_cast<uint32_t *>(o) = pack_bf2(acc[j][0], acc[j][1]);
-    if (ok1) *reinterpret_cast<uint32_t *>(o + (size_t)8 * p.n_head * p.width) = pack_bf2(acc[j][2], acc[j][3]);
+    if (ok1) *reinterpret_cast<uint32_t *>(o + (size_t)8 * p.n_head * p.row_ld) = pack_bf2(acc[j][2], acc[j][3]);
   }
 }
 
@@ -366,19 +372,26 @@ __global__ void __launch_bounds__(EXPAND_WARPS * 32) expand_kernel(const Params 
 
 // ------------------------------------------------------------------------------------------ one token per sequence
 // Block: one run of pages of one sequence, 16 MT heads.  The rows [rotated part | latent] of a page lie once in shared memory and serve
-// as keys (warps w and w + 8: keys 8 w .., half of the row each) and, from column rot on, as values (warp w: latent dimensions 8 NT w ..).
-constexpr int DEC_WARPS = 16, DEC_THREADS = DEC_WARPS * 32, P_LD = TILE + 8;
-template <int MT> static size_t decode_smem(int width_pad) {
-  return (size_t)(16 * MT + 2 * TILE) * (width_pad + 8) * sizeof(bf) + (size_t)16 * MT * (P_LD * (2 * sizeof(float) + 2 * sizeof(bf)) + sizeof(float));
+// as keys and, from column rot on, as values; one bulk copy brings half a page into a slot of a ring (a block computes on two slots while
+// the others fill).  Rows are an odd number of 16-byte units long, so that eight of them meet in no bank.  Scores: warp (a quarter of the
+// row's dimensions, 8 KT keys), its part of the queries stays in registers (S steps of 32 dimensions); the quarters' sums meet in shared
+// memory.  Weighted sum: warp w takes latent dimensions 8 NT w ...
+constexpr int PARTS = 4, P_LD = TILE + 8, HALF = TILE / 2, kMaxSlots = 8;
+template <int MT> static size_t decode_smem(int row_ld, int slots) {
+  return (size_t)slots * HALF * row_ld * sizeof(bf) + (size_t)16 * MT * (P_LD * (PARTS * sizeof(float) + 2 * sizeof(bf)) + sizeof(float));
 }
-template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) decode_kernel(const Params p) {
-  constexpr int HB = 16 * MT;
+constexpr size_t kSmemLimit = 226 * 1024;
+constexpr int kMinSlots = 4;
+template <int MT, int NT, int S, int WARPS> __global__ void __launch_bounds__(WARPS * 32, 1) decode_kernel(const Params p) {
+  constexpr int HB = 16 * MT, KT = TILE / 8 / (WARPS / PARTS), THREADS = WARPS * 32;   // KT: groups of eight keys per warp
   extern __shared__ __align__(16) unsigned char sm_raw[];
-  const int ld = p.width_pad + 8;
-  bf *qs = reinterpret_cast<bf *>(sm_raw), *ks = qs + HB * ld;              // [HB][ld], [2][TILE][ld]
-  float *ps = reinterpret_cast<float *>(ks + 2 * TILE * ld);                // [2][HB][P_LD] scores, the two halves' sums
-  bf *ph = reinterpret_cast<bf *>(ps + 2 * HB * P_LD), *pl = ph + HB * P_LD;    // [HB][P_LD] the weights' two parts
+  const int ld = p.row_ld, k_end = ld - 8;        // k_end: the row's dimensions, a multiple of 16
+  bf *ks = reinterpret_cast<bf *>(sm_raw);                                  // [slots][HALF][ld]
+  float *ps = reinterpret_cast<float *>(ks + p.slots * HALF * ld);          // [PARTS][HB][P_LD]
+  bf *ph = reinterpret_cast<bf *>(ps + PARTS * HB * P_LD), *pl = ph + HB * P_LD;   // [HB][P_LD] the weights' two parts
   float *corr = reinterpret_cast<float *>(pl + HB * P_LD);                  // [HB]
+  __shared__ uint64_t full[kMaxSlots], q_full;
+  __shared__ volatile int abort_flag;
   launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3;
   const int t = blockIdx.z, h0 = blockIdx.y * HB, nh = min(HB, p.n_head - h0), x = blockIdx.x;
@@ -391,83 +404,116 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
   const int n_pages = pos / TILE + 1, per = pages_per_run(n_pages, p.n_split), pg0 = x * per, pg1 = min(n_pages, pg0 + per);
   if (pg0 >= pg1) return;
   const int *table = p.page_table + (size_t)p.slot[t] * p.max_pages;
-  const int units = p.width_pad / 8;
-  auto load_page = [&](int pg, int stage) {
-    const bf *src = reinterpret_cast<const bf *>(p.pool) + (size_t)table[pg] * TILE * p.width;
-    bf *dst = ks + stage * TILE * ld;
-#pragma unroll 2
-    for (int r = warp; r < TILE; r += DEC_WARPS) {
-      const bool row_in = pg * TILE + r <= pos;
-      for (int u = lane; u < units; u += 32) {
-        const bool in = row_in && u * 8 < p.width;
-        cp16(dst + r * ld + u * 8, src + (in ? (size_t)r * p.width + u * 8 : 0), in);
-      }
+  const int first = pg0 * TILE, halves = (min(pg1 * TILE, pos + 1) - first + HALF - 1) / HALF;
+  int issued = 0, fill_slot = 0, phys = table[pg0];
+  auto load_half = [&]() {                        // the next half page of the run into the next slot
+    const int rows = min(HALF, pos + 1 - first - issued * HALF);      // rows behind the newest position: zeros (their weights are zero, but what is multiplied must be a number)
+    bf *dst = ks + fill_slot * HALF * ld;
+    if (tid == 0) {
+      const uint32_t bar = smem_addr(&full[fill_slot]), bytes = (uint32_t)(rows * ld * sizeof(bf));
+      mbar_expect_tx(bar, bytes);
+      bulk_g2s(smem_addr(dst), reinterpret_cast<const bf *>(p.pool) + ((size_t)phys * TILE + (issued & 1) * HALF) * ld, bytes, bar);
+      if (issued & 1) phys = table[min(pg0 + (issued + 1) / 2, pg1 - 1)];
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    for (int r = rows + warp; r < HALF; r += WARPS)
+      for (int i = lane; i < ld / 2; i += 32) reinterpret_cast<uint32_t *>(dst + r * ld)[i] = 0u;
+    ++issued;
+    if (++fill_slot == p.slots) fill_slot = 0;
   };
-  for (int r = warp; r < HB; r += DEC_WARPS)
-    for (int u = lane; u < units; u += 32) {
-      const bool in = r < nh && u * 8 < p.width;
-      const bf *src = reinterpret_cast<const bf *>(p.q_cat) + ((size_t)t * p.n_head + h0) * p.width;
-      cp16(qs + r * ld + u * 8, src + (in ? (size_t)r * p.width + u * 8 : 0), in);
-    }
-  load_page(pg0, 0);
-  const float sc2 = p.scale * kLog2e;
-  float m_run[MT], l_run[MT];                     // heads MT warp .. (the same in all lanes)
+  if (tid == 0) {
+    abort_flag = 0;
+    for (int i = 0; i < kMaxSlots; ++i) mbar_init(smem_addr(&full[i]), 1);
+    mbar_init(smem_addr(&q_full), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    // the queries pass through the last slot
+    const uint32_t bytes = (uint32_t)(nh * ld * sizeof(bf));
+    mbar_expect_tx(smem_addr(&q_full), bytes);
+    bulk_g2s(smem_addr(ks + (p.slots - 1) * HALF * ld), reinterpret_cast<const bf *>(p.q_cat) + ((size_t)t * p.n_head + h0) * ld, bytes, smem_addr(&q_full));
+  }
+  __syncthreads();
+  while (issued < min(halves, p.slots - 1)) load_half();
+  const int part = warp & (PARTS - 1), keys = warp / PARTS * (KT * 8), k0 = part * S * 32;   // this warp's scores: dimensions k0 .., keys keys ..
+  auto failed = [&]() {
+    if (!abort_flag && p.error_flag) atomicCAS(p.error_flag, 0, 11);
+    abort_flag = 1;
+  };
+  if (!mbar_wait(smem_addr(&q_full), 0, &abort_flag)) failed();
+  uint32_t qa[MT][2 * S][4];
+  {
+    const uint32_t q_lane = smem_addr(ks + ((p.slots - 1) * HALF + (lane & 15)) * ld + k0 + (lane >> 4) * 8);
 #pragma unroll
-  for (int i = 0; i < MT; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int kk = 0; kk < 2 * S; ++kk) {
+        qa[mt][kk][0] = qa[mt][kk][1] = qa[mt][kk][2] = qa[mt][kk][3] = 0u;
+        if (k0 + kk * 16 < k_end) ldsm4(q_lane + (uint32_t)(mt * 16 * ld + kk * 16) * 2u, qa[mt][kk][0], qa[mt][kk][1], qa[mt][kk][2], qa[mt][kk][3]);
+      }
+  }
+  __syncthreads();
+  if (issued < halves) load_half();
+  const float sc2 = p.scale * kLog2e;
+  constexpr int ROWS = HB / WARPS;
+  float m_run[ROWS], l_run[ROWS];                 // heads ROWS warp .. (the same in all lanes)
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
   float o[MT][NT][4];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
     for (int j = 0; j < NT; ++j) o[mt][j][0] = o[mt][j][1] = o[mt][j][2] = o[mt][j][3] = 0.f;
   const int c0 = warp * NT * 8;                   // this warp's latent dimensions
-  int stage = 0;
-  for (int pg = pg0; pg < pg1; ++pg, stage ^= 1) {
-    if (pg + 1 < pg1) {
-      load_page(pg + 1, stage ^ 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();
-    const bf *K = ks + stage * TILE * ld;
-    {
-      float sc[MT][2][4] = {};
-      const int keys = (warp & 7) * 8, part = warp >> 3, steps = p.width_pad / 32, k0 = part ? (steps + 1) / 2 * 32 : 0, k1 = part ? p.width_pad : (steps + 1) / 2 * 32;
-      const uint32_t k_lane = smem_addr(K + (keys + (lane & 7)) * ld + (lane >> 3) * 8);     // matrices: k 0-7, 8-15, 16-23, 24-31 of eight keys
-      const uint32_t q_lane = smem_addr(qs + (lane & 15) * ld + (lane >> 4) * 8);
-#pragma unroll 3
-      for (int k = k0; k < k1; k += 32) {
-        uint32_t b0, b1, b2, b3;
-        ldsm4(k_lane + k * 2u, b0, b1, b2, b3);
+  int slot0 = 0, turn0 = 0;                       // of the tile's first half: its slot, and how often the ring was used up before
+  for (int h = 0; h < halves; h += 2) {
+    const int slot1 = slot0 + 1 == p.slots ? 0 : slot0 + 1, turn1 = turn0 + (slot1 == 0);
+    const bool two = h + 1 < halves;
+    if (!mbar_wait(smem_addr(&full[slot0]), turn0 & 1, &abort_flag) || (two && !mbar_wait(smem_addr(&full[slot1]), turn1 & 1, &abort_flag))) failed();
+    const bf *K0 = ks + slot0 * HALF * ld, *K1 = ks + slot1 * HALF * ld;
+    if (two || keys < HALF) {
+      float sc[MT][KT][4] = {};
+      const uint32_t k_lane = smem_addr((keys < HALF ? K0 : K1) + ((keys & (HALF - 1)) + (lane & 7)) * ld + k0 + (lane >> 3) * 8);     // matrices: k 0-7, 8-15, 16-23, 24-31 of eight keys
 #pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          uint32_t a0, a1, a2, a3;
-          const uint32_t qa = q_lane + (uint32_t)(mt * 16 * ld + k) * 2u;
-          ldsm4(qa, a0, a1, a2, a3);
-          mma16816_bf16(sc[mt][0], a0, a1, a2, a3, b0, b1);
-          ldsm4(qa + 32u, a0, a1, a2, a3);
-          mma16816_bf16(sc[mt][1], a0, a1, a2, a3, b2, b3);
+      for (int s = 0; s < S; ++s) {
+        if (k0 + s * 32 >= k_end) break;          // (uniform over the warp)
+        const bool both = k0 + s * 32 + 16 < k_end;
+#pragma unroll
+        for (int j = 0; j < KT; ++j) {
+          uint32_t b0, b1, b2, b3;
+          ldsm4(k_lane + (uint32_t)(j * 8 * ld + s * 32) * 2u, b0, b1, b2, b3);
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            const uint32_t(&a)[4] = qa[mt][2 * s], (&b)[4] = qa[mt][2 * s + 1];
+            mma16816_bf16(sc[mt][j], a[0], a[1], a[2], a[3], b0, b1);
+            if (both) mma16816_bf16(sc[mt][j], b[0], b[1], b[2], b[3], b2, b3);
+          }
         }
       }
-      const int key = keys + 2 * tig, seen = pos - pg * TILE;           // keys 0 .. seen of this page
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const float a = (sc[mt][0][2 * r] + sc[mt][1][2 * r]) * sc2, b = (sc[mt][0][2 * r + 1] + sc[mt][1][2 * r + 1]) * sc2;
-          *reinterpret_cast<float2 *>(ps + (part * HB + mt * 16 + g + 8 * r) * P_LD + key) = make_float2(key <= seen ? a : -INFINITY, key + 1 <= seen ? b : -INFINITY);
-        }
+        for (int j = 0; j < KT; ++j)
+#pragma unroll
+          for (int r = 0; r < 2; ++r)
+            *reinterpret_cast<float2 *>(ps + (part * HB + mt * 16 + g + 8 * r) * P_LD + keys + j * 8 + 2 * tig) = make_float2(sc[mt][j][2 * r], sc[mt][j][2 * r + 1]);
     }
     __syncthreads();
+    if (abort_flag) {                             // (the same for the whole block) what is still in flight lands before the block ends
+      mbar_wait_all(smem_addr(&q_full), 0);
+      for (int i = h; i < issued; ++i) mbar_wait_all(smem_addr(&full[i % p.slots]), (i / p.slots) & 1);
+      return;
+    }
+    const int seen = pos - first - h * HALF;      // keys 0 .. seen of this tile
 #pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const int r = warp * MT + i;
-      float2 v = *reinterpret_cast<const float2 *>(ps + r * P_LD + 2 * lane);
-      const float2 v2 = *reinterpret_cast<const float2 *>(ps + (HB + r) * P_LD + 2 * lane);
-      v.x += v2.x;
-      v.y += v2.y;
+    for (int i = 0; i < ROWS; ++i) {
+      const int r = warp * ROWS + i;
+      float2 v = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int j = 0; j < PARTS; ++j) {
+        const float2 part_sum = *reinterpret_cast<const float2 *>(ps + (j * HB + r) * P_LD + 2 * lane);
+        v.x += part_sum.x;
+        v.y += part_sum.y;
+      }
+      v.x = 2 * lane <= seen ? v.x * sc2 : -INFINITY;
+      v.y = 2 * lane + 1 <= seen ? v.y * sc2 : -INFINITY;
       const float m = fmaxf(m_run[i], warp_max(fmaxf(v.x, v.y)));           // (a page of a run holds at least one visible key)
       const float a = exp2f(v.x - m), b = exp2f(v.y - m), c = exp2f(m_run[i] - m);
       uint32_t hi, lo;
@@ -488,10 +534,11 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
         o[mt][j][2] *= c_hi; o[mt][j][3] *= c_hi;
       }
     }
-    const uint32_t v_lane = smem_addr(K + (lane & 15) * ld + p.rot + c0 + (lane >> 4) * 8);
+    const uint32_t v_off = (uint32_t)((lane & 15) * ld + p.rot + c0 + (lane >> 4) * 8) * 2u, v_lane0 = smem_addr(K0) + v_off, v_lane1 = smem_addr(K1) + v_off;
     const uint32_t h_lane = smem_addr(ph + (lane & 15) * P_LD + (lane >> 4) * 8), l_lane = smem_addr(pl + (lane & 15) * P_LD + (lane >> 4) * 8);
 #pragma unroll
     for (int k2 = 0; k2 < TILE / 16; ++k2) {
+      if (k2 * 16 >= HALF && !two) break;         // (uniform)
       uint32_t h[MT][4], l[MT][4];
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
@@ -502,7 +549,7 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
       for (int jn = 0; jn < NT; jn += 2) {
         if (c0 + jn * 8 >= p.rank) break;         // (uniform over the warp)
         uint32_t b0, b1, b2, b3;
-        ldsm4t(v_lane + (uint32_t)(k2 * 16 * ld + jn * 8) * 2u, b0, b1, b2, b3);
+        ldsm4t((k2 * 16 < HALF ? v_lane0 : v_lane1) + (uint32_t)((k2 * 16 & (HALF - 1)) * ld + jn * 8) * 2u, b0, b1, b2, b3);
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           mma16816_bf16(o[mt][jn], h[mt][0], h[mt][1], h[mt][2], h[mt][3], b0, b1);
@@ -512,7 +559,11 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
         }
       }
     }
-    __syncthreads();                              // the stage may be refilled
+    __syncthreads();                              // both slots may be refilled
+    if (issued < halves) load_half();
+    if (issued < halves) load_half();
+    turn0 = turn1 + (slot1 + 1 == p.slots);
+    slot0 = slot1 + 1 == p.slots ? 0 : slot1 + 1;
   }
   const size_t head0 = (size_t)t * p.n_head + h0;
 #pragma unroll
@@ -527,33 +578,38 @@ template <int MT, int NT> __global__ void __launch_bounds__(DEC_THREADS, 1) deco
         if (c0 + j * 8 < p.rank) *reinterpret_cast<float2 *>(dst + j * 8) = make_float2(o[mt][j][2 * r], o[mt][j][2 * r + 1]);
     }
 #pragma unroll
-  for (int i = 0; i < MT; ++i) {
-    const int row = warp * MT + i;
+  for (int i = 0; i < ROWS; ++i) {
+    const int row = warp * ROWS + i;
     if (lane == 0 && row < nh) p.ws_ml[(head0 + row) * p.n_split + x] = make_float2(m_run[i], l_run[i]);
   }
 }
 
-template <int MT, int NT> static int launch_decode(const Params &p, cudaStream_t st) {
-  const size_t smem = decode_smem<MT>(p.width_pad);
+template <int MT, int NT, int S, int WARPS> static int launch_decode(Params p, cudaStream_t st) {
+  p.slots = kMaxSlots;
+  while (p.slots > kMinSlots && decode_smem<MT>(p.row_ld, p.slots) > kSmemLimit) --p.slots;
+  const size_t smem = decode_smem<MT>(p.row_ld, p.slots);
   static bool set = false;
-  if (!set) { PT_CUDA(cudaFuncSetAttribute(decode_kernel<MT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)); set = true; }
-  PT_CUDA(launch_early(decode_kernel<MT, NT>, dim3(p.n_split, ceil_div(p.n_head, 16 * MT), p.n_tok), DEC_THREADS, smem, st, p));
+  if (!set) { PT_CUDA(cudaFuncSetAttribute(decode_kernel<MT, NT, S, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemLimit)); set = true; }
+  PT_CUDA(launch_early(decode_kernel<MT, NT, S, WARPS>, dim3(p.n_split, ceil_div(p.n_head, 16 * MT), p.n_tok), WARPS * 32, smem, st, p));
   count_launch();
   return PT_OK;
 }
-template <int MT> static int dispatch_decode(const Params &p, cudaStream_t st) {
-  return p.rank <= 256 ? launch_decode<MT, 2>(p, st) : launch_decode<MT, 4>(p, st);
+template <int MT, int NT, int WARPS> static int dispatch_width(const Params &p, cudaStream_t st) {
+  return p.row_ld - 8 <= PARTS * 32 * 2 ? launch_decode<MT, NT, 2, WARPS>(p, st) : launch_decode<MT, NT, 5, WARPS>(p, st);
+}
+static int dispatch_decode(const Params &p, bool two_tiles, cudaStream_t st) {
+  if (!two_tiles) return p.rank <= 256 ? dispatch_width<1, 2, 16>(p, st) : launch_decode<1, 4, 5, 16>(p, st);
+  if (p.rank <= 128) return dispatch_width<2, 2, 8>(p, st);
+  return p.rank <= 256 ? dispatch_width<2, 4, 8>(p, st) : launch_decode<2, 8, 5, 8>(p, st);
 }
 
-constexpr size_t kSmemLimit = 226 * 1024;
-static int pad32(int v) { return (v + 31) / 32 * 32; }
-static bool two_tiles(int n_head, int width) { return n_head > 16 && decode_smem<2>(pad32(width)) <= kSmemLimit; }
-static int splits(int n_tok, int n_head, int width, int max_len) {
-  const int blocks = n_tok * ceil_div(n_head, two_tiles(n_head, width) ? 32 : 16);
+static bool two_tiles(int n_head, int row_ld) { return n_head > 16 && decode_smem<2>(row_ld, kMinSlots) <= kSmemLimit; }
+static int splits(int n_tok, int n_head, int row_ld, int max_len) {
+  const int blocks = n_tok * ceil_div(n_head, two_tiles(n_head, row_ld) ? 32 : 16);
   return std::max(1, std::min({sm_count() / blocks, kMaxSplit, ceil_div(max_len, TILE)}));
 }
 static bool decode_takes(int dtype, int page, int dim, int rot, int vdim, int rank) {
-  return dtype == PT_DT_BF16 && page == TILE && dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && rank <= 512 && decode_smem<1>(pad32(rot + rank)) <= kSmemLimit &&
+  return dtype == PT_DT_BF16 && page == TILE && dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && rank <= 512 && pt_latent_row(rot, rank) - 8 <= PARTS * 32 * 5 && decode_smem<1>(pt_latent_row(rot, rank), kMinSlots) <= kSmemLimit &&
          (size_t)16 * (rank + 32) * sizeof(bf) <= 40 * 1024;
 }
 static size_t align256(size_t v) { return (v + 255) / 256 * 256; }
@@ -562,6 +618,8 @@ static size_t align256(size_t v) { return (v + 255) / 256 * 256; }
 }  // namespace pt
 
 using namespace pt;
+
+extern "C" int pt_latent_row(int rot_dim, int rank) { return (rot_dim + rank + 15) / 16 * 16 + 8; }
 
 extern "C" int pt_latent_prep(const pt_latent_prep_args *a, void *stream) {
   PT_REQUIRE(a, "pt_latent_prep: null args");
@@ -573,7 +631,7 @@ extern "C" int pt_latent_prep(const pt_latent_prep_args *a, void *stream) {
   PT_REQUIRE(a->q && a->kv && a->q_norm && a->kv_norm && a->cq && a->pool && a->page_table && (!a->rot_dim || a->rope), "pt_latent_prep: null pointer argument");
   PT_REQUIRE(a->ld >= std::max(a->q_rank, a->rank + a->rot_dim) && a->cq_ld >= a->q_rank, "pt_latent_prep: row strides %d, %d", a->ld, a->cq_ld);
   lat::PrepParams p{};
-  p.q_rank = a->q_rank; p.rank = a->rank; p.rot = a->rot_dim; p.page = a->page_size; p.max_pages = a->max_pages; p.ld = a->ld; p.cq_ld = a->cq_ld; p.eps = a->eps;
+  p.q_rank = a->q_rank; p.rank = a->rank; p.rot = a->rot_dim; p.row_ld = pt_latent_row(a->rot_dim, a->rank); p.page = a->page_size; p.max_pages = a->max_pages; p.ld = a->ld; p.cq_ld = a->cq_ld; p.eps = a->eps;
   p.max_len = a->max_len > 0 ? a->max_len : a->page_size * a->max_pages;
   PT_REQUIRE(p.max_len <= a->page_size * a->max_pages, "pt_latent_prep: max_len=%d exceeds the page table", p.max_len);
   p.q = a->q; p.kv = a->kv; p.q_norm = a->q_norm; p.kv_norm = a->kv_norm; p.rope = (const float2 *)a->rope; p.cq = a->cq; p.pool = a->pool;
@@ -597,7 +655,7 @@ extern "C" int pt_latent_context(const pt_latent_context_args *a, void *stream) 
   PT_REQUIRE(a->pool && a->page_table && a->shared && a->latent && aligned_to(a->pool, 16) && aligned_to(a->shared, 16) && aligned_to(a->latent, 16),
              "pt_latent_context: null or unaligned pointer");
   lat::context_kernel<<<ceil_div(a->n_ctx, 8), 256, 0, as_stream(stream)>>>((const uint4 *)a->pool, a->page_table, b.slot, a->ctx_cu, b.n_seq, a->n_ctx, a->page_size, a->max_pages,
-                                                                            a->rot_dim / 8, (a->rot_dim + a->rank) / 8, (uint4 *)a->shared, (uint4 *)a->latent,
+                                                                            a->rot_dim / 8, (a->rot_dim + a->rank) / 8, pt_latent_row(a->rot_dim, a->rank) / 8, (uint4 *)a->shared, (uint4 *)a->latent,
                                                                             a->latent_ld / 8);
   PT_LAUNCH_CHECK("pt_latent_context");
   return PT_OK;
@@ -606,7 +664,7 @@ extern "C" int pt_latent_context(const pt_latent_context_args *a, void *stream) 
 extern "C" size_t pt_latent_attn_workspace_bytes(int n_tok, int n_head, int rot_dim, int rank, int dtype) {
   const size_t heads = (size_t)n_tok * n_head, es = dtype == PT_DT_F32 ? 4 : 2;
   const size_t plain = heads * rank * es, runs = ((size_t)n_tok + sm_count()) * n_head * (rank + 2) * sizeof(float) + 512;   // (tokens x runs stay below tokens + SMs)
-  return lat::align256(heads * (rot_dim + rank) * es) + std::max(plain, runs);
+  return lat::align256(heads * pt_latent_row(rot_dim, rank) * es) + std::max(plain, runs);
 }
 
 extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
@@ -623,7 +681,7 @@ extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
   PT_REQUIRE(a->workspace && a->workspace_bytes >= need && aligned_to(a->workspace, 16), "pt_latent_attn: %zu workspace bytes needed, got %zu", need, a->workspace_bytes);
   lat::Params p{};
   p.n_tok = b.n_tok; p.n_head = a->n_head; p.dim = a->dim; p.rot = a->rot_dim; p.vdim = a->vdim; p.rank = a->rank; p.width = a->rot_dim + a->rank;
-  p.width_pad = lat::pad32(p.width); p.q_ld = a->q_ld; p.max_pages = a->max_pages; p.gate_ld = a->gate_ld; p.out_ld = a->out_ld;
+  p.row_ld = pt_latent_row(a->rot_dim, a->rank); p.q_ld = a->q_ld; p.max_pages = a->max_pages; p.gate_ld = a->gate_ld; p.out_ld = a->out_ld;
   p.out_cols = a->out_cols > 0 ? a->out_cols : a->out_ld;
   PT_REQUIRE(p.out_cols >= a->n_head * a->vdim && p.out_cols <= a->out_ld, "pt_latent_attn: out_cols=%d", a->out_cols);
   p.max_len = a->max_len > 0 ? a->max_len : a->page_size * a->max_pages;
@@ -633,19 +691,19 @@ extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
   const size_t es = a->dtype == PT_DT_F32 ? 4 : 2;
   char *ws = (char *)a->workspace;
   p.q_cat = ws;
-  ws += lat::align256((size_t)b.n_tok * a->n_head * p.width * es);
+  ws += lat::align256((size_t)b.n_tok * a->n_head * p.row_ld * es);
   cudaStream_t st = as_stream(stream);
   const bool tc = !a->plain && b.n_tok == b.n_seq && b.n_seq <= 65535 && lat::decode_takes(a->dtype, a->page_size, a->dim, a->rot_dim, a->vdim, a->rank) && a->q_ld % 8 == 0 &&
                   a->out_ld % 2 == 0 && aligned_to(a->out, 4) && aligned_to(a->q, 16) && aligned_to(a->w_k, 16) && aligned_to(a->w_v, 16) && aligned_to(a->pool, 16);
   if (tc) {
-    p.n_split = lat::splits(b.n_tok, a->n_head, p.width, p.max_len);
+    p.n_split = lat::splits(b.n_tok, a->n_head, p.row_ld, p.max_len);
     p.ws_ml = (float2 *)ws;
     ws += lat::align256((size_t)b.n_tok * a->n_head * p.n_split * sizeof(float2));
     p.ws_o = (float *)ws;
     const int tokens16 = ceil_div(b.n_tok, 16);
     PT_CUDA(lat::launch_early(lat::absorb_kernel, dim3(ceil_div(a->rank, 16 * lat::ABSORB_WARPS), a->n_head, tokens16), lat::ABSORB_WARPS * 32, 0, st, p));
     count_launch();
-    if (int rc = lat::two_tiles(a->n_head, p.width) ? lat::dispatch_decode<2>(p, st) : lat::dispatch_decode<1>(p, st)) return rc;
+    if (int rc = lat::dispatch_decode(p, lat::two_tiles(a->n_head, p.row_ld), st)) return rc;
     p.ng = 2;
     while (p.ng < lat::EXPAND_WARPS && (long long)ceil_div(a->vdim, 16 * p.ng) * a->n_head * tokens16 > 2 * sm_count()) p.ng *= 2;
     PT_CUDA(lat::launch_early(lat::expand_kernel, dim3(ceil_div(a->vdim, 16 * p.ng), a->n_head, tokens16), lat::EXPAND_WARPS * 32, (size_t)16 * (a->rank + 32) * sizeof(__nv_bfloat16),
@@ -660,7 +718,7 @@ extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
   p.o_lat = ws;
   pt_window_attn_args w{};
   w.batch = b; w.dtype = a->dtype; w.n_head = a->n_head; w.n_kv = 1; w.dim = p.width; w.vdim = a->rank; w.page_size = a->page_size; w.max_pages = a->max_pages;
-  w.scale = a->scale; w.q = p.q_cat; w.q_ld = a->n_head * p.width; w.pool = const_cast<void *>(a->pool); w.page_table = a->page_table; w.out = p.o_lat; w.out_ld = a->n_head * a->rank;
+  w.scale = a->scale; w.q = p.q_cat; w.q_ld = a->n_head * p.row_ld; w.row_ld = p.row_ld; w.pool = const_cast<void *>(a->pool); w.page_table = a->page_table; w.out = p.o_lat; w.out_ld = a->n_head * a->rank;
   w.max_len = p.max_len; w.plain = 1; w.error_flag = a->error_flag; w.values_in_keys = 1; w.value_col = a->rot_dim;
   if (int rc = pt_window_attn(&w, stream)) return rc;
   if (a->dtype == PT_DT_F32) lat::expand_plain_kernel<float><<<grid, lat::PLAIN_THREADS, 0, st>>>(p);

@@ -29,21 +29,22 @@ struct Params {
 
 template <int VEC> __device__ __forceinline__ void put_f32(float *p, const float (&v)[VEC]) { store_vec<VEC>(p, v); }
 
-// NORM_Y: what is added is normalised (a residual step, without a second copy)
-template <typename T, typename E, int VEC, bool NORM_Y> __global__ void __launch_bounds__(1024, NORM_Y ? 2 : 1) post_norm_kernel(const Params p) {
+// RESIDUAL: a step whose addend is normalised, without a second copy.  ADD: nothing is normalised before it is added.  ANY: the rest.
+enum { RESIDUAL = 0, ADD = 1, ANY = 2 };
+template <typename T, typename E, int VEC, int MODE> __global__ void __launch_bounds__(1024, MODE == RESIDUAL ? 2 : 1) post_norm_kernel(const Params p) {
   extern __shared__ __align__(16) float row[];     // [width]: y, then the new x
   __shared__ float red[32], pw[kMaxTop];
   __shared__ int pr[kMaxTop];
   launch_dependents();
   const int r = blockIdx.x, src = p.row_index ? p.row_index[r] : r, tid = threadIdx.x;
   float *xo = p.x_out ? p.x_out + (size_t)r * p.width : nullptr;
-  T *hrow = p.h ? reinterpret_cast<T *>(p.h) + (size_t)r * p.h_ld : nullptr, *crow = !NORM_Y && p.copy ? reinterpret_cast<T *>(p.copy) + (size_t)r * p.copy_ld : nullptr;
+  T *hrow = p.h ? reinterpret_cast<T *>(p.h) + (size_t)r * p.h_ld : nullptr, *crow = MODE != RESIDUAL && p.copy ? reinterpret_cast<T *>(p.copy) + (size_t)r * p.copy_ld : nullptr;
   if (hrow)
     for (int i = p.width + tid; i < p.h_cols; i += blockDim.x) hrow[i] = from_f<T>(0.f);     // k padding of the next product
   if (crow)
     for (int i = p.width + tid; i < p.copy_cols; i += blockDim.x) crow[i] = from_f<T>(0.f);
   const T *emb = nullptr;
-  if (!NORM_Y && p.table) {
+  if (MODE != RESIDUAL && p.table) {
     const int step = p.step ? *p.step : 0;
     const int id = min(max(p.ids[(size_t)src * p.ids_ld + step], 0), p.vocab - 1);
     emb = reinterpret_cast<const T *>(p.table) + (size_t)id * p.table_ld;
@@ -58,10 +59,8 @@ template <typename T, typename E, int VEC, bool NORM_Y> __global__ void __launch
     pr[tid] = p.pair_row ? p.pair_row[k] : (int)k;
   }
   __syncthreads();
-  float ss = 0.f;
-  for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
-    float v[VEC];
-    if (!NORM_Y && emb) {
+  auto addend = [&](int i, float (&v)[VEC]) {
+    if (MODE != RESIDUAL && emb) {
       load_vec<VEC>(emb + i, v);
     } else if (p.y) {
       load_vec<VEC>(p.y + (size_t)src * p.y_ld + i, v);
@@ -77,31 +76,39 @@ template <typename T, typename E, int VEC, bool NORM_Y> __global__ void __launch
 #pragma unroll
       for (int j = 0; j < VEC; ++j) v[j] = fmaf(w, e[j], v[j]);
     }
-    put_f32<VEC>(row + i, v);
+  };
+  float ss = 0.f, inv = 1.f;
+  if (MODE != ADD) {
+    for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
+      float v[VEC];
+      addend(i, v);
+      put_f32<VEC>(row + i, v);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
+      for (int j = 0; j < VEC; ++j) ss = fmaf(v[j], v[j], ss);
+    }
+    inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);     // (every thread reads back what it wrote)
+    ss = 0.f;
   }
-  const bool norm = NORM_Y || p.norm_w;
-  const float inv = norm ? 1.0f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps) : 1.f;     // (every thread reads back what it wrote)
   const float *x = p.x_in ? p.x_in + (size_t)src * p.width : nullptr;
-  ss = 0.f;
   for (int i = tid * VEC; i < p.width; i += blockDim.x * VEC) {
     float v[VEC], o[VEC];
-    load_vec<VEC>(row + i, v);
-    if (norm) {
+    if (MODE == RESIDUAL || x) {
+      load_vec<VEC>(x + i, o);
+    } else {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+    }
+    if (MODE == ADD) {
+      addend(i, v);
+    } else {
       float w[VEC];
+      load_vec<VEC>(row + i, v);
       load_vec<VEC>(p.norm_w + i, w);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) v[j] *= inv * w[j];
     }
-    if (NORM_Y || x) {
-      load_vec<VEC>(x + i, o);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) o[j] += v[j];
-    } else {
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) o[j] = v[j];
-    }
+    for (int j = 0; j < VEC; ++j) o[j] += v[j];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) ss = fmaf(o[j], o[j], ss);
     if (xo) put_f32<VEC>(xo + i, o);
@@ -121,21 +128,22 @@ template <typename T, typename E, int VEC, bool NORM_Y> __global__ void __launch
   }
 }
 
-template <typename T, typename E, int VEC, bool NORM_Y> static int launch(const Params &p, cudaStream_t st) {
+template <typename T, typename E, int VEC, int MODE> static int launch(const Params &p, cudaStream_t st) {
   const size_t smem = (size_t)p.width * sizeof(float);
   if (smem > 48 * 1024) {
     static bool set = false;
-    if (!set) { PT_CUDA(cudaFuncSetAttribute(post_norm_kernel<T, E, VEC, NORM_Y>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
+    if (!set) { PT_CUDA(cudaFuncSetAttribute(post_norm_kernel<T, E, VEC, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); set = true; }
   }
   // few rows: as many threads per row as it has work for; many rows: more rows per SM
   const int want = ceil_div(ceil_div(p.width, VEC), 32) * 32, cap = p.rows <= 2 * sm_count() ? 1024 : 256;
-  post_norm_kernel<T, E, VEC, NORM_Y><<<p.rows, std::max(64, std::min(want, cap)), smem, st>>>(p);
+  post_norm_kernel<T, E, VEC, MODE><<<p.rows, std::max(64, std::min(want, cap)), smem, st>>>(p);
   PT_LAUNCH_CHECK("pt_post_norm");
   return PT_OK;
 }
 
 template <typename T, typename E, int VEC> static int launch(const Params &p, cudaStream_t st) {
-  return p.norm_w && p.x_in && !p.copy ? launch<T, E, VEC, true>(p, st) : launch<T, E, VEC, false>(p, st);
+  if (!p.norm_w) return launch<T, E, VEC, ADD>(p, st);
+  return p.x_in && !p.copy ? launch<T, E, VEC, RESIDUAL>(p, st) : launch<T, E, VEC, ANY>(p, st);
 }
 
 }  // namespace post

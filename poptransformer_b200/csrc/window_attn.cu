@@ -40,8 +40,8 @@ struct Params {
   int rope_half, out_cols;
   const void *gate;          // [n_tok][gate_ld]: n_head * vdim columns, or n_head with gate_heads
   int gate_ld;
-  bool gate_heads, v_in_k;   // v_in_k: the pool holds keys only, the values are their dimensions v_col ..
-  int v_col, hsplit;         // hsplit: blocks that share a kv head's query heads (plain kernel)
+  bool gate_heads, v_in_k;   // v_in_k: the pool holds keys only, the values are their dimensions v_col ..; row_ld: stride of its rows and of query heads
+  int v_col, row_ld, hsplit;         // hsplit: blocks that share a kv head's query heads (plain kernel)
   float softcap;
   // rows of the whole context (prompts)
   const __nv_bfloat16 *ctx_k, *ctx_shared, *ctx_v;
@@ -56,9 +56,9 @@ struct Params {
 };
 
 // (ANY: the values may be inside the keys; the tensor-core kernels do not take such pools)
-template <bool ANY> __device__ __forceinline__ size_t page_elems(const Params &p) { return (size_t)p.n_kv * p.page * (ANY && p.v_in_k ? p.dim : p.dim + p.vdim); }
+template <bool ANY> __device__ __forceinline__ size_t page_elems(const Params &p) { return (size_t)p.n_kv * p.page * (ANY && p.v_in_k ? p.row_ld : p.dim + p.vdim); }
 template <typename T, bool ANY = false> __device__ __forceinline__ T *k_page(const Params &p, int phys, int g) {
-  return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems<ANY>(p) + (size_t)g * p.page * p.dim;
+  return reinterpret_cast<T *>(p.pool) + (size_t)phys * page_elems<ANY>(p) + (size_t)g * p.page * (ANY && p.v_in_k ? p.row_ld : p.dim);
 }
 template <typename T, bool ANY = false> __device__ __forceinline__ T *v_page(const Params &p, int phys, int g) {
   if (ANY && p.v_in_k) return k_page<T, ANY>(p, phys, g) + p.v_col;
@@ -230,7 +230,7 @@ template <typename T> __global__ void kv_append_kernel(const Params p) {
 constexpr int PLAIN_THREADS = 128;
 template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plain_kernel(const Params p) {
   extern __shared__ __align__(16) float sm[];
-  const int nh = p.qpk / p.hsplit, g = blockIdx.y / p.hsplit, h0 = blockIdx.y * nh, v_ld = p.v_in_k ? p.dim : p.vdim;   // (heads h0 .. h0 + nh - 1)
+  const int nh = p.qpk / p.hsplit, g = blockIdx.y / p.hsplit, h0 = blockIdx.y * nh, k_ld = p.v_in_k ? p.row_ld : p.dim, v_ld = p.v_in_k ? p.row_ld : p.vdim;   // (heads h0 .. h0 + nh - 1)
   float *q = sm, *sc = q + nh * p.dim, *o = sc + nh * p.page, *st = o + nh * p.vdim;   // st: running max, sum, correction
   const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int s = p.tok_seq[t], pos = p.start[s] + t - p.cu[s];
@@ -239,8 +239,8 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
     return;
   }
   const int *table = p.page_table + (size_t)p.slot[s] * p.max_pages;
-  const T *qrow = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * p.dim;
-  for (int i = tid; i < nh * p.dim; i += PLAIN_THREADS) q[i] = to_f(qrow[i]);
+  const T *qrow = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h0 * k_ld;
+  for (int i = tid; i < nh * p.dim; i += PLAIN_THREADS) q[i] = to_f(qrow[(size_t)(i / p.dim) * k_ld + i % p.dim]);
   for (int i = tid; i < nh * p.vdim; i += PLAIN_THREADS) o[i] = 0.f;
   for (int h = tid; h < nh; h += PLAIN_THREADS) {
     st[3 * h] = p.sink ? p.sink[h0 + h] : -INFINITY;
@@ -255,7 +255,7 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) attn_plai
     for (int i = warp; i < nh * nk; i += PLAIN_THREADS / 32) {
       const int h = i / nk, key = i - h * nk;
       float a = 0.f;
-      for (int c = lane; c < p.dim; c += 32) a = fmaf(q[h * p.dim + c], to_f(K[(size_t)key * p.dim + c]), a);
+      for (int c = lane; c < p.dim; c += 32) a = fmaf(q[h * p.dim + c], to_f(K[(size_t)key * k_ld + c]), a);
       a = warp_sum(a);
       a *= p.scale;
       if (p.softcap > 0.f) a = p.softcap * tanhf(a / p.softcap);
@@ -816,14 +816,15 @@ extern "C" int pt_window_attn(const pt_window_attn_args *a, void *stream) {
   PT_REQUIRE(!a->values_in_keys || (!a->k && !ctx && a->value_col >= 0 && a->value_col + a->vdim <= a->dim),
              "pt_window_attn: values that are dimensions of the cached keys need value_col + vdim within dim and nothing to append");
   p.softcap = a->softcap; p.gate = a->gate; p.gate_ld = a->gate_ld; p.gate_heads = a->gate_per_head != 0;
-  p.v_in_k = a->values_in_keys != 0; p.v_col = a->value_col;
+  p.v_in_k = a->values_in_keys != 0; p.v_col = a->value_col; p.row_ld = a->row_ld > 0 ? a->row_ld : a->dim;
+  PT_REQUIRE(p.row_ld >= a->dim && (!p.v_in_k || a->q_ld >= a->n_head * p.row_ld) && (p.v_in_k || p.row_ld == a->dim), "pt_window_attn: row_ld=%d", a->row_ld);
   p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.0f;
   p.out_cols = a->out_cols > 0 ? a->out_cols : a->out_ld;
   p.prep = a->q_norm || a->k_norm || a->rope_dims;
   {
     const int pair = a->dtype == PT_DT_F32 ? 8 : 4;
     auto al = [](const void *x, int bytes) { return ((uintptr_t)x & (bytes - 1)) == 0; };
-    p.pair_rows = a->dim % 4 == 0 && a->dim <= 128 && a->rope_dims % 4 == 0 && a->q_ld % 2 == 0 && a->n_kv * a->page_size * (p.v_in_k ? a->dim : a->dim + a->vdim) % 2 == 0 && al(a->q, pair) && al(a->pool, pair) && al(a->rope, 16) && al(a->q_norm, 8) &&
+    p.pair_rows = a->dim % 4 == 0 && a->dim <= 128 && a->rope_dims % 4 == 0 && a->q_ld % 2 == 0 && a->n_kv * a->page_size * (p.v_in_k ? p.row_ld : a->dim + a->vdim) % 2 == 0 && al(a->q, pair) && al(a->pool, pair) && al(a->rope, 16) && al(a->q_norm, 8) &&
                   al(a->k_norm, 8) && (!a->k || (a->kv_ld % 2 == 0 && al(a->k, pair)));
   }
   PT_REQUIRE(a->rope_dims >= 0 && a->rope_dims % 2 == 0 && a->rope_dims <= a->dim && (!a->rope_dims || a->rope), "pt_window_attn: %d rotated dimensions of %d",

@@ -405,6 +405,11 @@ def window_attn(view, qkv, qkv_ld, cache, out, out_ld, n_head, scale, window=0, 
     check(_lib.lib().pt_window_attn(ctypes.byref(a), _stream()), "pt_window_attn")
 
 
+def latent_cache(rows, w, max_len, page_size=64, device="cuda", page_table=None, dtype=torch.bfloat16, n_pages=None):
+    """Page pool of a latent attention layer: per position one row [rotated key part | latent] and padding."""
+    return PagedKVCache(rows, 1, _lib.lib().pt_latent_row(w.rot_dim, w.rank), max_len, page_size, device, page_table, v_dim=0, dtype=dtype, n_pages=n_pages)
+
+
 def latent_prep(view, rows, ld, q_col, kv_col, w, cq, cq_ld, cache, eps, rope, error_flag=None):
     """Norms of both latents, rotation of the shared key part, append (see pt_latent_prep).  q_col, kv_col: first columns of the query latent
     and of [latent | key part] in `rows`; w: an object with q_rank, rank, rot_dim and the fp32 tensors q_norm, kv_norm."""

@@ -177,9 +177,11 @@ class PivavikDecoder(SequenceDecoder):
         self.caches = {}                                              # a run's own (the passes of a loop share weights, not positions)
         for r in self.runs:
             lay = r.sub.lay
-            heads, dim, vdim = (1, lay.rot_dim + lay.rank, 0) if lay.kind == "latent_attention" else (lay.kv_heads, lay.dim, lay.vdim)
-            self.caches[r.index] = ops.PagedKVCache(B, heads, dim, c.max_len, self._state_opts["page_size"], self.device, self.slots.page_table, v_dim=vdim,
-                                                    dtype=self.dtype, n_pages=self.slots.n_pages)
+            kw = dict(page_size=self._state_opts["page_size"], device=self.device, page_table=self.slots.page_table, dtype=self.dtype, n_pages=self.slots.n_pages)
+            if lay.kind == "latent_attention":
+                self.caches[r.index] = ops.latent_cache(B, r.sub.lat, c.max_len, **kw)
+            else:
+                self.caches[r.index] = ops.PagedKVCache(B, lay.kv_heads, lay.dim, c.max_len, v_dim=lay.vdim, **kw)
         self.attn_ws = self._attn_workspace([(s.lay.heads, s.lay.vdim, s.lay.window, 0) for s in self.subs if s.lay.kind == "attention"])
 
     def _row_buffers(self, rows):

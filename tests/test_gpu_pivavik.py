@@ -263,7 +263,7 @@ class LatentSite:
         self.rope = as_type(np.stack([np.cos(a), np.sin(a)], -1), F32, dev)
         pages = -(-max_len // page)
         table = np.random.default_rng(seed).permutation(n_slots * pages).reshape(n_slots, pages)
-        self.cache = ops.PagedKVCache(n_slots, 1, R + rank, max_len, page, dev, i32(table, dev), v_dim=0, dtype=dt)
+        self.cache = ops.latent_cache(n_slots, self.w, max_len, page, dev, i32(table, dev), dtype=dt)
         self.cache.pool.fill_(float("nan"))                   # nothing may be read that was not written
         self.flag = torch.zeros(1, dtype=torch.int32, device=dev)
 
