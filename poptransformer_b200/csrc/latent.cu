@@ -12,11 +12,10 @@
 //   absorb_kernel    W_uk^T q per head beside the rotated part of q (tensor cores; absorb_plain_kernel: any sizes, fp32 or bf16)
 //   decode_kernel    bf16, one token per sequence: 16 or 32 heads x a run of pages, scores and weighted sum on tensor cores from one copy
 //                    of the rows in shared memory, two pages in flight
-//   expand_kernel    the runs of pages combined, then W_uv and the gate per head (expand_plain_kernel: any sizes)
+//   combine_kernel   the runs of pages become one latent vector per head, with the gate
+//   expand_kernel    W_uv per head (expand_plain_kernel: any sizes, with the gate)
 // Prompts in fp32, or of sizes the tensor-core kernels do not take, go through pt_window_attn's any-size kernel with the values inside
 // the keys.  Norms, angles, scores, softmax and weights are fp32; weights enter the tensor cores as two bf16 parts (hi + lo).
-#include <type_traits>
-
 #include "chunk.cuh"
 #include "mbarrier.cuh"
 
@@ -252,94 +251,69 @@ __global__ void __launch_bounds__(ABSORB_WARPS * 32) absorb_kernel(const Params 
 
 __device__ __forceinline__ int pages_per_run(int n_pages, int n_split) { return (n_pages + n_split - 1) / n_split; }
 
-constexpr int EXPAND_WARPS = 8;
-// os[m] = sum over the runs of cw[m][run] * o[m][run], V neighbouring dimensions per item; a thread has the loads of U items x PB runs in
-// flight together.
-template <int V, int U, int PB>
-__device__ __forceinline__ void combine_runs(const float *src, size_t m_stride, int rank, int n_split, int tokens, const int *act, const float (*cw)[kMaxSplit + 1], bf *os, int ld) {
-  typedef typename std::conditional<V == 4, float4, float2>::type Vec;
-  const int per = rank / V, items = tokens * per, step = EXPAND_WARPS * 32;
-  for (int i = threadIdx.x; i < items; i += U * step) {
-    float a[U][V] = {};
-    int top = 0;
-    const float *s[U];
-    int ms[U], n_act[U];
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int k = i + u * step;
-      ms[u] = k < items ? k / per : 0;
-      n_act[u] = k < items ? act[ms[u]] : 0;
-      s[u] = src + ms[u] * m_stride + (k < items ? k - ms[u] * per : 0) * V;
-      top = max(top, n_act[u]);
-    }
-    for (int i0 = 0; i0 < top; i0 += PB) {
-      Vec v[U][PB];
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-#pragma unroll
-        for (int j = 0; j < PB; ++j)
-          if (i0 + j < n_act[u]) v[u][j] = __ldcg(reinterpret_cast<const Vec *>(s[u] + (size_t)(i0 + j) * rank));
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-#pragma unroll
-        for (int j = 0; j < PB; ++j)
-          if (i0 + j < n_act[u]) {
-            const float x = cw[ms[u]][i0 + j];
-            const float *f = reinterpret_cast<const float *>(&v[u][j]);
-#pragma unroll
-            for (int e = 0; e < V; ++e) a[u][e] = fmaf(f[e], x, a[u][e]);
-          }
-    }
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int k = i + u * step;
-      if (k >= items) break;
-      uint32_t *o = reinterpret_cast<uint32_t *>(os + ms[u] * ld + (k - ms[u] * per) * V);
-#pragma unroll
-      for (int e = 0; e < V; e += 2) o[e / 2] = pack_bf2(a[u][e], a[u][e + 1]);
-    }
+// The runs of one token and head become one latent vector (with the gate): a thread takes four neighbouring dimensions, a warp-wide
+// softmax over the runs' maxima gives their weights.
+constexpr int COMBINE_THREADS = 128;
+__global__ void __launch_bounds__(COMBINE_THREADS) combine_kernel(const Params p) {   // grid: (head, token)
+  __shared__ float cw[kMaxSplit];
+  launch_dependents();
+  const int tid = threadIdx.x, lane = tid & 31, h = blockIdx.x, t = blockIdx.y;
+  wait_for_prerequisites();
+  const int pos = p.start[t];
+  const bool ok = pos >= 0 && pos < p.max_len;
+  const int n_pages = pos / TILE + 1, per = pages_per_run(n_pages, p.n_split), n_act = ok ? (n_pages + per - 1) / per : 0;
+  const size_t head = (size_t)t * p.n_head + h;
+  constexpr int PB = 8;
+  const float *src = p.ws_o + head * p.n_split * p.rank;
+  if (tid < 32) {
+    const float2 ml = lane < n_act ? __ldcg(p.ws_ml + head * p.n_split + lane) : make_float2(-INFINITY, 0.f);
+    const float top = warp_max(ml.x), e = lane < n_act ? exp2f(ml.x - top) : 0.f, l = warp_sum(ml.y * e);
+    cw[lane] = lane < n_act ? e / l * sigmoid_gate<bf>(p, t, h) : 0.f;
   }
+  float4 v[PB];                                    // (the first runs' loads do not wait for the weights)
+  const int c = tid * 4;
+#pragma unroll
+  for (int j = 0; j < PB; ++j)
+    if (j < n_act && c < p.rank) v[j] = __ldcg(reinterpret_cast<const float4 *>(src + (size_t)j * p.rank + c));
+  __syncthreads();
+  if (c >= p.rank) return;                         // (rank is at most 512)
+  float a[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int i0 = 0; i0 < n_act; i0 += PB) {
+#pragma unroll
+    for (int j = 0; j < PB; ++j)
+      if (i0 + j < n_act) {
+        const float x = cw[i0 + j];
+        a[0] = fmaf(v[j].x, x, a[0]);
+        a[1] = fmaf(v[j].y, x, a[1]);
+        a[2] = fmaf(v[j].z, x, a[2]);
+        a[3] = fmaf(v[j].w, x, a[3]);
+      }
+#pragma unroll
+    for (int j = 0; j < PB; ++j)
+      if (i0 + PB + j < n_act) v[j] = __ldcg(reinterpret_cast<const float4 *>(src + (size_t)(i0 + PB + j) * p.rank + c));
+  }
+  *reinterpret_cast<uint2 *>(reinterpret_cast<bf *>(p.o_lat) + head * p.rank + c) = make_uint2(pack_bf2(a[0], a[1]), pack_bf2(a[2], a[3]));
 }
+
+constexpr int EXPAND_WARPS = 8;
 // Grid: (16 ng outputs, head, 16 tokens).  Warp (n group, k group): 8 / ng warps share an output group's k.
 __global__ void __launch_bounds__(EXPAND_WARPS * 32) expand_kernel(const Params p) {
-  extern __shared__ __align__(16) unsigned char sm_raw[];
-  __shared__ float cw[16][kMaxSplit + 1];
   __shared__ float red[EXPAND_WARPS * 32 * 8];
-  __shared__ int act[16];
   launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tig = lane & 3, h = blockIdx.y, t0 = blockIdx.z * 16;
   const int ks = EXPAND_WARPS / p.ng, wn = warp % p.ng, wk = warp / p.ng, n0 = (blockIdx.x * p.ng + wn) * 16;
-  const int k_per = ((p.rank + ks - 1) / ks + 31) / 32 * 32, kb = wk * k_per, ke = min(p.rank, kb + k_per), ld = p.rank + 32;
-  bf *os = reinterpret_cast<bf *>(sm_raw);          // [16][rank + 32]
+  const int k_per = ((p.rank + ks - 1) / ks + 31) / 32 * 32, kb = wk * k_per, ke = min(p.rank, kb + k_per);
   const bf *w = reinterpret_cast<const bf *>(p.w_v) + (size_t)h * p.vdim * p.rank;
   const bf *w0 = w + (size_t)(n0 + g) * p.rank, *w1 = w + (size_t)(n0 + 8 + g) * p.rank;
-  const bool n_ok0 = n0 + g < p.vdim, n_ok1 = n0 + 8 + g < p.vdim;
+  const bool n_ok0 = n0 + g < p.vdim, n_ok1 = n0 + 8 + g < p.vdim, ok0 = t0 + g < p.n_tok, ok1 = t0 + g + 8 < p.n_tok;
   Frag128 wf, xf;
   load128(wf, w0, w1, kb, ke, tig, n_ok0, n_ok1, true);
   wait_for_prerequisites();
-  // ---- the runs' weights (with the gate), then the latent vectors
-  for (int m = warp; m < 16; m += EXPAND_WARPS) {
-    const int t = t0 + m, pos = t < p.n_tok ? p.start[t] : -1;
-    const bool ok = pos >= 0 && pos < p.max_len;
-    const int n_pages = pos / TILE + 1, per = pages_per_run(n_pages, p.n_split), n_act = ok ? (n_pages + per - 1) / per : 0;
-    const float2 ml = lane < n_act ? __ldcg(p.ws_ml + ((size_t)t * p.n_head + h) * p.n_split + lane) : make_float2(-INFINITY, 0.f);
-    const float top = warp_max(ml.x), e = lane < n_act ? exp2f(ml.x - top) : 0.f, l = warp_sum(ml.y * e);
-    cw[m][lane] = n_act ? e / l * sigmoid_gate<bf>(p, t, h) : 0.f;
-    if (lane == 0) act[m] = n_act;
-  }
-  __syncthreads();
-  const int tokens = min(16, p.n_tok - t0);
-  const float *src = p.ws_o + ((size_t)t0 * p.n_head + h) * p.n_split * p.rank;
-  const size_t m_stride = (size_t)p.n_head * p.n_split * p.rank;
-  if (tokens == 1) combine_runs<2, 1, 16>(src, m_stride, p.rank, p.n_split, tokens, act, cw, os, ld);
-  else combine_runs<4, 4, 4>(src, m_stride, p.rank, p.n_split, tokens, act, cw, os, ld);
-  for (int i = tid; i < (16 - tokens) * p.rank / 2; i += blockDim.x) reinterpret_cast<uint32_t *>(os + (tokens + i / (p.rank / 2)) * ld)[i % (p.rank / 2)] = 0u;
-  __syncthreads();
-  // ---- W_uv
+  const bf *x0 = reinterpret_cast<const bf *>(p.o_lat) + ((size_t)(t0 + g) * p.n_head + h) * p.rank, *x1 = x0 + (size_t)8 * p.n_head * p.rank;
   float acc[2][4] = {};
   for (int k0 = kb; k0 < ke; k0 += 128) {
     if (k0 > kb) load128(wf, w0, w1, k0, ke, tig, n_ok0, n_ok1, true);
-    load128(xf, os + g * ld, os + (g + 8) * ld, k0, ke, tig, true, true, false);
+    load128(xf, x0, x1, k0, ke, tig, ok0, ok1, false);
     mma128(acc, xf, wf);
   }
   if (ks > 1) {
@@ -355,7 +329,6 @@ __global__ void __launch_bounds__(EXPAND_WARPS * 32) expand_kernel(const Params 
     }
   }
   bf *out = reinterpret_cast<bf *>(p.out) + (size_t)(t0 + g) * p.out_ld;
-  const bool ok0 = t0 + g < p.n_tok, ok1 = t0 + g + 8 < p.n_tok;
 #pragma unroll
   for (int j = 0; j < 2; ++j) {
     const int n = n0 + 8 * j + 2 * tig;
@@ -609,8 +582,7 @@ static int splits(int n_tok, int n_head, int row_ld, int max_len) {
   return std::max(1, std::min({sm_count() / blocks, kMaxSplit, ceil_div(max_len, TILE)}));
 }
 static bool decode_takes(int dtype, int page, int dim, int rot, int vdim, int rank) {
-  return dtype == PT_DT_BF16 && page == TILE && dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && rank <= 512 && pt_latent_row(rot, rank) - 8 <= PARTS * 32 * 5 && decode_smem<1>(pt_latent_row(rot, rank), kMinSlots) <= kSmemLimit &&
-         (size_t)16 * (rank + 32) * sizeof(bf) <= 40 * 1024;
+  return dtype == PT_DT_BF16 && page == TILE && dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && rank <= 512 && pt_latent_row(rot, rank) - 8 <= PARTS * 32 * 5 && decode_smem<1>(pt_latent_row(rot, rank), kMinSlots) <= kSmemLimit;
 }
 static size_t align256(size_t v) { return (v + 255) / 256 * 256; }
 
@@ -663,8 +635,8 @@ extern "C" int pt_latent_context(const pt_latent_context_args *a, void *stream) 
 
 extern "C" size_t pt_latent_attn_workspace_bytes(int n_tok, int n_head, int rot_dim, int rank, int dtype) {
   const size_t heads = (size_t)n_tok * n_head, es = dtype == PT_DT_F32 ? 4 : 2;
-  const size_t plain = heads * rank * es, runs = ((size_t)n_tok + sm_count()) * n_head * (rank + 2) * sizeof(float) + 512;   // (tokens x runs stay below tokens + SMs)
-  return lat::align256(heads * pt_latent_row(rot_dim, rank) * es) + std::max(plain, runs);
+  const size_t plain = heads * rank * es, runs = ((size_t)n_tok + sm_count()) * n_head * (rank + 2) * sizeof(float) + 1024;   // (tokens x runs stay below tokens + SMs)
+  return lat::align256(heads * pt_latent_row(rot_dim, rank) * es) + plain + (dtype == PT_DT_BF16 ? runs : 0);
 }
 
 extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
@@ -700,14 +672,17 @@ extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
     p.ws_ml = (float2 *)ws;
     ws += lat::align256((size_t)b.n_tok * a->n_head * p.n_split * sizeof(float2));
     p.ws_o = (float *)ws;
+    ws += lat::align256((size_t)b.n_tok * a->n_head * p.n_split * a->rank * sizeof(float));
+    p.o_lat = ws;
     const int tokens16 = ceil_div(b.n_tok, 16);
     PT_CUDA(lat::launch_early(lat::absorb_kernel, dim3(ceil_div(a->rank, 16 * lat::ABSORB_WARPS), a->n_head, tokens16), lat::ABSORB_WARPS * 32, 0, st, p));
     count_launch();
     if (int rc = lat::dispatch_decode(p, lat::two_tiles(a->n_head, p.row_ld), st)) return rc;
+    PT_CUDA(lat::launch_early(lat::combine_kernel, dim3(a->n_head, b.n_tok), lat::COMBINE_THREADS, 0, st, p));
+    count_launch();
     p.ng = 2;
     while (p.ng < lat::EXPAND_WARPS && (long long)ceil_div(a->vdim, 16 * p.ng) * a->n_head * tokens16 > 2 * sm_count()) p.ng *= 2;
-    PT_CUDA(lat::launch_early(lat::expand_kernel, dim3(ceil_div(a->vdim, 16 * p.ng), a->n_head, tokens16), lat::EXPAND_WARPS * 32, (size_t)16 * (a->rank + 32) * sizeof(__nv_bfloat16),
-                              st, p));
+    PT_CUDA(lat::launch_early(lat::expand_kernel, dim3(ceil_div(a->vdim, 16 * p.ng), a->n_head, tokens16), lat::EXPAND_WARPS * 32, 0, st, p));
     count_launch();
     return PT_OK;
   }

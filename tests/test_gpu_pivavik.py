@@ -190,7 +190,8 @@ def gate_rows(g, dt, dev):
 
 @pytest.mark.parametrize("dtype,plain", KINDS)
 @pytest.mark.parametrize("H,G,D,V,window,cap,per_head", [(4, 2, 32, 64, 70, 2.0, False), (3, 1, 128, 96, 128, 5.0, False), (2, 2, 40, 24, 1, 1.0, True), (12, 1, 64, 32, 65, 0.0, False),
-                                                         (5, 5, 14, 9, 33, 3.0, False), (6, 2, 96, 128, 0, 8.0, True), (4, 4, 64, 64, 300, 50.0, False)])
+                                                         (5, 5, 14, 9, 33, 3.0, False), (6, 2, 96, 128, 0, 8.0, True), (4, 4, 64, 64, 300, 50.0, False),
+                                                         (2, 1, 160, 136, 100, 4.0, False)])
 def test_attention_with_softcap_and_gate(cuda, dtype, plain, H, G, D, V, window, cap, per_head):
     """Three sequences of unequal length in portions (down to two tokens) and single tokens."""
     r = np.random.default_rng(5)
@@ -331,7 +332,7 @@ class LatentSite:
 
 LATENTS = [  # heads, plain key width, rotated width, value width, rank, query rank
     (4, 24, 16, 32, 48, 40), (20, 128, 64, 128, 512, 96), (3, 16, 8, 8, 136, 72), (33, 64, 32, 64, 256, 300), (16, 32, 64, 40, 320, 16), (3, 13, 6, 11, 21, 17), (2, 200, 48, 120, 72, 8),
-    (1, 8, 200, 16, 16, 24), (40, 16, 8, 24, 64, 64)]
+    (1, 8, 200, 16, 16, 24), (40, 16, 8, 24, 64, 64), (2, 24, 16, 32, 520, 24), (3, 40, 32, 136, 64, 48), (17, 264, 16, 16, 96, 32)]
 
 
 @pytest.mark.parametrize("dtype,plain", KINDS)
