@@ -690,7 +690,7 @@ typedef struct pt_latent_attn_args {
   int plain;              /* 1: the kernels for any sizes, whatever the shape        */
   void *workspace;        /* pt_latent_attn_workspace_bytes                          */
   size_t workspace_bytes;
-  int32_t *error_flag;
+  int32_t *error_flag;    /* optional, set to 11 when a bounded wait gave up, 12 when a position has no page */
 } pt_latent_attn_args;
 size_t pt_latent_attn_workspace_bytes(int n_tok, int n_head, int rot_dim, int rank, int dtype);
 int pt_latent_attn(const pt_latent_attn_args *args, void *stream);

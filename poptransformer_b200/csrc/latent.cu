@@ -11,7 +11,7 @@
 //   context_kernel   the cached rows of every sequence's context, one after the other
 //   absorb_kernel    W_uk^T q per head beside the rotated part of q (tensor cores; absorb_plain_kernel: any sizes, fp32 or bf16)
 //   decode_kernel    bf16, one token per sequence: 16 or 32 heads x a run of pages, scores and weighted sum on tensor cores from one copy
-//                    of the rows in shared memory, two pages in flight
+//                    of the rows in shared memory, which half pages enter through a ring of bulk copies
 //   combine_kernel   the runs of pages become one latent vector per head, with the gate
 //   expand_kernel    W_uv per head (expand_plain_kernel: any sizes, with the gate)
 // Prompts in fp32, or of sizes the tensor-core kernels do not take, go through pt_window_attn's any-size kernel with the values inside

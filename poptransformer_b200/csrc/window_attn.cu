@@ -1,6 +1,6 @@
 // Masked attention over a paged cache with per-sequence positions: a sliding window, kept first tokens, a softmax sink, grouped
-// heads, key and value widths of their own, optionally a norm and a rotation of every query and key head.  Position i sees key j when j <= i and (i - j < window or j < keep_first);
-// window = 0 means every earlier key.  sink[h] acts as one more logit of head h that brings weight to the denominator only.  With a
+// heads, key and value widths of their own, optionally a norm and a rotation of every query and key head.  Position i sees key j when
+// j <= i and (i - j < window or j < keep_first); window = 0 means every earlier key.  sink[h] acts as one more logit of head h that brings weight to the denominator only.  With a
 // softcap c a score s becomes c tanh(s / c).  The output can be multiplied with the sigmoid of a gate, per element or per head.
 // The values can be a part of the cached keys (a latent that all heads share), and prompts can read keys and values from rows of the
 // whole context instead of pages (pt_context_rows: a latent that was projected up), with a part of the key shared by all heads.
@@ -13,9 +13,10 @@
 //   attn_plain_kernel   any sizes, fp32 or bf16 caches, CUDA cores: the 32-bit path and the shapes the others do not take
 //   attn_prompt_kernel  bf16 prompts: 64 queries of one head per block, Q K^T and P V on the tensor cores, online softmax; only key
 //                       tiles that hold a visible key are touched
-//   (EXT instantiations of these two take a softcap and a gate)
 //   attn_decode_kernel  bf16, one token per sequence: one block per (visible page, kv head, sequence), scores and P V on the tensor
 //                       cores, pages combined by the last block to arrive; norm, rotation and append are fused
+//   attn_rotate_kernel  rotation alone, of a prompt's bf16 queries
+// Softcap and gate are in instantiations of their own (EXT) of the prompt and decode kernels.
 // Scores, softmax and weights are fp32.  The tensor-core kernels multiply V with weights split into two bf16 parts (hi + lo), which
 // keeps 16 significant bits of each weight.
 #include "chunk.cuh"
