@@ -835,7 +835,7 @@ def run_beside(args):
         else:
             flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(e.top * (size(e.up) + size(e.back)) for e in dec.expert_groups()))
             if name == "pivavik":
-                flops += 2 * prompt * sum(size(r.sub.up) for r in dec.runs if r.sub.lay.kind == "latent_attention")
+                flops += 2 * prompt * sum(size(r.sub.lat.up) for r in dec.runs if r.sub.lay.kind == "latent_attention")
         for n_seq in (1, 4):
             best = time_prompts(dec, cfg["vocab"], n_seq, prompt)
             pre.append({"sequences": n_seq, "prompt": prompt, "ms": best, "tokens_per_s": n_seq * prompt / best * 1e3, "linear_tflops": n_seq * flops / best / 1e9})

@@ -70,6 +70,7 @@ uint64_t pt_launch_count(void);
 #define PT_EPI_GLU 7          /* gated unit of row pairs (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
 #define PT_EPI_GELU_MUL 8     /* gelu_tanh(acc) * mul[mul_ids[row]]  (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
 #define PT_EPI_SOFTCAP 9      /* limit * tanh(acc / limit)  (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
+#define PT_EPI_XIELU 10       /* quadratic / exponential unit (PT_W_BF16 and pt_gemm_f32, see pt_dense_ext) */
 #define PT_GLU_CLAMPED 0      /* kinds of gated units */
 #define PT_GLU_SILU 1
 #define PT_GLU_GELU 2
@@ -82,6 +83,7 @@ uint64_t pt_launch_count(void);
  *              PT_GLU_CLAMPED  g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(1.702 g) (u + 1)
  *              PT_GLU_SILU     gate sigmoid(gate) up            PT_GLU_GELU  gelu_tanh(gate) up
  *   PT_EPI_SOFTCAP   out = limit tanh(y / limit)
+ *   PT_EPI_XIELU     out = pos y^2 + y / 2 for y > 0, neg (exp(y) - 1 - y) + y / 2 for the others
  *   PT_EPI_GELU_MUL  out[m, n] = gelu_tanh(y) * mul[mul_ids[m] * mul_ld + n], mul of the output's type
  *   groups     n_groups > 0: the weights are n_groups matrices one after the other (each as packed for the entry point), and tile t of
  *              group_rows activation rows is multiplied with matrix group_of[t] (device; negative: the tile is skipped).  pt_gemm:
@@ -99,6 +101,7 @@ typedef struct pt_dense_ext {
   const int32_t *group_used; /* pt_gemm, optional: rows in use of every tile (the rest is neither multiplied nor written) */
   int glu;
   const float *row_scale;
+  float pos, neg;           /* PT_EPI_XIELU                                           */
 } pt_dense_ext;
 
 /* ---- Int4ToHalf -------------------------------------------------------------------
@@ -554,13 +557,61 @@ typedef struct pt_post_norm_args {
 } pt_post_norm_args;
 int pt_post_norm(const pt_post_norm_args *args, void *stream);
 
+/* Residual step of layers that read two norms of the stream, the first of them mixed with the token before (csrc/shift_norm.cu), x fp32
+ * [rows, width]; s = row_index ? row_index[r] : r.
+ *   x = table != NULL ? N(table[ids[r * ids_ld + *step_dev]]) * embed_w (step_dev NULL: column 0; pos_out[r] <- the step)
+ *       : x_in[s] + y[s] + sum_k pair_w[s, k] (pair_row[s, k] < 0 ? self[s] : pair_y[pair_row[s, k]])      (pair_row NULL: s * top + k)
+ *   x_out[r] = x;   h2[r] = N(x) * w2;   n = N(x) * w1, h1[r] = n + (n' - n) * shift with n' the n of the same sequence's token before
+ * N divides each of `groups` equal parts of a row by its root mean square.  n' of a sequence's first new token comes from
+ * state_in[slot] (fp32 [slots, width]; zeros at position 0); the n of its last one goes to state_out[slot], or with state_by_seq to
+ * state_out[index of the sequence in the batch], which then must not be state_in.  h1 and h2 are in the activation type, columns from
+ * width on zeroed.  x_out, h1, h2 may be NULL.  x_out is not x_in unless every sequence brings one token. */
+typedef struct pt_shift_norm_args {
+  pt_batch_view batch;    /* used with h1                                            */
+  int rows, width, groups, dtype;
+  float eps;
+  const float *x_in;
+  float *x_out;
+  const void *table;
+  int table_ld, vocab;
+  const int32_t *ids;
+  int ids_ld;
+  const int32_t *step_dev;
+  int32_t *pos_out;
+  const float *embed_w;
+  const int32_t *row_index;
+  const float *y;
+  int y_ld;
+  const void *pair_y;     /* rows of width, pair_dtype PT_DT_F32 or PT_DT_BF16       */
+  int pair_dtype, pair_ld, top; /* top at most 64                                    */
+  const float *pair_w;
+  const int32_t *pair_row;
+  const void *self;       /* rows of the activation type                             */
+  int self_ld;
+  const float *w1, *shift;
+  void *h1;
+  int h1_ld;
+  const float *state_in;
+  float *state_out;
+  int state_by_seq;
+  const float *w2;
+  void *h2;
+  int h2_ld;
+} pt_shift_norm_args;
+int pt_shift_norm(const pt_shift_norm_args *args, void *stream);
+
 /* Mixture of experts (csrc/moe.cu): the `top` experts of every token by router logit, their weights (by `score`: the softmax over the
  * chosen logits, or the sigmoid of each), and the layout of the grouped products.  tile = 0: only expert and weight are written.  tile > 0: the pairs (token, choice) are sorted by
  * expert into tiles of `tile` rows: pair_row [n_tok, top], tile_expert [max_tiles] (-1: unused), tile_rows [max_tiles] (rows in use), row_token
  * [max_tiles * tile] (-1: padding), and with h the rows of h_bytes each are copied to gathered [max_tiles * tile] (padding
- * rows are left as they are), and row_weight [max_tiles * tile] (optional) gets the weight of every placed row. */
+ * rows are left as they are), and row_weight [max_tiles * tile] (optional) gets the weight of every placed row.
+ * PT_MOE_SOFTMAX_ALL: s = the softmax over all logits; experts are chosen by s + correction among the `keep` of `groups` equal groups of
+ * neighbours whose largest s + correction is largest, and the weights are the chosen s over their sum.  The last `identity` of the
+ * experts + identity logits have no matrices: a pair that chose one has expert = pair_row = -1 and no row (with tile = 0 pair_row, if
+ * given, is the pair's own index for the others). */
 #define PT_MOE_SOFTMAX 0
 #define PT_MOE_SIGMOID 1
+#define PT_MOE_SOFTMAX_ALL 2    /* see correction                                  */
 typedef struct pt_moe_route_args {
   int n_tok, experts, top;        /* at most 64 of 1024                              */
   const float *logits;
@@ -575,6 +626,8 @@ typedef struct pt_moe_route_args {
   void *gathered;
   int score;                      /* PT_MOE_*                                        */
   float *row_weight;
+  const float *correction;        /* PT_MOE_SOFTMAX_ALL: [experts + identity] or NULL; the rest is 0 for the other kinds */
+  int groups, keep, identity;     /* groups 0: one                                   */
 } pt_moe_route_args;
 int pt_moe_max_tiles(int n_tok, int experts, int top, int tile);
 int pt_moe_route(const pt_moe_route_args *args, void *stream);
@@ -641,7 +694,7 @@ typedef struct pt_latent_prep_args {
   int dtype;              /* PT_DT_F32 or PT_DT_BF16: q, kv, cq, pool                */
   int q_rank, rank, rot_dim;
   float eps;
-  const void *q, *kv;     /* [n_tok] rows of q_rank and of rank + rot_dim            */
+  const void *q, *kv;     /* [n_tok] rows of q_rank and of rank + rot_dim; kv NULL: nothing is cached (a layer that reads another's cache) */
   int ld;                 /* row stride of both                                      */
   const float *q_norm, *kv_norm;
   const float *rope;      /* fp32 [positions, rot_dim / 2, 2]                        */
@@ -691,6 +744,7 @@ typedef struct pt_latent_attn_args {
   void *workspace;        /* pt_latent_attn_workspace_bytes                          */
   size_t workspace_bytes;
   int32_t *error_flag;    /* optional, set to 11 when a bounded wait gave up, 12 when a position has no page */
+  int gate_per_value;     /* 1: the gate has n_head * vdim columns, one per output   */
 } pt_latent_attn_args;
 size_t pt_latent_attn_workspace_bytes(int n_tok, int n_head, int rot_dim, int rank, int dtype);
 int pt_latent_attn(const pt_latent_attn_args *args, void *stream);

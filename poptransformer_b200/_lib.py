@@ -19,7 +19,7 @@ class PtError(RuntimeError):
 class DenseExt(ctypes.Structure):
     _fields_ = [("bias", c_void_p), ("out2", c_void_p), ("out2_ld", c_int), ("split_n", c_int), ("limit", c_float), ("mul", c_void_p), ("mul_ld", c_int),
                 ("mul_ids", c_void_p), ("n_groups", c_int), ("group_rows", c_int), ("group_x_div", c_int), ("group_of", c_void_p),
-                ("group_used", c_void_p), ("glu", c_int), ("row_scale", c_void_p)]
+                ("group_used", c_void_p), ("glu", c_int), ("row_scale", c_void_p), ("pos", c_float), ("neg", c_float)]
 
 
 class LinearArgs(ctypes.Structure):
@@ -103,7 +103,7 @@ class LatentAttnArgs(ctypes.Structure):
                [("scale", c_float), ("q", c_void_p), ("q_ld", c_int)] + [(n, c_void_p) for n in ("rope", "w_k", "w_v", "gate")] + \
                [("gate_ld", c_int), ("pool", c_void_p), ("page_table", c_void_p)] + [(n, c_int) for n in ("page_size", "max_pages", "max_len")] + \
                [("out", c_void_p), ("out_ld", c_int), ("out_cols", c_int), ("plain", c_int), ("workspace", c_void_p), ("workspace_bytes", c_size_t),
-                ("error_flag", c_void_p)]
+                ("error_flag", c_void_p), ("gate_per_value", c_int)]
 
 
 class SsmArgs(ctypes.Structure):
@@ -127,10 +127,18 @@ class PostNormArgs(ctypes.Structure):
                [(n, c_void_p) for n in ("pair_w", "pair_row", "norm_w", "final_w", "h")] + [("h_ld", c_int), ("h_cols", c_int), ("copy", c_void_p), ("copy_ld", c_int), ("copy_cols", c_int)]
 
 
+class ShiftNormArgs(ctypes.Structure):
+    _fields_ = [("batch", BatchView)] + [(n, c_int) for n in ("rows", "width", "groups", "dtype")] + \
+               [("eps", c_float), ("x_in", c_void_p), ("x_out", c_void_p), ("table", c_void_p), ("table_ld", c_int), ("vocab", c_int), ("ids", c_void_p), ("ids_ld", c_int)] + \
+               [(n, c_void_p) for n in ("step_dev", "pos_out", "embed_w", "row_index", "y")] + [("y_ld", c_int), ("pair_y", c_void_p), ("pair_dtype", c_int), ("pair_ld", c_int), ("top", c_int)] + \
+               [(n, c_void_p) for n in ("pair_w", "pair_row", "self")] + [("self_ld", c_int), ("w1", c_void_p), ("shift", c_void_p), ("h1", c_void_p), ("h1_ld", c_int)] + \
+               [("state_in", c_void_p), ("state_out", c_void_p), ("state_by_seq", c_int), ("w2", c_void_p), ("h2", c_void_p), ("h2_ld", c_int)]
+
+
 class MoeRouteArgs(ctypes.Structure):
     _fields_ = [("n_tok", c_int), ("experts", c_int), ("top", c_int), ("logits", c_void_p), ("logits_ld", c_int), ("expert", c_void_p), ("weight", c_void_p),
                 ("tile", c_int), ("max_tiles", c_int), ("pair_row", c_void_p), ("tile_expert", c_void_p), ("tile_rows", c_void_p), ("row_token", c_void_p), ("counts", c_void_p), ("h", c_void_p), ("h_bytes", c_int),
-                ("gathered", c_void_p), ("score", c_int), ("row_weight", c_void_p)]
+                ("gathered", c_void_p), ("score", c_int), ("row_weight", c_void_p), ("correction", c_void_p), ("groups", c_int), ("keep", c_int), ("identity", c_int)]
 
 
 class LlamaLayer(ctypes.Structure):
@@ -164,6 +172,7 @@ SIGNATURES = {
     "pt_gemm_repack": (c_int, [c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]),
     "pt_gemm_f32": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, ctypes.POINTER(DenseExt), c_void_p]),
     "pt_post_norm": (c_int, [ctypes.POINTER(PostNormArgs), c_void_p]),
+    "pt_shift_norm": (c_int, [ctypes.POINTER(ShiftNormArgs), c_void_p]),
     "pt_moe_max_tiles": (c_int, [c_int] * 4),
     "pt_moe_route": (c_int, [ctypes.POINTER(MoeRouteArgs), c_void_p]),
     "pt_mlstm_workspace_bytes": (c_size_t, [c_int] * 5),

@@ -7,11 +7,11 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.environ.get("PT_B200_LIB", os.path.join(HERE, "libpt_b200.so"))   # same override as _lib.LIB_PATH
 SOURCES = ["api.cu", "linear.cu", "attention.cu", "ops.cu", "decode_llama.cu", "decode_llama_short.cu", "gemm_tc.cu", "prefill.cu",
-           "gemm_f32.cu", "hyper.cu", "window_attn.cu", "ssm.cu", "post_norm.cu", "moe.cu", "mlstm.cu", "latent.cu"]
+           "gemm_f32.cu", "hyper.cu", "window_attn.cu", "ssm.cu", "post_norm.cu", "moe.cu", "mlstm.cu", "latent.cu", "shift_norm.cu"]
 # Sources of a library that serves one architecture: what a program builds that runs only that model and finds no full library.
 _SEQUENCES = ["api.cu", "ops.cu", "linear.cu", "gemm_tc.cu", "gemm_f32.cu", "window_attn.cu"]
 PARTS = {"Sabisun": _SEQUENCES + ["hyper.cu", "ssm.cu"], "Padetar": _SEQUENCES + ["post_norm.cu", "moe.cu", "mlstm.cu"],
-         "Pivavik": _SEQUENCES + ["post_norm.cu", "moe.cu", "latent.cu"]}
+         "Pivavik": _SEQUENCES + ["post_norm.cu", "moe.cu", "latent.cu"], "Puputar": _SEQUENCES + ["shift_norm.cu", "moe.cu", "latent.cu"]}
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--threads", "0",
     "-Xcompiler", "-fPIC", "-shared",

@@ -5,6 +5,7 @@
 //   RELU2      out[m, n] = max(y, 0)^2
 //   GELU_MUL   out[m, n] = gelu_tanh(y) * mul[mul_ids[m], n]
 //   SOFTCAP    out[m, n] = limit * tanh(y / limit)
+//   XIELU      out[m, n] = y / 2 + (y > 0 ? pos y^2 : neg (exp(y) - 1 - y))
 //   GLU        weight rows alternate in blocks of eight, eight gate features and then the same eight up features; by `glu`:
 //     CLAMPED    out[m, f] = g sigmoid(1.702 g) (u + 1),  g = min(gate, limit), u = clamp(up, -limit, limit)
 //     SILU       out[m, f] = gate sigmoid(gate) up
@@ -28,6 +29,7 @@ struct DenseOut {
   float alpha, limit;
   int glu;
   const float *row_scale;
+  float pos, neg;
 };
 
 static inline DenseOut make_dense_out(void *out, int out_ld, int out_dt, int epilogue, float alpha, const pt_dense_ext *e) {
@@ -37,16 +39,16 @@ static inline DenseOut make_dense_out(void *out, int out_ld, int out_dt, int epi
   o.split_n = INT_MAX;
   if (e) {
     o.bias = e->bias; o.mul = e->mul; o.mul_ids = e->mul_ids; o.mul_ld = e->mul_ld; o.limit = e->limit;
-    o.glu = e->glu; o.row_scale = e->row_scale;
+    o.glu = e->glu; o.row_scale = e->row_scale; o.pos = e->pos; o.neg = e->neg;
     if (e->out2) { o.out2 = e->out2; o.out2_ld = e->out2_ld; o.split_n = e->split_n; }
   }
   return o;
 }
-static inline bool dense_needs_ext(int epilogue, const pt_dense_ext *e) { return e && (e->row_scale || epilogue == PT_EPI_SOFTCAP || (epilogue == PT_EPI_GLU && e->glu != PT_GLU_CLAMPED)); }
-static inline bool dense_epilogue_known(int e) { return e == PT_EPI_STORE || e == PT_EPI_RELU2 || e == PT_EPI_GLU || e == PT_EPI_GELU_MUL || e == PT_EPI_SOFTCAP; }
+static inline bool dense_needs_ext(int epilogue, const pt_dense_ext *e) { return e && (e->row_scale || epilogue == PT_EPI_SOFTCAP || epilogue == PT_EPI_XIELU || (epilogue == PT_EPI_GLU && e->glu != PT_GLU_CLAMPED)); }
+static inline bool dense_epilogue_known(int e) { return e == PT_EPI_STORE || e == PT_EPI_RELU2 || e == PT_EPI_GLU || e == PT_EPI_GELU_MUL || e == PT_EPI_SOFTCAP || e == PT_EPI_XIELU; }
 // nullptr, or what is wrong with the combination.
 static inline const char *dense_ext_error(int epilogue, int n_out, const pt_dense_ext *e) {
-  if ((epilogue == PT_EPI_GLU || epilogue == PT_EPI_GELU_MUL || epilogue == PT_EPI_SOFTCAP) && !e) return "the epilogue needs its extra arguments";
+  if ((epilogue == PT_EPI_GLU || epilogue == PT_EPI_GELU_MUL || epilogue == PT_EPI_SOFTCAP || epilogue == PT_EPI_XIELU) && !e) return "the epilogue needs its extra arguments";
   if (!e) return nullptr;
   if (epilogue == PT_EPI_GELU_MUL && !(e->mul && e->mul_ids)) return "a gelu-times-row epilogue needs mul and mul_ids";
   if (e->out2 && (e->split_n < 0 || e->split_n % 32 || e->split_n > n_out || e->out2_ld < n_out - e->split_n))
@@ -89,6 +91,10 @@ __device__ __forceinline__ void dense_put(const DenseOut &o, int m, int n, float
 template <bool EXT> __device__ __forceinline__ float dense_factor(const DenseOut &o, int m) { return EXT && o.row_scale ? o.alpha * __ldcg(o.row_scale + m) : o.alpha; }
 template <bool EXT> __device__ __forceinline__ float dense_value(const DenseOut &o, int m, int n, float acc) { return fmaf(acc, dense_factor<EXT>(o, m), o.bias ? __ldg(o.bias + n) : 0.f); }
 __device__ __forceinline__ float softcap_fast(float x, float limit) { return limit * (1.0f - __fdividef(2.0f, 1.0f + __expf(__fdividef(2.0f * x, limit)))); }
+template <bool EXACT> __device__ __forceinline__ float xielu_f(float y, float pos, float neg) {
+  const float e = EXACT ? expm1f(y) - y : __expf(y) - 1.0f - y;       // (not used for y > 0, where it may overflow)
+  return fmaf(0.5f, y, y > 0.f ? pos * y * y : neg * e);
+}
 // One finished sum (any epilogue but GLU, whose sums come in pairs).  EXACT: for models that run in 32-bit.
 template <bool EXT, bool EXACT = false> __device__ __forceinline__ void dense_store(const DenseOut &o, int m, int n, float acc) {
   float y = dense_value<EXT>(o, m, n, acc);
@@ -101,6 +107,8 @@ template <bool EXT, bool EXACT = false> __device__ __forceinline__ void dense_st
     y *= y;
   } else if (EXT && o.epilogue == PT_EPI_SOFTCAP) {
     y = EXACT ? o.limit * tanhf(y / o.limit) : softcap_fast(y, o.limit);
+  } else if (EXT && o.epilogue == PT_EPI_XIELU) {
+    y = xielu_f<EXACT>(y, o.pos, o.neg);
   } else if (o.epilogue == PT_EPI_GELU_MUL) {
     const size_t i = (size_t)o.mul_ids[m] * o.mul_ld + n;
     y = (EXACT ? gelu_tanh_f(y) : gelu_tanh_fast(y)) * (o.out_dt == PT_DT_F32 ? reinterpret_cast<const float *>(o.mul)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16 *>(o.mul)[i]));
@@ -134,7 +142,7 @@ __device__ __forceinline__ void dense_put4(void *out, size_t i, bool f32, const 
 template <bool EXT> __device__ __forceinline__ void dense_store4(const DenseOut &o, int m, int n, const float4 &acc) {
   const float a[4] = {acc.x, acc.y, acc.z, acc.w};
   const bool second = n >= o.split_n;
-  if (!second && o.epilogue != PT_EPI_STORE && o.epilogue != PT_EPI_RELU2) {
+  if (!second && o.epilogue != PT_EPI_STORE && o.epilogue != PT_EPI_RELU2 && !(EXT && o.epilogue == PT_EPI_XIELU)) {
 #pragma unroll 1
     for (int j = 0; j < 4; ++j) dense_store<EXT>(o, m, n + j, j == 0 ? acc.x : j == 1 ? acc.y : j == 2 ? acc.z : acc.w);
     return;
@@ -148,6 +156,7 @@ template <bool EXT> __device__ __forceinline__ void dense_store4(const DenseOut 
       y[j] = fmaxf(y[j], 0.f);
       y[j] *= y[j];
     }
+    if (EXT && !second && o.epilogue == PT_EPI_XIELU) y[j] = xielu_f<false>(y[j], o.pos, o.neg);
   }
   if (second) dense_put4(o.out2, (size_t)m * o.out2_ld + n - o.split_n, true, y);
   else dense_put4(o.out, (size_t)m * o.out_ld + n, o.out_dt == PT_DT_F32, y);

@@ -72,7 +72,7 @@ extern "C" int pt_gemm_f32(const float *x, int x_ld, const float *w, int w_ld, i
   const int n_y = epilogue == PT_EPI_GLU ? 0 : (ext && ext->out2 ? ext->split_n : n);
   PT_REQUIRE(m > 0 && n > 0 && k > 0 && x_ld >= k && w_ld >= k && y_ld >= n_y, "pt_gemm_f32: bad shape m=%d n=%d k=%d (row strides %d %d %d)", m, n, k, x_ld,
              w_ld, y_ld);
-  PT_REQUIRE(dense_epilogue_known(epilogue), "pt_gemm_f32: epilogue %d (store, relu2, glu, gelu-mul or softcap)", epilogue);
+  PT_REQUIRE(dense_epilogue_known(epilogue), "pt_gemm_f32: epilogue %d (store, relu2, glu, gelu-mul, softcap or xielu)", epilogue);
   const char *bad = dense_ext_error(epilogue, n, ext);
   PT_REQUIRE(!bad, "pt_gemm_f32: %s", bad);
   const bool grouped = ext && ext->n_groups > 0;

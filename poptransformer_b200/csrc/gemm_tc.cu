@@ -225,7 +225,7 @@ __device__ __forceinline__ void epilogue(const GemmParams &p, uint32_t tmem, int
 // bf16 output: neighbouring lanes (n, n + 1) trade values of two columns, so every store writes 4 bytes per lane.
 // Gated features: lanes n and n + 8 trade likewise, and each computes one column of the pair's feature.
 enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_GLU = 2, OUT_GELU_MUL = 3 };
-enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2, ACT_SCALED = 16 };   // OUT_GLU: the kind of unit, plus ACT_SCALED with a factor per row
+enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2, ACT_XIELU = 3, ACT_SCALED = 16 };   // OUT_GLU: the kind of unit, plus ACT_SCALED with a factor per row
 template <int KIND, int ACT>
 __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, int ld, const uint32_t (&v)[32], int n, int m, int lane) {
   const float b = d.bias ? __ldg(d.bias + n + (KIND == OUT_F32 && out == d.out2 ? d.split_n : 0)) : 0.f;
@@ -233,6 +233,7 @@ __device__ __forceinline__ void epilogue_rows32(const DenseOut &d, void *out, in
     float y = fmaf(__uint_as_float(x), d.alpha, b);
     if (ACT == ACT_RELU2) { y = fmaxf(y, 0.f); y *= y; }
     if (ACT == ACT_SOFTCAP) y = softcap_fast(y, d.limit);
+    if (ACT == ACT_XIELU) y = xielu_f<false>(y, d.pos, d.neg);
     return y;
   };
   if (KIND == OUT_F32) {
@@ -282,7 +283,7 @@ template <bool EXT> __device__ __forceinline__ void epilogue_bf16(const GemmPara
   // (warp-uniform) where this warp's 32 outputs go
   const bool second = nq >= d.split_n, glu = d.epilogue == PT_EPI_GLU && !second, f32 = second || d.out_dt == PT_DT_F32;
   // whole columns of 32 rows inside the output; 4-byte aligned pairs for bf16
-  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) && (!EXT || ((!d.row_scale || (glu && d.glu == PT_GLU_SILU)) && (second || f32 || d.epilogue != PT_EPI_SOFTCAP))) &&
+  const bool fast = p.ksplit == 1 && nq + 32 <= p.N && !(!second && d.epilogue == PT_EPI_GELU_MUL && f32) && !(glu && f32) && (!EXT || ((!d.row_scale || (glu && d.glu == PT_GLU_SILU)) && (second || (f32 ? d.epilogue != PT_EPI_XIELU : d.epilogue != PT_EPI_SOFTCAP)))) &&
                     (f32 || glu || (d.out_ld % 2 == 0 && ((uintptr_t)d.out & 3) == 0));
   const int rows = min(p.mb, m_end - m0), whole = fast ? rows & ~31 : 0;
   for (int c0 = 0; c0 < whole; c0 += 32) {
@@ -302,6 +303,7 @@ template <bool EXT> __device__ __forceinline__ void epilogue_bf16(const GemmPara
     } else {
       if (d.epilogue == PT_EPI_GELU_MUL) epilogue_rows32<OUT_GELU_MUL, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
       else if (d.epilogue == PT_EPI_RELU2) epilogue_rows32<OUT_BF16, ACT_RELU2>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
+      else if (EXT && d.epilogue == PT_EPI_XIELU) epilogue_rows32<OUT_BF16, ACT_XIELU>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
       else epilogue_rows32<OUT_BF16, ACT_NONE>(d, d.out, d.out_ld, v, n, m0 + c0, lane);
     }
   }
@@ -803,7 +805,7 @@ extern "C" int pt_gemm(const pt_gemm_args *a, void *stream) {
   PT_REQUIRE(a->x && a->w && a->out, "pt_gemm: null x / w / out");
   PT_REQUIRE(((uintptr_t)a->x & 15) == 0 && ((uintptr_t)a->w & 15) == 0, "pt_gemm: x and w must be 16-byte aligned");
   if (bf16) {
-    PT_REQUIRE(dense_epilogue_known(a->epilogue), "pt_gemm: BF16 epilogue %d (store, relu2, glu, gelu-mul or softcap)", a->epilogue);
+    PT_REQUIRE(dense_epilogue_known(a->epilogue), "pt_gemm: BF16 epilogue %d (store, relu2, glu, gelu-mul, softcap or xielu)", a->epilogue);
     const char *bad = dense_ext_error(a->epilogue, a->n_out, a->ext);
     PT_REQUIRE(!bad, "pt_gemm: %s", bad);
     PT_REQUIRE(a->out_dtype == PT_DT_BF16 || a->out_dtype == PT_DT_F32, "pt_gemm: BF16 weights write bf16 or fp32, got type %d", a->out_dtype);

@@ -12,8 +12,9 @@
 //   absorb_kernel    W_uk^T q per head beside the rotated part of q (tensor cores; absorb_plain_kernel: any sizes, fp32 or bf16)
 //   decode_kernel    bf16, one token per sequence: 16 or 32 heads x a run of pages, scores and weighted sum on tensor cores from one copy
 //                    of the rows in shared memory, which half pages enter through a ring of bulk copies
-//   combine_kernel   the runs of pages become one latent vector per head, with the gate
-//   expand_kernel    W_uv per head (expand_plain_kernel: any sizes, with the gate)
+//   combine_kernel   the runs of pages become one latent vector per head, with a gate per head
+//   expand_kernel    W_uv per head, with a gate per output (expand_plain_kernel: any sizes, with either gate)
+// A layer may read the latents that another one caches: its own prep then norms the query latent only.
 // Prompts in fp32, or of sizes the tensor-core kernels do not take, go through pt_window_attn's any-size kernel with the values inside
 // the keys.  Norms, angles, scores, softmax and weights are fp32; weights enter the tensor cores as two bf16 parts (hi + lo).
 #include "chunk.cuh"
@@ -63,10 +64,10 @@ template <typename T, int VEC> __global__ void __launch_bounds__(PREP_THREADS) p
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.ld, *kv = reinterpret_cast<const T *>(p.kv) + (size_t)t * p.ld;
   // the first half of the block takes the query latent, the second half the cached one
   constexpr int HALF = PREP_THREADS / 2;
-  const bool second = tid >= HALF;
-  const T *mine = second ? kv : q;
+  const bool second = tid >= HALF, append = p.kv != nullptr;
+  const T *mine = second && append ? kv : q;
   const float *norm = second ? p.kv_norm : p.q_norm;
-  const int n = second ? p.rank : p.q_rank, lane = tid & 31, warp = tid >> 5, at = tid & (HALF - 1);
+  const int n = second ? (append ? p.rank : 0) : p.q_rank, lane = tid & 31, warp = tid >> 5, at = tid & (HALF - 1);
   float ss = 0.f;
   for (int i = at * VEC; i < n; i += HALF * VEC) {
     float v[VEC];
@@ -80,6 +81,7 @@ template <typename T, int VEC> __global__ void __launch_bounds__(PREP_THREADS) p
   float sum = 0.f;
   for (int i = 0; i < HALF / 32; ++i) sum += red[(second ? HALF / 32 : 0) + i];
   const float inv = 1.0f / sqrtf(sum / (float)n + p.eps);
+  if (second && !append) return;
   if (second && !ok) {
     if (at == 0 && p.error_flag) atomicExch(p.error_flag, 12);
     return;
@@ -140,12 +142,13 @@ struct Params {
   float *ws_o;                       // [n_tok][n_head][n_split][rank]
   float2 *ws_ml;                     // [n_tok][n_head][n_split]
   int *error_flag;
+  bool gate_values;                  // a gate per output instead of one per head
 };
 
-template <typename T> __device__ __forceinline__ float sigmoid_gate(const Params &p, int t, int h) {
-  if (!p.gate) return 1.f;
-  return 1.0f / (1.0f + expf(-to_f(reinterpret_cast<const T *>(p.gate)[(size_t)t * p.gate_ld + h])));
+template <typename T> __device__ __forceinline__ float sigmoid_at(const Params &p, int t, int c) {
+  return 1.0f / (1.0f + expf(-to_f(reinterpret_cast<const T *>(p.gate)[(size_t)t * p.gate_ld + c])));
 }
+template <typename T> __device__ __forceinline__ float head_gate(const Params &p, int t, int h) { return p.gate && !p.gate_values ? sigmoid_at<T>(p, t, h) : 1.f; }
 template <typename T> __device__ __forceinline__ void rotate_query(const Params &p, int t, int h, int pos, int i, T *dst) {   // pair i
   const int half = p.rot / 2;
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)t * p.q_ld + (size_t)h * (p.rot + p.dim);
@@ -175,12 +178,12 @@ template <typename T> __global__ void __launch_bounds__(PLAIN_THREADS) expand_pl
   const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const T *o = reinterpret_cast<const T *>(p.o_lat) + ((size_t)t * p.n_head + h) * p.rank, *w = reinterpret_cast<const T *>(p.w_v) + (size_t)h * p.vdim * p.rank;
   T *out = reinterpret_cast<T *>(p.out) + (size_t)t * p.out_ld;
-  const float gate = sigmoid_gate<T>(p, t, h);
+  const float gate = head_gate<T>(p, t, h);
   for (int n = warp; n < p.vdim; n += PLAIN_THREADS / 32) {
     float a = 0.f;
     for (int r = lane; r < p.rank; r += 32) a = fmaf(to_f(o[r]), to_f(w[(size_t)n * p.rank + r]), a);
     a = warp_sum(a);
-    if (lane == 0) out[h * p.vdim + n] = from_f<T>(a * gate);
+    if (lane == 0) out[h * p.vdim + n] = from_f<T>(a * (p.gate_values ? sigmoid_at<T>(p, t, h * p.vdim + n) : gate));
   }
   if (h == p.n_head - 1)
     for (int i = p.n_head * p.vdim + tid; i < p.out_cols; i += PLAIN_THREADS) out[i] = from_f<T>(0.f);
@@ -268,7 +271,7 @@ __global__ void __launch_bounds__(COMBINE_THREADS) combine_kernel(const Params p
   if (tid < 32) {
     const float2 ml = lane < n_act ? __ldcg(p.ws_ml + head * p.n_split + lane) : make_float2(-INFINITY, 0.f);
     const float top = warp_max(ml.x), e = lane < n_act ? exp2f(ml.x - top) : 0.f, l = warp_sum(ml.y * e);
-    cw[lane] = lane < n_act ? e / l * sigmoid_gate<bf>(p, t, h) : 0.f;
+    cw[lane] = lane < n_act ? e / l * head_gate<bf>(p, t, h) : 0.f;
   }
   float4 v[PB];                                    // (the first runs' loads do not wait for the weights)
   const int c = tid * 4;
@@ -333,6 +336,11 @@ __global__ void __launch_bounds__(EXPAND_WARPS * 32) expand_kernel(const Params 
   for (int j = 0; j < 2; ++j) {
     const int n = n0 + 8 * j + 2 * tig;
     if (n >= p.vdim) continue;               // (vdim is a multiple of 8)
+    if (p.gate_values) {
+      const int c = h * p.vdim + n;
+      if (ok0) { acc[j][0] *= sigmoid_at<bf>(p, t0 + g, c); acc[j][1] *= sigmoid_at<bf>(p, t0 + g, c + 1); }
+      if (ok1) { acc[j][2] *= sigmoid_at<bf>(p, t0 + g + 8, c); acc[j][3] *= sigmoid_at<bf>(p, t0 + g + 8, c + 1); }
+    }
     if (ok0) *reinterpret_cast<uint32_t *>(out + h * p.vdim + n) = pack_bf2(acc[j][0], acc[j][1]);
     if (ok1) *reinterpret_cast<uint32_t *>(out + (size_t)8 * p.out_ld + h * p.vdim + n) = pack_bf2(acc[j][2], acc[j][3]);
   }
@@ -600,8 +608,8 @@ extern "C" int pt_latent_prep(const pt_latent_prep_args *a, void *stream) {
   PT_REQUIRE(a->dtype == PT_DT_F32 || a->dtype == PT_DT_BF16, "pt_latent_prep: type %d (fp32 or bf16)", a->dtype);
   PT_REQUIRE(a->q_rank > 0 && a->rank > 0 && a->rot_dim >= 0 && a->rot_dim % 2 == 0 && a->page_size > 0 && a->max_pages > 0, "pt_latent_prep: bad shape q_rank=%d rank=%d rot_dim=%d",
              a->q_rank, a->rank, a->rot_dim);
-  PT_REQUIRE(a->q && a->kv && a->q_norm && a->kv_norm && a->cq && a->pool && a->page_table && (!a->rot_dim || a->rope), "pt_latent_prep: null pointer argument");
-  PT_REQUIRE(a->ld >= std::max(a->q_rank, a->rank + a->rot_dim) && a->cq_ld >= a->q_rank, "pt_latent_prep: row strides %d, %d", a->ld, a->cq_ld);
+  PT_REQUIRE(a->q && a->q_norm && a->cq && a->page_table && (!a->kv || (a->kv_norm && a->pool && (!a->rot_dim || a->rope))), "pt_latent_prep: null pointer argument");
+  PT_REQUIRE(a->ld >= std::max(a->q_rank, a->kv ? a->rank + a->rot_dim : 0) && a->cq_ld >= a->q_rank, "pt_latent_prep: row strides %d, %d", a->ld, a->cq_ld);
   lat::PrepParams p{};
   p.q_rank = a->q_rank; p.rank = a->rank; p.rot = a->rot_dim; p.row_ld = pt_latent_row(a->rot_dim, a->rank); p.page = a->page_size; p.max_pages = a->max_pages; p.ld = a->ld; p.cq_ld = a->cq_ld; p.eps = a->eps;
   p.max_len = a->max_len > 0 ? a->max_len : a->page_size * a->max_pages;
@@ -647,7 +655,7 @@ extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
   PT_REQUIRE(a->n_head > 0 && a->n_head <= 65535 && a->dim > 0 && a->vdim > 0 && a->rank > 0 && a->rot_dim >= 0 && a->rot_dim % 2 == 0 && a->page_size > 0 && a->max_pages > 0,
              "pt_latent_attn: bad shape heads=%d dim=%d rot_dim=%d vdim=%d rank=%d", a->n_head, a->dim, a->rot_dim, a->vdim, a->rank);
   PT_REQUIRE(a->q && a->w_k && a->w_v && a->pool && a->page_table && a->out && (!a->rot_dim || a->rope), "pt_latent_attn: null pointer argument");
-  PT_REQUIRE(a->q_ld >= a->n_head * (a->rot_dim + a->dim) && a->out_ld >= a->n_head * a->vdim && (!a->gate || a->gate_ld >= a->n_head), "pt_latent_attn: row strides q %d, out %d, gate %d",
+  PT_REQUIRE(a->q_ld >= a->n_head * (a->rot_dim + a->dim) && a->out_ld >= a->n_head * a->vdim && (!a->gate || a->gate_ld >= a->n_head * (a->gate_per_value ? a->vdim : 1)), "pt_latent_attn: row strides q %d, out %d, gate %d",
              a->q_ld, a->out_ld, a->gate_ld);
   const size_t need = pt_latent_attn_workspace_bytes(b.n_tok, a->n_head, a->rot_dim, a->rank, a->dtype);
   PT_REQUIRE(a->workspace && a->workspace_bytes >= need && aligned_to(a->workspace, 16), "pt_latent_attn: %zu workspace bytes needed, got %zu", need, a->workspace_bytes);
@@ -658,6 +666,7 @@ extern "C" int pt_latent_attn(const pt_latent_attn_args *a, void *stream) {
   PT_REQUIRE(p.out_cols >= a->n_head * a->vdim && p.out_cols <= a->out_ld, "pt_latent_attn: out_cols=%d", a->out_cols);
   p.max_len = a->max_len > 0 ? a->max_len : a->page_size * a->max_pages;
   PT_REQUIRE(p.max_len <= a->page_size * a->max_pages, "pt_latent_attn: max_len=%d exceeds the page table", p.max_len);
+  p.gate_values = a->gate && a->gate_per_value;
   p.scale = a->scale; p.q = a->q; p.w_k = a->w_k; p.w_v = a->w_v; p.gate = a->gate; p.pool = a->pool; p.rope = (const float2 *)a->rope; p.page_table = a->page_table;
   p.cu = b.cu; p.start = b.start; p.slot = b.slot; p.tok_seq = b.tok_seq; p.out = a->out; p.error_flag = a->error_flag;
   const size_t es = a->dtype == PT_DT_F32 ? 4 : 2;

@@ -96,7 +96,9 @@ __global__ void __launch_bounds__(kThreads) linear_kernel(const LinearParams p) 
   if constexpr (WFMT == PT_W_BF16) {
     if (p.group_of) {
       if (p.pdl) wait_for_prerequisites();            // the router may be among the kernels before
-      w_base = (size_t)p.group_of[z] * p.group_stride;
+      const int grp = p.group_of[z];
+      if (grp < 0) return;                            // a row without a matrix
+      w_base = (size_t)grp * p.group_stride;
       px += (size_t)(z / p.group_x_div) * p.K;
     }
   }
@@ -606,7 +608,7 @@ extern "C" int pt_linear(const pt_linear_args *a, void *stream) {
   PT_REQUIRE(a->prologue >= PT_PRO_NONE && a->prologue <= PT_PRO_NORMCE, "pt_linear: bad prologue %d", a->prologue);
   if (a->wfmt == PT_W_BF16) {
     PT_REQUIRE(a->prologue == PT_PRO_NONE && dense_epilogue_known(a->epilogue),
-               "pt_linear: bf16 weights take no prologue and the store, relu2, glu, gelu-mul or softcap epilogue, got %d / %d", a->prologue, a->epilogue);
+               "pt_linear: bf16 weights take no prologue and the store, relu2, glu, gelu-mul, softcap or xielu epilogue, got %d / %d", a->prologue, a->epilogue);
     const char *bad = dense_ext_error(a->epilogue, a->n_out, a->ext);
     PT_REQUIRE(!bad, "pt_linear: %s", bad);
     PT_REQUIRE(!grouped || (a->ext->group_rows == 1 && a->ext->group_x_div >= 1), "pt_linear: groups come row by row");

@@ -1,6 +1,8 @@
 // Mixture of experts: which experts a token goes to, and where its rows lie for the grouped products.
 //   choose   per token the `top` experts with the largest router logits (the lowest index first among equals), and as weights the
 //            softmax over those logits or their sigmoids.  fp32.
+//            Or: scores are the softmax over all logits, corrected scores decide, only the best groups of neighbours take part, and the
+//            weights are the chosen scores over their sum.  Experts at the end may have no matrices (their output is the input).
 //   place    pair i = token i / top with its choice i % top gets a row of its own among its expert's rows.  The rows of an expert are
 //            padded to whole tiles; tile_expert names the expert of every tile (-1: unused) and tile_rows its rows in use, so a grouped
 //            product can look its weights up per tile.  Pairs keep their order within an expert.
@@ -23,6 +25,8 @@ struct Params {
   float *weight, *row_weight;                         // [n_tok][top], [max_tiles * tile] or null: the weight of every placed row
   int sigmoid;                                        // weights: sigmoid(logit) instead of the softmax over the chosen
   const int *counts;                                  // [experts], or null: counted while placing
+  int all, groups, keep;                              // logits: experts and identity experts
+  const float *correction;
 };
 
 // One warp per token; lane l holds the logits of experts l, l + 32, ...
@@ -63,6 +67,76 @@ __global__ void choose_kernel(const Params p) {
   if (lane + 32 < p.top) p.weight[(size_t)t * p.top + lane + 32] = w1 / sum;
 }
 
+// Corrected scores, groups and identity experts.  One warp per token; shared memory per warp: [all] scores, [all] corrected, [groups].
+constexpr int CHOOSE_WARPS = 4;
+__global__ void __launch_bounds__(CHOOSE_WARPS * 32) choose_corrected_kernel(const Params p) {
+  extern __shared__ float choose_sm[];
+  launch_dependents();
+  const int t = blockIdx.x * CHOOSE_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= p.n_tok) return;
+  float *s = choose_sm + (size_t)(threadIdx.x >> 5) * (2 * p.all + p.groups), *c = s + p.all, *best = c + p.all;
+  const float *z = p.logits + (size_t)t * p.logits_ld;
+  float top = -INFINITY, sum = 0.f;
+  for (int e = lane; e < p.all; e += 32) top = fmaxf(top, z[e]);
+  top = warp_max(top);
+  for (int e = lane; e < p.all; e += 32) {
+    s[e] = expf(z[e] - top);
+    sum += s[e];
+  }
+  sum = warp_sum(sum);
+  for (int e = lane; e < p.all; e += 32) {
+    s[e] /= sum;
+    c[e] = s[e] + (p.correction ? __ldg(p.correction + e) : 0.f);
+  }
+  __syncwarp();
+  if (p.keep < p.groups) {
+    const int size = p.all / p.groups;
+    for (int g = lane; g < p.groups; g += 32) {
+      float m = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, c[e]);
+      best[g] = m;
+    }
+    __syncwarp();
+    for (int g = lane; g < p.groups; g += 32) {
+      const float mine = best[g];
+      int before = 0;                                   // groups in front of this one (the lowest index first among equals)
+      for (int o = 0; o < p.groups; ++o) before += best[o] > mine || (best[o] == mine && o < g);
+      if (before >= p.keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) c[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  sum = 0.f;
+  float w0 = 0.f, w1 = 0.f;                             // lane k keeps the weights of choices k and k + 32
+  for (int k = 0; k < p.top; ++k) {
+    float most = -INFINITY;
+    int at = INT_MAX;
+    for (int e = lane; e < p.all; e += 32)
+      if (c[e] > most) { most = c[e]; at = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float b = __shfl_xor_sync(0xffffffffu, most, o);
+      const int a = __shfl_xor_sync(0xffffffffu, at, o);
+      if (b > most || (b == most && a < at)) { most = b; at = a; }
+    }
+    if (at == INT_MAX) at = k;                          // only infinities or NaN are left
+    const float w = s[at];
+    sum += w;
+    __syncwarp();
+    if (lane == (k & 31)) {
+      (k < 32 ? w0 : w1) = w;
+      const size_t i = (size_t)t * p.top + k;
+      p.expert[i] = at < p.experts ? at : -1;
+      if (p.pair_row) p.pair_row[i] = at < p.experts ? (int)i : -1;      // (placed experts get their rows later)
+      c[at] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  sum += 1e-20f;
+  if (lane < p.top) p.weight[(size_t)t * p.top + lane] = w0 / sum;
+  if (lane + 32 < p.top) p.weight[(size_t)t * p.top + lane + 32] = w1 / sum;
+}
+
 // Pairs per expert, for many pairs: block e counts those of expert e.
 __global__ void __launch_bounds__(PLACE_THREADS) count_kernel(const int *expert, int pairs, int *counts) {
   __shared__ int warps[PLACE_THREADS / 32];
@@ -96,7 +170,7 @@ __global__ void __launch_bounds__(PLACE_THREADS) place_kernel(const Params p) {
   __syncthreads();
   int hits = 0;
   auto count_one = [&](int x) {
-    if (!p.counts) atomicAdd(mine + x, 1);
+    if (!p.counts && x >= 0) atomicAdd(mine + x, 1);
     hits += x == e;
   };
   int i = i0;
@@ -193,16 +267,26 @@ extern "C" int pt_moe_max_tiles(int n_tok, int experts, int top, int tile) {
 
 extern "C" int pt_moe_route(const pt_moe_route_args *a, void *stream) {
   PT_REQUIRE(a, "pt_moe_route: null args");
-  PT_REQUIRE(a->n_tok > 0 && a->experts > 0 && a->experts <= moe::kMaxExperts && a->top > 0 && a->top <= std::min(a->experts, moe::kMaxTop),
-             "pt_moe_route: %d tokens, %d of %d experts (at most %d of %d)", a->n_tok, a->top, a->experts, moe::kMaxTop, moe::kMaxExperts);
+  const int all = a->experts + a->identity;       // logits
+  PT_REQUIRE(a->identity >= 0 && (!a->identity || a->score == PT_MOE_SOFTMAX_ALL), "pt_moe_route: %d identity experts", a->identity);
+  PT_REQUIRE(a->n_tok > 0 && a->experts > 0 && all <= moe::kMaxExperts && a->top > 0 && a->top <= std::min(all, moe::kMaxTop),
+             "pt_moe_route: %d tokens, %d of %d experts (at most %d of %d)", a->n_tok, a->top, all, moe::kMaxTop, moe::kMaxExperts);
   PT_REQUIRE((long long)a->n_tok * a->top < (1 << 28), "pt_moe_route: %d tokens x %d choices", a->n_tok, a->top);
-  PT_REQUIRE(a->logits && a->logits_ld >= a->experts && a->expert && a->weight, "pt_moe_route: null pointer argument");
+  PT_REQUIRE(a->logits && a->logits_ld >= all && a->expert && a->weight, "pt_moe_route: null pointer argument");
   moe::Params p{};
   p.n_tok = a->n_tok; p.experts = a->experts; p.top = a->top; p.logits_ld = a->logits_ld; p.logits = a->logits; p.expert = a->expert; p.weight = a->weight;
-  PT_REQUIRE(a->score == PT_MOE_SOFTMAX || a->score == PT_MOE_SIGMOID, "pt_moe_route: weights of kind %d", a->score);
+  PT_REQUIRE(a->score == PT_MOE_SOFTMAX || a->score == PT_MOE_SIGMOID || a->score == PT_MOE_SOFTMAX_ALL, "pt_moe_route: weights of kind %d", a->score);
   p.sigmoid = a->score == PT_MOE_SIGMOID;
   cudaStream_t st = as_stream(stream);
-  moe::choose_kernel<<<ceil_div(p.n_tok, 4), 128, 0, st>>>(p);
+  if (a->score == PT_MOE_SOFTMAX_ALL) {
+    p.all = all; p.groups = std::max(1, a->groups); p.keep = a->groups ? a->keep : 1; p.correction = a->correction; p.pair_row = a->pair_row;
+    PT_REQUIRE(all % p.groups == 0 && p.keep >= 1 && p.keep <= p.groups && a->top <= all / p.groups * p.keep, "pt_moe_route: %d of %d groups of %d experts, %d choices", p.keep,
+               p.groups, all, a->top);
+    PT_REQUIRE(!a->identity || a->pair_row, "pt_moe_route: identity experts need pair_row");
+    moe::choose_corrected_kernel<<<ceil_div(p.n_tok, moe::CHOOSE_WARPS), moe::CHOOSE_WARPS * 32, (size_t)moe::CHOOSE_WARPS * (2 * all + p.groups) * sizeof(float), st>>>(p);
+  } else {
+    moe::choose_kernel<<<ceil_div(p.n_tok, 4), 128, 0, st>>>(p);
+  }
   PT_LAUNCH_CHECK("pt_moe_route");
   if (!a->tile) return PT_OK;
   PT_REQUIRE(a->tile > 0 && a->pair_row && a->tile_expert && a->tile_rows && a->row_token && a->max_tiles >= pt_moe_max_tiles(a->n_tok, a->experts, a->top, a->tile),

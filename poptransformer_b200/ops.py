@@ -21,14 +21,14 @@ import torch
 
 from . import _lib
 from ._lib import (AttnArgs, BatchView, ContextRows, DenseExt, GemmArgs, HyperArgs, LatentAttnArgs, LatentContextArgs, LatentPrepArgs, LinearArgs, MlstmArgs,
-                   MoeRouteArgs, PostNormArgs, PtError, SsmArgs, WindowAttnArgs, check)
+                   MoeRouteArgs, PostNormArgs, PtError, ShiftNormArgs, SsmArgs, WindowAttnArgs, check)
 
 W_INT4, W_FP16, W_FP8, W_BF16 = 0, 1, 2, 3
 DT_F16, DT_F32, DT_BF16 = 0, 1, 2
 PRO_NONE, PRO_RMSNORM, PRO_CAST_FP8, PRO_RMSNORM_CAST_FP8, PRO_NORMCE = 0, 1, 2, 3, 4
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL, EPI_RELU2, EPI_GLU, EPI_GELU_MUL, EPI_SOFTCAP = range(10)
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL, EPI_RELU2, EPI_GLU, EPI_GELU_MUL, EPI_SOFTCAP, EPI_XIELU = range(11)
 GLU_CLAMPED, GLU_SILU, GLU_GELU = 0, 1, 2
-MOE_SOFTMAX, MOE_SIGMOID = 0, 1
+MOE_SOFTMAX, MOE_SIGMOID, MOE_SOFTMAX_ALL = 0, 1, 2
 ROPE_NONE, ROPE_LLAMA, ROPE_CHATGLM2 = 0, 1, 2
 SOFTMAX_F32, SOFTMAX_F16 = 0, 1
 
@@ -220,13 +220,13 @@ class DenseLinear:
     # Up to a million weights (128 x 2048, 2048 x 128, 1024 x 1024) the skinny kernel takes 0.6 - 0.75 of the GEMM's time at 8 and 16 rows.
     SKINNY_ROWS, SMALL_ROWS, SMALL_SIZE = 7, 16, 1 << 20
 
-    def __init__(self, w, dtype, pad_rows=0, keep=False, bias=None, split=None, limit=0.0, glu=GLU_CLAMPED):
+    def __init__(self, w, dtype, pad_rows=0, keep=False, bias=None, split=None, limit=0.0, glu=GLU_CLAMPED, xielu=None):
         """pad_rows: zero rows are appended up to this many outputs (an output that is the padded input of the next linear).
         keep: keep the padded matrix itself as `w` (a table that also serves look-ups).  bias: fp32 [n_out].  split: outputs from this
         row on (a multiple of 32) go to a second, fp32 output and skip the epilogue.  limit, glu: of a gated epilogue (rows as glu_rows);
-        limit also of the softcap."""
+        limit also of the softcap.  xielu: (pos, neg) of that epilogue."""
         self.dtype, self.n_out, self.k_in = dtype, w.shape[0], w.shape[1]
-        self.split, self.limit, self.glu = split, float(limit), glu
+        self.split, self.limit, self.glu, self.xielu = split, float(limit), glu, xielu
         self.ld = pad_to(self.k_in, self.K_PAD) if dtype == torch.bfloat16 else self.k_in
         if self.ld != self.k_in or pad_rows > self.n_out:
             full = torch.zeros((max(pad_rows, self.n_out), self.ld), dtype=w.dtype, device=w.device)
@@ -254,10 +254,12 @@ class DenseLinear:
     def _ext(self, out2, out2_ld, mul, mul_ids, bias):
         """mul: (a table of the output's type, its row stride, its first column)."""
         bias = self.bias if bias is None else bias
-        if bias is None and self.split is None and mul is None and not self.limit and self.glu == GLU_CLAMPED:
+        if bias is None and self.split is None and mul is None and not self.limit and self.glu == GLU_CLAMPED and self.xielu is None:
             return None
         e = DenseExt()
         e.bias, e.limit, e.glu = _ptr(bias), self.limit, self.glu
+        if self.xielu is not None:
+            e.pos, e.neg = self.xielu
         if self.split is not None:
             e.out2, e.out2_ld, e.split_n = _ptr(out2), out2_ld, self.split
         if mul is not None:
@@ -412,12 +414,12 @@ def latent_cache(rows, w, max_len, page_size=64, device="cuda", page_table=None,
 
 def latent_prep(view, rows, ld, q_col, kv_col, w, cq, cq_ld, cache, eps, rope, error_flag=None):
     """Norms of both latents, rotation of the shared key part, append (see pt_latent_prep).  q_col, kv_col: first columns of the query latent
-    and of [latent | key part] in `rows`; w: an object with q_rank, rank, rot_dim and the fp32 tensors q_norm, kv_norm."""
+    and of [latent | key part] in `rows` (kv_col None: the layer reads what another one caches); w: an object with q_rank, rank, rot_dim and the fp32 tensors q_norm, kv_norm."""
     a = LatentPrepArgs()
     es = rows.element_size()
     a.batch, a.dtype, a.q_rank, a.rank, a.rot_dim, a.eps = view, dtype_code(rows.dtype), w.q_rank, w.rank, w.rot_dim, float(eps)
-    a.q, a.kv, a.ld = rows.data_ptr() + q_col * es, rows.data_ptr() + kv_col * es, ld
-    a.q_norm, a.kv_norm, a.rope, a.cq, a.cq_ld = _ptr(w.q_norm), _ptr(w.kv_norm), _ptr(rope), _ptr(cq), cq_ld
+    a.q, a.kv, a.ld = rows.data_ptr() + q_col * es, None if kv_col is None else rows.data_ptr() + kv_col * es, ld
+    a.q_norm, a.kv_norm, a.rope, a.cq, a.cq_ld = _ptr(w.q_norm), None if kv_col is None else _ptr(w.kv_norm), _ptr(rope), _ptr(cq), cq_ld
     a.pool, a.page_table, a.page_size, a.max_pages, a.max_len = _ptr(cache.pool), _ptr(cache.page_table), cache.page_size, cache.page_table.shape[1], cache.max_len
     a.error_flag = _ptr(error_flag)
     check(_lib.lib().pt_latent_prep(ctypes.byref(a), _stream()), "pt_latent_prep")
@@ -436,13 +438,13 @@ def latent_workspace_bytes(n_tok, w, dtype):
     return _lib.lib().pt_latent_attn_workspace_bytes(n_tok, w.heads, w.rot_dim, w.rank, dtype_code(dtype))
 
 
-def latent_attn(view, q, q_ld, w, cache, out, out_ld, scale, rope, workspace, gate=None, gate_ld=0, out_cols=0, error_flag=None, plain=False):
+def latent_attn(view, q, q_ld, w, cache, out, out_ld, scale, rope, workspace, gate=None, gate_ld=0, out_cols=0, error_flag=None, plain=False, gate_per_value=False):
     """Attention over the cached latents (see pt_latent_attn).  w: an object with heads, dim, rot_dim, vdim, rank and the tensors w_k [heads,
-    rank, dim] and w_v [heads, vdim, rank].  gate: a view that starts at the heads' gates."""
+    rank, dim] and w_v [heads, vdim, rank].  gate: a view that starts at the heads' gates (gate_per_value: one per output)."""
     a = LatentAttnArgs()
     a.batch, a.dtype, a.n_head, a.dim, a.rot_dim, a.vdim, a.rank, a.scale = view, dtype_code(q.dtype), w.heads, w.dim, w.rot_dim, w.vdim, w.rank, float(scale)
     a.q, a.q_ld, a.rope, a.w_k, a.w_v = _ptr(q), q_ld, _ptr(rope), _ptr(w.w_k), _ptr(w.w_v)
-    a.gate, a.gate_ld = gate.data_ptr() if gate is not None else None, gate_ld
+    a.gate, a.gate_ld, a.gate_per_value = gate.data_ptr() if gate is not None else None, gate_ld, 1 if gate_per_value else 0
     a.pool, a.page_table, a.page_size, a.max_pages, a.max_len = _ptr(cache.pool), _ptr(cache.page_table), cache.page_size, cache.page_table.shape[1], cache.max_len
     a.out, a.out_ld, a.out_cols, a.plain, a.error_flag = _ptr(out), out_ld, out_cols, 1 if plain else 0, _ptr(error_flag)
     a.workspace, a.workspace_bytes = _ptr(workspace), workspace.numel()
@@ -498,19 +500,41 @@ def post_norm(rows, width, eps, dtype, x_in=None, x_out=None, y=None, y_ld=0, pa
     check(_lib.lib().pt_post_norm(ctypes.byref(a), _stream()), "pt_post_norm")
 
 
+def shift_norm(view, rows, width, groups, eps, dtype, x_in=None, x_out=None, y=None, y_ld=0, pair_y=None, pair_ld=0, top=0, pair_w=None, pair_row=None, self_rows=None,
+               self_ld=0, w1=None, shift=None, h1=None, h1_ld=0, state_in=None, state_out=None, state_by_seq=False, w2=None, h2=None, h2_ld=0, row_index=None, table=None, vocab=0,
+               ids=None, ids_ld=1, step=None, pos_out=None, embed_w=None):
+    """Residual step with two grouped norms of the stream, the first mixed with the token before, or the start of a token from an embedding
+    table (see pt_shift_norm).  view: needed with h1.  self_rows: what the experts without matrices give back."""
+    a = ShiftNormArgs()
+    if view is not None:
+        a.batch = view
+    a.rows, a.width, a.groups, a.dtype, a.eps, a.x_in, a.x_out = rows, width, groups, dtype_code(dtype), float(eps), _ptr(x_in), _ptr(x_out)
+    if table is not None:
+        a.table, a.table_ld, a.vocab, a.ids, a.ids_ld = _ptr(table), table.shape[1], vocab or table.shape[0], _ptr(ids), ids_ld
+        a.step_dev, a.pos_out, a.embed_w = _ptr(step), _ptr(pos_out), _ptr(embed_w)
+    a.row_index, a.y, a.y_ld = _ptr(row_index), _ptr(y), y_ld
+    if pair_y is not None:
+        a.pair_dtype = dtype_code(pair_y.dtype)
+    a.pair_y, a.pair_ld, a.top, a.pair_w, a.pair_row, a.self, a.self_ld = _ptr(pair_y), pair_ld, top, _ptr(pair_w), _ptr(pair_row), _ptr(self_rows), self_ld
+    a.w1, a.shift, a.h1, a.h1_ld, a.state_in, a.state_out, a.state_by_seq = _ptr(w1), _ptr(shift), _ptr(h1), h1_ld, _ptr(state_in), _ptr(state_out), 1 if state_by_seq else 0
+    a.w2, a.h2, a.h2_ld = _ptr(w2), _ptr(h2), h2_ld
+    check(_lib.lib().pt_shift_norm(ctypes.byref(a), _stream()), "pt_shift_norm")
+
+
 def moe_max_tiles(n_tok, experts, top, tile):
     return int(_lib.lib().pt_moe_max_tiles(n_tok, experts, top, tile))
 
 
 def moe_route(logits, n_tok, experts, top, expert, weight, tile=0, pair_row=None, tile_expert=None, tile_rows=None, row_token=None, counts=None, h=None, h_ld=0, gathered=None,
-              score=MOE_SOFTMAX, row_weight=None):
+              score=MOE_SOFTMAX, row_weight=None, correction=None, groups=0, keep=0, identity=0):
     """Experts and weights of every token, and with `tile` the rows of the grouped products (see pt_moe_route)."""
     a = MoeRouteArgs()
-    a.n_tok, a.experts, a.top, a.logits, a.logits_ld = n_tok, experts, top, _ptr(logits), logits.shape[-1]
+    a.n_tok, a.experts, a.top, a.logits, a.logits_ld = n_tok, experts, top, _ptr(logits), logits.shape[-1]     # experts: those with matrices
     a.expert, a.weight, a.tile, a.score, a.row_weight = _ptr(expert), _ptr(weight), tile, score, _ptr(row_weight)
+    a.correction, a.groups, a.keep, a.identity, a.pair_row = _ptr(correction), groups, keep, identity, _ptr(pair_row)
     if tile:
         a.max_tiles = moe_max_tiles(n_tok, experts, top, tile)
-        a.pair_row, a.tile_expert, a.tile_rows, a.row_token = _ptr(pair_row), _ptr(tile_expert), _ptr(tile_rows), _ptr(row_token)
+        a.tile_expert, a.tile_rows, a.row_token = _ptr(tile_expert), _ptr(tile_rows), _ptr(row_token)
         a.counts = _ptr(counts)
         if h is not None:
             a.h, a.h_bytes, a.gathered = _ptr(h), h_ld * h.element_size(), _ptr(gathered)

@@ -3,7 +3,7 @@
 One fp32 residual stream; a layer reads one RMS norm of it (weights stored as their distance from one) and adds mixer and feed-forward at
 once (csrc/post_norm.cu).  Mixers and feed-forwards, in any order:
   latent_attention  queries through a latent; keys and values from a cached latent plus one rotated key part shared by all heads; a gate
-                    per head (csrc/latent.cu).  Decode steps stay in the latent's space, prompts project the context up
+                    per head (latent.py, csrc/latent.cu).  Decode steps stay in the latent's space, prompts project the context up
   attention         grouped heads with biases, a sliding window, a softcap on the scores, a gate per element; no rotation
                     (csrc/window_attn.cu)
   dense             gelu gated unit with biases
@@ -20,13 +20,12 @@ inputs are bfloat16, accumulation, residual stream, norms, rotation, scores, sof
 true 32-bit."""
 from types import SimpleNamespace
 
-import numpy as np
 import torch
 
 from . import ops
 from .experts import Experts
-from .padetar import rope_frequencies
-from .sequences import SequenceDecoder
+from .latent import LatentAttention, latent_mixer
+from .sequences import JointRows, SequenceDecoder
 
 
 class PivavikConfig:
@@ -38,19 +37,17 @@ class PivavikConfig:
         self.logit_softcap = float(config.get("logit_softcap") or 0.0)
         self.layers = []
         for i, lay in enumerate(config["layers"]):
-            m, mlp = lay["mixer"], lay.get("mlp")
-            layer = SimpleNamespace(kind=lay["type"], heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]), ff=0, moe=None)
-            if layer.kind == "latent_attention":
-                rot = m["rot"]
-                layer.q_rank, layer.rank, layer.rot_dim, layer.base = int(m["q_rank"]), int(m["kv_rank"]), int(m["rot_dim"]), float(rot["base"])
-                if int(rot["dims"]) != layer.rot_dim or layer.rot_dim % 2:
-                    raise ops.PtError(f"layer {i}: {rot['dims']} rotated dimensions of a rotated part of {layer.rot_dim}")
-            elif layer.kind == "attention":
+            kind, m, mlp = lay["type"], lay["mixer"], lay.get("mlp")
+            if kind == "latent_attention":
+                layer = latent_mixer(i, kind, m)
+            elif kind == "attention":
+                layer = SimpleNamespace(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]))
                 layer.kv_heads, layer.window, layer.softcap = int(m["kv_heads"]), int((m.get("mask") or {}).get("size") or 0), float(m.get("softcap") or 0.0)
                 if layer.heads % layer.kv_heads:
                     raise ops.PtError(f"layer {i}: {layer.heads} heads do not divide over {layer.kv_heads} key/value heads")
             else:
-                raise ops.PtError(f"layer {i}: unknown mixer {layer.kind!r}")
+                raise ops.PtError(f"layer {i}: unknown mixer {kind!r}")
+            layer.ff, layer.moe = 0, None
             if mlp is not None:
                 if mlp["kind"] == "dense":
                     layer.ff = int(mlp["ff"])
@@ -81,7 +78,7 @@ class PivavikDecoder(SequenceDecoder):
         c, dt, dev, f32, mat = self.cfg, self.dtype, self.device, w.f32, w.mat
         W = c.width
         bf16 = dt == torch.bfloat16
-        zeros = lambda rows, cols=W: torch.zeros((rows, cols), dtype=dt, device=dev)
+        zeros = lambda rows, cols: torch.zeros((rows, cols), dtype=dt, device=dev)
         self.head = w.lin(["embed"], [(c.vocab, W)], keep=True, limit=c.logit_softcap)     # also the look-up table
         self.table, self.h_ld = self.head.w, self.head.ld
         self.embed_norm, self.final_norm = 1.0 + f32("embed.norm", (W,)), 1.0 + f32("final.norm", (W,))
@@ -91,52 +88,24 @@ class PivavikDecoder(SequenceDecoder):
         for i, lay in enumerate(c.layers):
             p, M = f"l{i}.", f"l{i}.mix."
             sub = SimpleNamespace(layer=i, lay=lay, norm=1.0 + f32(p + "norm1", (W,)), ff=None, experts=None)
-            parts, bias = [], []
-
-            def add(rows, b=None):
-                parts.append(rows)
-                bias.append(torch.zeros(len(rows), dtype=torch.float32, device=dev) if b is None else b)
-
-            def col():
-                """First column of what is added next, on a 16-byte boundary."""
-                add(zeros(-sum(map(len, parts)) % 8))
-                return sum(map(len, parts))
-
+            rows = JointRows(W, dt, dev)
             H, D, V = lay.heads, lay.dim, lay.vdim
             if lay.kind == "attention":
                 for name, n in (("q", H * D), ("k", lay.kv_heads * D), ("v", lay.kv_heads * V)):
-                    add(mat(M + name, (n, W)), f32(M + name + ".b", (n,)))
-                sub.gate_col = col()
-                add(mat(M + "g", (H * V, W)))
+                    rows.add(mat(M + name, (n, W)), f32(M + name + ".b", (n,)))
+                sub.gate_col = rows.column()
+                rows.add(mat(M + "g", (H * V, W)))
             else:
-                R, rank = lay.rot_dim, lay.rank
-                add(mat(M + "dq", (lay.q_rank, W)))
-                sub.kv_col = col()
-                add(mat(M + "dkv", (rank + R, W)))
-                sub.gate_col = col()
-                add(mat(M + "g", (H, W)))
-                uq = mat(M + "uq", (H * (D + R), lay.q_rank)).view(H, D + R, lay.q_rank)
-                sub.uq = ops.DenseLinear(torch.cat([uq[:, D:], uq[:, :D]], 1).reshape(-1, lay.q_rank), dt)       # a head: the rotated part first
-                sub.q_ld = ops.pad_to(sub.uq.n_out, 8)
-                uk, uv = mat(M + "uk", (H * D, rank)), mat(M + "uv", (H * V, rank))
-                sub.lat = SimpleNamespace(heads=H, dim=D, rot_dim=R, vdim=V, rank=rank, q_rank=lay.q_rank, q_norm=f32(M + "dq.norm", (lay.q_rank,)),
-                                          kv_norm=f32(M + "dkv.norm", (rank,)), w_k=uk.view(H, D, rank).transpose(1, 2).contiguous(), w_v=uv.view(H, V, rank).contiguous())
-                # prompts on tensor cores: keys and values of the whole context by one product
-                sub.up = ops.DenseLinear(torch.cat([uk, uv], 0), dt) if bf16 and R and not any(x % 8 for x in (D, R, V, rank)) and D + R <= 256 and V <= 128 else None
-                if (R, lay.base) not in ropes:
-                    ang = np.arange(c.max_len)[:, None] * rope_frequencies(R, lay.base)
-                    ropes[R, lay.base] = torch.from_numpy(np.stack([np.cos(ang), np.sin(ang)], -1).astype(np.float32)).to(dev) if R else None
-                sub.rope = ropes[R, lay.base]
+                sub.lat = LatentAttention(w, M, lay, W, rows, ropes, c.max_len)
             split = None
             if lay.moe:
                 E, F = lay.moe.experts, lay.moe.ff
-                add(zeros(-sum(map(len, parts)) % 32))
-                split = sum(map(len, parts))
-                add(mat(p + "mlp.router", (E, W)))
+                split = rows.column(32)
+                rows.add(mat(p + "mlp.router", (E, W)))
                 gates, ups = ([mat(p + f"mlp.e{e}.{n}", (F, W)) for e in range(E)] for n in ("gate", "up"))
                 sub.experts = Experts(dt, lay.moe.top, gates, ups, [mat(p + f"mlp.e{e}.down", (W, F)) for e in range(E)], glu=ops.GLU_SILU, score=ops.MOE_SIGMOID,
                                       weigh_input=True)
-            sub.proj = ops.DenseLinear(torch.cat(parts, 0), dt, bias=torch.cat(bias) if lay.kind == "attention" else None, split=split)
+            sub.proj = rows.linear(biased=lay.kind == "attention", split=split)
             sub.ld = ops.pad_to(sub.proj.n_out if split is None else split, 8)
             # ---- outputs: the mixer's columns, then the dense feed-forward's
             sub.ff_col = ops.pad_to(H * V, 8)
@@ -157,15 +126,14 @@ class PivavikDecoder(SequenceDecoder):
     def _linears(self):
         """Every linear once per time a token runs through it."""
         once = [self.head] + [self.loop_in for r in self.runs if r.entry is not None]
-        return once + [x for r in self.runs for x in (r.sub.proj, r.sub.ff, r.sub.uq if r.sub.lay.kind != "attention" else None, r.sub.out) if x is not None]
+        return once + [x for r in self.runs for x in (r.sub.proj, r.sub.ff, r.sub.lat.uq if r.sub.lay.kind != "attention" else None, r.sub.out) if x is not None]
 
     def expert_groups(self):
         return [r.sub.experts for r in self.runs if r.sub.experts]
 
     def fixed_bytes(self):
         """Weight bytes that every decode step streams, whatever the experts: the linears and the latents' per-head up-projections."""
-        heads = [x for r in self.runs if r.sub.lay.kind != "attention" for x in (r.sub.lat.w_k, r.sub.lat.w_v)]
-        return sum(x.nbytes for x in self._linears()) + sum(x.numel() * x.element_size() for x in heads)
+        return sum(x.nbytes for x in self._linears()) + sum(r.sub.lat.head_bytes for r in self.runs if r.sub.lay.kind != "attention")
 
     def weight_bytes(self, rows=1):
         """Algorithmic weight bytes one decode step of `rows` tokens streams, of the experts as many as the rows can choose at most."""
@@ -179,7 +147,7 @@ class PivavikDecoder(SequenceDecoder):
             lay = r.sub.lay
             kw = dict(page_size=self._state_opts["page_size"], device=self.device, page_table=self.slots.page_table, dtype=self.dtype, n_pages=self.slots.n_pages)
             if lay.kind == "latent_attention":
-                self.caches[r.index] = ops.latent_cache(B, r.sub.lat, c.max_len, **kw)
+                self.caches[r.index] = r.sub.lat.new_cache(self)
             else:
                 self.caches[r.index] = ops.PagedKVCache(B, lay.kv_heads, lay.dim, c.max_len, v_dim=lay.vdim, **kw)
         self.attn_ws = self._attn_workspace([(s.lay.heads, s.lay.vdim, s.lay.window, 0) for s in self.subs if s.lay.kind == "attention"])
@@ -187,7 +155,7 @@ class PivavikDecoder(SequenceDecoder):
     def _row_buffers(self, rows):
         c, dev, dt = self.cfg, self.device, self.dtype
         f32, act = dict(dtype=torch.float32, device=dev), dict(dtype=dt, device=dev)
-        latents, moes = [s for s in self.subs if s.lay.kind == "latent_attention"], [s for s in self.subs if s.experts]
+        moes = [s for s in self.subs if s.experts]
         r = SimpleNamespace(rows=rows)
         r.x = torch.empty((rows, c.width), **f32)                                              # residual stream
         r.h = torch.empty(rows * self.h_ld, **act)
@@ -201,39 +169,16 @@ class PivavikDecoder(SequenceDecoder):
             self._linear_workspaces(r.beside, rows, [s.ff for s in self.subs if s.ff] + [x for s in moes for x in (s.experts.up, s.experts.back)])
         if moes:
             Experts.buffers(r, rows, [s.experts for s in moes], self.h_ld, dev, r.beside)
-        r.lat_ws = r.ctx = None
-        if latents:
-            r.q, r.cq = torch.empty(rows * max(s.q_ld for s in latents), **act), torch.empty(rows * max(s.uq.ld for s in latents), **act)
-            if rows <= self.batch or self.plain or any(s.up is None for s in latents):
-                r.lat_ws = torch.empty(max(ops.latent_workspace_bytes(rows, s.lat, dt) for s in latents), dtype=torch.uint8, device=dev)
+        LatentAttention.buffers(r, rows, self._latents(), self)
         return r
 
-    def _context(self, r, rows):
-        """Buffers for `rows` rows of context that prompts project up."""
-        if r.ctx is None or r.ctx.rows < rows:
-            r.ctx = None
-            ups = [s for s in self.subs if s.lay.kind == "latent_attention" and s.up]
-            size = lambda n: torch.empty(rows * n, dtype=self.dtype, device=self.device)
-            r.ctx = SimpleNamespace(rows=rows, shared=size(max(s.lat.rot_dim for s in ups)), latent=size(max(s.up.ld for s in ups)), kv=size(max(s.up.n_out for s in ups)))
-            self._linear_workspaces(r.ctx, rows, [s.up for s in ups])
-        return r.ctx
+    def _latents(self):
+        return [s.lat for s in self.subs if s.lay.kind == "latent_attention"]
 
     # ---- the layers -----------------------------------------------------------------------------
     def _latent_attention(self, run, r, view, longest):
-        s, n, cache = run.sub, view.n_tok, self.caches[run.index]
-        lay, w = s.lay, s.lat
-        ops.latent_prep(view, r.a, s.ld, 0, s.kv_col, w, r.cq, s.uq.ld, cache, self.cfg.eps, s.rope, self.error_flag)
-        self._linear(s.uq, r.cq, r.q, n, s.q_ld, r, pdl=1)
-        gate = dict(gate=r.a[s.gate_col:], gate_ld=s.ld)
-        if n == view.n_seq or s.up is None or self.plain:
-            ops.latent_attn(view, r.q, s.q_ld, w, cache, r.b, s.out.ld, lay.scale, s.rope, r.lat_ws, out_cols=s.mix_cols, error_flag=self.error_flag, plain=self.plain, **gate)
-            return
-        ctx = self._context(r, view.n_ctx)
-        ops.latent_context(view, view.ctx_cu, view.n_ctx, w, cache, ctx.shared, ctx.latent, s.up.ld)
-        self._linear(s.up, ctx.latent, ctx.kv, view.n_ctx, s.up.n_out, ctx)
-        rows = SimpleNamespace(k=ctx.kv, v=ctx.kv[w.heads * w.dim:], shared=ctx.shared, ld=s.up.n_out, shared_dim=w.rot_dim, cu=view.ctx_cu, dim=w.dim + w.rot_dim, vdim=w.vdim)
-        ops.window_attn(view, r.q, s.q_ld, cache, r.b, s.out.ld, w.heads, lay.scale, append=False, max_tokens_per_seq=longest, error_flag=self.error_flag, rope=s.rope,
-                        rope_dims=w.rot_dim, out_cols=s.mix_cols, gate_per_head=True, context=rows, **gate)
+        s = run.sub
+        s.lat(self, r, view, longest, r.a, s.ld, self.caches[run.index], r.b, s.out.ld, s.mix_cols, self._latents())
 
     def _attention(self, run, r, view, longest):
         s, lay = run.sub, run.sub.lay

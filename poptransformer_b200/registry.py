@@ -51,6 +51,11 @@ def _pivavik(c, sd, batch, max_len, dtype, **kw):
     return PivavikDecoder(PivavikConfig(c, max_len), sd, batch, dtype=dtype, **kw)
 
 
+def _puputar(c, sd, batch, max_len, dtype, **kw):
+    from .puputar import PuputarConfig, PuputarDecoder
+    return PuputarDecoder(PuputarConfig(c, max_len), sd, batch, dtype=dtype, **kw)
+
+
 # name -> (builder, dtypes the decoder runs in; the first is the default)
 ARCHITECTURES = {
     "LlamaForCausalLM": (_llama, ("float16",)),
@@ -61,6 +66,7 @@ ARCHITECTURES = {
     "Sabisun": (_sabisun, ("bfloat16", "float32")),
     "Padetar": (_padetar, ("bfloat16", "float32")),
     "Pivavik": (_pivavik, ("bfloat16", "float32")),
+    "Puputar": (_puputar, ("bfloat16", "float32")),
 }
 
 

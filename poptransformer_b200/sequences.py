@@ -46,6 +46,28 @@ class Weights:
         return ops.DenseLinear(torch.cat(ws, 0) if len(ws) > 1 else ws[0], self.dtype, **kw)
 
 
+class JointRows:
+    """Matrices that read the same activations, gathered row by row into one linear."""
+
+    def __init__(self, width, dtype, device):
+        self.width, self.dtype, self.device, self.parts, self.biases, self.n = width, dtype, device, [], [], 0
+
+    def add(self, rows, bias=None):
+        """bias: fp32 [rows] (default zeros)."""
+        self.parts.append(rows)
+        self.biases.append(torch.zeros(len(rows), dtype=torch.float32, device=self.device) if bias is None else bias)
+        self.n += len(rows)
+
+    def column(self, multiple=8):
+        """First column of what is added next: zero rows come before it up to a multiple (8: a 16-byte boundary)."""
+        if self.n % multiple:
+            self.add(torch.zeros((-self.n % multiple, self.width), dtype=self.dtype, device=self.device))
+        return self.n
+
+    def linear(self, biased=False, **kw):
+        return ops.DenseLinear(torch.cat(self.parts, 0), self.dtype, bias=torch.cat(self.biases) if biased else None, **kw)
+
+
 class SequenceDecoder(DecodeLoop):
     _side_stream = None
     PROMPT_TOKENS = 8192     # most packed prompt tokens of one pass (longer prompts go in portions)

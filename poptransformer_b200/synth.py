@@ -193,6 +193,55 @@ def pivavik_state_dict(config, seed=0, device="cpu"):
     return sd
 
 
+def puputar_state_dict(config, seed=0, device="cpu"):
+    """Random bf16 weights of a Puputar (config: its parsed config.json)."""
+    gen = torch.Generator(device=device)
+    gen.manual_seed(seed)
+    W, V, sd = config["width"], config["vocab"], {}
+
+    def put(key, shape, std=1.0, mean=0.0):
+        sd[key] = torch.empty(shape, dtype=torch.bfloat16, device=device).normal_(mean, std, generator=gen)
+
+    def lin(key, o, i, bias=False):
+        put(key, (o, i), i ** -0.5)
+        if bias:
+            put(key + ".b", (o,), 0.1)
+
+    for key in ("embed", "head"):
+        lin(key, V, W)
+    for key in ("embed.norm", "final.norm"):
+        put(key, (W,), 0.02, 1.0)
+    for i, lay in enumerate(config["layers"]):
+        p, m, mlp = f"l{i}.", lay["mixer"], lay.get("mlp")
+        M, Q, H = p + "mix.", p + "mlp.", m["heads"]
+        put(p + "norm1", (W,), 0.02, 1.0)
+        put(p + "shift", (W,), 0.2, 0.5)
+        lin(M + "dq", m["q_rank"], W)
+        put(M + "dq.norm", (m["q_rank"],), 0.02, 1.0)
+        lin(M + "uq", H * (m["dim"] + m["rot_dim"]), m["q_rank"])
+        if m.get("kv_from") is None:
+            lin(M + "dkv", m["kv_rank"] + m["rot_dim"], W)
+            put(M + "dkv.norm", (m["kv_rank"],), 0.02, 1.0)
+        lin(M + "uk", H * m["dim"], m["kv_rank"])
+        lin(M + "uv", H * m["vdim"], m["kv_rank"])
+        lin(M + "g", H if lay["type"] == "latent_attention" else H * m["vdim"], W)
+        lin(M + "o", W, H * m["vdim"])
+        if mlp:
+            put(p + "norm2", (W,), 0.02, 1.0)
+        if mlp and mlp["kind"] == "dense":
+            lin(Q + "up", mlp["ff"], W, True)
+            lin(Q + "down", W, mlp["ff"], True)
+            put(Q + "act", (2,), 0.5)
+        elif mlp:
+            r = mlp["router"]
+            lin(Q + "router", r["experts"] + r.get("identity", 0), W)
+            put(Q + "correction", (r["experts"] + r.get("identity", 0),), 0.02)
+            for e in range(r["experts"]):
+                lin(Q + f"e{e}.up", mlp["expert"]["ff"], W)
+                lin(Q + f"e{e}.down", W, mlp["expert"]["ff"])
+    return sd
+
+
 def gpt2_state_dict(n_layer, d_model, n_head, vocab, n_positions, seed=0, device="cpu"):
     """GPT-2 architecture with the reference's key names after its checkpoint pre-processing (gpt2/model.py:154-166): linear
     weights [out, in], the query third of c_attn (weight and bias) multiplied by 1/sqrt(head_size).  fp16, N(0, 0.02);
