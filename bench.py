@@ -636,6 +636,16 @@ def latent_config(width, n_layer, loop, heads, kv_heads, dim, rot, kv_rank, q_ra
             "layers": [dict(win if i % 2 else lat, mlp=moe if i else {"kind": "dense", "ff": dense_ff}) for i in range(n_layer)]}
 
 
+def shifted_config(width, n_layer, norm_groups, heads, dim, rot, kv_rank, q_rank, experts, identity, groups, keep, top, ff, dense_ff, vocab):
+    """A Puputar of real-model layer sizes: both kinds of latent attention in turn, every fourth layer over the latents of the one two before
+    it, the first layer with a dense feed-forward."""
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "kv_rank": kv_rank, "q_rank": q_rank, "rot": {"base": 1e4, "dims": rot}, "scale": (dim + rot) ** -0.5}
+    moe = {"kind": "moe", "router": {"experts": experts, "identity": identity, "groups": {"count": groups, "keep": keep}, "top": top}, "expert": {"ff": ff}}
+    return {"architecture": "Puputar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6, "groups": norm_groups},
+            "layers": [{"type": "latent_attention_2" if i % 2 else "latent_attention", "mixer": dict(mixer, kv_from=i - 2) if i % 4 == 3 else mixer,
+                        "mlp": moe if i else {"kind": "dense", "ff": dense_ff}} for i in range(n_layer)]}
+
+
 EXPERTS = {   # name: configuration, then the Sabisun of equal width, depth and vocabulary whose feed-forward has as many weights as a token uses here
     "padetar-2k": (dict(width=2048, n_layer=16, heads=16, kv_heads=4, dim=128, mem_heads=16, mem_dim=128, mem_vdim=128, experts=32, top=4, ff=1024, shared_ff=2048,
                         side=128, vocab=32000),
@@ -651,6 +661,14 @@ LATENT = {    # name: configuration, then the Padetar of equal width, vocabulary
                         dense_ff=6144, vocab=32000), EXPERTS["padetar-2k"][0]),
     "pivavik-4k": (dict(width=4096, n_layer=6, loop=(2, 4, 2), heads=32, kv_heads=8, dim=128, rot=64, kv_rank=512, q_rank=1536, window=1024, softcap=50.0, experts=32, top=4, ff=1536,
                         dense_ff=12288, vocab=32000), EXPERTS["padetar-4k"][0]),
+}
+
+SHIFTED = {   # name: configuration, then the Pivavik of equal width, vocabulary, heads and latents with as many
+              # layers as run there; its experts have three matrices and these two, so 3 / 2 the features
+    "puputar-2k": (dict(width=2048, n_layer=16, norm_groups=8, heads=16, dim=128, rot=64, kv_rank=512, q_rank=768, experts=30, identity=2, groups=4, keep=2, top=4, ff=1536, dense_ff=9216,
+                        vocab=32000), LATENT["pivavik-2k"][0]),
+    "puputar-4k": (dict(width=4096, n_layer=8, norm_groups=16, heads=32, dim=128, rot=64, kv_rank=512, q_rank=1536, experts=30, identity=2, groups=4, keep=2, top=4, ff=2304, dense_ff=18432,
+                        vocab=32000), LATENT["pivavik-4k"][0]),
 }
 
 
@@ -793,16 +811,22 @@ def pivavik_state_bytes(dims, ctx):
     return sum(2 * 2 * dims["kv_heads"] * dims["dim"] * min(ctx, dims["window"]) if i % 2 else 2 * (dims["rot"] + dims["kv_rank"]) * ctx for i in runs)
 
 
+def puputar_state_bytes(dims, ctx):
+    """Cached latents of one row and step (a layer without latents of its own reads another's again) and the shift's state, read and written."""
+    return dims["n_layer"] * (2 * (dims["rot"] + dims["kv_rank"]) * ctx + 2 * 4 * dims["width"])
+
+
 def run_beside(args):
     """Decode and prompt throughput of an architecture beside its closest one of equal size.  One JSON line, marked `secondary`."""
     import torch
     from poptransformer_b200 import registry, synth
     if not torch.cuda.is_available():
         raise SystemExit("bench.py needs a CUDA device (there is no CPU fallback)")
-    mine, other, table, what = ("pivavik", "padetar", LATENT, "a decoder with latent attention, experts and looped layers") if args.workload in LATENT else \
+    mine, other, table, what = ("puputar", "pivavik", SHIFTED, "a decoder with latent attention, a token shift and experts in groups") if args.workload in SHIFTED else \
+        ("pivavik", "padetar", LATENT, "a decoder with latent attention, experts and looped layers") if args.workload in LATENT else \
         ("padetar", "sabisun", EXPERTS, "a decoder with experts and a matrix memory")
     make = {"pivavik": (latent_config, synth.pivavik_state_dict, pivavik_state_bytes), "padetar": (expert_config, synth.padetar_state_dict, padetar_state_bytes),
-            "sabisun": (hybrid_config, synth.sabisun_state_dict, None)}
+            "sabisun": (hybrid_config, synth.sabisun_state_dict, None), "puputar": (shifted_config, synth.puputar_state_dict, puputar_state_bytes)}
     dims, odims = table[args.workload]
     dev = torch.device("cuda", 0)
     ctx, prompt, K = 2048, 2048, max(8, min(args.steps, 64))
@@ -823,7 +847,7 @@ def run_beside(args):
                 need = dec.weight_bytes() + batch * sabisun_state_bytes(cfg)
             else:
                 # every linear once, and the experts that `batch` independent choices are expected to hit
-                hit = d["experts"] * (1.0 - (1.0 - d["top"] / d["experts"]) ** batch)
+                hit = d["experts"] * (1.0 - (1.0 - d["top"] / (d["experts"] + d.get("identity", 0))) ** batch)
                 need = dec.fixed_bytes() + sum(hit * (e.up.nbytes + e.back.nbytes) for e in dec.expert_groups()) + batch * state_bytes(d, ctx)
             rows.append({"batch": batch, "decode_ms": ms, "decode_tokens_per_s": batch / ms * 1e3, "bytes_per_step": int(need), "decode_frac_of_measured": need / ms / 1e6 / peak})
             del dec
@@ -833,9 +857,11 @@ def run_beside(args):
         if name == "sabisun":
             flops = 2 * prompt * sum(size(s.proj) + size(s.out) for s in dec.subs)
         else:
-            flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(e.top * (size(e.up) + size(e.back)) for e in dec.expert_groups()))
+            flops = 2 * prompt * (sum(size(x) for x in dec._linears()[1:]) + sum(e.top * e.experts / e.logits * (size(e.up) + size(e.back)) for e in dec.expert_groups()))
             if name == "pivavik":
                 flops += 2 * prompt * sum(size(r.sub.lat.up) for r in dec.runs if r.sub.lay.kind == "latent_attention")
+            if name == "puputar":
+                flops += 2 * prompt * sum(size(s.lat.up) for s in dec.subs)
         for n_seq in (1, 4):
             best = time_prompts(dec, cfg["vocab"], n_seq, prompt)
             pre.append({"sequences": n_seq, "prompt": prompt, "ms": best, "tokens_per_s": n_seq * prompt / best * 1e3, "linear_tflops": n_seq * flops / best / 1e9})
@@ -868,7 +894,7 @@ def main():
                     "stays small; the line is then marked profiling_only and is not a benchmark result")
     ap.add_argument("--pdl", type=int, default=-1, help="secondary workloads: programmatic dependent launch, bit 0 = linear kernels, bit 1 = "
                     "attention kernel (-1: the decoder's default)")
-    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY) + list(HYBRID) + list(EXPERTS) + list(LATENT),
+    ap.add_argument("--workload", default="llama2-7b-int4", choices=["llama2-7b-int4"] + list(SECONDARY) + list(HYBRID) + list(EXPERTS) + list(LATENT) + list(SHIFTED),
                     help="llama2-7b-int4 is the benchmark; the others time a parity configuration, or an architecture of this framework beside the "
                     "closest one of equal size, on one GPU (line marked `secondary`)")
     args = ap.parse_args()
@@ -878,7 +904,7 @@ def main():
         run_secondary(args)
     elif args.workload in HYBRID:
         run_hybrid(args)
-    elif args.workload in EXPERTS or args.workload in LATENT:
+    elif args.workload in EXPERTS or args.workload in LATENT or args.workload in SHIFTED:
         run_beside(args)
     else:
         run_b200(args)

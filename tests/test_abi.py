@@ -34,7 +34,8 @@ def test_library_exports_every_declared_symbol():
 
 
 @pytest.mark.parametrize("arch,own,other", [("Sabisun", ("pt_hyper", "pt_ssm"), "pt_mlstm"), ("Padetar", ("pt_post_norm", "pt_moe_route", "pt_mlstm"), "pt_ssm"),
-                                            ("Pivavik", ("pt_post_norm", "pt_moe_route", "pt_latent_attn"), "pt_mlstm")])
+                                            ("Pivavik", ("pt_post_norm", "pt_moe_route", "pt_latent_attn"), "pt_mlstm"),
+                                            ("Puputar", ("pt_shift_norm", "pt_moe_route", "pt_latent_attn"), "pt_post_norm")])
 def test_parts_link_on_their_own(tmp_path, monkeypatch, arch, own, other):
     """A library with one architecture's sources resolves all of its symbols and has the entry points that the decoder calls."""
     from poptransformer_b200 import build
