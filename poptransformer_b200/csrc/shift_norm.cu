@@ -5,14 +5,18 @@
 // feed-forward's input back.  The kernel also starts a token (x = n(embedding row) w) and ends the model (h2 only).
 //
 // A block takes a run of rows.  For the row above the first one it computes the sum again from the same inputs (which is why x_out is
-// another buffer than x_in), so no block waits for another.  Rows lie in shared memory once; a warp sums the squares of a part of a
-// group at a time.  All of it is fp32; only h1 and h2 are rounded.
+// another buffer than x_in), so no block waits for another.  All of it is fp32; only h1 and h2 are rounded.
+//   rows_kernel        four columns per thread: a row lives in registers while the next one's loads are on their way, the a of the row
+//                      above stays where it is, and weights are read once per run.  Groups in units of 128 columns (a warp's share)
+//   shift_norm_kernel  any width and groups: the run's rows in shared memory, a warp sums the squares of a part of a group at a time
+#include <type_traits>
+
 #include "elem.cuh"
 
 namespace pt {
 namespace shift {
 
-constexpr int kMaxTop = 64, kMaxRun = 4, kRows = kMaxRun + 1;
+constexpr int kMaxTop = 64, kMaxRun = 4, kRows = kMaxRun + 1, kMaxFastRun = 16;
 
 struct Params {
   int rows, width, groups, part, run, segs, h1_ld, h2_ld, table_ld, vocab, ids_ld, y_ld, pair_ld, top, self_ld;   // part: columns of a group; segs: warps' shares of one
@@ -183,6 +187,164 @@ template <typename T, typename E, int VEC, bool START> __global__ void __launch_
   }
 }
 
+__device__ __forceinline__ void fetch4(const float *p, float4 &v) { v = *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ void fetch4(const __nv_bfloat16 *p, uint2 &v) { v = *reinterpret_cast<const uint2 *>(p); }
+__device__ __forceinline__ void add4(float (&a)[4], float w, const float4 &v) {
+  a[0] = fmaf(w, v.x, a[0]); a[1] = fmaf(w, v.y, a[1]); a[2] = fmaf(w, v.z, a[2]); a[3] = fmaf(w, v.w, a[3]);
+}
+__device__ __forceinline__ void add4(float (&a)[4], float w, const uint2 &v) {
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.y));
+  a[0] = fmaf(w, lo.x, a[0]); a[1] = fmaf(w, lo.y, a[1]); a[2] = fmaf(w, hi.x, a[2]); a[3] = fmaf(w, hi.y, a[3]);
+}
+template <typename T> struct Raw4 { typedef float4 type; };
+template <> struct Raw4<__nv_bfloat16> { typedef uint2 type; };
+
+constexpr int CHUNK = 128;                       // columns of a warp
+template <typename T, bool START> __global__ void __launch_bounds__(1024) rows_kernel(const Params p) {
+  __shared__ __align__(16) float pw[(kMaxFastRun + 1) * kMaxTop];      // every row's pairs, in fours (of the last four the rest repeats a row with weight 0)
+  __shared__ __align__(16) int pr[(kMaxFastRun + 1) * kMaxTop];
+  __shared__ float red[2][32];
+  __shared__ int before[kMaxFastRun + 1], from[kMaxFastRun + 1], to[kMaxFastRun + 1];
+  launch_dependents();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, c = tid * 4, r0 = blockIdx.x * p.run, r1 = min(p.rows, r0 + p.run);
+  const bool mix = p.h1 != nullptr;
+  const int lead = mix && p.run > 1 && r0 > p.cu[p.tok_seq[r0]] ? 1 : 0, base = r0 - lead, n = r1 - base;      // (a run of one row: every sequence brings one token)
+  auto source = [&](int i) { return p.row_index ? p.row_index[base + i] : base + i; };
+  // ---- loads of one row, and their sum once they are there
+  typedef typename Raw4<T>::type Raw;
+  float4 xv, yv;
+  Raw ev[4], tv;                                 // four experts' rows, the embedding's row
+  const int quads = (p.top + 3) / 4;
+  auto request = [&](int i) {
+    const int src = source(i);
+    if (START) {
+      const int r = base + i, id = min(max(p.ids[(size_t)r * p.ids_ld + (p.step ? *p.step : 0)], 0), p.vocab - 1);
+      fetch4(reinterpret_cast<const T *>(p.table) + (size_t)id * p.table_ld + c, tv);
+      return;
+    }
+    fetch4(p.x_in + (size_t)src * p.width + c, xv);
+    if (p.y) fetch4(p.y + (size_t)src * p.y_ld + c, yv);
+  };
+  auto request_pairs = [&](int i, int quad) {    // (after the block's pr are in place)
+    const int4 rows = *reinterpret_cast<const int4 *>(pr + (i * quads + quad) * 4);
+    const T *self = reinterpret_cast<const T *>(p.self) + (size_t)source(i) * p.self_ld + c, *pair = reinterpret_cast<const T *>(p.pair_y) + c;
+    fetch4(rows.x < 0 ? self : pair + (size_t)rows.x * p.pair_ld, ev[0]);
+    fetch4(rows.y < 0 ? self : pair + (size_t)rows.y * p.pair_ld, ev[1]);
+    fetch4(rows.z < 0 ? self : pair + (size_t)rows.z * p.pair_ld, ev[2]);
+    fetch4(rows.w < 0 ? self : pair + (size_t)rows.w * p.pair_ld, ev[3]);
+  };
+  auto add_pairs = [&](int i, int quad, float (&v)[4]) {
+    const float4 w = *reinterpret_cast<const float4 *>(pw + (i * quads + quad) * 4);
+    add4(v, w.x, ev[0]);
+    add4(v, w.y, ev[1]);
+    add4(v, w.z, ev[2]);
+    add4(v, w.w, ev[3]);
+  };
+  auto sum = [&](int i, float (&v)[4]) {
+    v[0] = v[1] = v[2] = v[3] = 0.f;
+    if (START) {
+      add4(v, 1.f, tv);
+      return;
+    }
+    if (p.y) {
+      add4(v, 1.f, yv);
+      if (quads) add_pairs(i, 0, v);
+      for (int q = 1; q < quads; ++q) {
+        request_pairs(i, q);
+        add_pairs(i, q, v);
+      }
+    }
+    v[0] += xv.x; v[1] += xv.y; v[2] += xv.z; v[3] += xv.w;
+  };
+  request(0);
+  float above[4] = {0.f, 0.f, 0.f, 0.f}, w1[4], w2[4], share[4], we[4];
+  int first_to = -1;
+  if (mix && p.run == 1) {                       // sequence r0: its state is on its way at once
+    const int at = START && p.step ? *p.step : p.start[r0], slot = p.slot[r0];
+    if (at > 0) load_vec<4>(p.state_in + (size_t)slot * p.width + c, above);
+    first_to = p.by_seq ? r0 : slot;
+  }
+  if (mix) {
+    load_vec<4>(p.w1 + c, w1);
+    load_vec<4>(p.shift + c, share);
+  }
+  if (p.h2) load_vec<4>(p.w2 + c, w2);
+  if (START) load_vec<4>(p.embed_w + c, we);
+  for (int i = tid; i < n * quads * 4; i += blockDim.x) {
+    const int row = i / (quads * 4), j = i % (quads * 4);
+    const size_t k = (size_t)source(row) * p.top + min(j, p.top - 1);
+    const int at = p.pair_row ? p.pair_row[k] : (int)k;
+    const bool none = j >= p.top || (at < 0 && !p.self);
+    pw[i] = none ? 0.f : p.pair_w ? p.pair_w[k] : 1.f;
+    pr[i] = at < 0 && !p.self ? 0 : at;
+  }
+  if (mix && p.run > 1 && tid < n) {
+    const int r = base + tid, s = p.tok_seq[r], at = START && p.step ? *p.step : p.start[s];
+    before[tid] = r > p.cu[s] ? ABOVE : at > 0 ? STATE : NOTHING;
+    from[tid] = p.slot[s];
+    to[tid] = r >= r0 && r + 1 == p.cu[s + 1] ? (p.by_seq ? s : p.slot[s]) : -1;
+  }
+  const int per = p.part / CHUNK, g0 = c / p.part * per;         // the warps of this column's group
+  int turn = 0;
+  auto inv_rms = [&](const float (&v)[4]) {
+    const float ss = warp_sum(fmaf(v[0], v[0], fmaf(v[1], v[1], fmaf(v[2], v[2], v[3] * v[3]))));
+    if (lane == 0) red[turn][warp] = ss;
+    __syncthreads();
+    float all = 0.f;
+    for (int i = 0; i < per; ++i) all += red[turn][g0 + i];
+    turn ^= 1;                                   // (the next sums land in the other half: one barrier per row)
+    return 1.0f / sqrtf(all / (float)p.part + p.eps);
+  };
+  if (quads || p.run > 1) __syncthreads();
+  if (!START && quads) request_pairs(0, 0);
+  for (int i = 0; i < n; ++i) {
+    const int r = base + i;
+    const bool mine = r >= r0;
+    float v[4], o[4];
+    sum(i, v);
+    if (i + 1 < n) {
+      request(i + 1);
+      if (!START && quads) request_pairs(i + 1, 0);
+    }
+    const int kind = mix && p.run > 1 ? before[i] : ABOVE;
+    if (kind == STATE) load_vec<4>(p.state_in + (size_t)from[i] * p.width + c, above);
+    if (START) {
+      if (tid == 0 && mine && p.pos_out) p.pos_out[r] = p.step ? *p.step : 0;
+      const float f = inv_rms(v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] *= f * we[j];
+    }
+    if (p.x_out && mine) store_vec<4>(p.x_out + (size_t)r * p.width + c, v);
+    if (!mix && !p.h2) continue;
+    const float f = inv_rms(v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] *= f;
+    if (p.h2 && mine) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[j] = v[j] * w2[j];
+      store_vec<4>(reinterpret_cast<T *>(p.h2) + (size_t)r * p.h2_ld + c, o);
+    }
+    if (!mix) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      v[j] *= w1[j];
+      o[j] = fmaf((kind == NOTHING ? 0.f : above[j]) - v[j], share[j], v[j]);
+      above[j] = v[j];
+    }
+    if (mine) {
+      store_vec<4>(reinterpret_cast<T *>(p.h1) + (size_t)r * p.h1_ld + c, o);
+      const int dst = p.run > 1 ? to[i] : first_to;
+      if (dst >= 0) store_vec<4>(p.state_out + (size_t)dst * p.width + c, v);
+    }
+  }
+  for (int r = r0; r < r1; ++r) {                // k padding of the next products
+    if (mix)
+      for (int k = p.width + tid; k < p.h1_ld; k += blockDim.x) reinterpret_cast<T *>(p.h1)[(size_t)r * p.h1_ld + k] = from_f<T>(0.f);
+    if (p.h2)
+      for (int k = p.width + tid; k < p.h2_ld; k += blockDim.x) reinterpret_cast<T *>(p.h2)[(size_t)r * p.h2_ld + k] = from_f<T>(0.f);
+  }
+}
+
 constexpr size_t kSmemLimit = 200 * 1024;
 static size_t smem_bytes(const Params &p, int run) {
   const size_t rows = run + (p.h1 ? 1 : 0);
@@ -190,6 +352,13 @@ static size_t smem_bytes(const Params &p, int run) {
 }
 
 template <typename T, typename E, int VEC, bool START> static int launch(Params p, bool single, cudaStream_t st) {
+  if (VEC == 4 && p.part % CHUNK == 0 && p.width <= 4096 && (!p.top || std::is_same<T, E>::value)) {
+    const int threads = p.width / 4, resident = std::max(1, 1024 / threads) * sm_count();        // blocks on the GPU at a time
+    p.run = single ? 1 : std::min(kMaxFastRun, std::max(2, ceil_div(p.rows, resident)));
+    rows_kernel<T, START><<<ceil_div(p.rows, p.run), threads, 0, st>>>(p);
+    PT_LAUNCH_CHECK("pt_shift_norm");
+    return PT_OK;
+  }
   // few rows: as many threads as a row has work for; many: several rows of a sequence per block, so that few are computed twice
   const int want = ceil_div(ceil_div(p.width, VEC), 32) * 32, cap = p.rows <= 2 * sm_count() ? 1024 : 256, threads = std::max(64, std::min(want, cap));
   p.run = single ? 1 : p.rows >= 8 * sm_count() ? kMaxRun : p.rows >= 4 * sm_count() ? 2 : 1;

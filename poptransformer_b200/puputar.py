@@ -92,6 +92,7 @@ class PuputarDecoder(SequenceDecoder):
             rows = JointRows(W, dt, dev)
             sub.lat = LatentAttention(w, M, lay, W, rows, ropes, c.max_len, gate_per_value=GATE_PER_VALUE[lay.kind], interleaved=True, own=lay.kv_from is None)
             sub.cache = i if lay.kv_from is None else lay.kv_from
+            rows.column(32)                      # (the GEMM's fast epilogue takes whole groups of 32 outputs)
             sub.proj = rows.linear()
             sub.ld = ops.pad_to(sub.proj.n_out, 8)
             if lay.ff or lay.moe:

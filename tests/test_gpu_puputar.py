@@ -54,7 +54,7 @@ class ShiftSite:
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("W,G", [(33, 3), (96, 4), (96, 1), (50, 50), (2048, 8), (260, 13)])
+@pytest.mark.parametrize("W,G", [(33, 3), (96, 4), (96, 1), (50, 50), (2048, 8), (260, 13), (128, 1), (384, 3), (768, 3), (4096, 1), (4224, 33)])
 def test_residual_step_with_token_shift(cuda, dtype, W, G):
     """Three sequences in portions (down to two tokens) and single tokens: dense outputs, experts' outputs with weights, and experts that
     give the feed-forward's input back."""
@@ -93,11 +93,12 @@ def test_residual_step_with_token_shift(cuda, dtype, W, G):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("W,G", [(64, 2), (256, 2)])
 @pytest.mark.parametrize("rows", [3, 700, 1300])
-def test_residual_step_over_many_rows(cuda, dtype, rows):
-    """Runs of one, two and four rows per block, with sequences that begin and end anywhere in them, and an embedding start."""
+def test_residual_step_over_many_rows(cuda, dtype, rows, W, G):
+    """Runs of one row per block and more, with sequences that begin and end anywhere in them, and an embedding start."""
     r = np.random.default_rng(2)
-    W, G, vocab = 64, 2, 31
+    vocab = 31
     lens = []
     while sum(lens) < rows:
         lens.append(int(min(r.integers(1, 12), rows - sum(lens))))
@@ -123,11 +124,12 @@ def test_residual_step_over_many_rows(cuda, dtype, rows):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-def test_residual_step_of_the_decode_loop_and_the_end(cuda, dtype):
+@pytest.mark.parametrize("W,G", [(96, 4), (512, 2)])
+def test_residual_step_of_the_decode_loop_and_the_end(cuda, dtype, W, G):
     """One token per row from an id container at a position that is read on the device; and the norm in front of the output layer."""
     from poptransformer_b200 import ops
     r = np.random.default_rng(3)
-    W, G, B, vocab = 96, 4, 5, 17
+    B, vocab = 5, 17
     site, tol = ShiftSite(cuda, dtype, W, G, B), 1e-6 if dtype == F32 else 4e-3
     table, ids = bf16(r.standard_normal((vocab, W))), r.integers(0, vocab, (B, 4))
     pos, step, rows = torch.full((B,), 77, dtype=torch.int32, device=cuda), i32([0], cuda), i32(np.arange(B + 1), cuda)
